@@ -47,6 +47,8 @@ class Config:
     #   "original":   number of tokens the request has really seen
     position_mode: str = "compressed"
     prefix_caching: bool = True
+    # slots of per-request recurrent state (models with recurrent layers only; 0: one per running request)
+    num_state_slots: int = 0
     seed: int = 0
     extra: dict = field(default_factory=dict)
 
@@ -93,6 +95,17 @@ class ModelConfig:
             if "rope_scaling" not in kw:
                 kind = rp.get("rope_type", rp.get("type", "default"))
                 self.rope_scaling = None if kind in (None, "default") else dict(rp)
+
+        # a hybrid layer list ("layers": one dict per layer) names its sizes `vocab` and `width`; the engine reads
+        # the HuggingFace field names
+        if isinstance(kw.get("layers"), list):
+            for src, dst in (("vocab", "vocab_size"), ("width", "hidden_size")):
+                if src in kw and dst not in kw:
+                    setattr(self, dst, kw[src])
+            if "num_hidden_layers" not in kw:
+                self.num_hidden_layers = len(kw["layers"])
+            if "architectures" not in kw and isinstance(kw.get("architecture"), str):
+                self.architectures = [kw["architecture"]]
 
     def get(self, name: str, default: Any = None) -> Any:
         return getattr(self, name, default)

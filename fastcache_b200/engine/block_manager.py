@@ -39,7 +39,7 @@ class Block:
 
 
 class BlockManager:
-    def __init__(self, num_blocks: int, block_size: int, prefix_caching: bool = True):
+    def __init__(self, num_blocks: int, block_size: int, prefix_caching: bool = True, num_state_slots: int = 0):
         if num_blocks <= 0:
             raise ValueError("the KV pool needs at least one block")
         self.block_size = block_size
@@ -48,6 +48,12 @@ class BlockManager:
         self.hash_to_block_id: Dict[int, int] = {}
         self.free_block_ids: Deque[int] = deque(range(num_blocks))
         self.used_block_ids: Set[int] = set()
+        # one slot of recurrent state per request that holds blocks (0: the model keeps none).  A state belongs to
+        # one request and one position, so it cannot be found through the prefix cache
+        self.num_state_slots = num_state_slots
+        self.free_state_slots: Deque[int] = deque(range(num_state_slots))
+        if num_state_slots and prefix_caching:
+            raise ValueError("prefix caching cannot be combined with recurrent state slots")
 
     # ------------------------------------------------------------------ hashing
     @staticmethod
@@ -108,6 +114,8 @@ class BlockManager:
 
     # -------------------------------------------------------------- allocation
     def can_allocate(self, seq: Sequence) -> bool:
+        if self.num_state_slots and not self.free_state_slots:
+            return False
         return len(self.free_block_ids) >= seq.num_blocks
 
     def allocate(self, seq: Sequence) -> None:
@@ -118,6 +126,8 @@ class BlockManager:
         """
         if seq.block_table:
             raise RuntimeError("sequence already holds blocks")
+        if self.num_state_slots:
+            seq.state_slot = self.free_state_slots.popleft()
         use_cache = self.prefix_caching and not seq.has_image
         h = -1
         cache_miss = not use_cache
@@ -150,6 +160,9 @@ class BlockManager:
             self._release(block_id)
         seq.num_cached_tokens = 0
         seq.block_table.clear()
+        if seq.state_slot >= 0:
+            self.free_state_slots.append(seq.state_slot)
+            seq.state_slot = -1
 
     # ------------------------------------------------------------------- decode
     def can_append(self, seq: Sequence) -> bool:
@@ -286,6 +299,14 @@ class BlockManager:
                 raise AssertionError("negative reference count")
             if (b.ref_count > 0) != (b.block_id in self.used_block_ids):
                 raise AssertionError(f"block {b.block_id}: refs and used set disagree")
+        slots = list(self.free_state_slots)
+        if len(set(slots)) != len(slots):
+            raise AssertionError("duplicate state slot on the free list")
+        if live is not None and self.num_state_slots:
+            live = list(live)
+            held = [s.state_slot for s in live if s.block_table]
+            if min(held, default=0) < 0 or sorted(held + slots) != list(range(self.num_state_slots)):
+                raise AssertionError("state slots leaked or handed out twice")
         if live is not None:
             refs: Dict[int, int] = {}
             for s in live:

@@ -32,8 +32,9 @@ from ..layers.sampler import Sampler
 from ..models.registry import build_model, detect_model_type
 from ..parallel import tp as tpmod
 from ..utils.context import reset_context, set_context
-from ..utils.loader import init_random_weights, load_model
+from ..utils.loader import checkpoint_shapes, init_random_weights, load_model
 from ..utils.memory import get_gpu_memory
+from . import layer_cache
 from .async_compression import AsyncCompressionManager  # noqa: F401  (the reference exports it from here)
 from .sequence import CompressionState, Sequence  # noqa: F401  (CompressionState: the reference defines it in llava_model_runner.py:43)
 
@@ -104,6 +105,9 @@ class ModelRunner:
         self.model_type = detect_model_type(hf)
         self.is_multimodal = self.model_type in ("llava", "minicpm")
 
+        if self.config.model:
+            # a size that only a tensor's shape gives (see the model) is read from the checkpoint's headers
+            hf.checkpoint_shapes = checkpoint_shapes(self.config.model) if self.model_type == "bagedra" else None
         prev = torch.get_default_dtype()
         torch.set_default_dtype(self.dtype)
         try:
@@ -116,7 +120,9 @@ class ModelRunner:
 
         tc = self.text_config
         self.num_hidden_layers = tc.num_hidden_layers
-        heads = tc.num_attention_heads
+        # a model that describes its own cache keeps no per-head K/V rows: pages and state slots instead of `kv_cache`
+        self.cache_layout = self.model.cache_layout() if hasattr(self.model, "cache_layout") else None
+        heads = getattr(tc, "num_attention_heads", 1) if self.cache_layout is not None else tc.num_attention_heads
         kvh = getattr(tc, "num_key_value_heads", None) or heads
         self.head_dim = getattr(tc, "head_dim", None) or tc.hidden_size // heads
         self.total_kv_heads = kvh
@@ -143,6 +149,9 @@ class ModelRunner:
         self.allocate_kv_cache()
 
         # ------------------------------------------------------ compression
+        if enable_compression and not getattr(self.model, "supports_compression", True):
+            print(f"[fastcache_b200] {self.model_type} keeps no per-head K/V rows; compression disabled")
+            enable_compression = False
         self.enable_compression = enable_compression
         self.async_compression = async_compression
         self.compression_backend = compression_backend
@@ -232,26 +241,48 @@ class ModelRunner:
             self.compressor = None
             self.packed_compressor = None
 
+    def allocate_layer_caches(self) -> None:
+        """Pages and state slots of a model with a cache layout of its own.  The slots come first (their number is
+        the number of requests that can run), the pages share what is left."""
+        cfg, bs = self.config, self.block_size
+        if layer_cache.state_bytes(self.cache_layout):
+            cfg.num_state_slots = cfg.num_state_slots or cfg.max_num_seqs
+            cfg.max_num_seqs = min(cfg.max_num_seqs, cfg.num_state_slots)
+            cfg.prefix_caching = False           # a cached prefix has no recurrent state to continue from
+            layer_cache.allocate_states(self.cache_layout, cfg.num_state_slots, self.device)
+        block_bytes = max(1, bs * layer_cache.row_bytes(self.cache_layout, self.dtype))
+        if cfg.num_kvcache_blocks <= 0:
+            cap = cfg.max_num_seqs * -(-cfg.max_model_len // bs)       # more can never be in use
+            cfg.num_kvcache_blocks = min(cap, self._blocks_that_fit(block_bytes))
+        self.num_blocks = cfg.num_kvcache_blocks
+        layer_cache.allocate_rows(self.cache_layout, self.num_blocks, bs, self.dtype, self.device)
+        self.kv_cache = None
+
+    def _blocks_that_fit(self, block_bytes: int) -> int:
+        cfg, bs = self.config, self.block_size
+        if self.device.type != "cuda":
+            need = cfg.max_num_seqs * -(-cfg.max_model_len // bs)
+            return max(1, min(need, (1 << 30) // block_bytes))
+        total, used, free = get_gpu_memory(self.device.index)
+        budget = int(total * cfg.gpu_memory_utilization) - used
+        need = -(-cfg.max_model_len // bs)
+        if budget < need * block_bytes:
+            raise RuntimeError(
+                f"not enough device memory for the KV pool: {max(budget, 0) / 2**30:.1f} GiB left under "
+                f"gpu_memory_utilization={cfg.gpu_memory_utilization} ({used / 2**30:.1f} of "
+                f"{total / 2**30:.1f} GiB in use), one request of max_model_len={cfg.max_model_len} needs "
+                f"{need * block_bytes / 2**30:.1f} GiB; free other engines in this process "
+                f"(`llm.exit()`) or pass num_kvcache_blocks")
+        return budget // block_bytes
+
     def allocate_kv_cache(self) -> None:
+        if self.cache_layout is not None:
+            return self.allocate_layer_caches()
         cfg = self.config
         L, H, D, bs = self.num_hidden_layers, self.num_key_value_heads, self.head_dim, self.block_size
         block_bytes = 2 * L * bs * H * D * torch.empty((), dtype=self.dtype).element_size()
         if cfg.num_kvcache_blocks <= 0:
-            if self.device.type == "cuda":
-                total, used, free = get_gpu_memory(self.device.index)
-                budget = int(total * cfg.gpu_memory_utilization) - used
-                need = -(-cfg.max_model_len // bs)
-                if budget < need * block_bytes:
-                    raise RuntimeError(
-                        f"not enough device memory for the KV pool: {max(budget, 0) / 2**30:.1f} GiB left under "
-                        f"gpu_memory_utilization={cfg.gpu_memory_utilization} ({used / 2**30:.1f} of "
-                        f"{total / 2**30:.1f} GiB in use), one request of max_model_len={cfg.max_model_len} needs "
-                        f"{need * block_bytes / 2**30:.1f} GiB; free other engines in this process "
-                        f"(`llm.exit()`) or pass num_kvcache_blocks")
-                cfg.num_kvcache_blocks = budget // block_bytes
-            else:
-                need = cfg.max_num_seqs * -(-cfg.max_model_len // bs)
-                cfg.num_kvcache_blocks = max(1, min(need, (1 << 30) // block_bytes))
+            cfg.num_kvcache_blocks = self._blocks_that_fit(block_bytes)
         self.num_blocks = cfg.num_kvcache_blocks
         self.kv_cache = torch.zeros(L, 2, self.num_blocks, H, bs, D, dtype=self.dtype, device=self.device)
         i = 0
@@ -322,8 +353,23 @@ class ModelRunner:
             window = {"indices": self._to_dev(np.concatenate(idx), torch.int64), "q": {},
                       "counts": [len(x) for x in idx]}
         set_context(True, cu, cu, max_q, max_k, slot_mapping, kvl, block_tables, window_q=window,
-                    obs_window=self.obs_window)
+                    obs_window=self.obs_window, **self._layer_metadata(seqs, cu_q, kv_lens))
         return input_ids, positions, image_rows
+
+    def _state_slots(self, seqs: Seq[Sequence]) -> np.ndarray:
+        return np.asarray([s.state_slot for s in seqs], dtype=np.int32)
+
+    def _layer_metadata(self, seqs: Seq[Sequence], cu_q: List[int], kv_lens: List[int]) -> Dict[str, Any]:
+        """Prefill metadata of models with a cache layout of their own (see `Context`)."""
+        if self.cache_layout is None:
+            return {}
+        lens = np.diff(cu_q)
+        ctx = np.concatenate([np.arange(k - n, k, dtype=np.int32) + 1 for n, k in zip(lens, kv_lens)])
+        cu_kv = np.concatenate([[0], np.cumsum(kv_lens)])
+        return {"state_slots": self._to_dev(self._state_slots(seqs), torch.int32),
+                "row_seq": self._to_dev(np.repeat(np.arange(len(seqs), dtype=np.int32), lens), torch.int32),
+                "row_ctx": self._to_dev(ctx, torch.int32),
+                "cu_seqlens_kv": self._to_dev(cu_kv.astype(np.int32), torch.int32), "total_kv": int(cu_kv[-1])}
 
     def prepare_decode(self, seqs: Seq[Sequence]):
         bs = self.block_size
@@ -367,10 +413,14 @@ class ModelRunner:
             embed_head.set_local_logits(prev)
 
     @torch.inference_mode()
-    def run_prefill(self, seqs: Seq[Sequence], local_logits: bool = False) -> torch.Tensor:
+    def run_prefill(self, seqs: Seq[Sequence], local_logits: bool = False,
+                    logits_rows: Optional[Seq[int]] = None) -> torch.Tensor:
+        """Logits of the last row of every request, or of the given rows of the concatenated pieces."""
         input_ids, positions, image_rows = self.prepare_prefill(seqs)
         from ..utils.context import get_context
         ctx = get_context()
+        if logits_rows is not None:
+            ctx.logits_indices = self._to_dev(np.asarray(logits_rows, dtype=np.int64), torch.int64)
         if self.timer is not None:
             self.timer.start(self.main_stream)
         logits = self._forward(input_ids, positions, seqs, image_rows, local_logits=local_logits)
@@ -398,7 +448,9 @@ class ModelRunner:
             set_context(False, slot_mapping=self._to_dev(slots, torch.int32),
                         context_lens=self._to_dev(lens, torch.int32),
                         block_tables=self._to_dev(bt, torch.int32),
-                        attn_workspace=getattr(self, "attn_workspace", None))
+                        attn_workspace=getattr(self, "attn_workspace", None),
+                        **({} if self.cache_layout is None else
+                           {"state_slots": self._to_dev(self._state_slots(seqs), torch.int32)}))
             ids_d, pos_d = self._to_dev(ids, torch.int64), self._to_dev(pos, torch.int64)
             if self.timer is not None:
                 self.timer.start(self.main_stream)
@@ -415,7 +467,10 @@ class ModelRunner:
         h["context_lens"][n:bucket] = 0
         h["block_tables"][:bucket].fill_(0)
         h["block_tables"][:n, : bt.shape[1]] = torch.from_numpy(np.maximum(bt, 0))
-        for k in ("input_ids", "positions", "slot_mapping", "context_lens", "block_tables"):
+        self._stage_state_slots(seqs, bucket)
+        for k in ("input_ids", "positions", "slot_mapping", "context_lens", "block_tables", "state_slots"):
+            if k not in gv:
+                continue
             gv[k][:bucket].copy_(h[k][:bucket], non_blocking=True)
             if self.device.type == "cuda":
                 self.io["h2d_bytes"] += h[k][:bucket].numel() * h[k].element_size()
@@ -426,6 +481,12 @@ class ModelRunner:
         if self.local_logits and not local_logits:          # the graphs hold shards: gather for a caller who asked
             logits = tpmod.tp_all_gather(logits, dim=-1)[:, : self.text_config.vocab_size]
         return logits
+
+    def _stage_state_slots(self, seqs: Seq[Sequence], bucket: int) -> None:
+        if self.cache_layout is not None:
+            h = self._staging["state_slots"]
+            h[: len(seqs)] = torch.from_numpy(self._state_slots(seqs))
+            h[len(seqs):bucket] = -1
 
     def _replay(self, bucket: int) -> None:
         g = self.graphs[bucket]
@@ -440,7 +501,8 @@ class ModelRunner:
         gv = self.graph_vars
         set_context(False, slot_mapping=gv["slot_mapping"][:bucket], context_lens=gv["context_lens"][:bucket],
                     block_tables=gv["block_tables"][:bucket],
-                    attn_workspace=getattr(self, "attn_workspace", None))
+                    attn_workspace=getattr(self, "attn_workspace", None),
+                    **({"state_slots": gv["state_slots"][:bucket]} if "state_slots" in gv else {}))
         gv["logits"][:bucket] = self._forward(gv["input_ids"][:bucket], gv["positions"][:bucket],
                                               local_logits=self.local_logits)
 
@@ -459,6 +521,8 @@ class ModelRunner:
             "block_tables": torch.zeros(max_bs, max_blocks, dtype=torch.int32, device=dev),
             "logits": torch.zeros(max_bs, vocab, dtype=self.dtype, device=dev),
         }
+        if self.cache_layout is not None:
+            self.graph_vars["state_slots"] = torch.full((max_bs,), -1, dtype=torch.int32, device=dev)
         pin = dev.type == "cuda"
         self._staging = {k: torch.zeros(v.shape, dtype=v.dtype, pin_memory=pin)
                          for k, v in self.graph_vars.items() if k != "logits"}
@@ -523,7 +587,8 @@ class ModelRunner:
             h["input_ids"][n:bucket] = 0
             h["block_tables"][:bucket].fill_(0)
             h["block_tables"][:n, : bt.shape[1]] = torch.from_numpy(np.maximum(bt, 0))
-            for key in ("input_ids", "block_tables"):
+            self._stage_state_slots(seqs, bucket)
+            for key in ("input_ids", "block_tables") + (("state_slots",) if "state_slots" in gv else ()):
                 gv[key][:bucket].copy_(h[key][:bucket], non_blocking=True)
                 if self.device.type == "cuda":
                     self.io["h2d_bytes"] += h[key][:bucket].numel() * h[key].element_size()
@@ -761,7 +826,7 @@ class ModelRunner:
 
     def reset_graph_vars(self) -> None:
         for name, t in getattr(self, "graph_vars", {}).items():
-            if name == "slot_mapping":
+            if name in ("slot_mapping", "state_slots"):
                 t.fill_(-1)
             elif name != "logits":
                 t.zero_()
@@ -838,6 +903,8 @@ class ModelRunner:
             for module in model.modules():
                 if hasattr(module, "k_cache") and hasattr(module, "v_cache"):
                     module.k_cache = module.v_cache = None
+        if self.cache_layout is not None:
+            layer_cache.release(self.cache_layout)
         self.kv_cache = None
         self.model = None
         self.packed_compressor = None

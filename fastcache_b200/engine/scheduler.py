@@ -46,7 +46,8 @@ class Scheduler:
         self._piece_last = False         # the previous step ran a piece of a split prompt
         self.one_image_per_prefill = bool(config.extra.get("one_image_per_prefill", False))
         self.block_manager = BlockManager(config.num_kvcache_blocks, config.kvcache_block_size,
-                                          prefix_caching=config.prefix_caching)
+                                          prefix_caching=config.prefix_caching,
+                                          num_state_slots=config.num_state_slots)
         self.waiting: Deque[Sequence] = deque()
         self.running: Deque[Sequence] = deque()
         self.compress_queue: Deque[Sequence] = deque()
@@ -118,6 +119,26 @@ class Scheduler:
         if room < self.max_num_batched_tokens:       # other requests share the step: wait for an emptier one
             return 0
         return take if take > 0 else min(room, cost - 1)
+
+    def schedule_pieces(self, pieces: List[Tuple[Sequence, List[int]]]) -> List[Sequence]:
+        """A batch chosen by the caller: the next given tokens of each request, as one piece of its prompt.  A new
+        request is admitted (blocks, state slot), a known one grows its block table; nothing is sampled."""
+        for seq, tokens in pieces:
+            done = seq.prefill_start
+            if seq.block_table:
+                seq.extend_tokens(tokens)
+                if self.block_manager.blocks_short_for(seq, 0) > self.block_manager.num_free_blocks:
+                    raise RuntimeError(f"no free blocks for request {seq.seq_id}")
+                self.block_manager.reserve_rows(seq, 0)
+            else:
+                if not self.block_manager.can_allocate(seq):
+                    raise RuntimeError(f"no free blocks or state slot for request {seq.seq_id}")
+                self.block_manager.allocate(seq)
+                self.running.append(seq)
+                seq.status = SequenceStatus.RUNNING
+                done = seq.prefill_start
+            seq.num_computed_tokens, seq.prefill_end = done, len(seq)
+        return [seq for seq, _ in pieces]
 
     # ------------------------------------------------------------------ decode
     def _schedule_decode(self) -> List[Sequence]:

@@ -54,6 +54,7 @@ class Sequence:
         self.num_computed_tokens = 0
         self.prefill_end: Optional[int] = None
         self.block_table: List[int] = []
+        self.state_slot = -1          # slot of the recurrent state (models with recurrent layers)
         self.temperature = sp.temperature
         self.max_tokens = sp.max_tokens
         self.ignore_eos = sp.ignore_eos
@@ -176,6 +177,12 @@ class Sequence:
         if self._kv_cache_len is not None:
             self._kv_cache_len += 1
         self._pending_row = True
+
+    def extend_tokens(self, token_ids: List[int]) -> None:
+        """Append given (not sampled) tokens whose rows the next prefill piece computes."""
+        self.token_ids.extend(int(t) for t in token_ids)
+        self.last_token = self.token_ids[-1]
+        self.num_tokens = self.num_prompt_tokens = len(self.token_ids)
 
     @property
     def rows_in_pool(self) -> int:

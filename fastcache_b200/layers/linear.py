@@ -15,7 +15,7 @@ Differences by design:
 """
 from __future__ import annotations
 
-from typing import List, Optional
+from typing import Dict, List, Optional, Sequence
 
 import torch
 from torch import nn
@@ -98,6 +98,44 @@ class MergedColumnParallelLinear(LinearBase):
         if loaded.shape[0] != size:
             loaded = loaded.narrow(0, self.tp_rank * size, size)
         _copy(param.data.narrow(0, off, size), loaded)
+
+
+def pad8(n: int) -> int:
+    return -(-n // 8) * 8
+
+
+class PackedLinear(nn.Module):
+    """Named projections of one input in one weight (one GEMM, not split over ranks).
+
+    `sizes`: output width by name, in order.  A projection named in `tight` follows its predecessor directly, any
+    other starts at a multiple of 8 columns; the input width and the total are padded to multiples of 8 with zero
+    weights, so that every size meets the GEMMs' 16-byte rows.  `offset[name]` is the first output column."""
+
+    def __init__(self, input_size: int, sizes: Dict[str, int], bias: bool = False, tight: Sequence[str] = ()):
+        super().__init__()
+        self.input_size = input_size
+        self.sizes = dict(sizes)
+        self.offset: Dict[str, int] = {}
+        n = 0
+        for name, size in sizes.items():
+            n = n if name in tight else pad8(n)
+            self.offset[name] = n
+            n += size
+        self.output_size = pad8(n)
+        self.weight = nn.Parameter(torch.zeros(self.output_size, pad8(input_size)), requires_grad=False)
+        self.weight.weight_loader = self.weight_loader
+        if bias:
+            self.bias = nn.Parameter(torch.zeros(self.output_size), requires_grad=False)
+            self.bias.weight_loader = self.weight_loader
+        else:
+            self.register_parameter("bias", None)
+
+    def weight_loader(self, param: nn.Parameter, loaded: torch.Tensor, shard_id=None) -> None:
+        dst = param.data.narrow(0, self.offset[shard_id], self.sizes[shard_id])
+        _copy(dst if param.data.dim() == 1 else dst[:, :self.input_size], loaded)
+
+    def forward(self, x: torch.Tensor) -> torch.Tensor:
+        return ops.linear(x, self.weight, self.bias)
 
 
 class QKVParallelLinear(LinearBase):

@@ -1,0 +1,87 @@
+"""Recurrent mixers with a fixed-size state per request: gated linear attention and the gated delta rule.
+
+Both read the state that earlier steps left in the request's slot (`state`, and `conv_state` for the short
+convolutions), advance it by the rows of the batch and leave it there; prefill portions of any length and decode
+steps go through the same call.
+"""
+from __future__ import annotations
+
+from typing import Dict, Optional, Tuple
+
+import torch
+from torch import nn
+
+from .. import ops
+from ..ops.hybrid import DeltaDims, GlaDims
+from ..utils.context import get_context
+from .linear import PackedLinear
+
+
+def fp32_vector(*shape: int) -> nn.Parameter:
+    """A small parameter that is used in 32-bit whatever the model's dtype."""
+    return nn.Parameter(torch.zeros(*shape, dtype=torch.float32), requires_grad=False)
+
+
+class GatedLinearAttention(nn.Module):
+    """S <- diag(alpha) S + k v^T, o = S^T q per head, with a decay alpha per key channel and token from a low-rank
+    projection, alpha = sigmoid(z)^(1 / tau); the head outputs are RMS-normed and gated with silu."""
+
+    def __init__(self, width: int, heads: int, dim: int, vdim: int, rank: int, tau: float, eps: float):
+        super().__init__()
+        self.eps = eps
+        self.in_proj = PackedLinear(width, {"q": heads * dim, "k": heads * dim, "v": heads * vdim,
+                                            "g": heads * vdim, "a1": rank})
+        self.a2 = PackedLinear(rank, {"a2": heads * dim})
+        self.z_bias = fp32_vector(heads * dim)
+        self.norm = fp32_vector(vdim)
+        self.o_proj = PackedLinear(heads * vdim, {"o": width})
+        o = self.in_proj.offset
+        self.dims = GlaDims(heads, dim, vdim, rank, float(tau), o["q"], o["k"], o["v"], o["g"], o["a1"])
+        self.state: Optional[torch.Tensor] = None           # [slots, heads, dim, vdim], bound by the runner
+
+    def state_shapes(self) -> Dict[str, Tuple[int, ...]]:
+        d = self.dims
+        return {"state": (d.heads, d.dim, d.vdim)}
+
+    def forward(self, positions: torch.Tensor, h: torch.Tensor) -> torch.Tensor:
+        return ops.hybrid.gla(h, self.in_proj.weight, self.dims, self.a2.weight, self.z_bias, self.norm, self.eps,
+                              self.state, get_context())
+
+
+class GatedDeltaRule(nn.Module):
+    """S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q per head, with q, k, v from projections followed
+    by a short causal convolution and silu, unit-norm q and k shared by groups of heads, one decay and one step size
+    per head; the head outputs are RMS-normed and gated with silu."""
+
+    def __init__(self, width: int, heads: int, kv_heads: int, dim: int, vdim: int, taps: int, eps: float,
+                 unit_eps: float = 1e-6):
+        super().__init__()
+        if heads % kv_heads:
+            raise ValueError(f"{heads} heads cannot share {kv_heads} q/k heads evenly")
+        self.eps = eps
+        self.taps = taps
+        self.in_proj = PackedLinear(width, {"q": kv_heads * dim, "k": kv_heads * dim, "v": heads * vdim,
+                                            "g": heads * vdim, "b": heads, "a": heads}, tight=("k", "v"))
+        self.channels = 2 * kv_heads * dim + heads * vdim
+        self.conv = fp32_vector(self.channels, taps)
+        self.conv.weight_loader = self._load_conv
+        self.a_log = fp32_vector(heads)
+        self.dt_bias = fp32_vector(heads)
+        self.norm = fp32_vector(vdim)
+        self.o_proj = PackedLinear(heads * vdim, {"o": width})
+        o = self.in_proj.offset
+        self.dims = DeltaDims(heads, kv_heads, dim, vdim, o["g"], o["b"], o["a"], unit_eps)
+        self.state: Optional[torch.Tensor] = None           # [slots, heads, dim, vdim], bound by the runner
+        self.conv_state: Optional[torch.Tensor] = None      # [slots, taps - 1, channels]: the last inputs
+
+    def _load_conv(self, param: nn.Parameter, loaded: torch.Tensor, shard_id=None) -> None:
+        off, size = self.in_proj.offset[shard_id], self.in_proj.sizes[shard_id]
+        param.data[off:off + size].copy_(loaded)
+
+    def state_shapes(self) -> Dict[str, Tuple[int, ...]]:
+        d = self.dims
+        return {"state": (d.heads, d.dim, d.vdim), "conv_state": (self.taps - 1, self.channels)}
+
+    def forward(self, positions: torch.Tensor, h: torch.Tensor) -> torch.Tensor:
+        return ops.hybrid.delta_rule(h, self.in_proj.weight, self.dims, self.conv, self.a_log, self.dt_bias,
+                                     self.norm, self.eps, self.conv_state, self.state, get_context())

@@ -20,6 +20,8 @@ def detect_model_type(hf_config: Any) -> str:
         return "qwen3"
     if "qwen2" in mt or "qwen2" in joined:
         return "qwen2"
+    if "bagedra" in mt or "bagedra" in joined:
+        return "bagedra"
     if "llama" in mt or "llama" in joined or "mistral" in mt:
         return "llama"
     raise ValueError(f"unsupported model type {mt!r} / architectures {archs}")
@@ -50,8 +52,14 @@ def _minicpm(cfg):
     return MiniCPMForConditionalGeneration(cfg)
 
 
+def _bagedra(cfg):
+    from .bagedra import BagedraForCausalLM
+    return BagedraForCausalLM(cfg)
+
+
 MODEL_REGISTRY: Dict[str, Callable] = {
     "llama": _llama, "qwen3": _qwen3, "qwen2": _qwen2, "llava": _llava, "minicpm": _minicpm,
+    "bagedra": _bagedra,
 }
 
 

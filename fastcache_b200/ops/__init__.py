@@ -19,6 +19,8 @@ from .loader import ext, ext_available  # noqa: F401
 
 COUNTERS = {"launches": 0}
 
+from . import hybrid  # noqa: E402,F401
+
 
 def _n(k: int = 1) -> None:
     COUNTERS["launches"] += k

@@ -1,0 +1,146 @@
+"""Ops of hybrid models (recurrent layers, latent attention, sublayer-output norms on a 32-bit residual stream).
+
+Same rule as the other ops of this package: the device of the data decides between the sm_100a kernels and the
+PyTorch statements of `reference_hybrid.py`.  Inputs and outputs are in the model's dtype (bf16, or fp32 for runs
+in 32-bit); the residual stream, the recurrent states and the small per-head vectors are always fp32.
+"""
+from __future__ import annotations
+
+from dataclasses import dataclass
+from typing import Optional
+
+import torch
+
+from . import reference_hybrid as ref
+from .loader import ext
+
+
+def _n(k: int = 1) -> None:
+    from . import COUNTERS
+    COUNTERS["launches"] += k
+
+
+@dataclass(frozen=True)
+class GlaDims:
+    """Gated linear attention: sizes, decay temperature, first columns of the packed projections."""
+    heads: int
+    dim: int
+    vdim: int
+    rank: int
+    tau: float
+    q: int
+    k: int
+    v: int
+    g: int
+    a1: int
+
+
+@dataclass(frozen=True)
+class DeltaDims:
+    """Gated delta rule; q | k | v are the first columns of the packed projections, without gaps."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    g: int
+    b: int
+    a: int
+    unit_eps: float = 1e-6
+
+
+@dataclass(frozen=True)
+class LatentDims:
+    """Latent attention; `kv` is None for a layer that reads another layer's cache rows."""
+    heads: int
+    dim: int
+    rot: int
+    vdim: int
+    rank: int
+    scale: float
+    base: float
+    rot_dims: int
+    q: int
+    g: int
+    kv: Optional[int]
+
+
+# ------------------------------------------------------------------ residual stream
+def embed_scaled(ids, weight, width: int, scale: float):
+    """(fp32 residual [T, width], its copy in the model's dtype [T, padded width]) of table rows times `scale`."""
+    if weight.is_cuda:
+        _n()
+        return ext().embed_scaled(ids, weight, int(width), float(scale))
+    return ref.embed_scaled(ids, weight, width, scale)
+
+
+def linear_post_norm_add(a, weight, bias, x, norm_w, eps: float):
+    """x += RMSNorm(a @ weight.T + bias) * norm_w in fp32, in place; returns x in the model's dtype (padded width)."""
+    if a.is_cuda:
+        _n(2)
+        return ext().linear_post_norm_add(a, weight, bias, x, norm_w, float(eps))
+    return ref.post_norm_add(ref_linear(a, weight, bias), x, norm_w, eps)
+
+
+def rms_norm_wide(x, norm_w, eps: float, width: int, dtype):
+    """RMSNorm of the fp32 residual in the model's dtype, zero-padded to `width` columns."""
+    if x.is_cuda:
+        _n()
+        return ext().rms_norm_wide(x, norm_w, float(eps), int(width), dtype == torch.float32)
+    return ref.rms_norm_wide(x, norm_w, eps, width, dtype)
+
+
+def linear_gelu_mul(h, weight, bias, up_off: int, width: int):
+    """gelu_tanh(gate) * up of the packed projections gate | up (`up` from column `up_off`), padded to 8 columns."""
+    if h.is_cuda:
+        _n(2)
+        return ext().linear_gelu_mul(h, weight, bias, int(up_off), int(width))
+    return ref.gelu_tanh_and_mul(ref_linear(h, weight, bias), up_off, width)
+
+
+def ref_linear(x, weight, bias=None):
+    from . import linear
+    return linear(x, weight, bias)
+
+
+# ------------------------------------------------------------------ recurrent layers
+def gla(h, weight, d: GlaDims, a2_weight, z_bias, norm_w, eps: float, state, ctx):
+    """Gated linear attention of a batch of runs up to (not including) the output projection."""
+    if h.is_cuda:
+        _n(4)
+        return ext().gla(h, weight, a2_weight, z_bias, norm_w, float(eps), state,
+                         [d.heads, d.dim, d.vdim, d.rank, d.q, d.k, d.v, d.g, d.a1], float(d.tau), *_run_args(ctx))
+    p = ref_linear(h, weight)
+    z = ref_linear(p[:, d.a1:d.a1 + a2_weight.shape[1]], a2_weight)
+    return ref.gla(p, z, d, z_bias, norm_w, eps, state, ctx)
+
+
+def delta_rule(h, weight, d: DeltaDims, conv_w, a_log, dt_bias, norm_w, eps: float, conv_state, state, ctx):
+    """Gated delta rule (with its short convolutions) of a batch of runs up to the output projection."""
+    if h.is_cuda:
+        _n(4)
+        return ext().delta_rule(h, weight, conv_w, a_log, dt_bias, norm_w, float(eps), conv_state, state,
+                                [d.heads, d.kv_heads, d.dim, d.vdim, d.g, d.b, d.a], float(d.unit_eps),
+                                *_run_args(ctx))
+    return ref.delta_rule(ref_linear(h, weight), d, conv_w, a_log, dt_bias, norm_w, eps, conv_state, state, ctx)
+
+
+def _run_args(ctx):
+    """Batch layout for the recurrent kernels: run boundaries (None: one row per request), rows per request after
+    this step, state slots, longest run."""
+    return ctx.cu_seqlens_q, ctx.context_lens, ctx.state_slots, int(ctx.max_seqlen_q) if ctx.is_prefill else 1
+
+
+# ------------------------------------------------------------------ latent attention
+def latent_attention(h, weight, d: LatentDims, kv_norm_w, eps: float, kv_proj, w_ukt, w_uv, pool, positions, ctx):
+    """Projections, cache store, attention and output gate of a latent-attention layer up to the output projection.
+
+    `kv_proj` (packed uk | uv) expands cache rows to keys and values (prefill); `w_ukt` [H, rank, dim] and `w_uv`
+    [H, vdim, rank] are the same weights for the absorbed form (decode), which never expands a row."""
+    if h.is_cuda:
+        from .latent import latent_attention_cuda
+        return latent_attention_cuda(h, weight, d, kv_norm_w, eps, kv_proj, w_ukt, w_uv, pool, positions, ctx)
+    p = ref_linear(h, weight)
+    q = ref.latent_project(p, d, kv_norm_w, eps, positions, pool, ctx.slot_mapping)
+    w, off = kv_proj.weight, kv_proj.offset
+    return ref.latent_attention(q, p[:, d.g:d.g + d.heads * d.vdim], d, w[off["uk"]:off["uk"] + d.heads * d.dim],
+                                w[off["uv"]:off["uv"] + d.heads * d.vdim], pool, ctx)

@@ -1,0 +1,157 @@
+"""Plain PyTorch statements of the ops of hybrid models: sublayer-output norm on a 32-bit residual, short
+convolution, gated linear attention, gated delta rule and paged latent attention.
+
+Like `reference.py`: the execution path on CPU tensors.  A batch is a concatenation of runs of rows, one run per
+request, with the request's state slot and the position of its first row; a run that starts at position 0 starts
+from a zero state.
+"""
+from __future__ import annotations
+
+from typing import List, Optional, Tuple
+
+import torch
+import torch.nn.functional as F
+
+from .reference import _rotate
+
+
+def runs(ctx) -> List[Tuple[int, int, int, int, int]]:
+    """(request, first row, end row, position of the first row, state slot) of every run of the batch."""
+    lens = ctx.context_lens.tolist()
+    cu = list(range(len(lens) + 1)) if ctx.cu_seqlens_q is None else ctx.cu_seqlens_q.tolist()
+    slots = ctx.state_slots.tolist() if ctx.state_slots is not None else [-1] * len(lens)
+    return [(i, cu[i], cu[i + 1], n - (cu[i + 1] - cu[i]), slots[i]) for i, n in enumerate(lens)
+            if n > 0 and cu[i + 1] > cu[i]]
+
+
+def _pad_to(x: torch.Tensor, width: int) -> torch.Tensor:
+    return F.pad(x, (0, width - x.shape[-1]))
+
+
+def _rms(x: torch.Tensor, eps: float) -> torch.Tensor:
+    return x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps)
+
+
+# ------------------------------------------------------------------ residual stream
+def embed_scaled(ids, weight, width: int, scale: float):
+    h = F.embedding(ids, weight)
+    x = h[:, :width].float() * scale
+    return x, _pad_to(x.to(weight.dtype), weight.shape[1])
+
+
+def post_norm_add(y, x, weight, eps: float):
+    x += _rms(y[:, : x.shape[1]].float(), eps) * weight
+    return _pad_to(x.to(y.dtype), y.shape[1])
+
+
+def rms_norm_wide(x, weight, eps: float, width: int, dtype):
+    return _pad_to((_rms(x, eps) * weight).to(dtype), width)
+
+
+def gelu_tanh_and_mul(gu, up_off: int, width: int):
+    a = F.gelu(gu[:, :width].float(), approximate="tanh") * gu[:, up_off:up_off + width].float()
+    return _pad_to(a.to(gu.dtype), -(-width // 8) * 8)
+
+
+# ------------------------------------------------------------------ recurrent layers
+def short_conv(p, conv_w, conv_state, ctx):
+    """silu(depthwise causal convolution) of the first C columns of p, per run; updates the kept inputs."""
+    C, taps = conv_w.shape
+    x = p[:, :C].float()
+    out = torch.zeros_like(x)
+    for _, lo, hi, start, slot in runs(ctx):
+        past = x.new_zeros(taps - 1, C) if start == 0 else conv_state[slot]
+        seq = torch.cat([past, x[lo:hi]])
+        out[lo:hi] = F.silu(sum(seq[j:j + hi - lo] * conv_w[:, j] for j in range(taps)))
+        if taps > 1:
+            conv_state[slot] = seq[hi - lo:]
+    return out
+
+
+def gated_head_norm(o, gate, norm_w, eps: float, dtype):
+    """rms(o) * norm_w * silu(gate) per head; o [T, H, V] fp32 -> [T, pad8(H * V)]."""
+    T, H, V = o.shape
+    y = (_rms(o, eps) * norm_w).reshape(T, H * V) * F.silu(gate.float())
+    return _pad_to(y.to(dtype), -(-H * V // 8) * 8)
+
+
+def gla(p, z, d, z_bias, norm_w, eps: float, state, ctx):
+    """d: sizes and column offsets (`ops.hybrid.GlaDims`); p packed projections, z decay projection [T, H * D]."""
+    T, H, D, V = p.shape[0], d.heads, d.dim, d.vdim
+    q = p[:, d.q:d.q + H * D].float().view(T, H, D) * D ** -0.5
+    k = p[:, d.k:d.k + H * D].float().view(T, H, D)
+    v = p[:, d.v:d.v + H * V].float().view(T, H, V)
+    alpha = torch.exp(F.logsigmoid(z[:, : H * D].float() + z_bias) / d.tau).view(T, H, D)
+    o = q.new_zeros(T, H, V)
+    for _, lo, hi, start, slot in runs(ctx):
+        S = state.new_zeros(H, D, V) if start == 0 else state[slot].clone()
+        for t in range(lo, hi):
+            S = alpha[t][:, :, None] * S + k[t][:, :, None] * v[t][:, None, :]
+            o[t] = torch.einsum("hdv,hd->hv", S, q[t])
+        state[slot] = S
+    return gated_head_norm(o, p[:, d.g:d.g + H * V], norm_w, eps, p.dtype)
+
+
+def delta_rule(p, d, conv_w, a_log, dt_bias, norm_w, eps: float, conv_state, state, ctx):
+    """d: `ops.hybrid.DeltaDims`; p packed projections whose first columns are q | k | v."""
+    T, H, K, D, V = p.shape[0], d.heads, d.kv_heads, d.dim, d.vdim
+    c = short_conv(p, conv_w, conv_state, ctx)
+    q, k = c[:, : K * D].reshape(T, K, D), c[:, K * D: 2 * K * D].reshape(T, K, D)
+    q, k = (x * torch.rsqrt(x.pow(2).sum(-1, keepdim=True) + d.unit_eps) for x in (q, k))
+    q, k = (x.repeat_interleave(H // K, 1) for x in (q * D ** -0.5, k))
+    v = c[:, 2 * K * D:].to(p.dtype).float().view(T, H, V)
+    beta = torch.sigmoid(p[:, d.b:d.b + H].float())
+    g = torch.exp(-torch.exp(a_log) * F.softplus(p[:, d.a:d.a + H].float() + dt_bias))
+    o = q.new_zeros(T, H, V)
+    for _, lo, hi, start, slot in runs(ctx):
+        S = state.new_zeros(H, D, V) if start == 0 else state[slot].clone()
+        for t in range(lo, hi):
+            S = g[t][:, None, None] * S
+            u = beta[t][:, None] * (v[t] - torch.einsum("hdv,hd->hv", S, k[t]))
+            S = S + k[t][:, :, None] * u[:, None, :]
+            o[t] = torch.einsum("hdv,hd->hv", S, q[t])
+        state[slot] = S
+    return gated_head_norm(o, p[:, d.g:d.g + H * V], norm_w, eps, p.dtype)
+
+
+# ------------------------------------------------------------------ latent attention
+def _rope(x, positions, base: float, dims: int):
+    i = torch.arange(dims // 2, dtype=torch.float64, device=x.device)
+    a = positions.double()[:, None, None] * base ** (-2 * i / dims)
+    cos, sin = a.cos().float(), a.sin().float()
+    return torch.cat([_rotate(x[..., :dims].float(), cos, sin), x[..., dims:].float()], -1).to(x.dtype)
+
+
+def latent_project(p, d, norm_w, eps: float, positions, pool, slots):
+    """Writes the cache rows (normed latent | rotated shared key part) of a layer that owns a cache and returns the
+    queries with their rotated part rotated, [T, H, dim + rot]."""
+    T = p.shape[0]
+    q = p[:, d.q:d.q + d.heads * (d.dim + d.rot)].reshape(T, d.heads, d.dim + d.rot).clone()
+    q[..., d.dim:] = _rope(q[..., d.dim:], positions, d.base, d.rot_dims)
+    if d.kv is not None:
+        kv = p[:, d.kv:d.kv + d.rank + d.rot]
+        c = (_rms(kv[:, : d.rank].float(), eps) * norm_w).to(p.dtype)
+        r = _rope(kv[:, None, d.rank:], positions, d.base, d.rot_dims)[:, 0]
+        ok = slots >= 0
+        flat = pool.view(-1, pool.shape[-1])
+        flat[slots[ok].long(), : d.rank + d.rot] = torch.cat([c, r], -1)[ok].to(pool.dtype)
+    return q
+
+
+def latent_attention(q, gate, d, w_uk, w_uv, pool, ctx):
+    """Causal attention of the rows of `q` over the cache rows of their requests, times sigmoid(gate)."""
+    T, H = q.shape[0], d.heads
+    out = torch.zeros(T, H, d.vdim, dtype=torch.float32)
+    for i, lo, hi, start, _ in runs(ctx):
+        n = start + hi - lo
+        blocks = ctx.block_tables[i][: -(-n // pool.shape[1])].long()
+        rows = pool[blocks].reshape(-1, pool.shape[-1])[:n].float()
+        c, r = rows[:, : d.rank], rows[:, d.rank: d.rank + d.rot]
+        kn = (c @ w_uk[:, : d.rank].float().T).view(n, H, d.dim)
+        v = (c @ w_uv[:, : d.rank].float().T).view(n, H, d.vdim)
+        s = torch.einsum("ihd,jhd->hij", q[lo:hi, :, : d.dim].float(), kn)
+        s = (s + torch.einsum("ihd,jd->hij", q[lo:hi, :, d.dim:].float(), r)) * d.scale
+        hidden = torch.arange(n)[None, :] > torch.arange(start, n)[:, None]
+        out[lo:hi] = torch.einsum("hij,jhv->ihv", torch.softmax(s.masked_fill(hidden, float("-inf")), -1), v)
+    y = out.reshape(T, H * d.vdim) * torch.sigmoid(gate.float())
+    return _pad_to(y.to(q.dtype), -(-H * d.vdim // 8) * 8)

@@ -31,6 +31,14 @@ class Context:
     obs_window: int = 0
     attn_workspace: Any = None
     tp: Any = None
+    # models with recurrent or latent-attention layers: the state slot of every request (-1: padding row of a
+    # captured batch) and, in prefill, the request and the visible rows (position + 1) of every flat row
+    state_slots: Optional[torch.Tensor] = None
+    row_seq: Optional[torch.Tensor] = None
+    row_ctx: Optional[torch.Tensor] = None
+    # latent attention in prefill: first row of every request in the batch's gathered cache rows, their total
+    cu_seqlens_kv: Optional[torch.Tensor] = None
+    total_kv: int = 0
 
 
 _CONTEXT = Context()
@@ -42,11 +50,11 @@ def get_context() -> Context:
 
 def set_context(is_prefill: bool, cu_seqlens_q=None, cu_seqlens_k=None, max_seqlen_q=0, max_seqlen_k=0,
                 slot_mapping=None, context_lens=None, block_tables=None, logits_indices=None,
-                window_q=None, obs_window=0, attn_workspace=None, tp=None) -> Context:
+                window_q=None, obs_window=0, attn_workspace=None, tp=None, **layer_fields) -> Context:
     global _CONTEXT
     _CONTEXT = Context(is_prefill, cu_seqlens_q, cu_seqlens_k, max_seqlen_q, max_seqlen_k,
                        slot_mapping, context_lens, block_tables, logits_indices, window_q,
-                       obs_window, attn_workspace, tp)
+                       obs_window, attn_workspace, tp, **layer_fields)
     return _CONTEXT
 
 

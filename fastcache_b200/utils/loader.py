@@ -37,6 +37,7 @@ def load_weights(model: nn.Module, named_tensors: Iterable[Tuple[str, torch.Tens
     packed = getattr(model, "packed_modules_mapping", {})
     prefix_map = getattr(model, "checkpoint_prefix_map", {})
     skip = tuple(getattr(model, "skip_weight_substrings", ()))
+    table = getattr(model, "checkpoint_map", None)       # explicit: checkpoint name -> (parameter, shard id)
     params = dict(model.named_parameters())
     buffers = dict(model.named_buffers())
     stats = {"loaded": 0, "skipped": 0, "unknown": 0}
@@ -52,12 +53,14 @@ def load_weights(model: nn.Module, named_tensors: Iterable[Tuple[str, torch.Tens
             continue
         name = _resolve(model, name, prefix_map)
         target, shard_id = name, None
+        if table is not None:
+            target, shard_id = table.get(name, (None, None))
         for key, (packed_name, sid) in packed.items():
             if f".{key}." in name or name.startswith(key + "."):
                 target = name.replace(key, packed_name)
                 shard_id = sid
                 break
-        if target not in params and name in params:
+        if table is None and target not in params and name in params:
             # the name only looks packed: the vision towers keep separate q / k / v projections under the same
             # leaf names that the language model packs
             target, shard_id = name, None
@@ -84,6 +87,9 @@ def missing_parameters(model: nn.Module, seen) -> list:
     """Parameters of `model` that no checkpoint tensor reached: a plain parameter needs its own tensor, a packed
     one (qkv_proj, gate_up_proj) every shard of its group.  Tied parameters (the LM head sharing the embedding
     table) count once.  Modules listed in `model.optional_weight_substrings` may stay at their initial values."""
+    table = getattr(model, "checkpoint_map", None)
+    if table is not None:
+        return sorted(name for name, entry in table.items() if entry not in seen)
     packed = getattr(model, "packed_modules_mapping", {})
     optional = tuple(o for m in model.modules() for o in getattr(m, "optional_weight_substrings", ()))
     groups: Dict[str, set] = {}
@@ -121,6 +127,17 @@ def iter_safetensors(path: str) -> Iterable[Tuple[str, torch.Tensor]]:
                 yield name, f.get_tensor(name)
 
 
+def checkpoint_shapes(path: str) -> Dict[str, Tuple[int, ...]]:
+    """Tensor names and shapes of a checkpoint directory (headers only)."""
+    from safetensors import safe_open
+    shapes: Dict[str, Tuple[int, ...]] = {}
+    for file in sorted(glob(os.path.join(path, "*.safetensors"))):
+        with safe_open(file, "pt", "cpu") as f:
+            for name in f.keys():
+                shapes[name] = tuple(f.get_slice(name).get_shape())
+    return shapes
+
+
 def load_model(model: nn.Module, path: str, strip_prefix: str = "", verbose: bool = False,
                strict: bool = True) -> Dict[str, int]:
     """Load every `*.safetensors` file of `path`.  With `strict` (default) a parameter that no checkpoint tensor
@@ -154,9 +171,8 @@ def random_named_tensors(shapes: Dict[str, Tuple[int, ...]], seed: int = 0, std:
     """
     import zlib
     for name, shape in shapes.items():
-        leaf = name.rsplit(".", 2)
-        is_norm_w = name.endswith("weight") and len(shape) == 1 and any(
-            k in name for k in ("norm", "layernorm", "ln_", ".ln", "layer_norm"))
+        is_norm_w = len(shape) == 1 and (name.rsplit(".", 1)[-1].startswith("norm") or name.endswith("weight") and any(
+            k in name for k in ("norm", "layernorm", "ln_", ".ln", "layer_norm")))
         if is_norm_w:
             yield name, torch.ones(shape, dtype=dtype, device=device)
             continue
