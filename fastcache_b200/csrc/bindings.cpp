@@ -547,7 +547,8 @@ Tensor dense_attention(const Tensor& q, const Tensor& k, const Tensor& v, double
 // entries >= v_limit (-1: none) are padding.
 Tensor sample(const Tensor& logits, const Tensor& temps, int64_t seed, bool with_status, int64_t vocab_offset,
               int64_t v_limit) {
-  check_bf16(logits, "logits");
+  const bool f32 = logits.scalar_type() == torch::kFloat32 && logits.is_cuda();
+  if (!f32) check_bf16(logits, "logits");
   TORCH_CHECK(logits.dim() == 2 && logits.stride(1) == 1, "logits must be [B, V] with unit inner stride");
   TORCH_CHECK(temps.is_cuda() && temps.scalar_type() == torch::kFloat32 && temps.numel() == logits.size(0),
               "temperatures must be fp32 [B] on the device");
@@ -557,7 +558,7 @@ Tensor sample(const Tensor& logits, const Tensor& temps, int64_t seed, bool with
   if (B == 0 && with_status) out.zero_();
   fc::launch_sample(logits.data_ptr(), temps.data_ptr(), out.data_ptr(), int(B), int(logits.size(1)),
                     logits.stride(0), uint32_t(seed), at::cuda::getCurrentCUDAStream(), int(vocab_offset),
-                    int(v_limit), with_status ? status_ptr(logits.get_device()) : nullptr);
+                    int(v_limit), with_status ? status_ptr(logits.get_device()) : nullptr, f32);
   return out;
 }
 
@@ -606,6 +607,7 @@ void register_stream_sms(int64_t stream_ptr, int64_t sms) {
 void register_greenctx(pybind11::module_& m);
 void register_compress(pybind11::module_& m);
 void register_comm(pybind11::module_& m);
+void register_hybrid(pybind11::module_& m);
 void register_symm(pybind11::module_& m);
 
 namespace fc {
@@ -669,5 +671,6 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   register_greenctx(m);
   register_compress(m);
   register_comm(m);
+  register_hybrid(m);
   register_symm(m);
 }

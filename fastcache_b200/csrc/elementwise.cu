@@ -402,8 +402,9 @@ rope_qknorm_store_d128_kernel(const bf16* __restrict__ qkv, const long long* __r
 constexpr int SAMPLE_SPLIT = 4;
 constexpr int SAMPLE_THREADS = 512;
 
+template <typename T>
 __global__ void __launch_bounds__(SAMPLE_THREADS)
-sample_kernel(const bf16* __restrict__ logits, const float* __restrict__ temps, long long* __restrict__ out,
+sample_kernel(const T* __restrict__ logits, const float* __restrict__ temps, long long* __restrict__ out,
               int V, long long ld, uint32_t seed, int vocab_offset, int v_limit, const uint32_t* status) {
   __shared__ float s_val[32];
   __shared__ int s_idx[32];
@@ -499,12 +500,14 @@ void launch_rope_qknorm_store(const void* qkv, const void* positions, const void
 }
 
 void launch_sample(const void* logits, const void* temps, void* out, int B, int V, long long ld, uint32_t seed,
-                   cudaStream_t s, int vocab_offset, int v_limit, const uint32_t* status) {
+                   cudaStream_t s, int vocab_offset, int v_limit, const uint32_t* status, bool f32) {
   if (B == 0) return;
-  const cudaError_t e =
-      launch_pdl_cluster(PDL_SAMPLE, sample_kernel, dim3(B, SAMPLE_SPLIT), dim3(SAMPLE_THREADS), 0, s, SAMPLE_SPLIT,
-                         (const bf16*)logits, (const float*)temps, (long long*)out, V, ld, seed, vocab_offset,
-                         v_limit < 0 ? vocab_offset + V : v_limit, status);
+  auto go = [&](auto* rows, auto kern) {
+    return launch_pdl_cluster(PDL_SAMPLE, kern, dim3(B, SAMPLE_SPLIT), dim3(SAMPLE_THREADS), 0, s, SAMPLE_SPLIT, rows,
+                              (const float*)temps, (long long*)out, V, ld, seed, vocab_offset,
+                              v_limit < 0 ? vocab_offset + V : v_limit, status);
+  };
+  const cudaError_t e = f32 ? go((const float*)logits, sample_kernel<float>) : go((const bf16*)logits, sample_kernel<bf16>);
   // a cluster that the stream's SM set cannot place is a launch error, not a kernel that ran: say so here
   if (e != cudaSuccess) throw std::runtime_error(std::string("sampler launch: ") + cudaGetErrorString(e));
 }

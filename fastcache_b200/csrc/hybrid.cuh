@@ -1,0 +1,111 @@
+// Device helpers of the hybrid-model kernels: element type conversion and reads of projection outputs.
+#pragma once
+#include <cuda_bf16.h>
+#include <cuda_runtime.h>
+#include <stdint.h>
+
+#include "hybrid.h"
+#include "ptx.cuh"
+
+namespace fc {
+
+template <typename T>
+struct Elem;
+template <>
+struct Elem<float> {
+  static __device__ __forceinline__ float get(float v) { return v; }
+  static __device__ __forceinline__ float put(float v) { return v; }
+};
+template <>
+struct Elem<__nv_bfloat16> {
+  static __device__ __forceinline__ float get(__nv_bfloat16 v) { return __bfloat162float(v); }
+  static __device__ __forceinline__ __nv_bfloat16 put(float v) { return __float2bfloat16(v); }
+};
+
+// one element of a projection output
+template <typename T>
+__device__ __forceinline__ float proj_at(const ProjSrc& s, long long row, int col) {
+  if (s.splits > 1) {
+    float v = 0.f;
+    const float* p = s.part + row * s.part_ld + col;
+    for (int i = 0; i < s.splits; ++i) v += __ldcg(p + i * s.part_stride);
+    return v;
+  }
+  return Elem<T>::get(reinterpret_cast<const T*>(s.p)[row * s.ld + col]);
+}
+
+// four consecutive elements; `col` and the pitches are multiples of 4
+template <typename T>
+__device__ __forceinline__ float4 proj_at4(const ProjSrc& s, long long row, int col) {
+  if (s.splits > 1) {
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+    const float* p = s.part + row * s.part_ld + col;
+#pragma unroll 4
+    for (int i = 0; i < s.splits; ++i) {
+      const float4 a = __ldcg(reinterpret_cast<const float4*>(p + i * s.part_stride));
+      v.x += a.x;
+      v.y += a.y;
+      v.z += a.z;
+      v.w += a.w;
+    }
+    return v;
+  }
+  const T* q = reinterpret_cast<const T*>(s.p) + row * s.ld + col;
+  if constexpr (sizeof(T) == 4) {
+    return __ldcg(reinterpret_cast<const float4*>(q));
+  } else {
+    const uint2 u = __ldcg(reinterpret_cast<const uint2*>(q));
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x));
+    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
+    return make_float4(a.x, a.y, b.x, b.y);
+  }
+}
+
+template <typename T>
+__device__ __forceinline__ void store4(T* dst, float a, float b, float c, float d) {
+  if constexpr (sizeof(T) == 4) {
+    *reinterpret_cast<float4*>(dst) = make_float4(a, b, c, d);
+  } else {
+    uint2 u;
+    u.x = pack_bf16(a, b);
+    u.y = pack_bf16(c, d);
+    *reinterpret_cast<uint2*>(dst) = u;
+  }
+}
+
+__device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
+__device__ __forceinline__ float silu_f(float x) { return x / (1.f + expf(-x)); }
+// log(sigmoid(x)) and log(1 + exp(x)) without overflow
+__device__ __forceinline__ float log_sigmoid_f(float x) { return fminf(x, 0.f) - log1pf(expf(-fabsf(x))); }
+__device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
+__device__ __forceinline__ float gelu_tanh_f(float z) {
+  return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+}
+
+struct Run {
+  int lo, len, start, slot;
+};
+__device__ __forceinline__ Run get_run(const RunBatch& r, int b) {
+  Run o;
+  o.lo = r.cu != nullptr ? r.cu[b] : b;
+  o.len = r.cu != nullptr ? r.cu[b + 1] - o.lo : 1;
+  const int n = r.ctx[b];
+  o.slot = r.slots[b];
+  o.start = n - o.len;
+  if (n <= 0 || o.slot < 0 || o.slot >= r.num_slots) o.slot = -1;
+  return o;
+}
+
+template <int THREADS>
+__device__ __forceinline__ float cta_sum(float v, float* red) {
+  v = warp_sum(v);
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+  __syncthreads();
+  float t = 0.f;
+#pragma unroll
+  for (int i = 0; i < THREADS / 32; ++i) t += red[i];
+  __syncthreads();
+  return t;
+}
+
+}  // namespace fc

@@ -1,0 +1,515 @@
+// Python bindings of the hybrid-model kernels.  Tensors are checked here, so that the kernels can assume their layout.
+#include <ATen/cuda/CUDAContext.h>
+#include <c10/cuda/CUDAGuard.h>
+#include <torch/extension.h>
+
+#include <tuple>
+#include <vector>
+
+#include "gemm.h"
+#include "hybrid.h"
+#include "workspace.h"
+
+namespace {
+
+using torch::Tensor;
+using OptTensor = c10::optional<Tensor>;
+
+bool is_f32(const Tensor& t) { return t.scalar_type() == torch::kFloat32; }
+cudaStream_t stream_now() { return at::cuda::getCurrentCUDAStream(); }
+const fc::StreamWorkspace& ws_of(const Tensor& t) { return fc::stream_workspace(t.get_device(), stream_now()); }
+int pad8(int n) { return (n + 7) / 8 * 8; }
+
+void check_elem(const Tensor& t, const char* name) {
+  TORCH_CHECK(t.is_cuda() && (t.scalar_type() == torch::kBFloat16 || is_f32(t)), name, " must be a bf16 or fp32 CUDA tensor");
+}
+void check_f32(const Tensor& t, const char* name, int64_t n) {
+  TORCH_CHECK(t.is_cuda() && is_f32(t) && t.is_contiguous() && t.numel() == n, name, " must be a contiguous fp32 tensor of ",
+              n, " elements");
+}
+void check_i32(const Tensor& t, const char* name, int64_t n) {
+  TORCH_CHECK(t.is_cuda() && t.scalar_type() == torch::kInt32 && t.is_contiguous() && t.numel() >= n, name,
+              " must be a contiguous int32 tensor of at least ", n, " elements");
+}
+
+// x @ w.T.  `partial`: decode-size bf16 products may stay split-K partial sums in the stream's scratch, valid until
+// the next product on this stream.  `hold` keeps the finished output alive.
+fc::ProjSrc project(const Tensor& x, const Tensor& w, const OptTensor& bias, bool partial, Tensor& hold) {
+  check_elem(x, "x");
+  TORCH_CHECK(x.scalar_type() == w.scalar_type() && x.dim() == 2 && w.dim() == 2 && x.size(1) == w.size(1) &&
+                  x.stride(1) == 1 && w.is_contiguous() && w.size(1) % 8 == 0 && w.size(0) % 8 == 0 &&
+                  x.stride(0) % 8 == 0, "projection operands must be row-major matrices padded to multiples of 8");
+  const int M = int(x.size(0)), N = int(w.size(0)), K = int(x.size(1));
+  const void* bp = nullptr;
+  if (bias.has_value() && bias->defined()) {
+    TORCH_CHECK(bias->scalar_type() == x.scalar_type() && bias->is_contiguous() && bias->numel() == N, "bad bias");
+    bp = bias->data_ptr();
+  }
+  fc::ProjSrc src;
+  hold = torch::empty({M, N}, x.options());
+  src.p = hold.data_ptr();
+  src.ld = N;
+  if (M == 0) return src;
+  if (is_f32(x)) {
+    fc::SimtLinear a;
+    a.x = x.data_ptr();
+    a.w = w.data_ptr();
+    a.bias = bp;
+    a.y = hold.data_ptr();
+    a.M = M;
+    a.N = N;
+    a.K = K;
+    a.ldx = x.stride(0);
+    a.ldw = K;
+    a.ldy = N;
+    fc::launch_linear_simt(a, true, stream_now());
+    return src;
+  }
+  const auto& ws = ws_of(x);
+  fc::GemmWorkspace gw;
+  gw.scratch = ws.gemm_scratch;
+  gw.counters = ws.gemm_counters;
+  gw.status = ws.status;
+  gw.grid_sync = ws.grid_sync;
+  const int sms = fc::stream_sm_limit(stream_now());
+  if (partial && M <= 256 && bp == nullptr) {
+    const int splits = fc::gemm_skinny_bf16(x.data_ptr(), w.data_ptr(), hold.data_ptr(), nullptr, M, N, K, x.stride(0),
+                                            K, N, 0, gw, sms, 0, false, stream_now());
+    if (splits > 1) {
+      src.part = ws.gemm_scratch;
+      src.splits = splits;
+      src.part_stride = (long long)M * N;
+      src.part_ld = N;
+    }
+    return src;
+  }
+  fc::gemm_bf16(x.data_ptr(), w.data_ptr(), hold.data_ptr(), bp, M, N, K, x.stride(0), K, N, 0, gw, sms, stream_now());
+  return src;
+}
+
+Tensor linear_wide(const Tensor& x, const Tensor& w, const OptTensor& bias) {
+  c10::cuda::CUDAGuard guard(x.device());
+  Tensor y;
+  project(x, w, bias, false, y);
+  return y;
+}
+
+std::tuple<Tensor, Tensor> embed_scaled(const Tensor& ids, const Tensor& weight, int64_t W, double scale) {
+  check_elem(weight, "weight");
+  TORCH_CHECK(ids.is_cuda() && ids.scalar_type() == torch::kInt64 && ids.is_contiguous(), "ids must be int64 CUDA");
+  TORCH_CHECK(weight.is_contiguous() && weight.dim() == 2 && weight.size(1) >= W, "bad embedding table");
+  c10::cuda::CUDAGuard guard(weight.device());
+  const int64_t T = ids.numel(), Wp = weight.size(1);
+  Tensor x = torch::empty({T, W}, weight.options().dtype(torch::kFloat32)), h = torch::empty({T, Wp}, weight.options());
+  fc::launch_embed_scaled(ids.data_ptr(), weight.data_ptr(), x.data_ptr<float>(), h.data_ptr(), int(T), int(W), int(Wp),
+                          weight.size(0), float(scale), is_f32(weight), ws_of(weight).status, stream_now());
+  return {x, h};
+}
+
+// x += rms(a @ w.T + bias) * norm_w; returns x in the element type of a, padded to the width of w's output
+Tensor linear_post_norm_add(const Tensor& a, const Tensor& w, const OptTensor& bias, Tensor x, const Tensor& norm_w,
+                            double eps) {
+  c10::cuda::CUDAGuard guard(a.device());
+  const int64_t T = a.size(0), W = x.size(1), Wp = w.size(0);
+  check_f32(x, "residual", T * W);
+  check_f32(norm_w, "norm weight", W);
+  TORCH_CHECK(Wp >= W, "projection narrower than the residual");
+  Tensor hold;
+  const void* bp = nullptr;
+  if (bias.has_value() && bias->defined()) {
+    TORCH_CHECK(bias->scalar_type() == a.scalar_type() && bias->is_contiguous() && bias->numel() == Wp, "bad bias");
+    bp = bias->data_ptr();
+  }
+  const fc::ProjSrc src = project(a, w, c10::nullopt, true, hold);
+  Tensor h = torch::empty({T, Wp}, a.options());
+  fc::launch_post_norm_add(src, bp, x.data_ptr<float>(), norm_w.data_ptr<float>(), h.data_ptr(), int(T), int(W), int(Wp),
+                           float(eps), is_f32(a), stream_now());
+  return h;
+}
+
+Tensor rms_norm_wide(const Tensor& x, const Tensor& norm_w, double eps, int64_t Wp, bool f32) {
+  const int64_t T = x.size(0), W = x.size(1);
+  check_f32(x, "residual", T * W);
+  check_f32(norm_w, "norm weight", W);
+  c10::cuda::CUDAGuard guard(x.device());
+  Tensor h = torch::empty({T, Wp}, x.options().dtype(f32 ? torch::kFloat32 : torch::kBFloat16));
+  fc::launch_rms_norm_wide(x.data_ptr<float>(), norm_w.data_ptr<float>(), h.data_ptr(), int(T), int(W), int(Wp),
+                           float(eps), f32, stream_now());
+  return h;
+}
+
+Tensor linear_gelu_mul(const Tensor& h, const Tensor& w, const OptTensor& bias, int64_t up_off, int64_t width) {
+  c10::cuda::CUDAGuard guard(h.device());
+  const int64_t T = h.size(0), N = w.size(0), wp = pad8(int(width));
+  TORCH_CHECK(up_off % 8 == 0 && up_off >= width && up_off + wp <= N, "bad gate | up layout");
+  const void* bp = nullptr;
+  if (bias.has_value() && bias->defined()) {
+    TORCH_CHECK(bias->scalar_type() == h.scalar_type() && bias->is_contiguous() && bias->numel() == N, "bad bias");
+    bp = bias->data_ptr();
+  }
+  Tensor hold;
+  const fc::ProjSrc src = project(h, w, c10::nullopt, true, hold);
+  Tensor out = torch::empty({T, wp}, h.options());
+  fc::launch_gelu_mul(src, bp, out.data_ptr(), int(T), int(up_off), int(width), int(wp), is_f32(h), stream_now());
+  return out;
+}
+
+fc::RunBatch run_batch(const OptTensor& cu, const Tensor& ctx, const Tensor& slots, const Tensor& state) {
+  fc::RunBatch r;
+  r.B = int(slots.numel());
+  check_i32(slots, "state slots", r.B);
+  check_i32(ctx, "context lengths", r.B);
+  if (cu.has_value() && cu->defined()) {
+    check_i32(*cu, "run boundaries", r.B + 1);
+    r.cu = cu->data_ptr<int>();
+  }
+  r.ctx = ctx.data_ptr<int>();
+  r.slots = slots.data_ptr<int>();
+  r.num_slots = int(state.size(0));
+  return r;
+}
+
+constexpr int CHUNK_MIN_ROWS = 24;      // longest run of a batch from which the chunked kernels are used
+
+void run_recurrence(fc::StepParams& p, const Tensor& h, bool delta, bool chunk, int T, int max_len, Tensor& out,
+                    Tensor& o_raw) {
+  const bool f32 = is_f32(h);
+  out = torch::empty({T, pad8(p.H * p.V)}, h.options());
+  const bool fused = !chunk && fc::step_fuses_norm(p.D, p.V);
+  p.ld_out = out.size(1);
+  if (fused) {
+    p.out = out.data_ptr();
+  } else {
+    o_raw = torch::empty({T, p.H * p.V}, h.options().dtype(torch::kFloat32));
+    p.o_raw = o_raw.data_ptr<float>();
+  }
+  if (chunk) {
+    if (delta) fc::launch_delta_chunk(p, max_len, stream_now());
+    else fc::launch_gla_chunk(p, max_len, stream_now());
+  } else {
+    if (delta) fc::launch_delta_step(p, f32, stream_now());
+    else fc::launch_gla_step(p, f32, stream_now());
+  }
+  if (!fused)
+    fc::launch_gated_head_norm(p.o_raw, p.proj, p.off_g, p.norm_w, p.eps, out.data_ptr(), p.ld_out, T, p.H, p.V, f32,
+                               stream_now());
+}
+
+Tensor gla(const Tensor& h, const Tensor& w, const Tensor& w_a2, const Tensor& z_bias, const Tensor& norm_w, double eps,
+           Tensor state, const std::vector<int64_t>& d, double tau, const OptTensor& cu, const Tensor& ctx,
+           const Tensor& slots, int64_t max_len) {
+  TORCH_CHECK(d.size() == 9, "gla: nine sizes and offsets");
+  const int H = int(d[0]), D = int(d[1]), V = int(d[2]), rank = int(d[3]);
+  c10::cuda::CUDAGuard guard(h.device());
+  const int T = int(h.size(0));
+  check_f32(state, "state", state.size(0) * H * D * V);
+  check_f32(z_bias, "decay bias", (int64_t)H * D);
+  check_f32(norm_w, "head norm", V);
+  TORCH_CHECK(w_a2.scalar_type() == h.scalar_type() && w_a2.is_contiguous() && w_a2.size(0) >= H * D &&
+                  w_a2.size(1) >= rank && d[8] + w_a2.size(1) <= w.size(0), "bad decay projection");
+  fc::StepParams p;
+  p.H = H;
+  p.D = D;
+  p.V = V;
+  p.runs = run_batch(cu, ctx, slots, state);
+  TORCH_CHECK(p.runs.cu != nullptr || p.runs.B == T, "one row per request expected");
+  p.state = state.data_ptr<float>();
+  p.off_q = int(d[4]);
+  p.off_k = int(d[5]);
+  p.off_v = int(d[6]);
+  p.off_g = int(d[7]);
+  p.off_a1 = int(d[8]);
+  p.z_bias = z_bias.data_ptr<float>();
+  p.inv_tau = float(1.0 / tau);
+  p.q_scale = 1.f / std::sqrt(float(D));
+  p.norm_w = norm_w.data_ptr<float>();
+  p.eps = float(eps);
+  const bool chunk = !is_f32(h) && max_len >= CHUNK_MIN_ROWS && fc::chunk_supported(D, V);
+  Tensor hold, z, out, o_raw;
+  const bool decode = p.runs.cu == nullptr;
+  p.proj = project(h, w, c10::nullopt, decode, hold);
+  if (decode) {
+    p.w_a2 = w_a2.data_ptr();
+    p.ld_a2 = w_a2.size(1);
+    p.rank = rank;
+  } else {
+    project(hold.narrow(1, d[8], w_a2.size(1)), w_a2, c10::nullopt, false, z);
+    p.z = z.data_ptr();
+    p.ld_z = z.size(1);
+  }
+  run_recurrence(p, h, false, chunk, T, int(max_len), out, o_raw);
+  return out;
+}
+
+Tensor delta_rule(const Tensor& h, const Tensor& w, const Tensor& conv_w, const Tensor& a_log, const Tensor& dt_bias,
+                  const Tensor& norm_w, double eps, Tensor conv_state, Tensor state, const std::vector<int64_t>& d,
+                  double unit_eps, const OptTensor& cu, const Tensor& ctx, const Tensor& slots, int64_t max_len,
+                  const OptTensor& row_seq) {
+  TORCH_CHECK(d.size() == 7, "delta rule: seven sizes and offsets");
+  const int H = int(d[0]), K = int(d[1]), D = int(d[2]), V = int(d[3]);
+  const int C = 2 * K * D + H * V, taps = int(conv_w.size(1));
+  c10::cuda::CUDAGuard guard(h.device());
+  const int T = int(h.size(0));
+  check_f32(state, "state", state.size(0) * H * D * V);
+  check_f32(conv_w, "convolution weights", (int64_t)C * taps);
+  check_f32(conv_state, "convolution state", state.size(0) * (taps - 1) * C);
+  check_f32(a_log, "A_log", H);
+  check_f32(dt_bias, "dt_bias", H);
+  check_f32(norm_w, "head norm", V);
+  TORCH_CHECK(H % K == 0, "heads must be a multiple of the q/k heads");
+  const auto f32o = h.options().dtype(torch::kFloat32);
+  Tensor hold, out, o_raw;
+  Tensor qk = torch::empty({T, 2 * K * D}, f32o), v = torch::empty({T, H * V}, h.options());
+  Tensor gates = torch::empty({2, T, H}, f32o);
+  fc::StepParams p;
+  p.H = H;
+  p.group = H / K;
+  p.D = D;
+  p.V = V;
+  p.runs = run_batch(cu, ctx, slots, state);
+  fc::DeltaPrepare q;
+  if (p.runs.cu != nullptr) {
+    TORCH_CHECK(row_seq.has_value() && row_seq->defined(), "runs of several rows need the request of every row");
+    check_i32(*row_seq, "row_seq", T);
+    q.row_seq = row_seq->data_ptr<int>();
+  } else {
+    TORCH_CHECK(p.runs.B == T, "one row per request expected");
+  }
+  p.proj = project(h, w, c10::nullopt, true, hold);
+  q.H = H;
+  q.K = K;
+  q.D = D;
+  q.V = V;
+  q.taps = taps;
+  q.T = T;
+  q.runs = p.runs;
+  q.proj = p.proj;
+  p.off_g = int(d[4]);
+  q.off_b = int(d[5]);
+  q.off_a = int(d[6]);
+  q.conv_w = conv_w.data_ptr<float>();
+  q.conv_state = conv_state.data_ptr<float>();
+  q.a_log = a_log.data_ptr<float>();
+  q.dt_bias = dt_bias.data_ptr<float>();
+  q.unit_eps = float(unit_eps);
+  q.q_scale = 1.f / std::sqrt(float(D));
+  q.qk = qk.data_ptr<float>();
+  q.v = v.data_ptr();
+  q.log_g = gates.data_ptr<float>();
+  q.beta = q.log_g + (long long)T * H;
+  fc::launch_delta_prepare(q, is_f32(h), stream_now());
+  p.qk = q.qk;
+  p.v = q.v;
+  p.log_g = q.log_g;
+  p.beta = q.beta;
+  p.state = state.data_ptr<float>();
+  p.norm_w = norm_w.data_ptr<float>();
+  p.eps = float(eps);
+  const bool chunk = !is_f32(h) && max_len >= CHUNK_MIN_ROWS && fc::chunk_supported(D, V);
+  run_recurrence(p, h, true, chunk, T, int(max_len), out, o_raw);
+  return out;
+}
+
+// Projection, cache store and attention of a latent-attention layer (up to the output projection).
+// d: heads, dim, rot, vdim, rank, rot_dims, offsets of q, kv (-1: none), g
+Tensor latent_attention(const Tensor& h, const Tensor& w, const std::vector<int64_t>& d, double scale, double base,
+                        const OptTensor& kv_norm, double eps, const Tensor& w_kv, int64_t off_uv, const Tensor& w_ukt,
+                        const Tensor& w_uv, Tensor pool, const Tensor& positions, const OptTensor& slots,
+                        const Tensor& block_tables, const Tensor& ctx, const OptTensor& cu_q, const OptTensor& cu_kv,
+                        const OptTensor& row_seq, const OptTensor& row_ctx, int64_t max_q, int64_t max_ctx,
+                        int64_t total_kv, int64_t impl) {
+  TORCH_CHECK(d.size() == 9, "latent attention: nine sizes and offsets");
+  const int H = int(d[0]), D = int(d[1]), R = int(d[2]), V = int(d[3]), rank = int(d[4]), rot_dims = int(d[5]);
+  c10::cuda::CUDAGuard guard(h.device());
+  const int T = int(h.size(0)), B = int(ctx.numel());
+  const bool f32 = is_f32(h);
+  check_elem(pool, "cache rows");
+  TORCH_CHECK(pool.scalar_type() == h.scalar_type() && pool.is_contiguous() && pool.dim() == 3 &&
+                  pool.size(2) >= rank + R && pool.size(2) % 8 == 0, "cache rows must be [blocks, block, row width]");
+  TORCH_CHECK(positions.is_cuda() && positions.scalar_type() == torch::kInt64 && positions.is_contiguous() &&
+                  positions.numel() == T, "positions must be int64 [T]");
+  check_i32(ctx, "context lengths", B);
+  TORCH_CHECK(block_tables.is_cuda() && block_tables.scalar_type() == torch::kInt32 && block_tables.dim() == 2 &&
+                  block_tables.is_contiguous() && block_tables.size(0) >= B, "block_tables must be int32 [B, blocks]");
+  TORCH_CHECK(w_ukt.is_contiguous() && w_ukt.numel() == (int64_t)H * rank * D && w_uv.is_contiguous() &&
+                  w_uv.numel() == (int64_t)H * V * rank && w_ukt.scalar_type() == h.scalar_type() &&
+                  w_uv.scalar_type() == h.scalar_type(), "bad expansion weights");
+  TORCH_CHECK(rot_dims % 2 == 0 && rot_dims <= R, "rotated dimensions must be even and inside the rotated part");
+  const auto& ws = ws_of(h);
+  fc::LatentStore st;
+  st.T = T;
+  st.H = H;
+  st.D = D;
+  st.R = R;
+  st.V = V;
+  st.rank = rank;
+  st.rot_dims = rot_dims;
+  st.off_q = int(d[6]);
+  st.off_kv = int(d[7]);
+  st.off_g = int(d[8]);
+  st.eps = float(eps);
+  st.base = base;
+  st.positions = reinterpret_cast<const long long*>(positions.data_ptr<int64_t>());
+  st.pool = pool.data_ptr();
+  st.row_width = int(pool.size(2));
+  st.num_rows = pool.size(0) * pool.size(1);
+  st.status = ws.status;
+  if (st.off_kv >= 0) {
+    TORCH_CHECK(kv_norm.has_value() && slots.has_value(), "a layer with cache rows needs its norm and the slot map");
+    check_f32(*kv_norm, "latent norm", rank);
+    check_i32(*slots, "slot map", T);
+    st.norm_w = kv_norm->data_ptr<float>();
+    st.slots = slots->data_ptr<int>();
+  }
+  const bool prefill = cu_q.has_value() && cu_q->defined();
+  Tensor out = torch::empty({T, pad8(H * V)}, h.options());
+  if (T == 0) return out;
+  Tensor hold;
+  st.proj = project(h, w, c10::nullopt, true, hold);
+
+  if (prefill && !f32 && impl != 1) {
+    // expanded form: the cache rows of every request become per-head keys and values
+    fc::LatentPrefill a;
+    a.T = T;
+    a.B = B;
+    a.H = H;
+    a.D = D;
+    a.R = R;
+    a.V = V;
+    a.max_q = int(max_q);
+    a.total_kv = total_kv;
+    if (fc::latent_prefill_supported(a)) {
+      check_i32(*cu_q, "cu_q", B + 1);
+      check_i32(*cu_kv, "cu_kv", B + 1);
+      Tensor q = torch::empty({T, H, D + R}, h.options()), gate = torch::empty({T, H * V}, h.options());
+      st.q = q.data_ptr();
+      const bool partial = st.proj.splits > 1;
+      if (partial) st.gate = gate.data_ptr();
+      fc::launch_latent_store(st, false, stream_now());
+      Tensor rows = torch::empty({total_kv, pool.size(2)}, h.options());
+      fc::launch_gather_rows(pool.data_ptr(), block_tables.data_ptr<int>(), ctx.data_ptr<int>(), cu_kv->data_ptr<int>(),
+                             rows.data_ptr(), B, int(max_ctx), int(pool.size(2)), int(pool.size(1)),
+                             int(block_tables.size(1)), int(pool.size(0)), false, ws.status, stream_now());
+      Tensor kv;
+      project(rows.narrow(1, 0, w_kv.size(1)), w_kv, c10::nullopt, false, kv);
+      a.q = q.data_ptr();
+      a.k = kv.data_ptr();
+      a.v = reinterpret_cast<const char*>(kv.data_ptr()) + off_uv * 2;
+      a.ld_kv = kv.size(1);
+      a.rot = reinterpret_cast<const char*>(rows.data_ptr()) + rank * 2;
+      a.ld_rot = rows.size(1);
+      a.cu_q = cu_q->data_ptr<int>();
+      a.cu_kv = cu_kv->data_ptr<int>();
+      if (partial) {
+        a.gate = gate.data_ptr();
+        a.ld_gate = H * V;
+      } else {
+        a.gate = reinterpret_cast<const char*>(st.proj.p) + (long long)st.off_g * 2;
+        a.ld_gate = st.proj.ld;
+      }
+      a.out = out.data_ptr();
+      a.ld_out = out.size(1);
+      a.scale = float(scale);
+      a.status = ws.status;
+      fc::launch_latent_prefill(a, stream_now());
+      return out;
+    }
+  }
+  // absorbed form: queries into the latent space, attention over the rows as they are, outputs out of it
+  Tensor qn = torch::empty({T, H, D}, h.options()), q_abs = torch::empty({T, H, rank + R}, h.options());
+  Tensor gate, o_lat = torch::empty({T, H, rank}, h.options());
+  st.q = qn.data_ptr();
+  st.q_abs = q_abs.data_ptr();
+  fc::launch_latent_store(st, f32, stream_now());
+  fc::SimtLinear a;
+  a.x = qn.data_ptr();
+  a.w = w_ukt.data_ptr();
+  a.y = q_abs.data_ptr();
+  a.M = T;
+  a.N = rank;
+  a.K = D;
+  a.groups = H;
+  a.ldx = (long long)H * D;
+  a.ldw = D;
+  a.ldy = (long long)H * (rank + R);
+  a.gx = D;
+  a.gw = (long long)rank * D;
+  a.gy = rank + R;
+  auto head_linear = [&](const fc::SimtLinear& l) {
+    if (!f32 && impl != 1 && fc::head_linear_mma_supported(l)) fc::launch_head_linear_mma(l, stream_now());
+    else fc::launch_linear_simt(l, f32, stream_now());
+  };
+  head_linear(a);
+  fc::LatentAttn at;
+  at.T = T;
+  at.H = H;
+  at.rank = rank;
+  at.R = R;
+  at.row_width = int(pool.size(2));
+  at.block_size = int(pool.size(1));
+  at.max_blocks = int(block_tables.size(1));
+  at.num_blocks = int(pool.size(0));
+  at.q_abs = q_abs.data_ptr();
+  at.pool = pool.data_ptr();
+  at.block_tables = block_tables.data_ptr<int>();
+  if (prefill) {
+    TORCH_CHECK(row_seq.has_value() && row_ctx.has_value(), "prefill rows need their request and visible rows");
+    check_i32(*row_seq, "row_seq", T);
+    check_i32(*row_ctx, "row_ctx", T);
+    at.row_seq = row_seq->data_ptr<int>();
+    at.row_ctx = row_ctx->data_ptr<int>();
+  } else {
+    TORCH_CHECK(B >= T, "one row per request expected");
+    at.row_ctx = ctx.data_ptr<int>();
+  }
+  at.o_lat = o_lat.data_ptr();
+  at.scale = float(scale);
+  at.status = ws.status;
+  if (!f32 && impl != 1 && fc::latent_decode_supported(at)) {
+    const int64_t mc = max_ctx > 0 ? max_ctx : block_tables.size(1) * pool.size(1);
+    at.splits = fc::latent_decode_splits(at, int(mc), fc::gemm_num_sms());
+    Tensor po, pl;
+    if (at.splits > 1) {
+      po = torch::empty({(int64_t)T * H * at.splits * rank}, h.options().dtype(torch::kFloat32));
+      pl = torch::empty({(int64_t)T * H * at.splits}, h.options().dtype(torch::kFloat32));
+      at.part_o = po.data_ptr<float>();
+      at.part_lse = pl.data_ptr<float>();
+    }
+    fc::launch_latent_decode(at, stream_now());
+  } else {
+    fc::launch_latent_attn_simt(at, f32, stream_now());
+  }
+  a = fc::SimtLinear();
+  a.x = o_lat.data_ptr();
+  a.w = w_uv.data_ptr();
+  a.y = out.data_ptr();
+  a.M = T;
+  a.N = V;
+  a.K = rank;
+  a.groups = H;
+  a.ldx = (long long)H * rank;
+  a.ldw = rank;
+  a.ldy = out.size(1);
+  a.gx = rank;
+  a.gw = (long long)V * rank;
+  a.gy = V;
+  a.gate = st.proj;                    // no product has used the scratch since
+  a.gate_off = st.off_g;
+  a.y_pad = int(out.size(1));
+  head_linear(a);
+  return out;
+}
+
+}  // namespace
+
+void register_hybrid(pybind11::module_& m) {
+  m.def("linear_wide", &linear_wide, "x @ w.T (+ bias), bf16 on tcgen05 or true fp32 on the CUDA cores", py::arg("x"),
+        py::arg("w"), py::arg("bias") = py::none());
+  m.def("embed_scaled", &embed_scaled);
+  m.def("linear_post_norm_add", &linear_post_norm_add);
+  m.def("rms_norm_wide", &rms_norm_wide);
+  m.def("linear_gelu_mul", &linear_gelu_mul);
+  m.def("gla", &gla);
+  m.def("delta_rule", &delta_rule);
+  m.def("latent_attention", &latent_attention);
+}

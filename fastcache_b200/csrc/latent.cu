@@ -1,0 +1,219 @@
+// Latent attention around the cache: norm of the latent, rotation of the shared key part and of the queries, store of
+// the cache rows, gather of a request's rows for the expanded form, and the general (any size, fp32 or bf16) form of
+// absorbed attention over the paged rows.
+#include <algorithm>
+#include <stdexcept>
+#include <string>
+
+#include "hybrid.cuh"
+#include "launch.h"
+
+namespace fc {
+
+using bf16 = __nv_bfloat16;
+constexpr int LS_THREADS = 256;
+
+// cos and sin of position * base^(-2 i / dims): the angle is reduced in double, so that far positions lose nothing
+__device__ __forceinline__ void rope_angle(double pos, double log2_base, int i, int dims, float& c, float& s) {
+  const double turns = pos * exp2(-log2_base * (2.0 * i / dims)) * 0.15915494309189535;   // 1 / (2 pi)
+  sincospif(float(2.0 * (turns - rint(turns))), &s, &c);
+}
+
+template <typename T>
+__global__ void __launch_bounds__(LS_THREADS)
+latent_store_kernel(const LatentStore p) {
+  __shared__ float red[LS_THREADS / 32];
+  extern __shared__ float cs[];                   // cos | sin of this token, rot_dims / 2 each
+  const int half = p.rot_dims / 2;
+  pdl_launch_dependents();
+  pdl_wait();
+  const long long t = blockIdx.x;
+  const double pos = double(p.positions[t]);
+  const double l2b = log2(p.base);
+  for (int i = threadIdx.x; i < half; i += LS_THREADS) rope_angle(pos, l2b, i, p.rot_dims, cs[i], cs[half + i]);
+  __syncthreads();
+  const int part = blockIdx.y, parts = gridDim.y;
+  // queries: every (head, column) of this part
+  const int Q = p.D + p.R;
+  T* q_abs = reinterpret_cast<T*>(p.q_abs);
+  T* q = reinterpret_cast<T*>(p.q);
+  const int qw = q_abs != nullptr ? p.D : Q;
+  for (int idx = part * LS_THREADS + threadIdx.x; idx < p.H * Q; idx += parts * LS_THREADS) {
+    const int h = idx / Q, c = idx - h * Q;
+    float v = proj_at<T>(p.proj, t, p.off_q + idx);
+    const int r = c - p.D;
+    if (r >= 0 && r < p.rot_dims) {
+      const bool first = r < half;
+      const int i = first ? r : r - half;
+      const float o = proj_at<T>(p.proj, t, p.off_q + idx + (first ? half : -half));
+      v = first ? v * cs[i] - o * cs[half + i] : v * cs[i] + o * cs[half + i];
+    }
+    if (r < 0 || q_abs == nullptr) q[(t * p.H + h) * qw + c] = Elem<T>::put(v);
+    else q_abs[(t * p.H + h) * (p.rank + p.R) + p.rank + r] = Elem<T>::put(v);
+  }
+  if (p.gate != nullptr) {
+    T* gate = reinterpret_cast<T*>(p.gate);
+    for (int c = part * LS_THREADS + threadIdx.x; c < p.H * p.V; c += parts * LS_THREADS)
+      gate[t * p.H * p.V + c] = Elem<T>::put(proj_at<T>(p.proj, t, p.off_g + c));
+  }
+  if (p.off_kv < 0 || part != 0) return;
+  // cache row: normed latent | rotated shared key part
+  const int slot = p.slots[t];
+  if (slot < 0) return;
+  if (slot >= p.num_rows) {
+    if (threadIdx.x == 0) report(p.status, ST_BAD_INDEX);
+    return;
+  }
+  T* row = reinterpret_cast<T*>(p.pool) + (long long)slot * p.row_width;
+  float ss = 0.f;
+  for (int c = threadIdx.x; c < p.rank; c += LS_THREADS) {
+    const float v = proj_at<T>(p.proj, t, p.off_kv + c);
+    ss += v * v;
+  }
+  const float inv = rsqrtf(cta_sum<LS_THREADS>(ss, red) / float(p.rank) + p.eps);
+  for (int c = threadIdx.x; c < p.rank; c += LS_THREADS)
+    row[c] = Elem<T>::put(proj_at<T>(p.proj, t, p.off_kv + c) * inv * p.norm_w[c]);
+  for (int r = threadIdx.x; r < p.R; r += LS_THREADS) {
+    const int col = p.off_kv + p.rank + r;
+    float v = proj_at<T>(p.proj, t, col);
+    if (r < p.rot_dims) {
+      const bool first = r < half;
+      const int i = first ? r : r - half;
+      const float o = proj_at<T>(p.proj, t, col + (first ? half : -half));
+      v = first ? v * cs[i] - o * cs[half + i] : v * cs[i] + o * cs[half + i];
+    }
+    row[p.rank + r] = Elem<T>::put(v);
+  }
+}
+
+void launch_latent_store(const LatentStore& p, bool f32, cudaStream_t s) {
+  if (p.T == 0) return;
+  const int work = p.H * (p.D + p.R);
+  const int parts = p.T >= 592 ? 1 : std::max(1, std::min(16, (work + LS_THREADS * 4 - 1) / (LS_THREADS * 4)));
+  const dim3 grid(p.T, parts);
+  const size_t smem = size_t(std::max(2, p.rot_dims)) * 4;
+  if (f32) launch_pdl(PDL_ROPE, latent_store_kernel<float>, grid, dim3(LS_THREADS), smem, s, p);
+  else launch_pdl(PDL_ROPE, latent_store_kernel<bf16>, grid, dim3(LS_THREADS), smem, s, p);
+  const cudaError_t e = cudaGetLastError();
+  if (e != cudaSuccess) throw std::runtime_error(std::string("latent store: ") + cudaGetErrorString(e));
+}
+
+// ------------------------------------------------------------------ gather
+// rows [0, ctx[b]) of every request, one after another (cu_kv), 16 bytes per thread
+template <int BYTES>
+__global__ void __launch_bounds__(256)
+gather_rows_kernel(const uint8_t* __restrict__ pool, const int* __restrict__ block_tables, const int* __restrict__ ctx,
+                   const int* __restrict__ cu_kv, uint8_t* __restrict__ out, int chunks, int block_size,
+                   int max_blocks, int num_blocks, uint32_t* status) {
+  const int b = blockIdx.y;
+  const int n = ctx[b];
+  const int per = 256 / chunks > 0 ? 256 / chunks : 1;
+  const int row0 = blockIdx.x * per;
+  for (int i = threadIdx.x; i < per * chunks; i += 256) {
+    const int row = row0 + i / chunks, c = i % chunks;
+    if (row >= n) return;
+    const int blk = block_tables[(long long)b * max_blocks + row / block_size];
+    if (blk < 0 || blk >= num_blocks) {
+      report(status, ST_BAD_INDEX);
+      continue;
+    }
+    const long long src = (long long)blk * block_size + row % block_size;
+    reinterpret_cast<uint4*>(out)[((long long)cu_kv[b] + row) * chunks + c] =
+        reinterpret_cast<const uint4*>(pool)[src * chunks + c];
+  }
+}
+
+void launch_gather_rows(const void* pool, const int* block_tables, const int* ctx, const int* cu_kv, void* out,
+                        int B, int max_ctx, int row_width, int block_size, int max_blocks, int num_blocks, bool f32,
+                        uint32_t* status, cudaStream_t s) {
+  if (B == 0 || max_ctx == 0) return;
+  const int chunks = row_width * (f32 ? 4 : 2) / 16;
+  const int per = std::max(1, 256 / chunks);
+  gather_rows_kernel<16><<<dim3((max_ctx + per - 1) / per, B), 256, 0, s>>>(
+      (const uint8_t*)pool, block_tables, ctx, cu_kv, (uint8_t*)out, chunks, block_size, max_blocks, num_blocks, status);
+  const cudaError_t e = cudaGetLastError();
+  if (e != cudaSuccess) throw std::runtime_error(std::string("gather rows: ") + cudaGetErrorString(e));
+}
+
+// ------------------------------------------------------------------ absorbed attention, general form
+constexpr int LA_THREADS = 128;
+constexpr int LA_TILE = 64;
+constexpr int LA_COLS = 8;           // latent columns per thread: rank <= 1024
+
+template <typename T>
+__global__ void __launch_bounds__(LA_THREADS)
+latent_attn_simt_kernel(const LatentAttn p) {
+  extern __shared__ float sq[];                    // rank + R query values
+  __shared__ float ss[LA_TILE];
+  __shared__ const T* srow[LA_TILE];
+  const int t = blockIdx.x, h = blockIdx.y;
+  const int w = p.rank + p.R;
+  const int ctx = p.row_ctx[t];
+  const int b = p.row_seq != nullptr ? p.row_seq[t] : t;
+  const T* q = reinterpret_cast<const T*>(p.q_abs) + ((long long)t * p.H + h) * w;
+  const T* pool = reinterpret_cast<const T*>(p.pool);
+  const int* bt = p.block_tables + (long long)b * p.max_blocks;
+  for (int c = threadIdx.x; c < w; c += LA_THREADS) sq[c] = ctx > 0 ? Elem<T>::get(q[c]) * p.scale : 0.f;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  float acc[LA_COLS];
+#pragma unroll
+  for (int i = 0; i < LA_COLS; ++i) acc[i] = 0.f;
+  float m = -INFINITY, l = 0.f;
+  for (int k0 = 0; k0 < ctx; k0 += LA_TILE) {
+    const int n = min(LA_TILE, ctx - k0);
+    __syncthreads();
+    if (threadIdx.x < n) {
+      const int j = k0 + threadIdx.x;
+      int blk = bt[j / p.block_size];
+      if (blk < 0 || blk >= p.num_blocks) {
+        report(p.status, ST_BAD_INDEX);
+        blk = 0;
+      }
+      srow[threadIdx.x] = pool + ((long long)blk * p.block_size + j % p.block_size) * p.row_width;
+    }
+    __syncthreads();
+    for (int j = warp; j < n; j += LA_THREADS / 32) {
+      float d = 0.f;
+      for (int c = lane; c < w; c += 32) d = fmaf(sq[c], Elem<T>::get(srow[j][c]), d);
+      d = warp_sum(d);
+      if (lane == 0) ss[j] = d;
+    }
+    __syncthreads();
+    float mx = m;
+    for (int j = 0; j < n; ++j) mx = fmaxf(mx, ss[j]);
+    const float corr = expf(m - mx);
+    m = mx;
+    l *= corr;
+#pragma unroll
+    for (int i = 0; i < LA_COLS; ++i) acc[i] *= corr;
+    for (int j = 0; j < n; ++j) {
+      const float e = expf(ss[j] - mx);
+      l += e;
+#pragma unroll
+      for (int i = 0; i < LA_COLS; ++i) {
+        const int c = threadIdx.x + i * LA_THREADS;
+        if (c < p.rank) acc[i] = fmaf(e, Elem<T>::get(srow[j][c]), acc[i]);
+      }
+    }
+  }
+  const float inv = l > 0.f ? 1.f / l : 0.f;
+  T* o = reinterpret_cast<T*>(p.o_lat) + ((long long)t * p.H + h) * p.rank;
+#pragma unroll
+  for (int i = 0; i < LA_COLS; ++i) {
+    const int c = threadIdx.x + i * LA_THREADS;
+    if (c < p.rank) o[c] = Elem<T>::put(acc[i] * inv);
+  }
+}
+
+void launch_latent_attn_simt(const LatentAttn& p, bool f32, cudaStream_t s) {
+  if (p.T == 0) return;
+  if (p.rank > LA_THREADS * LA_COLS) throw std::runtime_error("latent attention: kv_rank is limited to 1024");
+  const dim3 grid(p.T, p.H);
+  const size_t smem = size_t(p.rank + p.R) * 4;
+  if (f32) latent_attn_simt_kernel<float><<<grid, LA_THREADS, smem, s>>>(p);
+  else latent_attn_simt_kernel<bf16><<<grid, LA_THREADS, smem, s>>>(p);
+  const cudaError_t e = cudaGetLastError();
+  if (e != cudaSuccess) throw std::runtime_error(std::string("latent attention: ") + cudaGetErrorString(e));
+}
+
+}  // namespace fc

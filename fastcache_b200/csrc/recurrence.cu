@@ -1,0 +1,422 @@
+// Recurrent layers, token by token: gated linear attention and the gated delta rule with the state in registers.
+//
+// One CTA owns (request, head, block of value columns): its part of the fp32 state [D, V] is read from the request's
+// slot once, advanced over the rows of the request's run and written back.  A decode step is a run of one row; it is
+// bound by reading and writing the states (each exactly once).  Threads form CG column groups of four value columns x
+// 256 / CG row groups; sums over the key dimension go through warp shuffles and one exchange in shared memory per
+// token.  Also here: what surrounds the recurrence (short convolutions, unit norms, gates, head norm).
+#include <algorithm>
+#include <stdexcept>
+#include <string>
+
+#include "hybrid.cuh"
+#include "launch.h"
+
+namespace fc {
+
+using bf16 = __nv_bfloat16;
+constexpr int ST_THREADS = 256;
+constexpr int ST_WARPS = ST_THREADS / 32;
+constexpr int ST_MAX_D = 1024;
+
+template <typename T, bool DELTA, int CG, int R>
+__global__ void __launch_bounds__(ST_THREADS)
+step_kernel(const StepParams p) {
+  constexpr int RG = ST_THREADS / CG;
+  constexpr int VB = CG * 4;
+  constexpr int NV = DELTA ? 2 * VB + 1 : VB;               // values exchanged per warp and token
+  constexpr int NL = (RG * R + ST_THREADS - 1) / ST_THREADS; // staged entries per thread
+  extern __shared__ float sm[];
+  const int D = p.D;
+  float* s_q = sm;                                           // [3][D]
+  float* s_k = sm + 3 * D;
+  float* s_a = sm + 6 * D;                                   // decay per key channel (GLA)
+  float* red = sm + 9 * D;                                   // [2][ST_WARPS][NV]
+  pdl_launch_dependents();
+  pdl_wait();
+  const int vb = blockIdx.x, h = blockIdx.y, b = blockIdx.z;
+  const Run run = get_run(p.runs, b);
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int cl = tid % CG, rg = tid / CG;
+  const int col = vb * VB + cl * 4;
+  T* out = reinterpret_cast<T*>(p.out);
+  const bool vec = (p.V & 3) == 0;
+  if (run.slot < 0) {                                        // padding row of a captured batch
+    if (rg == 0)
+      for (int t = run.lo; t < run.lo + run.len; ++t)
+        for (int j = 0; j < 4; ++j)
+          if (col + j < p.V) {
+            if (out != nullptr) out[t * p.ld_out + h * p.V + col + j] = Elem<T>::put(0.f);
+            else p.o_raw[((long long)t * p.H + h) * p.V + col + j] = 0.f;
+          }
+    return;
+  }
+  float* st = p.state + ((long long)run.slot * p.H + h) * D * p.V;
+  float S[R][4];
+#pragma unroll
+  for (int i = 0; i < R; ++i) {
+    const int r = rg + i * RG;
+    S[i][0] = S[i][1] = S[i][2] = S[i][3] = 0.f;
+    if (run.start > 0 && r < D) {
+      const float* src = st + (long long)r * p.V + col;
+      if (vec && col < p.V) {
+        const float4 v = *reinterpret_cast<const float4*>(src);
+        S[i][0] = v.x; S[i][1] = v.y; S[i][2] = v.z; S[i][3] = v.w;
+      } else {
+#pragma unroll
+        for (int j = 0; j < 4; ++j)
+          if (col + j < p.V) S[i][j] = src[j];
+      }
+    }
+  }
+  const int hk = h / p.group, K = p.H / p.group;
+  float pq[NL], pk[NL], pa[NL];
+  auto fetch = [&](int t) {
+#pragma unroll
+    for (int i = 0; i < NL; ++i) {
+      const int r = tid + i * ST_THREADS;
+      if (r >= D) continue;
+      if (DELTA) {
+        const float* row = p.qk + ((long long)t * 2 * K + hk) * D + r;
+        pq[i] = __ldcg(row);
+        pk[i] = __ldcg(row + (long long)K * D);
+      } else {
+        pq[i] = proj_at<T>(p.proj, t, p.off_q + h * D + r) * p.q_scale;
+        pk[i] = proj_at<T>(p.proj, t, p.off_k + h * D + r);
+        float z = p.z_bias[h * D + r];
+        if (p.z != nullptr) {
+          z += Elem<T>::get(reinterpret_cast<const T*>(p.z)[(long long)t * p.ld_z + h * D + r]);
+        } else {
+          const T* w = reinterpret_cast<const T*>(p.w_a2) + (long long)(h * D + r) * p.ld_a2;
+          for (int j = 0; j < p.rank; ++j) z = fmaf(proj_at<T>(p.proj, t, p.off_a1 + j), Elem<T>::get(w[j]), z);
+        }
+        pa[i] = expf(log_sigmoid_f(z) * p.inv_tau);
+      }
+    }
+  };
+  auto put = [&](int buf) {
+#pragma unroll
+    for (int i = 0; i < NL; ++i) {
+      const int r = tid + i * ST_THREADS;
+      if (r >= D) continue;
+      s_q[buf * D + r] = pq[i];
+      s_k[buf * D + r] = pk[i];
+      if (!DELTA) s_a[buf * D + r] = pa[i];
+    }
+  };
+  const int t1 = run.lo + run.len;
+  if (run.len > 0) {
+    fetch(run.lo);
+    put(0);
+  }
+  __syncthreads();
+  for (int t = run.lo, n = 0; t < t1; ++t, ++n) {
+    const int buf = n % 3;
+    if (t + 1 < t1) fetch(t + 1);
+    float v[4] = {0.f, 0.f, 0.f, 0.f};
+    float g = 0.f, beta = 0.f;
+    if (DELTA) {
+      const T* vr = reinterpret_cast<const T*>(p.v) + ((long long)t * p.H + h) * p.V + col;
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+        if (col + j < p.V) v[j] = Elem<T>::get(vr[j]);
+      g = expf(__ldcg(p.log_g + (long long)t * p.H + h));
+      beta = __ldcg(p.beta + (long long)t * p.H + h);
+    } else {
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+        if (col + j < p.V) v[j] = proj_at<T>(p.proj, t, p.off_v + h * p.V + col + j);
+    }
+    const float *q_s = s_q + buf * D, *k_s = s_k + buf * D, *a_s = s_a + buf * D;
+    float oq[4] = {0.f, 0.f, 0.f, 0.f}, ok[4] = {0.f, 0.f, 0.f, 0.f}, kq = 0.f;
+#pragma unroll
+    for (int i = 0; i < R; ++i) {
+      const int r = rg + i * RG;
+      if (r >= D) continue;
+      const float qv = q_s[r], kv = k_s[r];
+      const float a = DELTA ? g : a_s[r];
+      if (DELTA) kq = fmaf(qv, kv, kq);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        S[i][j] = DELTA ? S[i][j] * a : fmaf(S[i][j], a, kv * v[j]);
+        oq[j] = fmaf(qv, S[i][j], oq[j]);
+        if (DELTA) ok[j] = fmaf(kv, S[i][j], ok[j]);
+      }
+    }
+#pragma unroll
+    for (int o = CG; o < 32; o <<= 1) {
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        oq[j] += __shfl_xor_sync(0xffffffffu, oq[j], o);
+        if (DELTA) ok[j] += __shfl_xor_sync(0xffffffffu, ok[j], o);
+      }
+      if (DELTA) kq += __shfl_xor_sync(0xffffffffu, kq, o);
+    }
+    float* rd = red + (n & 1) * ST_WARPS * NV;
+    if (lane < CG) {
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        rd[warp * NV + cl * 4 + j] = oq[j];
+        if (DELTA) rd[warp * NV + VB + cl * 4 + j] = ok[j];
+      }
+      if (DELTA && cl == 0) rd[warp * NV + 2 * VB] = kq;
+    }
+    if (t + 1 < t1) put((n + 1) % 3);
+    __syncthreads();
+    float o[4] = {0.f, 0.f, 0.f, 0.f};
+    if (DELTA) {
+      float s[4] = {0.f, 0.f, 0.f, 0.f};
+      kq = 0.f;
+#pragma unroll
+      for (int w = 0; w < ST_WARPS; ++w) {
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          o[j] += rd[w * NV + cl * 4 + j];
+          s[j] += rd[w * NV + VB + cl * 4 + j];
+        }
+        kq += rd[w * NV + 2 * VB];
+      }
+      float u[4];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        u[j] = beta * (v[j] - s[j]);
+        o[j] = fmaf(kq, u[j], o[j]);                        // S^T q after the write: (g S)^T q + (k . q) u
+      }
+#pragma unroll
+      for (int i = 0; i < R; ++i) {
+        const int r = rg + i * RG;
+        if (r >= D) continue;
+        const float kv = k_s[r];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) S[i][j] = fmaf(kv, u[j], S[i][j]);
+      }
+    } else if (warp == 0) {
+#pragma unroll
+      for (int w = 0; w < ST_WARPS; ++w)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) o[j] += rd[w * NV + cl * 4 + j];
+    }
+    if (warp == 0) {
+      if (out == nullptr) {
+        if (rg == 0) {
+          float* dst = p.o_raw + ((long long)t * p.H + h) * p.V + col;
+#pragma unroll
+          for (int j = 0; j < 4; ++j)
+            if (col + j < p.V) dst[j] = o[j];
+        }
+      } else {                                              // this CTA holds the whole head: norm and gate here
+        float sq = 0.f;
+#pragma unroll
+        for (int j = 0; j < 4; ++j) sq += col + j < p.V ? o[j] * o[j] : 0.f;
+#pragma unroll
+        for (int x = 1; x < CG; x <<= 1) sq += __shfl_xor_sync(0xffffffffu, sq, x);
+        const float inv = rsqrtf(sq / float(p.V) + p.eps);
+        if (rg == 0) {
+          T* dst = out + t * p.ld_out + h * p.V + col;
+#pragma unroll
+          for (int j = 0; j < 4; ++j)
+            if (col + j < p.V)
+              dst[j] = Elem<T>::put(o[j] * inv * p.norm_w[col + j] *
+                                    silu_f(proj_at<T>(p.proj, t, p.off_g + h * p.V + col + j)));
+        }
+        if (h == 0 && lane < int(p.ld_out) - p.H * p.V) out[t * p.ld_out + p.H * p.V + lane] = Elem<T>::put(0.f);
+      }
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < R; ++i) {
+    const int r = rg + i * RG;
+    if (r >= D || run.len <= 0) continue;
+    float* dst = st + (long long)r * p.V + col;
+    if (vec && col < p.V) {
+      *reinterpret_cast<float4*>(dst) = make_float4(S[i][0], S[i][1], S[i][2], S[i][3]);
+    } else {
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+        if (col + j < p.V) dst[j] = S[i][j];
+    }
+  }
+}
+
+// column groups of the state tile: as wide as the head where the rows then fit the registers
+static int step_col_groups(int D, int V) {
+  int cg = V <= 32 ? 8 : V <= 64 ? 16 : 32;
+  while (cg > 8 && D > 32 * (ST_THREADS / cg)) cg >>= 1;
+  return cg;
+}
+bool step_fuses_norm(int D, int V) { return V <= step_col_groups(D, V) * 4; }
+
+template <typename T, bool DELTA>
+static void launch_step(const StepParams& p, cudaStream_t s) {
+  if (p.runs.B == 0) return;
+  if (p.D > ST_MAX_D) throw std::runtime_error("recurrent layers: the key dimension is limited to 1024");
+  const int cg = step_col_groups(p.D, p.V);
+  const int vb = cg * 4, rows = (p.D + ST_THREADS / cg - 1) / (ST_THREADS / cg);
+  const dim3 grid((p.V + vb - 1) / vb, p.H, p.runs.B);
+  const size_t smem = (size_t(9) * p.D + 2 * ST_WARPS * (DELTA ? 2 * vb + 1 : vb)) * 4;
+  auto go = [&](auto kern) {
+    if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem));
+    launch_pdl(PDL_PARTIALS, kern, grid, dim3(ST_THREADS), smem, s, p);
+  };
+  auto pick = [&](auto c) {
+    constexpr int CG = decltype(c)::value;
+    if (rows <= 4) go(step_kernel<T, DELTA, CG, 4>);
+    else if (rows <= 16) go(step_kernel<T, DELTA, CG, 16>);
+    else go(step_kernel<T, DELTA, CG, 32>);
+  };
+  if (cg == 8) pick(std::integral_constant<int, 8>{});
+  else if (cg == 16) pick(std::integral_constant<int, 16>{});
+  else pick(std::integral_constant<int, 32>{});
+  const cudaError_t e = cudaGetLastError();
+  if (e != cudaSuccess) throw std::runtime_error(std::string("recurrent step: ") + cudaGetErrorString(e));
+}
+void launch_gla_step(const StepParams& p, bool f32, cudaStream_t s) {
+  if (f32) launch_step<float, false>(p, s);
+  else launch_step<bf16, false>(p, s);
+}
+void launch_delta_step(const StepParams& p, bool f32, cudaStream_t s) {
+  if (f32) launch_step<float, true>(p, s);
+  else launch_step<bf16, true>(p, s);
+}
+
+// ------------------------------------------------------------------ head norm and gate
+// one warp per (row, head)
+template <typename T>
+__global__ void __launch_bounds__(256)
+gated_head_norm_kernel(const float* __restrict__ o_raw, const ProjSrc proj, int off_g, const float* __restrict__ norm_w,
+                       float eps, T* __restrict__ out, long long ld_out, long long units, int H, int V) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const long long u = blockIdx.x * 8ll + (threadIdx.x >> 5);
+  if (u >= units) return;
+  const int lane = threadIdx.x & 31;
+  const long long t = u / H;
+  const int h = int(u - t * H);
+  const float* o = o_raw + u * V;
+  float ss = 0.f;
+  for (int c = lane; c < V; c += 32) ss += o[c] * o[c];
+  const float inv = rsqrtf(warp_sum(ss) / float(V) + eps);
+  for (int c = lane; c < V; c += 32)
+    out[t * ld_out + h * V + c] = Elem<T>::put(o[c] * inv * norm_w[c] * silu_f(proj_at<T>(proj, t, off_g + h * V + c)));
+  if (h == 0 && lane < int(ld_out) - H * V) out[t * ld_out + H * V + lane] = Elem<T>::put(0.f);
+}
+void launch_gated_head_norm(const float* o_raw, const ProjSrc& proj, int off_g, const float* norm_w, float eps,
+                            void* out, long long ld_out, int T, int H, int V, bool f32, cudaStream_t s) {
+  const long long units = (long long)T * H;
+  if (units == 0) return;
+  const dim3 grid((unsigned)((units + 7) / 8));
+  if (f32)
+    launch_pdl(PDL_NORM, gated_head_norm_kernel<float>, grid, dim3(256), 0, s, o_raw, proj, off_g, norm_w, eps,
+               (float*)out, ld_out, units, H, V);
+  else
+    launch_pdl(PDL_NORM, gated_head_norm_kernel<bf16>, grid, dim3(256), 0, s, o_raw, proj, off_g, norm_w, eps,
+               (bf16*)out, ld_out, units, H, V);
+  const cudaError_t e = cudaGetLastError();
+  if (e != cudaSuccess) throw std::runtime_error(std::string("head norm: ") + cudaGetErrorString(e));
+}
+
+// ------------------------------------------------------------------ inputs of the delta rule
+// One warp per unit: a q or k head (convolution, silu, unit norm), 128 value channels (convolution, silu) or the
+// decays and step sizes of a row.  A run of one row (decode) also moves the kept inputs of its channels on; for longer
+// runs conv_state_kernel does that afterwards, when every row has read them.
+constexpr int DP_REGS = ST_MAX_D / 32;
+template <typename T>
+__global__ void __launch_bounds__(256)
+delta_prepare_kernel(const DeltaPrepare p, int units, int advance) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.x, u = blockIdx.y * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (u >= units) return;
+  const int b = p.row_seq != nullptr ? p.row_seq[t] : t;
+  const Run run = get_run(p.runs, b);
+  if (run.slot < 0) return;
+  const int i = t - run.lo, C = 2 * p.K * p.D + p.H * p.V;
+  if (u == units - 1) {
+    for (int h = lane; h < p.H; h += 32) {
+      p.log_g[(long long)t * p.H + h] = -expf(p.a_log[h]) * softplus_f(proj_at<T>(p.proj, t, p.off_a + h) + p.dt_bias[h]);
+      p.beta[(long long)t * p.H + h] = sigmoid_f(proj_at<T>(p.proj, t, p.off_b + h));
+    }
+    return;
+  }
+  float* cst = p.conv_state + (long long)run.slot * (p.taps - 1) * C;
+  auto conv = [&](int c) {
+    const float x0 = proj_at<T>(p.proj, t, c);
+    float y = x0 * p.conv_w[(long long)c * p.taps + p.taps - 1];
+    for (int j = 1; j < p.taps; ++j) {                       // the input j rows back
+      float x;
+      if (i - j >= 0) x = proj_at<T>(p.proj, t - j, c);
+      else if (run.start + i - j >= 0) x = cst[(long long)(p.taps - 1 + i - j) * C + c];
+      else x = 0.f;
+      y = fmaf(x, p.conv_w[(long long)c * p.taps + p.taps - 1 - j], y);
+    }
+    if (advance) {
+      for (int j = 0; j < p.taps - 2; ++j)
+        cst[(long long)j * C + c] = run.start > 0 ? cst[(long long)(j + 1) * C + c] : 0.f;
+      if (p.taps > 1) cst[(long long)(p.taps - 2) * C + c] = x0;
+    }
+    return silu_f(y);
+  };
+  if (u < 2 * p.K) {
+    const int which = u / p.K, hk = u - which * p.K;
+    float v[DP_REGS];
+    float ss = 0.f;
+    const int n = (p.D + 31) / 32;
+#pragma unroll
+    for (int x = 0; x < DP_REGS; ++x) {
+      if (x >= n) break;
+      const int d = lane + x * 32;
+      v[x] = d < p.D ? conv(u * p.D + d) : 0.f;
+      ss += v[x] * v[x];
+    }
+    const float inv = rsqrtf(warp_sum(ss) + p.unit_eps) * (which == 0 ? p.q_scale : 1.f);
+    float* dst = p.qk + (((long long)t * 2 + which) * p.K + hk) * p.D;
+#pragma unroll
+    for (int x = 0; x < DP_REGS; ++x) {
+      if (x >= n) break;
+      const int d = lane + x * 32;
+      if (d < p.D) dst[d] = v[x] * inv;
+    }
+    return;
+  }
+  const int c0 = (u - 2 * p.K) * 128, HV = p.H * p.V;
+  T* dst = reinterpret_cast<T*>(p.v) + (long long)t * HV;
+  for (int c = c0 + lane; c < min(c0 + 128, HV); c += 32) dst[c] = Elem<T>::put(conv(2 * p.K * p.D + c));
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256)
+conv_state_kernel(const DeltaPrepare p) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const Run run = get_run(p.runs, blockIdx.y);
+  const int C = 2 * p.K * p.D + p.H * p.V, c = blockIdx.x * 256 + threadIdx.x;
+  if (run.slot < 0 || run.len <= 0 || c >= C) return;
+  float* cst = p.conv_state + (long long)run.slot * (p.taps - 1) * C;
+  for (int j = 0; j < p.taps - 1; ++j) {                     // ascending: an old entry moves towards the front
+    const int i = run.len - (p.taps - 1) + j;
+    float x = 0.f;
+    if (i >= 0) x = proj_at<T>(p.proj, run.lo + i, c);
+    else if (run.start + i >= 0) x = cst[(long long)(j + run.len) * C + c];
+    cst[(long long)j * C + c] = x;
+  }
+}
+
+template <typename T>
+static void delta_prepare_t(const DeltaPrepare& p, cudaStream_t s) {
+  const int units = 2 * p.K + (p.H * p.V + 127) / 128 + 1;
+  const int advance = p.runs.cu == nullptr ? 1 : 0;
+  launch_pdl(PDL_PARTIALS, delta_prepare_kernel<T>, dim3(p.T, (units + 7) / 8), dim3(256), 0, s, p, units, advance);
+  if (!advance && p.taps > 1)
+    launch_pdl(PDL_PARTIALS, conv_state_kernel<T>, dim3((2 * p.K * p.D + p.H * p.V + 255) / 256, p.runs.B), dim3(256),
+               0, s, p);
+}
+void launch_delta_prepare(const DeltaPrepare& p, bool f32, cudaStream_t s) {
+  if (p.T == 0) return;
+  if (p.D > ST_MAX_D) throw std::runtime_error("recurrent layers: the key dimension is limited to 1024");
+  if (f32) delta_prepare_t<float>(p, s);
+  else delta_prepare_t<bf16>(p, s);
+  const cudaError_t e = cudaGetLastError();
+  if (e != cudaSuccess) throw std::runtime_error(std::string("delta rule inputs: ") + cudaGetErrorString(e));
+}
+
+}  // namespace fc

@@ -1,0 +1,200 @@
+// fp32 residual stream of models that norm a sublayer's output before adding it: embedding with a scale, norm + add,
+// final norm, and the gelu gate of the feed-forward.  Readers of a projection take split-K partial sums as they are.
+#include <algorithm>
+#include <stdexcept>
+#include <string>
+
+#include "hybrid.cuh"
+#include "launch.h"
+
+namespace fc {
+
+using bf16 = __nv_bfloat16;
+constexpr int RS_THREADS = 256;
+constexpr int RS_CHUNKS = 8;        // 4-column chunks per thread: rows up to 8192 columns
+
+template <typename T>
+__global__ void __launch_bounds__(RS_THREADS)
+embed_scaled_kernel(const long long* __restrict__ ids, const T* __restrict__ weight, float* __restrict__ x,
+                    T* __restrict__ h, int W, int Wp, long long V, float scale, uint32_t* status) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const long long row = blockIdx.x;
+  long long id = ids[row];
+  const bool ok = id >= 0 && id < V;
+  if (!ok) {
+    if (threadIdx.x == 0) report(status, ST_BAD_INDEX);
+    id = 0;
+  }
+  for (int c = threadIdx.x; c < Wp; c += RS_THREADS) {
+    const float v = (c < W && ok) ? Elem<T>::get(weight[id * Wp + c]) * scale : 0.f;
+    if (c < W) x[row * W + c] = v;
+    h[row * Wp + c] = Elem<T>::put(v);
+  }
+}
+
+// x += rms(y + bias) * w;  h = x in the model's type, zero-padded from W to Wp columns
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(RS_THREADS)
+post_norm_add_kernel(const ProjSrc y, const T* __restrict__ bias, float* __restrict__ x, const float* __restrict__ w,
+                     T* __restrict__ h, int W, int Wp, float eps) {
+  __shared__ float red[RS_THREADS / 32];
+  pdl_launch_dependents();
+  pdl_wait();
+  const long long row = blockIdx.x;
+  float v[RS_CHUNKS][4];
+  float ss = 0.f;
+#pragma unroll
+  for (int c = 0; c < RS_CHUNKS; ++c) {
+    const int col = (threadIdx.x + c * RS_THREADS) * 4;
+    if (col >= W) continue;
+    const float4 a = proj_at4<T>(y, row, col);           // the pad columns of a projection exist and are zero
+    v[c][0] = a.x;
+    v[c][1] = a.y;
+    v[c][2] = a.z;
+    v[c][3] = a.w;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      if (bias != nullptr) v[c][i] += Elem<T>::get(bias[col + i]);
+      if (!VEC && col + i >= W) v[c][i] = 0.f;
+      ss += v[c][i] * v[c][i];
+    }
+  }
+  const float inv = rsqrtf(cta_sum<RS_THREADS>(ss, red) / float(W) + eps);
+#pragma unroll
+  for (int c = 0; c < RS_CHUNKS; ++c) {
+    const int col = (threadIdx.x + c * RS_THREADS) * 4;
+    if (col >= W) continue;
+    float* xr = x + row * W + col;
+    if (VEC) {
+      float4 xv = *reinterpret_cast<const float4*>(xr);
+      const float4 wv = *reinterpret_cast<const float4*>(w + col);
+      xv.x += v[c][0] * inv * wv.x;
+      xv.y += v[c][1] * inv * wv.y;
+      xv.z += v[c][2] * inv * wv.z;
+      xv.w += v[c][3] * inv * wv.w;
+      *reinterpret_cast<float4*>(xr) = xv;
+      store4(h + row * Wp + col, xv.x, xv.y, xv.z, xv.w);
+    } else {
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        if (col + i >= W) break;
+        const float n = xr[i] + v[c][i] * inv * w[col + i];
+        xr[i] = n;
+        h[row * Wp + col + i] = Elem<T>::put(n);
+      }
+    }
+  }
+  for (int c = W + threadIdx.x; c < Wp; c += RS_THREADS) h[row * Wp + c] = Elem<T>::put(0.f);
+}
+
+template <typename T>
+__global__ void __launch_bounds__(RS_THREADS)
+rms_norm_wide_kernel(const float* __restrict__ x, const float* __restrict__ w, T* __restrict__ h, int W, int Wp,
+                     float eps) {
+  __shared__ float red[RS_THREADS / 32];
+  pdl_launch_dependents();
+  pdl_wait();
+  const long long row = blockIdx.x;
+  float ss = 0.f;
+  for (int c = threadIdx.x; c < W; c += RS_THREADS) {
+    const float v = x[row * W + c];
+    ss += v * v;
+  }
+  const float inv = rsqrtf(cta_sum<RS_THREADS>(ss, red) / float(W) + eps);
+  for (int c = threadIdx.x; c < Wp; c += RS_THREADS)
+    h[row * Wp + c] = Elem<T>::put(c < W ? x[row * W + c] * inv * w[c] : 0.f);
+}
+
+// out = gelu_tanh(gate + bias) * (up + bias), four columns per thread
+template <typename T>
+__global__ void __launch_bounds__(RS_THREADS)
+gelu_mul_kernel(const ProjSrc gu, const T* __restrict__ bias, T* __restrict__ out, long long total, int quads,
+                int up_off, int width, int width_p) {
+  pdl_launch_dependents();
+  pdl_wait();
+  for (long long i = blockIdx.x * (long long)RS_THREADS + threadIdx.x; i < total;
+       i += (long long)gridDim.x * RS_THREADS) {
+    const long long row = i / quads;
+    const int col = int(i - row * quads) * 4;
+    const float4 g = proj_at4<T>(gu, row, col), u = proj_at4<T>(gu, row, up_off + col);
+    const float gv[4] = {g.x, g.y, g.z, g.w}, uv[4] = {u.x, u.y, u.z, u.w};
+    float o[4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      float a = gv[j], b = uv[j];
+      if (bias != nullptr) {
+        a += Elem<T>::get(bias[col + j]);
+        b += Elem<T>::get(bias[up_off + col + j]);
+      }
+      o[j] = col + j < width ? gelu_tanh_f(a) * b : 0.f;
+    }
+    store4(out + row * width_p + col, o[0], o[1], o[2], o[3]);
+  }
+}
+
+// ================================================================= launchers
+static void check_launch(const char* what) {
+  const cudaError_t e = cudaGetLastError();
+  if (e != cudaSuccess) throw std::runtime_error(std::string(what) + ": " + cudaGetErrorString(e));
+}
+
+template <typename T>
+static void embed_t(const void* ids, const void* weight, float* x, void* h, int T_, int W, int Wp, long long V,
+                    float scale, uint32_t* status, cudaStream_t s) {
+  launch_pdl(PDL_EMBEDDING, embed_scaled_kernel<T>, dim3(T_), dim3(RS_THREADS), 0, s, (const long long*)ids,
+             (const T*)weight, x, (T*)h, W, Wp, V, scale, status);
+}
+void launch_embed_scaled(const void* ids, const void* weight, float* x, void* h, int T, int W, int Wp, long long V,
+                         float scale, bool f32, uint32_t* status, cudaStream_t s) {
+  if (T == 0) return;
+  if (f32) embed_t<float>(ids, weight, x, h, T, W, Wp, V, scale, status, s);
+  else embed_t<bf16>(ids, weight, x, h, T, W, Wp, V, scale, status, s);
+  check_launch("embedding");
+}
+
+template <typename T>
+static void post_norm_t(const ProjSrc& y, const void* bias, float* x, const float* w, void* h, int T_, int W, int Wp,
+                        float eps, cudaStream_t s) {
+  if (W % 4 == 0)
+    launch_pdl(PDL_NORM, post_norm_add_kernel<T, true>, dim3(T_), dim3(RS_THREADS), 0, s, y, (const T*)bias, x, w,
+               (T*)h, W, Wp, eps);
+  else
+    launch_pdl(PDL_NORM, post_norm_add_kernel<T, false>, dim3(T_), dim3(RS_THREADS), 0, s, y, (const T*)bias, x, w,
+               (T*)h, W, Wp, eps);
+}
+void launch_post_norm_add(const ProjSrc& y, const void* bias, float* x, const float* w, void* h, int T, int W, int Wp,
+                          float eps, bool f32, cudaStream_t s) {
+  if (T == 0) return;
+  if (W > RS_THREADS * RS_CHUNKS * 4) throw std::runtime_error("norm rows are limited to 8192 columns");
+  if (f32) post_norm_t<float>(y, bias, x, w, h, T, W, Wp, eps, s);
+  else post_norm_t<bf16>(y, bias, x, w, h, T, W, Wp, eps, s);
+  check_launch("norm + add");
+}
+
+void launch_rms_norm_wide(const float* x, const float* w, void* h, int T, int W, int Wp, float eps, bool f32,
+                          cudaStream_t s) {
+  if (T == 0) return;
+  if (f32)
+    launch_pdl(PDL_NORM, rms_norm_wide_kernel<float>, dim3(T), dim3(RS_THREADS), 0, s, x, w, (float*)h, W, Wp, eps);
+  else
+    launch_pdl(PDL_NORM, rms_norm_wide_kernel<bf16>, dim3(T), dim3(RS_THREADS), 0, s, x, w, (bf16*)h, W, Wp, eps);
+  check_launch("final norm");
+}
+
+void launch_gelu_mul(const ProjSrc& gu, const void* bias, void* out, int T, int up_off, int width, int width_p,
+                     bool f32, cudaStream_t s) {
+  if (T == 0) return;
+  const int quads = width_p / 4;
+  const long long total = (long long)T * quads;
+  const int blocks = (int)std::min<long long>((total + RS_THREADS - 1) / RS_THREADS, 148 * 16);
+  if (f32)
+    launch_pdl(PDL_PARTIALS, gelu_mul_kernel<float>, dim3(blocks), dim3(RS_THREADS), 0, s, gu, (const float*)bias,
+               (float*)out, total, quads, up_off, width, width_p);
+  else
+    launch_pdl(PDL_PARTIALS, gelu_mul_kernel<bf16>, dim3(blocks), dim3(RS_THREADS), 0, s, gu, (const bf16*)bias,
+               (bf16*)out, total, quads, up_off, width, width_p);
+  check_launch("gelu gate");
+}
+
+}  // namespace fc

@@ -21,6 +21,9 @@ __device__ __forceinline__ bool sample_better(float v, int i, float best, int be
   return v > best || (v == best && i < best_i);
 }
 
+__device__ __forceinline__ float sample_value(float v) { return v; }
+__device__ __forceinline__ float sample_value(__nv_bfloat16 v) { return __bfloat162float(v); }
+
 // Best (value, global index) of row `row` [V logits, global indices vocab_offset + j, indices >= v_limit are
 // padding and never win] for the calling CTA; valid in thread 0 after the call.  `s_val` / `s_idx`: 32 words each.
 //
@@ -28,7 +31,8 @@ __device__ __forceinline__ bool sample_better(float v, int i, float best, int be
 // plus a constant, hence the same winner for one multiply-add and two lg2 per entry.  u = (k + 0.5) / 2^23 with k
 // the top 23 bits of the hash: k + 0.5 is exact in fp32, so u stays inside (0, 1) and the noise inside (-2.9, 16.7)
 // (with 24 bits the largest k + 0.5 would round up to u = 1 and give that entry infinite noise).
-__device__ __forceinline__ void sample_row_best(const __nv_bfloat16* row, int V, int vocab_offset, int v_limit,
+template <typename T_>      // bf16 or fp32 logits
+__device__ __forceinline__ void sample_row_best(const T_* row, int V, int vocab_offset, int v_limit,
                                                 float T, uint32_t row_seed, float* s_val, int* s_idx,
                                                 float& best, int& best_i) {
   best = -INFINITY;
@@ -49,7 +53,7 @@ __device__ __forceinline__ void sample_row_best(const __nv_bfloat16* row, int V,
       local_i = j;
     }
   };
-  const bool vec = ((reinterpret_cast<uintptr_t>(row) & 15) == 0);
+  const bool vec = sizeof(T_) == 2 && ((reinterpret_cast<uintptr_t>(row) & 15) == 0);
   const int v8 = (vec && n > 0) ? (n >> 3) : 0;
   for (int c = threadIdx.x; c < v8; c += blockDim.x) {           // 16-byte loads: 8 logits at a time
     const uint4 u = __ldcg(reinterpret_cast<const uint4*>(row) + c);
@@ -61,7 +65,7 @@ __device__ __forceinline__ void sample_row_best(const __nv_bfloat16* row, int V,
       consider(f.y, c * 8 + 2 * i + 1);
     }
   }
-  for (int j = v8 * 8 + threadIdx.x; j < n; j += blockDim.x) consider(__bfloat162float(row[j]), j);
+  for (int j = v8 * 8 + threadIdx.x; j < n; j += blockDim.x) consider(sample_value(row[j]), j);
   if (local_i >= 0) best_i = vocab_offset + local_i;
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) {

@@ -17,7 +17,11 @@ def gemm(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor] = N
     x2 = x.reshape(-1, x.shape[-1])
     if x2.stride(-1) != 1:
         x2 = x2.contiguous()
-    if act == "swiglu":
+    if x2.dtype == torch.float32:                                # true 32-bit, CUDA cores
+        if act != "none" or out is not None:
+            raise ValueError("fp32 products take no activation or output buffer")
+        y = ext().linear_wide(x2, weight, bias)
+    elif act == "swiglu":
         if x2.shape[0] > 256 and weight.shape[0] % 256 == 0 and bias is None:
             y = ext().gemm(x2, weight, None, 6, None)        # SwiGLU applied in the GEMM epilogue
         else:

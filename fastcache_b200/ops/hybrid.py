@@ -15,6 +15,9 @@ from . import reference_hybrid as ref
 from .loader import ext
 
 
+LATENT_IMPL = 0         # 1: the general kernels also where a tensor-core form exists (tests)
+
+
 def _n(k: int = 1) -> None:
     from . import COUNTERS
     COUNTERS["launches"] += k
@@ -120,7 +123,7 @@ def delta_rule(h, weight, d: DeltaDims, conv_w, a_log, dt_bias, norm_w, eps: flo
         _n(4)
         return ext().delta_rule(h, weight, conv_w, a_log, dt_bias, norm_w, float(eps), conv_state, state,
                                 [d.heads, d.kv_heads, d.dim, d.vdim, d.g, d.b, d.a], float(d.unit_eps),
-                                *_run_args(ctx))
+                                *_run_args(ctx), ctx.row_seq)
     return ref.delta_rule(ref_linear(h, weight), d, conv_w, a_log, dt_bias, norm_w, eps, conv_state, state, ctx)
 
 
@@ -137,8 +140,12 @@ def latent_attention(h, weight, d: LatentDims, kv_norm_w, eps: float, kv_proj, w
     `kv_proj` (packed uk | uv) expands cache rows to keys and values (prefill); `w_ukt` [H, rank, dim] and `w_uv`
     [H, vdim, rank] are the same weights for the absorbed form (decode), which never expands a row."""
     if h.is_cuda:
-        from .latent import latent_attention_cuda
-        return latent_attention_cuda(h, weight, d, kv_norm_w, eps, kv_proj, w_ukt, w_uv, pool, positions, ctx)
+        _n(6)
+        return ext().latent_attention(
+            h, weight, [d.heads, d.dim, d.rot, d.vdim, d.rank, d.rot_dims, d.q, -1 if d.kv is None else d.kv, d.g],
+            d.scale, d.base, kv_norm_w, float(eps), kv_proj.weight, kv_proj.offset["uv"], w_ukt, w_uv, pool, positions,
+            ctx.slot_mapping, ctx.block_tables, ctx.context_lens, ctx.cu_seqlens_q, ctx.cu_seqlens_kv, ctx.row_seq,
+            ctx.row_ctx, int(ctx.max_seqlen_q), int(ctx.max_seqlen_k), int(ctx.total_kv), LATENT_IMPL)
     p = ref_linear(h, weight)
     q = ref.latent_project(p, d, kv_norm_w, eps, positions, pool, ctx.slot_mapping)
     w, off = kv_proj.weight, kv_proj.offset
