@@ -45,6 +45,10 @@ int gemm_num_sms();
 CUtensorMap make_tmap_bf16_2d(const void* base, uint64_t rows, uint64_t cols, uint64_t ld, uint32_t box_rows,
                               uint32_t box_cols);
 
+// The same for [n2][n1][n0] with pitches ld1 (between n1) and ld2 (between n2) in elements; box columns past n0 read zero.
+CUtensorMap make_tmap_bf16_3d(const void* base, uint64_t n0, uint64_t n1, uint64_t n2, uint64_t ld1, uint64_t ld2,
+                              uint32_t box0, uint32_t box1, uint32_t box2);
+
 // c[M, N] = act(x[M, K] @ w[N, K]^T + bias[N]); bf16 in/out, fp32 accumulate.
 // ldx / ldw / ldc are row pitches in elements.  sm_limit > 0 caps the persistent grid
 // (used when the launching stream belongs to a green context with fewer SMs).

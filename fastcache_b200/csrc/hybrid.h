@@ -156,7 +156,7 @@ void launch_gather_rows(const void* pool, const int* block_tables, const int* ct
                         uint32_t* status, cudaStream_t s);
 // expanded causal attention on tcgen05 (latent_prefill.cu)
 struct LatentPrefill {
-  int T = 0, B = 0, H = 0, D = 0, R = 0, V = 0, max_q = 0;
+  int T = 0, B = 0, H = 0, D = 0, R = 0, V = 0, rank = 0, max_q = 0;
   long long total_kv = 0;
   const void* q = nullptr;           // [T, H, D + R]
   const void* k = nullptr;           // [total_kv, ld_kv]: keys, head by head

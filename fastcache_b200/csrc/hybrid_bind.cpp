@@ -376,6 +376,7 @@ Tensor latent_attention(const Tensor& h, const Tensor& w, const std::vector<int6
     a.D = D;
     a.R = R;
     a.V = V;
+    a.rank = rank;
     a.max_q = int(max_q);
     a.total_kv = total_kv;
     if (fc::latent_prefill_supported(a)) {

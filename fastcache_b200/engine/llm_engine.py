@@ -105,7 +105,7 @@ class LLMEngine:
         self.config = config
         Sequence.block_size = config.kvcache_block_size
 
-        self.tokenizer = tokenizer
+        self.tokenizer = None if tokenizer is False else tokenizer      # False: token ids only, look for none
         self.processor = None
         if tokenizer is None and model:
             self._load_tokenizer(model)
