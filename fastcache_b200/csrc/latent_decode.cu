@@ -1,9 +1,413 @@
-#include "hybrid.cuh"
+// Absorbed latent attention of decode-size batches (bf16): every query row attends to the cache rows of its request as
+// they are, key = [latent | rotated part], value = latent, shared by all heads.
+//
+// Grid (query row, group of 16 * MT heads, split of the context).  A CTA streams 64-row tiles of the cache through a
+// two-stage TMA ring (128-byte swizzle, boxes that never straddle a page); one tile in shared memory is both the keys
+// and the values of all its heads, so a row is read once.  Per tile:
+//   scores   warp w: 16 keys (w & 3) against all heads, half of the columns (w >> 2), mma.sync m16n8k16; the two halves
+//            are added when they are read back
+//   softmax  16 / MT threads per head, running maximum and sum in registers, P to shared memory as bf16
+//   values   warp w owns the latent columns of 16-column groups w, w + 8, ...; P V accumulates in registers
+// With several splits a CTA writes normalised partials with their log-sum-exp and a second kernel merges them.
+//
+// Also here: the per-head products around it (queries into the latent space, outputs out of it).
+#include <algorithm>
 #include <stdexcept>
+#include <string>
+
+#include "gemm.h"
+#include "hybrid.cuh"
+#include "launch.h"
+#include "mma.cuh"
+
 namespace fc {
-bool head_linear_mma_supported(const SimtLinear&) { return false; }
-void launch_head_linear_mma(const SimtLinear&, cudaStream_t) { throw std::runtime_error("-"); }
-bool latent_decode_supported(const LatentAttn&) { return false; }
-int latent_decode_splits(const LatentAttn&, int, int) { return 1; }
-void launch_latent_decode(const LatentAttn&, cudaStream_t) { throw std::runtime_error("-"); }
+
+using bf16 = __nv_bfloat16;
+constexpr int LD_TILE = 64, LD_STAGES = 2, LD_THREADS = 256;
+constexpr int LD_SUB = LD_TILE * 128;             // bytes of a [64 rows x 64 columns] sub-tile
+constexpr int LD_MAX_SPLITS = 32;
+
+// byte offset of 16-byte chunk `chunk` of row `row` in sub-tiles of `rows` rows x 128 bytes
+__device__ __forceinline__ uint32_t ld_swz(int rows, int row, int chunk) {
+  return uint32_t((chunk >> 3) * rows * 128 + row * 128 + (((chunk & 7) ^ (row & 7)) << 4));
 }
+
+template <int MT, int NPW>
+__global__ void __launch_bounds__(LD_THREADS, 1)
+latent_decode_kernel(const __grid_constant__ CUtensorMap tm, const LatentAttn p, int box_rows, int nc, float scale_log2) {
+  constexpr int HR = MT * 16;                     // head rows of this CTA
+  constexpr int TPR = LD_THREADS / HR;            // softmax threads per head row
+  constexpr int KPT = LD_TILE / TPR;              // keys per softmax thread
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+  const int stage_bytes = nc * LD_SUB;
+  uint8_t* s_kv = smem;                                            // [LD_STAGES]
+  uint8_t* s_q = s_kv + LD_STAGES * stage_bytes;                   // [nc][HR][128 B]
+  uint8_t* s_p = s_q + nc * HR * 128;                              // [HR][128 B]
+  float* s_s = reinterpret_cast<float*>(s_p + HR * 128);           // [2][HR][LD_TILE + 4]
+  float* s_cor = s_s + 2 * HR * (LD_TILE + 4);                     // [HR]
+  float* s_l = s_cor + HR;                                         // [HR]
+  uint64_t* full = reinterpret_cast<uint64_t*>(s_l + HR);          // [LD_STAGES]
+  constexpr int SLD = LD_TILE + 4;
+
+  const int t = blockIdx.x, h0 = blockIdx.y * HR, split = blockIdx.z;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  pdl_launch_dependents();
+  if (tid == 0) {
+    for (int s = 0; s < LD_STAGES; ++s) mbar_init(&full[s], 1);
+    fence_barrier_init();
+    tma_prefetch_desc(&tm);
+  }
+  pdl_wait();
+  asm volatile("fence.proxy.async.global;" ::: "memory");          // rows were written with ordinary stores
+  const int ctx = p.row_ctx[t];
+  const int b = p.row_seq != nullptr ? p.row_seq[t] : t;
+  const int tiles = (ctx + LD_TILE - 1) / LD_TILE;
+  const int per = (tiles + p.splits - 1) / p.splits;
+  const int tile0 = split * per, n_tiles = max(0, min(tiles, tile0 + per) - tile0);
+  const int* bt = p.block_tables + (long long)b * p.max_blocks;
+  const int w = p.rank + p.R;
+
+  // Q, zero-padded to whole sub-tiles and head rows
+  for (int i = tid; i < HR * nc * 8; i += LD_THREADS) {
+    const int r = i / (nc * 8), ch = i - r * (nc * 8);
+    uint4 v = make_uint4(0, 0, 0, 0);
+    if (h0 + r < p.H && ch * 8 < w)
+      v = __ldcg(reinterpret_cast<const uint4*>(reinterpret_cast<const bf16*>(p.q_abs) +
+                                                ((long long)t * p.H + h0 + r) * w + ch * 8));
+    *reinterpret_cast<uint4*>(s_q + ld_swz(HR, r, ch)) = v;
+  }
+  if (n_tiles <= LD_STAGES) {
+    // boxes past the context are never loaded: what they would hold must be finite
+    for (int i = tid; i < n_tiles * stage_bytes / 16; i += LD_THREADS)
+      reinterpret_cast<uint4*>(s_kv)[i] = make_uint4(0, 0, 0, 0);
+    fence_proxy_async();
+  }
+  __syncthreads();
+
+  auto load_tile = [&](int tile, int stage) {
+    const int row0 = tile * LD_TILE;
+    const int pieces = min(LD_TILE / box_rows, (ctx - row0 + box_rows - 1) / box_rows);
+    mbar_expect_tx(&full[stage], uint32_t(pieces) * nc * box_rows * 128);
+    for (int pc = 0; pc < pieces; ++pc) {
+      const int tok = row0 + pc * box_rows;
+      int blk = bt[tok / p.block_size];
+      if (blk < 0 || blk >= p.num_blocks) {
+        report(p.status, ST_BAD_INDEX);
+        blk = 0;
+      }
+      const int grow = blk * p.block_size + tok % p.block_size;
+      for (int c = 0; c < nc; ++c)
+        tma_load_2d(s_kv + stage * stage_bytes + c * LD_SUB + pc * box_rows * 128, &tm, &full[stage], c * 64, grow);
+    }
+  };
+  if (tid == 0)
+    for (int s = 0; s < LD_STAGES; ++s)
+      if (s < n_tiles) load_tile(tile0 + s, s);
+
+  const int g = lane >> 2, q4 = lane & 3;
+  float o[MT][NPW][2][4];
+#pragma unroll
+  for (int m = 0; m < MT; ++m)
+#pragma unroll
+    for (int n = 0; n < NPW; ++n)
+#pragma unroll
+      for (int e = 0; e < 8; ++e) o[m][n][e >> 2][e & 3] = 0.f;
+  const int srow = tid / TPR, sk0 = (tid % TPR) * KPT;             // softmax: head row and first key of this thread
+  float m_run = -INFINITY, l_run = 0.f;
+  const int ksteps = (p.row_width + 15) / 16, khalf = (ksteps + 1) / 2;
+  const int kg = (warp & 3) * 16, part = warp >> 2;
+  const int k_lo = part * khalf, k_hi = min(ksteps, k_lo + khalf);
+  const uint32_t q_base = smem_u32(s_q), p_base = smem_u32(s_p);
+  bool alive = true;
+  for (int it = 0; it < n_tiles; ++it) {
+    const int stage = it % LD_STAGES;
+    if (!mbar_wait(&full[stage], (it / LD_STAGES) & 1, p.status, ST_TIMEOUT_FULL)) alive = false;
+    if (__syncthreads_or(!alive)) {
+      alive = false;
+      break;
+    }
+    const uint32_t kv = smem_u32(s_kv + stage * stage_bytes);
+    // ---- scores of 16 keys, half of the columns
+    float sc[MT][2][4];
+#pragma unroll
+    for (int m = 0; m < MT; ++m)
+#pragma unroll
+      for (int e = 0; e < 8; ++e) sc[m][e >> 2][e & 3] = 0.f;
+    const int mat = lane >> 3;
+#pragma unroll 4
+    for (int kk = k_lo; kk < k_hi; ++kk) {
+      uint32_t b0, b1, b2, b3;
+      ldsm_x4(kv + ld_swz(LD_TILE, kg + (mat >> 1) * 8 + (lane & 7), kk * 2 + (mat & 1)), b0, b1, b2, b3);
+#pragma unroll
+      for (int m = 0; m < MT; ++m) {
+        uint32_t a[4];
+        ldsm_x4(q_base + ld_swz(HR, m * 16 + (mat & 1) * 8 + (lane & 7), kk * 2 + (mat >> 1)), a[0], a[1], a[2], a[3]);
+        mma_bf16(sc[m][0], a, b0, b1);
+        mma_bf16(sc[m][1], a, b2, b3);
+      }
+    }
+#pragma unroll
+    for (int m = 0; m < MT; ++m)
+#pragma unroll
+      for (int n = 0; n < 2; ++n) {
+        float* d = s_s + (part * HR + m * 16 + g) * SLD + kg + n * 8 + q4 * 2;
+        *reinterpret_cast<float2*>(d) = make_float2(sc[m][n][0], sc[m][n][1]);
+        *reinterpret_cast<float2*>(d + 8 * SLD) = make_float2(sc[m][n][2], sc[m][n][3]);
+      }
+    __syncthreads();
+    // ---- softmax of one head row by TPR threads
+    {
+      const int valid = ctx - (tile0 + it) * LD_TILE;              // keys of this tile that exist
+      float v[KPT];
+      float mx = -INFINITY;
+#pragma unroll
+      for (int i = 0; i < KPT; ++i) {
+        const float s = s_s[srow * SLD + sk0 + i] + s_s[(HR + srow) * SLD + sk0 + i];
+        v[i] = sk0 + i < valid ? s * scale_log2 : -INFINITY;
+        mx = fmaxf(mx, v[i]);
+      }
+#pragma unroll
+      for (int x = 1; x < TPR; x <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, x));
+      const float mn = fmaxf(m_run, mx);                           // a tile has at least one key
+      const float cor = exp2f(m_run - mn);
+      m_run = mn;
+      float rs = 0.f;
+#pragma unroll
+      for (int i = 0; i < KPT; i += 2) {
+        const float e0 = exp2f(v[i] - mn), e1 = exp2f(v[i + 1] - mn);
+        rs += e0 + e1;
+        const int key = sk0 + i;
+        *reinterpret_cast<uint32_t*>(s_p + ld_swz(HR, srow, key >> 3) + (key & 7) * 2) = pack_bf16(e0, e1);
+      }
+      l_run = l_run * cor + rs;
+      if (tid % TPR == 0) s_cor[srow] = cor;
+    }
+    __syncthreads();
+    // ---- O = O * cor + P V
+#pragma unroll
+    for (int m = 0; m < MT; ++m) {
+      const float c0 = s_cor[m * 16 + g], c1 = s_cor[m * 16 + g + 8];
+#pragma unroll
+      for (int n = 0; n < NPW; ++n)
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          o[m][n][e][0] *= c0;
+          o[m][n][e][1] *= c0;
+          o[m][n][e][2] *= c1;
+          o[m][n][e][3] *= c1;
+        }
+    }
+#pragma unroll
+    for (int ks = 0; ks < LD_TILE / 16; ++ks) {
+      uint32_t a[MT][4];
+#pragma unroll
+      for (int m = 0; m < MT; ++m)
+        ldsm_x4(p_base + ld_swz(HR, m * 16 + (mat & 1) * 8 + (lane & 7), ks * 2 + (mat >> 1)), a[m][0], a[m][1], a[m][2],
+                a[m][3]);
+#pragma unroll
+      for (int n = 0; n < NPW; ++n) {
+        const int cg = warp + n * 8;                               // 16-column group of the latent
+        if (cg * 16 >= p.rank) continue;
+        uint32_t b0, b1, b2, b3;
+        ldsm_x4_t(kv + ld_swz(LD_TILE, ks * 16 + (mat & 1) * 8 + (lane & 7), cg * 2 + (mat >> 1)), b0, b1, b2, b3);
+#pragma unroll
+        for (int m = 0; m < MT; ++m) {
+          mma_bf16(o[m][n][0], a[m], b0, b1);
+          mma_bf16(o[m][n][1], a[m], b2, b3);
+        }
+      }
+    }
+    __syncthreads();                                               // every warp is done with this stage, S and P
+    if (tid == 0 && it + LD_STAGES < n_tiles) load_tile(tile0 + it + LD_STAGES, stage);
+  }
+  // ---- finish: 1 / l per head row, then either the result or a normalised partial
+#pragma unroll
+  for (int x = 1; x < TPR; x <<= 1) l_run += __shfl_xor_sync(0xffffffffu, l_run, x);
+  if (tid % TPR == 0) {
+    s_l[srow] = alive && l_run > 0.f ? 1.f / l_run : 0.f;
+    if (p.splits > 1 && h0 + srow < p.H)
+      p.part_lse[((long long)t * p.H + h0 + srow) * p.splits + split] =
+          alive && l_run > 0.f ? m_run + log2f(l_run) : -INFINITY;
+  }
+  __syncthreads();
+#pragma unroll
+  for (int m = 0; m < MT; ++m)
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+      const int r = m * 16 + half * 8 + g;
+      if (h0 + r >= p.H) continue;
+      const float inv = s_l[r];
+      const long long row = (long long)t * p.H + h0 + r;
+#pragma unroll
+      for (int n = 0; n < NPW; ++n) {
+        const int cg = warp + n * 8;
+        if (cg * 16 >= p.rank) continue;
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const int col = cg * 16 + e * 8 + q4 * 2;
+          const float a = o[m][n][e][half * 2] * inv, c = o[m][n][e][half * 2 + 1] * inv;
+          if (p.splits == 1)
+            *reinterpret_cast<uint32_t*>(reinterpret_cast<bf16*>(p.o_lat) + row * p.rank + col) = pack_bf16(a, c);
+          else
+            *reinterpret_cast<float2*>(p.part_o + (row * p.splits + split) * p.rank + col) = make_float2(a, c);
+        }
+      }
+    }
+}
+
+// o_lat[row] = sum_s 2^(lse_s - max) part_o[row, s] / sum_s 2^(lse_s - max); one warp per (row, head), 4 columns a lane
+__global__ void __launch_bounds__(256)
+latent_merge_kernel(const LatentAttn p) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const long long row = blockIdx.x * 8ll + (threadIdx.x >> 5);
+  if (row >= (long long)p.T * p.H) return;
+  const int lane = threadIdx.x & 31;
+  const float l = lane < p.splits ? __ldcg(p.part_lse + row * p.splits + lane) : -INFINITY;
+  const float mx = warp_max(l);
+  const float wgt = l == -INFINITY ? 0.f : exp2f(l - mx);
+  const float den = warp_sum(wgt);
+  const float inv = den > 0.f ? 1.f / den : 0.f;
+  for (int c0 = 0; c0 < p.rank; c0 += 128) {                       // every lane stays for the shuffles
+    const int c = c0 + lane * 4;
+    float a[4] = {0.f, 0.f, 0.f, 0.f};
+    for (int s = 0; s < p.splits; ++s) {
+      const float f = __shfl_sync(0xffffffffu, wgt, s) * inv;
+      if (c >= p.rank) continue;
+      const float4 v = __ldcg(reinterpret_cast<const float4*>(p.part_o + (row * p.splits + s) * p.rank + c));
+      a[0] = fmaf(f, v.x, a[0]);
+      a[1] = fmaf(f, v.y, a[1]);
+      a[2] = fmaf(f, v.z, a[2]);
+      a[3] = fmaf(f, v.w, a[3]);
+    }
+    if (c < p.rank) store4(reinterpret_cast<bf16*>(p.o_lat) + row * p.rank + c, a[0], a[1], a[2], a[3]);
+  }
+}
+
+static int ld_box_rows(int block_size) {
+  int box = LD_TILE;
+  while (box > block_size || block_size % box != 0) box >>= 1;
+  return box;
+}
+static int ld_nc(const LatentAttn& p) { return (p.row_width + 63) / 64; }
+static int ld_smem(int mt, int nc) {
+  return LD_STAGES * nc * LD_SUB + nc * mt * 16 * 128 + mt * 16 * 128 + 2 * mt * 16 * (LD_TILE + 4) * 4 +
+         2 * mt * 16 * 4 + 64 + 1024;
+}
+static int ld_mt(const LatentAttn& p) {
+  int mt = p.H > 32 ? 4 : p.H > 16 ? 2 : 1;
+  while (mt > 1 && ld_smem(mt, ld_nc(p)) > 227 * 1024) mt >>= 1;
+  return mt;
+}
+
+bool latent_decode_supported(const LatentAttn& p) {
+  return p.rank % 16 == 0 && p.rank <= 512 && (p.rank + p.R) % 8 == 0 && ld_box_rows(p.block_size) >= 8 &&
+         ld_smem(ld_mt(p), ld_nc(p)) <= 227 * 1024;
+}
+
+int latent_decode_splits(const LatentAttn& p, int max_ctx, int num_sms) {
+  const int hr = ld_mt(p) * 16;
+  const int ctas = p.T * ((p.H + hr - 1) / hr);
+  const int by_len = std::max(1, max_ctx / (4 * LD_TILE));
+  int s = std::max(1, std::min({num_sms / std::max(1, ctas), by_len, LD_MAX_SPLITS}));
+  if (ctas < num_sms && ctas * 3 > num_sms * 2) s = 1;             // nearly a full wave already
+  return s;
+}
+
+void launch_latent_decode(const LatentAttn& p, cudaStream_t s) {
+  if (p.T == 0) return;
+  const int box = ld_box_rows(p.block_size), nc = ld_nc(p), mt = ld_mt(p), smem = ld_smem(mt, nc);
+  const CUtensorMap tm = make_tmap_bf16_2d(p.pool, (uint64_t)p.num_blocks * p.block_size, p.row_width, p.row_width, box, 64);
+  const dim3 grid(p.T, (p.H + mt * 16 - 1) / (mt * 16), p.splits);
+  const float scale_log2 = p.scale * 1.4426950408889634f;
+  auto go = [&](auto kern) {
+    cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    // ordinary launch like the other paged decode attention
+    launch_pdl(PDL_DECODE_ATTN, kern, grid, dim3(LD_THREADS), smem, s, tm, p, box, nc, scale_log2);
+  };
+  auto pick = [&](auto m) {
+    constexpr int MT = decltype(m)::value;
+    if (p.rank <= 128) go(latent_decode_kernel<MT, 1>);
+    else if (p.rank <= 256) go(latent_decode_kernel<MT, 2>);
+    else go(latent_decode_kernel<MT, 4>);
+  };
+  if (mt == 1) pick(std::integral_constant<int, 1>{});
+  else if (mt == 2) pick(std::integral_constant<int, 2>{});
+  else pick(std::integral_constant<int, 4>{});
+  if (p.splits > 1)
+    launch_pdl(PDL_DECODE_MERGE, latent_merge_kernel, dim3(unsigned(((long long)p.T * p.H + 7) / 8)), dim3(256), 0, s, p);
+  const cudaError_t e = cudaGetLastError();
+  if (e != cudaSuccess) throw std::runtime_error(std::string("latent decode: ") + cudaGetErrorString(e));
+}
+
+// ------------------------------------------------------------------ per-head products
+// y[g][m, n] = sum_k x[g][m, k] w[g][n, k] for few rows m: bound by reading w once.  One warp per 16 rows of w (they are
+// the M side of mma.sync m16n8k16, so no row of the tensor-core tile is wasted on a small batch); NT n8-tiles hold up to
+// 8 * NT batch rows.  Four warps of a CTA take consecutive 16-row groups.
+constexpr int HL_WARPS = 4;
+template <int NT>
+__global__ void __launch_bounds__(HL_WARPS * 32)
+head_linear_kernel(const SimtLinear a) {
+  pdl_launch_dependents();
+  const int g = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int n0 = (blockIdx.x * HL_WARPS + warp) * 16, m0 = blockIdx.z * NT * 8;
+  const int r = lane >> 2, c = (lane & 3) * 2;
+  const bf16* w = reinterpret_cast<const bf16*>(a.w) + g * a.gw;
+  const bf16* x = reinterpret_cast<const bf16*>(a.x) + g * a.gx;
+  float acc[NT][4];
+#pragma unroll
+  for (int i = 0; i < NT; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
+  pdl_wait();
+  if (n0 < a.N) {
+    const bool w0ok = n0 + r < a.N, w1ok = n0 + r + 8 < a.N;
+    const bf16 *w0 = w + (long long)(n0 + r) * a.ldw + c, *w1 = w0 + 8 * a.ldw;
+    auto ld = [](const bf16* q, bool ok) { return ok ? __ldcg(reinterpret_cast<const uint32_t*>(q)) : 0u; };
+#pragma unroll 2
+    for (int k = 0; k < a.K; k += 16) {
+      const bool hi = k + 8 < a.K;                                 // K is a multiple of 8
+      const uint32_t af[4] = {ld(w0 + k, w0ok), ld(w1 + k, w1ok), ld(w0 + k + 8, w0ok && hi), ld(w1 + k + 8, w1ok && hi)};
+#pragma unroll
+      for (int i = 0; i < NT; ++i) {
+        const int m = m0 + i * 8 + r;
+        const bf16* xr = x + (long long)m * a.ldx + c + k;
+        mma_bf16(acc[i], af, ld(xr, m < a.M), ld(xr + 8, m < a.M && hi));
+      }
+    }
+    const bool gated = a.gate.p != nullptr || a.gate.part != nullptr;
+    bf16* y = reinterpret_cast<bf16*>(a.y) + g * a.gy;
+#pragma unroll
+    for (int i = 0; i < NT; ++i)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int n = n0 + r + (e >> 1) * 8, m = m0 + i * 8 + c + (e & 1);
+        if (n >= a.N || m >= a.M) continue;
+        float v = acc[i][e];
+        if (gated) v *= sigmoid_f(proj_at<bf16>(a.gate, m, a.gate_off + g * a.N + n));
+        y[(long long)m * a.ldy + n] = __float2bfloat16(v);
+      }
+  }
+  if (a.y_pad > a.groups * a.N && g == 0 && blockIdx.x == 0)
+    for (int i = threadIdx.x; i < NT * 8 * (a.y_pad - a.groups * a.N); i += HL_WARPS * 32) {
+      const int pad = a.y_pad - a.groups * a.N, m = m0 + i / pad;
+      if (m < a.M) reinterpret_cast<bf16*>(a.y)[(long long)m * a.ldy + a.groups * a.N + i % pad] = __float2bfloat16(0.f);
+    }
+}
+
+bool head_linear_mma_supported(const SimtLinear& a) {
+  return a.K % 8 == 0 && a.ldx % 2 == 0 && a.ldw % 2 == 0 && a.gx % 2 == 0 && a.gw % 2 == 0 && a.bias == nullptr;
+}
+void launch_head_linear_mma(const SimtLinear& a, cudaStream_t s) {
+  if (a.M == 0 || a.N == 0) return;
+  auto go = [&](auto kern, int rows) {
+    launch_pdl(PDL_SKINNY_GEMM, kern, dim3((a.N + HL_WARPS * 16 - 1) / (HL_WARPS * 16), a.groups, (a.M + rows - 1) / rows),
+               dim3(HL_WARPS * 32), 0, s, a);
+  };
+  if (a.M <= 8) go(head_linear_kernel<1>, 8);
+  else if (a.M <= 32) go(head_linear_kernel<4>, 32);
+  else go(head_linear_kernel<8>, 64);
+  const cudaError_t e = cudaGetLastError();
+  if (e != cudaSuccess) throw std::runtime_error(std::string("per-head product: ") + cudaGetErrorString(e));
+}
+
+}  // namespace fc
