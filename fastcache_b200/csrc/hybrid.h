@@ -76,6 +76,7 @@ struct StepParams {
   const void* v = nullptr;           // [T, H * V]
   const float* log_g = nullptr;      // [T, H]
   const float* beta = nullptr;       // [T, H]
+  uint8_t* scratch = nullptr;        // chunked form: chunk_scratch_bytes()
   // output: `out` with the head norm and gate applied, or raw fp32 head outputs in `o_raw`
   float* o_raw = nullptr;            // [T, H * V]
   void* out = nullptr;
@@ -108,7 +109,7 @@ void launch_delta_prepare(const DeltaPrepare& p, bool f32, cudaStream_t s);
 
 // ---- recurrence_chunk.cu (bf16 runs of many rows): o_raw [T, H * V] and the state after every run
 bool chunk_supported(int D, int V);
-size_t gla_chunk_scratch_floats(const StepParams& p, int T, int max_len);
+long long chunk_scratch_bytes(const StepParams& p, int T, bool delta);
 void launch_gla_chunk(const StepParams& p, int max_len, cudaStream_t s);
 void launch_delta_chunk(const StepParams& p, int max_len, cudaStream_t s);
 

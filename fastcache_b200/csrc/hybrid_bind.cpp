@@ -183,7 +183,10 @@ void run_recurrence(fc::StepParams& p, const Tensor& h, bool delta, bool chunk, 
     o_raw = torch::empty({T, p.H * p.V}, h.options().dtype(torch::kFloat32));
     p.o_raw = o_raw.data_ptr<float>();
   }
+  Tensor scratch;
   if (chunk) {
+    scratch = torch::empty({fc::chunk_scratch_bytes(p, T, delta)}, h.options().dtype(torch::kUInt8));
+    p.scratch = scratch.data_ptr<uint8_t>();
     if (delta) fc::launch_delta_chunk(p, max_len, stream_now());
     else fc::launch_gla_chunk(p, max_len, stream_now());
   } else {

@@ -1,7 +1,633 @@
-#include "hybrid.cuh"
+// Recurrent layers over long runs (bf16 models): chunks of 64 rows, products on the tensor cores.
+//
+// With S the state before a chunk and b the decay accumulated inside it, both recurrences have the form
+//     U = U0 - W S,   O = Q' S + P U,   S <- diag(dec) S + K'^T U
+//   gated linear attention: U = V, no W, b per key channel:
+//       Q' = q e^b,  K' = k e^(b_end - b),  P_ij = sum_d q_id k_jd e^(b_id - b_jd) for j <= i,  dec = e^b_end
+//   gated delta rule (b per head): the writes of a chunk depend on one another through the unit lower triangular
+//       I + L, L_ij = beta_i e^(b_i - b_j) k_i.k_j for j < i; W and U0 solve (I + L) [W | U0] = diag(beta) [e^b k | v]
+//       (Yang, Kautz, Hatamizadeh, "Gated Delta Networks: Improving Mamba2 with Delta Rule"), P_ij = e^(b_i - b_j) q_i.k_j
+// The first kernel computes W, U0, Q', K', P and dec of every chunk in parallel; the second walks the chunks of a
+// run with S in registers.  No exponent is ever positive: P of different 16-row blocks uses the decay at the block
+// border as reference, P inside a block the exact difference.
+//
+// Everything that enters the recurrence stays 32-bit grade: a tensor-core operand is the sum of two bf16 terms
+// (hi + lo) and a product hi hi + hi lo + lo hi, accumulated in fp32.  Operands of the second kernel are stored in the
+// register layout of mma.sync m16n8k16's A fragment (1 KiB per 16 x 16 block: hi, then lo), ready to load.
 #include <stdexcept>
+#include <string>
+
+#include "hybrid.cuh"
+#include "mma.cuh"
+
 namespace fc {
-bool chunk_supported(int D, int V) { return false; }
-void launch_gla_chunk(const StepParams&, int, cudaStream_t) { throw std::runtime_error("no chunked form"); }
-void launch_delta_chunk(const StepParams&, int, cudaStream_t) { throw std::runtime_error("no chunked form"); }
+
+using bf16 = __nv_bfloat16;
+constexpr int CK = 64;                 // rows per chunk
+constexpr int CK_MAX_D = 128;
+constexpr int CK_P = 10;               // lower-triangular 16 x 16 blocks of P
+
+// scratch of one (chunk, head): fragments of Q', K', P, W, then U0 [64, V] and dec [Dp]
+struct ChunkLayout {
+  int kd;                              // 16-column blocks of the key dimension
+  int q, k, p, w;                      // first fragment
+  long long u, dec, bytes;             // byte offsets, total
+};
+__host__ __device__ inline ChunkLayout chunk_layout(int D, int V, bool delta) {
+  ChunkLayout l;
+  l.kd = (D + 15) / 16;
+  l.q = 0;
+  l.k = 4 * l.kd;
+  l.p = 8 * l.kd;
+  l.w = l.p + CK_P;
+  const long long frags = l.w + (delta ? 4 * l.kd : 0);
+  l.u = frags * 1024;
+  l.dec = l.u + (delta ? (long long)CK * ((V + 3) / 4 * 4) * 4 : 0);
+  l.bytes = (l.dec + l.kd * 64 + 255) / 256 * 256;
+  return l;
 }
+bool chunk_supported(int D, int V) { return D % 2 == 0 && D <= CK_MAX_D && V % 2 == 0; }
+long long chunk_scratch_bytes(const StepParams& p, int T, bool delta) {
+  return (long long)(T / CK + p.runs.B) * p.H * chunk_layout(p.D, p.V, delta).bytes;
+}
+
+__device__ __forceinline__ void split_pack(float a, float b, uint32_t& hi, uint32_t& lo) {
+  const __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
+  const float2 f = __bfloat1622float2(h);
+  hi = *reinterpret_cast<const uint32_t*>(&h);
+  lo = pack_bf16(a - f.x, b - f.y);
+}
+struct Frag {                          // hi and lo registers of an A (4) or B (2) operand
+  uint32_t h[4], l[4];
+};
+__device__ __forceinline__ void mma3(float (&c)[4], const Frag& a, uint32_t bh0, uint32_t bh1, uint32_t bl0, uint32_t bl1) {
+  mma_bf16(c, a.l, bh0, bh1);
+  mma_bf16(c, a.h, bl0, bl1);
+  mma_bf16(c, a.h, bh0, bh1);
+}
+__device__ __forceinline__ void store_frag(uint8_t* unit, int f, int lane, const Frag& a) {
+  uint4* d = reinterpret_cast<uint4*>(unit + (long long)f * 1024);
+  d[lane] = make_uint4(a.h[0], a.h[1], a.h[2], a.h[3]);
+  d[32 + lane] = make_uint4(a.l[0], a.l[1], a.l[2], a.l[3]);
+}
+__device__ __forceinline__ Frag load_frag(const uint8_t* unit, int f, int lane) {
+  const uint4* s = reinterpret_cast<const uint4*>(unit + (long long)f * 1024);
+  const uint4 h = __ldcg(s + lane), l = __ldcg(s + 32 + lane);
+  Frag a;
+  a.h[0] = h.x; a.h[1] = h.y; a.h[2] = h.z; a.h[3] = h.w;
+  a.l[0] = l.x; a.l[1] = l.y; a.l[2] = l.z; a.l[3] = l.w;
+  return a;
+}
+// accumulators of a 16 x 16 block (two n8 tiles) as an A fragment
+__device__ __forceinline__ Frag acc_frag(const float (&c0)[4], const float (&c1)[4]) {
+  Frag a;
+  split_pack(c0[0], c0[1], a.h[0], a.l[0]);
+  split_pack(c0[2], c0[3], a.h[1], a.l[1]);
+  split_pack(c1[0], c1[1], a.h[2], a.l[2]);
+  split_pack(c1[2], c1[3], a.h[3], a.l[3]);
+  return a;
+}
+// row pitch (floats) of a [64][Dp] tile: 8 mod 32, so that the 8-byte fragment reads are free of bank conflicts
+__host__ __device__ inline int chunk_pitch(int kd) { return (kd * 16 + 31) / 32 * 32 + 8; }
+
+struct ChunkId {
+  Run run;
+  int n, row0;                         // rows of this chunk, first flat row
+  uint8_t* unit;                       // scratch of (chunk, head)
+};
+__device__ __forceinline__ bool chunk_of(const StepParams& p, const ChunkLayout& l, int c, int h, int b, ChunkId& o) {
+  o.run = get_run(p.runs, b);
+  o.n = min(CK, o.run.len - c * CK);
+  o.row0 = o.run.lo + c * CK;
+  // floor(lo / 64) + b leaves room for ceil(len / 64) chunks before the next run's first
+  o.unit = p.scratch + ((long long)(o.run.lo / CK + b + c) * p.H + h) * l.bytes;
+  return o.run.slot >= 0 && o.n > 0;
+}
+
+constexpr int CA_THREADS = 256;
+
+// blocks (I, J) of the lower triangle in order
+__device__ __forceinline__ void tri_block(int idx, int& I, int& J) {
+  I = idx >= 6 ? 3 : idx >= 3 ? 2 : idx >= 1 ? 1 : 0;
+  J = idx - I * (I + 1) / 2;
+}
+
+// ------------------------------------------------------------------ first kernel, gated delta rule
+__global__ void __launch_bounds__(CA_THREADS)
+delta_chunk_prepare_kernel(const StepParams p) {
+  extern __shared__ float sm[];
+  const ChunkLayout lay = chunk_layout(p.D, p.V, true);
+  const int pitch = chunk_pitch(lay.kd), Dp = lay.kd * 16;
+  float* s_k = sm;                                  // [64][pitch]
+  float* s_q = s_k + CK * pitch;                    // [64][pitch], later W
+  float* s_l = s_q + CK * pitch;                    // [64][64]
+  float* s_g = s_l + CK * CK;                       // accumulated log decay
+  float* s_beta = s_g + CK;
+  float* s_lg = s_beta + CK;
+  const int h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  ChunkId id;
+  if (!chunk_of(p, lay, blockIdx.x, h, blockIdx.z, id)) return;
+  const int K = p.H / p.group, hk = h / p.group;
+  if (tid < CK) {
+    s_lg[tid] = tid < id.n ? p.log_g[(long long)(id.row0 + tid) * p.H + h] : 0.f;
+    s_beta[tid] = tid < id.n ? p.beta[(long long)(id.row0 + tid) * p.H + h] : 0.f;
+  }
+  for (int i = tid; i < CK * (Dp / 2); i += CA_THREADS) {
+    const int r = i / (Dp / 2), c = (i - r * (Dp / 2)) * 2;
+    float2 q = make_float2(0.f, 0.f), k = q;
+    if (r < id.n && c < p.D) {
+      const float* src = p.qk + ((long long)(id.row0 + r) * 2 * K + hk) * p.D + c;
+      q = *reinterpret_cast<const float2*>(src);
+      k = *reinterpret_cast<const float2*>(src + (long long)K * p.D);
+    }
+    *reinterpret_cast<float2*>(s_q + r * pitch + c) = q;
+    *reinterpret_cast<float2*>(s_k + r * pitch + c) = k;
+  }
+  __syncthreads();
+  if (tid < CK) {
+    float g = 0.f;
+    for (int j = 0; j <= tid; ++j) g += s_lg[j];
+    s_g[tid] = g;
+  }
+  __syncthreads();
+  const float g_end = s_g[CK - 1];
+  const int gr = lane >> 2, gc = (lane & 3) * 2;
+  // L and P, block by block
+  for (int idx = warp; idx < CK_P; idx += CA_THREADS / 32) {
+    int I, J;
+    tri_block(idx, I, J);
+    float ak[2][4] = {}, aq[2][4] = {};
+    for (int kk = 0; kk < lay.kd; ++kk) {
+      auto row2 = [&](const float* base, int r, int c) { return *reinterpret_cast<const float2*>(base + r * pitch + kk * 16 + c); };
+      Frag fk, fq;
+#pragma unroll
+      for (int x = 0; x < 4; ++x) {
+        const int r = I * 16 + gr + (x & 1) * 8, c = gc + (x >> 1) * 8;
+        const float2 kv = row2(s_k, r, c), qv = row2(s_q, r, c);
+        split_pack(kv.x, kv.y, fk.h[x], fk.l[x]);
+        split_pack(qv.x, qv.y, fq.h[x], fq.l[x]);
+      }
+#pragma unroll
+      for (int n = 0; n < 2; ++n) {
+        uint32_t bh[2], bl[2];
+#pragma unroll
+        for (int x = 0; x < 2; ++x) {
+          const float2 kv = row2(s_k, J * 16 + n * 8 + gr, gc + x * 8);
+          split_pack(kv.x, kv.y, bh[x], bl[x]);
+        }
+        mma3(ak[n], fk, bh[0], bh[1], bl[0], bl[1]);
+        mma3(aq[n], fq, bh[0], bh[1], bl[0], bl[1]);
+      }
+    }
+#pragma unroll
+    for (int n = 0; n < 2; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int i = I * 16 + gr + (e >> 1) * 8, j = J * 16 + n * 8 + gc + (e & 1);
+        const float f = j <= i ? expf(s_g[i] - s_g[j]) : 0.f;
+        aq[n][e] *= f;
+        s_l[i * CK + j] = j < i ? s_beta[i] * f * ak[n][e] : 0.f;
+      }
+    store_frag(id.unit, lay.p + idx, lane, acc_frag(aq[0], aq[1]));
+  }
+  // Q' and K'^T fragments
+  for (int f = warp; f < 8 * lay.kd; f += CA_THREADS / 32) {
+    Frag a;
+    if (f < 4 * lay.kd) {
+      const int I = f / lay.kd, kk = f - I * lay.kd;
+#pragma unroll
+      for (int x = 0; x < 4; ++x) {
+        const int r = I * 16 + gr + (x & 1) * 8, c = kk * 16 + gc + (x >> 1) * 8;
+        const float e = expf(s_g[r]);
+        split_pack(s_q[r * pitch + c] * e, s_q[r * pitch + c + 1] * e, a.h[x], a.l[x]);
+      }
+      store_frag(id.unit, lay.q + f, lane, a);
+    } else {
+      const int m = (f - 4 * lay.kd) / 4, kt = (f - 4 * lay.kd) & 3;
+#pragma unroll
+      for (int x = 0; x < 4; ++x) {
+        const int d = m * 16 + gr + (x & 1) * 8, r = kt * 16 + gc + (x >> 1) * 8;
+        split_pack(s_k[r * pitch + d] * expf(g_end - s_g[r]), s_k[(r + 1) * pitch + d] * expf(g_end - s_g[r + 1]),
+                   a.h[x], a.l[x]);
+      }
+      store_frag(id.unit, lay.k + f - 4 * lay.kd, lane, a);
+    }
+  }
+  for (int d = tid; d < Dp; d += CA_THREADS) reinterpret_cast<float*>(id.unit + lay.dec)[d] = expf(g_end);
+  __syncthreads();
+  // forward substitution, one right-hand-side column per thread: key columns give W, value columns U0
+  const int V4 = (p.V + 3) / 4 * 4;
+  float* u0 = reinterpret_cast<float*>(id.unit + lay.u);
+  const bf16* v = reinterpret_cast<const bf16*>(p.v) + (long long)id.row0 * p.H * p.V + h * p.V;
+  for (int c = tid; c < Dp + V4; c += CA_THREADS) {
+    float x[CK];
+    const bool key = c < Dp;
+    const int vc = c - Dp;
+#pragma unroll
+    for (int i = 0; i < CK; ++i) {
+      float rhs = 0.f;
+      if (key) rhs = s_k[i * pitch + c] * expf(s_g[i]);
+      else if (i < id.n && vc < p.V) rhs = __bfloat162float(v[(long long)i * p.H * p.V + vc]);
+      x[i] = rhs * s_beta[i];
+    }
+#pragma unroll
+    for (int i = 1; i < CK; ++i) {
+      float a0 = 0.f, a1 = 0.f, a2 = 0.f, a3 = 0.f;
+#pragma unroll
+      for (int j = 0; j < i; j += 4) {
+        const float4 lv = *reinterpret_cast<const float4*>(s_l + i * CK + j);   // entries j >= i of the row are zero
+        a0 = fmaf(lv.x, x[j], a0);
+        if (j + 1 < i) a1 = fmaf(lv.y, x[j + 1], a1);
+        if (j + 2 < i) a2 = fmaf(lv.z, x[j + 2], a2);
+        if (j + 3 < i) a3 = fmaf(lv.w, x[j + 3], a3);
+      }
+      x[i] -= (a0 + a1) + (a2 + a3);
+    }
+#pragma unroll
+    for (int i = 0; i < CK; ++i) {
+      if (key) s_q[i * pitch + c] = x[i];
+      else u0[i * V4 + vc] = x[i];
+    }
+  }
+  __syncthreads();
+  for (int f = warp; f < 4 * lay.kd; f += CA_THREADS / 32) {
+    const int I = f / lay.kd, kk = f - I * lay.kd;
+    Frag a;
+#pragma unroll
+    for (int x = 0; x < 4; ++x) {
+      const float2 w = *reinterpret_cast<const float2*>(s_q + (I * 16 + gr + (x & 1) * 8) * pitch + kk * 16 + gc + (x >> 1) * 8);
+      split_pack(w.x, w.y, a.h[x], a.l[x]);
+    }
+    store_frag(id.unit, lay.w + f, lane, a);
+  }
+}
+
+// ------------------------------------------------------------------ first kernel, gated linear attention
+__global__ void __launch_bounds__(CA_THREADS)
+gla_chunk_prepare_kernel(const StepParams p) {
+  extern __shared__ float sm[];
+  const ChunkLayout lay = chunk_layout(p.D, p.V, false);
+  const int pitch = chunk_pitch(lay.kd), Dp = lay.kd * 16;
+  float* s_k = sm;                                  // [64][pitch]
+  float* s_q = s_k + CK * pitch;
+  float* s_b = s_q + CK * pitch;                    // accumulated decay, log2
+  float* s_d = s_b + CK * pitch;                    // [4][16][18] diagonal blocks of P
+  const int h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  ChunkId id;
+  if (!chunk_of(p, lay, blockIdx.x, h, blockIdx.z, id)) return;
+  const bf16* proj = reinterpret_cast<const bf16*>(p.proj.p);
+  const bf16* zp = reinterpret_cast<const bf16*>(p.z);
+  for (int i = tid; i < CK * Dp; i += CA_THREADS) {
+    const int r = i / Dp, c = i - r * Dp;
+    float q = 0.f, k = 0.f, b = 0.f;
+    if (r < id.n && c < p.D) {
+      const bf16* row = proj + (long long)(id.row0 + r) * p.proj.ld + h * p.D + c;
+      q = __bfloat162float(row[p.off_q]) * p.q_scale;
+      k = __bfloat162float(row[p.off_k]);
+      const float z = __bfloat162float(zp[(long long)(id.row0 + r) * p.ld_z + h * p.D + c]) + p.z_bias[h * p.D + c];
+      b = log_sigmoid_f(z) * p.inv_tau * 1.4426950408889634f;
+    }
+    s_q[r * pitch + c] = q;
+    s_k[r * pitch + c] = k;
+    s_b[r * pitch + c] = b;
+  }
+  __syncthreads();
+  for (int c = tid; c < Dp; c += CA_THREADS) {
+    float acc = 0.f;
+#pragma unroll 8
+    for (int r = 0; r < CK; ++r) {
+      acc += s_b[r * pitch + c];
+      s_b[r * pitch + c] = acc;
+    }
+    reinterpret_cast<float*>(id.unit + lay.dec)[c] = exp2f(acc);
+  }
+  __syncthreads();
+  const int gr = lane >> 2, gc = (lane & 3) * 2;
+  if (warp < 4) {
+    // diagonal block: exact decay differences, lanes over the key channels
+    const int r0 = warp * 16;
+    float* s_p = s_d + warp * 16 * 18;
+    for (int i = 0; i < 16; ++i) {
+      float q[CK_MAX_D / 32], b[CK_MAX_D / 32];
+#pragma unroll
+      for (int x = 0; x < CK_MAX_D / 32; ++x) {
+        const int c = lane + x * 32;
+        q[x] = c < Dp ? s_q[(r0 + i) * pitch + c] : 0.f;
+        b[x] = c < Dp ? s_b[(r0 + i) * pitch + c] : 0.f;
+      }
+#pragma unroll 4
+      for (int j = 0; j <= i; ++j) {
+        float a = 0.f;
+#pragma unroll
+        for (int x = 0; x < CK_MAX_D / 32; ++x) {
+          const int c = lane + x * 32;
+          if (c < Dp) a = fmaf(q[x] * exp2f(b[x] - s_b[(r0 + j) * pitch + c]), s_k[(r0 + j) * pitch + c], a);
+        }
+        a = warp_sum(a);
+        if (lane == 0) s_p[i * 18 + j] = a;
+      }
+      if (lane > i && lane < 16) s_p[i * 18 + lane] = 0.f;
+    }
+    __syncwarp();
+    Frag a;
+#pragma unroll
+    for (int x = 0; x < 4; ++x) {
+      const float* s = s_p + (gr + (x & 1) * 8) * 18 + gc + (x >> 1) * 8;
+      split_pack(s[0], s[1], a.h[x], a.l[x]);
+    }
+    store_frag(id.unit, lay.p + warp * (warp + 1) / 2 + warp, lane, a);
+  } else {
+    // blocks below the diagonal: both factors decayed to the row before block I
+    for (int idx = warp - 4; idx < 6; idx += 4) {
+      const int I = idx >= 3 ? 3 : idx >= 1 ? 2 : 1, J = idx - (I - 1) * I / 2;
+      const float* ref = s_b + (I * 16 - 1) * pitch;
+      float acc[2][4] = {};
+      for (int kk = 0; kk < lay.kd; ++kk) {
+        Frag fq;
+#pragma unroll
+        for (int x = 0; x < 4; ++x) {
+          const int r = (I * 16 + gr + (x & 1) * 8) * pitch, c = kk * 16 + gc + (x >> 1) * 8;
+          split_pack(s_q[r + c] * exp2f(s_b[r + c] - ref[c]), s_q[r + c + 1] * exp2f(s_b[r + c + 1] - ref[c + 1]),
+                     fq.h[x], fq.l[x]);
+        }
+#pragma unroll
+        for (int n = 0; n < 2; ++n) {
+          uint32_t bh[2], bl[2];
+#pragma unroll
+          for (int x = 0; x < 2; ++x) {
+            const int r = (J * 16 + n * 8 + gr) * pitch, c = kk * 16 + gc + x * 8;
+            split_pack(s_k[r + c] * exp2f(ref[c] - s_b[r + c]), s_k[r + c + 1] * exp2f(ref[c + 1] - s_b[r + c + 1]),
+                       bh[x], bl[x]);
+          }
+          mma3(acc[n], fq, bh[0], bh[1], bl[0], bl[1]);
+        }
+      }
+      store_frag(id.unit, lay.p + I * (I + 1) / 2 + J, lane, acc_frag(acc[0], acc[1]));
+    }
+  }
+  for (int f = warp; f < 8 * lay.kd; f += CA_THREADS / 32) {
+    Frag a;
+    if (f < 4 * lay.kd) {
+      const int I = f / lay.kd, kk = f - I * lay.kd;
+#pragma unroll
+      for (int x = 0; x < 4; ++x) {
+        const int o = (I * 16 + gr + (x & 1) * 8) * pitch + kk * 16 + gc + (x >> 1) * 8;
+        split_pack(s_q[o] * exp2f(s_b[o]), s_q[o + 1] * exp2f(s_b[o + 1]), a.h[x], a.l[x]);
+      }
+      store_frag(id.unit, lay.q + f, lane, a);
+    } else {
+      const int m = (f - 4 * lay.kd) / 4, kt = (f - 4 * lay.kd) & 3;
+#pragma unroll
+      for (int x = 0; x < 4; ++x) {
+        const int d = m * 16 + gr + (x & 1) * 8, o = (kt * 16 + gc + (x >> 1) * 8) * pitch + d;
+        const float end = s_b[(CK - 1) * pitch + d];
+        split_pack(s_k[o] * exp2f(end - s_b[o]), s_k[o + pitch] * exp2f(end - s_b[o + pitch]), a.h[x], a.l[x]);
+      }
+      store_frag(id.unit, lay.k + f - 4 * lay.kd, lane, a);
+    }
+  }
+}
+
+// ------------------------------------------------------------------ second kernel
+// CTA = (block of VB value columns, head, request), four warps.  Warp w owns rows 16 w .. 16 w + 15 of a chunk for U and
+// O, and the 16-row blocks w, w + 4 of S in registers; S and U go through shared memory as hi / lo operands.
+constexpr int CB_THREADS = 128;
+
+template <bool DELTA, int VB>
+__global__ void __launch_bounds__(CB_THREADS)
+chunk_scan_kernel(const StepParams p) {
+  constexpr int N8 = VB / 8;
+  constexpr int PITCH = VB + 8;                     // bf16; rows an odd number of 16-byte units apart
+  extern __shared__ uint8_t smem_raw[];
+  const ChunkLayout lay = chunk_layout(p.D, p.V, DELTA);
+  const int kd = lay.kd, Dp = kd * 16;
+  bf16* s_sh = reinterpret_cast<bf16*>(smem_raw);   // [Dp][PITCH] state, hi
+  bf16* s_sl = s_sh + Dp * PITCH;
+  bf16* s_uh = s_sl + Dp * PITCH;                   // [64][PITCH]
+  bf16* s_ul = s_uh + CK * PITCH;
+  const int h = blockIdx.y, b = blockIdx.z, v0 = blockIdx.x * VB;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gr = lane >> 2, gc = (lane & 3) * 2;
+  const Run run = get_run(p.runs, b);
+  if (run.slot < 0 || run.len <= 0) {
+    for (int i = tid; i < run.len * VB; i += CB_THREADS)
+      if (v0 + i % VB < p.V) p.o_raw[((long long)(run.lo + i / VB) * p.H + h) * p.V + v0 + i % VB] = 0.f;
+    return;
+  }
+  float* st = p.state + ((long long)run.slot * p.H + h) * p.D * p.V;
+  float S[2][N8][4];
+  auto state_io = [&](bool load) {
+#pragma unroll
+    for (int mi = 0; mi < 2; ++mi)
+#pragma unroll
+      for (int n = 0; n < N8; ++n)
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+          const int d = (warp + mi * 4) * 16 + gr + half * 8, v = v0 + n * 8 + gc;
+          if (d >= p.D || v >= p.V) continue;       // V is even: a pair of columns exists or not
+          float2* s = reinterpret_cast<float2*>(st + (long long)d * p.V + v);
+          if (load) {
+            const float2 x = *s;
+            S[mi][n][half * 2] = x.x;
+            S[mi][n][half * 2 + 1] = x.y;
+          } else {
+            *s = make_float2(S[mi][n][half * 2], S[mi][n][half * 2 + 1]);
+          }
+        }
+  };
+#pragma unroll
+  for (int mi = 0; mi < 2; ++mi)
+#pragma unroll
+    for (int n = 0; n < N8; ++n) S[mi][n][0] = S[mi][n][1] = S[mi][n][2] = S[mi][n][3] = 0.f;
+  if (run.start > 0) state_io(true);
+  auto put_state = [&]() {
+#pragma unroll
+    for (int mi = 0; mi < 2; ++mi) {
+      if (warp + mi * 4 >= kd) continue;
+#pragma unroll
+      for (int n = 0; n < N8; ++n)
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+          const int o = ((warp + mi * 4) * 16 + gr + half * 8) * PITCH + n * 8 + gc;
+          uint32_t hi, lo;
+          split_pack(S[mi][n][half * 2], S[mi][n][half * 2 + 1], hi, lo);
+          *reinterpret_cast<uint32_t*>(s_sh + o) = hi;
+          *reinterpret_cast<uint32_t*>(s_sl + o) = lo;
+        }
+    }
+  };
+  put_state();
+  __syncthreads();
+  const uint32_t a_sh = smem_u32(s_sh), a_sl = smem_u32(s_sl), a_uh = smem_u32(s_uh), a_ul = smem_u32(s_ul);
+  // B fragments (k16 x n16) of a [rows][PITCH] tile
+  const uint32_t b_off = uint32_t((((lane >> 3) & 1) * 8 + (lane & 7)) * PITCH + (lane >> 4) * 8) * 2;
+  auto ld_b = [&](uint32_t base, int kk, int n2, uint32_t (&r)[4]) {
+    ldsm_x4_t(base + b_off + uint32_t(kk * 16 * PITCH + n2 * 16) * 2, r[0], r[1], r[2], r[3]);
+  };
+  const int V4 = (p.V + 3) / 4 * 4;
+  const int n_chunks = (run.len + CK - 1) / CK;
+  for (int c = 0; c < n_chunks; ++c) {
+    ChunkId id;
+    chunk_of(p, lay, c, h, b, id);
+    const int i0 = warp * 16 + gr;                  // rows i0 and i0 + 8 of the chunk
+    // ---- U0 (or V) and the products with the state before the chunk
+    float u[N8][4], o[N8][4];
+#pragma unroll
+    for (int n = 0; n < N8; ++n)
+#pragma unroll
+      for (int half = 0; half < 2; ++half) {
+        const int i = i0 + half * 8, v = v0 + n * 8 + gc;
+        float2 x = make_float2(0.f, 0.f);
+        if (v < p.V) {
+          if (DELTA)
+            x = __ldcg(reinterpret_cast<const float2*>(reinterpret_cast<const float*>(id.unit + lay.u) + i * V4 + v));
+          else if (i < id.n)
+            x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(
+                reinterpret_cast<const bf16*>(p.proj.p) + (long long)(id.row0 + i) * p.proj.ld + p.off_v + h * p.V + v));
+        }
+        u[n][half * 2] = x.x;
+        u[n][half * 2 + 1] = x.y;
+        o[n][half * 2] = o[n][half * 2 + 1] = 0.f;
+      }
+    Frag fq = load_frag(id.unit, lay.q + warp * kd, lane), fw;
+    if (DELTA) fw = load_frag(id.unit, lay.w + warp * kd, lane);
+    for (int kk = 0; kk < kd; ++kk) {
+      Frag nq = fq, nw = fw;
+      if (kk + 1 < kd) {
+        nq = load_frag(id.unit, lay.q + warp * kd + kk + 1, lane);
+        if (DELTA) nw = load_frag(id.unit, lay.w + warp * kd + kk + 1, lane);
+      }
+      if (DELTA) {                                  // U = U0 - W S
+#pragma unroll
+        for (int x = 0; x < 4; ++x) {
+          fw.h[x] ^= 0x80008000u;
+          fw.l[x] ^= 0x80008000u;
+        }
+      }
+#pragma unroll
+      for (int n2 = 0; n2 < N8 / 2; ++n2) {
+        uint32_t bh[4], bl[4];
+        ld_b(a_sh, kk, n2, bh);
+        ld_b(a_sl, kk, n2, bl);
+#pragma unroll
+        for (int y = 0; y < 2; ++y) {
+          mma3(o[n2 * 2 + y], fq, bh[y * 2], bh[y * 2 + 1], bl[y * 2], bl[y * 2 + 1]);
+          if (DELTA) mma3(u[n2 * 2 + y], fw, bh[y * 2], bh[y * 2 + 1], bl[y * 2], bl[y * 2 + 1]);
+        }
+      }
+      fq = nq;
+      fw = nw;
+    }
+    Frag fp = load_frag(id.unit, lay.p + warp * (warp + 1) / 2, lane);
+    Frag fk = load_frag(id.unit, lay.k + warp * 4, lane);          // warp < kd or an unused fragment of this unit
+#pragma unroll
+    for (int n = 0; n < N8; ++n)
+#pragma unroll
+      for (int half = 0; half < 2; ++half) {
+        const int off = (i0 + half * 8) * PITCH + n * 8 + gc;
+        uint32_t hi, lo;
+        split_pack(u[n][half * 2], u[n][half * 2 + 1], hi, lo);
+        *reinterpret_cast<uint32_t*>(s_uh + off) = hi;
+        if (DELTA) *reinterpret_cast<uint32_t*>(s_ul + off) = lo;  // a bf16 value has no second term
+      }
+    __syncthreads();
+    // ---- O += P U
+    for (int kt = 0; kt <= warp; ++kt) {
+      Frag np = fp;
+      if (kt < warp) np = load_frag(id.unit, lay.p + warp * (warp + 1) / 2 + kt + 1, lane);
+#pragma unroll
+      for (int n2 = 0; n2 < N8 / 2; ++n2) {
+        uint32_t bh[4], bl[4];
+        ld_b(a_uh, kt, n2, bh);
+        if (DELTA) ld_b(a_ul, kt, n2, bl);
+#pragma unroll
+        for (int y = 0; y < 2; ++y) {
+          if (DELTA) {
+            mma3(o[n2 * 2 + y], fp, bh[y * 2], bh[y * 2 + 1], bl[y * 2], bl[y * 2 + 1]);
+          } else {
+            mma_bf16(o[n2 * 2 + y], fp.l, bh[y * 2], bh[y * 2 + 1]);
+            mma_bf16(o[n2 * 2 + y], fp.h, bh[y * 2], bh[y * 2 + 1]);
+          }
+        }
+      }
+      fp = np;
+    }
+    // ---- S = dec S + K'^T U
+    const float* dec = reinterpret_cast<const float*>(id.unit + lay.dec);
+#pragma unroll
+    for (int mi = 0; mi < 2; ++mi) {
+      const int m = warp + mi * 4;
+      if (m >= kd) continue;
+      const float d0 = __ldcg(dec + m * 16 + gr), d1 = __ldcg(dec + m * 16 + gr + 8);
+#pragma unroll
+      for (int n = 0; n < N8; ++n) {
+        S[mi][n][0] *= d0;
+        S[mi][n][1] *= d0;
+        S[mi][n][2] *= d1;
+        S[mi][n][3] *= d1;
+      }
+      for (int kt = 0; kt < 4; ++kt) {
+        Frag nk = fk;
+        if (kt < 3) nk = load_frag(id.unit, lay.k + m * 4 + kt + 1, lane);
+        else if (mi == 0 && m + 4 < kd) nk = load_frag(id.unit, lay.k + (m + 4) * 4, lane);
+#pragma unroll
+        for (int n2 = 0; n2 < N8 / 2; ++n2) {
+          uint32_t bh[4], bl[4];
+          ld_b(a_uh, kt, n2, bh);
+          if (DELTA) ld_b(a_ul, kt, n2, bl);
+#pragma unroll
+          for (int y = 0; y < 2; ++y) {
+            if (DELTA) {
+              mma3(S[mi][n2 * 2 + y], fk, bh[y * 2], bh[y * 2 + 1], bl[y * 2], bl[y * 2 + 1]);
+            } else {
+              mma_bf16(S[mi][n2 * 2 + y], fk.l, bh[y * 2], bh[y * 2 + 1]);
+              mma_bf16(S[mi][n2 * 2 + y], fk.h, bh[y * 2], bh[y * 2 + 1]);
+            }
+          }
+        }
+        fk = nk;
+      }
+    }
+#pragma unroll
+    for (int n = 0; n < N8; ++n)
+#pragma unroll
+      for (int half = 0; half < 2; ++half) {
+        const int i = i0 + half * 8, v = v0 + n * 8 + gc;
+        if (i < id.n && v < p.V)
+          *reinterpret_cast<float2*>(p.o_raw + ((long long)(id.row0 + i) * p.H + h) * p.V + v) =
+              make_float2(o[n][half * 2], o[n][half * 2 + 1]);
+      }
+    put_state();                                    // the products with the old state ended before the barrier above
+    __syncthreads();
+  }
+  state_io(false);
+}
+
+template <bool DELTA>
+static void launch_chunks(const StepParams& p, int max_len, cudaStream_t s) {
+  const ChunkLayout lay = chunk_layout(p.D, p.V, DELTA);
+  const int chunks = (max_len + CK - 1) / CK, pitch = chunk_pitch(lay.kd);
+  const dim3 grid(chunks, p.H, p.runs.B);
+  if (DELTA) {
+    const int smem = (2 * CK * pitch + CK * CK + 3 * CK) * 4;
+    cudaFuncSetAttribute(delta_chunk_prepare_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    delta_chunk_prepare_kernel<<<grid, CA_THREADS, smem, s>>>(p);
+  } else {
+    const int smem = (3 * CK * pitch + 4 * 16 * 18) * 4;
+    cudaFuncSetAttribute(gla_chunk_prepare_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    gla_chunk_prepare_kernel<<<grid, CA_THREADS, smem, s>>>(p);
+  }
+  auto scan = [&](auto kern, int vb) {
+    const int smem = 2 * (lay.kd * 16 + CK) * (vb + 8) * 2;
+    cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    kern<<<dim3((p.V + vb - 1) / vb, p.H, p.runs.B), CB_THREADS, smem, s>>>(p);
+  };
+  // few (request, head) pairs: narrower column blocks for more CTAs
+  if (p.runs.B * p.H * ((p.V + 63) / 64) >= 148) scan(chunk_scan_kernel<DELTA, 64>, 64);
+  else scan(chunk_scan_kernel<DELTA, 32>, 32);
+  const cudaError_t e = cudaGetLastError();
+  if (e != cudaSuccess) throw std::runtime_error(std::string("chunked recurrence: ") + cudaGetErrorString(e));
+}
+void launch_gla_chunk(const StepParams& p, int max_len, cudaStream_t s) { launch_chunks<false>(p, max_len, s); }
+void launch_delta_chunk(const StepParams& p, int max_len, cudaStream_t s) { launch_chunks<true>(p, max_len, s); }
+
+}  // namespace fc
