@@ -78,8 +78,9 @@ __device__ __forceinline__ float silu_f(float x) { return x / (1.f + expf(-x)); 
 // log(sigmoid(x)) and log(1 + exp(x)) without overflow
 __device__ __forceinline__ float log_sigmoid_f(float x) { return fminf(x, 0.f) - log1pf(expf(-fabsf(x))); }
 __device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
+// 0.5 z (1 + tanh y) = z sigmoid(2 y) with y = sqrt(2 / pi) (z + 0.044715 z^3)
 __device__ __forceinline__ float gelu_tanh_f(float z) {
-  return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+  return z / (1.f + expf(-1.5957691216057308f * (z + 0.044715f * z * z * z)));
 }
 
 struct Run {

@@ -131,7 +131,8 @@ struct LatentStore {
   void* gate = nullptr;              // [T, H * V] copy of the gate projection (nullptr: not wanted)
   uint32_t* status = nullptr;
 };
-void launch_latent_store(const LatentStore& p, bool f32, cudaStream_t s);
+void launch_latent_store(const LatentStore& p, bool f32, cudaStream_t s);   // q == nullptr: queries stay in `proj`
+bool latent_rotate_supported(const LatentStore& p);
 
 struct LatentAttn {
   int T = 0, H = 0, rank = 0, R = 0, row_width = 0, block_size = 0, max_blocks = 0, num_blocks = 0;
@@ -159,7 +160,8 @@ void launch_gather_rows(const void* pool, const int* block_tables, const int* ct
 struct LatentPrefill {
   int T = 0, B = 0, H = 0, D = 0, R = 0, V = 0, rank = 0, max_q = 0;
   long long total_kv = 0;
-  const void* q = nullptr;           // [T, H, D + R]
+  const void* q = nullptr;           // [T, ld_q]: D + R columns per head
+  long long ld_q = 0;
   const void* k = nullptr;           // [total_kv, ld_kv]: keys, head by head
   const void* v = nullptr;           // values, head by head, same pitch
   long long ld_kv = 0;

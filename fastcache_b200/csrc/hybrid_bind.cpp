@@ -385,10 +385,21 @@ Tensor latent_attention(const Tensor& h, const Tensor& w, const std::vector<int6
     if (fc::latent_prefill_supported(a)) {
       check_i32(*cu_q, "cu_q", B + 1);
       check_i32(*cu_kv, "cu_kv", B + 1);
-      Tensor q = torch::empty({T, H, D + R}, h.options()), gate = torch::empty({T, H * V}, h.options());
-      st.q = q.data_ptr();
+      Tensor q, gate;
       const bool partial = st.proj.splits > 1;
-      if (partial) st.gate = gate.data_ptr();
+      if (fc::latent_rotate_supported(st)) {
+        a.q = reinterpret_cast<const char*>(st.proj.p) + (long long)st.off_q * 2;
+        a.ld_q = st.proj.ld;
+      } else {
+        q = torch::empty({T, H, D + R}, h.options());
+        st.q = q.data_ptr();
+        a.q = st.q;
+        a.ld_q = (long long)H * (D + R);
+      }
+      if (partial) {
+        gate = torch::empty({T, H * V}, h.options());
+        st.gate = gate.data_ptr();
+      }
       fc::launch_latent_store(st, false, stream_now());
       Tensor rows = torch::empty({total_kv, pool.size(2)}, h.options());
       fc::launch_gather_rows(pool.data_ptr(), block_tables.data_ptr<int>(), ctx.data_ptr<int>(), cu_kv->data_ptr<int>(),
@@ -396,7 +407,6 @@ Tensor latent_attention(const Tensor& h, const Tensor& w, const std::vector<int6
                              int(block_tables.size(1)), int(pool.size(0)), false, ws.status, stream_now());
       Tensor kv;
       project(rows.narrow(1, 0, w_kv.size(1)), w_kv, c10::nullopt, false, kv);
-      a.q = q.data_ptr();
       a.k = kv.data_ptr();
       a.v = reinterpret_cast<const char*>(kv.data_ptr()) + off_uv * 2;
       a.ld_kv = kv.size(1);

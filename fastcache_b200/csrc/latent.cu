@@ -86,8 +86,73 @@ latent_store_kernel(const LatentStore p) {
   }
 }
 
+// The same for many rows of a finished projection whose queries are then read where they are: the rotated parts are
+// rotated in place, nothing is copied.  Four columns per access (sizes and offsets multiples of 4); one warp per row for
+// the cache row, the other warps rotate the heads.
+constexpr int LR_WARPS = 4;
+template <typename T>
+__global__ void __launch_bounds__(LR_WARPS * 32)
+latent_rotate_kernel(const LatentStore p) {
+  extern __shared__ float cs[];
+  const int half = p.rot_dims / 2, quads = half / 4;
+  pdl_launch_dependents();
+  pdl_wait();
+  const long long t = blockIdx.x;
+  const int tid = threadIdx.x, lane = tid & 31;
+  const double pos = double(p.positions[t]), l2b = log2(p.base);
+  for (int i = tid; i < half; i += LR_WARPS * 32) rope_angle(pos, l2b, i, p.rot_dims, cs[i], cs[half + i]);
+  __syncthreads();
+  T* row = const_cast<T*>(reinterpret_cast<const T*>(p.proj.p)) + t * p.proj.ld;
+  auto rotate = [&](const T* su, T* du, int i0) {            // quads at columns i0 and half + i0 of a rotated part
+    ProjSrc s;
+    s.p = su;
+    const float4 u = proj_at4<T>(s, 0, i0), v = proj_at4<T>(s, 0, half + i0);
+    const float4 c = *reinterpret_cast<const float4*>(cs + i0), d = *reinterpret_cast<const float4*>(cs + half + i0);
+    store4(du + i0, u.x * c.x - v.x * d.x, u.y * c.y - v.y * d.y, u.z * c.z - v.z * d.z, u.w * c.w - v.w * d.w);
+    store4(du + half + i0, v.x * c.x + u.x * d.x, v.y * c.y + u.y * d.y, v.z * c.z + u.z * d.z, v.w * c.w + u.w * d.w);
+  };
+  for (int i = tid; i < p.H * quads; i += LR_WARPS * 32) {
+    const int h = i / quads;
+    T* q = row + p.off_q + h * (p.D + p.R) + p.D;
+    rotate(q, q, (i - h * quads) * 4);
+  }
+  if (p.off_kv < 0 || tid >= 32) return;
+  const int slot = p.slots[t];
+  if (slot < 0) return;
+  if (slot >= p.num_rows) {
+    if (lane == 0) report(p.status, ST_BAD_INDEX);
+    return;
+  }
+  T* dst = reinterpret_cast<T*>(p.pool) + (long long)slot * p.row_width;
+  ProjSrc s;
+  s.p = row + p.off_kv;
+  float ss = 0.f;
+  for (int c = lane * 4; c < p.rank; c += 128) {
+    const float4 v = proj_at4<T>(s, 0, c);
+    ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+  }
+  const float inv = rsqrtf(warp_sum(ss) / float(p.rank) + p.eps);
+  for (int c = lane * 4; c < p.rank; c += 128) {
+    const float4 v = proj_at4<T>(s, 0, c), w = *reinterpret_cast<const float4*>(p.norm_w + c);
+    store4(dst + c, v.x * inv * w.x, v.y * inv * w.y, v.z * inv * w.z, v.w * inv * w.w);
+  }
+  for (int i = lane; i < quads; i += 32) rotate(row + p.off_kv + p.rank, dst + p.rank, i * 4);
+}
+bool latent_rotate_supported(const LatentStore& p) {
+  return p.proj.splits <= 1 && p.rot_dims == p.R && p.R % 8 == 0 && p.D % 4 == 0 && p.rank % 4 == 0;
+}
+
 void launch_latent_store(const LatentStore& p, bool f32, cudaStream_t s) {
   if (p.T == 0) return;
+  if (p.q == nullptr) {                                      // in place
+    if (!latent_rotate_supported(p)) throw std::runtime_error("latent store: queries cannot stay in place");
+    const size_t smem = size_t(p.rot_dims) * 4;
+    if (f32) launch_pdl(PDL_ROPE, latent_rotate_kernel<float>, dim3(p.T), dim3(LR_WARPS * 32), smem, s, p);
+    else launch_pdl(PDL_ROPE, latent_rotate_kernel<bf16>, dim3(p.T), dim3(LR_WARPS * 32), smem, s, p);
+    const cudaError_t e = cudaGetLastError();
+    if (e != cudaSuccess) throw std::runtime_error(std::string("latent store: ") + cudaGetErrorString(e));
+    return;
+  }
   const int work = p.H * (p.D + p.R);
   const int parts = p.T >= 592 ? 1 : std::max(1, std::min(16, (work + LS_THREADS * 4 - 1) / (LS_THREADS * 4)));
   const dim3 grid(p.T, parts);

@@ -4,10 +4,10 @@
 // Grid (query row, group of 16 * MT heads, split of the context).  A CTA streams 64-row tiles of the cache through a
 // two-stage TMA ring (128-byte swizzle, boxes that never straddle a page); one tile in shared memory is both the keys
 // and the values of all its heads, so a row is read once.  Per tile:
-//   scores   warp w: 16 keys (w & 3) against all heads, half of the columns (w >> 2), mma.sync m16n8k16; the two halves
-//            are added when they are read back
-//   softmax  16 / MT threads per head, running maximum and sum in registers, P to shared memory as bf16
-//   values   warp w owns the latent columns of 16-column groups w, w + 8, ...; P V accumulates in registers
+//   scores   warp w: 16 keys (w & 3) against all heads, a quarter of the columns (w >> 2), mma.sync m16n8k16; the
+//            quarters are added when they are read back
+//   softmax  32 / MT threads per head, running maximum and sum in registers, P to shared memory as bf16
+//   values   warp w owns the latent columns of 16-column groups w, w + 16, ...; P V accumulates in registers
 // With several splits a CTA writes normalised partials with their log-sum-exp and a second kernel merges them.
 //
 // Also here: the per-head products around it (queries into the latent space, outputs out of it).
@@ -23,7 +23,8 @@
 namespace fc {
 
 using bf16 = __nv_bfloat16;
-constexpr int LD_TILE = 64, LD_STAGES = 2, LD_THREADS = 256;
+constexpr int LD_TILE = 64, LD_STAGES = 2, LD_WARPS = 16, LD_THREADS = LD_WARPS * 32;
+constexpr int LD_PARTS = LD_WARPS / 4;           // column ranges of the scores
 constexpr int LD_SUB = LD_TILE * 128;             // bytes of a [64 rows x 64 columns] sub-tile
 constexpr int LD_MAX_SPLITS = 32;
 
@@ -44,8 +45,8 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm, const LatentAttn p,
   uint8_t* s_kv = smem;                                            // [LD_STAGES]
   uint8_t* s_q = s_kv + LD_STAGES * stage_bytes;                   // [nc][HR][128 B]
   uint8_t* s_p = s_q + nc * HR * 128;                              // [HR][128 B]
-  float* s_s = reinterpret_cast<float*>(s_p + HR * 128);           // [2][HR][LD_TILE + 4]
-  float* s_cor = s_s + 2 * HR * (LD_TILE + 4);                     // [HR]
+  float* s_s = reinterpret_cast<float*>(s_p + HR * 128);           // [LD_PARTS][HR][LD_TILE + 4]
+  float* s_cor = s_s + LD_PARTS * HR * (LD_TILE + 4);                     // [HR]
   float* s_l = s_cor + HR;                                         // [HR]
   uint64_t* full = reinterpret_cast<uint64_t*>(s_l + HR);          // [LD_STAGES]
   constexpr int SLD = LD_TILE + 4;
@@ -115,9 +116,9 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm, const LatentAttn p,
       for (int e = 0; e < 8; ++e) o[m][n][e >> 2][e & 3] = 0.f;
   const int srow = tid / TPR, sk0 = (tid % TPR) * KPT;             // softmax: head row and first key of this thread
   float m_run = -INFINITY, l_run = 0.f;
-  const int ksteps = (p.row_width + 15) / 16, khalf = (ksteps + 1) / 2;
+  const int ksteps = (p.row_width + 15) / 16, kpart = (ksteps + LD_PARTS - 1) / LD_PARTS;
   const int kg = (warp & 3) * 16, part = warp >> 2;
-  const int k_lo = part * khalf, k_hi = min(ksteps, k_lo + khalf);
+  const int k_lo = part * kpart, k_hi = min(ksteps, k_lo + kpart);
   const uint32_t q_base = smem_u32(s_q), p_base = smem_u32(s_p);
   bool alive = true;
   for (int it = 0; it < n_tiles; ++it) {
@@ -163,7 +164,9 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm, const LatentAttn p,
       float mx = -INFINITY;
 #pragma unroll
       for (int i = 0; i < KPT; ++i) {
-        const float s = s_s[srow * SLD + sk0 + i] + s_s[(HR + srow) * SLD + sk0 + i];
+        float s = 0.f;
+#pragma unroll
+        for (int x = 0; x < LD_PARTS; ++x) s += s_s[(x * HR + srow) * SLD + sk0 + i];
         v[i] = sk0 + i < valid ? s * scale_log2 : -INFINITY;
         mx = fmaxf(mx, v[i]);
       }
@@ -207,7 +210,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm, const LatentAttn p,
                 a[m][3]);
 #pragma unroll
       for (int n = 0; n < NPW; ++n) {
-        const int cg = warp + n * 8;                               // 16-column group of the latent
+        const int cg = warp + n * LD_WARPS;                               // 16-column group of the latent
         if (cg * 16 >= p.rank) continue;
         uint32_t b0, b1, b2, b3;
         ldsm_x4_t(kv + ld_swz(LD_TILE, ks * 16 + (mat & 1) * 8 + (lane & 7), cg * 2 + (mat >> 1)), b0, b1, b2, b3);
@@ -241,7 +244,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm, const LatentAttn p,
       const long long row = (long long)t * p.H + h0 + r;
 #pragma unroll
       for (int n = 0; n < NPW; ++n) {
-        const int cg = warp + n * 8;
+        const int cg = warp + n * LD_WARPS;
         if (cg * 16 >= p.rank) continue;
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
@@ -292,7 +295,7 @@ static int ld_box_rows(int block_size) {
 }
 static int ld_nc(const LatentAttn& p) { return (p.row_width + 63) / 64; }
 static int ld_smem(int mt, int nc) {
-  return LD_STAGES * nc * LD_SUB + nc * mt * 16 * 128 + mt * 16 * 128 + 2 * mt * 16 * (LD_TILE + 4) * 4 +
+  return LD_STAGES * nc * LD_SUB + nc * mt * 16 * 128 + mt * 16 * 128 + LD_PARTS * mt * 16 * (LD_TILE + 4) * 4 +
          2 * mt * 16 * 4 + 64 + 1024;
 }
 static int ld_mt(const LatentAttn& p) {
@@ -328,9 +331,8 @@ void launch_latent_decode(const LatentAttn& p, cudaStream_t s) {
   };
   auto pick = [&](auto m) {
     constexpr int MT = decltype(m)::value;
-    if (p.rank <= 128) go(latent_decode_kernel<MT, 1>);
-    else if (p.rank <= 256) go(latent_decode_kernel<MT, 2>);
-    else go(latent_decode_kernel<MT, 4>);
+    if (p.rank <= 256) go(latent_decode_kernel<MT, 1>);
+    else go(latent_decode_kernel<MT, 2>);
   };
   if (mt == 1) pick(std::integral_constant<int, 1>{});
   else if (mt == 2) pick(std::integral_constant<int, 2>{});
@@ -342,66 +344,99 @@ void launch_latent_decode(const LatentAttn& p, cudaStream_t s) {
 }
 
 // ------------------------------------------------------------------ per-head products
-// y[g][m, n] = sum_k x[g][m, k] w[g][n, k] for few rows m: bound by reading w once.  One warp per 16 rows of w (they are
-// the M side of mma.sync m16n8k16, so no row of the tensor-core tile is wasted on a small batch); NT n8-tiles hold up to
-// 8 * NT batch rows.  Four warps of a CTA take consecutive 16-row groups.
-constexpr int HL_WARPS = 4;
+// y[g][m, n] = sum_k x[g][m, k] w[g][n, k] for decode-size batches.  CTA: 64 rows n of w (the M side of mma.sync m16n8k16,
+// 16 per warp, so that no row of the tensor-core tile is wasted on a small batch) x NT * 8 rows m of x; both operands
+// come in 64-column steps through a three-stage cp.async ring.
+constexpr int HL_N = 64, HL_K = 64, HL_STAGES = 3, HL_THREADS = 128;
 template <int NT>
-__global__ void __launch_bounds__(HL_WARPS * 32)
+__global__ void __launch_bounds__(HL_THREADS)
 head_linear_kernel(const SimtLinear a) {
+  constexpr int XR = NT * 8;                                       // rows of x
+  __shared__ __align__(128) uint8_t s_w[HL_STAGES][HL_N * 128], s_x[HL_STAGES][XR * 128];
   pdl_launch_dependents();
-  const int g = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int n0 = (blockIdx.x * HL_WARPS + warp) * 16, m0 = blockIdx.z * NT * 8;
-  const int r = lane >> 2, c = (lane & 3) * 2;
+  const int g = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int n0 = blockIdx.x * HL_N, m0 = blockIdx.z * XR;
   const bf16* w = reinterpret_cast<const bf16*>(a.w) + g * a.gw;
   const bf16* x = reinterpret_cast<const bf16*>(a.x) + g * a.gx;
+  const int steps = (a.K + HL_K - 1) / HL_K;
+  auto load = [&](int st, bool wpart, bool xpart) {
+    const int k0 = st * HL_K;
+    if (wpart)
+      for (int i = tid; i < HL_N * 8; i += HL_THREADS) {
+        const int r = i >> 3, c = i & 7;
+        const bool ok = n0 + r < a.N && k0 + c * 8 < a.K;
+        cp_async16(smem_u32(s_w[st % HL_STAGES]) + r * 128 + ((c ^ (r & 7)) << 4),
+                   ok ? w + (long long)(n0 + r) * a.ldw + k0 + c * 8 : w, ok);
+      }
+    if (xpart)
+      for (int i = tid; i < XR * 8; i += HL_THREADS) {
+        const int r = i >> 3, c = i & 7;
+        const bool ok = m0 + r < a.M && k0 + c * 8 < a.K;
+        cp_async16(smem_u32(s_x[st % HL_STAGES]) + r * 128 + ((c ^ (r & 7)) << 4),
+                   ok ? x + (long long)(m0 + r) * a.ldx + k0 + c * 8 : x, ok);
+      }
+  };
+  load(0, true, false);                                            // weights do not depend on the kernel before
+  if (steps > 1) load(1, true, false);
+  pdl_wait();
+  load(0, false, true);
+  cp_async_commit();
+  if (steps > 1) load(1, false, true);
+  cp_async_commit();
   float acc[NT][4];
 #pragma unroll
   for (int i = 0; i < NT; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
-  pdl_wait();
-  if (n0 < a.N) {
-    const bool w0ok = n0 + r < a.N, w1ok = n0 + r + 8 < a.N;
-    const bf16 *w0 = w + (long long)(n0 + r) * a.ldw + c, *w1 = w0 + 8 * a.ldw;
-    auto ld = [](const bf16* q, bool ok) { return ok ? __ldcg(reinterpret_cast<const uint32_t*>(q)) : 0u; };
-#pragma unroll 2
-    for (int k = 0; k < a.K; k += 16) {
-      const bool hi = k + 8 < a.K;                                 // K is a multiple of 8
-      const uint32_t af[4] = {ld(w0 + k, w0ok), ld(w1 + k, w1ok), ld(w0 + k + 8, w0ok && hi), ld(w1 + k + 8, w1ok && hi)};
+  const int mat = lane >> 3;
+  for (int st = 0; st < steps; ++st) {
+    cp_async_wait<1>();
+    __syncthreads();
+    if (st + 2 < steps) load(st + 2, true, true);
+    cp_async_commit();
+    const uint32_t ws = smem_u32(s_w[st % HL_STAGES]), xs = smem_u32(s_x[st % HL_STAGES]);
 #pragma unroll
-      for (int i = 0; i < NT; ++i) {
-        const int m = m0 + i * 8 + r;
-        const bf16* xr = x + (long long)m * a.ldx + c + k;
-        mma_bf16(acc[i], af, ld(xr, m < a.M), ld(xr + 8, m < a.M && hi));
+    for (int kk = 0; kk < HL_K / 16; ++kk) {
+      uint32_t af[4];
+      {
+        const int r = warp * 16 + (mat & 1) * 8 + (lane & 7), c = kk * 2 + (mat >> 1);
+        ldsm_x4(ws + r * 128 + ((c ^ (r & 7)) << 4), af[0], af[1], af[2], af[3]);
+      }
+#pragma unroll
+      for (int i = 0; i < NT; i += 2) {
+        uint32_t b0, b1, b2, b3;
+        const int r = min(i * 8 + (mat >> 1) * 8 + (lane & 7), XR - 1), c = kk * 2 + (mat & 1);
+        ldsm_x4(xs + r * 128 + ((c ^ (r & 7)) << 4), b0, b1, b2, b3);
+        mma_bf16(acc[i], af, b0, b1);
+        if (i + 1 < NT) mma_bf16(acc[i + 1], af, b2, b3);
       }
     }
-    const bool gated = a.gate.p != nullptr || a.gate.part != nullptr;
-    bf16* y = reinterpret_cast<bf16*>(a.y) + g * a.gy;
-#pragma unroll
-    for (int i = 0; i < NT; ++i)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int n = n0 + r + (e >> 1) * 8, m = m0 + i * 8 + c + (e & 1);
-        if (n >= a.N || m >= a.M) continue;
-        float v = acc[i][e];
-        if (gated) v *= sigmoid_f(proj_at<bf16>(a.gate, m, a.gate_off + g * a.N + n));
-        y[(long long)m * a.ldy + n] = __float2bfloat16(v);
-      }
   }
-  if (a.y_pad > a.groups * a.N && g == 0 && blockIdx.x == 0)
-    for (int i = threadIdx.x; i < NT * 8 * (a.y_pad - a.groups * a.N); i += HL_WARPS * 32) {
-      const int pad = a.y_pad - a.groups * a.N, m = m0 + i / pad;
-      if (m < a.M) reinterpret_cast<bf16*>(a.y)[(long long)m * a.ldy + a.groups * a.N + i % pad] = __float2bfloat16(0.f);
+  const bool gated = a.gate.p != nullptr || a.gate.part != nullptr;
+  bf16* y = reinterpret_cast<bf16*>(a.y) + g * a.gy;
+#pragma unroll
+  for (int i = 0; i < NT; ++i)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int n = n0 + warp * 16 + (lane >> 2) + (e >> 1) * 8, m = m0 + i * 8 + (lane & 3) * 2 + (e & 1);
+      if (n >= a.N || m >= a.M) continue;
+      float v = acc[i][e];
+      if (gated) v *= sigmoid_f(proj_at<bf16>(a.gate, m, a.gate_off + g * a.N + n));
+      y[(long long)m * a.ldy + n] = __float2bfloat16(v);
     }
+  const int pad = a.y_pad - a.groups * a.N;
+  if (pad > 0 && g == 0 && blockIdx.x == 0)
+    for (int i = tid; i < XR * pad; i += HL_THREADS)
+      if (m0 + i / pad < a.M)
+        reinterpret_cast<bf16*>(a.y)[(long long)(m0 + i / pad) * a.ldy + a.groups * a.N + i % pad] = __float2bfloat16(0.f);
 }
 
 bool head_linear_mma_supported(const SimtLinear& a) {
-  return a.K % 8 == 0 && a.ldx % 2 == 0 && a.ldw % 2 == 0 && a.gx % 2 == 0 && a.gw % 2 == 0 && a.bias == nullptr;
+  return a.K % 8 == 0 && a.ldx % 8 == 0 && a.ldw % 8 == 0 && a.gx % 8 == 0 && a.gw % 8 == 0 && a.bias == nullptr;
 }
 void launch_head_linear_mma(const SimtLinear& a, cudaStream_t s) {
   if (a.M == 0 || a.N == 0) return;
   auto go = [&](auto kern, int rows) {
-    launch_pdl(PDL_SKINNY_GEMM, kern, dim3((a.N + HL_WARPS * 16 - 1) / (HL_WARPS * 16), a.groups, (a.M + rows - 1) / rows),
-               dim3(HL_WARPS * 32), 0, s, a);
+    launch_pdl(PDL_SKINNY_GEMM, kern, dim3((a.N + HL_N - 1) / HL_N, a.groups, (a.M + rows - 1) / rows), dim3(HL_THREADS), 0,
+               s, a);
   };
   if (a.M <= 8) go(head_linear_kernel<1>, 8);
   else if (a.M <= 32) go(head_linear_kernel<4>, 32);

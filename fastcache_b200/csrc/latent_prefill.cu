@@ -344,8 +344,8 @@ void launch_latent_prefill(const LatentPrefill& p, cudaStream_t s) {
   LpMaps tm;
   const uint64_t Q = uint64_t(p.D + p.R);
   const bf16* q = reinterpret_cast<const bf16*>(p.q);
-  tm.qn = make_tmap_bf16_3d(q, p.D, p.H, p.T, Q, Q * p.H, 64, 1, LP_BM);
-  tm.qr = make_tmap_bf16_3d(q + p.D, p.R, p.H, p.T, Q, Q * p.H, 64, 1, LP_BM);
+  tm.qn = make_tmap_bf16_3d(q, p.D, p.H, p.T, Q, p.ld_q, 64, 1, LP_BM);
+  tm.qr = make_tmap_bf16_3d(q + p.D, p.R, p.H, p.T, Q, p.ld_q, 64, 1, LP_BM);
   tm.kn = make_tmap_bf16_3d(p.k, p.D, p.H, p.total_kv, p.D, p.ld_kv, 64, 1, LP_BN);
   tm.v = make_tmap_bf16_3d(p.v, p.V, p.H, p.total_kv, p.V, p.ld_kv, 64, 1, LP_BN);
   tm.kr = make_tmap_bf16_2d(p.rot, p.total_kv, p.R, p.ld_rot, LP_BN, 64);

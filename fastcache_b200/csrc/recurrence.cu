@@ -294,6 +294,21 @@ gated_head_norm_kernel(const float* __restrict__ o_raw, const ProjSrc proj, int 
   const int h = int(u - t * H);
   const float* o = o_raw + u * V;
   float ss = 0.f;
+  if ((V & 3) == 0 && (off_g & 3) == 0) {
+    for (int c = lane * 4; c < V; c += 128) {
+      const float4 x = *reinterpret_cast<const float4*>(o + c);
+      ss += x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
+    }
+    const float inv = rsqrtf(warp_sum(ss) / float(V) + eps);
+    for (int c = lane * 4; c < V; c += 128) {
+      const float4 x = *reinterpret_cast<const float4*>(o + c), w = *reinterpret_cast<const float4*>(norm_w + c);
+      const float4 g = proj_at4<T>(proj, t, off_g + h * V + c);
+      store4(out + t * ld_out + h * V + c, x.x * inv * w.x * silu_f(g.x), x.y * inv * w.y * silu_f(g.y),
+             x.z * inv * w.z * silu_f(g.z), x.w * inv * w.w * silu_f(g.w));
+    }
+    if (h == 0 && lane < int(ld_out) - H * V) out[t * ld_out + H * V + lane] = Elem<T>::put(0.f);
+    return;
+  }
   for (int c = lane; c < V; c += 32) ss += o[c] * o[c];
   const float inv = rsqrtf(warp_sum(ss) / float(V) + eps);
   for (int c = lane; c < V; c += 32)
@@ -383,6 +398,97 @@ delta_prepare_kernel(const DeltaPrepare p, int units, int advance) {
   for (int c = c0 + lane; c < min(c0 + 128, HV); c += 32) dst[c] = Elem<T>::put(conv(2 * p.K * p.D + c));
 }
 
+// The same for long runs: a warp takes 16 consecutive rows of 128 channels (four per lane) and slides the window of the
+// convolution over them in registers, so that every input is read about once.  Heads of up to 128 channels sit in LPH
+// lanes (a power of two), several to a warp.  Up to four taps.
+constexpr int DR_ROWS = 16;
+template <typename T>
+__global__ void __launch_bounds__(256)
+delta_prepare_rows_kernel(const DeltaPrepare p, int units, int lph, int qk_units) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t0 = blockIdx.x * DR_ROWS, u = blockIdx.y * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (u >= units) return;
+  const int t1 = min(p.T, t0 + DR_ROWS), C = 2 * p.K * p.D + p.H * p.V;
+  if (u == units - 1) {
+    for (int i = lane; i < (t1 - t0) * p.H; i += 32) {
+      const int t = t0 + i / p.H, h = i % p.H;
+      p.log_g[(long long)t * p.H + h] = -expf(p.a_log[h]) * softplus_f(proj_at<T>(p.proj, t, p.off_a + h) + p.dt_bias[h]);
+      p.beta[(long long)t * p.H + h] = sigmoid_f(proj_at<T>(p.proj, t, p.off_b + h));
+    }
+    return;
+  }
+  const bool is_qk = u < qk_units;
+  int head = 0, c;
+  bool on;
+  if (is_qk) {                                               // head of q | k, channel inside it
+    head = u * (32 / lph) + lane / lph;
+    const int d = (lane % lph) * 4;
+    on = head < 2 * p.K && d < p.D;
+    c = head * p.D + d;
+  } else {
+    const int x = (u - qk_units) * 128 + lane * 4;
+    on = x < p.H * p.V;
+    c = 2 * p.K * p.D + x;
+  }
+  float w[4][4];                                             // [tap: 0 = current row][channel]
+#pragma unroll
+  for (int j = 0; j < 4; ++j)
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+      w[j][i] = on && j < p.taps ? p.conv_w[(long long)(c + i) * p.taps + p.taps - 1 - j] : 0.f;
+  float x1[4] = {}, x2[4] = {}, x3[4] = {};                  // inputs one, two and three rows back
+  int b = -1;
+  Run run{};
+  const float scale_q = is_qk && head < p.K ? p.q_scale : 1.f;
+  auto back = [&](int t, int j, float (&x)[4]) {             // input j rows before row t of the current run
+    x[0] = x[1] = x[2] = x[3] = 0.f;
+    const int i = t - run.lo - j;
+    if (!on || j >= p.taps || run.slot < 0) return;
+    if (i >= 0) {
+      const float4 v = proj_at4<T>(p.proj, t - j, c);
+      x[0] = v.x; x[1] = v.y; x[2] = v.z; x[3] = v.w;
+    } else if (run.start + i >= 0) {
+      const float* s = p.conv_state + ((long long)run.slot * (p.taps - 1) + p.taps - 1 + i) * C + c;
+#pragma unroll
+      for (int k = 0; k < 4; ++k) x[k] = s[k];
+    }
+  };
+  float4 nxt = on ? proj_at4<T>(p.proj, t0, c) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 2
+  for (int t = t0; t < t1; ++t) {
+    const int bt = p.row_seq[t];
+    if (bt != b) {
+      b = bt;
+      run = get_run(p.runs, b);
+      back(t, 1, x1);
+      back(t, 2, x2);
+      back(t, 3, x3);
+    }
+    const float x0[4] = {nxt.x, nxt.y, nxt.z, nxt.w};
+    if (on && t + 1 < t1) nxt = proj_at4<T>(p.proj, t + 1, c);
+    float y[4], ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      y[i] = silu_f(fmaf(x3[i], w[3][i], fmaf(x2[i], w[2][i], fmaf(x1[i], w[1][i], x0[i] * w[0][i]))));
+      ss += y[i] * y[i];
+      x3[i] = x2[i];
+      x2[i] = x1[i];
+      x1[i] = x0[i];
+    }
+    if (is_qk) {
+      if (!on) ss = 0.f;
+      for (int x = 1; x < lph; x <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, x);
+      const float inv = rsqrtf(ss + p.unit_eps) * scale_q;
+      if (on)
+        *reinterpret_cast<float4*>(p.qk + (long long)t * 2 * p.K * p.D + c) =
+            make_float4(y[0] * inv, y[1] * inv, y[2] * inv, y[3] * inv);
+    } else if (on) {
+      store4(reinterpret_cast<T*>(p.v) + (long long)t * p.H * p.V + c - 2 * p.K * p.D, y[0], y[1], y[2], y[3]);
+    }
+  }
+}
+
 template <typename T>
 __global__ void __launch_bounds__(256)
 conv_state_kernel(const DeltaPrepare p) {
@@ -403,6 +509,17 @@ conv_state_kernel(const DeltaPrepare p) {
 
 template <typename T>
 static void delta_prepare_t(const DeltaPrepare& p, cudaStream_t s) {
+  if (p.runs.cu != nullptr && p.T >= 256 && p.taps <= 4 && p.D % 4 == 0 && p.D <= 128 && p.H * p.V % 4 == 0) {
+    int lph = 1;
+    while (lph * 4 < p.D) lph <<= 1;
+    const int qk_units = (2 * p.K * lph + 31) / 32, units = qk_units + (p.H * p.V + 127) / 128 + 1;
+    launch_pdl(PDL_PARTIALS, delta_prepare_rows_kernel<T>, dim3((p.T + DR_ROWS - 1) / DR_ROWS, (units + 7) / 8),
+               dim3(256), 0, s, p, units, lph, qk_units);
+    if (p.taps > 1)
+      launch_pdl(PDL_PARTIALS, conv_state_kernel<T>, dim3((2 * p.K * p.D + p.H * p.V + 255) / 256, p.runs.B), dim3(256),
+                 0, s, p);
+    return;
+  }
   const int units = 2 * p.K + (p.H * p.V + 127) / 128 + 1;
   const int advance = p.runs.cu == nullptr ? 1 : 0;
   launch_pdl(PDL_PARTIALS, delta_prepare_kernel<T>, dim3(p.T, (units + 7) / 8), dim3(256), 0, s, p, units, advance);

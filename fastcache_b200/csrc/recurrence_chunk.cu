@@ -8,8 +8,7 @@
 //       I + L, L_ij = beta_i e^(b_i - b_j) k_i.k_j for j < i; W and U0 solve (I + L) [W | U0] = diag(beta) [e^b k | v]
 //       (Yang, Kautz, Hatamizadeh, "Gated Delta Networks: Improving Mamba2 with Delta Rule"), P_ij = e^(b_i - b_j) q_i.k_j
 // The first kernel computes W, U0, Q', K', P and dec of every chunk in parallel; the second walks the chunks of a
-// run with S in registers.  No exponent is ever positive: P of different 16-row blocks uses the decay at the block
-// border as reference, P inside a block the exact difference.
+// run with S in registers.
 //
 // Everything that enters the recurrence stays 32-bit grade: a tensor-core operand is the sum of two bf16 terms
 // (hi + lo) and a product hi hi + hi lo + lo hi, accumulated in fp32.  Operands of the second kernel are stored in the
@@ -119,8 +118,8 @@ delta_chunk_prepare_kernel(const StepParams p) {
   const ChunkLayout lay = chunk_layout(p.D, p.V, true);
   const int pitch = chunk_pitch(lay.kd), Dp = lay.kd * 16;
   float* s_k = sm;                                  // [64][pitch]
-  float* s_q = s_k + CK * pitch;                    // [64][pitch], later W
-  float* s_l = s_q + CK * pitch;                    // [64][64]
+  float* s_q = s_k + CK * pitch;                    // [64][pitch], later columns of U0
+  float* s_l = s_q + CK * max(pitch, CA_THREADS / 2);   // L transposed: [column j][row i], 64 x 64
   float* s_g = s_l + CK * CK;                       // accumulated log decay
   float* s_beta = s_g + CK;
   float* s_lg = s_beta + CK;
@@ -132,17 +131,18 @@ delta_chunk_prepare_kernel(const StepParams p) {
     s_lg[tid] = tid < id.n ? p.log_g[(long long)(id.row0 + tid) * p.H + h] : 0.f;
     s_beta[tid] = tid < id.n ? p.beta[(long long)(id.row0 + tid) * p.H + h] : 0.f;
   }
-  for (int i = tid; i < CK * (Dp / 2); i += CA_THREADS) {
-    const int r = i / (Dp / 2), c = (i - r * (Dp / 2)) * 2;
-    float2 q = make_float2(0.f, 0.f), k = q;
-    if (r < id.n && c < p.D) {
-      const float* src = p.qk + ((long long)(id.row0 + r) * 2 * K + hk) * p.D + c;
-      q = *reinterpret_cast<const float2*>(src);
-      k = *reinterpret_cast<const float2*>(src + (long long)K * p.D);
+#pragma unroll 4
+  for (int r = warp; r < CK; r += CA_THREADS / 32)
+    for (int c = lane * 2; c < Dp; c += 64) {
+      float2 q = make_float2(0.f, 0.f), k = q;
+      if (r < id.n && c < p.D) {
+        const float* src = p.qk + ((long long)(id.row0 + r) * 2 * K + hk) * p.D + c;
+        q = *reinterpret_cast<const float2*>(src);
+        k = *reinterpret_cast<const float2*>(src + (long long)K * p.D);
+      }
+      *reinterpret_cast<float2*>(s_q + r * pitch + c) = q;
+      *reinterpret_cast<float2*>(s_k + r * pitch + c) = k;
     }
-    *reinterpret_cast<float2*>(s_q + r * pitch + c) = q;
-    *reinterpret_cast<float2*>(s_k + r * pitch + c) = k;
-  }
   __syncthreads();
   if (tid < CK) {
     float g = 0.f;
@@ -186,7 +186,7 @@ delta_chunk_prepare_kernel(const StepParams p) {
         const int i = I * 16 + gr + (e >> 1) * 8, j = J * 16 + n * 8 + gc + (e & 1);
         const float f = j <= i ? expf(s_g[i] - s_g[j]) : 0.f;
         aq[n][e] *= f;
-        s_l[i * CK + j] = j < i ? s_beta[i] * f * ak[n][e] : 0.f;
+        s_l[j * CK + i] = j < i ? s_beta[i] * f * ak[n][e] : 0.f;
       }
     store_frag(id.unit, lay.p + idx, lane, acc_frag(aq[0], aq[1]));
   }
@@ -215,38 +215,57 @@ delta_chunk_prepare_kernel(const StepParams p) {
   }
   for (int d = tid; d < Dp; d += CA_THREADS) reinterpret_cast<float*>(id.unit + lay.dec)[d] = expf(g_end);
   __syncthreads();
-  // forward substitution, one right-hand-side column per thread: key columns give W, value columns U0
+  // forward substitution, one right-hand-side column per thread and 16 rows at a time: the first half of the CTA takes
+  // the key columns (W, in place of k), the second half value columns (U0, in slots of the q tile)
   const int V4 = (p.V + 3) / 4 * 4;
   float* u0 = reinterpret_cast<float*>(id.unit + lay.u);
   const bf16* v = reinterpret_cast<const bf16*>(p.v) + (long long)id.row0 * p.H * p.V + h * p.V;
-  for (int c = tid; c < Dp + V4; c += CA_THREADS) {
-    float x[CK];
-    const bool key = c < Dp;
-    const int vc = c - Dp;
+  constexpr int HALF = CA_THREADS / 2;              // >= CK_MAX_D
+  const bool key = tid < HALF;
+  float* col = key ? s_k + tid : s_q + tid - HALF;
+  const int ld = key ? pitch : HALF;
+  for (int c = key ? tid : tid - HALF; c < (key ? Dp : V4); c += HALF) {
+#pragma unroll 1
+    for (int I = 0; I < 4; ++I) {
+      float x[16];
 #pragma unroll
-    for (int i = 0; i < CK; ++i) {
-      float rhs = 0.f;
-      if (key) rhs = s_k[i * pitch + c] * expf(s_g[i]);
-      else if (i < id.n && vc < p.V) rhs = __bfloat162float(v[(long long)i * p.H * p.V + vc]);
-      x[i] = rhs * s_beta[i];
-    }
-#pragma unroll
-    for (int i = 1; i < CK; ++i) {
-      float a0 = 0.f, a1 = 0.f, a2 = 0.f, a3 = 0.f;
-#pragma unroll
-      for (int j = 0; j < i; j += 4) {
-        const float4 lv = *reinterpret_cast<const float4*>(s_l + i * CK + j);   // entries j >= i of the row are zero
-        a0 = fmaf(lv.x, x[j], a0);
-        if (j + 1 < i) a1 = fmaf(lv.y, x[j + 1], a1);
-        if (j + 2 < i) a2 = fmaf(lv.z, x[j + 2], a2);
-        if (j + 3 < i) a3 = fmaf(lv.w, x[j + 3], a3);
+      for (int i = 0; i < 16; ++i) {
+        const int r = I * 16 + i;
+        if (key) x[i] = col[r * ld] * expf(s_g[r]);
+        else x[i] = r < id.n && c < p.V ? __bfloat162float(v[(long long)r * p.H * p.V + c]) : 0.f;
+        x[i] *= s_beta[r];
       }
-      x[i] -= (a0 + a1) + (a2 + a3);
-    }
+#pragma unroll 2
+      for (int j = 0; j < I * 16; ++j) {
+        const float xj = col[j * ld];
+        const float4* lc = reinterpret_cast<const float4*>(s_l + j * CK + I * 16);
 #pragma unroll
-    for (int i = 0; i < CK; ++i) {
-      if (key) s_q[i * pitch + c] = x[i];
-      else u0[i * V4 + vc] = x[i];
+        for (int q = 0; q < 4; ++q) {
+          const float4 lv = lc[q];
+          x[q * 4] = fmaf(-lv.x, xj, x[q * 4]);
+          x[q * 4 + 1] = fmaf(-lv.y, xj, x[q * 4 + 1]);
+          x[q * 4 + 2] = fmaf(-lv.z, xj, x[q * 4 + 2]);
+          x[q * 4 + 3] = fmaf(-lv.w, xj, x[q * 4 + 3]);
+        }
+      }
+#pragma unroll
+      for (int j = 0; j < 16; ++j) {                // entries of L on and above the diagonal are zero
+        const float4* lc = reinterpret_cast<const float4*>(s_l + (I * 16 + j) * CK + I * 16);
+#pragma unroll
+        for (int q = j / 4; q < 4; ++q) {
+          const float4 lv = lc[q];
+          const float xj = x[j];
+          if (q * 4 > j) x[q * 4] = fmaf(-lv.x, xj, x[q * 4]);
+          if (q * 4 + 1 > j) x[q * 4 + 1] = fmaf(-lv.y, xj, x[q * 4 + 1]);
+          if (q * 4 + 2 > j) x[q * 4 + 2] = fmaf(-lv.z, xj, x[q * 4 + 2]);
+          if (q * 4 + 3 > j) x[q * 4 + 3] = fmaf(-lv.w, xj, x[q * 4 + 3]);
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < 16; ++i) {
+        col[(I * 16 + i) * ld] = x[i];
+        if (!key) u0[(I * 16 + i) * V4 + c] = x[i];
+      }
     }
   }
   __syncthreads();
@@ -255,7 +274,7 @@ delta_chunk_prepare_kernel(const StepParams p) {
     Frag a;
 #pragma unroll
     for (int x = 0; x < 4; ++x) {
-      const float2 w = *reinterpret_cast<const float2*>(s_q + (I * 16 + gr + (x & 1) * 8) * pitch + kk * 16 + gc + (x >> 1) * 8);
+      const float2 w = *reinterpret_cast<const float2*>(s_k + (I * 16 + gr + (x & 1) * 8) * pitch + kk * 16 + gc + (x >> 1) * 8);
       split_pack(w.x, w.y, a.h[x], a.l[x]);
     }
     store_frag(id.unit, lay.w + f, lane, a);
@@ -277,93 +296,106 @@ gla_chunk_prepare_kernel(const StepParams p) {
   if (!chunk_of(p, lay, blockIdx.x, h, blockIdx.z, id)) return;
   const bf16* proj = reinterpret_cast<const bf16*>(p.proj.p);
   const bf16* zp = reinterpret_cast<const bf16*>(p.z);
-  for (int i = tid; i < CK * Dp; i += CA_THREADS) {
-    const int r = i / Dp, c = i - r * Dp;
-    float q = 0.f, k = 0.f, b = 0.f;
-    if (r < id.n && c < p.D) {
-      const bf16* row = proj + (long long)(id.row0 + r) * p.proj.ld + h * p.D + c;
-      q = __bfloat162float(row[p.off_q]) * p.q_scale;
-      k = __bfloat162float(row[p.off_k]);
-      const float z = __bfloat162float(zp[(long long)(id.row0 + r) * p.ld_z + h * p.D + c]) + p.z_bias[h * p.D + c];
-      b = log_sigmoid_f(z) * p.inv_tau * 1.4426950408889634f;
+#pragma unroll 4
+  for (int r = warp; r < CK; r += CA_THREADS / 32)
+    for (int c = lane * 2; c < Dp; c += 64) {
+      float2 q = make_float2(0.f, 0.f), k = q, g = q;
+      if (r < id.n && c < p.D) {
+        auto two = [](const bf16* s) { return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(s)); };
+        const bf16* row = proj + (long long)(id.row0 + r) * p.proj.ld + h * p.D + c;
+        q = two(row + p.off_q);
+        k = two(row + p.off_k);
+        g = two(zp + (long long)(id.row0 + r) * p.ld_z + h * p.D + c);
+        const float2 zb = *reinterpret_cast<const float2*>(p.z_bias + h * p.D + c);
+        const float f = p.inv_tau * 1.4426950408889634f;
+        g = make_float2(log_sigmoid_f(g.x + zb.x) * f, log_sigmoid_f(g.y + zb.y) * f);
+      }
+      *reinterpret_cast<float2*>(s_q + r * pitch + c) = make_float2(q.x * p.q_scale, q.y * p.q_scale);
+      *reinterpret_cast<float2*>(s_k + r * pitch + c) = k;
+      *reinterpret_cast<float2*>(s_b + r * pitch + c) = g;
     }
-    s_q[r * pitch + c] = q;
-    s_k[r * pitch + c] = k;
-    s_b[r * pitch + c] = b;
-  }
   __syncthreads();
   for (int c = tid; c < Dp; c += CA_THREADS) {
     float acc = 0.f;
-#pragma unroll 8
-    for (int r = 0; r < CK; ++r) {
-      acc += s_b[r * pitch + c];
-      s_b[r * pitch + c] = acc;
+#pragma unroll 1
+    for (int r = 0; r < CK; r += 16) {
+      float x[16];
+#pragma unroll
+      for (int i = 0; i < 16; ++i) x[i] = s_b[(r + i) * pitch + c];
+#pragma unroll
+      for (int i = 0; i < 16; ++i) {
+        acc += x[i];
+        s_b[(r + i) * pitch + c] = acc;
+      }
     }
     reinterpret_cast<float*>(id.unit + lay.dec)[c] = exp2f(acc);
   }
   __syncthreads();
   const int gr = lane >> 2, gc = (lane & 3) * 2;
-  if (warp < 4) {
-    // diagonal block: exact decay differences, lanes over the key channels
-    const int r0 = warp * 16;
-    float* s_p = s_d + warp * 16 * 18;
-    for (int i = 0; i < 16; ++i) {
-      float q[CK_MAX_D / 32], b[CK_MAX_D / 32];
-#pragma unroll
-      for (int x = 0; x < CK_MAX_D / 32; ++x) {
-        const int c = lane + x * 32;
-        q[x] = c < Dp ? s_q[(r0 + i) * pitch + c] : 0.f;
-        b[x] = c < Dp ? s_b[(r0 + i) * pitch + c] : 0.f;
-      }
-#pragma unroll 4
-      for (int j = 0; j <= i; ++j) {
-        float a = 0.f;
-#pragma unroll
-        for (int x = 0; x < CK_MAX_D / 32; ++x) {
-          const int c = lane + x * 32;
-          if (c < Dp) a = fmaf(q[x] * exp2f(b[x] - s_b[(r0 + j) * pitch + c]), s_k[(r0 + j) * pitch + c], a);
-        }
-        a = warp_sum(a);
-        if (lane == 0) s_p[i * 18 + j] = a;
-      }
-      if (lane > i && lane < 16) s_p[i * 18 + lane] = 0.f;
-    }
-    __syncwarp();
-    Frag a;
-#pragma unroll
-    for (int x = 0; x < 4; ++x) {
-      const float* s = s_p + (gr + (x & 1) * 8) * 18 + gc + (x >> 1) * 8;
-      split_pack(s[0], s[1], a.h[x], a.l[x]);
-    }
-    store_frag(id.unit, lay.p + warp * (warp + 1) / 2 + warp, lane, a);
-  } else {
-    // blocks below the diagonal: both factors decayed to the row before block I
-    for (int idx = warp - 4; idx < 6; idx += 4) {
-      const int I = idx >= 3 ? 3 : idx >= 1 ? 2 : 1, J = idx - (I - 1) * I / 2;
-      const float* ref = s_b + (I * 16 - 1) * pitch;
-      float acc[2][4] = {};
-      for (int kk = 0; kk < lay.kd; ++kk) {
-        Frag fq;
+  // P: both factors of a 16 x 16 block decayed to a common row, the row before block I or, on the diagonal, its first
+  // row.  There the key factor grows with the decay inside the block; should that leave the range of the format, the
+  // block is computed from the exact differences instead.
+  for (int idx = warp; idx < CK_P; idx += CA_THREADS / 32) {
+    int I, J;
+    tri_block(idx, I, J);
+    const float* ref = s_b + (I == J ? I * 16 : I * 16 - 1) * pitch;
+    if (I == J) {
+      bool far = false;
+      for (int c = lane; c < Dp; c += 32) far |= ref[c] - s_b[(I * 16 + 15) * pitch + c] > 60.f;
+      if (__any_sync(0xffffffffu, far)) {
+        float* s_p = s_d + I * 16 * 18;
+        for (int i = 0; i < 16; ++i)
+          for (int j = 0; j < 16; ++j) {
+            float a = 0.f;
+            if (j <= i)
+              for (int c = lane; c < Dp; c += 32) {
+                const int x = (I * 16 + i) * pitch + c, y = (I * 16 + j) * pitch + c;
+                a = fmaf(s_q[x] * exp2f(s_b[x] - s_b[y]), s_k[y], a);
+              }
+            a = warp_sum(a);
+            if (lane == 0) s_p[i * 18 + j] = a;
+          }
+        __syncwarp();
+        Frag a;
 #pragma unroll
         for (int x = 0; x < 4; ++x) {
-          const int r = (I * 16 + gr + (x & 1) * 8) * pitch, c = kk * 16 + gc + (x >> 1) * 8;
-          split_pack(s_q[r + c] * exp2f(s_b[r + c] - ref[c]), s_q[r + c + 1] * exp2f(s_b[r + c + 1] - ref[c + 1]),
-                     fq.h[x], fq.l[x]);
+          const float* s = s_p + (gr + (x & 1) * 8) * 18 + gc + (x >> 1) * 8;
+          split_pack(s[0], s[1], a.h[x], a.l[x]);
         }
-#pragma unroll
-        for (int n = 0; n < 2; ++n) {
-          uint32_t bh[2], bl[2];
-#pragma unroll
-          for (int x = 0; x < 2; ++x) {
-            const int r = (J * 16 + n * 8 + gr) * pitch, c = kk * 16 + gc + x * 8;
-            split_pack(s_k[r + c] * exp2f(ref[c] - s_b[r + c]), s_k[r + c + 1] * exp2f(ref[c + 1] - s_b[r + c + 1]),
-                       bh[x], bl[x]);
-          }
-          mma3(acc[n], fq, bh[0], bh[1], bl[0], bl[1]);
-        }
+        store_frag(id.unit, lay.p + idx, lane, a);
+        continue;
       }
-      store_frag(id.unit, lay.p + I * (I + 1) / 2 + J, lane, acc_frag(acc[0], acc[1]));
     }
+    float acc[2][4] = {};
+    for (int kk = 0; kk < lay.kd; ++kk) {
+      Frag fq;
+#pragma unroll
+      for (int x = 0; x < 4; ++x) {
+        const int r = (I * 16 + gr + (x & 1) * 8) * pitch, c = kk * 16 + gc + (x >> 1) * 8;
+        const float2 q = *reinterpret_cast<const float2*>(s_q + r + c), b = *reinterpret_cast<const float2*>(s_b + r + c),
+                     f = *reinterpret_cast<const float2*>(ref + c);
+        split_pack(q.x * exp2f(b.x - f.x), q.y * exp2f(b.y - f.y), fq.h[x], fq.l[x]);
+      }
+#pragma unroll
+      for (int n = 0; n < 2; ++n) {
+        uint32_t bh[2], bl[2];
+#pragma unroll
+        for (int x = 0; x < 2; ++x) {
+          const int r = (J * 16 + n * 8 + gr) * pitch, c = kk * 16 + gc + x * 8;
+          const float2 k = *reinterpret_cast<const float2*>(s_k + r + c), b = *reinterpret_cast<const float2*>(s_b + r + c),
+                       f = *reinterpret_cast<const float2*>(ref + c);
+          split_pack(k.x * exp2f(f.x - b.x), k.y * exp2f(f.y - b.y), bh[x], bl[x]);
+        }
+        mma3(acc[n], fq, bh[0], bh[1], bl[0], bl[1]);
+      }
+    }
+    if (I == J)
+#pragma unroll
+      for (int n = 0; n < 2; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e)
+          if (n * 8 + gc + (e & 1) > gr + (e >> 1) * 8) acc[n][e] = 0.f;
+    store_frag(id.unit, lay.p + idx, lane, acc_frag(acc[0], acc[1]));
   }
   for (int f = warp; f < 8 * lay.kd; f += CA_THREADS / 32) {
     Frag a;
@@ -608,7 +640,7 @@ static void launch_chunks(const StepParams& p, int max_len, cudaStream_t s) {
   const int chunks = (max_len + CK - 1) / CK, pitch = chunk_pitch(lay.kd);
   const dim3 grid(chunks, p.H, p.runs.B);
   if (DELTA) {
-    const int smem = (2 * CK * pitch + CK * CK + 3 * CK) * 4;
+    const int smem = (CK * pitch + CK * (pitch > CA_THREADS / 2 ? pitch : CA_THREADS / 2) + CK * CK + 3 * CK) * 4;
     cudaFuncSetAttribute(delta_chunk_prepare_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     delta_chunk_prepare_kernel<<<grid, CA_THREADS, smem, s>>>(p);
   } else {
