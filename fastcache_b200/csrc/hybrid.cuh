@@ -73,14 +73,53 @@ __device__ __forceinline__ void store4(T* dst, float a, float b, float c, float 
   }
 }
 
+// eight consecutive elements; `col` and the pitches are multiples of 8
+template <typename T>
+__device__ __forceinline__ void proj_at8(const ProjSrc& s, long long row, int col, float (&v)[8]) {
+  if (sizeof(T) == 2 && s.splits <= 1) {
+    const uint4 u = __ldcg(reinterpret_cast<const uint4*>(reinterpret_cast<const T*>(s.p) + row * s.ld + col));
+    const uint32_t w[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&w[i]));
+      v[2 * i] = f.x;
+      v[2 * i + 1] = f.y;
+    }
+    return;
+  }
+  const float4 a = proj_at4<T>(s, row, col), b = proj_at4<T>(s, row, col + 4);
+  v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
+  v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+}
+template <typename T>
+__device__ __forceinline__ void store8(T* dst, const float (&v)[8]) {
+  if constexpr (sizeof(T) == 2) {
+    *reinterpret_cast<uint4*>(dst) =
+        make_uint4(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]), pack_bf16(v[4], v[5]), pack_bf16(v[6], v[7]));
+  } else {
+    store4(dst, v[0], v[1], v[2], v[3]);
+    store4(dst + 4, v[4], v[5], v[6], v[7]);
+  }
+}
+
 __device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
-__device__ __forceinline__ float silu_f(float x) { return x / (1.f + expf(-x)); }
+// activations of a model in T: the fast intrinsics where the result is rounded to bf16 anyway
+template <typename T>
+__device__ __forceinline__ float over_one_plus_exp(float x, float e) {      // x / (1 + exp(e))
+  if constexpr (sizeof(T) == 2) return __fdividef(x, 1.f + __expf(e));
+  return x / (1.f + expf(e));
+}
+template <typename T>
+__device__ __forceinline__ float silu_t(float x) { return over_one_plus_exp<T>(x, -x); }
+template <typename T>
+__device__ __forceinline__ float sigmoid_t(float x) { return over_one_plus_exp<T>(1.f, -x); }
 // log(sigmoid(x)) and log(1 + exp(x)) without overflow
 __device__ __forceinline__ float log_sigmoid_f(float x) { return fminf(x, 0.f) - log1pf(expf(-fabsf(x))); }
 __device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
 // 0.5 z (1 + tanh y) = z sigmoid(2 y) with y = sqrt(2 / pi) (z + 0.044715 z^3)
-__device__ __forceinline__ float gelu_tanh_f(float z) {
-  return z / (1.f + expf(-1.5957691216057308f * (z + 0.044715f * z * z * z)));
+template <typename T>
+__device__ __forceinline__ float gelu_tanh_t(float z) {
+  return over_one_plus_exp<T>(z, -1.5957691216057308f * (z + 0.044715f * z * z * z));
 }
 
 struct Run {

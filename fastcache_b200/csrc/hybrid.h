@@ -120,7 +120,7 @@ struct LatentStore {
   int off_q = 0, off_kv = -1, off_g = 0;       // off_kv < 0: the layer reads another layer's rows
   const float* norm_w = nullptr;
   float eps = 0.f;
-  double base = 10000.0;
+  double log2_base = 0.0;            // rotation: position * base^(-2 i / rot_dims)
   const long long* positions = nullptr;
   const int* slots = nullptr;
   void* pool = nullptr;

@@ -3,6 +3,7 @@
 #include <c10/cuda/CUDAGuard.h>
 #include <torch/extension.h>
 
+#include <cmath>
 #include <tuple>
 #include <vector>
 
@@ -351,7 +352,7 @@ Tensor latent_attention(const Tensor& h, const Tensor& w, const std::vector<int6
   st.off_kv = int(d[7]);
   st.off_g = int(d[8]);
   st.eps = float(eps);
-  st.base = base;
+  st.log2_base = std::log2(base);
   st.positions = reinterpret_cast<const long long*>(positions.data_ptr<int64_t>());
   st.pool = pool.data_ptr();
   st.row_width = int(pool.size(2));
@@ -434,6 +435,10 @@ Tensor latent_attention(const Tensor& h, const Tensor& w, const std::vector<int6
   Tensor gate, o_lat = torch::empty({T, H, rank}, h.options());
   st.q = qn.data_ptr();
   st.q_abs = q_abs.data_ptr();
+  if (st.proj.splits > 1) {
+    gate = torch::empty({T, H * V}, h.options());
+    st.gate = gate.data_ptr();
+  }
   fc::launch_latent_store(st, f32, stream_now());
   fc::SimtLinear a;
   a.x = qn.data_ptr();
@@ -507,8 +512,13 @@ Tensor latent_attention(const Tensor& h, const Tensor& w, const std::vector<int6
   a.gx = rank;
   a.gw = (long long)V * rank;
   a.gy = V;
-  a.gate = st.proj;                    // no product has used the scratch since
-  a.gate_off = st.off_g;
+  if (st.gate != nullptr) {
+    a.gate.p = st.gate;
+    a.gate.ld = H * V;
+  } else {
+    a.gate = st.proj;
+    a.gate_off = st.off_g;
+  }
   a.y_pad = int(out.size(1));
   head_linear(a);
   return out;

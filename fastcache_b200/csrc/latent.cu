@@ -29,8 +29,7 @@ latent_store_kernel(const LatentStore p) {
   pdl_wait();
   const long long t = blockIdx.x;
   const double pos = double(p.positions[t]);
-  const double l2b = log2(p.base);
-  for (int i = threadIdx.x; i < half; i += LS_THREADS) rope_angle(pos, l2b, i, p.rot_dims, cs[i], cs[half + i]);
+  for (int i = threadIdx.x; i < half; i += LS_THREADS) rope_angle(pos, p.log2_base, i, p.rot_dims, cs[i], cs[half + i]);
   __syncthreads();
   const int part = blockIdx.y, parts = gridDim.y;
   // queries: every (head, column) of this part
@@ -99,8 +98,8 @@ latent_rotate_kernel(const LatentStore p) {
   pdl_wait();
   const long long t = blockIdx.x;
   const int tid = threadIdx.x, lane = tid & 31;
-  const double pos = double(p.positions[t]), l2b = log2(p.base);
-  for (int i = tid; i < half; i += LR_WARPS * 32) rope_angle(pos, l2b, i, p.rot_dims, cs[i], cs[half + i]);
+  const double pos = double(p.positions[t]);
+  for (int i = tid; i < half; i += LR_WARPS * 32) rope_angle(pos, p.log2_base, i, p.rot_dims, cs[i], cs[half + i]);
   __syncthreads();
   T* row = const_cast<T*>(reinterpret_cast<const T*>(p.proj.p)) + t * p.proj.ld;
   auto rotate = [&](const T* su, T* du, int i0) {            // quads at columns i0 and half + i0 of a rotated part

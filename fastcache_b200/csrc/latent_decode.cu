@@ -410,18 +410,38 @@ head_linear_kernel(const SimtLinear a) {
       }
     }
   }
-  const bool gated = a.gate.p != nullptr || a.gate.part != nullptr;
-  bf16* y = reinterpret_cast<bf16*>(a.y) + g * a.gy;
+  // through shared memory, so that a row of y is written (and its gate read) 16 bytes at a time
+  __syncthreads();
+  constexpr int YP = HL_N + 8;
+  static_assert(XR * YP * 2 <= int(sizeof(s_w)), "staging fits the weight ring");
+  bf16* s_y = reinterpret_cast<bf16*>(&s_w[0][0]);
 #pragma unroll
   for (int i = 0; i < NT; ++i)
 #pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      const int n = n0 + warp * 16 + (lane >> 2) + (e >> 1) * 8, m = m0 + i * 8 + (lane & 3) * 2 + (e & 1);
-      if (n >= a.N || m >= a.M) continue;
-      float v = acc[i][e];
-      if (gated) v *= sigmoid_f(proj_at<bf16>(a.gate, m, a.gate_off + g * a.N + n));
-      y[(long long)m * a.ldy + n] = __float2bfloat16(v);
+    for (int e = 0; e < 4; ++e)
+      s_y[(i * 8 + (lane & 3) * 2 + (e & 1)) * YP + warp * 16 + (lane >> 2) + (e >> 1) * 8] = __float2bfloat16(acc[i][e]);
+  __syncthreads();
+  bf16* y = reinterpret_cast<bf16*>(a.y) + g * a.gy;
+  const bf16* gate = reinterpret_cast<const bf16*>(a.gate.p);
+  for (int i = tid; i < XR * (HL_N / 8); i += HL_THREADS) {
+    const int m = i / (HL_N / 8), n = (i % (HL_N / 8)) * 8;
+    if (m0 + m >= a.M || n0 + n >= a.N) continue;                  // N is a multiple of 8
+    uint4 u = *reinterpret_cast<const uint4*>(s_y + m * YP + n);
+    if (gate != nullptr) {
+      const uint4 gu = __ldcg(reinterpret_cast<const uint4*>(gate + (long long)(m0 + m) * a.gate.ld + a.gate_off + g * a.N +
+                                                             n0 + n));
+      uint32_t uw[4] = {u.x, u.y, u.z, u.w};
+      const uint32_t gw[4] = {gu.x, gu.y, gu.z, gu.w};
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&uw[e]));
+        const float2 q = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&gw[e]));
+        uw[e] = pack_bf16(v.x * sigmoid_t<bf16>(q.x), v.y * sigmoid_t<bf16>(q.y));
+      }
+      u = make_uint4(uw[0], uw[1], uw[2], uw[3]);
     }
+    *reinterpret_cast<uint4*>(y + (long long)(m0 + m) * a.ldy + n0 + n) = u;
+  }
   const int pad = a.y_pad - a.groups * a.N;
   if (pad > 0 && g == 0 && blockIdx.x == 0)
     for (int i = tid; i < XR * pad; i += HL_THREADS)
@@ -430,6 +450,8 @@ head_linear_kernel(const SimtLinear a) {
 }
 
 bool head_linear_mma_supported(const SimtLinear& a) {
+  if (a.N % 8 != 0 || a.ldy % 8 != 0 || a.gy % 8 != 0 || a.gate.part != nullptr) return false;
+  if (a.gate.p != nullptr && (a.gate.ld % 8 != 0 || a.gate_off % 8 != 0)) return false;
   return a.K % 8 == 0 && a.ldx % 8 == 0 && a.ldw % 8 == 0 && a.gx % 8 == 0 && a.gw % 8 == 0 && a.bias == nullptr;
 }
 void launch_head_linear_mma(const SimtLinear& a, cudaStream_t s) {

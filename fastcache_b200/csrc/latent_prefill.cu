@@ -310,7 +310,7 @@ latent_prefill_kernel(const __grid_constant__ LpMaps tm, const LpParams p) {
                 b = fmaf(s_o[(col + 2 * e + 1) * 128 + row], w1, b);
               }
               const float2 g = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&gw[e]));
-              ow[e] = pack_bf16(a * sigmoid_f(g.x), b * sigmoid_f(g.y));
+              ow[e] = pack_bf16(a * sigmoid_t<bf16>(g.x), b * sigmoid_t<bf16>(g.y));
             }
             *reinterpret_cast<uint4*>(dst + col) = make_uint4(ow[0], ow[1], ow[2], ow[3]);
           }

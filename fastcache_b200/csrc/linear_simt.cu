@@ -54,7 +54,7 @@ linear_simt_kernel(const SimtLinear a) {
       if (n >= a.N) break;
       float v = acc[i][j];
       if (bias != nullptr) v += Elem<T>::get(bias[n]);
-      if (gated) v *= sigmoid_f(proj_at<T>(a.gate, m, a.gate_off + g * a.N + n));
+      if (gated) v *= sigmoid_t<T>(proj_at<T>(a.gate, m, a.gate_off + g * a.N + n));
       y[(long long)m * a.ldy + n] = Elem<T>::put(v);
     }
     if (g == 0 && blockIdx.x == 0)

@@ -217,7 +217,7 @@ step_kernel(const StepParams p) {
           for (int j = 0; j < 4; ++j)
             if (col + j < p.V)
               dst[j] = Elem<T>::put(o[j] * inv * p.norm_w[col + j] *
-                                    silu_f(proj_at<T>(p.proj, t, p.off_g + h * p.V + col + j)));
+                                    silu_t<T>(proj_at<T>(p.proj, t, p.off_g + h * p.V + col + j)));
         }
         if (h == 0 && lane < int(p.ld_out) - p.H * p.V) out[t * p.ld_out + p.H * p.V + lane] = Elem<T>::put(0.f);
       }
@@ -303,8 +303,8 @@ gated_head_norm_kernel(const float* __restrict__ o_raw, const ProjSrc proj, int 
     for (int c = lane * 4; c < V; c += 128) {
       const float4 x = *reinterpret_cast<const float4*>(o + c), w = *reinterpret_cast<const float4*>(norm_w + c);
       const float4 g = proj_at4<T>(proj, t, off_g + h * V + c);
-      store4(out + t * ld_out + h * V + c, x.x * inv * w.x * silu_f(g.x), x.y * inv * w.y * silu_f(g.y),
-             x.z * inv * w.z * silu_f(g.z), x.w * inv * w.w * silu_f(g.w));
+      store4(out + t * ld_out + h * V + c, x.x * inv * w.x * silu_t<T>(g.x), x.y * inv * w.y * silu_t<T>(g.y),
+             x.z * inv * w.z * silu_t<T>(g.z), x.w * inv * w.w * silu_t<T>(g.w));
     }
     if (h == 0 && lane < int(ld_out) - H * V) out[t * ld_out + H * V + lane] = Elem<T>::put(0.f);
     return;
@@ -312,7 +312,7 @@ gated_head_norm_kernel(const float* __restrict__ o_raw, const ProjSrc proj, int 
   for (int c = lane; c < V; c += 32) ss += o[c] * o[c];
   const float inv = rsqrtf(warp_sum(ss) / float(V) + eps);
   for (int c = lane; c < V; c += 32)
-    out[t * ld_out + h * V + c] = Elem<T>::put(o[c] * inv * norm_w[c] * silu_f(proj_at<T>(proj, t, off_g + h * V + c)));
+    out[t * ld_out + h * V + c] = Elem<T>::put(o[c] * inv * norm_w[c] * silu_t<T>(proj_at<T>(proj, t, off_g + h * V + c)));
   if (h == 0 && lane < int(ld_out) - H * V) out[t * ld_out + H * V + lane] = Elem<T>::put(0.f);
 }
 void launch_gated_head_norm(const float* o_raw, const ProjSrc& proj, int off_g, const float* norm_w, float eps,
@@ -369,7 +369,7 @@ delta_prepare_kernel(const DeltaPrepare p, int units, int advance) {
         cst[(long long)j * C + c] = run.start > 0 ? cst[(long long)(j + 1) * C + c] : 0.f;
       if (p.taps > 1) cst[(long long)(p.taps - 2) * C + c] = x0;
     }
-    return silu_f(y);
+    return silu_t<T>(y);
   };
   if (u < 2 * p.K) {
     const int which = u / p.K, hk = u - which * p.K;
@@ -398,18 +398,18 @@ delta_prepare_kernel(const DeltaPrepare p, int units, int advance) {
   for (int c = c0 + lane; c < min(c0 + 128, HV); c += 32) dst[c] = Elem<T>::put(conv(2 * p.K * p.D + c));
 }
 
-// The same for long runs: a warp takes 16 consecutive rows of 128 channels (four per lane) and slides the window of the
-// convolution over them in registers, so that every input is read about once.  Heads of up to 128 channels sit in LPH
+// The same with four channels per lane: a warp takes 128 channels of one row (decode) or of 16 consecutive rows, over which
+// it slides the window of the convolution in registers, so that every input is read about once.  Heads of up to 128 channels sit in LPH
 // lanes (a power of two), several to a warp.  Up to four taps.
 constexpr int DR_ROWS = 16;
 template <typename T>
 __global__ void __launch_bounds__(256)
-delta_prepare_rows_kernel(const DeltaPrepare p, int units, int lph, int qk_units) {
+delta_prepare_rows_kernel(const DeltaPrepare p, int units, int lph, int qk_units, int rows, int advance) {
   pdl_launch_dependents();
   pdl_wait();
-  const int t0 = blockIdx.x * DR_ROWS, u = blockIdx.y * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  const int t0 = blockIdx.x * rows, u = blockIdx.y * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (u >= units) return;
-  const int t1 = min(p.T, t0 + DR_ROWS), C = 2 * p.K * p.D + p.H * p.V;
+  const int t1 = min(p.T, t0 + rows), C = 2 * p.K * p.D + p.H * p.V;
   if (u == units - 1) {
     for (int i = lane; i < (t1 - t0) * p.H; i += 32) {
       const int t = t0 + i / p.H, h = i % p.H;
@@ -457,7 +457,7 @@ delta_prepare_rows_kernel(const DeltaPrepare p, int units, int lph, int qk_units
   float4 nxt = on ? proj_at4<T>(p.proj, t0, c) : make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll 2
   for (int t = t0; t < t1; ++t) {
-    const int bt = p.row_seq[t];
+    const int bt = p.row_seq != nullptr ? p.row_seq[t] : t;
     if (bt != b) {
       b = bt;
       run = get_run(p.runs, b);
@@ -470,7 +470,7 @@ delta_prepare_rows_kernel(const DeltaPrepare p, int units, int lph, int qk_units
     float y[4], ss = 0.f;
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
-      y[i] = silu_f(fmaf(x3[i], w[3][i], fmaf(x2[i], w[2][i], fmaf(x1[i], w[1][i], x0[i] * w[0][i]))));
+      y[i] = silu_t<T>(fmaf(x3[i], w[3][i], fmaf(x2[i], w[2][i], fmaf(x1[i], w[1][i], x0[i] * w[0][i]))));
       ss += y[i] * y[i];
       x3[i] = x2[i];
       x2[i] = x1[i];
@@ -485,6 +485,15 @@ delta_prepare_rows_kernel(const DeltaPrepare p, int units, int lph, int qk_units
             make_float4(y[0] * inv, y[1] * inv, y[2] * inv, y[3] * inv);
     } else if (on) {
       store4(reinterpret_cast<T*>(p.v) + (long long)t * p.H * p.V + c - 2 * p.K * p.D, y[0], y[1], y[2], y[3]);
+    }
+    if (advance && on && run.slot >= 0) {                    // a run of one row: this thread read what it now replaces
+      float* s = p.conv_state + (long long)run.slot * (p.taps - 1) * C + c;
+#pragma unroll
+      for (int k = 0; k < 4; ++k) {
+        if (p.taps > 1) s[(long long)(p.taps - 2) * C + k] = x1[k];
+        if (p.taps > 2) s[(long long)(p.taps - 3) * C + k] = x2[k];
+        if (p.taps > 3) s[(long long)(p.taps - 4) * C + k] = x3[k];
+      }
     }
   }
 }
@@ -509,19 +518,20 @@ conv_state_kernel(const DeltaPrepare p) {
 
 template <typename T>
 static void delta_prepare_t(const DeltaPrepare& p, cudaStream_t s) {
-  if (p.runs.cu != nullptr && p.T >= 256 && p.taps <= 4 && p.D % 4 == 0 && p.D <= 128 && p.H * p.V % 4 == 0) {
+  const int advance = p.runs.cu == nullptr ? 1 : 0;
+  if (p.taps <= 4 && p.D % 4 == 0 && p.D <= 128 && p.H * p.V % 4 == 0) {
     int lph = 1;
     while (lph * 4 < p.D) lph <<= 1;
     const int qk_units = (2 * p.K * lph + 31) / 32, units = qk_units + (p.H * p.V + 127) / 128 + 1;
-    launch_pdl(PDL_PARTIALS, delta_prepare_rows_kernel<T>, dim3((p.T + DR_ROWS - 1) / DR_ROWS, (units + 7) / 8),
-               dim3(256), 0, s, p, units, lph, qk_units);
-    if (p.taps > 1)
+    const int rows = advance || p.T < 256 ? 1 : DR_ROWS;
+    launch_pdl(PDL_PARTIALS, delta_prepare_rows_kernel<T>, dim3((p.T + rows - 1) / rows, (units + 7) / 8), dim3(256), 0, s,
+               p, units, lph, qk_units, rows, advance);
+    if (!advance && p.taps > 1)
       launch_pdl(PDL_PARTIALS, conv_state_kernel<T>, dim3((2 * p.K * p.D + p.H * p.V + 255) / 256, p.runs.B), dim3(256),
                  0, s, p);
     return;
   }
   const int units = 2 * p.K + (p.H * p.V + 127) / 128 + 1;
-  const int advance = p.runs.cu == nullptr ? 1 : 0;
   launch_pdl(PDL_PARTIALS, delta_prepare_kernel<T>, dim3(p.T, (units + 7) / 8), dim3(256), 0, s, p, units, advance);
   if (!advance && p.taps > 1)
     launch_pdl(PDL_PARTIALS, conv_state_kernel<T>, dim3((2 * p.K * p.D + p.H * p.V + 255) / 256, p.runs.B), dim3(256),

@@ -123,6 +123,8 @@ delta_chunk_prepare_kernel(const StepParams p) {
   float* s_g = s_l + CK * CK;                       // accumulated log decay
   float* s_beta = s_g + CK;
   float* s_lg = s_beta + CK;
+  float* s_eg = s_lg + CK;                          // e^b of a row, e^(b_end - b)
+  float* s_ek = s_eg + CK;
   const int h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   ChunkId id;
   if (!chunk_of(p, lay, blockIdx.x, h, blockIdx.z, id)) return;
@@ -151,6 +153,11 @@ delta_chunk_prepare_kernel(const StepParams p) {
   }
   __syncthreads();
   const float g_end = s_g[CK - 1];
+  if (tid < CK) {
+    s_eg[tid] = expf(s_g[tid]);
+    s_ek[tid] = expf(g_end - s_g[tid]);
+  }
+  __syncthreads();
   const int gr = lane >> 2, gc = (lane & 3) * 2;
   // L and P, block by block
   for (int idx = warp; idx < CK_P; idx += CA_THREADS / 32) {
@@ -198,7 +205,7 @@ delta_chunk_prepare_kernel(const StepParams p) {
 #pragma unroll
       for (int x = 0; x < 4; ++x) {
         const int r = I * 16 + gr + (x & 1) * 8, c = kk * 16 + gc + (x >> 1) * 8;
-        const float e = expf(s_g[r]);
+        const float e = s_eg[r];
         split_pack(s_q[r * pitch + c] * e, s_q[r * pitch + c + 1] * e, a.h[x], a.l[x]);
       }
       store_frag(id.unit, lay.q + f, lane, a);
@@ -207,13 +214,13 @@ delta_chunk_prepare_kernel(const StepParams p) {
 #pragma unroll
       for (int x = 0; x < 4; ++x) {
         const int d = m * 16 + gr + (x & 1) * 8, r = kt * 16 + gc + (x >> 1) * 8;
-        split_pack(s_k[r * pitch + d] * expf(g_end - s_g[r]), s_k[(r + 1) * pitch + d] * expf(g_end - s_g[r + 1]),
+        split_pack(s_k[r * pitch + d] * s_ek[r], s_k[(r + 1) * pitch + d] * s_ek[r + 1],
                    a.h[x], a.l[x]);
       }
       store_frag(id.unit, lay.k + f - 4 * lay.kd, lane, a);
     }
   }
-  for (int d = tid; d < Dp; d += CA_THREADS) reinterpret_cast<float*>(id.unit + lay.dec)[d] = expf(g_end);
+  for (int d = tid; d < Dp; d += CA_THREADS) reinterpret_cast<float*>(id.unit + lay.dec)[d] = s_eg[CK - 1];
   __syncthreads();
   // forward substitution, one right-hand-side column per thread and 16 rows at a time: the first half of the CTA takes
   // the key columns (W, in place of k), the second half value columns (U0, in slots of the q tile)
@@ -231,7 +238,7 @@ delta_chunk_prepare_kernel(const StepParams p) {
 #pragma unroll
       for (int i = 0; i < 16; ++i) {
         const int r = I * 16 + i;
-        if (key) x[i] = col[r * ld] * expf(s_g[r]);
+        if (key) x[i] = col[r * ld] * s_eg[r];
         else x[i] = r < id.n && c < p.V ? __bfloat162float(v[(long long)r * p.H * p.V + c]) : 0.f;
         x[i] *= s_beta[r];
       }
@@ -426,7 +433,7 @@ gla_chunk_prepare_kernel(const StepParams p) {
 constexpr int CB_THREADS = 128;
 
 template <bool DELTA, int VB>
-__global__ void __launch_bounds__(CB_THREADS)
+__global__ void __launch_bounds__(CB_THREADS, VB == 16 ? 3 : 2)
 chunk_scan_kernel(const StepParams p) {
   constexpr int N8 = VB / 8;
   constexpr int PITCH = VB + 8;                     // bf16; rows an odd number of 16-byte units apart
@@ -497,12 +504,12 @@ chunk_scan_kernel(const StepParams p) {
   };
   const int V4 = (p.V + 3) / 4 * 4;
   const int n_chunks = (run.len + CK - 1) / CK;
-  for (int c = 0; c < n_chunks; ++c) {
-    ChunkId id;
-    chunk_of(p, lay, c, h, b, id);
-    const int i0 = warp * 16 + gr;                  // rows i0 and i0 + 8 of the chunk
-    // ---- U0 (or V) and the products with the state before the chunk
-    float u[N8][4], o[N8][4];
+  const int i0 = warp * 16 + gr;                    // this thread's rows of a chunk: i0 and i0 + 8
+  constexpr int MAX_KD = CK_MAX_D / 16;
+  float u[N8][4];
+  Frag fq[3], fw[3];
+  // U0 (or V) of this thread's rows and the first fragments of a chunk
+  auto fetch = [&](const ChunkId& id) {
 #pragma unroll
     for (int n = 0; n < N8; ++n)
 #pragma unroll
@@ -518,39 +525,64 @@ chunk_scan_kernel(const StepParams p) {
         }
         u[n][half * 2] = x.x;
         u[n][half * 2 + 1] = x.y;
-        o[n][half * 2] = o[n][half * 2 + 1] = 0.f;
       }
-    Frag fq = load_frag(id.unit, lay.q + warp * kd, lane), fw;
-    if (DELTA) fw = load_frag(id.unit, lay.w + warp * kd, lane);
-    for (int kk = 0; kk < kd; ++kk) {
-      Frag nq = fq, nw = fw;
-      if (kk + 1 < kd) {
-        nq = load_frag(id.unit, lay.q + warp * kd + kk + 1, lane);
-        if (DELTA) nw = load_frag(id.unit, lay.w + warp * kd + kk + 1, lane);
-      }
-      if (DELTA) {                                  // U = U0 - W S
 #pragma unroll
-        for (int x = 0; x < 4; ++x) {
-          fw.h[x] ^= 0x80008000u;
-          fw.l[x] ^= 0x80008000u;
-        }
-      }
+    for (int x = 0; x < 2; ++x) {
+      if (x >= kd) continue;
+      fq[x] = load_frag(id.unit, lay.q + warp * kd + x, lane);
+      if (DELTA) fw[x] = load_frag(id.unit, lay.w + warp * kd + x, lane);
+    }
+  };
+  ChunkId id;
+  chunk_of(p, lay, 0, h, b, id);
+  fetch(id);
+  for (int c = 0; c < n_chunks; ++c) {
+    // ---- products with the state before the chunk: O = Q' S, U = U0 - W S
+    float o[N8][4];
+#pragma unroll
+    for (int n = 0; n < N8; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
+    Frag fp[2], fk[2][2];                           // P and K'^T (two blocks of S) of a 16-row step
+    {
+      uint32_t bh[2][N8 / 2][4], bl[2][N8 / 2][4];
 #pragma unroll
       for (int n2 = 0; n2 < N8 / 2; ++n2) {
-        uint32_t bh[4], bl[4];
-        ld_b(a_sh, kk, n2, bh);
-        ld_b(a_sl, kk, n2, bl);
+        ld_b(a_sh, 0, n2, bh[0][n2]);
+        ld_b(a_sl, 0, n2, bl[0][n2]);
+      }
 #pragma unroll
-        for (int y = 0; y < 2; ++y) {
-          mma3(o[n2 * 2 + y], fq, bh[y * 2], bh[y * 2 + 1], bl[y * 2], bl[y * 2 + 1]);
-          if (DELTA) mma3(u[n2 * 2 + y], fw, bh[y * 2], bh[y * 2 + 1], bl[y * 2], bl[y * 2 + 1]);
+      for (int kk = 0; kk < MAX_KD; ++kk) {
+        if (kk >= kd) continue;
+        if (kk + 2 < kd) {
+          fq[(kk + 2) % 3] = load_frag(id.unit, lay.q + warp * kd + kk + 2, lane);
+          if (DELTA) fw[(kk + 2) % 3] = load_frag(id.unit, lay.w + warp * kd + kk + 2, lane);
+        }
+        if (kk + 1 < kd)
+#pragma unroll
+          for (int n2 = 0; n2 < N8 / 2; ++n2) {
+            ld_b(a_sh, kk + 1, n2, bh[(kk + 1) & 1][n2]);
+            ld_b(a_sl, kk + 1, n2, bl[(kk + 1) & 1][n2]);
+          }
+        if (kk == kd - 1) {                         // what follows the barrier
+          fp[0] = load_frag(id.unit, lay.p + warp * (warp + 1) / 2, lane);
+          if (warp < kd) fk[0][0] = load_frag(id.unit, lay.k + warp * 4, lane);
+          if (warp + 4 < kd) fk[0][1] = load_frag(id.unit, lay.k + (warp + 4) * 4, lane);
+        }
+        Frag& q = fq[kk % 3];
+        Frag& w = fw[kk % 3];
+        if (DELTA)
+#pragma unroll
+          for (int x = 0; x < 4; ++x) {
+            w.h[x] ^= 0x80008000u;
+            w.l[x] ^= 0x80008000u;
+          }
+#pragma unroll
+        for (int n = 0; n < N8; ++n) {
+          const uint32_t *hh = bh[kk & 1][n / 2] + (n & 1) * 2, *ll = bl[kk & 1][n / 2] + (n & 1) * 2;
+          mma3(o[n], q, hh[0], hh[1], ll[0], ll[1]);
+          if (DELTA) mma3(u[n], w, hh[0], hh[1], ll[0], ll[1]);
         }
       }
-      fq = nq;
-      fw = nw;
     }
-    Frag fp = load_frag(id.unit, lay.p + warp * (warp + 1) / 2, lane);
-    Frag fk = load_frag(id.unit, lay.k + warp * 4, lane);          // warp < kd or an unused fragment of this unit
 #pragma unroll
     for (int n = 0; n < N8; ++n)
 #pragma unroll
@@ -561,35 +593,11 @@ chunk_scan_kernel(const StepParams p) {
         *reinterpret_cast<uint32_t*>(s_uh + off) = hi;
         if (DELTA) *reinterpret_cast<uint32_t*>(s_ul + off) = lo;  // a bf16 value has no second term
       }
-    __syncthreads();
-    // ---- O += P U
-    for (int kt = 0; kt <= warp; ++kt) {
-      Frag np = fp;
-      if (kt < warp) np = load_frag(id.unit, lay.p + warp * (warp + 1) / 2 + kt + 1, lane);
-#pragma unroll
-      for (int n2 = 0; n2 < N8 / 2; ++n2) {
-        uint32_t bh[4], bl[4];
-        ld_b(a_uh, kt, n2, bh);
-        if (DELTA) ld_b(a_ul, kt, n2, bl);
-#pragma unroll
-        for (int y = 0; y < 2; ++y) {
-          if (DELTA) {
-            mma3(o[n2 * 2 + y], fp, bh[y * 2], bh[y * 2 + 1], bl[y * 2], bl[y * 2 + 1]);
-          } else {
-            mma_bf16(o[n2 * 2 + y], fp.l, bh[y * 2], bh[y * 2 + 1]);
-            mma_bf16(o[n2 * 2 + y], fp.h, bh[y * 2], bh[y * 2 + 1]);
-          }
-        }
-      }
-      fp = np;
-    }
-    // ---- S = dec S + K'^T U
     const float* dec = reinterpret_cast<const float*>(id.unit + lay.dec);
 #pragma unroll
     for (int mi = 0; mi < 2; ++mi) {
-      const int m = warp + mi * 4;
-      if (m >= kd) continue;
-      const float d0 = __ldcg(dec + m * 16 + gr), d1 = __ldcg(dec + m * 16 + gr + 8);
+      if (warp + mi * 4 >= kd) continue;
+      const float d0 = __ldcg(dec + (warp + mi * 4) * 16 + gr), d1 = __ldcg(dec + (warp + mi * 4) * 16 + gr + 8);
 #pragma unroll
       for (int n = 0; n < N8; ++n) {
         S[mi][n][0] *= d0;
@@ -597,26 +605,48 @@ chunk_scan_kernel(const StepParams p) {
         S[mi][n][2] *= d1;
         S[mi][n][3] *= d1;
       }
+    }
+    __syncthreads();
+    const ChunkId now = id;
+    // ---- O += P U, S = dec S + K'^T U
+    {
+      uint32_t bh[2][N8 / 2][4], bl[2][N8 / 2][4];
+#pragma unroll
+      for (int n2 = 0; n2 < N8 / 2; ++n2) {
+        ld_b(a_uh, 0, n2, bh[0][n2]);
+        if (DELTA) ld_b(a_ul, 0, n2, bl[0][n2]);
+      }
+#pragma unroll
       for (int kt = 0; kt < 4; ++kt) {
-        Frag nk = fk;
-        if (kt < 3) nk = load_frag(id.unit, lay.k + m * 4 + kt + 1, lane);
-        else if (mi == 0 && m + 4 < kd) nk = load_frag(id.unit, lay.k + (m + 4) * 4, lane);
+        if (kt < 3) {
+          if (kt + 1 <= warp) fp[(kt + 1) & 1] = load_frag(now.unit, lay.p + warp * (warp + 1) / 2 + kt + 1, lane);
+          if (warp < kd) fk[(kt + 1) & 1][0] = load_frag(now.unit, lay.k + warp * 4 + kt + 1, lane);
+          if (warp + 4 < kd) fk[(kt + 1) & 1][1] = load_frag(now.unit, lay.k + (warp + 4) * 4 + kt + 1, lane);
 #pragma unroll
-        for (int n2 = 0; n2 < N8 / 2; ++n2) {
-          uint32_t bh[4], bl[4];
-          ld_b(a_uh, kt, n2, bh);
-          if (DELTA) ld_b(a_ul, kt, n2, bl);
-#pragma unroll
-          for (int y = 0; y < 2; ++y) {
-            if (DELTA) {
-              mma3(S[mi][n2 * 2 + y], fk, bh[y * 2], bh[y * 2 + 1], bl[y * 2], bl[y * 2 + 1]);
-            } else {
-              mma_bf16(S[mi][n2 * 2 + y], fk.l, bh[y * 2], bh[y * 2 + 1]);
-              mma_bf16(S[mi][n2 * 2 + y], fk.h, bh[y * 2], bh[y * 2 + 1]);
-            }
+          for (int n2 = 0; n2 < N8 / 2; ++n2) {
+            ld_b(a_uh, kt + 1, n2, bh[(kt + 1) & 1][n2]);
+            if (DELTA) ld_b(a_ul, kt + 1, n2, bl[(kt + 1) & 1][n2]);
           }
+        } else if (c + 1 < n_chunks) {
+          chunk_of(p, lay, c + 1, h, b, id);
+          fetch(id);
         }
-        fk = nk;
+        auto add = [&](float (&acc)[4], const Frag& f, int n) {
+          const uint32_t* hh = bh[kt & 1][n / 2] + (n & 1) * 2;
+          if (DELTA) {
+            const uint32_t* ll = bl[kt & 1][n / 2] + (n & 1) * 2;
+            mma3(acc, f, hh[0], hh[1], ll[0], ll[1]);
+          } else {
+            mma_bf16(acc, f.l, hh[0], hh[1]);
+            mma_bf16(acc, f.h, hh[0], hh[1]);
+          }
+        };
+#pragma unroll
+        for (int n = 0; n < N8; ++n) {
+          if (kt <= warp) add(o[n], fp[kt & 1], n);
+          if (warp < kd) add(S[0][n], fk[kt & 1][0], n);
+          if (warp + 4 < kd) add(S[1][n], fk[kt & 1][1], n);
+        }
       }
     }
 #pragma unroll
@@ -624,8 +654,8 @@ chunk_scan_kernel(const StepParams p) {
 #pragma unroll
       for (int half = 0; half < 2; ++half) {
         const int i = i0 + half * 8, v = v0 + n * 8 + gc;
-        if (i < id.n && v < p.V)
-          *reinterpret_cast<float2*>(p.o_raw + ((long long)(id.row0 + i) * p.H + h) * p.V + v) =
+        if (i < now.n && v < p.V)
+          *reinterpret_cast<float2*>(p.o_raw + ((long long)(now.row0 + i) * p.H + h) * p.V + v) =
               make_float2(o[n][half * 2], o[n][half * 2 + 1]);
       }
     put_state();                                    // the products with the old state ended before the barrier above
@@ -640,7 +670,7 @@ static void launch_chunks(const StepParams& p, int max_len, cudaStream_t s) {
   const int chunks = (max_len + CK - 1) / CK, pitch = chunk_pitch(lay.kd);
   const dim3 grid(chunks, p.H, p.runs.B);
   if (DELTA) {
-    const int smem = (CK * pitch + CK * (pitch > CA_THREADS / 2 ? pitch : CA_THREADS / 2) + CK * CK + 3 * CK) * 4;
+    const int smem = (CK * pitch + CK * (pitch > CA_THREADS / 2 ? pitch : CA_THREADS / 2) + CK * CK + 5 * CK) * 4;
     cudaFuncSetAttribute(delta_chunk_prepare_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     delta_chunk_prepare_kernel<<<grid, CA_THREADS, smem, s>>>(p);
   } else {
@@ -654,8 +684,8 @@ static void launch_chunks(const StepParams& p, int max_len, cudaStream_t s) {
     kern<<<dim3((p.V + vb - 1) / vb, p.H, p.runs.B), CB_THREADS, smem, s>>>(p);
   };
   // few (request, head) pairs: narrower column blocks for more CTAs
-  if (p.runs.B * p.H * ((p.V + 63) / 64) >= 148) scan(chunk_scan_kernel<DELTA, 64>, 64);
-  else scan(chunk_scan_kernel<DELTA, 32>, 32);
+  if (p.runs.B * p.H * ((p.V + 31) / 32) >= 2 * 148) scan(chunk_scan_kernel<DELTA, 32>, 32);
+  else scan(chunk_scan_kernel<DELTA, 16>, 16);
   const cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess) throw std::runtime_error(std::string("chunked recurrence: ") + cudaGetErrorString(e));
 }

@@ -106,30 +106,29 @@ rms_norm_wide_kernel(const float* __restrict__ x, const float* __restrict__ w, T
     h[row * Wp + c] = Elem<T>::put(c < W ? x[row * W + c] * inv * w[c] : 0.f);
 }
 
-// out = gelu_tanh(gate + bias) * (up + bias), four columns per thread
+// out = gelu_tanh(gate + bias) * (up + bias), eight columns per thread; grid (column blocks, row groups)
 template <typename T>
 __global__ void __launch_bounds__(RS_THREADS)
-gelu_mul_kernel(const ProjSrc gu, const T* __restrict__ bias, T* __restrict__ out, long long total, int quads,
-                int up_off, int width, int width_p) {
+gelu_mul_kernel(const ProjSrc gu, const T* __restrict__ bias, T* __restrict__ out, int rows, int up_off, int width,
+                int width_p) {
   pdl_launch_dependents();
   pdl_wait();
-  for (long long i = blockIdx.x * (long long)RS_THREADS + threadIdx.x; i < total;
-       i += (long long)gridDim.x * RS_THREADS) {
-    const long long row = i / quads;
-    const int col = int(i - row * quads) * 4;
-    const float4 g = proj_at4<T>(gu, row, col), u = proj_at4<T>(gu, row, up_off + col);
-    const float gv[4] = {g.x, g.y, g.z, g.w}, uv[4] = {u.x, u.y, u.z, u.w};
-    float o[4];
+  const int col = (blockIdx.x * RS_THREADS + threadIdx.x) * 8;
+  if (col >= width_p) return;
+  float bg[8], bu[8];
 #pragma unroll
-    for (int j = 0; j < 4; ++j) {
-      float a = gv[j], b = uv[j];
-      if (bias != nullptr) {
-        a += Elem<T>::get(bias[col + j]);
-        b += Elem<T>::get(bias[up_off + col + j]);
-      }
-      o[j] = col + j < width ? gelu_tanh_f(a) * b : 0.f;
-    }
-    store4(out + row * width_p + col, o[0], o[1], o[2], o[3]);
+  for (int j = 0; j < 8; ++j) {
+    bg[j] = bias != nullptr ? Elem<T>::get(bias[col + j]) : 0.f;
+    bu[j] = bias != nullptr ? Elem<T>::get(bias[up_off + col + j]) : 0.f;
+  }
+#pragma unroll 2
+  for (int row = blockIdx.y; row < rows; row += gridDim.y) {
+    float g[8], u[8], o[8];
+    proj_at8<T>(gu, row, col, g);
+    proj_at8<T>(gu, row, up_off + col, u);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) o[j] = col + j < width ? gelu_tanh_t<T>(g[j] + bg[j]) * (u[j] + bu[j]) : 0.f;
+    store8(out + (long long)row * width_p + col, o);
   }
 }
 
@@ -185,15 +184,14 @@ void launch_rms_norm_wide(const float* x, const float* w, void* h, int T, int W,
 void launch_gelu_mul(const ProjSrc& gu, const void* bias, void* out, int T, int up_off, int width, int width_p,
                      bool f32, cudaStream_t s) {
   if (T == 0) return;
-  const int quads = width_p / 4;
-  const long long total = (long long)T * quads;
-  const int blocks = (int)std::min<long long>((total + RS_THREADS - 1) / RS_THREADS, 148 * 16);
+  const int cols = (width_p / 8 + RS_THREADS - 1) / RS_THREADS;
+  const dim3 grid(cols, std::min(T, std::max(1, 148 * 8 / cols)));
   if (f32)
-    launch_pdl(PDL_PARTIALS, gelu_mul_kernel<float>, dim3(blocks), dim3(RS_THREADS), 0, s, gu, (const float*)bias,
-               (float*)out, total, quads, up_off, width, width_p);
+    launch_pdl(PDL_PARTIALS, gelu_mul_kernel<float>, grid, dim3(RS_THREADS), 0, s, gu, (const float*)bias, (float*)out, T,
+               up_off, width, width_p);
   else
-    launch_pdl(PDL_PARTIALS, gelu_mul_kernel<bf16>, dim3(blocks), dim3(RS_THREADS), 0, s, gu, (const bf16*)bias,
-               (bf16*)out, total, quads, up_off, width, width_p);
+    launch_pdl(PDL_PARTIALS, gelu_mul_kernel<bf16>, grid, dim3(RS_THREADS), 0, s, gu, (const bf16*)bias, (bf16*)out, T,
+               up_off, width, width_p);
   check_launch("gelu gate");
 }
 
