@@ -113,7 +113,10 @@ struct SmemLayout {
   static constexpr int TOTAL = BAR_OFF + 256 + 1024;  // + barriers + alignment slack
 };
 
-template <int BN, int STAGES, bool TRANS_OUT, bool SWIGLU = false>
+// GLU: gated epilogue, out = act(gate) * up of w = [gate; up]
+enum Glu : int { GLU_NONE = 0, GLU_SILU = 1, GLU_GELU_TANH = 2 };   // GLU_GELU_TANH takes a bias [gate | up]
+
+template <int BN, int STAGES, bool TRANS_OUT, int GLU = GLU_NONE>
 __global__ void __launch_bounds__(GEMM_THREADS, 1)
 gemm_bf16_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_constant__ CUtensorMap tma_b,
                  const GemmParams p) {
@@ -192,7 +195,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_constan
           uint8_t* sb = sa + L::A_BYTES;
           mbar_expect_tx(&full_bar[stage], L::STAGE_BYTES);
           tma_load_2d(sa, &tma_a, &full_bar[stage], kb * BK, m_blk * BM);
-          if constexpr (SWIGLU) {
+          if constexpr (GLU != GLU_NONE) {
             // B tile = 128 rows of the gate half + the matching 128 rows of the up half
             tma_load_2d(sb, &tma_b, &full_bar[stage], kb * BK, n_blk * (BN / 2));
             tma_load_2d(sb + L::B_BYTES / 2, &tma_b, &full_bar[stage], kb * BK, p.up_row0 + n_blk * (BN / 2));
@@ -342,7 +345,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_constan
         }
       };
 
-      if constexpr (SWIGLU) {
+      if constexpr (GLU != GLU_NONE) {
         // accumulator columns [0, BN/2) = gate, [BN/2, BN) = up; out[:, n_blk * BN/2 + j] = silu(gate_j) * up_j
         const int jo = n_blk * (BN / 2);
 #pragma unroll 1
@@ -363,9 +366,25 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_constan
 #pragma unroll
               for (int e = 0; e < 4; ++e) {
                 const int t = q * 8 + e * 2;
-                const float g0 = __uint_as_float(rg[t]), g1 = __uint_as_float(rg[t + 1]);
-                const float a = g0 / (1.f + __expf(-g0)) * __uint_as_float(ru[t]);
-                const float b = g1 / (1.f + __expf(-g1)) * __uint_as_float(ru[t + 1]);
+                float g0 = __uint_as_float(rg[t]), g1 = __uint_as_float(rg[t + 1]);
+                float u0 = __uint_as_float(ru[t]), u1 = __uint_as_float(ru[t + 1]);
+                float a, b;
+                if constexpr (GLU == GLU_GELU_TANH) {
+                  if (p.bias != nullptr) {            // pairs of a bias that starts at a multiple of 16 bytes
+                    const uint32_t bg = *reinterpret_cast<const uint32_t*>(p.bias + jo + c * 32 + t);
+                    const uint32_t bu = *reinterpret_cast<const uint32_t*>(p.bias + p.up_row0 + jo + c * 32 + t);
+                    g0 += __uint_as_float(bg << 16);
+                    g1 += __uint_as_float(bg & 0xffff0000u);
+                    u0 += __uint_as_float(bu << 16);
+                    u1 += __uint_as_float(bu & 0xffff0000u);
+                  }
+                  // 0.5 z (1 + tanh y) = z / (1 + exp(-2 y)), y = sqrt(2 / pi) (z + 0.044715 z^3)
+                  a = __fdividef(g0, 1.f + __expf(-1.5957691216057308f * (g0 + 0.044715f * g0 * g0 * g0))) * u0;
+                  b = __fdividef(g1, 1.f + __expf(-1.5957691216057308f * (g1 + 0.044715f * g1 * g1 * g1))) * u1;
+                } else {
+                  a = g0 / (1.f + __expf(-g0)) * u0;
+                  b = g1 / (1.f + __expf(-g1)) * u1;
+                }
                 u[e] = pack_bf16(a, b);
               }
               *reinterpret_cast<uint4*>(dst + q * 8) = make_uint4(u[0], u[1], u[2], u[3]);
@@ -492,11 +511,11 @@ CUtensorMap make_tmap_bf16_3d(const void* base, uint64_t n0, uint64_t n1, uint64
   return m;
 }
 
-template <int BN, int STAGES, bool TRANS, bool SWIGLU = false>
+template <int BN, int STAGES, bool TRANS, int GLU = GLU_NONE>
 static void launch_one(const CUtensorMap& ta, const CUtensorMap& tb, const GemmParams& p, int grid,
                        cudaStream_t stream) {
   using L = SmemLayout<BN, STAGES>;
-  auto kern = gemm_bf16_kernel<BN, STAGES, TRANS, SWIGLU>;
+  auto kern = gemm_bf16_kernel<BN, STAGES, TRANS, GLU>;
   // the attribute belongs to the (function, device) pair: remember it per device, not per process
   static std::atomic<uint64_t> configured{0};
   int dev = 0;
@@ -543,7 +562,7 @@ void gemm_bf16(const void* x, const void* w, void* c, const void* bias, int M, i
   p.counters = ws.counters;
   const int num_kb = (K + BK - 1) / BK;
   const bool swapped = (M <= 256);
-  if (!swapped && gemm_pairs_mode() &&
+  if (!swapped && gemm_pairs_mode() && act != ACT_GEGLU_TANH &&
       gemm_bf16_2cta(x, w, c, bias, M, N, K, ldx, ldw, ldc, act, sm_limit, ws.status, stream))
     return;
   if (!swapped) {
@@ -558,19 +577,21 @@ void gemm_bf16(const void* x, const void* w, void* c, const void* bias, int M, i
     p.num_m = (M + BM - 1) / BM;
     p.group_m = 16;
     CUtensorMap ta = make_tmap_bf16_2d(x, M, K, ldx, BM, BK);
-    if (act == ACT_SWIGLU) {
+    if (act == ACT_SWIGLU || act == ACT_GEGLU_TANH) {
       // w = [gate; up] stacked ([N, K], N = 2 x width); c is [M, N / 2]
       constexpr int BN = 256;
       const int width = N / 2;
-      if (N % 256 != 0 || ldc % 8 != 0 || (reinterpret_cast<uintptr_t>(c) & 15) != 0 || bias != nullptr)
-        throw std::runtime_error("fused SwiGLU GEMM needs N % 256 == 0, a 16-byte aligned output and no bias");
+      if (N % 256 != 0 || ldc % 8 != 0 || (reinterpret_cast<uintptr_t>(c) & 15) != 0 ||
+          (bias != nullptr && (act == ACT_SWIGLU || (reinterpret_cast<uintptr_t>(bias) & 15) != 0)))
+        throw std::runtime_error("fused gated GEMM needs N % 256 == 0, a 16-byte aligned output and no (SwiGLU) or a 16-byte aligned (GEGLU) bias");
       p.N = width;
       p.act = ACT_NONE;
       p.up_row0 = width;
       p.num_n = width / (BN / 2);
       p.total_work = p.num_m * p.num_n;
       CUtensorMap tb = make_tmap_bf16_2d(w, N, K, ldw, BN / 2, BK);
-      launch_one<BN, 4, false, true>(ta, tb, p, std::min(p.total_work, sms), stream);
+      if (act == ACT_SWIGLU) launch_one<BN, 4, false, GLU_SILU>(ta, tb, p, std::min(p.total_work, sms), stream);
+      else launch_one<BN, 4, false, GLU_GELU_TANH>(ta, tb, p, std::min(p.total_work, sms), stream);
       return;
     }
     if (N >= 256 || N % 256 == 0) {
@@ -588,7 +609,7 @@ void gemm_bf16(const void* x, const void* w, void* c, const void* bias, int M, i
     }
     return;
   }
-  if (act == ACT_SWIGLU) throw std::runtime_error("fused SwiGLU GEMM is for M > 256; use linear_silu_mul below that");
+  if (act == ACT_SWIGLU || act == ACT_GEGLU_TANH) throw std::runtime_error("fused gated GEMM is for M > 256; use linear_silu_mul below that");
   // decode-size batch with more 256-row tiles than SMs (the LM head): equal spans of (tile, K block) units per SM
   if (M <= 128 && streamk_enabled() && (N + 255) / 256 >= sms &&
       gemm_streamk_bf16(x, w, c, bias, M, N, K, ldx, ldw, ldc, act, false, ws, sm_limit, stream))

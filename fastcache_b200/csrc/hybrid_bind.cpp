@@ -149,8 +149,23 @@ Tensor linear_gelu_mul(const Tensor& h, const Tensor& w, const OptTensor& bias, 
     bp = bias->data_ptr();
   }
   Tensor hold;
-  const fc::ProjSrc src = project(h, w, c10::nullopt, true, hold);
   Tensor out = torch::empty({T, wp}, h.options());
+  if (!is_f32(h) && T > 256 && width % 128 == 0 && up_off == width && N == 2 * width) {
+    // prefill sizes: the gate runs in the GEMM's epilogue
+    const auto& ws = ws_of(h);
+    fc::GemmWorkspace gw;
+    gw.scratch = ws.gemm_scratch;
+    gw.counters = ws.gemm_counters;
+    gw.status = ws.status;
+    gw.grid_sync = ws.grid_sync;
+    check_elem(h, "h");
+    TORCH_CHECK(h.scalar_type() == w.scalar_type() && h.dim() == 2 && h.size(1) == w.size(1) && h.stride(1) == 1 &&
+                    h.stride(0) % 8 == 0 && w.is_contiguous() && w.size(1) % 8 == 0, "bad projection operands");
+    fc::gemm_bf16(h.data_ptr(), w.data_ptr(), out.data_ptr(), bp, int(T), int(N), int(h.size(1)), h.stride(0), w.size(1),
+                  wp, fc::ACT_GEGLU_TANH, gw, fc::stream_sm_limit(stream_now()), stream_now());
+    return out;
+  }
+  const fc::ProjSrc src = project(h, w, c10::nullopt, true, hold);
   fc::launch_gelu_mul(src, bp, out.data_ptr(), int(T), int(up_off), int(width), int(wp), is_f32(h), stream_now());
   return out;
 }

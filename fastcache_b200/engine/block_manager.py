@@ -118,17 +118,18 @@ class BlockManager:
             return False
         return len(self.free_block_ids) >= seq.num_blocks
 
-    def allocate(self, seq: Sequence) -> None:
+    def allocate(self, seq: Sequence, reuse_prefix: bool = True) -> None:
         """Give `seq` blocks for its whole prompt, reusing cached prefix blocks.
 
         Prefix reuse is limited to text-only requests: the rows of an image
-        request depend on pixels that the token ids do not identify.
+        request depend on pixels that the token ids do not identify.  `reuse_prefix=False`: every row of this
+        request will be computed (the caller wants them), so it neither reuses nor publishes blocks.
         """
         if seq.block_table:
             raise RuntimeError("sequence already holds blocks")
         if self.num_state_slots:
             seq.state_slot = self.free_state_slots.popleft()
-        use_cache = self.prefix_caching and not seq.has_image
+        use_cache = self.prefix_caching and reuse_prefix and not seq.has_image
         h = -1
         cache_miss = not use_cache
         for i in range(seq.num_blocks):

@@ -133,7 +133,7 @@ class Scheduler:
             else:
                 if not self.block_manager.can_allocate(seq):
                     raise RuntimeError(f"no free blocks or state slot for request {seq.seq_id}")
-                self.block_manager.allocate(seq)
+                self.block_manager.allocate(seq, reuse_prefix=False)
                 self.running.append(seq)
                 seq.status = SequenceStatus.RUNNING
                 done = seq.prefill_start

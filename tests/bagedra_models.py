@@ -88,6 +88,27 @@ def weights(cfg, seed=0, rank=12):
     return out
 
 
+def pointer_model(at, n, spec, seed=2, strength=40.0):
+    """A latent layer whose token 1 asks for token 0: (cfg, weights, prompt) with token 0 only at place `at` and token 1
+    last.  Removing that one key changes the last logits completely."""
+    cfg = config([spec], width=40, ff=24, vocab=60)
+    w = weights(cfg, seed=seed)
+    m, p = spec[1], "l0.mix."
+    e0, e1 = w["embed"][0], w["embed"][1]
+    c0 = oracle.rms(w[p + "dkv"][:m["kv_rank"]] @ e0, 1e-6) * w[p + "dkv.norm"]
+    k0 = (w[p + "uk"] @ c0).view(m["heads"], m["dim"])
+    q = w[p + "q"].view(m["heads"], m["dim"] + m["rot_dim"], -1)
+    q *= 0.02
+    unit = e1 / e1.pow(2).sum()
+    for h in range(m["heads"]):
+        q[h, :m["dim"]] += strength * (k0[h] / k0[h].pow(2).sum())[:, None] * unit / m["scale"]
+    w[p + "q"] = w[p + "q"].bfloat16().float()
+    w[p + "o"] = (w[p + "o"] * 4).bfloat16().float()
+    prompt = [2 + t % (cfg["vocab"] - 2) for t in tokens(n, 10 ** 6, seed)]
+    prompt[at], prompt[-1] = 0, 1
+    return cfg, w, prompt
+
+
 def save(path, cfg, w):
     from safetensors.torch import save_file
     os.makedirs(path, exist_ok=True)

@@ -20,9 +20,20 @@ MODELS = {
                          bm.delta(heads=4, kv_heads=2, dim=128, vdim=128, conv=4),
                          bm.latent(heads=8, dim=64, rot=64, vdim=96, rank=256, kv_from=0),
                          bm.gla(heads=2, dim=64, vdim=256), bm.delta(heads=2, kv_heads=1, dim=96, vdim=64)],
-                 width=256, ff=320, vocab=520),
+                 width=256, ff=384, vocab=520),
     "mid": dict(mixers=[bm.gla(heads=2, dim=32, vdim=64, tau=2.0), bm.latent(heads=20, dim=96, rot=24, vdim=64, rank=128),
                         bm.delta(heads=2, kv_heads=1, dim=64, vdim=128)], width=128, ff=96, vocab=200),
+    "heads": dict(mixers=[bm.latent(heads=40, dim=32, rot=32, vdim=32, rank=128), bm.delta(heads=12, kv_heads=3, dim=16, vdim=16),
+                          bm.latent(heads=70, dim=16, rot=32, vdim=16, rank=128, kv_from=0), bm.gla(heads=12, dim=16, vdim=16)],
+                  width=192, ff=256, vocab=100),
+}
+SINGLE = {
+    "latent": [bm.latent(heads=2, dim=64, rot=32, vdim=64, rank=64)],
+    "latent odd": [bm.latent(heads=2, dim=33, rot=10, vdim=13, rank=37)],
+    "gla": [bm.gla(heads=2, dim=48, vdim=80, tau=4.0)],
+    "gla strong decay": [bm.gla(heads=2, dim=48, vdim=32, tau=0.25)],
+    "delta": [bm.delta(heads=4, kv_heads=2, dim=80, vdim=48, conv=4)],
+    "delta six taps": [bm.delta(heads=2, kv_heads=1, dim=24, vdim=40, conv=6)],
 }
 
 
@@ -50,6 +61,86 @@ def test_portions_decode_and_mixed_batches(name, dtype, tmp_path):
         for i in prompts:
             worst, mean = bm.errors(got[i], want[i])
             assert worst < LIMIT[dtype] and mean < MEAN_LIMIT[dtype], (i, schedule[0], worst, mean)
+    llm.exit()
+
+
+def _check(got, want, dtype, what):
+    worst, mean = bm.errors(got, want)
+    assert worst < LIMIT[dtype] and mean < MEAN_LIMIT[dtype], (what, worst, mean)
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("name", list(SINGLE))
+def test_each_mechanism_in_portions_of_several_sizes(name, dtype, tmp_path):
+    cfg = bm.config(SINGLE[name], width=96, ff=64, vocab=90)
+    w = bm.weights(cfg, seed=11)
+    llm = bm.engine(bm.save(tmp_path / "m", cfg, w), "cuda", dtype)
+    prompts = {"a": bm.tokens(206, cfg["vocab"], 5)}
+    want = bm.expected(cfg, w, prompts)["a"]
+    for sizes in ([206], [2] * 103, [64, 64, 64, 14], [63, 1, 65, 1, 76], [30, 1, 25, 150], [130] + [1] * 76):
+        got = bm.feed(llm, prompts, [[("a", n)] for n in sizes])["a"]
+        _check(got, want, dtype, sizes[:5])
+    llm.exit()
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_single_far_key_at_page_and_tile_borders(dtype, tmp_path):
+    """One key carries the whole answer: prompts, portions and decoding, pages of 16 and of 64 tokens."""
+    n = 420
+    for at in (0, 1, 15, 16, 63, 64, 127, 128, 129, 255, 256, 383, 384, 417):
+        cfg, w, prompt = bm.pointer_model(at, n, bm.latent(heads=2, dim=64, rot=32, vdim=64, rank=64))
+        want = bm.oracle.forward(cfg, w, prompt)[0]
+        path = bm.save(tmp_path / f"m{at}", cfg, w)
+        llm = bm.engine(path, "cuda", dtype, page=64 if at % 2 else 16, enforce_eager=True)
+        for cut in ([n], [n - 1, 1], [at + 1, n - at - 3, 2], [256, 129, n - 385]):
+            got = bm.feed(llm, {"a": prompt}, [[("a", c)] for c in cut if c])["a"]
+            worst, _ = bm.errors(got[-1:], want[-1:])
+            assert worst < (0.05 if dtype == "bfloat16" else 2e-4), (at, cut, worst)
+        llm.exit()
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_pages_and_slots_with_old_contents(dtype, tmp_path):
+    cfg, w, path = _model("wide", tmp_path)
+    llm = bm.engine(path, "cuda", dtype, max_tokens=20 * bm.PAGE, requests=2)
+    for c in llm.model_runner.cache_layout:
+        for name in c.state:
+            getattr(c.module, name).fill_(1e3)
+        if c.row_width:
+            c.module.rows.fill_(1e3)
+    for k in range(4):
+        prompts = {f"x{k}": bm.tokens(130 + k, cfg["vocab"], k), f"y{k}": bm.tokens(90 - 20 * k, cfg["vocab"], 50 + k)}
+        want = bm.expected(cfg, w, prompts)
+        a, b = prompts
+        n, m = len(prompts[a]), len(prompts[b])
+        got = bm.feed(llm, prompts, [[(b, 1)], [(a, 100), (b, 3)], [(a, n - 103), (b, 1)], [(b, m - 8), (a, 1)],
+                                     [(a, 1), (b, 1)], [(a, 1), (b, 1)], [(b, 1)]])
+        for i in prompts:
+            _check(got[i], want[i], dtype, i)
+    llm.exit()
+
+
+def test_general_kernels_in_bf16_agree(tmp_path, monkeypatch):
+    """The forms without tensor cores, where a tensor-core form exists."""
+    from fastcache_b200.ops import hybrid
+    monkeypatch.setattr(hybrid, "LATENT_IMPL", 1)
+    cfg, w, path = _model("wide", tmp_path)
+    prompts = {"a": bm.tokens(90, cfg["vocab"], 1)}
+    llm = bm.engine(path, "cuda", "bfloat16", enforce_eager=True)
+    _check(bm.feed(llm, prompts, [[("a", 70)], [("a", 18)], [("a", 1)], [("a", 1)]])["a"],
+           bm.expected(cfg, w, prompts)["a"], "bfloat16", "general")
+    llm.exit()
+
+
+def test_long_context_decode_with_splits(tmp_path):
+    cfg, w, path = _model("mid", tmp_path)
+    n = 1500
+    prompts = {"a": bm.tokens(n, cfg["vocab"], 1), "b": bm.tokens(n // 3, cfg["vocab"], 2)}
+    want = bm.expected(cfg, w, prompts)
+    llm = bm.engine(path, "cuda", "bfloat16", max_tokens=4096)
+    got = bm.feed(llm, prompts, [[("a", n - 40), ("b", n // 3 - 40)]] + [[("a", 1), ("b", 1)]] * 40)
+    for i in prompts:
+        _check(got[i], want[i], "bfloat16", i)
     llm.exit()
 
 
