@@ -631,6 +631,21 @@ def run_reference(args):
         emit(line)
 
 
+def run_layers(args):
+    """Layer throughput of the hybrid model beside the dense decoder at equal size (no job, no serving loop)."""
+    from benchmarks.hybrid_bench import run
+    from fastcache_b200 import ops
+    sampler = ClockSampler()
+    sampler.start()
+    res = run(max(5, args.steps), args.small)
+    clocks = sampler.stop()
+    last = list(res["sizes"].values())[-1]["rows"][0]
+    emit({"metric": "prefill tokens/s of 8 hybrid layers", "value": last["tok_s"], "unit": "tok/s", "n_gpus": 1,
+          "steps": max(5, args.steps), "warmup": 3, "ms_per_step": last["ms"], "higher_is_better": True, "scaling": "weak",
+          "vs_baseline": None, "dtype": "bf16", "data": "synthetic", "config": {"model": "Bagedra beside Qwen3", **res},
+          "gpu_launches": int(ops.COUNTERS["launches"]), "clocks": clocks})
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -663,6 +678,10 @@ def main():
     ap.add_argument("--check", action="store_true",
                     help="instead of timing: first tokens under --gpus N against the same prompts on one GPU "
                          "(shrunken config, greedy)")
+    ap.add_argument("--layers", action="store_true",
+                    help="instead of the job: prefill and decode throughput of the hybrid model's layers beside the dense "
+                         "decoder at a few equal sizes, and the roofline of their kernels (1 GPU)")
+    ap.add_argument("--small", action="store_true", help="--layers: the smallest size only")
     ap.add_argument("--check-out", default="", help=argparse.SUPPRESS)
     args = ap.parse_args()
     args.warmup = max(3, args.warmup)
@@ -671,7 +690,9 @@ def main():
     if args.check:
         run_check(args)
         return
-    if args.impl == "reference":
+    if args.layers:
+        run_layers(args)
+    elif args.impl == "reference":
         run_reference(args)
     elif args.config in SERVING:
         run_serving(args)

@@ -34,9 +34,17 @@ void check_i32(const Tensor& t, const char* name, int64_t n) {
 }
 
 // x @ w.T.  `partial`: decode-size bf16 products may stay split-K partial sums in the stream's scratch, valid until
-// the next product on this stream.  `hold` keeps the finished output alive.
+// the next product on this stream.  `hold` keeps the finished output alive.  An empty w: x is the projection output.
 fc::ProjSrc project(const Tensor& x, const Tensor& w, const OptTensor& bias, bool partial, Tensor& hold) {
   check_elem(x, "x");
+  if (w.numel() == 0) {
+    TORCH_CHECK(x.dim() == 2 && x.stride(1) == 1 && x.stride(0) % 8 == 0, "bad projection output");
+    fc::ProjSrc done;
+    hold = x;
+    done.p = x.data_ptr();
+    done.ld = x.stride(0);
+    return done;
+  }
   TORCH_CHECK(x.scalar_type() == w.scalar_type() && x.dim() == 2 && w.dim() == 2 && x.size(1) == w.size(1) &&
                   x.stride(1) == 1 && w.is_contiguous() && w.size(1) % 8 == 0 && w.size(0) % 8 == 0 &&
                   x.stride(0) % 8 == 0, "projection operands must be row-major matrices padded to multiples of 8");
@@ -111,7 +119,7 @@ std::tuple<Tensor, Tensor> embed_scaled(const Tensor& ids, const Tensor& weight,
 Tensor linear_post_norm_add(const Tensor& a, const Tensor& w, const OptTensor& bias, Tensor x, const Tensor& norm_w,
                             double eps) {
   c10::cuda::CUDAGuard guard(a.device());
-  const int64_t T = a.size(0), W = x.size(1), Wp = w.size(0);
+  const int64_t T = a.size(0), W = x.size(1), Wp = w.numel() ? w.size(0) : a.size(1);
   check_f32(x, "residual", T * W);
   check_f32(norm_w, "norm weight", W);
   TORCH_CHECK(Wp >= W, "projection narrower than the residual");
@@ -141,7 +149,7 @@ Tensor rms_norm_wide(const Tensor& x, const Tensor& norm_w, double eps, int64_t 
 
 Tensor linear_gelu_mul(const Tensor& h, const Tensor& w, const OptTensor& bias, int64_t up_off, int64_t width) {
   c10::cuda::CUDAGuard guard(h.device());
-  const int64_t T = h.size(0), N = w.size(0), wp = pad8(int(width));
+  const int64_t T = h.size(0), N = w.numel() ? w.size(0) : h.size(1), wp = pad8(int(width));
   TORCH_CHECK(up_off % 8 == 0 && up_off >= width && up_off + wp <= N, "bad gate | up layout");
   const void* bp = nullptr;
   if (bias.has_value() && bias->defined()) {
@@ -150,7 +158,7 @@ Tensor linear_gelu_mul(const Tensor& h, const Tensor& w, const OptTensor& bias, 
   }
   Tensor hold;
   Tensor out = torch::empty({T, wp}, h.options());
-  if (!is_f32(h) && T > 256 && width % 128 == 0 && up_off == width && N == 2 * width) {
+  if (w.numel() && !is_f32(h) && T > 256 && width % 128 == 0 && up_off == width && N == 2 * width) {
     // prefill sizes: the gate runs in the GEMM's epilogue
     const auto& ws = ws_of(h);
     fc::GemmWorkspace gw;
@@ -225,7 +233,7 @@ Tensor gla(const Tensor& h, const Tensor& w, const Tensor& w_a2, const Tensor& z
   check_f32(z_bias, "decay bias", (int64_t)H * D);
   check_f32(norm_w, "head norm", V);
   TORCH_CHECK(w_a2.scalar_type() == h.scalar_type() && w_a2.is_contiguous() && w_a2.size(0) >= H * D &&
-                  w_a2.size(1) >= rank && d[8] + w_a2.size(1) <= w.size(0), "bad decay projection");
+                  w_a2.size(1) >= rank && d[8] + w_a2.size(1) <= (w.numel() ? w.size(0) : h.size(1)), "bad decay projection");
   fc::StepParams p;
   p.H = H;
   p.D = D;
@@ -327,6 +335,23 @@ Tensor delta_rule(const Tensor& h, const Tensor& w, const Tensor& conv_w, const 
   const bool chunk = !is_f32(h) && max_len >= CHUNK_MIN_ROWS && fc::chunk_supported(D, V);
   run_recurrence(p, h, true, chunk, T, int(max_len), out, o_raw);
   return out;
+}
+
+// absorbed attention: the tensor-core form where it takes the sizes; `po` / `pl` keep its scratch alive
+void absorbed(fc::LatentAttn& at, bool f32, int64_t impl, int64_t max_ctx, const Tensor& like, Tensor& po, Tensor& pl) {
+  if (f32 || impl == 1 || !fc::latent_decode_supported(at)) {
+    fc::launch_latent_attn_simt(at, f32, stream_now());
+    return;
+  }
+  at.splits = fc::latent_decode_splits(at, int(max_ctx), fc::gemm_num_sms());
+  if (at.splits > 1) {
+    const auto opt = like.options().dtype(torch::kFloat32);
+    po = torch::empty({(int64_t)at.T * at.H * at.splits * at.rank}, opt);
+    pl = torch::empty({(int64_t)at.T * at.H * at.splits}, opt);
+    at.part_o = po.data_ptr<float>();
+    at.part_lse = pl.data_ptr<float>();
+  }
+  fc::launch_latent_decode(at, stream_now());
 }
 
 // Projection, cache store and attention of a latent-attention layer (up to the output projection).
@@ -499,20 +524,8 @@ Tensor latent_attention(const Tensor& h, const Tensor& w, const std::vector<int6
   at.o_lat = o_lat.data_ptr();
   at.scale = float(scale);
   at.status = ws.status;
-  if (!f32 && impl != 1 && fc::latent_decode_supported(at)) {
-    const int64_t mc = max_ctx > 0 ? max_ctx : block_tables.size(1) * pool.size(1);
-    at.splits = fc::latent_decode_splits(at, int(mc), fc::gemm_num_sms());
-    Tensor po, pl;
-    if (at.splits > 1) {
-      po = torch::empty({(int64_t)T * H * at.splits * rank}, h.options().dtype(torch::kFloat32));
-      pl = torch::empty({(int64_t)T * H * at.splits}, h.options().dtype(torch::kFloat32));
-      at.part_o = po.data_ptr<float>();
-      at.part_lse = pl.data_ptr<float>();
-    }
-    fc::launch_latent_decode(at, stream_now());
-  } else {
-    fc::launch_latent_attn_simt(at, f32, stream_now());
-  }
+  Tensor po, pl;
+  absorbed(at, f32, impl, max_ctx > 0 ? max_ctx : block_tables.size(1) * pool.size(1), o_lat, po, pl);
   a = fc::SimtLinear();
   a.x = o_lat.data_ptr();
   a.w = w_uv.data_ptr();
@@ -539,6 +552,81 @@ Tensor latent_attention(const Tensor& h, const Tensor& w, const std::vector<int6
   return out;
 }
 
+// Absorbed attention alone: q_abs [T, H, rank + R] over the paged rows, one request per row -> [T, H, rank]
+Tensor latent_decode_rows(const Tensor& q_abs, const Tensor& pool, const Tensor& block_tables, const Tensor& ctx,
+                          int64_t rank, double scale) {
+  check_elem(q_abs, "q");
+  check_elem(pool, "cache rows");
+  TORCH_CHECK(q_abs.dim() == 3 && q_abs.is_contiguous() && pool.dim() == 3 && pool.is_contiguous() &&
+                  pool.scalar_type() == q_abs.scalar_type() && pool.size(2) >= q_abs.size(2), "bad operands");
+  c10::cuda::CUDAGuard guard(q_abs.device());
+  const int64_t T = q_abs.size(0), H = q_abs.size(1);
+  check_i32(ctx, "context lengths", T);
+  check_i32(block_tables, "block tables", T);
+  TORCH_CHECK(block_tables.dim() == 2 && block_tables.size(0) >= T, "bad block tables");
+  Tensor o = torch::empty({T, H, rank}, q_abs.options()), po, pl;
+  fc::LatentAttn at;
+  at.T = int(T);
+  at.H = int(H);
+  at.rank = int(rank);
+  at.R = int(q_abs.size(2) - rank);
+  at.row_width = int(pool.size(2));
+  at.block_size = int(pool.size(1));
+  at.max_blocks = int(block_tables.size(1));
+  at.num_blocks = int(pool.size(0));
+  at.q_abs = q_abs.data_ptr();
+  at.pool = pool.data_ptr();
+  at.block_tables = block_tables.data_ptr<int>();
+  at.row_ctx = ctx.data_ptr<int>();
+  at.o_lat = o.data_ptr();
+  at.scale = float(scale);
+  at.status = ws_of(pool).status;
+  absorbed(at, is_f32(q_abs), 0, block_tables.size(1) * pool.size(1), o, po, pl);
+  return o;
+}
+
+// Expanded attention alone: q [T, H, D + R], kv [rows, H * D | H * V], rot [rows, R], gate [T, H * V] -> [T, H * V]
+Tensor latent_prefill_rows(const Tensor& q, const Tensor& kv, const Tensor& rot, const Tensor& gate, const Tensor& cu_q,
+                           const Tensor& cu_kv, int64_t D, int64_t V, double scale, int64_t max_q) {
+  const int64_t T = q.size(0), H = q.size(1), R = rot.size(1), B = cu_q.numel() - 1;
+  TORCH_CHECK(q.is_contiguous() && kv.is_contiguous() && gate.is_contiguous() && rot.stride(1) == 1 && q.size(2) == D + R &&
+                  kv.size(1) == H * (D + V) && gate.size(1) == H * V && gate.size(0) == T && rot.size(0) == kv.size(0) &&
+                  q.scalar_type() == torch::kBFloat16 && kv.scalar_type() == torch::kBFloat16 && q.is_cuda() &&
+                  rot.scalar_type() == torch::kBFloat16 && gate.scalar_type() == torch::kBFloat16, "bad operands");
+  check_i32(cu_q, "cu_q", B + 1);
+  check_i32(cu_kv, "cu_kv", B + 1);
+  c10::cuda::CUDAGuard guard(q.device());
+  Tensor out = torch::empty({T, H * V}, q.options());
+  fc::LatentPrefill a;
+  a.T = int(T);
+  a.B = int(B);
+  a.H = int(H);
+  a.D = int(D);
+  a.R = int(R);
+  a.V = int(V);
+  a.rank = 8;
+  a.max_q = int(max_q);
+  a.total_kv = kv.size(0);
+  TORCH_CHECK(fc::latent_prefill_supported(a), "sizes without a tensor-core form");
+  a.q = q.data_ptr();
+  a.ld_q = H * (D + R);
+  a.k = kv.data_ptr();
+  a.v = reinterpret_cast<const char*>(kv.data_ptr()) + H * D * 2;
+  a.ld_kv = kv.size(1);
+  a.rot = rot.data_ptr();
+  a.ld_rot = rot.stride(0);
+  a.cu_q = cu_q.data_ptr<int>();
+  a.cu_kv = cu_kv.data_ptr<int>();
+  a.gate = gate.data_ptr();
+  a.ld_gate = H * V;
+  a.out = out.data_ptr();
+  a.ld_out = H * V;
+  a.scale = float(scale);
+  a.status = ws_of(q).status;
+  fc::launch_latent_prefill(a, stream_now());
+  return out;
+}
+
 }  // namespace
 
 void register_hybrid(pybind11::module_& m) {
@@ -551,4 +639,6 @@ void register_hybrid(pybind11::module_& m) {
   m.def("gla", &gla);
   m.def("delta_rule", &delta_rule);
   m.def("latent_attention", &latent_attention);
+  m.def("latent_decode_rows", &latent_decode_rows);
+  m.def("latent_prefill_rows", &latent_prefill_rows);
 }

@@ -170,7 +170,7 @@ gather_rows_kernel(const uint8_t* __restrict__ pool, const int* __restrict__ blo
                    const int* __restrict__ cu_kv, uint8_t* __restrict__ out, int chunks, int block_size,
                    int max_blocks, int num_blocks, uint32_t* status) {
   const int b = blockIdx.y;
-  const int n = ctx[b];
+  const int n = min(min(ctx[b], cu_kv[b + 1] - cu_kv[b]), max_blocks * block_size);
   const int per = 256 / chunks > 0 ? 256 / chunks : 1;
   const int row0 = blockIdx.x * per;
   for (int i = threadIdx.x; i < per * chunks; i += 256) {
@@ -212,7 +212,7 @@ latent_attn_simt_kernel(const LatentAttn p) {
   __shared__ const T* srow[LA_TILE];
   const int t = blockIdx.x, h = blockIdx.y;
   const int w = p.rank + p.R;
-  const int ctx = p.row_ctx[t];
+  const int ctx = min(p.row_ctx[t], p.max_blocks * p.block_size);
   const int b = p.row_seq != nullptr ? p.row_seq[t] : t;
   const T* q = reinterpret_cast<const T*>(p.q_abs) + ((long long)t * p.H + h) * w;
   const T* pool = reinterpret_cast<const T*>(p.pool);

@@ -61,7 +61,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm, const LatentAttn p,
   }
   pdl_wait();
   asm volatile("fence.proxy.async.global;" ::: "memory");          // rows were written with ordinary stores
-  const int ctx = p.row_ctx[t];
+  const int ctx = min(p.row_ctx[t], p.max_blocks * p.block_size);
   const int b = p.row_seq != nullptr ? p.row_seq[t] : t;
   const int tiles = (ctx + LD_TILE - 1) / LD_TILE;
   const int per = (tiles + p.splits - 1) / p.splits;

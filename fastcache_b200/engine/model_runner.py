@@ -203,10 +203,17 @@ class ModelRunner:
         self.graph_bs: List[int] = []
         self.graph_vars: Dict[str, torch.Tensor] = {}
         self.graph_pool = None
+        self._main_follows_current()
         if not self.enforce_eager:
             self.capture_cudagraph()
 
     # ------------------------------------------------------------------ setup
+    def _main_follows_current(self) -> None:
+        """Weights, pools and static buffers are filled on the stream that is current while the engine is built; the
+        main stream must not read them before that is done."""
+        if self.main_stream is not None:
+            self.main_stream.wait_stream(torch.cuda.current_stream(self.device))
+
     def _load_weights(self) -> None:
         cfg = self.config
         random_init = bool(cfg.extra.get("random_init", False)) or not cfg.model
@@ -534,6 +541,7 @@ class ModelRunner:
             self.graphs = {b: None for b in self.graph_bs}
             return
         stream = self.main_stream or torch.cuda.current_stream()
+        self._main_follows_current()
         with torch.cuda.stream(stream):
             for b in reversed(self.graph_bs):
                 self._decode_on_static(b)            # warm-up (allocations, lazy init)

@@ -5,11 +5,13 @@ the same blocks and state slots and run by the same prefill and decode steps as 
 """
 from __future__ import annotations
 
+from contextlib import nullcontext
 from typing import Any, Dict, List, Sequence as Seq
 
 import numpy as np
 import torch
 
+from ..utils.context import reset_context
 from .llm_engine import LLMEngine
 from .sequence import Sequence
 
@@ -35,11 +37,14 @@ class TokenReplay:
             seqs = sch.schedule_pieces(pieces)
             offsets = np.concatenate([[0], np.cumsum([len(t) for _, t in pieces])])
             rows = [int(o) + int(w) for o, e in zip(offsets, entries) for w in e.get("want", ())]
-            if all(len(t) == 1 and s.prefill_start > 0 for s, t in pieces):
-                got = runner.run_decode(seqs)[rows]
-            else:
-                got = runner.run_prefill(seqs, logits_rows=rows)
-            logits = got.float().cpu()
+            stream = torch.cuda.stream(runner.main_stream) if runner.main_stream is not None else nullcontext()
+            with stream:
+                if all(len(t) == 1 and s.prefill_start > 0 for s, t in pieces):
+                    got = runner.run_decode(seqs)[rows]
+                else:
+                    got = runner.run_prefill(seqs, logits_rows=rows)
+                logits = got.float().cpu()
+            reset_context()
             for s in seqs:
                 s.num_computed_tokens, s.prefill_end = s.prefill_end, None
         self.llm.check_device_status()
