@@ -2,11 +2,11 @@
 its kernels beside the like kernels of the dense decoder.
 
     python bench.py --layers [--small]        # throughput and kernels, one JSON line
-    python benchmarks/hybrid_bench.py         # the same, a readable table
+    python benchmarks/hybrid_bench.py [--kernels]    # the same (or the kernels alone) as a readable table
 
 Random weights.  Throughput: whole forward steps through the engine's prefill and decode steps (CUDA graphs in decode),
 CUDA events on the engine's stream, 3 warm-up steps, median; the weights and caches of a step are larger than L2.
-Kernels: CUDA events around single operations, a 256 MB write between samples to flush L2, median; fractions are of the
+Kernels: CUDA events around single operations (replays of a CUDA graph), a 256 MB write between samples to flush L2, median; fractions are of the
 measured peaks in MEASURED_PEAKS.json (algorithmic bytes and FLOPs).
 """
 import json
@@ -122,6 +122,20 @@ def throughput(cfg, steps):
     return rows
 
 
+def graphed(fn):
+    """`fn` as a CUDA-graph replay: what is timed is the device, not the launches from Python."""
+    stream = torch.cuda.Stream()
+    stream.wait_stream(torch.cuda.current_stream())
+    with torch.cuda.stream(stream):
+        for _ in range(2):
+            fn()
+    stream.synchronize()
+    g = torch.cuda.CUDAGraph()
+    with torch.cuda.graph(g, stream=stream):
+        fn()
+    return g.replay
+
+
 def kernel_table():
     """Kernels of the 4k size and the like kernels of the dense decoder."""
     from benchmarks.kernel_bench import peaks, timeit
@@ -139,10 +153,11 @@ def kernel_table():
     def i32(*v):
         return torch.tensor(v, dtype=torch.int32, device=dev)
 
-    def add(kernel, case, fn, byts, flops=0.0, like=None):
-        ms = timeit(fn)
+    def add(kernel, case, fn, byts, flops=0.0, like=None, like_case=None):
+        ms = timeit(graphed(fn))
         roof = max(byts / (hbm * 1e9), flops / (tf * 1e12)) * 1e3
-        rows.append({"kernel": kernel, "case": case, "ms": round(ms, 4), "of_roofline": round(roof / ms, 3), "like": like})
+        rows.append({"kernel": kernel, "case": case, "ms": round(ms, 4), "of_roofline": round(roof / ms, 3), "like": like,
+                     "like_case": like_case or case})
 
     none = torch.empty(0, device=dev, dtype=bf)
     T = 8192
@@ -208,22 +223,24 @@ def kernel_table():
         add("delta: convolution, chunked recurrence, gates, head norm", f"{b} x {n}",
             lambda: e.delta_rule(dproj, none, cw, hv, hv, hn, 1e-6, cs, st, dd, 1e-6, cu, lens, slots, n, seq),
             T * 2 * (H * D + 3 * H * V), fl + b * n * H * 2 * D * V)
-    for b, n in ((64, 1), (8, 1), (1, 1)):
+    for b, dense in ((64, "64 x 2048"), (8, "8 x 8192"), (1, "1 x 4096")):
         st, cs = torch.zeros(b, H, D, V, device=dev), torch.zeros(b, 3, C, device=dev)
         lens, slots = i32(*([100] * b)), torch.arange(b, device=dev, dtype=torch.int32)
         p1, p2 = proj[:b].contiguous(), dproj[:b].contiguous()
         add("gla step", f"{b} requests",
             lambda: e.gla(p1, none, a2, zb, hn, 1e-6, st, gd, 16.0, None, lens, slots, 1), b * H * D * V * 8,
-            like="decode_attention (dense)")
+            like="decode_attention (dense)", like_case=dense)
         add("delta inputs + step", f"{b} requests",
             lambda: e.delta_rule(p2, none, cw, hv, hv, hn, 1e-6, cs, st, dd, 1e-6, None, lens, slots, 1, None),
-            b * H * D * V * 8, like="decode_attention (dense)")
+            b * H * D * V * 8, like="decode_attention (dense)", like_case=dense)
     by = {(r["kernel"], r["case"]): r["of_roofline"] for r in rows}
     for r in rows:
         if r["like"]:
-            ref = by.get((r["like"], r["case"])) or next((v for (k, _), v in by.items() if k == r["like"]), None)
+            ref = by.get((r["like"], r["like_case"])) or next(v for (k, _), v in by.items() if k == r["like"])
             r["like_of_roofline"] = ref
             r["times_as_far"] = round(ref / r["of_roofline"], 2)
+        else:
+            del r["like"], r["like_case"]
     return rows, src
 
 
@@ -242,6 +259,10 @@ def run(steps=5, small=False, kernels=True):
 
 
 def main():
+    if "--kernels" in sys.argv:
+        for r in kernel_table()[0]:
+            print(json.dumps(r))
+        return
     res = run()
     for name, s in res["sizes"].items():
         for r in s["rows"]:

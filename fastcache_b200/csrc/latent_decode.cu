@@ -1,14 +1,16 @@
 // Absorbed latent attention of decode-size batches (bf16): every query row attends to the cache rows of its request as
 // they are, key = [latent | rotated part], value = latent, shared by all heads.
 //
-// Grid (query row, group of 16 * MT heads, split of the context).  A CTA streams 64-row tiles of the cache through a
-// two-stage TMA ring (128-byte swizzle, boxes that never straddle a page); one tile in shared memory is both the keys
-// and the values of all its heads, so a row is read once.  Per tile:
-//   scores   warp w: 16 keys (w & 3) against all heads, a quarter of the columns (w >> 2), mma.sync m16n8k16; the
+// Grid (query row, group of 16 * MT heads, split of the context).  One tile of 32 cache rows in shared memory is both the
+// keys and the values of all heads of the CTA, so a row is read once.  Two groups of eight warps take alternate tiles, each
+// with its own two-stage TMA ring (128-byte swizzle, boxes that never straddle a page), running maximum and accumulators:
+// while one group is in a latency-bound phase the other keeps the pipes busy.  Per tile and group:
+//   scores   warp w: 16 keys (w & 1) against all heads, a quarter of the columns (w >> 1), mma.sync m16n8k16; the
 //            quarters are added when they are read back
-//   softmax  32 / MT threads per head, running maximum and sum in registers, P to shared memory as bf16
-//   values   warp w owns the latent columns of 16-column groups w, w + 16, ...; P V accumulates in registers
-// With several splits a CTA writes normalised partials with their log-sum-exp and a second kernel merges them.
+//   softmax  16 / MT threads per head, running maximum and sum in registers, P to shared memory as bf16
+//   values   warp w owns the latent columns of 16-column groups w, w + 8, ...; P V accumulates in registers
+// The groups are merged in shared memory at the end.  With several splits a CTA writes normalised partials with their
+// log-sum-exp and a second kernel merges them.
 //
 // Also here: the per-head products around it (queries into the latent space, outputs out of it).
 #include <algorithm>
@@ -23,9 +25,10 @@
 namespace fc {
 
 using bf16 = __nv_bfloat16;
-constexpr int LD_TILE = 64, LD_STAGES = 2, LD_WARPS = 16, LD_THREADS = LD_WARPS * 32;
-constexpr int LD_PARTS = LD_WARPS / 4;           // column ranges of the scores
-constexpr int LD_SUB = LD_TILE * 128;             // bytes of a [64 rows x 64 columns] sub-tile
+constexpr int LD_TILE = 32, LD_STAGES = 2, LD_GROUPS = 2;
+constexpr int LD_WARPS = 8, LD_GT = LD_WARPS * 32, LD_THREADS = LD_GROUPS * LD_GT;      // warps and threads of a group
+constexpr int LD_PARTS = 4;                      // column ranges of the scores
+constexpr int LD_SUB = LD_TILE * 128;             // bytes of a [32 rows x 64 columns] sub-tile
 constexpr int LD_MAX_SPLITS = 32;
 
 // byte offset of 16-byte chunk `chunk` of row `row` in sub-tiles of `rows` rows x 128 bytes
@@ -37,25 +40,28 @@ template <int MT, int NPW>
 __global__ void __launch_bounds__(LD_THREADS, 1)
 latent_decode_kernel(const __grid_constant__ CUtensorMap tm, const LatentAttn p, int box_rows, int nc, float scale_log2) {
   constexpr int HR = MT * 16;                     // head rows of this CTA
-  constexpr int TPR = LD_THREADS / HR;            // softmax threads per head row
+  constexpr int TPR = LD_GT / HR;                 // softmax threads per head row
   constexpr int KPT = LD_TILE / TPR;              // keys per softmax thread
+  constexpr int SLD = LD_TILE + 4;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   const int stage_bytes = nc * LD_SUB;
-  uint8_t* s_kv = smem;                                            // [LD_STAGES]
-  uint8_t* s_q = s_kv + LD_STAGES * stage_bytes;                   // [nc][HR][128 B]
-  uint8_t* s_p = s_q + nc * HR * 128;                              // [HR][128 B]
-  float* s_s = reinterpret_cast<float*>(s_p + HR * 128);           // [LD_PARTS][HR][LD_TILE + 4]
-  float* s_cor = s_s + LD_PARTS * HR * (LD_TILE + 4);                     // [HR]
-  float* s_l = s_cor + HR;                                         // [HR]
-  uint64_t* full = reinterpret_cast<uint64_t*>(s_l + HR);          // [LD_STAGES]
-  constexpr int SLD = LD_TILE + 4;
+  const int tid = threadIdx.x, grp = tid / LD_GT, gt = tid % LD_GT, warp = gt >> 5, lane = tid & 31;
+  uint8_t* s_all = smem;                                                     // [group][stage]
+  uint8_t* s_q = s_all + LD_GROUPS * LD_STAGES * stage_bytes;                // [nc][HR][128 B]
+  uint8_t* s_p = s_q + nc * HR * 128 + grp * HR * 128;                       // [group][HR][128 B]
+  float* s_s = reinterpret_cast<float*>(s_q + nc * HR * 128 + LD_GROUPS * HR * 128) + grp * LD_PARTS * HR * SLD;
+  float* s_m = reinterpret_cast<float*>(s_q + nc * HR * 128 + LD_GROUPS * HR * 128) + LD_GROUPS * LD_PARTS * HR * SLD;
+  float* s_cor = s_m + 2 * HR + grp * HR;                                    // s_m: [2][HR] maximum and sum of group 1
+  uint64_t* bars = reinterpret_cast<uint64_t*>(s_m + (2 + LD_GROUPS) * HR);  // [group][stage]
+  uint8_t* s_kv = s_all + grp * LD_STAGES * stage_bytes;
+  uint64_t* full = bars + grp * LD_STAGES;
+  auto group_sync = [&]() { asm volatile("bar.sync %0, %1;" ::"r"(grp + 1), "r"(LD_GT) : "memory"); };
 
   const int t = blockIdx.x, h0 = blockIdx.y * HR, split = blockIdx.z;
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   pdl_launch_dependents();
   if (tid == 0) {
-    for (int s = 0; s < LD_STAGES; ++s) mbar_init(&full[s], 1);
+    for (int s = 0; s < LD_GROUPS * LD_STAGES; ++s) mbar_init(&bars[s], 1);
     fence_barrier_init();
     tma_prefetch_desc(&tm);
   }
@@ -66,6 +72,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm, const LatentAttn p,
   const int tiles = (ctx + LD_TILE - 1) / LD_TILE;
   const int per = (tiles + p.splits - 1) / p.splits;
   const int tile0 = split * per, n_tiles = max(0, min(tiles, tile0 + per) - tile0);
+  const int n_mine = (n_tiles - grp + LD_GROUPS - 1) / LD_GROUPS;  // tiles grp, grp + 2, ...
   const int* bt = p.block_tables + (long long)b * p.max_blocks;
   const int w = p.rank + p.R;
 
@@ -78,16 +85,16 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm, const LatentAttn p,
                                                 ((long long)t * p.H + h0 + r) * w + ch * 8));
     *reinterpret_cast<uint4*>(s_q + ld_swz(HR, r, ch)) = v;
   }
-  if (n_tiles <= LD_STAGES) {
+  if (n_tiles <= LD_GROUPS * LD_STAGES) {
     // boxes past the context are never loaded: what they would hold must be finite
-    for (int i = tid; i < n_tiles * stage_bytes / 16; i += LD_THREADS)
-      reinterpret_cast<uint4*>(s_kv)[i] = make_uint4(0, 0, 0, 0);
+    for (int i = tid; i < LD_GROUPS * LD_STAGES * stage_bytes / 16; i += LD_THREADS)
+      reinterpret_cast<uint4*>(s_all)[i] = make_uint4(0, 0, 0, 0);
     fence_proxy_async();
   }
   __syncthreads();
 
-  auto load_tile = [&](int tile, int stage) {
-    const int row0 = tile * LD_TILE;
+  auto load_tile = [&](int it) {                                   // the group's it-th tile
+    const int stage = it % LD_STAGES, row0 = (tile0 + grp + it * LD_GROUPS) * LD_TILE;
     const int pieces = min(LD_TILE / box_rows, (ctx - row0 + box_rows - 1) / box_rows);
     mbar_expect_tx(&full[stage], uint32_t(pieces) * nc * box_rows * 128);
     for (int pc = 0; pc < pieces; ++pc) {
@@ -102,11 +109,11 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm, const LatentAttn p,
         tma_load_2d(s_kv + stage * stage_bytes + c * LD_SUB + pc * box_rows * 128, &tm, &full[stage], c * 64, grow);
     }
   };
-  if (tid == 0)
+  if (gt == 0)
     for (int s = 0; s < LD_STAGES; ++s)
-      if (s < n_tiles) load_tile(tile0 + s, s);
+      if (s < n_mine) load_tile(s);
 
-  const int g = lane >> 2, q4 = lane & 3;
+  const int g = lane >> 2, q4 = lane & 3, mat = lane >> 3;
   float o[MT][NPW][2][4];
 #pragma unroll
   for (int m = 0; m < MT; ++m)
@@ -114,29 +121,24 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm, const LatentAttn p,
     for (int n = 0; n < NPW; ++n)
 #pragma unroll
       for (int e = 0; e < 8; ++e) o[m][n][e >> 2][e & 3] = 0.f;
-  const int srow = tid / TPR, sk0 = (tid % TPR) * KPT;             // softmax: head row and first key of this thread
+  const int srow = gt / TPR, sk0 = (gt % TPR) * KPT;               // softmax: head row and first key of this thread
   float m_run = -INFINITY, l_run = 0.f;
   const int ksteps = (p.row_width + 15) / 16, kpart = (ksteps + LD_PARTS - 1) / LD_PARTS;
-  const int kg = (warp & 3) * 16, part = warp >> 2;
+  const int kg = (warp & 1) * 16, part = warp >> 1;
   const int k_lo = part * kpart, k_hi = min(ksteps, k_lo + kpart);
   const uint32_t q_base = smem_u32(s_q), p_base = smem_u32(s_p);
-  bool alive = true;
-  for (int it = 0; it < n_tiles; ++it) {
+  bool alive = true;                                               // false: a tile never landed (the status word says so)
+  for (int it = 0; it < n_mine; ++it) {
     const int stage = it % LD_STAGES;
-    if (!mbar_wait(&full[stage], (it / LD_STAGES) & 1, p.status, ST_TIMEOUT_FULL)) alive = false;
-    if (__syncthreads_or(!alive)) {
-      alive = false;
-      break;
-    }
+    if (alive) alive = mbar_wait(&full[stage], (it / LD_STAGES) & 1, p.status, ST_TIMEOUT_FULL);
     const uint32_t kv = smem_u32(s_kv + stage * stage_bytes);
-    // ---- scores of 16 keys, half of the columns
+    // ---- scores of 16 keys, a quarter of the columns
     float sc[MT][2][4];
 #pragma unroll
     for (int m = 0; m < MT; ++m)
 #pragma unroll
       for (int e = 0; e < 8; ++e) sc[m][e >> 2][e & 3] = 0.f;
-    const int mat = lane >> 3;
-#pragma unroll 4
+#pragma unroll 3
     for (int kk = k_lo; kk < k_hi; ++kk) {
       uint32_t b0, b1, b2, b3;
       ldsm_x4(kv + ld_swz(LD_TILE, kg + (mat >> 1) * 8 + (lane & 7), kk * 2 + (mat & 1)), b0, b1, b2, b3);
@@ -156,10 +158,10 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm, const LatentAttn p,
         *reinterpret_cast<float2*>(d) = make_float2(sc[m][n][0], sc[m][n][1]);
         *reinterpret_cast<float2*>(d + 8 * SLD) = make_float2(sc[m][n][2], sc[m][n][3]);
       }
-    __syncthreads();
+    group_sync();
     // ---- softmax of one head row by TPR threads
     {
-      const int valid = ctx - (tile0 + it) * LD_TILE;              // keys of this tile that exist
+      const int valid = ctx - (tile0 + grp + it * LD_GROUPS) * LD_TILE;      // keys of this tile that exist
       float v[KPT];
       float mx = -INFINITY;
 #pragma unroll
@@ -184,13 +186,14 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm, const LatentAttn p,
         *reinterpret_cast<uint32_t*>(s_p + ld_swz(HR, srow, key >> 3) + (key & 7) * 2) = pack_bf16(e0, e1);
       }
       l_run = l_run * cor + rs;
-      if (tid % TPR == 0) s_cor[srow] = cor;
+      if (gt % TPR == 0) s_cor[srow] = cor;
     }
-    __syncthreads();
+    group_sync();
     // ---- O = O * cor + P V
 #pragma unroll
     for (int m = 0; m < MT; ++m) {
       const float c0 = s_cor[m * 16 + g], c1 = s_cor[m * 16 + g + 8];
+      if (c0 == 1.f && c1 == 1.f) continue;
 #pragma unroll
       for (int n = 0; n < NPW; ++n)
 #pragma unroll
@@ -210,7 +213,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm, const LatentAttn p,
                 a[m][3]);
 #pragma unroll
       for (int n = 0; n < NPW; ++n) {
-        const int cg = warp + n * LD_WARPS;                               // 16-column group of the latent
+        const int cg = warp + n * LD_WARPS;                        // 16-column group of the latent
         if (cg * 16 >= p.rank) continue;
         uint32_t b0, b1, b2, b3;
         ldsm_x4_t(kv + ld_swz(LD_TILE, ks * 16 + (mat & 1) * 8 + (lane & 7), cg * 2 + (mat >> 1)), b0, b1, b2, b3);
@@ -221,26 +224,46 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm, const LatentAttn p,
         }
       }
     }
-    __syncthreads();                                               // every warp is done with this stage, S and P
-    if (tid == 0 && it + LD_STAGES < n_tiles) load_tile(tile0 + it + LD_STAGES, stage);
+    group_sync();                                                  // every warp is done with this stage, S and P
+    if (gt == 0 && alive && it + LD_STAGES < n_mine) load_tile(it + LD_STAGES);
   }
-  // ---- finish: 1 / l per head row, then either the result or a normalised partial
+  // ---- merge the groups: group 1 leaves its accumulators, maxima and sums in shared memory, group 0 combines and writes
 #pragma unroll
   for (int x = 1; x < TPR; x <<= 1) l_run += __shfl_xor_sync(0xffffffffu, l_run, x);
-  if (tid % TPR == 0) {
-    s_l[srow] = alive && l_run > 0.f ? 1.f / l_run : 0.f;
-    if (p.splits > 1 && h0 + srow < p.H)
-      p.part_lse[((long long)t * p.H + h0 + srow) * p.splits + split] =
-          alive && l_run > 0.f ? m_run + log2f(l_run) : -INFINITY;
+  __syncthreads();
+  float* s_o = reinterpret_cast<float*>(s_all);                    // [value of a thread][thread of the group]
+  if (grp == 1) {
+    if (gt % TPR == 0) {
+      s_m[srow] = m_run;
+      s_m[HR + srow] = l_run;
+    }
+#pragma unroll
+    for (int m = 0; m < MT; ++m)
+#pragma unroll
+      for (int n = 0; n < NPW; ++n)
+#pragma unroll
+        for (int e = 0; e < 8; ++e) s_o[((m * NPW + n) * 8 + e) * LD_GT + gt] = o[m][n][e >> 2][e & 3];
   }
   __syncthreads();
+  if (grp == 1) return;
+  float* s_w = s_cor;                                              // [2][HR] weight / sum of the two groups
+  if (gt % TPR == 0) {
+    const float m1 = s_m[srow], mm = fmaxf(m_run, m1);
+    const float w0 = m_run == -INFINITY ? 0.f : exp2f(m_run - mm), w1 = m1 == -INFINITY ? 0.f : exp2f(m1 - mm);
+    const float l = l_run * w0 + s_m[HR + srow] * w1, inv = l > 0.f ? 1.f / l : 0.f;
+    s_w[srow] = w0 * inv;
+    s_w[HR + srow] = w1 * inv;
+    if (p.splits > 1 && h0 + srow < p.H)
+      p.part_lse[((long long)t * p.H + h0 + srow) * p.splits + split] = l > 0.f ? mm + log2f(l) : -INFINITY;
+  }
+  group_sync();
 #pragma unroll
   for (int m = 0; m < MT; ++m)
 #pragma unroll
     for (int half = 0; half < 2; ++half) {
       const int r = m * 16 + half * 8 + g;
       if (h0 + r >= p.H) continue;
-      const float inv = s_l[r];
+      const float w0 = s_w[r], w1 = s_w[HR + r];
       const long long row = (long long)t * p.H + h0 + r;
 #pragma unroll
       for (int n = 0; n < NPW; ++n) {
@@ -248,8 +271,9 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm, const LatentAttn p,
         if (cg * 16 >= p.rank) continue;
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
-          const int col = cg * 16 + e * 8 + q4 * 2;
-          const float a = o[m][n][e][half * 2] * inv, c = o[m][n][e][half * 2 + 1] * inv;
+          const int col = cg * 16 + e * 8 + q4 * 2, i0 = (m * NPW + n) * 8 + e * 4 + half * 2;
+          const float a = o[m][n][e][half * 2] * w0 + s_o[i0 * LD_GT + gt] * w1;
+          const float c = o[m][n][e][half * 2 + 1] * w0 + s_o[(i0 + 1) * LD_GT + gt] * w1;
           if (p.splits == 1)
             *reinterpret_cast<uint32_t*>(reinterpret_cast<bf16*>(p.o_lat) + row * p.rank + col) = pack_bf16(a, c);
           else
@@ -258,34 +282,40 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm, const LatentAttn p,
       }
     }
 }
-
-// o_lat[row] = sum_s 2^(lse_s - max) part_o[row, s] / sum_s 2^(lse_s - max); one warp per (row, head), 4 columns a lane
-__global__ void __launch_bounds__(256)
+// o_lat[row] = sum_s 2^(lse_s - max) part_o[row, s] / sum_s 2^(lse_s - max); one CTA per (row, head), 4 columns a thread
+__global__ void __launch_bounds__(128)
 latent_merge_kernel(const LatentAttn p) {
+  __shared__ float s_w[LD_MAX_SPLITS];
   pdl_launch_dependents();
   pdl_wait();
-  const long long row = blockIdx.x * 8ll + (threadIdx.x >> 5);
-  if (row >= (long long)p.T * p.H) return;
-  const int lane = threadIdx.x & 31;
-  const float l = lane < p.splits ? __ldcg(p.part_lse + row * p.splits + lane) : -INFINITY;
-  const float mx = warp_max(l);
-  const float wgt = l == -INFINITY ? 0.f : exp2f(l - mx);
-  const float den = warp_sum(wgt);
-  const float inv = den > 0.f ? 1.f / den : 0.f;
-  for (int c0 = 0; c0 < p.rank; c0 += 128) {                       // every lane stays for the shuffles
-    const int c = c0 + lane * 4;
+  const long long row = blockIdx.x;
+  if (threadIdx.x < 32) {
+    const int lane = threadIdx.x;
+    const float l = lane < p.splits ? __ldcg(p.part_lse + row * p.splits + lane) : -INFINITY;
+    const float mx = warp_max(l);
+    const float wgt = l == -INFINITY ? 0.f : exp2f(l - mx);
+    const float den = warp_sum(wgt);
+    s_w[lane] = den > 0.f ? wgt / den : 0.f;
+  }
+  __syncthreads();
+  for (int c = threadIdx.x * 4; c < p.rank; c += 512) {
     float a[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll 8
     for (int s = 0; s < p.splits; ++s) {
-      const float f = __shfl_sync(0xffffffffu, wgt, s) * inv;
-      if (c >= p.rank) continue;
+      const float f = s_w[s];
       const float4 v = __ldcg(reinterpret_cast<const float4*>(p.part_o + (row * p.splits + s) * p.rank + c));
       a[0] = fmaf(f, v.x, a[0]);
       a[1] = fmaf(f, v.y, a[1]);
       a[2] = fmaf(f, v.z, a[2]);
       a[3] = fmaf(f, v.w, a[3]);
     }
-    if (c < p.rank) store4(reinterpret_cast<bf16*>(p.o_lat) + row * p.rank + c, a[0], a[1], a[2], a[3]);
+    store4(reinterpret_cast<bf16*>(p.o_lat) + row * p.rank + c, a[0], a[1], a[2], a[3]);
   }
+}
+void launch_latent_merge(const LatentAttn& p, cudaStream_t s) {
+  launch_pdl(PDL_DECODE_MERGE, latent_merge_kernel, dim3(unsigned((long long)p.T * p.H)), dim3(128), 0, s, p);
+  const cudaError_t e = cudaGetLastError();
+  if (e != cudaSuccess) throw std::runtime_error(std::string("latent merge: ") + cudaGetErrorString(e));
 }
 
 static int ld_box_rows(int block_size) {
@@ -295,12 +325,13 @@ static int ld_box_rows(int block_size) {
 }
 static int ld_nc(const LatentAttn& p) { return (p.row_width + 63) / 64; }
 static int ld_smem(int mt, int nc) {
-  return LD_STAGES * nc * LD_SUB + nc * mt * 16 * 128 + mt * 16 * 128 + LD_PARTS * mt * 16 * (LD_TILE + 4) * 4 +
-         2 * mt * 16 * 4 + 64 + 1024;
+  const int hr = mt * 16;
+  return LD_GROUPS * LD_STAGES * nc * LD_SUB + nc * hr * 128 + LD_GROUPS * hr * 128 +
+         LD_GROUPS * LD_PARTS * hr * (LD_TILE + 4) * 4 + (2 + LD_GROUPS) * hr * 4 + LD_GROUPS * LD_STAGES * 8 + 1024;
 }
 static int ld_mt(const LatentAttn& p) {
   int mt = p.H > 32 ? 4 : p.H > 16 ? 2 : 1;
-  while (mt > 1 && ld_smem(mt, ld_nc(p)) > 227 * 1024) mt >>= 1;
+  while (mt > 1 && (ld_smem(mt, ld_nc(p)) > 227 * 1024 || (mt == 4 && p.rank > 256))) mt >>= 1;
   return mt;
 }
 
@@ -312,7 +343,7 @@ bool latent_decode_supported(const LatentAttn& p) {
 int latent_decode_splits(const LatentAttn& p, int max_ctx, int num_sms) {
   const int hr = ld_mt(p) * 16;
   const int ctas = p.T * ((p.H + hr - 1) / hr);
-  const int by_len = std::max(1, max_ctx / (4 * LD_TILE));
+  const int by_len = std::max(1, max_ctx / (4 * LD_TILE));      // two tiles per group at least
   int s = std::max(1, std::min({num_sms / std::max(1, ctas), by_len, LD_MAX_SPLITS}));
   if (ctas < num_sms && ctas * 3 > num_sms * 2) s = 1;             // nearly a full wave already
   return s;
@@ -331,14 +362,13 @@ void launch_latent_decode(const LatentAttn& p, cudaStream_t s) {
   };
   auto pick = [&](auto m) {
     constexpr int MT = decltype(m)::value;
-    if (p.rank <= 256) go(latent_decode_kernel<MT, 1>);
-    else go(latent_decode_kernel<MT, 2>);
+    if (p.rank <= 128) go(latent_decode_kernel<MT, 1>);
+    else if (p.rank <= 256) go(latent_decode_kernel<MT, 2>);
+    else if constexpr (MT < 4) go(latent_decode_kernel<MT, 4>);    // ld_mt keeps the accumulators in registers
   };
   if (mt == 1) pick(std::integral_constant<int, 1>{});
   else if (mt == 2) pick(std::integral_constant<int, 2>{});
   else pick(std::integral_constant<int, 4>{});
-  if (p.splits > 1)
-    launch_pdl(PDL_DECODE_MERGE, latent_merge_kernel, dim3(unsigned(((long long)p.T * p.H + 7) / 8)), dim3(256), 0, s, p);
   const cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess) throw std::runtime_error(std::string("latent decode: ") + cudaGetErrorString(e));
 }

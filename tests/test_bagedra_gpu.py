@@ -120,16 +120,47 @@ def test_pages_and_slots_with_old_contents(dtype, tmp_path):
     llm.exit()
 
 
-def test_general_kernels_in_bf16_agree(tmp_path, monkeypatch):
-    """The forms without tensor cores, where a tensor-core form exists."""
+@pytest.mark.parametrize("impl", [1, 2])
+@pytest.mark.parametrize("name", ["wide", "heads"])
+def test_other_forms_of_latent_attention_agree(name, impl, tmp_path, monkeypatch):
+    """The forms without tcgen05 (1: no tensor cores, 2: mma.sync) where a tcgen05 form exists."""
     from fastcache_b200.ops import hybrid
-    monkeypatch.setattr(hybrid, "LATENT_IMPL", 1)
-    cfg, w, path = _model("wide", tmp_path)
+    monkeypatch.setattr(hybrid, "LATENT_IMPL", impl)
+    cfg, w, path = _model(name, tmp_path)
     prompts = {"a": bm.tokens(90, cfg["vocab"], 1)}
     llm = bm.engine(path, "cuda", "bfloat16", enforce_eager=True)
     _check(bm.feed(llm, prompts, [[("a", 70)], [("a", 18)], [("a", 1)], [("a", 1)]])["a"],
            bm.expected(cfg, w, prompts)["a"], "bfloat16", "general")
     llm.exit()
+
+
+def _absorbed(q, pool, bt, ctx, rank, scale):
+    out = []
+    for i, n in enumerate(ctx.tolist()):
+        rows = pool[bt[i].long()].reshape(-1, pool.shape[-1])[:n, :q.shape[-1]].double()
+        s = (q[i].double() @ rows.T) * scale
+        out.append(torch.softmax(s, -1) @ rows[:, :rank] if n else torch.zeros(q.shape[1], rank, device=q.device))
+    return torch.stack([o.double() for o in out])
+
+
+@pytest.mark.parametrize("impl", [0, 2])
+@pytest.mark.parametrize("H,rank,R,page", [(32, 512, 64, 64), (5, 128, 32, 16), (70, 256, 64, 256), (33, 64, 32, 8),
+                                           (16, 320, 64, 32), (1, 16, 8, 128)])
+def test_absorbed_attention_over_pages(H, rank, R, page, impl):
+    from fastcache_b200.ops.loader import ext
+    g = torch.Generator(device="cuda").manual_seed(H)
+    ctx = torch.tensor([1, 700, 0, 127, 128, 129, 1030, 2500, 64], dtype=torch.int32, device="cuda")
+    pages = -(-2500 // page)
+    B = ctx.numel()
+    pool = torch.randn(B * pages, page, rank + R, device="cuda", generator=g).bfloat16()
+    bt = torch.randperm(B * pages, device="cuda", generator=g).int().view(B, pages)
+    q = torch.randn(B, H, rank + R, device="cuda", generator=g).bfloat16()
+    for scale in (0.02, 0.5, 8.0):            # the last: scores hundreds of e-folds apart, one row takes all
+        got = ext().latent_decode_rows(q, pool, bt, ctx, rank, scale, impl).double()
+        want = _absorbed(q, pool, bt, ctx, rank, scale)
+        err = (got - want).abs().max().item()
+        assert err < 0.04, (scale, err)
+    assert ext().read_status(0) == 0
 
 
 def test_long_context_decode_with_splits(tmp_path):
