@@ -15,7 +15,7 @@ from . import reference_hybrid as ref
 from .loader import ext
 
 
-LATENT_IMPL = 0         # 1: the general kernels also where a tensor-core form exists (tests)
+LATENT_IMPL = 0         # tests: 1 the general kernels also where a tensor-core form exists, 2 absorbed also in prefill
 
 
 def _n(k: int = 1) -> None:

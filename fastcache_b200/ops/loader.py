@@ -1,7 +1,8 @@
 """Locates the compiled extension that holds the sm_100a kernels.
 
 The shared object is built in-tree (`python setup.py build_ext --inplace`, or
-`build()` in the repository's entry file) as `fastcache_b200/_C*.so`.
+`build()` in the repository's entry file) as `fastcache_b200/_C*.so`; with `FC_EXT=core` only the part that hybrid
+models need, as `_C_core`.
 """
 from __future__ import annotations
 
@@ -16,7 +17,10 @@ class ExtensionMissing(RuntimeError):
 @lru_cache(maxsize=1)
 def _load():
     import torch  # noqa: F401  (registers libc10/libtorch for the extension's loader)
-    return importlib.import_module("fastcache_b200._C")
+    try:
+        return importlib.import_module("fastcache_b200._C")
+    except ModuleNotFoundError:
+        return importlib.import_module("fastcache_b200._C_core")      # a build of the core sources alone
 
 
 def ext_available() -> bool:

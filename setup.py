@@ -10,7 +10,13 @@ from torch.utils.cpp_extension import BuildExtension, CUDAExtension
 
 ROOT = os.path.dirname(os.path.abspath(__file__))
 SRC = os.path.join("fastcache_b200", "csrc")
-sources = sorted(glob.glob(os.path.join(SRC, "*.cu")) + glob.glob(os.path.join(SRC, "*.cpp")))
+# FC_EXT=core: `fastcache_b200._C_core`, the part that models without per-head K/V attention, compression or tensor
+# parallelism need (ops/loader.py takes it where the whole extension is not built)
+CORE = os.environ.get("FC_EXT") == "core"
+CORE_SOURCES = ("bindings.cpp", "elementwise.cu", "gemm.cu", "gemm_2cta.cu", "gemm_skinny.cu", "gemm_streamk.cu",
+                "hybrid_bind.cpp", "latent.cu", "latent_decode.cu", "latent_prefill.cu", "linear_simt.cu", "partials.cu",
+                "recurrence.cu", "recurrence_chunk.cu", "resid.cu")
+sources = [os.path.join(SRC, f) for f in CORE_SOURCES] if CORE else sorted(glob.glob(os.path.join(SRC, "*.cu")) + glob.glob(os.path.join(SRC, "*.cpp")))
 
 nvcc_flags = ["-O3", "-std=c++17", "-lineinfo", "-gencode", "arch=compute_100a,code=sm_100a",
               "--expt-relaxed-constexpr", "-Xptxas", "-v"] if os.environ.get("FC_PTXAS_V") else \
@@ -22,7 +28,7 @@ setup(
     version="0.1.0",
     packages=[],
     ext_modules=[CUDAExtension(
-        name="fastcache_b200._C",
+        name="fastcache_b200._C_core" if CORE else "fastcache_b200._C",
         sources=sources,
         include_dirs=[os.path.join(ROOT, SRC)],
         extra_compile_args={"cxx": ["-O3", "-std=c++17"], "nvcc": nvcc_flags},
