@@ -44,6 +44,9 @@ class TokenReplay:
                 else:
                     got = runner.run_prefill(seqs, logits_rows=rows)
                 logits = got.float().cpu()
+            if runner.main_stream is not None:
+                # also when nothing was read back: the next step writes the pinned buffers that this one copies from
+                runner.main_stream.synchronize()
             reset_context()
             for s in seqs:
                 s.num_computed_tokens, s.prefill_end = s.prefill_end, None

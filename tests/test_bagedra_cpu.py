@@ -200,3 +200,19 @@ def test_trace_run_command(tmp_path):
     got = [torch.from_numpy(np.fromfile(out / f"{i}.f32", dtype="<f4").reshape(-1, cfg["vocab"])) for i in range(3)]
     for rows, at in zip(got, ([0, 29], [4], [39])):
         assert bm.errors(rows, want[at])[0] < TOL
+
+
+@pytest.mark.parametrize("mode", ["lazy", "none"])
+def test_server_with_its_default_settings(mode, tmp_path):
+    from fastcache_b200.serving.server import FastCacheServer
+    cfg, w, path = _model(tmp_path, MIX)
+    server = FastCacheServer(path, compression_mode=mode, max_model_len=128, device="cpu", dtype="float32",
+                             kvcache_block_size=16, num_kvcache_blocks=32, max_num_seqs=3, tokenizer=False)
+    try:
+        prompts = [bm.tokens(n, cfg["vocab"], n) for n in (20, 5, 33, 9)]
+        futures = [server.submit(p, 6, 0.0) for p in prompts]
+        for p, f in zip(prompts, futures):
+            out = f.result(60)["token_ids"]
+            assert oracle.forward(cfg, w, p + out)[0][len(p) - 1:-1].argmax(-1).tolist() == out
+    finally:
+        server.shutdown()

@@ -163,6 +163,24 @@ def test_absorbed_attention_over_pages(H, rank, R, page, impl):
     assert ext().read_status(0) == 0
 
 
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_steps_that_read_nothing_back(dtype, tmp_path):
+    """Decode steps whose logits nobody asks for, one after another, then one that is asked for."""
+    from fastcache_b200.engine.replay import TokenReplay
+    cfg, w, path = _model("general", tmp_path)
+    llm = bm.engine(path, "cuda", dtype)
+    replay = TokenReplay(llm)
+    for k, n in enumerate((97, 23, 140, 64)):
+        toks = bm.tokens(n, cfg["vocab"], k)
+        name = f"r{k}"
+        replay.step([{"id": name, "tokens": toks[:4], "want": []}])
+        for t in toks[4:-1]:
+            replay.step([{"id": name, "tokens": [t], "want": []}])
+        got = replay.step([{"id": name, "tokens": toks[-1:], "want": [0]}], [name])
+        assert bm.errors(got, bm.oracle.forward(cfg, w, toks)[0][-1:])[0] < LIMIT[dtype], n
+    llm.exit()
+
+
 def test_long_context_decode_with_splits(tmp_path):
     cfg, w, path = _model("mid", tmp_path)
     n = 1500
