@@ -635,7 +635,7 @@ def run_layers(args):
     """Layer throughput of the hybrid model beside the dense decoder at equal size (no job, no serving loop)."""
     from benchmarks.hybrid_bench import run
     from fastcache_b200 import ops
-    sampler = ClockSampler()
+    sampler = ClockSampler(0)
     sampler.start()
     res = run(max(5, args.steps), args.small)
     clocks = sampler.stop()
