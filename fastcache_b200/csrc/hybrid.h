@@ -152,7 +152,10 @@ void launch_latent_attn_simt(const LatentAttn& p, bool f32, cudaStream_t s);
 bool latent_decode_supported(const LatentAttn& p);
 int latent_decode_splits(const LatentAttn& p, int max_ctx, int num_sms);
 void launch_latent_decode(const LatentAttn& p, cudaStream_t s);
-// partials (splits > 1) to the result
+// the same on tcgen05 (latent_decode_tc.cu); both leave partials for launch_latent_merge when splits > 1
+bool latent_decode_tc_supported(const LatentAttn& p);
+int latent_decode_tc_splits(const LatentAttn& p, int max_ctx, int num_sms);
+void launch_latent_decode_tc(const LatentAttn& p, cudaStream_t s);
 void launch_latent_merge(const LatentAttn& p, cudaStream_t s);
 
 void launch_gather_rows(const void* pool, const int* block_tables, const int* ctx, const int* cu_kv, void* out,

@@ -339,11 +339,13 @@ Tensor delta_rule(const Tensor& h, const Tensor& w, const Tensor& conv_w, const 
 
 // absorbed attention: the tensor-core form where it takes the sizes; `po` / `pl` keep its scratch alive
 void absorbed(fc::LatentAttn& at, bool f32, int64_t impl, int64_t max_ctx, const Tensor& like, Tensor& po, Tensor& pl) {
-  if (f32 || impl == 1 || !fc::latent_decode_supported(at)) {
+  const bool tc = !f32 && impl != 1 && impl != 3 && fc::latent_decode_tc_supported(at);
+  if (!tc && (f32 || impl == 1 || !fc::latent_decode_supported(at))) {
     fc::launch_latent_attn_simt(at, f32, stream_now());
     return;
   }
-  at.splits = fc::latent_decode_splits(at, int(max_ctx), fc::gemm_num_sms());
+  at.splits = tc ? fc::latent_decode_tc_splits(at, int(max_ctx), fc::gemm_num_sms())
+                 : fc::latent_decode_splits(at, int(max_ctx), fc::gemm_num_sms());
   if (at.splits > 1) {
     const auto opt = like.options().dtype(torch::kFloat32);
     po = torch::empty({(int64_t)at.T * at.H * at.splits * at.rank}, opt);
@@ -351,13 +353,15 @@ void absorbed(fc::LatentAttn& at, bool f32, int64_t impl, int64_t max_ctx, const
     at.part_o = po.data_ptr<float>();
     at.part_lse = pl.data_ptr<float>();
   }
-  fc::launch_latent_decode(at, stream_now());
+  if (tc) fc::launch_latent_decode_tc(at, stream_now());
+  else fc::launch_latent_decode(at, stream_now());
   if (at.splits > 1) fc::launch_latent_merge(at, stream_now());
 }
 
 // Projection, cache store and attention of a latent-attention layer (up to the output projection).
 // d: heads, dim, rot, vdim, rank, rot_dims, offsets of q, kv (-1: none), g.  impl: 0 choose, 1 the forms without tensor
-// cores, 2 absorbed also in prefill
+// cores, 2 absorbed also in prefill, 3 the same
+// on mma.sync
 Tensor latent_attention(const Tensor& h, const Tensor& w, const std::vector<int64_t>& d, double scale, double base,
                         const OptTensor& kv_norm, double eps, const Tensor& w_kv, int64_t off_uv, const Tensor& w_ukt,
                         const Tensor& w_uv, Tensor pool, const Tensor& positions, const OptTensor& slots,
@@ -642,6 +646,6 @@ void register_hybrid(pybind11::module_& m) {
   m.def("delta_rule", &delta_rule);
   m.def("latent_attention", &latent_attention);
   m.def("latent_decode_rows", &latent_decode_rows, py::arg("q"), py::arg("pool"), py::arg("block_tables"), py::arg("ctx"),
-        py::arg("rank"), py::arg("scale"), py::arg("impl") = 0);      // 0 choose, 1 CUDA cores
+        py::arg("rank"), py::arg("scale"), py::arg("impl") = 0);      // 0 choose, 1 CUDA cores, 3 mma.sync
   m.def("latent_prefill_rows", &latent_prefill_rows);
 }

@@ -1,0 +1,429 @@
+// Absorbed latent attention of decode-size batches on tcgen05 (the general tensor-core form is in latent_decode.cu).
+//
+// Grid (query row, group of 32 heads, split of the context).  A CTA walks its rows of the cache in tiles of 64.  The wide
+// operand of both products is the cache, not the few heads:
+//     S^T [64 rows x 32 heads]    = rows (latent | rotated part) * Q^T        A: row tile, K-major; B: Q, K-major
+//     O^T [128 latents x 32 heads] += rows^T * P^T, one block per 128 latents  A: the same tile, MN-major; B: P, K-major
+// (S^T is issued with 128 rows; the upper 64 read the shared memory behind the tile and their lanes are ignored.)  Shared
+// memory holds a tile as pairs of 64-column sub-tiles (128 latents each) in a ring of ten pairs, and the columns behind
+// them in a ring of two sub-tiles; a pair is refilled as soon as its block of O^T is done.
+//   warp 0     TMA, boxes that never straddle a page
+//   warp 1     tcgen05.mma issuer; the scores of the next tile go first, so that they overlap the softmax of this one
+//   warps 2-5  one cache row per thread: P = 2^(s - ref) for all heads against a reference per head (the first row's
+//              score; should a score outgrow it by 2^64, all accumulators move to the new maximum), P to shared memory
+//              as bf16, sums per thread; at the end one latent per thread
+#include <algorithm>
+#include <stdexcept>
+#include <string>
+
+#include "gemm.h"
+#include "hybrid.cuh"
+#include "launch.h"
+
+namespace fc {
+
+using bf16 = __nv_bfloat16;
+constexpr int LT_ROWS = 64, LT_HEADS = 32, LT_PAIRS = 10, LT_THREADS = 192;
+constexpr int LT_SUB = LT_ROWS * 128;             // bytes of a [64 rows x 64 columns] sub-tile
+constexpr int LT_QSUB = LT_HEADS * 128;           // of a [32 heads x 64 columns] sub-tile
+constexpr int LT_TMEM = 256;                      // S^T of even / odd tiles [0, 32) [32, 64), O^T blocks [64 + 32 b, ...)
+constexpr float LT_RANGE = 64.f;                  // log2 units above the reference that P may reach
+constexpr int LT_MAX_SUBS = 9;
+
+__device__ __forceinline__ uint64_t lt_sdesc(uint32_t addr, uint32_t lbo_bytes, uint32_t sbo_bytes) {
+  uint64_t d = 0;
+  d |= uint64_t((addr & 0x3FFFF) >> 4);
+  d |= uint64_t((lbo_bytes >> 4) & 0x3FFF) << 16;
+  d |= uint64_t((sbo_bytes >> 4) & 0x3FFF) << 32;
+  d |= uint64_t(1) << 46;
+  d |= uint64_t(2) << 61;
+  return d;
+}
+
+__global__ void __launch_bounds__(LT_THREADS, 1)
+latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm, const LatentAttn p, int box_rows, int pairs, int extra,
+                        float scale_log2) {
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+  uint8_t* s_kv = smem;                                            // [LT_PAIRS] pairs of sub-tiles
+  uint8_t* s_x = s_kv + LT_PAIRS * 2 * LT_SUB;                     // the columns behind the pairs
+  uint8_t* s_q = s_x + 2 * LT_SUB;                                 // [LT_MAX_SUBS] sub-tiles
+  uint8_t* s_p = s_q + LT_MAX_SUBS * LT_QSUB;
+  float* s_ref = reinterpret_cast<float*>(s_p + 2 * LT_QSUB);      // (P of even / odd tiles)  [32] reference
+  float* s_red = s_ref + LT_HEADS;                                 // [4][32]
+  uint64_t* bars = reinterpret_cast<uint64_t*>(s_red + 4 * LT_HEADS);
+  uint64_t *full = bars, *empty = bars + LT_PAIRS, *x_full = bars + 2 * LT_PAIRS, *x_empty = x_full + 2;
+  uint64_t *s_full = x_full + 4, *p_ready = x_full + 6, *o_done = x_full + 7;      // o_done: O^T complete up to a tile
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(x_full + 8);
+  volatile int* s_abort = reinterpret_cast<volatile int*>(tmem_slot + 1);
+  int* s_at = reinterpret_cast<int*>(tmem_slot + 2);               // [LT_ROWS / 8]
+
+  const int t = blockIdx.x, h0 = blockIdx.y * LT_HEADS, split = blockIdx.z;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  pdl_launch_dependents();
+  if (tid == 0) {
+    for (int i = 0; i < LT_PAIRS; ++i) {
+      mbar_init(&full[i], 1);
+      mbar_init(&empty[i], 1);
+    }
+    for (int i = 0; i < 2; ++i) {
+      mbar_init(&x_full[i], 1);
+      mbar_init(&x_empty[i], 1);
+      mbar_init(&s_full[i], 1);
+    }
+    mbar_init(p_ready, 128);
+    mbar_init(o_done, 1);
+    *s_abort = 0;
+    fence_barrier_init();
+    tma_prefetch_desc(&tm);
+  }
+  if (warp == 1) {
+    tmem_alloc(tmem_slot, LT_TMEM);
+    tmem_relinquish();
+  }
+  pdl_wait();
+  asm volatile("fence.proxy.async.global;" ::: "memory");          // rows were written with ordinary stores
+  const int ctx = min(p.row_ctx[t], p.max_blocks * p.block_size);
+  const int b = p.row_seq != nullptr ? p.row_seq[t] : t;
+  const int tiles = (ctx + LT_ROWS - 1) / LT_ROWS;
+  const int per = (tiles + p.splits - 1) / p.splits;
+  const int tile0 = split * per, n_tiles = max(0, min(tiles, tile0 + per) - tile0);
+  const int* bt = p.block_tables + (long long)b * p.max_blocks;
+  const int w = p.rank + p.R, subs = pairs * 2 + extra;
+
+  {                                                                // Q, zero-padded to whole sub-tiles and head rows
+    const uint4* q = reinterpret_cast<const uint4*>(reinterpret_cast<const bf16*>(p.q_abs) + ((long long)t * p.H + h0) * w);
+    uint4 v[6];
+    for (int ch = lane; ch < subs * 8; ch += 32) {
+#pragma unroll
+      for (int i = 0; i < 6; ++i) {
+        const int r = warp + i * (LT_THREADS / 32);
+        v[i] = r < LT_HEADS && h0 + r < p.H && ch * 8 < w ? __ldcg(q + (long long)r * (w / 8) + ch) : make_uint4(0, 0, 0, 0);
+      }
+#pragma unroll
+      for (int i = 0; i < 6; ++i) {
+        const int r = warp + i * (LT_THREADS / 32);
+        if (r < LT_HEADS)
+          *reinterpret_cast<uint4*>(s_q + (ch >> 3) * LT_QSUB + r * 128 + (((ch & 7) ^ (r & 7)) << 4)) = v[i];
+      }
+    }
+  }
+  if (n_tiles <= LT_PAIRS)                                         // boxes past the context are never loaded: keep it finite
+    for (int i = tid; i < (LT_PAIRS * 2 + 2) * LT_SUB / 16; i += LT_THREADS)
+      reinterpret_cast<uint4*>(s_kv)[i] = make_uint4(0, 0, 0, 0);
+  fence_proxy_async();
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem = *tmem_slot;
+
+  if (warp == 0) {
+    // ------------------------------------------------------------------ TMA loader
+    if (lane == 0) {
+      int slot = 0;
+      uint32_t phase = 1;
+      constexpr int MAX_PIECES = LT_ROWS / 8;
+      int next[MAX_PIECES];                                        // pool row of every piece of a tile, one tile ahead
+      auto find = [&](int j) {
+        const int row0 = (tile0 + j) * LT_ROWS;
+#pragma unroll
+        for (int pc = 0; pc < MAX_PIECES; ++pc) {
+          const int tok = row0 + pc * box_rows;
+          if (j >= n_tiles || pc * box_rows >= LT_ROWS || tok >= ctx) continue;
+          int blk = bt[tok / p.block_size];
+          if (blk < 0 || blk >= p.num_blocks) {
+            report(p.status, ST_BAD_INDEX);
+            blk = 0;
+          }
+          next[pc] = blk * p.block_size + tok % p.block_size;
+        }
+      };
+      find(0);
+      for (int j = 0; j < n_tiles && !*s_abort; ++j) {
+        const int pieces = min(LT_ROWS / box_rows, (ctx - (tile0 + j) * LT_ROWS + box_rows - 1) / box_rows);
+        const uint32_t bytes = uint32_t(pieces) * box_rows * 128;
+        // through shared memory: the issue loop stays one instruction sequence for any number of pieces
+#pragma unroll
+        for (int pc = 0; pc < MAX_PIECES; ++pc) s_at[pc] = next[pc];
+        find(j + 1);
+        auto load = [&](uint8_t* dst, uint64_t* bar, int col) {
+#pragma unroll 1
+          for (int pc = 0; pc < pieces; ++pc)
+            tma_load_2d(dst + pc * box_rows * 128, &tm, bar, col, reinterpret_cast<volatile int*>(s_at)[pc]);
+        };
+        for (int i = 0; i < pairs; ++i) {
+          if (!mbar_wait(&empty[slot], phase, p.status, ST_TIMEOUT_EMPTY)) {
+            *s_abort = 1;
+            break;
+          }
+          mbar_expect_tx(&full[slot], 2 * bytes);
+          load(s_kv + slot * 2 * LT_SUB, &full[slot], i * 128);
+          load(s_kv + slot * 2 * LT_SUB + LT_SUB, &full[slot], i * 128 + 64);
+          if (++slot == LT_PAIRS) {
+            slot = 0;
+            phase ^= 1;
+          }
+        }
+        if (extra && !*s_abort) {
+          const int x = j & 1;
+          if (!mbar_wait(&x_empty[x], (uint32_t(j >> 1) & 1u) ^ 1u, p.status, ST_TIMEOUT_EMPTY)) {
+            *s_abort = 1;
+            break;
+          }
+          mbar_expect_tx(&x_full[x], bytes);
+          load(s_x + x * LT_SUB, &x_full[x], pairs * 128);
+        }
+      }
+    }
+  } else if (warp == 1) {
+    // ------------------------------------------------------------------ MMA issuer
+    if (lane == 0) {
+      constexpr uint32_t idesc_s = make_idesc_bf16(128, LT_HEADS, false, false);
+      constexpr uint32_t idesc_o = make_idesc_bf16(128, LT_HEADS, true, false);      // A (rows^T) is MN-major
+      const int ksteps = (p.row_width + 15) / 16;
+      const uint32_t qa = smem_u32(s_q), pa = smem_u32(s_p);
+      int slot = 0, sl = 0;                                        // next pair of O^T and of S^T
+      uint32_t ph = 0;
+      auto scores = [&](uint32_t tm_s, uint32_t base, int sub) {
+        for (int kk = 0; kk < 4; ++kk) {
+          if (sub * 4 + kk >= ksteps) break;
+          tc_mma_f16(tm_s, lt_sdesc(base + uint32_t(kk) * 32, 16, 1024),
+                     lt_sdesc(qa + uint32_t(sub) * LT_QSUB + uint32_t(kk) * 32, 16, 1024), idesc_s,
+                     (sub > 0 || kk > 0) ? 1u : 0u);
+        }
+      };
+      auto issue_s = [&](int j) {
+        const int x = j & 1;
+        for (int i = 0; i < pairs; ++i) {
+          if (!mbar_wait(&full[sl], ph, p.status, ST_TIMEOUT_FULL)) return false;
+          tc_fence_after();
+          const uint32_t base = smem_u32(s_kv + sl * 2 * LT_SUB);
+          scores(tmem + LT_HEADS * uint32_t(x), base, i * 2);
+          scores(tmem + LT_HEADS * uint32_t(x), base + LT_SUB, i * 2 + 1);
+          if (++sl == LT_PAIRS) {
+            sl = 0;
+            ph ^= 1;
+          }
+        }
+        if (extra) {
+          if (!mbar_wait(&x_full[x], uint32_t(j >> 1) & 1u, p.status, ST_TIMEOUT_FULL)) return false;
+          tc_fence_after();
+          scores(tmem + LT_HEADS * uint32_t(x), smem_u32(s_x + x * LT_SUB), pairs * 2);
+        }
+        tc_commit(&s_full[x]);
+        if (extra) tc_commit(&x_empty[x]);
+        return true;
+      };
+      bool ok = n_tiles == 0 || issue_s(0);
+      for (int j = 0; j < n_tiles && ok; ++j) {
+        if (j + 1 < n_tiles) ok = issue_s(j + 1);
+        ok = ok && mbar_wait(p_ready, uint32_t(j) & 1u, p.status, ST_TIMEOUT_FULL);
+        if (!ok) break;
+        tc_fence_after();
+        for (int i = 0; i < pairs; ++i) {
+          const uint32_t va = smem_u32(s_kv + slot * 2 * LT_SUB);
+#pragma unroll
+          for (int kk = 0; kk < LT_ROWS / 16; ++kk)
+            tc_mma_f16(tmem + LT_HEADS * uint32_t(2 + i), lt_sdesc(va + uint32_t(kk) * 2048, LT_SUB, 1024),
+                       lt_sdesc(pa + uint32_t(j & 1) * LT_QSUB + uint32_t(kk) * 32, 16, 1024), idesc_o,
+                       (j > 0 || kk > 0) ? 1u : 0u);
+          tc_commit(&empty[slot]);
+          if (++slot == LT_PAIRS) slot = 0;
+        }
+        tc_commit(o_done);
+      }
+      if (!ok) *s_abort = 1;
+    }
+  } else {
+    // ------------------------------------------------------------------ softmax, then epilogue
+    const int group = warp & 3;                                    // TMEM lanes this warp may touch
+    const int row = group * 32 + lane;
+    const uint32_t lanes = uint32_t(group * 32) << 16;
+    auto sync_or = [](bool x) {                                    // over the four warps
+      uint32_t r;
+      asm volatile(
+          "{\n\t.reg .pred p, q;\n\tsetp.ne.u32 p, %1, 0;\n\tbar.red.or.pred q, 1, 128, p;\n\tselp.u32 %0, 1, 0, q;\n\t}"
+          : "=r"(r)
+          : "r"(x ? 1u : 0u)
+          : "memory");
+      return r != 0;
+    };
+    float l[LT_HEADS];
+#pragma unroll
+    for (int h = 0; h < LT_HEADS; ++h) l[h] = 0.f;
+    uint8_t* prow = s_p + (row & 7) * 2;
+    const int chunk = (row & 63) >> 3;
+    const bool mine = row < LT_ROWS;                               // warp-uniform: the upper lanes hold no cache row
+    bool ok = true;
+    for (int j = 0; j < n_tiles; ++j) {
+      if (ok) ok = !*s_abort && mbar_wait(&s_full[j & 1], uint32_t(j >> 1) & 1u, p.status, ST_TIMEOUT_ACC_FULL);
+      if (sync_or(!ok)) {                                          // all four warps leave together
+        ok = false;
+        break;
+      }
+      tc_fence_after();
+      uint32_t s[LT_HEADS];
+      tmem_ld_32x32(tmem + lanes + LT_HEADS * uint32_t(j & 1), s);
+      tmem_ld_wait();
+      const bool valid = mine && (tile0 + j) * LT_ROWS + row < ctx;
+      if (j == 0) {
+        if (row == 0)
+#pragma unroll
+          for (int h = 0; h < LT_HEADS; ++h) s_ref[h] = __uint_as_float(s[h]) * scale_log2;
+        sync_or(false);
+      }
+      float v[LT_HEADS], top = -INFINITY;
+#pragma unroll
+      for (int h = 0; h < LT_HEADS; h += 4) {
+        const float4 r = *reinterpret_cast<const float4*>(s_ref + h);
+        const float rr[4] = {r.x, r.y, r.z, r.w};
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          v[h + e] = fmaf(__uint_as_float(s[h + e]), scale_log2, -rr[e]);      // relative to the reference
+          top = fmaxf(top, v[h + e]);
+        }
+      }
+      const bool far = top > LT_RANGE;
+      if (sync_or(far && valid)) {
+        // a score outgrew its reference: maximum over the tile, then sums and O^T (complete up to the tile before) move
+        // to the new reference
+#pragma unroll
+        for (int h = 0; h < LT_HEADS; ++h) {
+          const float m = warp_max(valid ? v[h] + s_ref[h] : -INFINITY);
+          if (lane == h) s_red[group * LT_HEADS + h] = m;
+        }
+        sync_or(false);
+        float f[LT_HEADS];
+#pragma unroll
+        for (int h = 0; h < LT_HEADS; ++h) {
+          const float m = fmaxf(fmaxf(s_red[h], s_red[LT_HEADS + h]), fmaxf(s_red[2 * LT_HEADS + h], s_red[3 * LT_HEADS + h]));
+          f[h] = exp2f(fminf(s_ref[h] - m, 0.f));
+          l[h] *= f[h];
+          v[h] += fminf(s_ref[h] - m, 0.f);
+        }
+        if (j > 0 && ok) ok = mbar_wait(o_done, uint32_t(j - 1) & 1u, p.status, ST_TIMEOUT_ACC_FULL);
+        tc_fence_after();
+        if (j > 0)
+          for (int i = 0; i < pairs; ++i) {
+            uint32_t r[32];
+            tmem_ld_32x32(tmem + lanes + LT_HEADS * uint32_t(2 + i), r);
+            tmem_ld_wait();
+#pragma unroll
+            for (int h = 0; h < LT_HEADS; ++h) r[h] = __float_as_uint(__uint_as_float(r[h]) * f[h]);
+            tmem_st_32x32(tmem + lanes + LT_HEADS * uint32_t(2 + i), r);
+            tmem_st_wait();
+          }
+        sync_or(false);
+        if (row < LT_HEADS) {
+          const int h = row;
+          s_ref[h] = fmaxf(s_ref[h], fmaxf(fmaxf(s_red[h], s_red[LT_HEADS + h]),
+                                           fmaxf(s_red[2 * LT_HEADS + h], s_red[3 * LT_HEADS + h])));
+        }
+        sync_or(false);
+      }
+      if (mine) {
+#pragma unroll
+        for (int h = 0; h < LT_HEADS; ++h) {
+          float e;
+          asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(valid ? v[h] : -INFINITY));
+          l[h] += e;
+          *reinterpret_cast<bf16*>(prow + (j & 1) * LT_QSUB + h * 128 + ((chunk ^ (h & 7)) << 4)) = __float2bfloat16(e);
+        }
+      }
+      fence_proxy_async();
+      tc_fence_before();
+      mbar_arrive(p_ready);
+    }
+    // the last two phases one by one: the scores of the last tile only say that the third-last product is done, and a
+    // parity cannot tell a phase from the one two before it
+    if (ok && n_tiles > 1) ok = mbar_wait(o_done, uint32_t(n_tiles - 2) & 1u, p.status, ST_TIMEOUT_ACC_FULL);
+    if (ok && n_tiles > 0) ok = mbar_wait(o_done, uint32_t(n_tiles - 1) & 1u, p.status, ST_TIMEOUT_ACC_FULL);
+    if (!ok) *s_abort = 1;
+    tc_fence_after();
+    // every product is done: the ring is free.  Sums over the rows, then O^T block by block through shared memory
+    const bool good = !sync_or(!ok) && n_tiles > 0;
+    float* s_l = reinterpret_cast<float*>(s_kv);                   // [LT_ROWS][33]
+    float* s_o = s_l + LT_ROWS * 33;                               // [32 heads][128 latents + 4]
+    const int et = tid - 64;                                       // 0..127
+    if (mine)
+#pragma unroll
+      for (int h = 0; h < LT_HEADS; ++h) s_l[row * 33 + h] = l[h];
+    sync_or(false);
+    {
+      float x = 0.f;
+      for (int r = et >> 5; r < LT_ROWS; r += 4) x += s_l[r * 33 + (et & 31)];
+      s_red[et] = x;
+    }
+    sync_or(false);
+    if (et < LT_HEADS) {
+      const float x = s_red[et] + s_red[LT_HEADS + et] + s_red[2 * LT_HEADS + et] + s_red[3 * LT_HEADS + et];
+      const bool has = good && x > 0.f;
+      if (p.splits > 1 && h0 + et < p.H)
+        p.part_lse[((long long)t * p.H + h0 + et) * p.splits + split] = has ? s_ref[et] + log2f(x) : -INFINITY;
+      s_red[et] = has ? 1.f / x : 0.f;
+    }
+    for (int i = 0; i < pairs; ++i) {
+      sync_or(false);                                              // s_red is there, the block before is written
+      if (good) {
+        uint32_t r[32];
+        tmem_ld_32x32(tmem + lanes + LT_HEADS * uint32_t(2 + i), r);
+        tmem_ld_wait();
+#pragma unroll
+        for (int h = 0; h < LT_HEADS; ++h) s_o[h * 132 + row] = __uint_as_float(r[h]);
+      }
+      sync_or(false);
+      const int c = i * 128 + (et & 31) * 4;                       // a warp writes 128 latents of a head
+      if (c < p.rank)
+        for (int h = et >> 5; h < LT_HEADS && h0 + h < p.H; h += 4) {
+          const float inv = s_red[h];
+          float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+          if (inv != 0.f) x = *reinterpret_cast<const float4*>(s_o + h * 132 + (et & 31) * 4);
+          const long long at = (long long)t * p.H + h0 + h;
+          if (p.splits == 1)
+            store4(reinterpret_cast<bf16*>(p.o_lat) + at * p.rank + c, x.x * inv, x.y * inv, x.z * inv, x.w * inv);
+          else
+            store4(p.part_o + (at * p.splits + split) * p.rank + c, x.x * inv, x.y * inv, x.z * inv, x.w * inv);
+        }
+    }
+  }
+  tc_fence_before();
+  __syncthreads();
+  if (warp == 1) {
+    tc_fence_after();
+    tmem_dealloc(tmem, LT_TMEM);
+  }
+}
+
+static int lt_box_rows(int block_size) {
+  int box = LT_ROWS;
+  while (box > block_size || block_size % box != 0) box >>= 1;
+  return box;
+}
+
+bool latent_decode_tc_supported(const LatentAttn& p) {
+  const int pairs = (p.rank + 127) / 128;
+  return p.rank % 8 == 0 && (p.rank + p.R) % 8 == 0 && pairs <= 4 && p.row_width - pairs * 128 <= 64 &&
+         lt_box_rows(p.block_size) >= 8;
+}
+
+int latent_decode_tc_splits(const LatentAttn& p, int max_ctx, int num_sms) {
+  const int ctas = p.T * ((p.H + LT_HEADS - 1) / LT_HEADS);
+  if (ctas * 3 > num_sms * 2) return 1;                            // nearly a full wave already
+  return std::max(1, std::min({num_sms / std::max(1, ctas), max_ctx / (2 * LT_ROWS), 32}));
+}
+
+void launch_latent_decode_tc(const LatentAttn& p, cudaStream_t s) {
+  if (p.T == 0) return;
+  const int box = lt_box_rows(p.block_size), pairs = (p.rank + 127) / 128, extra = p.row_width > pairs * 128 ? 1 : 0;
+  const CUtensorMap tm = make_tmap_bf16_2d(p.pool, (uint64_t)p.num_blocks * p.block_size, p.row_width, p.row_width, box, 64);
+  constexpr int smem = (LT_PAIRS * 2 + 2) * LT_SUB + (LT_MAX_SUBS + 2) * LT_QSUB + 5 * LT_HEADS * 4 +
+                       (2 * LT_PAIRS + 8) * 8 + 16 + LT_ROWS / 2 + 1024;
+  static_assert(smem <= 227 * 1024, "shared memory of a CTA");
+  cudaFuncSetAttribute(latent_decode_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+  launch_pdl(PDL_DECODE_ATTN, latent_decode_tc_kernel, dim3(p.T, (p.H + LT_HEADS - 1) / LT_HEADS, p.splits),
+             dim3(LT_THREADS), smem, s, tm, p, box, pairs, extra, p.scale * 1.4426950408889634f);
+  const cudaError_t e = cudaGetLastError();
+  if (e != cudaSuccess) throw std::runtime_error(std::string("latent decode (tcgen05): ") + cudaGetErrorString(e));
+}
+
+}  // namespace fc

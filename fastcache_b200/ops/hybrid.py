@@ -15,7 +15,8 @@ from . import reference_hybrid as ref
 from .loader import ext
 
 
-LATENT_IMPL = 0         # tests: 1 the general kernels also where a tensor-core form exists, 2 absorbed also in prefill
+LATENT_IMPL = 0         # tests: 1 the general kernels also where a tensor-core form exists, 2 absorbed also in prefill,
+                        # 3 the same on mma.sync
 
 
 def _n(k: int = 1) -> None:

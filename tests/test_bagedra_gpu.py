@@ -120,10 +120,11 @@ def test_pages_and_slots_with_old_contents(dtype, tmp_path):
     llm.exit()
 
 
-@pytest.mark.parametrize("impl", [1, 2])
+@pytest.mark.parametrize("impl", [1, 2, 3])
 @pytest.mark.parametrize("name", ["wide", "heads"])
 def test_other_forms_of_latent_attention_agree(name, impl, tmp_path, monkeypatch):
-    """Forms that are not the first choice: 1 without tensor cores, 2 absorbed attention also in prefill."""
+    """Forms that are not the first choice: 1 without tensor cores, 2 absorbed attention also in prefill,
+    3 the same on mma.sync."""
     from fastcache_b200.ops import hybrid
     monkeypatch.setattr(hybrid, "LATENT_IMPL", impl)
     cfg, w, path = _model(name, tmp_path)
@@ -143,7 +144,7 @@ def _absorbed(q, pool, bt, ctx, rank, scale):
     return torch.stack([o.double() for o in out])
 
 
-@pytest.mark.parametrize("impl", [0, 1])
+@pytest.mark.parametrize("impl", [0, 1, 3])
 @pytest.mark.parametrize("H,rank,R,page", [(32, 512, 64, 64), (5, 128, 32, 16), (70, 256, 64, 256), (33, 64, 32, 8),
                                            (16, 320, 64, 32), (1, 16, 8, 128)])
 def test_absorbed_attention_over_pages(H, rank, R, page, impl):
