@@ -40,6 +40,24 @@ __device__ __forceinline__ uint64_t lt_sdesc(uint32_t addr, uint32_t lbo_bytes, 
   return d;
 }
 
+// issue by one lane of a warp that is converged otherwise: loops and descriptors stay warp-uniform
+__device__ __forceinline__ void lt_mma(uint32_t tmem_d, uint64_t a, uint64_t b, uint32_t idesc, uint32_t accumulate,
+                                       uint32_t issue) {
+  asm volatile(
+      "{\n\t.reg .pred p, q;\n\t"
+      "setp.ne.b32 p, %4, 0;\n\tsetp.ne.b32 q, %5, 0;\n\t"
+      "@q tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t}"
+      ::"r"(tmem_d), "l"(a), "l"(b), "r"(idesc), "r"(accumulate), "r"(issue)
+      : "memory");
+}
+__device__ __forceinline__ void lt_commit(uint64_t* bar, uint32_t issue) {
+  asm volatile(
+      "{\n\t.reg .pred q;\n\tsetp.ne.b32 q, %1, 0;\n\t"
+      "@q tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];\n\t}"
+      ::"r"(smem_u32(bar)), "r"(issue)
+      : "memory");
+}
+
 __global__ void __launch_bounds__(LT_THREADS, 1)
 latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm, const LatentAttn p, int box_rows, int pairs, int extra,
                         float scale_log2) {
@@ -177,62 +195,68 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm, const LatentAttn
     }
   } else if (warp == 1) {
     // ------------------------------------------------------------------ MMA issuer
-    if (lane == 0) {
+    const uint32_t el = elect_one() ? 1u : 0u;
+    {
       constexpr uint32_t idesc_s = make_idesc_bf16(128, LT_HEADS, false, false);
       constexpr uint32_t idesc_o = make_idesc_bf16(128, LT_HEADS, true, false);      // A (rows^T) is MN-major
       const int ksteps = (p.row_width + 15) / 16;
-      const uint32_t qa = smem_u32(s_q), pa = smem_u32(s_p);
+      auto wait = [](uint64_t* bar, uint32_t parity, uint32_t* status, uint32_t code) {
+        return __all_sync(0xffffffffu, mbar_wait(bar, parity, status, code)) != 0;
+      };
       int slot = 0, sl = 0;                                        // next pair of O^T and of S^T
       uint32_t ph = 0;
-      auto scores = [&](uint32_t tm_s, uint32_t base, int sub) {
-        for (int kk = 0; kk < 4; ++kk) {
-          if (sub * 4 + kk >= ksteps) break;
-          tc_mma_f16(tm_s, lt_sdesc(base + uint32_t(kk) * 32, 16, 1024),
-                     lt_sdesc(qa + uint32_t(sub) * LT_QSUB + uint32_t(kk) * 32, 16, 1024), idesc_s,
-                     (sub > 0 || kk > 0) ? 1u : 0u);
-        }
+      // descriptors by addition on their address field (16-byte units)
+      const uint64_t d_rows = lt_sdesc(smem_u32(s_kv), 16, 1024), d_x = lt_sdesc(smem_u32(s_x), 16, 1024);
+      const uint64_t d_cols = lt_sdesc(smem_u32(s_kv), LT_SUB, 1024);
+      const uint64_t d_q = lt_sdesc(smem_u32(s_q), 16, 1024), d_p = lt_sdesc(smem_u32(s_p), 16, 1024);
+      auto scores = [&](uint32_t tm_s, uint64_t da, int sub) {
+        const uint64_t dq = d_q + uint64_t(sub * (LT_QSUB >> 4));
+        const int left = ksteps - sub * 4;
+#pragma unroll
+        for (int kk = 0; kk < 4; ++kk)
+          if (kk < left)
+            lt_mma(tm_s, da + uint64_t(kk * 2), dq + uint64_t(kk * 2), idesc_s, (sub > 0 || kk > 0) ? 1u : 0u, el);
       };
       auto issue_s = [&](int j) {
         const int x = j & 1;
         for (int i = 0; i < pairs; ++i) {
-          if (!mbar_wait(&full[sl], ph, p.status, ST_TIMEOUT_FULL)) return false;
+          if (!wait(&full[sl], ph, p.status, ST_TIMEOUT_FULL)) return false;
           tc_fence_after();
-          const uint32_t base = smem_u32(s_kv + sl * 2 * LT_SUB);
-          scores(tmem + LT_HEADS * uint32_t(x), base, i * 2);
-          scores(tmem + LT_HEADS * uint32_t(x), base + LT_SUB, i * 2 + 1);
+          const uint64_t da = d_rows + uint64_t(sl * (2 * LT_SUB >> 4));
+          scores(tmem + LT_HEADS * uint32_t(x), da, i * 2);
+          scores(tmem + LT_HEADS * uint32_t(x), da + uint64_t(LT_SUB >> 4), i * 2 + 1);
           if (++sl == LT_PAIRS) {
             sl = 0;
             ph ^= 1;
           }
         }
         if (extra) {
-          if (!mbar_wait(&x_full[x], uint32_t(j >> 1) & 1u, p.status, ST_TIMEOUT_FULL)) return false;
+          if (!wait(&x_full[x], uint32_t(j >> 1) & 1u, p.status, ST_TIMEOUT_FULL)) return false;
           tc_fence_after();
-          scores(tmem + LT_HEADS * uint32_t(x), smem_u32(s_x + x * LT_SUB), pairs * 2);
+          scores(tmem + LT_HEADS * uint32_t(x), d_x + uint64_t(x * (LT_SUB >> 4)), pairs * 2);
         }
-        tc_commit(&s_full[x]);
-        if (extra) tc_commit(&x_empty[x]);
+        lt_commit(&s_full[x], el);
+        if (extra) lt_commit(&x_empty[x], el);
         return true;
       };
       bool ok = n_tiles == 0 || issue_s(0);
       for (int j = 0; j < n_tiles && ok; ++j) {
         if (j + 1 < n_tiles) ok = issue_s(j + 1);
-        ok = ok && mbar_wait(p_ready, uint32_t(j) & 1u, p.status, ST_TIMEOUT_FULL);
+        ok = ok && wait(p_ready, uint32_t(j) & 1u, p.status, ST_TIMEOUT_FULL);
         if (!ok) break;
         tc_fence_after();
         for (int i = 0; i < pairs; ++i) {
-          const uint32_t va = smem_u32(s_kv + slot * 2 * LT_SUB);
+          const uint64_t dv = d_cols + uint64_t(slot * (2 * LT_SUB >> 4)), dp = d_p + uint64_t((j & 1) * (LT_QSUB >> 4));
+          const uint32_t tm_o = tmem + LT_HEADS * uint32_t(2 + i);
 #pragma unroll
           for (int kk = 0; kk < LT_ROWS / 16; ++kk)
-            tc_mma_f16(tmem + LT_HEADS * uint32_t(2 + i), lt_sdesc(va + uint32_t(kk) * 2048, LT_SUB, 1024),
-                       lt_sdesc(pa + uint32_t(j & 1) * LT_QSUB + uint32_t(kk) * 32, 16, 1024), idesc_o,
-                       (j > 0 || kk > 0) ? 1u : 0u);
-          tc_commit(&empty[slot]);
+            lt_mma(tm_o, dv + uint64_t(kk * 128), dp + uint64_t(kk * 2), idesc_o, (j > 0 || kk > 0) ? 1u : 0u, el);
+          lt_commit(&empty[slot], el);
           if (++slot == LT_PAIRS) slot = 0;
         }
-        tc_commit(o_done);
+        lt_commit(o_done, el);
       }
-      if (!ok) *s_abort = 1;
+      if (!ok && lane == 0) *s_abort = 1;
     }
   } else {
     // ------------------------------------------------------------------ softmax, then epilogue
