@@ -58,6 +58,21 @@ __device__ __forceinline__ void lt_commit(uint64_t* bar, uint32_t issue) {
       : "memory");
 }
 
+__device__ __forceinline__ void lt_expect(uint64_t* bar, uint32_t bytes, uint32_t issue) {
+  asm volatile(
+      "{\n\t.reg .pred q;\n\tsetp.ne.b32 q, %2, 0;\n\t"
+      "@q mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;\n\t}"
+      ::"r"(smem_u32(bar)), "r"(bytes), "r"(issue)
+      : "memory");
+}
+__device__ __forceinline__ void lt_load(void* dst, const CUtensorMap* m, uint64_t* bar, int x, int y, uint32_t issue) {
+  asm volatile(
+      "{\n\t.reg .pred q;\n\tsetp.ne.b32 q, %5, 0;\n\t"
+      "@q cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4}], [%2];\n\t}"
+      ::"r"(smem_u32(dst)), "l"(reinterpret_cast<uint64_t>(m)), "r"(smem_u32(bar)), "r"(x), "r"(y), "r"(issue)
+      : "memory");
+}
+
 __global__ void __launch_bounds__(LT_THREADS, 1)
 latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm, const LatentAttn p, int box_rows, int pairs, int extra,
                         float scale_log2) {
@@ -137,8 +152,10 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm, const LatentAttn
 
   if (warp == 0) {
     // ------------------------------------------------------------------ TMA loader
-    if (lane == 0) {
+    const uint32_t el = elect_one() ? 1u : 0u;
+    {
       int slot = 0;
+      bool ok = true;
       uint32_t phase = 1;
       constexpr int MAX_PIECES = LT_ROWS / 8;
       int next[MAX_PIECES];                                        // pool row of every piece of a tile, one tile ahead
@@ -150,31 +167,35 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm, const LatentAttn
           if (j >= n_tiles || pc * box_rows >= LT_ROWS || tok >= ctx) continue;
           int blk = bt[tok / p.block_size];
           if (blk < 0 || blk >= p.num_blocks) {
-            report(p.status, ST_BAD_INDEX);
+            if (lane == 0) report(p.status, ST_BAD_INDEX);
             blk = 0;
           }
           next[pc] = blk * p.block_size + tok % p.block_size;
         }
       };
       find(0);
-      for (int j = 0; j < n_tiles && !*s_abort; ++j) {
+      for (int j = 0; j < n_tiles && ok; ++j) {
         const int pieces = min(LT_ROWS / box_rows, (ctx - (tile0 + j) * LT_ROWS + box_rows - 1) / box_rows);
         const uint32_t bytes = uint32_t(pieces) * box_rows * 128;
         // through shared memory: the issue loop stays one instruction sequence for any number of pieces
+        ok = !__any_sync(0xffffffffu, *s_abort != 0);                // also: every lane is done with the tile before
 #pragma unroll
-        for (int pc = 0; pc < MAX_PIECES; ++pc) s_at[pc] = next[pc];
+        for (int pc = 0; pc < MAX_PIECES; ++pc)
+          if (lane == 0) s_at[pc] = next[pc];
+        __syncwarp();
         find(j + 1);
         auto load = [&](uint8_t* dst, uint64_t* bar, int col) {
 #pragma unroll 1
           for (int pc = 0; pc < pieces; ++pc)
-            tma_load_2d(dst + pc * box_rows * 128, &tm, bar, col, reinterpret_cast<volatile int*>(s_at)[pc]);
+            lt_load(dst + pc * box_rows * 128, &tm, bar, col, reinterpret_cast<volatile int*>(s_at)[pc], el);
         };
         for (int i = 0; i < pairs; ++i) {
-          if (!mbar_wait(&empty[slot], phase, p.status, ST_TIMEOUT_EMPTY)) {
-            *s_abort = 1;
+          if (!__all_sync(0xffffffffu, mbar_wait(&empty[slot], phase, p.status, ST_TIMEOUT_EMPTY))) {
+            if (lane == 0) *s_abort = 1;
+            ok = false;
             break;
           }
-          mbar_expect_tx(&full[slot], 2 * bytes);
+          lt_expect(&full[slot], 2 * bytes, el);
           load(s_kv + slot * 2 * LT_SUB, &full[slot], i * 128);
           load(s_kv + slot * 2 * LT_SUB + LT_SUB, &full[slot], i * 128 + 64);
           if (++slot == LT_PAIRS) {
@@ -182,13 +203,14 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm, const LatentAttn
             phase ^= 1;
           }
         }
-        if (extra && !*s_abort) {
+        if (extra && ok) {
           const int x = j & 1;
-          if (!mbar_wait(&x_empty[x], (uint32_t(j >> 1) & 1u) ^ 1u, p.status, ST_TIMEOUT_EMPTY)) {
-            *s_abort = 1;
+          if (!__all_sync(0xffffffffu, mbar_wait(&x_empty[x], (uint32_t(j >> 1) & 1u) ^ 1u, p.status, ST_TIMEOUT_EMPTY))) {
+            if (lane == 0) *s_abort = 1;
+            ok = false;
             break;
           }
-          mbar_expect_tx(&x_full[x], bytes);
+          lt_expect(&x_full[x], bytes, el);
           load(s_x + x * LT_SUB, &x_full[x], pairs * 128);
         }
       }
