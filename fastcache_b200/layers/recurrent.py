@@ -23,8 +23,9 @@ def fp32_vector(*shape: int) -> nn.Parameter:
 
 
 class GatedLinearAttention(nn.Module):
-    """S <- diag(alpha) S + k v^T, o = S^T q per head, with a decay alpha per key channel and token from a low-rank
-    projection, alpha = sigmoid(z)^(1 / tau); the head outputs are RMS-normed and gated with silu."""
+    """A memory M [dim, vdim] per head whose row r fades by its own factor at every token before the outer product of key
+    and value is added; a token reads M with its query.  The factors come from a low-rank projection through
+    sigmoid(.)^(1 / tau); the head outputs are RMS-normed and gated with silu."""
 
     def __init__(self, width: int, heads: int, dim: int, vdim: int, rank: int, tau: float, eps: float):
         super().__init__()
@@ -49,9 +50,10 @@ class GatedLinearAttention(nn.Module):
 
 
 class GatedDeltaRule(nn.Module):
-    """S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q per head, with q, k, v from projections followed
-    by a short causal convolution and silu, unit-norm q and k shared by groups of heads, one decay and one step size
-    per head; the head outputs are RMS-normed and gated with silu."""
+    """A memory M [dim, vdim] per head that fades as a whole and is then corrected towards the token's value: of the
+    difference between v and what M returns for k, the share `beta` is written under k; the query reads after the
+    write.  q, k, v pass a short causal convolution and silu, q and k are unit vectors shared by groups of heads, fading
+    and share are one number per head and token; the head outputs are RMS-normed and gated with silu."""
 
     def __init__(self, width: int, heads: int, kv_heads: int, dim: int, vdim: int, taps: int, eps: float,
                  unit_eps: float = 1e-6):

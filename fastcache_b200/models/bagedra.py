@@ -22,7 +22,7 @@ from ..parallel import tp as tpmod
 
 
 class BagedraMLP(nn.Module):
-    """W_down (gelu_tanh(W_gate h) * (W_up h)), all three with biases."""
+    """GEGLU feed-forward (tanh form of gelu) whose three projections have biases."""
 
     def __init__(self, width: int, ff: int):
         super().__init__()
