@@ -1,23 +1,28 @@
 """What the layers of a hybrid model keep between steps, and the pools that hold it.
 
 A model whose layers do not all keep the same K/V rows describes its needs with `cache_layout()`, one `LayerCache`
-per layer that owns something: `row_width` elements per token in pages (block tables and slots as for K/V rows),
-and named fp32 tensors per request in state slots.  A layer that reads another layer's rows is bound to that layer's
-pages by the model.
+per owner (a layer, or one pass through a layer that runs several times): `row_width` elements per token in pages (block
+tables and slots as for K/V rows), or keys and values of `kv` = (heads, dim) in pages of the layout of the K/V pool, and
+named fp32 tensors per request in state slots.  A layer that reads another layer's rows is bound to that layer's pages by
+the model.
 """
 from __future__ import annotations
 
 from dataclasses import dataclass, field
-from typing import Dict, List, Tuple
+from typing import Any, Dict, List, Optional, Tuple
 
 import torch
-from torch import nn
+
+
+class PassCache:
+    """What one pass through a layer keeps; the attributes are bound here (k_rows and v_rows, or the named states)."""
 
 
 @dataclass
 class LayerCache:
-    module: nn.Module
+    module: Any                                   # receives the tensors as attributes
     row_width: int = 0
+    kv: Optional[Tuple[int, int]] = None
     state: Dict[str, Tuple[int, ...]] = field(default_factory=dict)
 
 
@@ -28,7 +33,7 @@ def state_bytes(layout: List[LayerCache]) -> int:
 
 def row_bytes(layout: List[LayerCache], dtype: torch.dtype) -> int:
     """Bytes of paged rows of one token."""
-    return sum(c.row_width for c in layout) * torch.empty((), dtype=dtype).element_size()
+    return sum(c.row_width + (2 * c.kv[0] * c.kv[1] if c.kv else 0) for c in layout) * torch.empty((), dtype=dtype).element_size()
 
 
 def allocate_states(layout: List[LayerCache], num_slots: int, device: torch.device) -> None:
@@ -44,10 +49,15 @@ def allocate_rows(layout: List[LayerCache], num_blocks: int, block_size: int, dt
     for c in layout:
         if c.row_width:
             c.module.rows = torch.zeros(num_blocks, block_size, c.row_width, dtype=dtype, device=device)
+        if c.kv:
+            heads, dim = c.kv
+            for name in ("k_rows", "v_rows"):
+                setattr(c.module, name, torch.zeros(num_blocks, heads, block_size, dim, dtype=dtype, device=device))
 
 
 def release(layout: List[LayerCache]) -> None:
     for c in layout:
         for name in c.state:
             setattr(c.module, name, None)
-        c.module.rows = None
+        for name in ("rows",) if c.row_width else ("k_rows", "v_rows") if c.kv else ():
+            setattr(c.module, name, None)

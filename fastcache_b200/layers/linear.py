@@ -138,6 +138,35 @@ class PackedLinear(nn.Module):
         return ops.linear(x, self.weight, self.bias)
 
 
+class JoinedLinear(nn.Module):
+    """Projections of several inputs to one sum (one GEMM, not split over ranks): the inputs stand side by side in one
+    matrix, each from a multiple of 8 columns on, the weights likewise.  `offset[name]` is an input's first column."""
+
+    def __init__(self, inputs: Dict[str, int], output_size: int):
+        super().__init__()
+        self.sizes = dict(inputs)
+        self.output_size = output_size
+        self.offset: Dict[str, int] = {}
+        n = 0
+        for name, size in inputs.items():
+            self.offset[name] = n
+            n += pad8(size)
+        self.input_size = n
+        self.weight = nn.Parameter(torch.zeros(pad8(output_size), n), requires_grad=False)
+        self.weight.weight_loader = self.weight_loader
+
+    def weight_loader(self, param: nn.Parameter, loaded: torch.Tensor, shard_id=None) -> None:
+        """`shard_id` names one input; without it the tensor holds all of them, side by side and unpadded."""
+        names = list(self.sizes) if shard_id is None else [shard_id]
+        if loaded.shape != (self.output_size, sum(self.sizes[n] for n in names)):
+            raise ValueError(f"shape mismatch: {tuple(loaded.shape)} for inputs {names} of {self.sizes}")
+        at = 0
+        for n in names:
+            o = self.offset[n]
+            param.data[: self.output_size, o:o + self.sizes[n]].copy_(loaded[:, at:at + self.sizes[n]])
+            at += self.sizes[n]
+
+
 class QKVParallelLinear(LinearBase):
     def __init__(self, hidden_size: int, head_size: int, total_num_heads: int,
                  total_num_kv_heads: Optional[int] = None, bias: bool = False):

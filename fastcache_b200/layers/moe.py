@@ -1,0 +1,58 @@
+"""Mixture of experts: gated feed-forward experts and a router that reads a table of the token ids."""
+from __future__ import annotations
+
+import torch
+from torch import nn
+
+from .. import ops
+from ..ops.hybrid import GluSpec
+from ..utils.context import get_context
+from .linear import pad8
+
+
+class TableRouter(nn.Module):
+    """Every token id has its experts in a table [vocab, top]; they count equally."""
+
+    def __init__(self, vocab: int, experts: int, top: int):
+        super().__init__()
+        if not 0 < top <= experts:
+            raise ValueError(f"{top} experts per token of {experts}")
+        self.experts = experts
+        spread = (torch.arange(vocab)[:, None] * top + torch.arange(top)) % experts
+        self.table = nn.Parameter(spread.to(torch.int32), requires_grad=False)
+        self.table.weight_loader = self._load
+
+    def _load(self, param: nn.Parameter, loaded: torch.Tensor, shard_id=None) -> None:
+        if loaded.shape != param.data.shape or loaded.is_floating_point():
+            raise ValueError(f"an integer table of {tuple(param.data.shape)} expected, got {loaded.dtype} {tuple(loaded.shape)}")
+        if loaded.min() < 0 or loaded.max() >= self.experts:
+            raise ValueError(f"the table names experts outside 0 .. {self.experts - 1}")
+        param.data.copy_(loaded)
+
+    def forward(self, input_ids: torch.Tensor):
+        """The step's routing; depends on the ids alone, so passes that run a layer again share it."""
+        return ops.hybrid.route_by_table(input_ids, self.table, self.experts, get_context())
+
+
+class Experts(nn.Module):
+    """Gated feed-forward experts without biases, stacked: [E, gate rows | up rows, width] and [E, width, ff]."""
+
+    def __init__(self, width: int, experts: int, ff: int, spec: GluSpec):
+        super().__init__()
+        self.width, self.count, self.ff, self.spec = width, experts, ff, spec
+        fp = pad8(ff)
+        self.gate_up = nn.Parameter(torch.zeros(experts, 2 * fp, pad8(width)), requires_grad=False)
+        self.gate_up.weight_loader = self._load
+        self.down = nn.Parameter(torch.zeros(experts, pad8(width), fp), requires_grad=False)
+        self.down.weight_loader = self._load
+
+    def _load(self, param: nn.Parameter, loaded: torch.Tensor, shard_id=None) -> None:
+        e, name = shard_id
+        at = pad8(self.ff) if name == "up" else 0
+        want = (self.width, self.ff) if name == "down" else (self.ff, self.width)
+        if loaded.shape != want:
+            raise ValueError(f"shape mismatch: {tuple(loaded.shape)} for {name} of {want}")
+        param.data[e, at:at + want[0], :want[1]].copy_(loaded)
+
+    def forward(self, h: torch.Tensor, route, weights=None):
+        return ops.hybrid.experts(h, route, weights, self.gate_up, self.down, self.ff, self.spec)

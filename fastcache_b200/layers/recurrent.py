@@ -1,6 +1,6 @@
-"""Recurrent mixers with a fixed-size state per request: gated linear attention and the gated delta rule.
+"""Recurrent mixers with a fixed-size state per request: gated linear attention, the gated delta rule, matrix memory.
 
-Both read the state that earlier steps left in the request's slot (`state`, and `conv_state` for the short
+They read the state that earlier steps left in the request's slot (`state`, and `conv_state` for the short
 convolutions), advance it by the rows of the batch and leave it there; prefill portions of any length and decode
 steps go through the same call.
 """
@@ -12,7 +12,8 @@ import torch
 from torch import nn
 
 from .. import ops
-from ..ops.hybrid import DeltaDims, GlaDims
+from ..engine.layer_cache import LayerCache, PassCache
+from ..ops.hybrid import DeltaDims, GlaDims, MatrixMemoryDims
 from ..utils.context import get_context
 from .linear import PackedLinear
 
@@ -87,3 +88,35 @@ class GatedDeltaRule(nn.Module):
     def forward(self, positions: torch.Tensor, h: torch.Tensor) -> torch.Tensor:
         return ops.hybrid.delta_rule(h, self.in_proj.weight, self.dims, self.conv, self.a_log, self.dt_bias,
                                      self.norm, self.eps, self.conv_state, self.state, get_context())
+
+
+class MatrixMemory(nn.Module):
+    """mLSTM (Beck et al., "xLSTM: Extended Long Short-Term Memory"): a memory M [dim, vdim] and a normaliser n [dim] per
+    head, written with exponential gates that are kept in range by a running maximum of their logarithms (which starts
+    at 0).  Gates pass a soft cap; the head outputs are RMS-normed, weighted and gated with sigmoid.
+
+    Like `WindowedAttention` it works between projections that its owner holds."""
+
+    wide = ("i", "f")
+
+    def __init__(self, heads: int, dim: int, vdim: int, cap: float, eps: float):
+        super().__init__()
+        self.eps = eps
+        self.heads, self.dim, self.vdim, self.cap = heads, dim, vdim, float(cap)
+        self.sizes: Dict[str, int] = {"q": heads * dim, "k": heads * dim, "v": heads * vdim, "g": heads * vdim, "i": heads,
+                                      "f": heads}
+        self.out_width = heads * vdim
+        self.norm = fp32_vector(heads * vdim)
+        self.i_bias = fp32_vector(heads)
+        self.f_bias = fp32_vector(heads)
+        self.vectors = {"norm": "norm", "i.b": "i_bias", "f.b": "f_bias"}
+
+    def bind(self, offset: Dict[str, int]) -> None:
+        self.dims = MatrixMemoryDims(self.heads, self.dim, self.vdim, self.cap, *(offset[n] for n in "qkvgif"))
+
+    def cache(self) -> LayerCache:
+        return LayerCache(PassCache(), state={"state": (self.heads, self.dim, self.vdim),
+                                              "norm_state": (self.heads, self.dim), "max_state": (self.heads,)})
+
+    def forward(self, positions: torch.Tensor, p, cache: PassCache, out: torch.Tensor) -> None:
+        ops.hybrid.matrix_memory(p, self.dims, self.i_bias, self.f_bias, self.norm, self.eps, cache, get_context(), out)

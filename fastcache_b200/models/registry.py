@@ -22,6 +22,8 @@ def detect_model_type(hf_config: Any) -> str:
         return "qwen2"
     if "bagedra" in mt or "bagedra" in joined:
         return "bagedra"
+    if "lekilix" in mt or "lekilix" in joined:
+        return "lekilix"
     if "llama" in mt or "llama" in joined or "mistral" in mt:
         return "llama"
     raise ValueError(f"unsupported model type {mt!r} / architectures {archs}")
@@ -57,9 +59,14 @@ def _bagedra(cfg):
     return BagedraForCausalLM(cfg)
 
 
+def _lekilix(cfg):
+    from .lekilix import LekilixForCausalLM
+    return LekilixForCausalLM(cfg)
+
+
 MODEL_REGISTRY: Dict[str, Callable] = {
     "llama": _llama, "qwen3": _qwen3, "qwen2": _qwen2, "llava": _llava, "minicpm": _minicpm,
-    "bagedra": _bagedra,
+    "bagedra": _bagedra, "lekilix": _lekilix,
 }
 
 

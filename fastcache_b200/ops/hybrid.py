@@ -1,4 +1,4 @@
-"""Ops of hybrid models (recurrent layers, latent attention, sublayer-output norms on a 32-bit residual stream).
+"""Ops of hybrid models (recurrent layers, latent and windowed attention, experts, norms on a 32-bit residual stream).
 
 Same rule as the other ops of this package: the device of the data decides between the sm_100a kernels and the
 PyTorch statements of `reference_hybrid.py`.  Inputs and outputs are in the model's dtype (bf16, or fp32 for runs
@@ -66,6 +66,50 @@ class LatentDims:
     q: int
     g: int
     kv: Optional[int]
+
+
+@dataclass(frozen=True)
+class WindowDims:
+    """Windowed attention over keys that are also the values; first columns of the packed projections.  `window`: the
+    positions a query sees, itself included (0: all up to itself)."""
+    heads: int
+    kv_heads: int
+    dim: int
+    rot_dims: int
+    base: float
+    scale: float
+    window: int
+    q: int
+    k: int
+    g: int
+
+
+@dataclass(frozen=True)
+class MatrixMemoryDims:
+    """Matrix memory (mLSTM): sizes, soft cap of the gates, first columns of the packed projections; `floor` is added to
+    the normaliser."""
+    heads: int
+    dim: int
+    vdim: int
+    cap: float
+    q: int
+    k: int
+    v: int
+    g: int
+    i: int
+    f: int
+    floor: float = 1e-6
+
+
+@dataclass(frozen=True)
+class GluSpec:
+    """Gated activation: "silu", or "clamped" (see `reference_hybrid.glu`) with its limit."""
+    act: str = "silu"
+    limit: float = 0.0
+
+    @property
+    def code(self) -> int:
+        return {"silu": 0, "clamped": 1}[self.act]
 
 
 # ------------------------------------------------------------------ residual stream
@@ -152,3 +196,93 @@ def latent_attention(h, weight, d: LatentDims, kv_norm_w, eps: float, kv_proj, w
     w, off = kv_proj.weight, kv_proj.offset
     return ref.latent_attention(q, p[:, d.g:d.g + d.heads * d.vdim], d, w[off["uk"]:off["uk"] + d.heads * d.dim],
                                 w[off["uv"]:off["uv"] + d.heads * d.vdim], pool, ctx)
+
+
+# ------------------------------------------------------------------ pre-normed layers with parallel sublayers
+SMALL_ROWS = 256        # up to this many rows a projection stays fp32 split-K partial sums for its readers
+
+
+def project(h, weight, rows: Optional[int] = None, wide=None):
+    """h @ weight[:rows].T for the ops below: a matrix on CPU, an extension object on CUDA (for up to SMALL_ROWS rows its
+    fp32 partial sums, valid until the next product).  `wide` = (first, count): columns that are kept in fp32."""
+    if h.is_cuda:
+        _n()
+        first, count = wide or (0, 0)
+        return ext().project(h, weight, int(rows or weight.shape[0]), int(first), int(count))
+    return ref_linear(h, weight if rows is None else weight[:rows])
+
+
+def linear_add_norm(a, weight, x, norm_w, eps: float, add: bool = True, experts=None, out=None):
+    """x (+)= a @ weight.T + the mixed outputs of `experts` in fp32, in place; returns RMSNorm(x) * norm_w (norm_w None: x
+    itself) in the model's dtype, in `out` if given."""
+    if a.is_cuda:
+        _n(2)
+        y, row_of, mix = experts or (None, None, None)
+        return ext().linear_add_norm(a, weight, x, norm_w, float(eps), bool(add), y, row_of, mix, out)
+    h = ref.add_norm(ref_linear(a, weight), x, add, norm_w, eps, experts)
+    return h if out is None else out.copy_(h)
+
+
+def glu(p, gate: int, up: int, width: int, spec: GluSpec, out):
+    """act(gate) * up of a projection, to `out` (its columns past `width` are zeroed)."""
+    if out.is_cuda:
+        _n()
+        ext().glu(p, int(gate), int(up), int(width), spec.code, float(spec.limit), out)
+    else:
+        out.copy_(ref._pad_to(ref.glu(p[:, gate:gate + width], p[:, up:up + width], spec.act, spec.limit), out.shape[1]))
+
+
+def linear_glu(h, weight, up: int, width: int, spec: GluSpec, out):
+    """The same of the product h @ weight.T, weight = gate rows, then (from row `up`) up rows; prefill sizes run the gate in
+    the GEMM's epilogue."""
+    if out.is_cuda:
+        _n(2)
+        ext().linear_glu(h, weight, int(up), int(width), spec.code, float(spec.limit), out)
+    else:
+        glu(ref_linear(h, weight), 0, up, width, spec, out)
+
+
+# ------------------------------------------------------------------ experts
+def route_by_table(ids, table, experts: int, ctx):
+    """Which rows every expert gets when a token's id names its experts (table [vocab, top], int32).  CPU: [T, top]."""
+    if ids.is_cuda:
+        _n()
+        return ext().route_by_table(ids, table, int(experts), None if ctx.is_prefill else ctx.context_lens)
+    return table[ids].long()
+
+
+def experts(h, route, weights, w_gate_up, w_down, ff: int, spec: GluSpec):
+    """Expert outputs for `linear_add_norm`: every token's chosen experts, mixed there with `weights` [T, top] fp32 (None:
+    equal ones).  w_gate_up [E, 2 * padded ff, K]: gate rows, then up rows; w_down [E, N, padded ff]."""
+    if h.is_cuda:
+        _n(4)
+        row_of, plan = route
+        return ext().experts(h, plan, row_of.shape[1], w_gate_up, w_down, int(ff), spec.code, float(spec.limit)), row_of, weights
+    return ref.experts(h, route, weights, w_gate_up, w_down, ff, spec.act, spec.limit)
+
+
+# ------------------------------------------------------------------ windowed attention
+ATTN_IMPL = 0           # tests: 1 the general kernel also where a tensor-core form exists
+
+
+def windowed_attention(p, d: WindowDims, q_norm, k_norm, sink, eps: float, k_rows, v_rows, positions, ctx, out):
+    """Norm over the whole projection, rotation, cache store, attention with a sink and output gate, to `out`."""
+    if out.is_cuda:
+        _n(2)
+        ext().windowed_attention(p, [d.heads, d.kv_heads, d.dim, d.rot_dims, d.window, d.q, d.k, d.g], d.scale, d.base,
+                                 q_norm, k_norm, sink, float(eps), k_rows, v_rows, positions, ctx.slot_mapping,
+                                 ctx.block_tables, ctx.context_lens, ctx.cu_seqlens_q, ctx.row_seq, ctx.row_ctx,
+                                 int(ctx.max_seqlen_q), int(ctx.max_seqlen_k), out, ATTN_IMPL)
+    else:
+        ref.windowed_attention(p, d, q_norm, k_norm, sink, eps, k_rows, v_rows, positions, ctx, out)
+
+
+# ------------------------------------------------------------------ matrix memory
+def matrix_memory(p, d: MatrixMemoryDims, i_bias, f_bias, norm_w, eps: float, cache, ctx, out):
+    """mLSTM of a batch of runs with head norm and output gate, to `out`."""
+    if out.is_cuda:
+        _n(3)
+        ext().matrix_memory(p, [d.heads, d.dim, d.vdim, d.q, d.k, d.v, d.g, d.i, d.f], d.cap, d.floor, i_bias, f_bias,
+                            norm_w, float(eps), cache.state, cache.norm_state, cache.max_state, *_run_args(ctx), out)
+    else:
+        ref.matrix_memory(p, d, i_bias, f_bias, norm_w, eps, cache.state, cache.norm_state, cache.max_state, ctx, out)

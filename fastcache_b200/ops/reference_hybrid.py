@@ -1,5 +1,5 @@
-"""Plain PyTorch statements of the ops of hybrid models: sublayer-output norm on a 32-bit residual, short
-convolution, gated linear attention, gated delta rule and paged latent attention.
+"""Plain PyTorch statements of the ops of hybrid models: norms on a 32-bit residual, short convolution, gated linear
+attention, gated delta rule, matrix memory, paged latent attention, windowed attention with a sink, experts.
 
 Like `reference.py`: the execution path on CPU tensors.  A batch is a concatenation of runs of rows, one run per
 request, with the request's state slot and the position of its first row; a run that starts at position 0 starts
@@ -155,3 +155,101 @@ def latent_attention(q, gate, d, w_uk, w_uv, pool, ctx):
         out[lo:hi] = torch.einsum("hij,jhv->ihv", torch.softmax(s.masked_fill(hidden, float("-inf")), -1), v)
     y = out.reshape(T, H * d.vdim) * torch.sigmoid(gate.float())
     return _pad_to(y.to(q.dtype), -(-H * d.vdim // 8) * 8)
+
+
+# ------------------------------------------------------------------ pre-normed layers
+def add_norm(y, x, add: bool, norm_w, eps: float, experts=None):
+    """x (+)= y + the mixed expert outputs, in place; returns rms(x) * norm_w, or x itself where norm_w is None."""
+    if not add:
+        x.zero_()
+    x += y[:, : x.shape[1]].float()
+    if experts is not None:
+        x += experts[:, : x.shape[1]].float()
+    n = x if norm_w is None else _rms(x, eps) * norm_w
+    return _pad_to(n.to(y.dtype), y.shape[1])
+
+
+def glu(gate, up, act: str, limit: float):
+    """act(gate) * up ("silu"), or the clamped form ("clamped"): g * sigmoid(1.702 g) * (u + 1) with g = min(gate, limit)
+    and u = up clamped to +-limit."""
+    g, u = gate.float(), up.float()
+    if act == "silu":
+        return (F.silu(g) * u).to(gate.dtype)
+    g, u = g.clamp(max=limit), u.clamp(-limit, limit)
+    return (g * torch.sigmoid(1.702 * g) * (u + 1)).to(gate.dtype)
+
+
+def experts(h, ids, weights, w_gate_up, w_down, ff: int, act: str, limit: float):
+    """Sum over a token's experts `ids` [T, top] of weight * down(glu(gate, up)); weights None: equal ones."""
+    out = torch.zeros(h.shape[0], w_down.shape[1], dtype=torch.float32, device=h.device)
+    half = w_gate_up.shape[1] // 2
+    for e in ids.unique().tolist():
+        t, j = (ids == e).nonzero(as_tuple=True)
+        gu = h[t].float() @ w_gate_up[e].float().T
+        y = _pad_to(glu(gu[:, :ff], gu[:, half:half + ff], act, limit).to(h.dtype), w_down.shape[2]).float() @ w_down[e].float().T
+        out.index_add_(0, t, y * (1.0 / ids.shape[1] if weights is None else weights[t, j][:, None]))
+    return out
+
+
+def rope_pairs(x, positions, base: float, dims: int):
+    """Interleaved rotation: columns 2i and 2i + 1 below `dims` of x [T, H, D] turn by position * base^(-2i / dims)."""
+    i = torch.arange(dims // 2, dtype=torch.float64, device=x.device)
+    a = positions.double()[:, None, None] * base ** (-2 * i / dims)
+    c, s = a.cos().float(), a.sin().float()
+    u, v = x[..., 0:dims:2].float(), x[..., 1:dims:2].float()
+    turned = torch.stack([u * c - v * s, v * c + u * s], -1).flatten(-2)
+    return torch.cat([turned, x[..., dims:].float()], -1)
+
+
+def windowed_attention(p, d, q_norm, k_norm, sink, eps: float, k_rows, v_rows, positions, ctx, out):
+    """Stores the batch's keys and values (the raw keys) in the pages and writes attention times sigmoid(gate) to `out`.
+    d: `ops.hybrid.WindowDims`; a query at position i sees the last d.window positions up to i (0: all)."""
+    T, H, G, D = p.shape[0], d.heads, d.kv_heads, d.dim
+    q, k = p[:, d.q:d.q + H * D].float(), p[:, d.k:d.k + G * D]
+    q = rope_pairs((_rms(q, eps) * q_norm).view(T, H, D), positions, d.base, d.rot_dims).to(p.dtype)
+    kn = rope_pairs((_rms(k.float(), eps) * k_norm).view(T, G, D), positions, d.base, d.rot_dims)
+    ok = ctx.slot_mapping >= 0
+    slots = ctx.slot_mapping[ok].long()
+    bs = k_rows.shape[2]
+    k_rows[slots // bs, :, slots % bs] = kn[ok].to(k_rows.dtype)
+    v_rows[slots // bs, :, slots % bs] = k.reshape(T, G, D)[ok].to(v_rows.dtype)
+    o = torch.zeros(T, H, D)
+    for i, lo, hi, start, _ in runs(ctx):
+        n = start + hi - lo
+        blocks = ctx.block_tables[i][: -(-n // bs)].long()
+        ks, vs = (r[blocks].transpose(1, 2).reshape(-1, G, D)[:n].float().repeat_interleave(H // G, 1)
+                  for r in (k_rows, v_rows))
+        s = torch.einsum("ihd,jhd->hij", q[lo:hi].float(), ks) * d.scale
+        back = torch.arange(start, n)[:, None] - torch.arange(n)[None, :]
+        hidden = back < 0 if d.window <= 0 else (back < 0) | (back >= d.window)
+        s = torch.cat([s.masked_fill(hidden, float("-inf")), sink[:, None, None].expand(-1, hi - lo, 1)], -1)
+        o[lo:hi] = torch.einsum("hij,jhd->ihd", torch.softmax(s, -1)[..., :-1], vs)
+    y = o.reshape(T, H * D) * torch.sigmoid(p[:, d.g:d.g + H * D].float())
+    out.copy_(_pad_to(y.to(p.dtype), out.shape[1]))
+
+
+def matrix_memory(p, d, i_bias, f_bias, norm_w, eps: float, state, norm_state, max_state, ctx, out):
+    """d: `ops.hybrid.MatrixMemoryDims`; p packed projections."""
+    T, H, D, V = p.shape[0], d.heads, d.dim, d.vdim
+    q = p[:, d.q:d.q + H * D].float().view(T, H, D) * D ** -0.5
+    k = p[:, d.k:d.k + H * D].float().view(T, H, D)
+    v = p[:, d.v:d.v + H * V].float().view(T, H, V)
+    gi = d.cap * torch.tanh((p[:, d.i:d.i + H].float() + i_bias) / d.cap)
+    gf = F.logsigmoid(d.cap * torch.tanh((p[:, d.f:d.f + H].float() + f_bias) / d.cap))
+    o = q.new_zeros(T, H, V)
+    for _, lo, hi, start, slot in runs(ctx):
+        if start == 0:
+            S, n, m = state.new_zeros(H, D, V), state.new_zeros(H, D), state.new_zeros(H)
+        else:
+            S, n, m = state[slot].clone(), norm_state[slot].clone(), max_state[slot].clone()
+        for t in range(lo, hi):
+            top = torch.maximum(gf[t] + m, gi[t])
+            keep, write = torch.exp(gf[t] + m - top), torch.exp(gi[t] - top)
+            m = top
+            S = keep[:, None, None] * S + (write[:, None] * k[t])[:, :, None] * v[t][:, None, :]
+            n = keep[:, None] * n + write[:, None] * k[t]
+            den = torch.maximum((n * q[t]).sum(-1).abs(), torch.exp(-m)) + d.floor
+            o[t] = torch.einsum("hdv,hd->hv", S, q[t]) / den[:, None]
+        state[slot], norm_state[slot], max_state[slot] = S, n, m
+    y = _rms(o, eps).reshape(T, H * V) * norm_w * torch.sigmoid(p[:, d.g:d.g + H * V].float())
+    out.copy_(_pad_to(y.to(p.dtype), out.shape[1]))
