@@ -53,7 +53,7 @@ Tensor prefill_attention(const Tensor& q, const Tensor& kc, const Tensor& vc, co
   if (impl == 3 || (impl == 0 && tc_ok && max_q_len > 64)) {
     fc::launch_prefill_attention_tc2(q.data_ptr(), kc.data_ptr(), vc.data_ptr(), block_tables.data_ptr<int>(),
                                      cu_q.data_ptr<int>(), kv_lens.data_ptr<int>(), out.data_ptr(), q.size(0), int(B),
-                                     int(max_q_len), int(Hq), int(kc.size(1)), int(kc.size(2)),
+                                     int(max_q_len), int(Hq), int(kc.size(1)), int(D), int(kc.size(2)),
                                      int(block_tables.size(1)), int(kc.size(0)), float(scale),
                                      status_ptr(q.get_device()), at::cuda::getCurrentCUDAStream());
     return out;

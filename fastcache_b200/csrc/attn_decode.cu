@@ -17,6 +17,10 @@
 // This op is bound by HBM bandwidth (K and V are read exactly once, ~16 FLOP per
 // byte), so the legacy tensor path is enough to keep the memory system busy; the
 // tcgen05 path is used where the work is compute-bound.
+//
+// Options for other designs (AttnOptions): a sliding window (tiles before it are not read), a sink per head (one more
+// term of the denominator, added where the splits end up), heads narrower than the rows of the pool, and a gate that
+// multiplies the output.
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
 #include <stdint.h>
@@ -49,10 +53,25 @@ __device__ __forceinline__ uint32_t tswz(int row, int chunk) {
 // written; the last one to arrive merges all splits of the group's query heads
 //     out[b, h, :] = sum_s w_s * part_o[b, h, s, :],  w_s = 2^(lse_s - max) / sum
 // and puts the counter back to zero for the next launch (also a replay from a CUDA graph).
+// head output value `v` of column c (a row of the pool has D columns, the head opt.dim of them)
+__device__ __forceinline__ void put_head(const AttnOptions& opt, bf16* __restrict__ out, int b, int hq, int c, float v) {
+  const int dim = opt.dim;
+  if (c >= dim) return;
+  if (opt.gate != nullptr) {
+    const float g = __bfloat162float(reinterpret_cast<const bf16*>(opt.gate)[b * opt.ld_gate + hq * dim + c]);
+    v *= __fdividef(1.f, 1.f + __expf(-g));
+  }
+  out[b * opt.ld_out + hq * dim + c] = __float2bfloat16(v);
+}
+// the sink's share of a denominator whose terms are relative to `top` (log2 units)
+__device__ __forceinline__ float sink_term(const AttnOptions& opt, int hq, float top) {
+  return opt.sink != nullptr ? exp2f(opt.sink[hq] * 1.4426950408889634f - top) : 0.f;
+}
+
 template <int D>
 __device__ __forceinline__ void decode_merge_last(const float* __restrict__ part_o, const float* __restrict__ part_lse,
                                                   bf16* __restrict__ out, int* __restrict__ counters, int b, int hk,
-                                                  int G, int Hq, int Hkv, int splits) {
+                                                  int G, int Hq, int Hkv, int splits, const AttnOptions& opt) {
   __shared__ int s_last;
   __threadfence();
   __syncthreads();
@@ -77,9 +96,9 @@ __device__ __forceinline__ void decode_merge_last(const float* __restrict__ part
         den += w;
         acc += w * __ldcg(part_o + (bh * splits + s) * D + c);
       }
-      acc /= den;
+      acc /= den + sink_term(opt, hk * G + r, mx);
     }
-    out[bh * D + c] = __float2bfloat16(acc);
+    put_head(opt, out, b, hk * G + r, c, acc);
   }
   if (threadIdx.x == 0) counters[b * Hkv + hk] = 0;
 }
@@ -90,7 +109,7 @@ decode_attn_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_consta
                    const bf16* __restrict__ q, int box_rows, const int* __restrict__ block_tables, const int* __restrict__ context_lens,
                    bf16* __restrict__ out, float* __restrict__ part_o, float* __restrict__ part_lse, int Hq,
                    int Hkv, int block_size, int max_blocks, int num_blocks, int splits, float scale_log2,
-                   uint32_t* status, int* __restrict__ merge_counters) {
+                   uint32_t* status, int* __restrict__ merge_counters, const AttnOptions opt) {
   constexpr int CH = D / 8;                  // 16-byte chunks per row
   constexpr int TILE_BYTES = DEC_TILE * D * 2;
   extern __shared__ uint8_t smem_raw[];
@@ -116,10 +135,11 @@ decode_attn_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_consta
   const int g = lane >> 2, t = lane & 3;
 
   const int ctx = context_lens[b];
-  const int tiles_total = (ctx + DEC_TILE - 1) / DEC_TILE;
-  const int tiles_per = (tiles_total + splits - 1) / splits;
-  const int tile0 = split * tiles_per;
-  const int tile1 = min(tiles_total, tile0 + tiles_per);
+  const int first = opt.window > 0 ? max(0, ctx - opt.window) : 0;      // first visible row
+  const int tile_first = first / DEC_TILE, tile_end = (ctx + DEC_TILE - 1) / DEC_TILE;
+  const int tiles_per = (tile_end - tile_first + splits - 1) / splits;
+  const int tile0 = tile_first + split * tiles_per;
+  const int tile1 = min(tile_end, tile0 + tiles_per);
   const int n_tiles = max(0, tile1 - tile0);
   const int* bt = block_tables + (long long)b * max_blocks;
 
@@ -220,7 +240,7 @@ decode_attn_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_consta
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
         const int tok = tok_base + n * 8 + 2 * t + e;
-        if (tok >= ctx) {
+        if (tok >= ctx || tok < first) {
           sc[n][e] = -INFINITY;
           sc[n][2 + e] = -INFINITY;
         } else {
@@ -288,13 +308,13 @@ decode_attn_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_consta
       const int r = idx / D, c = idx - r * D;
       const int hq = hk * G + r;
       if (splits == 1) {
-        out[((long long)b * Hq + hq) * D + c] = __float2bfloat16(0.f);
+        put_head(opt, out, b, hq, c, 0.f);
       } else {
         part_o[(((long long)b * Hq + hq) * splits + split) * D + c] = 0.f;
         if (c == 0) part_lse[((long long)b * Hq + hq) * splits + split] = -INFINITY;
       }
     }
-    if (splits > 1 && merge_counters != nullptr) decode_merge_last<D>(part_o, part_lse, out, merge_counters, b, hk, G, Hq, Hkv, splits);
+    if (splits > 1 && merge_counters != nullptr) decode_merge_last<D>(part_o, part_lse, out, merge_counters, b, hk, G, Hq, Hkv, splits, opt);
     return;
   }
 
@@ -338,24 +358,25 @@ decode_attn_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_consta
       }
     }
     const int hq = hk * G + r;
-    const float val = (ll > 0.f) ? acc / ll : 0.f;
     if (splits == 1) {
-      out[((long long)b * Hq + hq) * D + c] = __float2bfloat16(val);
+      put_head(opt, out, b, hq, c, ll > 0.f ? acc / (ll + sink_term(opt, hq, mm)) : 0.f);
     } else {
+      const float val = (ll > 0.f) ? acc / ll : 0.f;
       part_o[(((long long)b * Hq + hq) * splits + split) * D + c] = val;
       if (c == 0)
         part_lse[((long long)b * Hq + hq) * splits + split] = (ll > 0.f) ? (mm + log2f(ll)) : -INFINITY;
     }
   }
-  if (splits > 1 && merge_counters != nullptr) decode_merge_last<D>(part_o, part_lse, out, merge_counters, b, hk, G, Hq, Hkv, splits);
+  if (splits > 1 && merge_counters != nullptr) decode_merge_last<D>(part_o, part_lse, out, merge_counters, b, hk, G, Hq, Hkv, splits, opt);
 }
 
 // out[b, h, :] = sum_s w_s * part_o[b, h, s, :],  w_s = 2^(lse_s - max) / sum
 __global__ void decode_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_lse,
-                                    bf16* __restrict__ out, int splits, int D) {
+                                    bf16* __restrict__ out, int splits, int D, int Hq, const AttnOptions opt) {
   pdl_launch_dependents();
   pdl_wait();
   const long long bh = blockIdx.x;
+  const int b = blockIdx.x / Hq, hq = blockIdx.x - b * Hq;
   const float* lse = part_lse + bh * splits;
   // the partials come from the kernel right before this one: L2 loads, not the read-only path (see above)
   float mx = -INFINITY;
@@ -365,6 +386,7 @@ __global__ void decode_merge_kernel(const float* __restrict__ part_o, const floa
     const float l = __ldcg(lse + s);
     den += (l == -INFINITY) ? 0.f : exp2f(l - mx);
   }
+  if (mx != -INFINITY) den += sink_term(opt, hq, mx);
   for (int c = threadIdx.x; c < D; c += blockDim.x) {
     float acc = 0.f;
     if (mx != -INFINITY) {
@@ -375,7 +397,7 @@ __global__ void decode_merge_kernel(const float* __restrict__ part_o, const floa
       }
       acc /= den;
     }
-    out[bh * D + c] = __float2bfloat16(acc);
+    put_head(opt, out, b, hq, c, acc);
   }
 }
 
@@ -390,8 +412,13 @@ int decode_attn_pick_splits(int B, int Hkv, int max_ctx, int num_sms) {
 void launch_decode_attention(const void* q, const void* k_cache, const void* v_cache, const int* block_tables,
                              const int* context_lens, void* out, float* part_o, float* part_lse, int B, int Hq,
                              int Hkv, int D, int block_size, int max_blocks, int num_blocks, int splits,
-                             float scale, uint32_t* status, cudaStream_t stream, int* merge_counters) {
+                             float scale, uint32_t* status, cudaStream_t stream, int* merge_counters,
+                             const AttnOptions* options) {
   if (B == 0) return;
+  AttnOptions opt;
+  if (options != nullptr) opt = *options;
+  if (opt.dim == 0) opt.dim = D;
+  if (opt.ld_out == 0) opt.ld_out = (long long)Hq * opt.dim;
   if (Hq % Hkv != 0 || Hq / Hkv > 16) throw std::runtime_error("decode attention: group size must divide and be <= 16");
   if (splits > 1 && (part_o == nullptr || part_lse == nullptr))
     throw std::runtime_error("decode attention: split-KV needs scratch");
@@ -409,7 +436,7 @@ void launch_decode_attention(const void* q, const void* k_cache, const void* v_c
     cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     launch_pdl(PDL_DECODE_ATTN, kern, grid, dim3(DEC_THREADS), smem, stream, tk, tv, (const bf16*)q, box_rows, block_tables,
                context_lens, (bf16*)out, part_o, part_lse, Hq, Hkv, block_size, max_blocks, num_blocks, splits,
-               scale_log2, status, merge_counters);
+               scale_log2, status, merge_counters, opt);
   };
   if (D == 128) launch(decode_attn_kernel<128>);
   else if (D == 64) launch(decode_attn_kernel<64>);
@@ -418,7 +445,7 @@ void launch_decode_attention(const void* q, const void* k_cache, const void* v_c
   // attention kernel itself; without them a second kernel does
   if (splits > 1 && merge_counters == nullptr)
     launch_pdl(PDL_DECODE_MERGE, decode_merge_kernel, dim3(B * Hq), dim3(128), 0, stream, (const float*)part_o, (const float*)part_lse,
-               (bf16*)out, splits, D);
+               (bf16*)out, splits, D, Hq, opt);
   cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess) throw std::runtime_error(std::string("decode attention launch: ") + cudaGetErrorString(e));
 }

@@ -33,7 +33,7 @@ __global__ void __launch_bounds__(PF_THREADS)
 prefill_attn_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_cache, const bf16* __restrict__ v_cache,
                     const int* __restrict__ block_tables, const int* __restrict__ cu_q,
                     const int* __restrict__ kv_lens, bf16* __restrict__ out, int Hq, int Hkv, int block_size,
-                    int max_blocks, int num_blocks, float scale_log2, uint32_t* status) {
+                    int max_blocks, int num_blocks, float scale_log2, uint32_t* status, const AttnOptions opt) {
   constexpr int CH = D / 8;
   constexpr int Q_BYTES = PF_BM * D * 2;
   constexpr int T_BYTES = PF_BN * D * 2;
@@ -54,7 +54,8 @@ prefill_attn_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_cache
   const int g = lane >> 2, t = lane & 3;
 
   const int kv_end = min(kv_len, offset + q0 + PF_BM);      // keys visible to this q tile
-  const int n_tiles = (kv_end + PF_BN - 1) / PF_BN;
+  const int tile0 = opt.window > 0 ? max(0, offset + q0 - opt.window + 1) / PF_BN : 0;      // tiles before the window
+  const int n_tiles = (kv_end + PF_BN - 1) / PF_BN - tile0;
 
   // ---- Q tile -> smem
 #pragma unroll
@@ -68,7 +69,7 @@ prefill_attn_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_cache
   auto load_tile = [&](int tile, int stage) {
     const uint32_t sk = s_kv + stage * 2 * T_BYTES;
     const uint32_t sv = sk + T_BYTES;
-    const int row0 = tile * PF_BN;
+    const int row0 = (tile0 + tile) * PF_BN;
 #pragma unroll
     for (int i = 0; i < (PF_BN * CH) / PF_THREADS; ++i) {
       const int c = threadIdx.x + i * PF_THREADS;
@@ -134,8 +135,10 @@ prefill_attn_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_cache
       }
     }
     // ---- scale, causal mask (only tiles that touch the diagonal or the end), row max
-    const int col0 = it * PF_BN;
-    const bool need_mask = (col0 + PF_BN - 1 > offset + q0 + warp * 16) || (col0 + PF_BN > kv_end);
+    const int col0 = (tile0 + it) * PF_BN;
+    const int win = opt.window > 0 ? opt.window : 0x40000000;           // visible: row - col < win
+    const bool need_mask = (col0 + PF_BN - 1 > offset + q0 + warp * 16) || (col0 + PF_BN > kv_end) ||
+                           (offset + q0 + warp * 16 + 15 - col0 >= win);
     float mx0 = -INFINITY, mx1 = -INFINITY;
 #pragma unroll
     for (int n = 0; n < PF_BN / 8; ++n) {
@@ -144,8 +147,8 @@ prefill_attn_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_cache
         const int col = col0 + n * 8 + 2 * t + e;
         float a = sc[n][e] * scale_log2, b = sc[n][2 + e] * scale_log2;
         if (need_mask) {
-          if (col > qrow0 || col >= kv_end) a = -INFINITY;
-          if (col > qrow1 || col >= kv_end) b = -INFINITY;
+          if (col > qrow0 || col >= kv_end || qrow0 - col >= win) a = -INFINITY;
+          if (col > qrow1 || col >= kv_end || qrow1 - col >= win) b = -INFINITY;
         }
         sc[n][e] = a;
         sc[n][2 + e] = b;
@@ -208,25 +211,45 @@ prefill_attn_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_cache
   l0 += __shfl_xor_sync(0xffffffffu, l0, 2);
   l1 += __shfl_xor_sync(0xffffffffu, l1, 1);
   l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
+  if (opt.sink != nullptr) {                                 // one more term of the denominator, without a value
+    const float sk = opt.sink[h] * 1.4426950408889634f;
+    if (m0 != -INFINITY) l0 += exp2f(sk - m0);
+    if (m1 != -INFINITY) l1 += exp2f(sk - m1);
+  }
   const float inv0 = l0 > 0.f ? 1.f / l0 : 0.f, inv1 = l1 > 0.f ? 1.f / l1 : 0.f;
   const int r0 = q0 + warp * 16 + g, r1 = r0 + 8;
 #pragma unroll
   for (int j = 0; j < D / 8; ++j) {
     const int c = j * 8 + 2 * t;
-    if (r0 < q_len)
-      *reinterpret_cast<uint32_t*>(out + ((long long)(q_begin + r0) * Hq + h) * D + c) =
-          pack_bf16(o[j][0] * inv0, o[j][1] * inv0);
-    if (r1 < q_len)
-      *reinterpret_cast<uint32_t*>(out + ((long long)(q_begin + r1) * Hq + h) * D + c) =
-          pack_bf16(o[j][2] * inv1, o[j][3] * inv1);
+    auto put = [&](int r, float a, float b) {
+      if (r >= q_len || c >= opt.dim) return;
+      bf16* dst = out + (q_begin + r) * opt.ld_out + h * opt.dim + c;
+      if (opt.gate != nullptr) {
+        const bf16* gate = reinterpret_cast<const bf16*>(opt.gate) + (q_begin + r) * opt.ld_gate + h * opt.dim + c;
+        a *= __fdividef(1.f, 1.f + __expf(-__bfloat162float(gate[0])));
+        if (c + 1 < opt.dim) b *= __fdividef(1.f, 1.f + __expf(-__bfloat162float(gate[1])));
+      }
+      if ((opt.dim & 1) == 0) {
+        *reinterpret_cast<uint32_t*>(dst) = pack_bf16(a, b);
+      } else {
+        dst[0] = __float2bfloat16(a);
+        if (c + 1 < opt.dim) dst[1] = __float2bfloat16(b);
+      }
+    };
+    put(r0, o[j][0] * inv0, o[j][1] * inv0);
+    put(r1, o[j][2] * inv1, o[j][3] * inv1);
   }
 }
 
 void launch_prefill_attention(const void* q, const void* k_cache, const void* v_cache, const int* block_tables,
                               const int* cu_seqlens_q, const int* kv_lens, void* out, int num_seqs, int max_q_len,
                               int Hq, int Hkv, int D, int block_size, int max_blocks, int num_blocks, float scale,
-                              uint32_t* status, cudaStream_t stream) {
+                              uint32_t* status, cudaStream_t stream, const AttnOptions* options) {
   if (num_seqs == 0 || max_q_len == 0) return;
+  AttnOptions opt;
+  if (options != nullptr) opt = *options;
+  if (opt.dim == 0) opt.dim = D;
+  if (opt.ld_out == 0) opt.ld_out = (long long)Hq * opt.dim;
   if (Hq % Hkv != 0) throw std::runtime_error("prefill attention: Hq must be a multiple of Hkv");
   const float scale_log2 = scale * 1.4426950408889634f;
   dim3 grid((max_q_len + PF_BM - 1) / PF_BM, Hq, num_seqs);
@@ -236,7 +259,7 @@ void launch_prefill_attention(const void* q, const void* k_cache, const void* v_
     cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     kern<<<grid, PF_THREADS, smem, stream>>>((const bf16*)q, (const bf16*)k_cache, (const bf16*)v_cache,
                                              block_tables, cu_seqlens_q, kv_lens, (bf16*)out, Hq, Hkv, block_size,
-                                             max_blocks, num_blocks, scale_log2, status);
+                                             max_blocks, num_blocks, scale_log2, status, opt);
   };
   if (D == 128) launch(prefill_attn_kernel<128>);
   else if (D == 64) launch(prefill_attn_kernel<64>);

@@ -1,4 +1,4 @@
-// Causal prefill attention on tcgen05, head_dim 128: two query tiles per CTA in ping-pong.
+// Causal prefill attention on tcgen05, head_dim 64 or 128: two query tiles per CTA in ping-pong.
 //
 // One CTA owns 256 query rows of one head (tiles A and B of 128 rows) and walks the visible keys
 // in tiles of 128 rows.  All accumulators live in tensor memory (512 columns):
@@ -15,6 +15,8 @@
 //                back as P.  O is rescaled only when a row maximum grows by more than 2^8 over the
 //                reference (all lanes of the warp then rescale their O row in tensor memory), so
 //                most tiles never touch O; the reference maximum cancels in O / l at the end.
+// Options (AttnOptions): a sliding window (key tiles before the first query's window are skipped), a sink per head, heads
+// narrower than the pool's rows, an output gate.
 #include <cuda.h>
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
@@ -33,10 +35,8 @@ using bf16 = __nv_bfloat16;
 
 constexpr int P2_BM = 128;             // rows per query tile (two tiles per CTA)
 constexpr int P2_BN = 128;
-constexpr int P2_D = 128;
 constexpr int P2_THREADS = 320;
-constexpr int P2_TILE_BYTES = P2_BN * P2_D * 2;        // 32 KiB: two [128 x 64] sub-tiles
-constexpr int P2_SUB_BYTES = P2_TILE_BYTES / 2;
+constexpr int P2_SUB_BYTES = P2_BN * 64 * 2;           // a [128 x 64] sub-tile; D / 64 of them make a tile
 constexpr float P2_RESCALE_THRESHOLD = 8.f;            // log2 units
 
 __device__ __forceinline__ uint64_t p2_sdesc(uint32_t addr, uint32_t lbo_bytes, uint32_t sbo_bytes) {
@@ -57,11 +57,14 @@ struct PrefillTc2Params {
   int Hq, Hkv, block_size, box_rows, max_blocks, num_blocks;
   float scale_log2;
   uint32_t* status;
+  AttnOptions opt;
 };
 
+template <int D>
 __global__ void __launch_bounds__(P2_THREADS, 1)
 prefill_attn_tc2_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_k,
                         const __grid_constant__ CUtensorMap tm_v, const PrefillTc2Params p) {
+  constexpr int SUBS = D / 64, P2_TILE_BYTES = SUBS * P2_SUB_BYTES;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   uint8_t* s_q = smem;                                   // 2 tiles
@@ -91,8 +94,10 @@ prefill_attn_tc2_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
   // keys visible to each query tile, in tiles of 128
   const int kv_end_a = min(kv_len, offset + q0 + P2_BM);
   const int kv_end_b = act_b ? min(kv_len, offset + q0 + 2 * P2_BM) : 0;
-  const int n_a = (kv_end_a + P2_BN - 1) / P2_BN;
-  const int n_b = (kv_end_b + P2_BN - 1) / P2_BN;
+  const int win = p.opt.window > 0 ? p.opt.window : 0x40000000;       // visible: row - key < win
+  const int tile0 = max(0, offset + q0 - win + 1) / P2_BN;            // tiles before it are out of every row's window
+  const int n_a = (kv_end_a + P2_BN - 1) / P2_BN - tile0;
+  const int n_b = act_b ? (kv_end_b + P2_BN - 1) / P2_BN - tile0 : 0;
   const int n_tiles = max(n_a, n_b);
   const int kv_end = max(kv_end_a, kv_end_b);
   const int* bt = p.block_tables + (long long)seq * p.max_blocks;
@@ -132,17 +137,18 @@ prefill_attn_tc2_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
     if (lane == 0) {
       mbar_expect_tx(q_full, (act_b ? 2 : 1) * P2_TILE_BYTES);
       for (int x = 0; x < (act_b ? 2 : 1); ++x) {
-        tma_load_2d(s_q + x * P2_TILE_BYTES, &tm_q, q_full, h * P2_D, q_begin + q0 + x * P2_BM);
-        tma_load_2d(s_q + x * P2_TILE_BYTES + P2_SUB_BYTES, &tm_q, q_full, h * P2_D + 64, q_begin + q0 + x * P2_BM);
+#pragma unroll
+        for (int s = 0; s < SUBS; ++s)
+          tma_load_2d(s_q + x * P2_TILE_BYTES + s * P2_SUB_BYTES, &tm_q, q_full, h * D + s * 64, q_begin + q0 + x * P2_BM);
       }
       const int pieces = P2_BN / p.box_rows;
       for (int j = 0; j < n_tiles && !*s_abort; ++j) {
         const int st = j & 1;
         const uint32_t ph = ((j >> 1) & 1) ^ 1;
-        const int row0 = j * P2_BN;
+        const int row0 = (tile0 + j) * P2_BN;
         uint32_t bytes = 0;
         for (int pc = 0; pc < pieces; ++pc)
-          if (row0 + pc * p.box_rows < kv_end) bytes += uint32_t(2 * p.box_rows * 128);
+          if (row0 + pc * p.box_rows < kv_end) bytes += uint32_t(SUBS * p.box_rows * 128);
         for (int which = 0; which < 2; ++which) {
           uint64_t* full = which == 0 ? &k_full[st] : &v_full[st];
           uint64_t* empty = which == 0 ? &k_empty[st] : &v_empty[st];
@@ -162,8 +168,9 @@ prefill_attn_tc2_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
             }
             const int grow = (blk * p.Hkv + hk) * p.block_size + tok % p.block_size;
             const CUtensorMap* tm = which == 0 ? &tm_k : &tm_v;
-            tma_load_2d(dst + pc * p.box_rows * 128, tm, full, 0, grow);
-            tma_load_2d(dst + P2_SUB_BYTES + pc * p.box_rows * 128, tm, full, 64, grow);
+#pragma unroll
+            for (int s = 0; s < SUBS; ++s)
+              tma_load_2d(dst + s * P2_SUB_BYTES + pc * p.box_rows * 128, tm, full, s * 64, grow);
           }
         }
       }
@@ -172,14 +179,14 @@ prefill_attn_tc2_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
     // ------------------------------------------------------------------ MMA issuer
     if (lane == 0) {
       constexpr uint32_t idesc_s = make_idesc_bf16(128, 128, false, false);
-      constexpr uint32_t idesc_o = make_idesc_bf16(128, 128, false, true);    // B (= V) is MN-major
+      constexpr uint32_t idesc_o = make_idesc_bf16(128, D, false, true);      // B (= V) is MN-major
       bool ok = mbar_wait(q_full, 0, p.status, ST_TIMEOUT_FULL);
       // S_x(j) = Q_x K(j)^T into tensor-memory columns [x * 128, x * 128 + 128)
       auto issue_s = [&](int x, int j) {
         const int st = j & 1;
         const uint32_t qa = smem_u32(s_q + x * P2_TILE_BYTES), ka = smem_u32(s_k + st * P2_TILE_BYTES);
 #pragma unroll
-        for (int kk = 0; kk < 8; ++kk) {
+        for (int kk = 0; kk < D / 16; ++kk) {
           const uint32_t off = uint32_t(kk >> 2) * P2_SUB_BYTES + uint32_t(kk & 3) * 32;
           tc_mma_f16(tmem_base + uint32_t(x * 128), p2_sdesc(qa + off, 16, 1024), p2_sdesc(ka + off, 16, 1024),
                      idesc_s, kk > 0 ? 1u : 0u);
@@ -248,7 +255,7 @@ prefill_attn_tc2_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
     const uint32_t to = tmem_base + lane_addr + 256u + uint32_t(x * 128);    // O_x
     const int qrow = q0 + x * P2_BM + row;                   // row among the sequence's new tokens
     const int qpos = offset + qrow;                          // last key position this row may see
-    float m_ref = 0.f, l = 0.f;
+    float m_ref = -INFINITY, l = 0.f;                        // -inf: no visible key yet
     bool ok = true;
     for (int j = 0; j < n_x && ok; ++j) {
       if (*s_abort || !mbar_wait(&s_full[x], uint32_t(j) & 1u, p.status, ST_TIMEOUT_ACC_FULL)) {
@@ -260,21 +267,21 @@ prefill_attn_tc2_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
 #pragma unroll
       for (int c = 0; c < 4; ++c) tmem_ld_32x32(ts + uint32_t(c * 32), *reinterpret_cast<uint32_t(*)[32]>(&s[c * 32]));
       tmem_ld_wait();
-      const int col0 = j * P2_BN;
-      const bool need_mask = (col0 + P2_BN - 1 > offset + q0 + x * P2_BM) || (col0 + P2_BN > kv_end_x);
+      const int col0 = (tile0 + j) * P2_BN;
+      const bool need_mask = (col0 + P2_BN - 1 > offset + q0 + x * P2_BM) || (col0 + P2_BN > kv_end_x) ||
+                             (offset + q0 + x * P2_BM + P2_BM - 1 - col0 >= win);
       if (need_mask) {
+        const int hi = min(qpos, kv_end_x - 1) - col0, lo = qpos - win + 1 - col0;     // visible columns of the tile
 #pragma unroll
-        for (int t = 0; t < 128; ++t) {
-          const int col = col0 + t;
-          if (col > qpos || col >= kv_end_x) s[t] = 0xff800000u;          // -inf
-        }
+        for (int t = 0; t < 128; ++t)
+          if (t > hi || t < lo) s[t] = 0xff800000u;                                     // -inf
       }
       float mx = -INFINITY;
 #pragma unroll
       for (int t = 0; t < 128; ++t) mx = fmaxf(mx, __uint_as_float(s[t]));
       mx *= p.scale_log2;
       if (j == 0) {
-        m_ref = (mx == -INFINITY) ? 0.f : mx;
+        m_ref = mx;
       } else if (__any_sync(__activemask(), mx > m_ref + P2_RESCALE_THRESHOLD)) {
         // some row of this warp outgrew its reference: bring O (complete up to tile j - 1) to the new one
         if (!mbar_wait(&o_done[x], uint32_t(j - 1) & 1u, p.status, ST_TIMEOUT_ACC_FULL)) {
@@ -283,11 +290,11 @@ prefill_attn_tc2_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
         }
         tc_fence_after();
         const float m_new = fmaxf(m_ref, mx);
-        const float f = exp2f(m_ref - m_new);
+        const float f = m_ref == -INFINITY ? 0.f : exp2f(m_ref - m_new);
         m_ref = m_new;
         l *= f;
 #pragma unroll 1
-        for (int c = 0; c < 4; ++c) {
+        for (int c = 0; c < D / 32; ++c) {
           uint32_t r[32];
           tmem_ld_32x32(to + uint32_t(c * 32), r);
           tmem_ld_wait();
@@ -297,13 +304,14 @@ prefill_attn_tc2_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
         }
         tmem_st_wait();
       }
+      const float base = m_ref == -INFINITY ? 0.f : m_ref;
       float rs = 0.f;
       uint32_t u[64];
 #pragma unroll
       for (int t = 0; t < 64; ++t) {
         float e0, e1;
-        const float a0 = fmaf(__uint_as_float(s[2 * t]), p.scale_log2, -m_ref);
-        const float a1 = fmaf(__uint_as_float(s[2 * t + 1]), p.scale_log2, -m_ref);
+        const float a0 = fmaf(__uint_as_float(s[2 * t]), p.scale_log2, -base);
+        const float a1 = fmaf(__uint_as_float(s[2 * t + 1]), p.scale_log2, -base);
         asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e0) : "f"(a0));
         asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e1) : "f"(a1));
         rs += e0 + e1;
@@ -319,24 +327,49 @@ prefill_attn_tc2_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
     if (!ok) *s_abort = 1;
     if (ok && n_x > 0 && mbar_wait(&o_done[x], uint32_t(n_x - 1) & 1u, p.status, ST_TIMEOUT_ACC_FULL)) {
       tc_fence_after();
+      if (p.opt.sink != nullptr && m_ref != -INFINITY)       // one more term of the denominator, without a value
+        l += exp2f(p.opt.sink[h] * 1.4426950408889634f - m_ref);
       const float inv = l > 0.f ? 1.f / l : 0.f;
-      bf16* dst = p.out + ((long long)(q_begin + qrow) * p.Hq + h) * P2_D;
+      const int dim = p.opt.dim;
+      bf16* dst = p.out + (q_begin + qrow) * p.opt.ld_out + h * dim;
+      const bf16* gate = p.opt.gate == nullptr ? nullptr
+          : reinterpret_cast<const bf16*>(p.opt.gate) + (q_begin + qrow) * p.opt.ld_gate + h * dim;
 #pragma unroll 1
-      for (int c = 0; c < 4; ++c) {
+      for (int c = 0; c < D / 32; ++c) {
         uint32_t r[32];
         tmem_ld_32x32(to + uint32_t(c * 32), r);
         tmem_ld_wait();
-        if (qrow < q_len) {
+        if (qrow < q_len && (dim & 7) == 0) {
 #pragma unroll
           for (int q = 0; q < 4; ++q) {
-            uint4 v;
-            v.x = pack_bf16(__uint_as_float(r[q * 8 + 0]) * inv, __uint_as_float(r[q * 8 + 1]) * inv);
-            v.y = pack_bf16(__uint_as_float(r[q * 8 + 2]) * inv, __uint_as_float(r[q * 8 + 3]) * inv);
-            v.z = pack_bf16(__uint_as_float(r[q * 8 + 4]) * inv, __uint_as_float(r[q * 8 + 5]) * inv);
-            v.w = pack_bf16(__uint_as_float(r[q * 8 + 6]) * inv, __uint_as_float(r[q * 8 + 7]) * inv);
-            reinterpret_cast<uint4*>(dst + c * 32)[q] = v;
+            const int col = c * 32 + q * 8;
+            if (col >= dim) continue;
+            float v[8];
+#pragma unroll
+            for (int e = 0; e < 8; ++e) v[e] = __uint_as_float(r[q * 8 + e]) * inv;
+            if (gate != nullptr) {
+              const uint4 gu = *reinterpret_cast<const uint4*>(gate + col);
+              const uint32_t gw[4] = {gu.x, gu.y, gu.z, gu.w};
+#pragma unroll
+              for (int e = 0; e < 4; ++e) {
+                const float2 g = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&gw[e]));
+                v[2 * e] *= __fdividef(1.f, 1.f + __expf(-g.x));
+                v[2 * e + 1] *= __fdividef(1.f, 1.f + __expf(-g.y));
+              }
+            }
+            *reinterpret_cast<uint4*>(dst + col) = make_uint4(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]),
+                                                              pack_bf16(v[4], v[5]), pack_bf16(v[6], v[7]));
+          }
+        } else if (qrow < q_len) {
+#pragma unroll
+          for (int t = 0; t < 32; ++t) {
+            if (c * 32 + t >= dim) continue;
+            float v = __uint_as_float(r[t]) * inv;
+            if (gate != nullptr) v *= __fdividef(1.f, 1.f + __expf(-__bfloat162float(gate[c * 32 + t])));
+            dst[c * 32 + t] = __float2bfloat16(v);
           }
         }
+        __syncwarp();                                        // the next tensor-memory load is a warp instruction
       }
     }
   }
@@ -348,15 +381,32 @@ prefill_attn_tc2_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
   }
 }
 
+template <int D>
+static void launch_tc2(const void* q, const void* k_cache, const void* v_cache, const PrefillTc2Params& p,
+                       long long total_q, int num_seqs, int max_q_len, cudaStream_t stream) {
+  const CUtensorMap tq = make_tmap_bf16_2d(q, (uint64_t)total_q, (uint64_t)p.Hq * D, (uint64_t)p.Hq * D, P2_BM, 64);
+  const uint64_t rows = (uint64_t)p.num_blocks * p.Hkv * p.block_size;
+  const CUtensorMap tk = make_tmap_bf16_2d(k_cache, rows, D, D, p.box_rows, 64);
+  const CUtensorMap tv = make_tmap_bf16_2d(v_cache, rows, D, D, p.box_rows, 64);
+  const int smem = 6 * (D / 64) * P2_SUB_BYTES + 256 + 1024;
+  cudaFuncSetAttribute(prefill_attn_tc2_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+  dim3 grid((max_q_len + 2 * P2_BM - 1) / (2 * P2_BM), p.Hq, num_seqs);
+  prefill_attn_tc2_kernel<D><<<grid, P2_THREADS, smem, stream>>>(tq, tk, tv, p);
+}
+
+bool prefill_attention_tc2_supported(int D, int block_size) { return (D == 64 || D == 128) && block_size % 8 == 0; }
+
 void launch_prefill_attention_tc2(const void* q, const void* k_cache, const void* v_cache, const int* block_tables,
                                   const int* cu_seqlens_q, const int* kv_lens, void* out, long long total_q,
-                                  int num_seqs, int max_q_len, int Hq, int Hkv, int block_size, int max_blocks,
-                                  int num_blocks, float scale, uint32_t* status, cudaStream_t stream) {
+                                  int num_seqs, int max_q_len, int Hq, int Hkv, int D, int block_size, int max_blocks,
+                                  int num_blocks, float scale, uint32_t* status, cudaStream_t stream,
+                                  const AttnOptions* options) {
   if (num_seqs == 0 || max_q_len == 0) return;
   if (Hq % Hkv != 0) throw std::runtime_error("prefill attention: Hq must be a multiple of Hkv");
+  if (!prefill_attention_tc2_supported(D, block_size))
+    throw std::runtime_error("prefill attention on tcgen05: head_dim 64 or 128 and a block_size that is a multiple of 8");
   int box_rows = P2_BN;
   while (box_rows > block_size || block_size % box_rows != 0) box_rows >>= 1;
-  if (box_rows < 8) throw std::runtime_error("prefill attention: block_size must be a multiple of 8");
   PrefillTc2Params p{};
   p.block_tables = block_tables;
   p.cu_q = cu_seqlens_q;
@@ -370,14 +420,11 @@ void launch_prefill_attention_tc2(const void* q, const void* k_cache, const void
   p.num_blocks = num_blocks;
   p.scale_log2 = scale * 1.4426950408889634f;
   p.status = status;
-  const CUtensorMap tq = make_tmap_bf16_2d(q, (uint64_t)total_q, (uint64_t)Hq * P2_D, (uint64_t)Hq * P2_D, P2_BM, 64);
-  const uint64_t rows = (uint64_t)num_blocks * Hkv * block_size;
-  const CUtensorMap tk = make_tmap_bf16_2d(k_cache, rows, P2_D, P2_D, box_rows, 64);
-  const CUtensorMap tv = make_tmap_bf16_2d(v_cache, rows, P2_D, P2_D, box_rows, 64);
-  const int smem = 6 * P2_TILE_BYTES + 256 + 1024;
-  cudaFuncSetAttribute(prefill_attn_tc2_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
-  dim3 grid((max_q_len + 2 * P2_BM - 1) / (2 * P2_BM), Hq, num_seqs);
-  prefill_attn_tc2_kernel<<<grid, P2_THREADS, smem, stream>>>(tq, tk, tv, p);
+  if (options != nullptr) p.opt = *options;
+  if (p.opt.dim == 0) p.opt.dim = D;
+  if (p.opt.ld_out == 0) p.opt.ld_out = (long long)Hq * p.opt.dim;
+  if (D == 128) launch_tc2<128>(q, k_cache, v_cache, p, total_q, num_seqs, max_q_len, stream);
+  else launch_tc2<64>(q, k_cache, v_cache, p, total_q, num_seqs, max_q_len, stream);
   cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess) throw std::runtime_error(std::string("prefill attention (tcgen05, 2 tiles) launch: ") + cudaGetErrorString(e));
 }

@@ -26,26 +26,38 @@ void launch_sample(const void* logits, const void* temps, void* out, int B, int 
                    cudaStream_t s, int vocab_offset = 0, int v_limit = -1, const uint32_t* status = nullptr,
                    bool f32 = false);     // f32: fp32 logits instead of bf16
 
+// Options of the paged attention kernels; the defaults are plain causal attention.
+struct AttnOptions {
+  int window = 0;                  // positions a query sees, itself included (0: all up to itself)
+  const float* sink = nullptr;     // [Hq] fp32: exp(sink) joins the denominator, without key or value
+  int dim = 0;                     // columns of a head that are written (0: all); the pool's rows may be wider
+  const void* gate = nullptr;      // bf16 [rows, ld_gate]: the output is multiplied by sigmoid(gate)
+  long long ld_gate = 0, ld_out = 0;   // row pitches in elements (ld_out 0: Hq * dim)
+};
+
 int decode_attn_pick_splits(int B, int Hkv, int max_ctx, int num_sms);
 void launch_decode_attention(const void* q, const void* k_cache, const void* v_cache, const int* block_tables,
                              const int* context_lens, void* out, float* part_o, float* part_lse, int B, int Hq,
                              int Hkv, int D, int block_size, int max_blocks, int num_blocks, int splits,
-                             float scale, uint32_t* status, cudaStream_t stream, int* merge_counters = nullptr);
+                             float scale, uint32_t* status, cudaStream_t stream, int* merge_counters = nullptr,
+                             const AttnOptions* options = nullptr);
 void launch_prefill_attention(const void* q, const void* k_cache, const void* v_cache, const int* block_tables,
                               const int* cu_seqlens_q, const int* kv_lens, void* out, int num_seqs, int max_q_len,
                               int Hq, int Hkv, int D, int block_size, int max_blocks, int num_blocks, float scale,
-                              uint32_t* status, cudaStream_t stream);
+                              uint32_t* status, cudaStream_t stream, const AttnOptions* options = nullptr);
 // tcgen05 version (head_dim 128, block_size a multiple of 8)
 bool prefill_attention_tc_supported(int D, int block_size);
 void launch_prefill_attention_tc(const void* q, const void* k_cache, const void* v_cache, const int* block_tables,
                                  const int* cu_seqlens_q, const int* kv_lens, void* out, long long total_q,
                                  int num_seqs, int max_q_len, int Hq, int Hkv, int block_size, int max_blocks,
                                  int num_blocks, float scale, uint32_t* status, cudaStream_t stream);
-// two query tiles per CTA in ping-pong, P and O in tensor memory (same limits)
+// two query tiles per CTA in ping-pong, P and O in tensor memory (head_dim 64 or 128, block_size a multiple of 8)
+bool prefill_attention_tc2_supported(int D, int block_size);
 void launch_prefill_attention_tc2(const void* q, const void* k_cache, const void* v_cache, const int* block_tables,
                                   const int* cu_seqlens_q, const int* kv_lens, void* out, long long total_q,
-                                  int num_seqs, int max_q_len, int Hq, int Hkv, int block_size, int max_blocks,
-                                  int num_blocks, float scale, uint32_t* status, cudaStream_t stream);
+                                  int num_seqs, int max_q_len, int Hq, int Hkv, int D, int block_size, int max_blocks,
+                                  int num_blocks, float scale, uint32_t* status, cudaStream_t stream,
+                                  const AttnOptions* options = nullptr);
 }  // namespace fc
 
 namespace fc {
