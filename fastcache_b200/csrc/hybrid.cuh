@@ -25,7 +25,7 @@ struct Elem<__nv_bfloat16> {
 // one element of a projection output
 template <typename T>
 __device__ __forceinline__ float proj_at(const ProjSrc& s, long long row, int col) {
-  if (s.splits > 1) {
+  if (s.part != nullptr) {
     float v = 0.f;
     const float* p = s.part + row * s.part_ld + col;
     for (int i = 0; i < s.splits; ++i) v += __ldcg(p + i * s.part_stride);
@@ -37,7 +37,7 @@ __device__ __forceinline__ float proj_at(const ProjSrc& s, long long row, int co
 // four consecutive elements; `col` and the pitches are multiples of 4
 template <typename T>
 __device__ __forceinline__ float4 proj_at4(const ProjSrc& s, long long row, int col) {
-  if (s.splits > 1) {
+  if (s.part != nullptr) {
     float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
     const float* p = s.part + row * s.part_ld + col;
 #pragma unroll 4
@@ -76,7 +76,7 @@ __device__ __forceinline__ void store4(T* dst, float a, float b, float c, float 
 // eight consecutive elements; `col` and the pitches are multiples of 8
 template <typename T>
 __device__ __forceinline__ void proj_at8(const ProjSrc& s, long long row, int col, float (&v)[8]) {
-  if (sizeof(T) == 2 && s.splits <= 1) {
+  if (sizeof(T) == 2 && s.part == nullptr) {
     const uint4 u = __ldcg(reinterpret_cast<const uint4*>(reinterpret_cast<const T*>(s.p) + row * s.ld + col));
     const uint32_t w[4] = {u.x, u.y, u.z, u.w};
 #pragma unroll
@@ -120,6 +120,21 @@ __device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.f) + lo
 template <typename T>
 __device__ __forceinline__ float gelu_tanh_t(float z) {
   return over_one_plus_exp<T>(z, -1.5957691216057308f * (z + 0.044715f * z * z * z));
+}
+
+// gated activations (GluKind)
+template <typename T, int KIND>
+__device__ __forceinline__ float glu_t(float g, float u, float limit) {
+  if (KIND == GLU_ACT_SILU) return silu_t<T>(g) * u;
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit);
+  return over_one_plus_exp<T>(g, -1.702f * g) * (u + 1.f);
+}
+
+// cos and sin of position * base^(-2 i / dims): the angle is reduced in double, so that far positions lose nothing
+__device__ __forceinline__ void rope_angle(double pos, double log2_base, int i, int dims, float& c, float& s) {
+  const double turns = pos * exp2(-log2_base * (2.0 * i / dims)) * 0.15915494309189535;   // 1 / (2 pi)
+  sincospif(float(2.0 * (turns - rint(turns))), &s, &c);
 }
 
 struct Run {

@@ -1,6 +1,7 @@
-// Launchers of the hybrid-model kernels: sublayer-output norm on an fp32 residual stream (resid.cu), recurrent
-// layers (recurrence.cu, recurrence_chunk.cu), latent attention (latent.cu, latent_decode.cu, latent_prefill.cu) and
-// the CUDA-core GEMM of 32-bit runs (linear_simt.cu).
+// Launchers of the hybrid-model kernels: norms on an fp32 residual stream and gated activations (resid.cu), recurrent
+// layers (recurrence.cu, recurrence_chunk.cu), latent attention (latent.cu, latent_decode.cu, latent_prefill.cu),
+// windowed attention (window_attn.cu, with the attn_*.cu kernels), experts (moe.cu, moe_gemm.cu) and the CUDA-core GEMM of
+// 32-bit runs (linear_simt.cu).
 //
 // `f32` selects the element type of activations and weights (fp32 or bf16); everything accumulates in fp32.
 #pragma once
@@ -9,12 +10,12 @@
 
 namespace fc {
 
-// Output of a projection: a finished matrix (element type of the model) or fp32 split-K partial sums that the reader
-// adds up.  row pitches in elements.
+// Output of a projection: a finished matrix (element type of the model) or, with `part`, fp32 split-K partial sums that
+// the reader adds up.  row pitches in elements.
 struct ProjSrc {
   const void* p = nullptr;
   long long ld = 0;
-  const float* part = nullptr;      // [splits, rows, part_ld] when splits > 1
+  const float* part = nullptr;      // [splits, rows, part_ld]
   int splits = 1;
   long long part_stride = 0;
   long long part_ld = 0;
@@ -39,6 +40,7 @@ struct SimtLinear {
   long long gx = 0, gw = 0, gy = 0;           // offsets between groups
   ProjSrc gate;                               // p == part == nullptr: no gate
   int gate_off = 0;
+  const int* group_rows = nullptr;            // [groups + 1]: group g has the rows [g, g + 1) of x and y (gx, gy unused)
   int y_pad = 0;                              // columns [groups * N, y_pad) of y are zeroed (groups stored side by side)
 };
 void launch_linear_simt(const SimtLinear& a, bool f32, cudaStream_t s);
@@ -53,6 +55,34 @@ void launch_post_norm_add(const ProjSrc& y, const void* bias, float* x, const fl
                           float eps, bool f32, cudaStream_t s);
 void launch_rms_norm_wide(const float* x, const float* w, void* h, int T, int W, int Wp, float eps, bool f32,
                           cudaStream_t s);
+// x (+)= y + sum_j mix_j experts[row_of_j] in fp32; h = rms(x) * w, or x itself without w
+struct AddNorm {
+  int T = 0, W = 0, Wp = 0;
+  const ProjSrc* y = nullptr;        // nullptr: x holds the sum already
+  bool add = true;                   // false: x is replaced
+  float* x = nullptr;                // [T, W]
+  const float* w = nullptr;
+  void* h = nullptr;                 // [T, ld_h], columns [W, Wp) are zeroed
+  long long ld_h = 0;
+  float eps = 0.f;
+  ProjSrc experts;
+  const int* row_of = nullptr;       // [T, top] rows of `experts` (-1: none); nullptr: no experts
+  const float* mix = nullptr;        // [T, top]; nullptr: 1 / top each
+  int top = 0;
+};
+void launch_add_norm(const AddNorm& p, bool f32, cudaStream_t s);
+// gated activations; CLAMPED: g sigmoid(1.702 g) (u + 1), g = min(gate, limit), u = up clamped to +-limit
+enum GluKind : int { GLU_ACT_SILU = 0, GLU_ACT_CLAMPED = 1 };
+struct GluMul {
+  int T = 0, width = 0, width_p = 0; // columns [width, width_p) of the output are zeroed
+  ProjSrc p;
+  int off_gate = 0, off_up = 0;
+  int kind = 0;
+  float limit = 0.f;
+  void* out = nullptr;
+  long long ld_out = 0;
+};
+void launch_glu_mul(const GluMul& p, bool f32, cudaStream_t s);
 void launch_gelu_mul(const ProjSrc& gu, const void* bias, void* out, int T, int up_off, int width, int width_p,
                      bool f32, cudaStream_t s);
 
@@ -77,19 +107,32 @@ struct StepParams {
   const float* log_g = nullptr;      // [T, H]
   const float* beta = nullptr;       // [T, H]
   uint8_t* scratch = nullptr;        // chunked form: chunk_scratch_bytes()
+  // matrix memory
+  float* nstate = nullptr;           // [slots, H, D] normaliser
+  float* mstate = nullptr;           // [slots, H] running maximum of the log gates
+  ProjSrc gates;                     // fp32 (or the 32-bit model's) gate projections
+  int off_i = 0, off_f = 0;
+  const float *i_bias = nullptr, *f_bias = nullptr;   // [H]
+  float cap = 1.f, floor = 0.f;
+  float *log_i = nullptr, *log_f = nullptr, *m_t = nullptr;   // [T, H] from launch_memory_gates (nullptr: the step kernel
+  float* m_0 = nullptr;                                       // makes its own gates); m_0 [B, H]: maximum before the run
+  float* den = nullptr;              // [T, H] raw normaliser n.q beside o_raw
   // output: `out` with the head norm and gate applied, or raw fp32 head outputs in `o_raw`
   float* o_raw = nullptr;            // [T, H * V]
   void* out = nullptr;
-  long long ld_out = 0;              // padded width of `out`; the pad is zeroed
-  const float* norm_w = nullptr;
+  long long ld_out = 0;              // row pitch of `out`
+  int pad_out = 0;                   // columns after H * V that are zeroed
+  const float* norm_w = nullptr;     // [V], matrix memory [H * V]
   float eps = 0.f;
 };
 // true: the step kernel writes `out` itself (one CTA holds a whole head)
 bool step_fuses_norm(int D, int V);
 void launch_gla_step(const StepParams& p, bool f32, cudaStream_t s);
 void launch_delta_step(const StepParams& p, bool f32, cudaStream_t s);
-void launch_gated_head_norm(const float* o_raw, const ProjSrc& proj, int off_g, const float* norm_w, float eps,
-                            void* out, long long ld_out, int T, int H, int V, bool f32, cudaStream_t s);
+void launch_memory_step(const StepParams& p, bool f32, cudaStream_t s);
+void launch_memory_gates(const StepParams& p, cudaStream_t s);
+// head norm and gate (silu; matrix memory: division by the normaliser first, gate sigmoid) of o_raw
+void launch_gated_head_norm(const StepParams& p, int T, bool memory, bool f32, cudaStream_t s);
 
 struct DeltaPrepare {
   int H = 0, K = 0, D = 0, V = 0, taps = 1, T = 0;
@@ -108,10 +151,12 @@ struct DeltaPrepare {
 void launch_delta_prepare(const DeltaPrepare& p, bool f32, cudaStream_t s);
 
 // ---- recurrence_chunk.cu (bf16 runs of many rows): o_raw [T, H * V] and the state after every run
+enum Recurrence : int { REC_GLA = 0, REC_DELTA = 1, REC_MEMORY = 2 };
 bool chunk_supported(int D, int V);
-long long chunk_scratch_bytes(const StepParams& p, int T, bool delta);
+long long chunk_scratch_bytes(const StepParams& p, int T, int kind);
 void launch_gla_chunk(const StepParams& p, int max_len, cudaStream_t s);
 void launch_delta_chunk(const StepParams& p, int max_len, cudaStream_t s);
+void launch_memory_chunk(const StepParams& p, int max_len, cudaStream_t s);
 
 // ---- latent.cu
 struct LatentStore {
@@ -182,5 +227,68 @@ struct LatentPrefill {
 };
 bool latent_prefill_supported(const LatentPrefill& p);
 void launch_latent_prefill(const LatentPrefill& p, cudaStream_t s);
+
+// ---- window_attn.cu: what surrounds attention over per-head K/V rows whose values are the raw keys
+struct WindowStore {
+  int T = 0, H = 0, G = 0, D = 0, pitch = 0, rot_dims = 0;     // pitch: row width of q and of the pools (>= D, zero-padded)
+  ProjSrc proj;
+  int off_q = 0, off_k = 0, off_g = 0;
+  const float *q_norm = nullptr, *k_norm = nullptr;            // over the whole projections
+  float eps = 0.f;
+  double log2_base = 0.0;
+  const long long* positions = nullptr;
+  const int* slots = nullptr;
+  void *k_rows = nullptr, *v_rows = nullptr;                   // [blocks, G, block, pitch]
+  int block_size = 0;
+  long long num_rows = 0;                                      // blocks * block
+  void* q = nullptr;                                           // [T, H, pitch]
+  void* gate = nullptr;                                        // [T, H * D] copy of the gate projection (nullptr: not wanted)
+  void* out = nullptr;                                         // attention output: columns [H * D, + pad_out) are zeroed
+  long long ld_out = 0;
+  int pad_out = 0;
+  uint32_t* status = nullptr;
+};
+void launch_window_store(const WindowStore& p, bool f32, cudaStream_t s);
+struct WindowAttn {                  // the general form: any head size, bf16 or fp32
+  int T = 0, H = 0, G = 0, D = 0, pitch = 0, window = 0, block_size = 0, max_blocks = 0, num_blocks = 0;
+  const void *q = nullptr, *k_rows = nullptr, *v_rows = nullptr;
+  const int *block_tables = nullptr, *row_seq = nullptr, *row_ctx = nullptr;      // as in LatentAttn
+  const float* sink = nullptr;
+  ProjSrc gate;
+  int off_g = 0;
+  void* out = nullptr;
+  long long ld_out = 0;
+  float scale = 1.f;
+  uint32_t* status = nullptr;
+};
+void launch_window_attn(const WindowAttn& p, bool f32, cudaStream_t s);
+
+// ---- moe.cu: tokens by expert.  plan: [E + 1] first sorted row of every expert, [1] number of 128-row tiles, then
+// (expert, first row) of every tile, then the token of every sorted row
+constexpr int MOE_TILE = 128;
+constexpr int MOE_MAX_EXPERTS = 1024;
+inline int moe_max_tiles(int pairs, int E) { return pairs / MOE_TILE + (pairs < E ? pairs : E); }
+inline long long moe_plan_size(int pairs, int E) { return E + 2 + 2ll * moe_max_tiles(pairs, E) + pairs; }
+inline int moe_token_offset(int pairs, int E) { return E + 2 + 2 * moe_max_tiles(pairs, E); }
+struct RouteTable {
+  const long long* ids = nullptr;
+  const int* table = nullptr;        // [vocab, top]
+  const int* ctx = nullptr;          // decode: rows of 0 are padding (nullptr: every row counts)
+  int T = 0, top = 0, E = 0;
+  long long vocab = 0;
+  int* row_of = nullptr;             // [T, top] sorted row, -1: none
+  int* plan = nullptr;
+  int token_at = 0;                  // (set by the launcher)
+  uint32_t* status = nullptr;
+};
+void launch_route_table(const RouteTable& p, cudaStream_t s);
+// decode-size expert products (moe_gemm.cu): partial [splits, pairs, N] of x [pairs, K] and w [E, N, K]; an expert has at
+// most max_rows <= 256 rows
+int moe_skinny_splits(int max_rows, int pairs, int E, int N, int K);
+void launch_moe_skinny(const void* x, const void* w, float* partial, int splits, const int* plan, int max_rows, int pairs,
+                       int E, int N, int K, uint32_t* status, cudaStream_t s);
+// out[r] = x[token of sorted row r]
+void launch_gather_tokens(const void* x, long long ldx, void* out, int cols, const int* plan, int pairs, int E, bool f32,
+                          cudaStream_t s);
 
 }  // namespace fc

@@ -13,12 +13,6 @@ namespace fc {
 using bf16 = __nv_bfloat16;
 constexpr int LS_THREADS = 256;
 
-// cos and sin of position * base^(-2 i / dims): the angle is reduced in double, so that far positions lose nothing
-__device__ __forceinline__ void rope_angle(double pos, double log2_base, int i, int dims, float& c, float& s) {
-  const double turns = pos * exp2(-log2_base * (2.0 * i / dims)) * 0.15915494309189535;   // 1 / (2 pi)
-  sincospif(float(2.0 * (turns - rint(turns))), &s, &c);
-}
-
 template <typename T>
 __global__ void __launch_bounds__(LS_THREADS)
 latent_store_kernel(const LatentStore p) {

@@ -16,7 +16,14 @@ __global__ void __launch_bounds__(256)
 linear_simt_kernel(const SimtLinear a) {
   __shared__ float sx[SL_K][SL_T + 4], sw[SL_K][SL_T + 4];
   const int g = blockIdx.z, m0 = blockIdx.y * SL_T, n0 = blockIdx.x * SL_T;
-  const T* x = reinterpret_cast<const T*>(a.x) + g * a.gx;
+  int M = a.M;
+  long long row0 = 0;
+  if (a.group_rows != nullptr) {
+    row0 = a.group_rows[g];
+    M = a.group_rows[g + 1] - int(row0);
+    if (m0 >= M) return;
+  }
+  const T* x = reinterpret_cast<const T*>(a.x) + (a.group_rows != nullptr ? row0 * a.ldx : g * a.gx);
   const T* w = reinterpret_cast<const T*>(a.w) + g * a.gw;
   const int tm = (threadIdx.x >> 4) * 4, tn = (threadIdx.x & 15) * 4;
   const int lr = threadIdx.x >> 2, lk = (threadIdx.x & 3) * 4;      // loader: row of the tile, first of 4 k
@@ -25,7 +32,7 @@ linear_simt_kernel(const SimtLinear a) {
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
       const int k = k0 + lk + i;
-      sx[lk + i][lr] = (m0 + lr < a.M && k < a.K) ? Elem<T>::get(x[(long long)(m0 + lr) * a.ldx + k]) : 0.f;
+      sx[lk + i][lr] = (m0 + lr < M && k < a.K) ? Elem<T>::get(x[(long long)(m0 + lr) * a.ldx + k]) : 0.f;
       sw[lk + i][lr] = (n0 + lr < a.N && k < a.K) ? Elem<T>::get(w[(long long)(n0 + lr) * a.ldw + k]) : 0.f;
     }
     __syncthreads();
@@ -41,13 +48,13 @@ linear_simt_kernel(const SimtLinear a) {
     }
     __syncthreads();
   }
-  T* y = reinterpret_cast<T*>(a.y) + g * a.gy;
+  T* y = reinterpret_cast<T*>(a.y) + (a.group_rows != nullptr ? row0 * a.ldy : g * a.gy);
   const T* bias = reinterpret_cast<const T*>(a.bias);
   const bool gated = a.gate.p != nullptr || a.gate.part != nullptr;
 #pragma unroll
   for (int i = 0; i < 4; ++i) {
     const int m = m0 + tm + i;
-    if (m >= a.M) break;
+    if (m >= M) break;
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int n = n0 + tn + j;

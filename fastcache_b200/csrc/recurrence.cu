@@ -1,4 +1,5 @@
-// Recurrent layers, token by token: gated linear attention and the gated delta rule with the state in registers.
+// Recurrent layers, token by token: gated linear attention, the gated delta rule and matrix memory (mLSTM) with the state
+// in registers.
 //
 // One CTA owns (request, head, block of value columns): its part of the fp32 state [D, V] is read from the request's
 // slot once, advanced over the rows of the request's run and written back.  A decode step is a run of one row; it is
@@ -19,12 +20,20 @@ constexpr int ST_THREADS = 256;
 constexpr int ST_WARPS = ST_THREADS / 32;
 constexpr int ST_MAX_D = 1024;
 
-template <typename T, bool DELTA, int CG, int R>
+// soft-capped log gates of matrix memory: log input gate and log(sigmoid) forget gate
+__device__ __forceinline__ float soft_cap(float x, float cap) { return cap * tanhf(x / cap); }
+__device__ __forceinline__ void memory_gates(const StepParams& p, long long t, int h, float& li, float& lf) {
+  li = soft_cap(proj_at<float>(p.gates, t, p.off_i + h) + p.i_bias[h], p.cap);
+  lf = log_sigmoid_f(soft_cap(proj_at<float>(p.gates, t, p.off_f + h) + p.f_bias[h], p.cap));
+}
+
+template <typename T, int KIND, int CG, int R>
 __global__ void __launch_bounds__(ST_THREADS)
 step_kernel(const StepParams p) {
+  constexpr bool DELTA = KIND == REC_DELTA, MEM = KIND == REC_MEMORY;
   constexpr int RG = ST_THREADS / CG;
   constexpr int VB = CG * 4;
-  constexpr int NV = DELTA ? 2 * VB + 1 : VB;               // values exchanged per warp and token
+  constexpr int NV = DELTA ? 2 * VB + 1 : MEM ? VB + 1 : VB;               // values exchanged per warp and token
   constexpr int NL = (RG * R + ST_THREADS - 1) / ST_THREADS; // staged entries per thread
   extern __shared__ float sm[];
   const int D = p.D;
@@ -46,13 +55,30 @@ step_kernel(const StepParams p) {
       for (int t = run.lo; t < run.lo + run.len; ++t)
         for (int j = 0; j < 4; ++j)
           if (col + j < p.V) {
-            if (out != nullptr) out[t * p.ld_out + h * p.V + col + j] = Elem<T>::put(0.f);
+            if (out != nullptr) out[(long long)t * p.ld_out + h * p.V + col + j] = Elem<T>::put(0.f);
             else p.o_raw[((long long)t * p.H + h) * p.V + col + j] = 0.f;
           }
+    if (MEM && out == nullptr && vb == 0)
+      for (int t = run.lo + tid; t < run.lo + run.len; t += ST_THREADS) {
+        p.den[(long long)t * p.H + h] = 0.f;
+        if (p.m_t != nullptr) p.m_t[(long long)t * p.H + h] = 0.f;
+      }
     return;
   }
   float* st = p.state + ((long long)run.slot * p.H + h) * D * p.V;
   float S[R][4];
+  float N[MEM ? R : 1];                                      // normaliser rows, in every column group
+  float m = 0.f;                                             // running maximum; starts at 0
+  if (MEM) {
+    const float* ns = p.nstate + ((long long)run.slot * p.H + h) * D;
+#pragma unroll
+    for (int i = 0; i < R; ++i) {
+      const int r = rg + i * RG;
+      N[MEM ? i : 0] = run.start > 0 && r < D ? ns[r] : 0.f;
+    }
+    if (p.m_t != nullptr) m = p.m_0[(long long)b * p.H + h];
+    else if (run.start > 0) m = p.mstate[(long long)run.slot * p.H + h];
+  }
 #pragma unroll
   for (int i = 0; i < R; ++i) {
     const int r = rg + i * RG;
@@ -83,6 +109,7 @@ step_kernel(const StepParams p) {
       } else {
         pq[i] = proj_at<T>(p.proj, t, p.off_q + h * D + r) * p.q_scale;
         pk[i] = proj_at<T>(p.proj, t, p.off_k + h * D + r);
+        if (MEM) continue;
         float z = p.z_bias[h * D + r];
         if (p.z != nullptr) {
           z += Elem<T>::get(reinterpret_cast<const T*>(p.z)[(long long)t * p.ld_z + h * D + r]);
@@ -101,7 +128,7 @@ step_kernel(const StepParams p) {
       if (r >= D) continue;
       s_q[buf * D + r] = pq[i];
       s_k[buf * D + r] = pk[i];
-      if (!DELTA) s_a[buf * D + r] = pa[i];
+      if (!DELTA && !MEM) s_a[buf * D + r] = pa[i];
     }
   };
   const int t1 = run.lo + run.len;
@@ -114,7 +141,22 @@ step_kernel(const StepParams p) {
     const int buf = n % 3;
     if (t + 1 < t1) fetch(t + 1);
     float v[4] = {0.f, 0.f, 0.f, 0.f};
-    float g = 0.f, beta = 0.f;
+    float g = 0.f, beta = 0.f;                               // matrix memory: kept and written shares
+    if (MEM) {
+      float li, lf, mt;
+      if (p.m_t != nullptr) {
+        const long long o = (long long)t * p.H + h;
+        li = __ldcg(p.log_i + o);
+        lf = __ldcg(p.log_f + o);
+        mt = __ldcg(p.m_t + o);
+      } else {
+        memory_gates(p, t, h, li, lf);
+        mt = fmaxf(lf + m, li);
+      }
+      g = expf(lf + m - mt);
+      beta = expf(li - mt);
+      m = mt;
+    }
     if (DELTA) {
       const T* vr = reinterpret_cast<const T*>(p.v) + ((long long)t * p.H + h) * p.V + col;
 #pragma unroll
@@ -134,11 +176,17 @@ step_kernel(const StepParams p) {
       const int r = rg + i * RG;
       if (r >= D) continue;
       const float qv = q_s[r], kv = k_s[r];
-      const float a = DELTA ? g : a_s[r];
+      const float a = DELTA || MEM ? g : a_s[r];
+      const float kw = MEM ? kv * beta : kv;
       if (DELTA) kq = fmaf(qv, kv, kq);
+      if (MEM) {
+        float& n_i = N[MEM ? i : 0];
+        n_i = fmaf(n_i, a, kw);
+        kq = fmaf(qv, n_i, kq);
+      }
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
-        S[i][j] = DELTA ? S[i][j] * a : fmaf(S[i][j], a, kv * v[j]);
+        S[i][j] = DELTA ? S[i][j] * a : fmaf(S[i][j], a, kw * v[j]);
         oq[j] = fmaf(qv, S[i][j], oq[j]);
         if (DELTA) ok[j] = fmaf(kv, S[i][j], ok[j]);
       }
@@ -150,7 +198,7 @@ step_kernel(const StepParams p) {
         oq[j] += __shfl_xor_sync(0xffffffffu, oq[j], o);
         if (DELTA) ok[j] += __shfl_xor_sync(0xffffffffu, ok[j], o);
       }
-      if (DELTA) kq += __shfl_xor_sync(0xffffffffu, kq, o);
+      if (DELTA || MEM) kq += __shfl_xor_sync(0xffffffffu, kq, o);
     }
     float* rd = red + (n & 1) * ST_WARPS * NV;
     if (lane < CG) {
@@ -159,7 +207,7 @@ step_kernel(const StepParams p) {
         rd[warp * NV + cl * 4 + j] = oq[j];
         if (DELTA) rd[warp * NV + VB + cl * 4 + j] = ok[j];
       }
-      if (DELTA && cl == 0) rd[warp * NV + 2 * VB] = kq;
+      if ((DELTA || MEM) && cl == 0) rd[warp * NV + NV - 1] = kq;
     }
     if (t + 1 < t1) put((n + 1) % 3);
     __syncthreads();
@@ -191,13 +239,17 @@ step_kernel(const StepParams p) {
         for (int j = 0; j < 4; ++j) S[i][j] = fmaf(kv, u[j], S[i][j]);
       }
     } else if (warp == 0) {
+      kq = 0.f;
 #pragma unroll
-      for (int w = 0; w < ST_WARPS; ++w)
+      for (int w = 0; w < ST_WARPS; ++w) {
 #pragma unroll
         for (int j = 0; j < 4; ++j) o[j] += rd[w * NV + cl * 4 + j];
+        if (MEM) kq += rd[w * NV + NV - 1];
+      }
     }
     if (warp == 0) {
       if (out == nullptr) {
+        if (MEM && vb == 0 && lane == 0) p.den[(long long)t * p.H + h] = kq;
         if (rg == 0) {
           float* dst = p.o_raw + ((long long)t * p.H + h) * p.V + col;
 #pragma unroll
@@ -206,20 +258,27 @@ step_kernel(const StepParams p) {
         }
       } else {                                              // this CTA holds the whole head: norm and gate here
         float sq = 0.f;
+        if (MEM) {
+          const float inv_n = 1.f / (fmaxf(fabsf(kq), expf(-m)) + p.floor);
+#pragma unroll
+          for (int j = 0; j < 4; ++j) o[j] *= inv_n;
+        }
 #pragma unroll
         for (int j = 0; j < 4; ++j) sq += col + j < p.V ? o[j] * o[j] : 0.f;
 #pragma unroll
         for (int x = 1; x < CG; x <<= 1) sq += __shfl_xor_sync(0xffffffffu, sq, x);
         const float inv = rsqrtf(sq / float(p.V) + p.eps);
         if (rg == 0) {
-          T* dst = out + t * p.ld_out + h * p.V + col;
+          T* dst = out + (long long)t * p.ld_out + h * p.V + col;
+          const float* nw = p.norm_w + (MEM ? h * p.V : 0) + col;
 #pragma unroll
           for (int j = 0; j < 4; ++j)
-            if (col + j < p.V)
-              dst[j] = Elem<T>::put(o[j] * inv * p.norm_w[col + j] *
-                                    silu_t<T>(proj_at<T>(p.proj, t, p.off_g + h * p.V + col + j)));
+            if (col + j < p.V) {
+              const float gv = proj_at<T>(p.proj, t, p.off_g + h * p.V + col + j);
+              dst[j] = Elem<T>::put(o[j] * inv * nw[j] * (MEM ? sigmoid_t<T>(gv) : silu_t<T>(gv)));
+            }
         }
-        if (h == 0 && lane < int(p.ld_out) - p.H * p.V) out[t * p.ld_out + p.H * p.V + lane] = Elem<T>::put(0.f);
+        if (h == 0 && lane < p.pad_out) out[(long long)t * p.ld_out + p.H * p.V + lane] = Elem<T>::put(0.f);
       }
     }
   }
@@ -236,6 +295,67 @@ step_kernel(const StepParams p) {
         if (col + j < p.V) dst[j] = S[i][j];
     }
   }
+  if (MEM && vb == 0 && run.len > 0) {
+    // with several column blocks the maximum was written by memory_gates_kernel; only this block writes the normaliser
+    if (cl == 0) {
+      float* ns = p.nstate + ((long long)run.slot * p.H + h) * D;
+#pragma unroll
+      for (int i = 0; i < R; ++i)
+        if (rg + i * RG < D) ns[rg + i * RG] = N[MEM ? i : 0];
+    }
+    if (p.m_t == nullptr && tid == 0) p.mstate[(long long)run.slot * p.H + h] = m;
+  }
+}
+
+// Log gates of matrix memory and their running maximum m_t = max(f_t + m_(t-1), i_t), one CTA per (head, request).  The
+// recurrence is a scan: (a, i) then (a', i') is (a + a', max(a' + i, i')).
+constexpr int MG_THREADS = 512;
+__global__ void __launch_bounds__(MG_THREADS)
+memory_gates_kernel(const StepParams p) {
+  __shared__ float s_a[MG_THREADS / 32], s_i[MG_THREADS / 32];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int h = blockIdx.x, b = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const Run run = get_run(p.runs, b);
+  if (run.slot < 0 || run.len <= 0) return;
+  float* mst = p.mstate + (long long)run.slot * p.H + h;
+  float m = run.start > 0 ? *mst : 0.f;
+  if (tid == 0) p.m_0[(long long)b * p.H + h] = m;
+  for (int t0 = 0; t0 < run.len; t0 += MG_THREADS) {
+    const bool on = t0 + tid < run.len;
+    const long long o = (long long)(run.lo + t0 + tid) * p.H + h;
+    float a = 0.f, i = -INFINITY;                            // identity of the scan
+    if (on) {
+      memory_gates(p, run.lo + t0 + tid, h, i, a);
+      p.log_i[o] = i;
+      p.log_f[o] = a;
+    }
+#pragma unroll
+    for (int d = 1; d < 32; d <<= 1) {
+      const float pa = __shfl_up_sync(0xffffffffu, a, d), pi = __shfl_up_sync(0xffffffffu, i, d);
+      if (lane >= d) {
+        i = fmaxf(a + pi, i);
+        a += pa;
+      }
+    }
+    __syncthreads();
+    if (lane == 31) {
+      s_a[warp] = a;
+      s_i[warp] = i;
+    }
+    __syncthreads();
+    for (int w = 0; w < warp; ++w) m = fmaxf(s_a[w] + m, s_i[w]);        // maximum before this warp's rows
+    if (on) p.m_t[o] = fmaxf(a + m, i);
+    for (int w = warp; w < MG_THREADS / 32; ++w) m = fmaxf(s_a[w] + m, s_i[w]);
+  }
+  __syncthreads();
+  if (tid == 0) *mst = m;
+}
+void launch_memory_gates(const StepParams& p, cudaStream_t s) {
+  if (p.runs.B == 0) return;
+  launch_pdl(PDL_PARTIALS, memory_gates_kernel, dim3(p.H, p.runs.B), dim3(MG_THREADS), 0, s, p);
+  const cudaError_t e = cudaGetLastError();
+  if (e != cudaSuccess) throw std::runtime_error(std::string("matrix memory gates: ") + cudaGetErrorString(e));
 }
 
 // column groups of the state tile: as wide as the head where the rows then fit the registers
@@ -246,23 +366,23 @@ static int step_col_groups(int D, int V) {
 }
 bool step_fuses_norm(int D, int V) { return V <= step_col_groups(D, V) * 4; }
 
-template <typename T, bool DELTA>
+template <typename T, int KIND>
 static void launch_step(const StepParams& p, cudaStream_t s) {
   if (p.runs.B == 0) return;
   if (p.D > ST_MAX_D) throw std::runtime_error("recurrent layers: the key dimension is limited to 1024");
   const int cg = step_col_groups(p.D, p.V);
   const int vb = cg * 4, rows = (p.D + ST_THREADS / cg - 1) / (ST_THREADS / cg);
   const dim3 grid((p.V + vb - 1) / vb, p.H, p.runs.B);
-  const size_t smem = (size_t(9) * p.D + 2 * ST_WARPS * (DELTA ? 2 * vb + 1 : vb)) * 4;
+  const size_t smem = (size_t(9) * p.D + 2 * ST_WARPS * (KIND == REC_DELTA ? 2 * vb + 1 : vb + 1)) * 4;
   auto go = [&](auto kern) {
     if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem));
     launch_pdl(PDL_PARTIALS, kern, grid, dim3(ST_THREADS), smem, s, p);
   };
   auto pick = [&](auto c) {
     constexpr int CG = decltype(c)::value;
-    if (rows <= 4) go(step_kernel<T, DELTA, CG, 4>);
-    else if (rows <= 16) go(step_kernel<T, DELTA, CG, 16>);
-    else go(step_kernel<T, DELTA, CG, 32>);
+    if (rows <= 4) go(step_kernel<T, KIND, CG, 4>);
+    else if (rows <= 16) go(step_kernel<T, KIND, CG, 16>);
+    else go(step_kernel<T, KIND, CG, 32>);
   };
   if (cg == 8) pick(std::integral_constant<int, 8>{});
   else if (cg == 16) pick(std::integral_constant<int, 16>{});
@@ -271,61 +391,67 @@ static void launch_step(const StepParams& p, cudaStream_t s) {
   if (e != cudaSuccess) throw std::runtime_error(std::string("recurrent step: ") + cudaGetErrorString(e));
 }
 void launch_gla_step(const StepParams& p, bool f32, cudaStream_t s) {
-  if (f32) launch_step<float, false>(p, s);
-  else launch_step<bf16, false>(p, s);
+  if (f32) launch_step<float, REC_GLA>(p, s);
+  else launch_step<bf16, REC_GLA>(p, s);
 }
 void launch_delta_step(const StepParams& p, bool f32, cudaStream_t s) {
-  if (f32) launch_step<float, true>(p, s);
-  else launch_step<bf16, true>(p, s);
+  if (f32) launch_step<float, REC_DELTA>(p, s);
+  else launch_step<bf16, REC_DELTA>(p, s);
+}
+void launch_memory_step(const StepParams& p, bool f32, cudaStream_t s) {
+  if (f32) launch_step<float, REC_MEMORY>(p, s);
+  else launch_step<bf16, REC_MEMORY>(p, s);
 }
 
 // ------------------------------------------------------------------ head norm and gate
 // one warp per (row, head)
-template <typename T>
+template <typename T, bool MEM>
 __global__ void __launch_bounds__(256)
-gated_head_norm_kernel(const float* __restrict__ o_raw, const ProjSrc proj, int off_g, const float* __restrict__ norm_w,
-                       float eps, T* __restrict__ out, long long ld_out, long long units, int H, int V) {
+gated_head_norm_kernel(const StepParams p, long long units) {
   pdl_launch_dependents();
   pdl_wait();
   const long long u = blockIdx.x * 8ll + (threadIdx.x >> 5);
   if (u >= units) return;
-  const int lane = threadIdx.x & 31;
+  const int lane = threadIdx.x & 31, H = p.H, V = p.V;
   const long long t = u / H;
   const int h = int(u - t * H);
-  const float* o = o_raw + u * V;
+  const float* o = p.o_raw + u * V;
+  T* out = reinterpret_cast<T*>(p.out) + t * p.ld_out;
+  const float* norm_w = p.norm_w + (MEM ? h * V : 0);
+  const float inv_n = MEM ? 1.f / (fmaxf(fabsf(p.den[u]), expf(-p.m_t[u])) + p.floor) : 1.f;
+  auto gate = [](float g) { return MEM ? sigmoid_t<T>(g) : silu_t<T>(g); };
   float ss = 0.f;
-  if ((V & 3) == 0 && (off_g & 3) == 0) {
+  if (h == 0 && lane < p.pad_out) out[H * V + lane] = Elem<T>::put(0.f);
+  if ((V & 3) == 0 && (p.off_g & 3) == 0) {
     for (int c = lane * 4; c < V; c += 128) {
       const float4 x = *reinterpret_cast<const float4*>(o + c);
       ss += x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
     }
-    const float inv = rsqrtf(warp_sum(ss) / float(V) + eps);
+    const float inv = inv_n * rsqrtf(warp_sum(ss) * inv_n * inv_n / float(V) + p.eps);
     for (int c = lane * 4; c < V; c += 128) {
       const float4 x = *reinterpret_cast<const float4*>(o + c), w = *reinterpret_cast<const float4*>(norm_w + c);
-      const float4 g = proj_at4<T>(proj, t, off_g + h * V + c);
-      store4(out + t * ld_out + h * V + c, x.x * inv * w.x * silu_t<T>(g.x), x.y * inv * w.y * silu_t<T>(g.y),
-             x.z * inv * w.z * silu_t<T>(g.z), x.w * inv * w.w * silu_t<T>(g.w));
+      const float4 g = proj_at4<T>(p.proj, t, p.off_g + h * V + c);
+      store4(out + h * V + c, x.x * inv * w.x * gate(g.x), x.y * inv * w.y * gate(g.y), x.z * inv * w.z * gate(g.z),
+             x.w * inv * w.w * gate(g.w));
     }
-    if (h == 0 && lane < int(ld_out) - H * V) out[t * ld_out + H * V + lane] = Elem<T>::put(0.f);
     return;
   }
   for (int c = lane; c < V; c += 32) ss += o[c] * o[c];
-  const float inv = rsqrtf(warp_sum(ss) / float(V) + eps);
+  const float inv = inv_n * rsqrtf(warp_sum(ss) * inv_n * inv_n / float(V) + p.eps);
   for (int c = lane; c < V; c += 32)
-    out[t * ld_out + h * V + c] = Elem<T>::put(o[c] * inv * norm_w[c] * silu_t<T>(proj_at<T>(proj, t, off_g + h * V + c)));
-  if (h == 0 && lane < int(ld_out) - H * V) out[t * ld_out + H * V + lane] = Elem<T>::put(0.f);
+    out[h * V + c] = Elem<T>::put(o[c] * inv * norm_w[c] * gate(proj_at<T>(p.proj, t, p.off_g + h * V + c)));
 }
-void launch_gated_head_norm(const float* o_raw, const ProjSrc& proj, int off_g, const float* norm_w, float eps,
-                            void* out, long long ld_out, int T, int H, int V, bool f32, cudaStream_t s) {
-  const long long units = (long long)T * H;
+void launch_gated_head_norm(const StepParams& p, int T, bool memory, bool f32, cudaStream_t s) {
+  const long long units = (long long)T * p.H;
   if (units == 0) return;
   const dim3 grid((unsigned)((units + 7) / 8));
-  if (f32)
-    launch_pdl(PDL_NORM, gated_head_norm_kernel<float>, grid, dim3(256), 0, s, o_raw, proj, off_g, norm_w, eps,
-               (float*)out, ld_out, units, H, V);
-  else
-    launch_pdl(PDL_NORM, gated_head_norm_kernel<bf16>, grid, dim3(256), 0, s, o_raw, proj, off_g, norm_w, eps,
-               (bf16*)out, ld_out, units, H, V);
+  if (memory) {
+    if (f32) launch_pdl(PDL_NORM, gated_head_norm_kernel<float, true>, grid, dim3(256), 0, s, p, units);
+    else launch_pdl(PDL_NORM, gated_head_norm_kernel<bf16, true>, grid, dim3(256), 0, s, p, units);
+  } else {
+    if (f32) launch_pdl(PDL_NORM, gated_head_norm_kernel<float, false>, grid, dim3(256), 0, s, p, units);
+    else launch_pdl(PDL_NORM, gated_head_norm_kernel<bf16, false>, grid, dim3(256), 0, s, p, units);
+  }
   const cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess) throw std::runtime_error(std::string("head norm: ") + cudaGetErrorString(e));
 }

@@ -1,14 +1,17 @@
 // Recurrent layers over long runs (bf16 models): chunks of 64 rows, products on the tensor cores.
 //
-// With S the state before a chunk and b the decay accumulated inside it, both recurrences have the form
+// With S the state before a chunk and b the decay accumulated inside it, the recurrences have the form
 //     U = U0 - W S,   O = Q' S + P U,   S <- diag(dec) S + K'^T U
 //   gated linear attention: U = V, no W, b per key channel:
 //       Q' = q e^b,  K' = k e^(b_end - b),  P_ij = sum_d q_id k_jd e^(b_id - b_jd) for j <= i,  dec = e^b_end
 //   gated delta rule (b per head): the writes of a chunk depend on one another through the unit lower triangular
 //       I + L, L_ij = beta_i e^(b_i - b_j) k_i.k_j for j < i; W and U0 solve (I + L) [W | U0] = diag(beta) [e^b k | v]
 //       (Yang, Kautz, Hatamizadeh, "Gated Delta Networks: Improving Mamba2 with Delta Rule"), P_ij = e^(b_i - b_j) q_i.k_j
-// The first kernel computes W, U0, Q', K', P and dec of every chunk in parallel; the second walks the chunks of a
-// run with S in registers.
+//   matrix memory: U = [V | 1] (the last column is the normaliser), no W.  With log gates f (summed to b) and i, running
+//       maximum m, c_j = i_j - b_j and u_i = m_i - b_i = max(m_0, max_(j <= i) c_j) every exponent is at most 0:
+//       Q' = q e^(m_0 - u_i),  K' = k e^(c_j - u_end),  P_ij = e^(c_j - u_i) q_i.k_j,  dec = e^(m_0 - u_end)
+// The first kernel computes W, U0, Q', K', P and dec of every chunk in parallel (m_0 of a chunk comes from the gate kernel
+// of recurrence.cu); the second walks the chunks of a run with S in registers.
 //
 // Everything that enters the recurrence stays 32-bit grade: a tensor-core operand is the sum of two bf16 terms
 // (hi + lo) and a product hi hi + hi lo + lo hi, accumulated in fp32.  Operands of the second kernel are stored in the
@@ -46,8 +49,8 @@ __host__ __device__ inline ChunkLayout chunk_layout(int D, int V, bool delta) {
   return l;
 }
 bool chunk_supported(int D, int V) { return D % 2 == 0 && D <= CK_MAX_D && V % 2 == 0; }
-long long chunk_scratch_bytes(const StepParams& p, int T, bool delta) {
-  return (long long)(T / CK + p.runs.B) * p.H * chunk_layout(p.D, p.V, delta).bytes;
+long long chunk_scratch_bytes(const StepParams& p, int T, int kind) {
+  return (long long)(T / CK + p.runs.B) * p.H * chunk_layout(p.D, p.V, kind == REC_DELTA).bytes;
 }
 
 __device__ __forceinline__ void split_pack(float a, float b, uint32_t& hi, uint32_t& lo) {
@@ -427,14 +430,132 @@ gla_chunk_prepare_kernel(const StepParams p) {
   }
 }
 
+// ------------------------------------------------------------------ first kernel, matrix memory
+__global__ void __launch_bounds__(CA_THREADS)
+memory_chunk_prepare_kernel(const StepParams p) {
+  extern __shared__ float sm[];
+  const ChunkLayout lay = chunk_layout(p.D, p.V, false);
+  const int pitch = chunk_pitch(lay.kd), Dp = lay.kd * 16;
+  float* s_k = sm;                                  // [64][pitch]
+  float* s_q = s_k + CK * pitch;
+  float* s_c = s_q + CK * pitch;                    // c_j, u_i
+  float* s_u = s_c + CK;
+  const int h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  ChunkId id;
+  if (!chunk_of(p, lay, blockIdx.x, h, blockIdx.z, id)) return;
+  const bf16* proj = reinterpret_cast<const bf16*>(p.proj.p);
+  const float m0 = blockIdx.x == 0 ? p.m_0[(long long)blockIdx.z * p.H + h] : p.m_t[(long long)(id.row0 - 1) * p.H + h];
+  if (warp == 0) {                                  // two rows per lane: sums of f, then running maxima of c
+    float f[2], g[2];
+#pragma unroll
+    for (int x = 0; x < 2; ++x) {
+      const int r = lane * 2 + x;
+      const long long o = (long long)(id.row0 + r) * p.H + h;
+      f[x] = r < id.n ? p.log_f[o] : 0.f;
+      g[x] = r < id.n ? p.log_i[o] : -INFINITY;     // rows past the run write nothing
+    }
+    float b = f[0] + f[1];
+#pragma unroll
+    for (int d = 1; d < 32; d <<= 1) {
+      const float y = __shfl_up_sync(0xffffffffu, b, d);
+      if (lane >= d) b += y;
+    }
+    const float c0 = g[0] - (b - f[1]), c1 = g[1] - b;
+    float u = fmaxf(c0, c1);
+#pragma unroll
+    for (int d = 1; d < 32; d <<= 1) {
+      const float y = __shfl_up_sync(0xffffffffu, u, d);
+      if (lane >= d) u = fmaxf(u, y);
+    }
+    const float before = __shfl_up_sync(0xffffffffu, u, 1);
+    const float u0 = fmaxf(m0, lane > 0 ? fmaxf(before, c0) : c0);
+    s_c[lane * 2] = c0;
+    s_c[lane * 2 + 1] = c1;
+    s_u[lane * 2] = u0;
+    s_u[lane * 2 + 1] = fmaxf(u0, c1);
+  }
+#pragma unroll 4
+  for (int r = warp; r < CK; r += CA_THREADS / 32)
+    for (int c = lane * 2; c < Dp; c += 64) {
+      float2 q = make_float2(0.f, 0.f), k = q;
+      if (r < id.n && c < p.D) {
+        auto two = [](const bf16* s) { return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(s)); };
+        const bf16* row = proj + (long long)(id.row0 + r) * p.proj.ld + h * p.D + c;
+        q = two(row + p.off_q);
+        k = two(row + p.off_k);
+      }
+      *reinterpret_cast<float2*>(s_q + r * pitch + c) = make_float2(q.x * p.q_scale, q.y * p.q_scale);
+      *reinterpret_cast<float2*>(s_k + r * pitch + c) = k;
+    }
+  __syncthreads();
+  const float u_end = s_u[CK - 1];
+  const int gr = lane >> 2, gc = (lane & 3) * 2;
+  for (int idx = warp; idx < CK_P; idx += CA_THREADS / 32) {
+    int I, J;
+    tri_block(idx, I, J);
+    float acc[2][4] = {};
+    for (int kk = 0; kk < lay.kd; ++kk) {
+      Frag fq;
+#pragma unroll
+      for (int x = 0; x < 4; ++x) {
+        const float2 q = *reinterpret_cast<const float2*>(s_q + (I * 16 + gr + (x & 1) * 8) * pitch + kk * 16 + gc + (x >> 1) * 8);
+        split_pack(q.x, q.y, fq.h[x], fq.l[x]);
+      }
+#pragma unroll
+      for (int n = 0; n < 2; ++n) {
+        uint32_t bh[2];                             // a key is a bf16 value: no second term
+#pragma unroll
+        for (int x = 0; x < 2; ++x) {
+          const float2 k = *reinterpret_cast<const float2*>(s_k + (J * 16 + n * 8 + gr) * pitch + kk * 16 + gc + x * 8);
+          bh[x] = pack_bf16(k.x, k.y);
+        }
+        mma_bf16(acc[n], fq.l, bh[0], bh[1]);
+        mma_bf16(acc[n], fq.h, bh[0], bh[1]);
+      }
+    }
+#pragma unroll
+    for (int n = 0; n < 2; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int i = I * 16 + gr + (e >> 1) * 8, j = J * 16 + n * 8 + gc + (e & 1);
+        acc[n][e] = j <= i ? acc[n][e] * expf(s_c[j] - s_u[i]) : 0.f;
+      }
+    store_frag(id.unit, lay.p + idx, lane, acc_frag(acc[0], acc[1]));
+  }
+  for (int f = warp; f < 8 * lay.kd; f += CA_THREADS / 32) {
+    Frag a;
+    if (f < 4 * lay.kd) {
+      const int I = f / lay.kd, kk = f - I * lay.kd;
+#pragma unroll
+      for (int x = 0; x < 4; ++x) {
+        const int r = I * 16 + gr + (x & 1) * 8, o = r * pitch + kk * 16 + gc + (x >> 1) * 8;
+        const float e = expf(m0 - s_u[r]);
+        split_pack(s_q[o] * e, s_q[o + 1] * e, a.h[x], a.l[x]);
+      }
+      store_frag(id.unit, lay.q + f, lane, a);
+    } else {
+      const int m = (f - 4 * lay.kd) / 4, kt = (f - 4 * lay.kd) & 3;
+#pragma unroll
+      for (int x = 0; x < 4; ++x) {
+        const int d = m * 16 + gr + (x & 1) * 8, r = kt * 16 + gc + (x >> 1) * 8;
+        split_pack(s_k[r * pitch + d] * expf(s_c[r] - u_end), s_k[(r + 1) * pitch + d] * expf(s_c[r + 1] - u_end), a.h[x], a.l[x]);
+      }
+      store_frag(id.unit, lay.k + f - 4 * lay.kd, lane, a);
+    }
+  }
+  for (int d = tid; d < Dp; d += CA_THREADS) reinterpret_cast<float*>(id.unit + lay.dec)[d] = expf(m0 - u_end);
+}
+
 // ------------------------------------------------------------------ second kernel
 // CTA = (block of VB value columns, head, request), four warps.  Warp w owns rows 16 w .. 16 w + 15 of a chunk for U and
-// O, and the 16-row blocks w, w + 4 of S in registers; S and U go through shared memory as hi / lo operands.
+// O, and the 16-row blocks w, w + 4 of S in registers; S and U go through shared memory as hi / lo operands.  Matrix memory
+// has one column more, V: its S is the normaliser, its U is 1 and its O goes to `den`.
 constexpr int CB_THREADS = 128;
 
-template <bool DELTA, int VB>
+template <int KIND, int VB>
 __global__ void __launch_bounds__(CB_THREADS, VB == 16 ? 3 : 2)
 chunk_scan_kernel(const StepParams p) {
+  constexpr bool DELTA = KIND == REC_DELTA, MEM = KIND == REC_MEMORY;
   constexpr int N8 = VB / 8;
   constexpr int PITCH = VB + 8;                     // bf16; rows an odd number of 16-byte units apart
   extern __shared__ uint8_t smem_raw[];
@@ -450,9 +571,11 @@ chunk_scan_kernel(const StepParams p) {
   if (run.slot < 0 || run.len <= 0) {
     for (int i = tid; i < run.len * VB; i += CB_THREADS)
       if (v0 + i % VB < p.V) p.o_raw[((long long)(run.lo + i / VB) * p.H + h) * p.V + v0 + i % VB] = 0.f;
+      else if (MEM && v0 + i % VB == p.V) p.den[(long long)(run.lo + i / VB) * p.H + h] = p.m_t[(long long)(run.lo + i / VB) * p.H + h] = 0.f;
     return;
   }
   float* st = p.state + ((long long)run.slot * p.H + h) * p.D * p.V;
+  float* ns = MEM ? p.nstate + ((long long)run.slot * p.H + h) * p.D : nullptr;
   float S[2][N8][4];
   auto state_io = [&](bool load) {
 #pragma unroll
@@ -462,6 +585,10 @@ chunk_scan_kernel(const StepParams p) {
 #pragma unroll
         for (int half = 0; half < 2; ++half) {
           const int d = (warp + mi * 4) * 16 + gr + half * 8, v = v0 + n * 8 + gc;
+          if (MEM && d < p.D && v == p.V) {
+            if (load) S[mi][n][half * 2] = ns[d];
+            else ns[d] = S[mi][n][half * 2];
+          }
           if (d >= p.D || v >= p.V) continue;       // V is even: a pair of columns exists or not
           float2* s = reinterpret_cast<float2*>(st + (long long)d * p.V + v);
           if (load) {
@@ -522,6 +649,8 @@ chunk_scan_kernel(const StepParams p) {
           else if (i < id.n)
             x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(
                 reinterpret_cast<const bf16*>(p.proj.p) + (long long)(id.row0 + i) * p.proj.ld + p.off_v + h * p.V + v));
+        } else if (MEM && v == p.V && i < id.n) {
+          x.x = 1.f;
         }
         u[n][half * 2] = x.x;
         u[n][half * 2 + 1] = x.y;
@@ -657,6 +786,8 @@ chunk_scan_kernel(const StepParams p) {
         if (i < now.n && v < p.V)
           *reinterpret_cast<float2*>(p.o_raw + ((long long)(now.row0 + i) * p.H + h) * p.V + v) =
               make_float2(o[n][half * 2], o[n][half * 2 + 1]);
+        else if (MEM && i < now.n && v == p.V)
+          p.den[(long long)(now.row0 + i) * p.H + h] = o[n][half * 2];
       }
     put_state();                                    // the products with the old state ended before the barrier above
     __syncthreads();
@@ -664,8 +795,9 @@ chunk_scan_kernel(const StepParams p) {
   state_io(false);
 }
 
-template <bool DELTA>
+template <int KIND>
 static void launch_chunks(const StepParams& p, int max_len, cudaStream_t s) {
+  constexpr bool DELTA = KIND == REC_DELTA;
   const ChunkLayout lay = chunk_layout(p.D, p.V, DELTA);
   const int chunks = (max_len + CK - 1) / CK, pitch = chunk_pitch(lay.kd);
   const dim3 grid(chunks, p.H, p.runs.B);
@@ -673,23 +805,29 @@ static void launch_chunks(const StepParams& p, int max_len, cudaStream_t s) {
     const int smem = (CK * pitch + CK * (pitch > CA_THREADS / 2 ? pitch : CA_THREADS / 2) + CK * CK + 5 * CK) * 4;
     cudaFuncSetAttribute(delta_chunk_prepare_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     delta_chunk_prepare_kernel<<<grid, CA_THREADS, smem, s>>>(p);
+  } else if (KIND == REC_MEMORY) {
+    const int smem = (2 * CK * pitch + 2 * CK) * 4;
+    cudaFuncSetAttribute(memory_chunk_prepare_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    memory_chunk_prepare_kernel<<<grid, CA_THREADS, smem, s>>>(p);
   } else {
     const int smem = (3 * CK * pitch + 4 * 16 * 18) * 4;
     cudaFuncSetAttribute(gla_chunk_prepare_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     gla_chunk_prepare_kernel<<<grid, CA_THREADS, smem, s>>>(p);
   }
+  const int columns = p.V + (KIND == REC_MEMORY ? 1 : 0);
   auto scan = [&](auto kern, int vb) {
     const int smem = 2 * (lay.kd * 16 + CK) * (vb + 8) * 2;
     cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
-    kern<<<dim3((p.V + vb - 1) / vb, p.H, p.runs.B), CB_THREADS, smem, s>>>(p);
+    kern<<<dim3((columns + vb - 1) / vb, p.H, p.runs.B), CB_THREADS, smem, s>>>(p);
   };
   // few (request, head) pairs: narrower column blocks for more CTAs
-  if (p.runs.B * p.H * ((p.V + 31) / 32) >= 2 * 148) scan(chunk_scan_kernel<DELTA, 32>, 32);
-  else scan(chunk_scan_kernel<DELTA, 16>, 16);
+  if (p.runs.B * p.H * ((p.V + 31) / 32) >= 2 * 148) scan(chunk_scan_kernel<KIND, 32>, 32);
+  else scan(chunk_scan_kernel<KIND, 16>, 16);
   const cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess) throw std::runtime_error(std::string("chunked recurrence: ") + cudaGetErrorString(e));
 }
-void launch_gla_chunk(const StepParams& p, int max_len, cudaStream_t s) { launch_chunks<false>(p, max_len, s); }
-void launch_delta_chunk(const StepParams& p, int max_len, cudaStream_t s) { launch_chunks<true>(p, max_len, s); }
+void launch_gla_chunk(const StepParams& p, int max_len, cudaStream_t s) { launch_chunks<REC_GLA>(p, max_len, s); }
+void launch_delta_chunk(const StepParams& p, int max_len, cudaStream_t s) { launch_chunks<REC_DELTA>(p, max_len, s); }
+void launch_memory_chunk(const StepParams& p, int max_len, cudaStream_t s) { launch_chunks<REC_MEMORY>(p, max_len, s); }
 
 }  // namespace fc
