@@ -1,5 +1,5 @@
-// fp32 residual stream of models that norm a sublayer's output before adding it: embedding with a scale, norm + add,
-// final norm, and the gelu gate of the feed-forward.  Readers of a projection take split-K partial sums as they are.
+// fp32 residual stream: embedding with a scale, norm of a sublayer's output + add, add + norm for the next sublayer, final
+// norm, and the gates of feed-forwards.  Readers of a projection take split-K partial sums as they are.
 #include <algorithm>
 #include <stdexcept>
 #include <string>
@@ -86,6 +86,99 @@ post_norm_add_kernel(const ProjSrc y, const T* __restrict__ bias, float* __restr
     }
   }
   for (int c = W + threadIdx.x; c < Wp; c += RS_THREADS) h[row * Wp + c] = Elem<T>::put(0.f);
+}
+
+// x (+)= y + mixed expert rows;  h = rms(x) * w (or x) in the model's type, zero-padded from W to Wp columns
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(RS_THREADS)
+add_norm_kernel(const AddNorm p, const ProjSrc y, int has_y) {
+  __shared__ float red[RS_THREADS / 32];
+  pdl_launch_dependents();
+  pdl_wait();
+  const long long row = blockIdx.x;
+  const int W = p.W;
+  float* x = p.x + row * W;
+  T* h = reinterpret_cast<T*>(p.h) + row * p.ld_h;
+  float v[RS_CHUNKS][4];
+  float ss = 0.f;
+#pragma unroll
+  for (int c = 0; c < RS_CHUNKS; ++c) {
+    const int col = (threadIdx.x + c * RS_THREADS) * 4;
+    if (col >= W) continue;
+    float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (has_y) a = proj_at4<T>(y, row, col);             // the pad columns of a projection exist and are zero
+    v[c][0] = a.x;
+    v[c][1] = a.y;
+    v[c][2] = a.z;
+    v[c][3] = a.w;
+    for (int j = 0; j < p.top; ++j) {
+      const int r = p.row_of[row * p.top + j];
+      if (r < 0) continue;
+      const float4 e = proj_at4<T>(p.experts, r, col);
+      const float f = p.mix != nullptr ? p.mix[row * p.top + j] : 1.f / float(p.top);
+      v[c][0] = fmaf(e.x, f, v[c][0]);
+      v[c][1] = fmaf(e.y, f, v[c][1]);
+      v[c][2] = fmaf(e.z, f, v[c][2]);
+      v[c][3] = fmaf(e.w, f, v[c][3]);
+    }
+    if (VEC) {
+      if (p.add) {
+        const float4 o = *reinterpret_cast<const float4*>(x + col);
+        v[c][0] += o.x;
+        v[c][1] += o.y;
+        v[c][2] += o.z;
+        v[c][3] += o.w;
+      }
+      if (has_y || p.top > 0) *reinterpret_cast<float4*>(x + col) = make_float4(v[c][0], v[c][1], v[c][2], v[c][3]);
+    } else {
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        if (col + i >= W) {
+          v[c][i] = 0.f;
+          continue;
+        }
+        if (p.add) v[c][i] += x[col + i];
+        x[col + i] = v[c][i];
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i) ss += v[c][i] * v[c][i];
+  }
+  const bool norm = p.w != nullptr;
+  const float inv = norm ? rsqrtf(cta_sum<RS_THREADS>(ss, red) / float(W) + p.eps) : 1.f;
+#pragma unroll
+  for (int c = 0; c < RS_CHUNKS; ++c) {
+    const int col = (threadIdx.x + c * RS_THREADS) * 4;
+    if (col >= W) continue;
+    if (VEC) {
+      const float4 w = norm ? *reinterpret_cast<const float4*>(p.w + col) : make_float4(1.f, 1.f, 1.f, 1.f);
+      store4(h + col, v[c][0] * inv * w.x, v[c][1] * inv * w.y, v[c][2] * inv * w.z, v[c][3] * inv * w.w);
+    } else {
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+        if (col + i < W) h[col + i] = Elem<T>::put(v[c][i] * inv * (norm ? p.w[col + i] : 1.f));
+    }
+  }
+  for (int c = W + threadIdx.x; c < p.Wp; c += RS_THREADS) h[c] = Elem<T>::put(0.f);
+}
+
+// eight columns per thread, grid as gelu_mul_kernel
+template <typename T, int KIND>
+__global__ void __launch_bounds__(RS_THREADS)
+glu_mul_kernel(const GluMul a) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int col = (blockIdx.x * RS_THREADS + threadIdx.x) * 8;
+  if (col >= a.width_p) return;
+#pragma unroll 2
+  for (int row = blockIdx.y; row < a.T; row += gridDim.y) {
+    float g[8], u[8], o[8];
+    proj_at8<T>(a.p, row, a.off_gate + col, g);
+    proj_at8<T>(a.p, row, a.off_up + col, u);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) o[j] = col + j < a.width ? glu_t<T, KIND>(g[j], u[j], a.limit) : 0.f;
+    store8(reinterpret_cast<T*>(a.out) + row * a.ld_out + col, o);
+  }
 }
 
 template <typename T>
@@ -179,6 +272,37 @@ void launch_rms_norm_wide(const float* x, const float* w, void* h, int T, int W,
   else
     launch_pdl(PDL_NORM, rms_norm_wide_kernel<bf16>, dim3(T), dim3(RS_THREADS), 0, s, x, w, (bf16*)h, W, Wp, eps);
   check_launch("final norm");
+}
+
+void launch_add_norm(const AddNorm& p, bool f32, cudaStream_t s) {
+  if (p.T == 0) return;
+  if (p.W > RS_THREADS * RS_CHUNKS * 4) throw std::runtime_error("norm rows are limited to 8192 columns");
+  const ProjSrc y = p.y != nullptr ? *p.y : ProjSrc();
+  const int has_y = p.y != nullptr ? 1 : 0;
+  auto go = [&](auto kern) { launch_pdl(PDL_NORM, kern, dim3(p.T), dim3(RS_THREADS), 0, s, p, y, has_y); };
+  if (f32) {
+    if (p.W % 4 == 0) go(add_norm_kernel<float, true>);
+    else go(add_norm_kernel<float, false>);
+  } else {
+    if (p.W % 4 == 0) go(add_norm_kernel<bf16, true>);
+    else go(add_norm_kernel<bf16, false>);
+  }
+  check_launch("add + norm");
+}
+
+void launch_glu_mul(const GluMul& p, bool f32, cudaStream_t s) {
+  if (p.T == 0) return;
+  const int cols = (p.width_p / 8 + RS_THREADS - 1) / RS_THREADS;
+  const dim3 grid(cols, std::min(p.T, std::max(1, 148 * 8 / cols)));
+  auto go = [&](auto kern) { launch_pdl(PDL_PARTIALS, kern, grid, dim3(RS_THREADS), 0, s, p); };
+  if (p.kind == GLU_ACT_SILU) {
+    if (f32) go(glu_mul_kernel<float, GLU_ACT_SILU>);
+    else go(glu_mul_kernel<bf16, GLU_ACT_SILU>);
+  } else {
+    if (f32) go(glu_mul_kernel<float, GLU_ACT_CLAMPED>);
+    else go(glu_mul_kernel<bf16, GLU_ACT_CLAMPED>);
+  }
+  check_launch("gated activation");
 }
 
 void launch_gelu_mul(const ProjSrc& gu, const void* bias, void* out, int T, int up_off, int width, int width_p,
