@@ -59,6 +59,14 @@ struct GemmParams {
   int num_m, num_n, group_m;
   int total_work;
   int up_row0;            // SWIGLU: row of W where the `up` half starts (= output width)
+  // other forms (GemmForm)
+  float* wide;            // GF_WIDE: columns [wide0, wide0 + wide_n) also go here in fp32, [M, wide_n]
+  int wide0, wide_n;
+  float* acc;             // GF_ACC: fp32 output, pitch ldc_i, replaced or added to
+  int acc_add;
+  const int* plan;        // GF_GROUPED: rows sorted by group, see gemm_bf16_grouped
+  int groups, group_rows; // groups, rows of W per group
+  float limit;            // GLU_CLAMPED
 };
 
 __device__ __forceinline__ float apply_act(float v, int act) {
@@ -114,9 +122,10 @@ struct SmemLayout {
 };
 
 // GLU: gated epilogue, out = act(gate) * up of w = [gate; up]
-enum Glu : int { GLU_NONE = 0, GLU_SILU = 1, GLU_GELU_TANH = 2 };   // GLU_GELU_TANH takes a bias [gate | up]
+enum Glu : int { GLU_NONE = 0, GLU_SILU = 1, GLU_GELU_TANH = 2, GLU_CLAMPED = 3 };   // GLU_GELU_TANH takes a bias [gate | up]
+enum GemmForm : int { GF_PLAIN = 0, GF_WIDE = 1, GF_ACC = 2, GF_GROUPED = 3 };
 
-template <int BN, int STAGES, bool TRANS_OUT, int GLU = GLU_NONE>
+template <int BN, int STAGES, bool TRANS_OUT, int GLU = GLU_NONE, int FORM = GF_PLAIN>
 __global__ void __launch_bounds__(GEMM_THREADS, 1)
 gemm_bf16_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_constant__ CUtensorMap tma_b,
                  const GemmParams p) {
@@ -160,6 +169,23 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_constan
   const uint32_t tmem_base = *tmem_slot;
 
   const int num_kb = (p.K + BK - 1) / BK;
+  // grouped form: how many 128-row tiles there are is known on the device only
+  const int num_m = FORM == GF_GROUPED ? __ldcg(p.plan + p.groups + 1) : p.num_m;
+  const int total_work = FORM == GF_GROUPED ? num_m * p.num_n : p.total_work;
+  // first row of a 128-row tile, end of its rows, first row of W
+  auto tile_rows = [&](int m_blk, int& row0, int& row_end, int& w0) {
+    if constexpr (FORM == GF_GROUPED) {
+      const int* t = p.plan + p.groups + 2 + 2 * m_blk;
+      const int group = __ldcg(t);
+      row0 = __ldcg(t + 1);
+      row_end = min(row0 + BM, __ldcg(p.plan + group + 1));
+      w0 = group * p.group_rows;
+    } else {
+      row0 = m_blk * BM;
+      row_end = p.M;
+      w0 = 0;
+    }
+  };
 
   auto decode_work = [&](int w, int& m_blk, int& n_blk, int& kb0, int& kb1, int& tile, int& split) {
     split = w % p.splits;
@@ -167,7 +193,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_constan
     const int per_group = p.group_m * p.num_n;
     const int g = tile / per_group;
     const int first_m = g * p.group_m;
-    const int gm = min(p.num_m - first_m, p.group_m);
+    const int gm = min(num_m - first_m, p.group_m);
     const int local = tile - g * per_group;
     m_blk = first_m + local % gm;
     n_blk = local / gm;
@@ -182,9 +208,10 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_constan
       uint32_t phase = 0;
       int issued = 0;
       bool ok = true;
-      for (int w = blockIdx.x; w < p.total_work && ok; w += gridDim.x) {
-        int m_blk, n_blk, kb0, kb1, tile, split;
+      for (int w = blockIdx.x; w < total_work && ok; w += gridDim.x) {
+        int m_blk, n_blk, kb0, kb1, tile, split, row0, row_end, w0;
         decode_work(w, m_blk, n_blk, kb0, kb1, tile, split);
+        tile_rows(m_blk, row0, row_end, w0);
         for (int kb = kb0; kb < kb1; ++kb) {
           if (s_flag[0] || !mbar_wait(&empty_bar[stage], phase ^ 1, p.status, ST_TIMEOUT_EMPTY)) {
             s_flag[0] = 1;
@@ -194,13 +221,13 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_constan
           uint8_t* sa = smem + stage * L::STAGE_BYTES;
           uint8_t* sb = sa + L::A_BYTES;
           mbar_expect_tx(&full_bar[stage], L::STAGE_BYTES);
-          tma_load_2d(sa, &tma_a, &full_bar[stage], kb * BK, m_blk * BM);
+          tma_load_2d(sa, &tma_a, &full_bar[stage], kb * BK, row0);
           if constexpr (GLU != GLU_NONE) {
             // B tile = 128 rows of the gate half + the matching 128 rows of the up half
-            tma_load_2d(sb, &tma_b, &full_bar[stage], kb * BK, n_blk * (BN / 2));
-            tma_load_2d(sb + L::B_BYTES / 2, &tma_b, &full_bar[stage], kb * BK, p.up_row0 + n_blk * (BN / 2));
+            tma_load_2d(sb, &tma_b, &full_bar[stage], kb * BK, w0 + n_blk * (BN / 2));
+            tma_load_2d(sb + L::B_BYTES / 2, &tma_b, &full_bar[stage], kb * BK, w0 + p.up_row0 + n_blk * (BN / 2));
           } else {
-            tma_load_2d(sb, &tma_b, &full_bar[stage], kb * BK, n_blk * BN);
+            tma_load_2d(sb, &tma_b, &full_bar[stage], kb * BK, w0 + n_blk * BN);
           }
           ++issued;
           if (++stage == STAGES) {
@@ -231,7 +258,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_constan
       int acc = 0;
       uint32_t acc_phase = 0;
       bool ok = true;
-      for (int w = blockIdx.x; w < p.total_work && ok; w += gridDim.x) {
+      for (int w = blockIdx.x; w < total_work && ok; w += gridDim.x) {
         int m_blk, n_blk, kb0, kb1, tile, split;
         decode_work(w, m_blk, n_blk, kb0, kb1, tile, split);
         if (s_flag[0] || !mbar_wait(&acc_empty[acc], acc_phase ^ 1, p.status, ST_TIMEOUT_ACC_EMPTY)) {
@@ -274,7 +301,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_constan
     const int ep_tid = (warp - 2) * 32 + lane;       // 0..127
     int acc = 0;
     uint32_t acc_phase = 0;
-    for (int w = blockIdx.x; w < p.total_work; w += gridDim.x) {
+    for (int w = blockIdx.x; w < total_work; w += gridDim.x) {
       int m_blk, n_blk, kb0, kb1, tile, split;
       decode_work(w, m_blk, n_blk, kb0, kb1, tile, split);
       if (s_flag[0] || !mbar_wait(&acc_full[acc], acc_phase, p.status, ST_TIMEOUT_ACC_FULL)) {
@@ -283,13 +310,42 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_constan
       }
       tc_fence_after();
       const uint32_t t_addr = tmem_base + (uint32_t(lane_group * 32) << 16) + uint32_t(acc * BN);
-      const int gi = m_blk * BM + row;
+      int row0, row_end, w0;
+      tile_rows(m_blk, row0, row_end, w0);
+      const int gi = row0 + row;
       const int j0 = n_blk * BN;
 
       auto finish_chunk = [&](float (&v)[32], int c) {
         // v: 32 consecutive columns of row `gi`, starting at column j0 + 32 c
         const int jb = j0 + c * 32;
-        if (gi >= p.M) return;
+        if (gi >= row_end) return;
+        if constexpr (FORM == GF_ACC) {
+          float* dst = p.acc + (long long)gi * p.ldc_i + jb;
+          if (jb + 32 <= p.N && (reinterpret_cast<uintptr_t>(dst) & 15) == 0) {
+            float4 o[8];
+#pragma unroll
+            for (int q = 0; q < 8; ++q)
+              o[q] = p.acc_add ? *reinterpret_cast<const float4*>(dst + q * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+            for (int q = 0; q < 8; ++q)
+              *reinterpret_cast<float4*>(dst + q * 4) =
+                  make_float4(o[q].x + v[q * 4], o[q].y + v[q * 4 + 1], o[q].z + v[q * 4 + 2], o[q].w + v[q * 4 + 3]);
+          } else {
+#pragma unroll
+            for (int t = 0; t < 32; ++t)
+              if (jb + t < p.N) dst[t] = p.acc_add ? dst[t] + v[t] : v[t];
+          }
+          return;
+        }
+        if constexpr (FORM == GF_WIDE) {
+          if (jb < p.wide0 + p.wide_n && jb + 32 > p.wide0) {
+#pragma unroll
+            for (int t = 0; t < 32; ++t) {
+              const int o = jb + t - p.wide0;
+              if (o >= 0 && o < p.wide_n) p.wide[(long long)gi * p.wide_n + o] = v[t];
+            }
+          }
+        }
         float bi = (p.bias != nullptr && p.bias_on_i) ? __bfloat162float(p.bias[gi]) : 0.f;
         if constexpr (!TRANS_OUT) {
           __nv_bfloat16* dst = p.C + (long long)gi * p.ldc_i + jb;
@@ -358,7 +414,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_constan
             tc_fence_before();
             mbar_arrive(&acc_empty[acc]);
           }
-          if (gi < p.M) {
+          if (gi < row_end) {
             __nv_bfloat16* dst = p.C + (long long)gi * p.ldc_i + jo + c * 32;
 #pragma unroll
             for (int q = 0; q < 4; ++q) {
@@ -381,6 +437,11 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_constan
                   // 0.5 z (1 + tanh y) = z / (1 + exp(-2 y)), y = sqrt(2 / pi) (z + 0.044715 z^3)
                   a = __fdividef(g0, 1.f + __expf(-1.5957691216057308f * (g0 + 0.044715f * g0 * g0 * g0))) * u0;
                   b = __fdividef(g1, 1.f + __expf(-1.5957691216057308f * (g1 + 0.044715f * g1 * g1 * g1))) * u1;
+                } else if constexpr (GLU == GLU_CLAMPED) {
+                  g0 = fminf(g0, p.limit);
+                  g1 = fminf(g1, p.limit);
+                  a = __fdividef(g0, 1.f + __expf(-1.702f * g0)) * (fminf(fmaxf(u0, -p.limit), p.limit) + 1.f);
+                  b = __fdividef(g1, 1.f + __expf(-1.702f * g1)) * (fminf(fmaxf(u1, -p.limit), p.limit) + 1.f);
                 } else {
                   a = g0 / (1.f + __expf(-g0)) * u0;
                   b = g1 / (1.f + __expf(-g1)) * u1;
@@ -511,11 +572,11 @@ CUtensorMap make_tmap_bf16_3d(const void* base, uint64_t n0, uint64_t n1, uint64
   return m;
 }
 
-template <int BN, int STAGES, bool TRANS, int GLU = GLU_NONE>
+template <int BN, int STAGES, bool TRANS, int GLU = GLU_NONE, int FORM = GF_PLAIN>
 static void launch_one(const CUtensorMap& ta, const CUtensorMap& tb, const GemmParams& p, int grid,
                        cudaStream_t stream) {
   using L = SmemLayout<BN, STAGES>;
-  auto kern = gemm_bf16_kernel<BN, STAGES, TRANS, GLU>;
+  auto kern = gemm_bf16_kernel<BN, STAGES, TRANS, GLU, FORM>;
   // the attribute belongs to the (function, device) pair: remember it per device, not per process
   static std::atomic<uint64_t> configured{0};
   int dev = 0;
@@ -616,6 +677,104 @@ void gemm_bf16(const void* x, const void* w, void* c, const void* bias, int M, i
     return;
   // decode-size batch: weight-streaming kernel (gemm_skinny.cu)
   gemm_skinny_bf16(x, w, c, bias, M, N, K, ldx, ldw, ldc, act, ws, sm_limit, 0, true, stream);
+}
+
+// ---- prefill-size forms
+static GemmParams prefill_params(void* c, int M, int N, int K, long long ldc, const GemmWorkspace& ws) {
+  GemmParams p{};
+  p.M = M;
+  p.N = N;
+  p.K = K;
+  p.C = reinterpret_cast<__nv_bfloat16*>(c);
+  p.ldc_i = ldc;
+  p.ldc_j = 1;
+  p.status = ws.status;
+  p.splits = 1;
+  p.kb_per_split = (K + BK - 1) / BK;
+  p.num_m = (M + BM - 1) / BM;
+  p.group_m = 16;
+  return p;
+}
+
+void gemm_bf16_wide(const void* x, const void* w, void* c, int M, int N, int K, long long ldx, long long ldw, long long ldc,
+                    int wide0, int wide_n, float* wide, const GemmWorkspace& ws, int sm_limit, cudaStream_t stream) {
+  if (M <= 0 || N <= 0 || K <= 0) return;
+  constexpr int BN = 256;
+  const int sms = sm_limit > 0 ? sm_limit : gemm_num_sms();
+  GemmParams p = prefill_params(c, M, N, K, ldc, ws);
+  p.wide = wide;
+  p.wide0 = wide0;
+  p.wide_n = wide_n;
+  p.num_n = (N + BN - 1) / BN;
+  p.total_work = p.num_m * p.num_n;
+  launch_one<BN, 4, false, GLU_NONE, GF_WIDE>(make_tmap_bf16_2d(x, M, K, ldx, BM, BK), make_tmap_bf16_2d(w, N, K, ldw, BN, BK),
+                                              p, std::min(p.total_work, sms), stream);
+}
+
+void gemm_bf16_acc(const void* x, const void* w, float* y, int M, int N, int K, long long ldx, long long ldw, long long ldy,
+                   bool add, const GemmWorkspace& ws, int sm_limit, cudaStream_t stream) {
+  if (M <= 0 || N <= 0 || K <= 0) return;
+  constexpr int BN = 256;
+  const int sms = sm_limit > 0 ? sm_limit : gemm_num_sms();
+  GemmParams p = prefill_params(nullptr, M, N, K, ldy, ws);
+  p.acc = y;
+  p.acc_add = add ? 1 : 0;
+  p.num_n = (N + BN - 1) / BN;
+  p.total_work = p.num_m * p.num_n;
+  launch_one<BN, 4, false, GLU_NONE, GF_ACC>(make_tmap_bf16_2d(x, M, K, ldx, BM, BK), make_tmap_bf16_2d(w, N, K, ldw, BN, BK),
+                                             p, std::min(p.total_work, sms), stream);
+}
+
+void gemm_bf16_clamped_glu(const void* x, const void* w, void* c, int M, int width, int K, long long ldx, long long ldw,
+                           long long ldc, float limit, const GemmWorkspace& ws, int sm_limit, cudaStream_t stream) {
+  if (M <= 0 || width <= 0 || K <= 0) return;
+  constexpr int BN = 256;
+  if (width % 128 != 0 || ldc % 8 != 0 || (reinterpret_cast<uintptr_t>(c) & 15) != 0)
+    throw std::runtime_error("fused gated GEMM needs a width that is a multiple of 128 and a 16-byte aligned output");
+  GemmParams p = prefill_params(c, M, width, K, ldc, ws);
+  p.limit = limit;
+  p.up_row0 = width;
+  p.num_n = width / (BN / 2);
+  p.total_work = p.num_m * p.num_n;
+  launch_one<BN, 4, false, GLU_CLAMPED>(make_tmap_bf16_2d(x, M, K, ldx, BM, BK),
+                                        make_tmap_bf16_2d(w, 2 * width, K, ldw, BN / 2, BK), p,
+                                        std::min(p.total_work, sm_limit > 0 ? sm_limit : gemm_num_sms()), stream);
+}
+
+void gemm_bf16_grouped(const void* x, const void* w, void* c, const int* plan, int rows, int groups, int max_tiles, int N,
+                       int K, long long ldx, long long ldc, int glu_kind, float limit, const GemmWorkspace& ws, int sm_limit,
+                       cudaStream_t stream) {
+  if (rows <= 0 || groups <= 0) return;
+  const int sms = sm_limit > 0 ? sm_limit : gemm_num_sms();
+  GemmParams p = prefill_params(c, rows, N, K, ldc, ws);
+  p.plan = plan;
+  p.groups = groups;
+  p.group_rows = N;
+  p.limit = limit;
+  const CUtensorMap ta = make_tmap_bf16_2d(x, rows, K, ldx, BM, BK);
+  if (glu_kind >= 0) {
+    constexpr int BN = 256;
+    const int width = N / 2;
+    if (N % 256 != 0 || ldc % 8 != 0 || (reinterpret_cast<uintptr_t>(c) & 15) != 0)
+      throw std::runtime_error("grouped gated GEMM needs a width that is a multiple of 128 and a 16-byte aligned output");
+    p.N = width;
+    p.up_row0 = width;
+    p.num_n = width / (BN / 2);
+    const CUtensorMap tb = make_tmap_bf16_2d(w, (uint64_t)groups * N, K, K, BN / 2, BK);
+    const int grid = std::min(max_tiles * p.num_n, sms);
+    if (glu_kind == 0) launch_one<BN, 4, false, GLU_SILU, GF_GROUPED>(ta, tb, p, grid, stream);
+    else launch_one<BN, 4, false, GLU_CLAMPED, GF_GROUPED>(ta, tb, p, grid, stream);
+  } else if (N >= 256) {
+    constexpr int BN = 256;
+    p.num_n = (N + BN - 1) / BN;
+    launch_one<BN, 4, false, GLU_NONE, GF_GROUPED>(ta, make_tmap_bf16_2d(w, (uint64_t)groups * N, K, K, BN, BK), p,
+                                                   std::min(max_tiles * p.num_n, sms), stream);
+  } else {
+    constexpr int BN = 128;
+    p.num_n = (N + BN - 1) / BN;
+    launch_one<BN, 6, false, GLU_NONE, GF_GROUPED>(ta, make_tmap_bf16_2d(w, (uint64_t)groups * N, K, K, BN, BK), p,
+                                                   std::min(max_tiles * p.num_n, sms), stream);
+  }
 }
 
 }  // namespace fc

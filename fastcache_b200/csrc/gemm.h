@@ -56,6 +56,23 @@ CUtensorMap make_tmap_bf16_3d(const void* base, uint64_t n0, uint64_t n1, uint64
 void gemm_bf16(const void* x, const void* w, void* c, const void* bias, int M, int N, int K, long long ldx,
                long long ldw, long long ldc, int act, const GemmWorkspace& ws, int sm_limit, cudaStream_t stream);
 
+// Prefill-size forms of the same kernel.
+// wide: columns [wide0, wide0 + wide_n) of the product also go to `wide` [M, wide_n] in fp32.
+void gemm_bf16_wide(const void* x, const void* w, void* c, int M, int N, int K, long long ldx, long long ldw, long long ldc,
+                    int wide0, int wide_n, float* wide, const GemmWorkspace& ws, int sm_limit, cudaStream_t stream);
+// acc: the fp32 product replaces y [M, N] (pitch ldy) or is added to it.
+void gemm_bf16_acc(const void* x, const void* w, float* y, int M, int N, int K, long long ldx, long long ldw, long long ldy,
+                   bool add, const GemmWorkspace& ws, int sm_limit, cudaStream_t stream);
+// clamped_glu: w = [gate; up], c [M, width] = g sigmoid(1.702 g) (u + 1), g = min(gate, limit), u = up clamped to +-limit.
+void gemm_bf16_clamped_glu(const void* x, const void* w, void* c, int M, int width, int K, long long ldx, long long ldw,
+                           long long ldc, float limit, const GemmWorkspace& ws, int sm_limit, cudaStream_t stream);
+// grouped: rows of x sorted by group, w [groups, N, K]; `plan` (device): [groups + 1] first row of every group, [1] number
+// of 128-row tiles, then (group, first row) of every tile (at most max_tiles).  glu_kind -1: c [rows, N]; 0 silu, 1 clamped:
+// w[g] = [gate; up], c [rows, N / 2].
+void gemm_bf16_grouped(const void* x, const void* w, void* c, const int* plan, int rows, int groups, int max_tiles, int N,
+                       int K, long long ldx, long long ldc, int glu_kind, float limit, const GemmWorkspace& ws, int sm_limit,
+                       cudaStream_t stream);
+
 // Decode-size batches (M <= 256).  Returns the number of K splits used; when that is > 1 and
 // `finalize` is false, ws.scratch holds fp32 partial sums [splits, M, N] for the caller to reduce.
 // `fused` != nullptr: the epilogue named there runs inside the kernel (`c` and `act` are unused).  Returns 0 without
@@ -65,7 +82,8 @@ void gemm_bf16(const void* x, const void* w, void* c, const void* bias, int M, i
 // width % 128 == 0 and the cluster form (returns 0 without launching when it cannot be taken).  SK_NO_CLUSTER: never
 // reduce the K splits inside a thread-block cluster (done where the shape allows when cluster_splitk_enabled(): the
 // result is then always finished bf16 in `c` and the return value is 1).
-enum SkinnyFlags : int { SK_SWIGLU = 1, SK_NO_CLUSTER = 2 };
+// SK_PARTIAL: ws.scratch receives the fp32 partial sums also when K is not split; with `finalize` `c` is written too.
+enum SkinnyFlags : int { SK_SWIGLU = 1, SK_NO_CLUSTER = 2, SK_PARTIAL = 4 };
 int gemm_skinny_bf16(const void* x, const void* w, void* c, const void* bias, int M, int N, int K, long long ldx,
                      long long ldw, long long ldc, int act, const GemmWorkspace& ws, int sm_limit,
                      int splits_request, bool finalize, cudaStream_t stream, const SkinnyFused* fused = nullptr,

@@ -71,6 +71,7 @@ struct SkinnyParams {
   int kb_per_split;
   uint32_t* status;
   int cluster;            // > 0: the splits are the CTAs of a cluster and reduce through shared memory
+  int keep;               // partial sums also with one split
   int swiglu;             // cluster mode only: tile = 128 gate rows + the matching 128 up rows, out [Mtok, Nw / 2]
   // fused epilogue (see the header comment); epi == EPI_NONE: everything below is unused
   int epi;
@@ -408,7 +409,7 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap tma_w, const __grid_const
   } else {
     const int lane_group = warp & 3;
     const int row = lane_group * 32 + lane;
-    const bool direct = p.splits == 1 && p.epi == EPI_NONE;     // bf16 result straight from the accumulator
+    const bool direct = p.splits == 1 && p.epi == EPI_NONE && !p.keep;     // bf16 result straight from the accumulator
     if (p.cluster > 0) {
       // the accumulators are exchanged and reduced after the role branches, by all CTAs of the cluster together
       if (*s_abort || !mbar_wait(acc_full, 0, p.status, ST_TIMEOUT_ACC_FULL)) *s_abort = 1;
@@ -761,7 +762,8 @@ int gemm_skinny_bf16(const void* x, const void* w, void* c, const void* bias, in
   if (fuse && tiles * splits > sms) splits = std::max(1, sms / tiles);
   // ---- the cluster form, where allowed: the splits become the CTAs of a cluster and nothing is left for a consumer
   int cluster = 0;
-  const bool want_cluster = !fuse && splits_request <= 0 && (flags & SK_NO_CLUSTER) == 0 && cluster_splitk_enabled();
+  const bool keep = (flags & SK_PARTIAL) != 0 && (size_t)M * N <= scratch_floats;
+  const bool want_cluster = !fuse && !keep && splits_request <= 0 && (flags & SK_NO_CLUSTER) == 0 && cluster_splitk_enabled();
   if (want_cluster || swiglu) {
     const int cap = sm_limit > 0 ? sm_limit : 0;
     int s_c = 0;
@@ -792,6 +794,7 @@ int gemm_skinny_bf16(const void* x, const void* w, void* c, const void* bias, in
   p.status = ws.status;
   p.cluster = cluster;
   p.swiglu = swiglu ? 1 : 0;
+  p.keep = keep ? 1 : 0;
   if (fuse) {
     p.epi = fused->epi;
     p.grid_sync = ws.grid_sync;
@@ -833,7 +836,7 @@ int gemm_skinny_bf16(const void* x, const void* w, void* c, const void* bias, in
             M, N, K, rows, tiles, cluster, splits, kb_per, act8[1], act8[2], act8[3], act8[4], act8[5], act8[6], act8[7], act8[8]);
   }
   if (cluster) return 1;               // finished bf16 result in `c`
-  if (splits > 1 && finalize && !fuse) {
+  if ((splits > 1 || keep) && finalize && !fuse) {
     const long long total = (long long)M * (N / 4);
     const int blocks = (int)std::min<long long>((total + 255) / 256, 2048);
     launch_pdl(PDL_FINALIZE, skinny_finalize_kernel, dim3(blocks), dim3(256), 0, stream, (const float*)ws.scratch, p.bias, p.out, M,
