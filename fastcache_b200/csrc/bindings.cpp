@@ -470,6 +470,7 @@ void register_compress(pybind11::module_& m) __attribute__((weak));
 void register_comm(pybind11::module_& m) __attribute__((weak));
 void register_symm(pybind11::module_& m) __attribute__((weak));
 void register_hybrid(pybind11::module_& m);
+void register_prenorm(pybind11::module_& m);
 void register_symm(pybind11::module_& m);
 
 namespace fc {
@@ -523,6 +524,7 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("num_sms", []() { return fc::gemm_num_sms(); });
   m.def("status_tensor", [](int64_t device) { return device_status(int(device)); });
   register_hybrid(m);
+  register_prenorm(m);
   if (register_attention) register_attention(m);
   if (register_greenctx) register_greenctx(m);
   if (register_compress) register_compress(m);

@@ -1,4 +1,5 @@
-// Python bindings of the hybrid-model kernels.  Tensors are checked here, so that the kernels can assume their layout.
+// Python bindings of the hybrid-model kernels (those of pre-normed layers with parallel sublayers: prenorm_bind.cpp).
+// Tensors are checked here, so that the kernels can assume their layout.
 #include <ATen/cuda/CUDAContext.h>
 #include <c10/cuda/CUDAGuard.h>
 #include <torch/extension.h>
@@ -7,31 +8,9 @@
 #include <tuple>
 #include <vector>
 
-#include "gemm.h"
-#include "hybrid.h"
-#include "workspace.h"
+#include "hybrid_bind.h"
 
 namespace {
-
-using torch::Tensor;
-using OptTensor = c10::optional<Tensor>;
-
-bool is_f32(const Tensor& t) { return t.scalar_type() == torch::kFloat32; }
-cudaStream_t stream_now() { return at::cuda::getCurrentCUDAStream(); }
-const fc::StreamWorkspace& ws_of(const Tensor& t) { return fc::stream_workspace(t.get_device(), stream_now()); }
-int pad8(int n) { return (n + 7) / 8 * 8; }
-
-void check_elem(const Tensor& t, const char* name) {
-  TORCH_CHECK(t.is_cuda() && (t.scalar_type() == torch::kBFloat16 || is_f32(t)), name, " must be a bf16 or fp32 CUDA tensor");
-}
-void check_f32(const Tensor& t, const char* name, int64_t n) {
-  TORCH_CHECK(t.is_cuda() && is_f32(t) && t.is_contiguous() && t.numel() == n, name, " must be a contiguous fp32 tensor of ",
-              n, " elements");
-}
-void check_i32(const Tensor& t, const char* name, int64_t n) {
-  TORCH_CHECK(t.is_cuda() && t.scalar_type() == torch::kInt32 && t.is_contiguous() && t.numel() >= n, name,
-              " must be a contiguous int32 tensor of at least ", n, " elements");
-}
 
 // x @ w.T.  `partial`: decode-size bf16 products may stay split-K partial sums in the stream's scratch, valid until
 // the next product on this stream.  `hold` keeps the finished output alive.  An empty w: x is the projection output.
@@ -178,38 +157,21 @@ Tensor linear_gelu_mul(const Tensor& h, const Tensor& w, const OptTensor& bias, 
   return out;
 }
 
-fc::RunBatch run_batch(const OptTensor& cu, const Tensor& ctx, const Tensor& slots, const Tensor& state) {
-  fc::RunBatch r;
-  r.B = int(slots.numel());
-  check_i32(slots, "state slots", r.B);
-  check_i32(ctx, "context lengths", r.B);
-  if (cu.has_value() && cu->defined()) {
-    check_i32(*cu, "run boundaries", r.B + 1);
-    r.cu = cu->data_ptr<int>();
-  }
-  r.ctx = ctx.data_ptr<int>();
-  r.slots = slots.data_ptr<int>();
-  r.num_slots = int(state.size(0));
-  return r;
-}
-
-constexpr int CHUNK_MIN_ROWS = 24;      // longest run of a batch from which the chunked kernels are used
-
 void run_recurrence(fc::StepParams& p, const Tensor& h, bool delta, bool chunk, int T, int max_len, Tensor& out,
                     Tensor& o_raw) {
   const bool f32 = is_f32(h);
   out = torch::empty({T, pad8(p.H * p.V)}, h.options());
   const bool fused = !chunk && fc::step_fuses_norm(p.D, p.V);
   p.ld_out = out.size(1);
-  if (fused) {
-    p.out = out.data_ptr();
-  } else {
+  p.pad_out = int(p.ld_out) - p.H * p.V;
+  p.out = fused ? out.data_ptr() : nullptr;
+  if (!fused) {
     o_raw = torch::empty({T, p.H * p.V}, h.options().dtype(torch::kFloat32));
     p.o_raw = o_raw.data_ptr<float>();
   }
   Tensor scratch;
   if (chunk) {
-    scratch = torch::empty({fc::chunk_scratch_bytes(p, T, delta)}, h.options().dtype(torch::kUInt8));
+    scratch = torch::empty({fc::chunk_scratch_bytes(p, T, delta ? fc::REC_DELTA : fc::REC_GLA)}, h.options().dtype(torch::kUInt8));
     p.scratch = scratch.data_ptr<uint8_t>();
     if (delta) fc::launch_delta_chunk(p, max_len, stream_now());
     else fc::launch_gla_chunk(p, max_len, stream_now());
@@ -217,9 +179,10 @@ void run_recurrence(fc::StepParams& p, const Tensor& h, bool delta, bool chunk, 
     if (delta) fc::launch_delta_step(p, f32, stream_now());
     else fc::launch_gla_step(p, f32, stream_now());
   }
-  if (!fused)
-    fc::launch_gated_head_norm(p.o_raw, p.proj, p.off_g, p.norm_w, p.eps, out.data_ptr(), p.ld_out, T, p.H, p.V, f32,
-                               stream_now());
+  if (!fused) {
+    p.out = out.data_ptr();
+    fc::launch_gated_head_norm(p, T, false, f32, stream_now());
+  }
 }
 
 Tensor gla(const Tensor& h, const Tensor& w, const Tensor& w_a2, const Tensor& z_bias, const Tensor& norm_w, double eps,

@@ -16,7 +16,13 @@ from .. import ops
 from ..engine.layer_cache import LayerCache, PassCache
 from ..ops.hybrid import WindowDims
 from ..utils.context import get_context
+from .linear import pad8
 from .recurrent import fp32_vector
+
+
+def padded_dim(dim: int) -> int:
+    """Row width of the pages: the head sizes that the tensor-core attention kernels take, larger ones as they are."""
+    return 64 if dim <= 64 else 128 if dim <= 128 else pad8(dim)
 
 
 class WindowedAttention(nn.Module):
@@ -44,7 +50,7 @@ class WindowedAttention(nn.Module):
                                offset["q"], offset["k"], offset["g"])
 
     def cache(self) -> LayerCache:
-        return LayerCache(PassCache(), kv=(self.kv_heads, self.dim))
+        return LayerCache(PassCache(), kv=(self.kv_heads, padded_dim(self.dim)))
 
     def forward(self, positions: torch.Tensor, p, cache: PassCache, out: torch.Tensor) -> None:
         ops.hybrid.windowed_attention(p, self.dims, self.q_norm, self.k_norm, self.sink, self.eps, cache.k_rows,

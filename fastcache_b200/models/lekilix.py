@@ -22,6 +22,7 @@ from ..layers.recurrent import MatrixMemory, fp32_vector
 from ..layers.windowed_attention import WindowedAttention
 from ..ops.hybrid import GluSpec
 from ..parallel import tp as tpmod
+from ..utils.context import get_context
 
 
 def one_plus(param: nn.Parameter, loaded: torch.Tensor, shard_id=None) -> None:
@@ -84,7 +85,7 @@ class LekilixLayer(nn.Module):
         a = h.new_empty(h.shape[0], self.out_proj.input_size)
         # many rows: the dense feed-forward is a product of its own, with the gate in its epilogue
         split = self.ff is not None and h.shape[0] > hy.SMALL_ROWS
-        p = hy.project(h, inp.weight, off["gate"] if split else None, self.wide)
+        p = hy.project(h, inp.weight, get_context(), off["gate"] if split else None, self.wide)
         self.mix(positions, p, cache, a[:, :pad8(self.mix.out_width)])
         y = None
         if self.ff is not None:

@@ -202,13 +202,17 @@ def latent_attention(h, weight, d: LatentDims, kv_norm_w, eps: float, kv_proj, w
 SMALL_ROWS = 256        # up to this many rows a projection stays fp32 split-K partial sums for its readers
 
 
-def project(h, weight, rows: Optional[int] = None, wide=None):
+CHUNK_ROWS = 24         # longest run of a batch from which recurrences work in chunks, on finished projections
+
+
+def project(h, weight, ctx, rows: Optional[int] = None, wide=None):
     """h @ weight[:rows].T for the ops below: a matrix on CPU, an extension object on CUDA (for up to SMALL_ROWS rows its
     fp32 partial sums, valid until the next product).  `wide` = (first, count): columns that are kept in fp32."""
     if h.is_cuda:
         _n()
         first, count = wide or (0, 0)
-        return ext().project(h, weight, int(rows or weight.shape[0]), int(first), int(count))
+        finish = ctx.is_prefill and int(ctx.max_seqlen_q) >= CHUNK_ROWS
+        return ext().project(h, weight, int(rows or weight.shape[0]), int(first), int(count), finish)
     return ref_linear(h, weight if rows is None else weight[:rows])
 
 

@@ -211,13 +211,13 @@ def windowed_attention(p, d, q_norm, k_norm, sink, eps: float, k_rows, v_rows, p
     ok = ctx.slot_mapping >= 0
     slots = ctx.slot_mapping[ok].long()
     bs = k_rows.shape[2]
-    k_rows[slots // bs, :, slots % bs] = kn[ok].to(k_rows.dtype)
-    v_rows[slots // bs, :, slots % bs] = k.reshape(T, G, D)[ok].to(v_rows.dtype)
+    k_rows[slots // bs, :, slots % bs, :D] = kn[ok].to(k_rows.dtype)
+    v_rows[slots // bs, :, slots % bs, :D] = k.reshape(T, G, D)[ok].to(v_rows.dtype)
     o = torch.zeros(T, H, D)
     for i, lo, hi, start, _ in runs(ctx):
         n = start + hi - lo
         blocks = ctx.block_tables[i][: -(-n // bs)].long()
-        ks, vs = (r[blocks].transpose(1, 2).reshape(-1, G, D)[:n].float().repeat_interleave(H // G, 1)
+        ks, vs = (r[blocks][..., :D].transpose(1, 2).reshape(-1, G, D)[:n].float().repeat_interleave(H // G, 1)
                   for r in (k_rows, v_rows))
         s = torch.einsum("ihd,jhd->hij", q[lo:hi].float(), ks) * d.scale
         back = torch.arange(start, n)[:, None] - torch.arange(n)[None, :]
