@@ -64,6 +64,9 @@ def weights(cfg, seed=0):
         else:
             VD = m["vdim"]
             put(p + "k", H * D, W)
+            # keys lean towards the queries: a first token whose k.q is near zero has outputs of either sign after the head
+            # norm, which no 16-bit run can decide
+            out[p + "k"] = (0.7 * out[p + "k"] + 0.7 * out[p + "q"]).bfloat16().float()
             put(p + "v", H * VD, W)
             put(p + "g", H * VD, W)
             put(p + "o", W, H * VD)
