@@ -637,12 +637,12 @@ def run_layers(args):
     from fastcache_b200 import ops
     sampler = ClockSampler(0)
     sampler.start()
-    res = run(max(5, args.steps), args.small)
+    res = run(max(5, args.steps), args.small, model=args.layers)
     clocks = sampler.stop()
     last = list(res["sizes"].values())[-1]["rows"][0]
     emit({"metric": "prefill tokens/s of 8 hybrid layers", "value": last["tok_s"], "unit": "tok/s", "n_gpus": 1,
           "steps": max(5, args.steps), "warmup": 3, "ms_per_step": last["ms"], "higher_is_better": True, "scaling": "weak",
-          "vs_baseline": None, "dtype": "bf16", "data": "synthetic", "config": {"model": "Bagedra beside Qwen3", **res},
+          "vs_baseline": None, "dtype": "bf16", "data": "synthetic", "config": {"model": f"{args.layers.capitalize()} beside Qwen3", **res},
           "gpu_launches": int(ops.COUNTERS["launches"]), "clocks": clocks})
 
 
@@ -678,8 +678,8 @@ def main():
     ap.add_argument("--check", action="store_true",
                     help="instead of timing: first tokens under --gpus N against the same prompts on one GPU "
                          "(shrunken config, greedy)")
-    ap.add_argument("--layers", action="store_true",
-                    help="instead of the job: prefill and decode throughput of the hybrid model's layers beside the dense "
+    ap.add_argument("--layers", nargs="?", const="bagedra", default="", choices=["bagedra", "lekilix"],
+                    help="instead of the job: prefill and decode throughput of a hybrid model's layers beside the dense "
                          "decoder at a few equal sizes, and the roofline of their kernels (1 GPU)")
     ap.add_argument("--small", action="store_true", help="--layers: the smallest size only")
     ap.add_argument("--check-out", default="", help=argparse.SUPPRESS)

@@ -100,8 +100,8 @@ def throughput(cfg, steps):
         release(seqs)
     for b, n in DECODE:
         seqs = requests(b, n)
-        for s in seqs:
-            s.append_token(7)
+        for i, s in enumerate(seqs):
+            s.append_token(7 + 11 * i)                  # different ids: they may choose the experts
             bm.may_append(s)
         with torch.cuda.stream(stream):
             r.run_decode(seqs)
@@ -233,6 +233,11 @@ def kernel_table():
         add("delta inputs + step", f"{b} requests",
             lambda: e.delta_rule(p2, none, cw, hv, hv, hn, 1e-6, cs, st, dd, 1e-6, None, lens, slots, 1, None),
             b * H * D * V * 8, like="decode_attention (dense)", like_case=dense)
+    return compare(rows), src
+
+
+def compare(rows):
+    """Adds to every row that names a like kernel how far that one is from its roofline."""
     by = {(r["kernel"], r["case"]): r["of_roofline"] for r in rows}
     for r in rows:
         if r["like"]:
@@ -241,20 +246,24 @@ def kernel_table():
             r["times_as_far"] = round(ref / r["of_roofline"], 2)
         else:
             del r["like"], r["like_case"]
-    return rows, src
+    return rows
 
 
-def run(steps=5, small=False, kernels=True):
+def run(steps=5, small=False, kernels=True, model="bagedra"):
     """The result as one dict (see `bench.py --layers`)."""
+    make, table = hybrid_config, kernel_table
+    if model == "lekilix":
+        from benchmarks import prenorm_bench
+        make, table = prenorm_bench.model_config, prenorm_bench.kernel_table
     sizes = {"2k": SIZES["2k"]} if small else SIZES
     out = {"layers": LAYERS, "sizes": {}}
     for name, size in sizes.items():
-        ours, dense = throughput(hybrid_config(*size), steps), throughput(dense_config(*size), steps)
+        ours, dense = throughput(make(*size), steps), throughput(dense_config(*size), steps)
         for a, b in zip(ours, dense):
             a["dense_ms"], a["dense_tok_s"] = b["ms"], b["tok_s"]
         out["sizes"][name] = {"width": size[0], "heads": size[1], "ff": size[2], "rows": ours}
     if kernels:
-        out["kernels"], out["peaks"] = kernel_table()
+        out["kernels"], out["peaks"] = table()
     return out
 
 

@@ -155,6 +155,34 @@ void linear_glu(const Tensor& h, const Tensor& w, int64_t up, int64_t width, int
   glu(project(h, w, w.size(0), 0, 0, false), 0, up, width, kind, limit, out);
 }
 
+// The add and the norm of linear_add_norm alone, for a stream that is complete already (kernel benchmarks)
+Tensor stream_norm(Tensor x, const Tensor& norm_w, double eps, const Projection* experts, const OptTensor& row_of) {
+  const int64_t T = x.size(0), W = x.size(1);
+  check_f32(x, "residual", T * W);
+  check_f32(norm_w, "norm weight", W);
+  c10::cuda::CUDAGuard guard(x.device());
+  fc::AddNorm n;
+  Tensor h = torch::empty({T, pad8(int(W))}, x.options().dtype(torch::kBFloat16));
+  n.T = int(T);
+  n.W = int(W);
+  n.Wp = pad8(int(W));
+  n.x = x.data_ptr<float>();
+  n.w = norm_w.data_ptr<float>();
+  n.h = h.data_ptr();
+  n.ld_h = n.Wp;
+  n.eps = float(eps);
+  if (experts != nullptr) {
+    TORCH_CHECK(row_of.has_value() && row_of->dim() == 2 && row_of->size(0) == T && experts->cols == n.Wp && !experts->f32,
+                "bad expert outputs");
+    check_i32(*row_of, "row_of", T);
+    n.experts = experts->src;
+    n.row_of = row_of->data_ptr<int>();
+    n.top = int(row_of->size(1));
+  }
+  fc::launch_add_norm(n, false, stream_now());
+  return h;
+}
+
 // x (+)= a @ w.T + mixed expert rows; returns rms(x) * norm_w (or x) in the element type of a
 Tensor linear_add_norm(const Tensor& a, const Tensor& w, Tensor x, const OptTensor& norm_w, double eps, bool add,
                        const Projection* experts, const OptTensor& row_of, const OptTensor& mix, const OptTensor& out) {
@@ -547,6 +575,7 @@ void register_prenorm(pybind11::module_& m) {
   m.def("glu", &glu);
   m.def("linear_glu", &linear_glu);
   m.def("linear_add_norm", &linear_add_norm);
+  m.def("stream_norm", &stream_norm);
   m.def("route_by_table", &route_by_table);
   m.def("experts", &experts);
   m.def("windowed_attention", &windowed_attention);
