@@ -101,6 +101,7 @@ def kernel_table():
     del gu, down, wg, wd
     # ---- windowed attention (norms, rotation, store, attention, gate)
     cols = [H, G, D, 64, WINDOW, 0, H * D, (H + G) * D]
+    freq = hybrid.rope_turns(1e4, 64).cuda()
     qn, kn, sink = torch.ones(H * D, device=dev), torch.ones(G * D, device=dev), torch.zeros(H, device=dev)
     cos_sin = torch.ones(16384, D, device=dev, dtype=torch.float32)
 
@@ -136,7 +137,7 @@ def kernel_table():
         out = torch.empty(t, H * D, device=dev, dtype=bf)
         ctx = (pos + 1).int()
         add(f"norms + store + windowed {kind} attention", case,
-            lambda: e.windowed_attention(pr, cols, D ** -0.5, 1e4, qn, kn, sink, 1e-6, kc, vc, pos, slots, bt, lens, cu,
+            lambda: e.windowed_attention(pr, cols, D ** -0.5, freq, qn, kn, sink, 1e-6, kc, vc, pos, slots, bt, lens, cu,
                                          seq if prefill else None, ctx if prefill else None, n if prefill else 0, 0, out, 0),
             io + t * H * D * 2 + b * min(n, WINDOW) * kv, seen * H * 4 * D, like=f"rope + store + {kind} attention (dense)")
         del kc, vc, qkv

@@ -98,6 +98,7 @@ prefill_attn_tc2_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
   const int tile0 = max(0, offset + q0 - win + 1) / P2_BN;            // tiles before it are out of every row's window
   const int n_a = (kv_end_a + P2_BN - 1) / P2_BN - tile0;
   const int n_b = act_b ? (kv_end_b + P2_BN - 1) / P2_BN - tile0 : 0;
+  const int f_b = max(0, offset + q0 + P2_BM - win + 1) / P2_BN - tile0;   // first tile of B's window (0 or 1; A's is 0)
   const int n_tiles = max(n_a, n_b);
   const int kv_end = max(kv_end_a, kv_end_b);
   const int* bt = p.block_tables + (long long)seq * p.max_blocks;
@@ -201,7 +202,7 @@ prefill_attn_tc2_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
         for (int kk = 0; kk < 8; ++kk) {
           const uint64_t db = p2_sdesc(va + uint32_t(kk) * 2048, P2_SUB_BYTES, 1024);
           tc_mma_f16_ts(tmem_base + 256u + uint32_t(x * 128), tmem_base + uint32_t(x * 128) + uint32_t(kk * 8), db,
-                        idesc_o, (j > 0 || kk > 0) ? 1u : 0u);
+                        idesc_o, (j > (x == 0 ? 0 : f_b) || kk > 0) ? 1u : 0u);
         }
         tc_commit(&o_done[x]);
       };
@@ -209,7 +210,7 @@ prefill_attn_tc2_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
       if (ok) {
         tc_fence_after();
         issue_s(0, 0);
-        if (act_b) issue_s(1, 0);
+        if (act_b && f_b == 0) issue_s(1, 0);
         tc_commit(&k_empty[0]);
       }
       for (int j = 0; j < n_tiles && ok; ++j) {
@@ -217,17 +218,19 @@ prefill_attn_tc2_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
         const bool more = j + 1 < n_tiles;
         bool v_waited = false, k_waited = false;
         for (int x = 0; x < 2 && ok; ++x) {
-          const int n_x = x == 0 ? n_a : n_b;
+          const int n_x = x == 0 ? n_a : n_b, f_x = x == 0 ? 0 : f_b;
           if (j >= n_x) continue;
-          ok = mbar_wait(&p_ready[x], uint32_t(j) & 1u, p.status, ST_TIMEOUT_FULL);
-          if (ok && !v_waited) {
-            ok = mbar_wait(&v_full[st], uint32_t(j >> 1) & 1u, p.status, ST_TIMEOUT_FULL);
-            v_waited = true;
+          if (j >= f_x) {
+            ok = mbar_wait(&p_ready[x], uint32_t(j - f_x) & 1u, p.status, ST_TIMEOUT_FULL);
+            if (ok && !v_waited) {
+              ok = mbar_wait(&v_full[st], uint32_t(j >> 1) & 1u, p.status, ST_TIMEOUT_FULL);
+              v_waited = true;
+            }
+            if (!ok) break;
+            tc_fence_after();
+            issue_pv(x, j);
           }
-          if (!ok) break;
-          tc_fence_after();
-          issue_pv(x, j);
-          if (j + 1 < n_x) {
+          if (j + 1 < n_x && j + 1 >= f_x) {
             if (!k_waited) {
               ok = mbar_wait(&k_full[st ^ 1], uint32_t((j + 1) >> 1) & 1u, p.status, ST_TIMEOUT_FULL);
               k_waited = true;
@@ -246,7 +249,7 @@ prefill_attn_tc2_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
   } else {
     // ------------------------------------------------ softmax of one query tile (x = 0: A, 1: B)
     const int x = (warp - 2) >> 2;
-    const int n_x = x == 0 ? n_a : n_b;
+    const int n_x = x == 0 ? n_a : n_b, f_x = x == 0 ? 0 : f_b;
     const int kv_end_x = x == 0 ? kv_end_a : kv_end_b;
     const int lane_group = warp & 3;                         // TMEM lanes this warp may touch
     const int row = lane_group * 32 + lane;
@@ -257,8 +260,8 @@ prefill_attn_tc2_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
     const int qpos = offset + qrow;                          // last key position this row may see
     float m_ref = -INFINITY, l = 0.f;                        // -inf: no visible key yet
     bool ok = true;
-    for (int j = 0; j < n_x && ok; ++j) {
-      if (*s_abort || !mbar_wait(&s_full[x], uint32_t(j) & 1u, p.status, ST_TIMEOUT_ACC_FULL)) {
+    for (int j = f_x; j < n_x && ok; ++j) {
+      if (*s_abort || !mbar_wait(&s_full[x], uint32_t(j - f_x) & 1u, p.status, ST_TIMEOUT_ACC_FULL)) {
         ok = false;
         break;
       }
@@ -280,11 +283,11 @@ prefill_attn_tc2_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
 #pragma unroll
       for (int t = 0; t < 128; ++t) mx = fmaxf(mx, __uint_as_float(s[t]));
       mx *= p.scale_log2;
-      if (j == 0) {
+      if (j == f_x) {
         m_ref = mx;
       } else if (__any_sync(__activemask(), mx > m_ref + P2_RESCALE_THRESHOLD)) {
         // some row of this warp outgrew its reference: bring O (complete up to tile j - 1) to the new one
-        if (!mbar_wait(&o_done[x], uint32_t(j - 1) & 1u, p.status, ST_TIMEOUT_ACC_FULL)) {
+        if (!mbar_wait(&o_done[x], uint32_t(j - 1 - f_x) & 1u, p.status, ST_TIMEOUT_ACC_FULL)) {
           ok = false;
           break;
         }
@@ -325,7 +328,7 @@ prefill_attn_tc2_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
       l += rs;
     }
     if (!ok) *s_abort = 1;
-    if (ok && n_x > 0 && mbar_wait(&o_done[x], uint32_t(n_x - 1) & 1u, p.status, ST_TIMEOUT_ACC_FULL)) {
+    if (ok && n_x > 0 && mbar_wait(&o_done[x], uint32_t(n_x - 1 - f_x) & 1u, p.status, ST_TIMEOUT_ACC_FULL)) {
       tc_fence_after();
       if (p.opt.sink != nullptr && m_ref != -INFINITY)       // one more term of the denominator, without a value
         l += exp2f(p.opt.sink[h] * 1.4426950408889634f - m_ref);

@@ -131,6 +131,11 @@ __device__ __forceinline__ float glu_t(float g, float u, float limit) {
   return over_one_plus_exp<T>(g, -1.702f * g) * (u + 1.f);
 }
 
+// cos and sin of `position` times a frequency in turns, reduced in double
+__device__ __forceinline__ void turn_angle(double pos, double freq, float& c, float& s) {
+  const double turns = pos * freq;
+  sincospif(float(2.0 * (turns - rint(turns))), &s, &c);
+}
 // cos and sin of position * base^(-2 i / dims): the angle is reduced in double, so that far positions lose nothing
 __device__ __forceinline__ void rope_angle(double pos, double log2_base, int i, int dims, float& c, float& s) {
   const double turns = pos * exp2(-log2_base * (2.0 * i / dims)) * 0.15915494309189535;   // 1 / (2 pi)

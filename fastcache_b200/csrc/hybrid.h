@@ -235,7 +235,7 @@ struct WindowStore {
   int off_q = 0, off_k = 0, off_g = 0;
   const float *q_norm = nullptr, *k_norm = nullptr;            // over the whole projections
   float eps = 0.f;
-  double log2_base = 0.0;
+  const double* freq = nullptr;                                // [rot_dims / 2] turns per position
   const long long* positions = nullptr;
   const int* slots = nullptr;
   void *k_rows = nullptr, *v_rows = nullptr;                   // [blocks, G, block, pitch]

@@ -339,7 +339,7 @@ Projection experts(const Tensor& h, const Tensor& plan, int64_t top, const Tenso
 
 // ------------------------------------------------------------------ windowed attention
 // d: heads, key heads, head size, rotated dimensions, window, first columns of q, k, gate.  impl: 0 choose, 1 general
-void windowed_attention(const Projection& pr, const std::vector<int64_t>& d, double scale, double base, const Tensor& q_norm,
+void windowed_attention(const Projection& pr, const std::vector<int64_t>& d, double scale, const Tensor& freq, const Tensor& q_norm,
                         const Tensor& k_norm, const Tensor& sink, double eps, Tensor k_rows, Tensor v_rows,
                         const Tensor& positions, const Tensor& slots, const Tensor& block_tables, const Tensor& ctx,
                         const OptTensor& cu_q, const OptTensor& row_seq, const OptTensor& row_ctx, int64_t max_q,
@@ -360,6 +360,8 @@ void windowed_attention(const Projection& pr, const std::vector<int64_t>& d, dou
   check_f32(q_norm, "query norm", (int64_t)H * D);
   check_f32(k_norm, "key norm", (int64_t)G * D);
   check_f32(sink, "sink", H);
+  TORCH_CHECK(freq.is_cuda() && freq.scalar_type() == torch::kFloat64 && freq.is_contiguous() && freq.numel() == rot / 2,
+              "freq must be float64 [rotated dimensions / 2]");
   check_i32(slots, "slot map", T);
   check_i32(ctx, "context lengths", B);
   TORCH_CHECK(positions.is_cuda() && positions.scalar_type() == torch::kInt64 && positions.is_contiguous() &&
@@ -385,7 +387,7 @@ void windowed_attention(const Projection& pr, const std::vector<int64_t>& d, dou
   st.q_norm = q_norm.data_ptr<float>();
   st.k_norm = k_norm.data_ptr<float>();
   st.eps = float(eps);
-  st.log2_base = std::log2(base);
+  st.freq = freq.data_ptr<double>();
   st.positions = reinterpret_cast<const long long*>(positions.data_ptr<int64_t>());
   st.slots = slots.data_ptr<int>();
   st.k_rows = k_rows.data_ptr();

@@ -88,8 +88,9 @@ post_norm_add_kernel(const ProjSrc y, const T* __restrict__ bias, float* __restr
   for (int c = W + threadIdx.x; c < Wp; c += RS_THREADS) h[row * Wp + c] = Elem<T>::put(0.f);
 }
 
-// x (+)= y + mixed expert rows;  h = rms(x) * w (or x) in the model's type, zero-padded from W to Wp columns
-template <typename T, bool VEC>
+// x (+)= y + mixed expert rows;  h = rms(x) * w (or x) in the model's type, zero-padded from W to Wp columns.  NC: 4-column
+// chunks per thread
+template <typename T, bool VEC, int NC>
 __global__ void __launch_bounds__(RS_THREADS)
 add_norm_kernel(const AddNorm p, const ProjSrc y, int has_y) {
   __shared__ float red[RS_THREADS / 32];
@@ -99,64 +100,77 @@ add_norm_kernel(const AddNorm p, const ProjSrc y, int has_y) {
   const int W = p.W;
   float* x = p.x + row * W;
   T* h = reinterpret_cast<T*>(p.h) + row * p.ld_h;
-  float v[RS_CHUNKS][4];
+  auto col_of = [&](int c) { return (int(threadIdx.x) + c * RS_THREADS) * 4; };
+  float4 v[NC];
+#pragma unroll
+  for (int c = 0; c < NC; ++c) {
+    const int col = col_of(c);
+    v[c] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (!p.add || col >= W) continue;
+    if (VEC) {
+      v[c] = __ldcg(reinterpret_cast<const float4*>(x + col));
+    } else {
+      v[c].x = x[col];
+      if (col + 1 < W) v[c].y = x[col + 1];
+      if (col + 2 < W) v[c].z = x[col + 2];
+      if (col + 3 < W) v[c].w = x[col + 3];
+    }
+  }
+  auto add4 = [&](int c, const float4& a, float f) {
+    v[c].x = fmaf(a.x, f, v[c].x);
+    v[c].y = fmaf(a.y, f, v[c].y);
+    v[c].z = fmaf(a.z, f, v[c].z);
+    v[c].w = fmaf(a.w, f, v[c].w);
+  };
+  if (has_y)
+#pragma unroll
+    for (int c = 0; c < NC; ++c)
+      if (col_of(c) < W) add4(c, proj_at4<T>(y, row, col_of(c)), 1.f);     // pad columns of a projection exist and are zero
+  for (int j = 0; j < p.top; ++j) {
+    const int r = p.row_of[row * p.top + j];
+    if (r < 0) continue;
+    const float f = p.mix != nullptr ? p.mix[row * p.top + j] : 1.f / float(p.top);
+    float4 e[NC];
+#pragma unroll
+    for (int c = 0; c < NC; ++c)
+      if (col_of(c) < W) e[c] = proj_at4<T>(p.experts, r, col_of(c));
+#pragma unroll
+    for (int c = 0; c < NC; ++c)
+      if (col_of(c) < W) add4(c, e[c], f);
+  }
+  const bool changed = has_y || p.top > 0;
   float ss = 0.f;
 #pragma unroll
-  for (int c = 0; c < RS_CHUNKS; ++c) {
-    const int col = (threadIdx.x + c * RS_THREADS) * 4;
+  for (int c = 0; c < NC; ++c) {
+    const int col = col_of(c);
     if (col >= W) continue;
-    float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (has_y) a = proj_at4<T>(y, row, col);             // the pad columns of a projection exist and are zero
-    v[c][0] = a.x;
-    v[c][1] = a.y;
-    v[c][2] = a.z;
-    v[c][3] = a.w;
-    for (int j = 0; j < p.top; ++j) {
-      const int r = p.row_of[row * p.top + j];
-      if (r < 0) continue;
-      const float4 e = proj_at4<T>(p.experts, r, col);
-      const float f = p.mix != nullptr ? p.mix[row * p.top + j] : 1.f / float(p.top);
-      v[c][0] = fmaf(e.x, f, v[c][0]);
-      v[c][1] = fmaf(e.y, f, v[c][1]);
-      v[c][2] = fmaf(e.z, f, v[c][2]);
-      v[c][3] = fmaf(e.w, f, v[c][3]);
-    }
     if (VEC) {
-      if (p.add) {
-        const float4 o = *reinterpret_cast<const float4*>(x + col);
-        v[c][0] += o.x;
-        v[c][1] += o.y;
-        v[c][2] += o.z;
-        v[c][3] += o.w;
-      }
-      if (has_y || p.top > 0) *reinterpret_cast<float4*>(x + col) = make_float4(v[c][0], v[c][1], v[c][2], v[c][3]);
+      if (changed) *reinterpret_cast<float4*>(x + col) = v[c];
     } else {
-#pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        if (col + i >= W) {
-          v[c][i] = 0.f;
-          continue;
-        }
-        if (p.add) v[c][i] += x[col + i];
-        x[col + i] = v[c][i];
-      }
+      if (col + 1 >= W) v[c].y = 0.f;
+      if (col + 2 >= W) v[c].z = 0.f;
+      if (col + 3 >= W) v[c].w = 0.f;
+      x[col] = v[c].x;
+      if (col + 1 < W) x[col + 1] = v[c].y;
+      if (col + 2 < W) x[col + 2] = v[c].z;
+      if (col + 3 < W) x[col + 3] = v[c].w;
     }
-#pragma unroll
-    for (int i = 0; i < 4; ++i) ss += v[c][i] * v[c][i];
+    ss += v[c].x * v[c].x + v[c].y * v[c].y + v[c].z * v[c].z + v[c].w * v[c].w;
   }
   const bool norm = p.w != nullptr;
   const float inv = norm ? rsqrtf(cta_sum<RS_THREADS>(ss, red) / float(W) + p.eps) : 1.f;
 #pragma unroll
-  for (int c = 0; c < RS_CHUNKS; ++c) {
-    const int col = (threadIdx.x + c * RS_THREADS) * 4;
+  for (int c = 0; c < NC; ++c) {
+    const int col = col_of(c);
     if (col >= W) continue;
     if (VEC) {
       const float4 w = norm ? *reinterpret_cast<const float4*>(p.w + col) : make_float4(1.f, 1.f, 1.f, 1.f);
-      store4(h + col, v[c][0] * inv * w.x, v[c][1] * inv * w.y, v[c][2] * inv * w.z, v[c][3] * inv * w.w);
+      store4(h + col, v[c].x * inv * w.x, v[c].y * inv * w.y, v[c].z * inv * w.z, v[c].w * inv * w.w);
     } else {
+      const float a[4] = {v[c].x, v[c].y, v[c].z, v[c].w};
 #pragma unroll
       for (int i = 0; i < 4; ++i)
-        if (col + i < W) h[col + i] = Elem<T>::put(v[c][i] * inv * (norm ? p.w[col + i] : 1.f));
+        if (col + i < W) h[col + i] = Elem<T>::put(a[i] * inv * (norm ? p.w[col + i] : 1.f));
     }
   }
   for (int c = W + threadIdx.x; c < p.Wp; c += RS_THREADS) h[c] = Elem<T>::put(0.f);
@@ -280,12 +294,18 @@ void launch_add_norm(const AddNorm& p, bool f32, cudaStream_t s) {
   const ProjSrc y = p.y != nullptr ? *p.y : ProjSrc();
   const int has_y = p.y != nullptr ? 1 : 0;
   auto go = [&](auto kern) { launch_pdl(PDL_NORM, kern, dim3(p.T), dim3(RS_THREADS), 0, s, p, y, has_y); };
-  if (f32) {
-    if (p.W % 4 == 0) go(add_norm_kernel<float, true>);
-    else go(add_norm_kernel<float, false>);
+  const int chunks = (p.W + RS_THREADS * 4 - 1) / (RS_THREADS * 4);
+  if (p.W % 4 != 0) {
+    if (f32) go(add_norm_kernel<float, false, RS_CHUNKS>);
+    else go(add_norm_kernel<bf16, false, RS_CHUNKS>);
+  } else if (f32) {
+    go(add_norm_kernel<float, true, RS_CHUNKS>);
+  } else if (chunks <= 2) {
+    go(add_norm_kernel<bf16, true, 2>);
+  } else if (chunks <= 4) {
+    go(add_norm_kernel<bf16, true, 4>);
   } else {
-    if (p.W % 4 == 0) go(add_norm_kernel<bf16, true>);
-    else go(add_norm_kernel<bf16, false>);
+    go(add_norm_kernel<bf16, true, RS_CHUNKS>);
   }
   check_launch("add + norm");
 }

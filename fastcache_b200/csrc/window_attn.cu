@@ -11,11 +11,10 @@
 namespace fc {
 
 using bf16 = __nv_bfloat16;
-constexpr int WS_THREADS = 256;
 
 // One CTA per token.  The projections are staged in shared memory as fp32 while their squares are summed; VEC: four
 // columns at a time (head size, pitch and offsets multiples of 4).
-template <typename T, bool VEC>
+template <typename T, bool VEC, int WS_THREADS>
 __global__ void __launch_bounds__(WS_THREADS)
 window_store_kernel(const WindowStore p) {
   __shared__ float red[WS_THREADS / 32];
@@ -30,7 +29,7 @@ window_store_kernel(const WindowStore p) {
   T* out = reinterpret_cast<T*>(p.out);
   if (tid < p.pad_out) out[t * p.ld_out + nq + tid] = Elem<T>::put(0.f);
   const double pos = double(p.positions[t]);
-  for (int i = tid; i < half; i += WS_THREADS) rope_angle(pos, p.log2_base, i, p.rot_dims, cs[i].x, cs[i].y);
+  for (int i = tid; i < half; i += WS_THREADS) turn_angle(pos, p.freq[i], cs[i].x, cs[i].y);
   float sq = 0.f, sk = 0.f;
   if (VEC) {
     for (int i = tid * 4; i < nq; i += WS_THREADS * 4) {
@@ -194,12 +193,13 @@ static void window_store_t(const WindowStore& p, cudaStream_t s) {
   const size_t smem = size_t((n + 3) / 4 * 4 + p.rot_dims) * 4;
   if (smem > 200 * 1024) throw std::runtime_error("windowed attention: query and key projections are limited to 50000 columns");
   const bool vec = p.D % 4 == 0 && p.pitch % 4 == 0 && p.off_q % 4 == 0 && p.off_k % 4 == 0 && p.off_g % 4 == 0;
-  auto go = [&](auto kern) {
+  auto go = [&](auto kern, int threads) {
     if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem));
-    launch_pdl(PDL_ROPE, kern, dim3(p.T), dim3(WS_THREADS), smem, s, p);
+    launch_pdl(PDL_ROPE, kern, dim3(p.T), dim3(threads), smem, s, p);
   };
-  if (vec) go(window_store_kernel<T, true>);
-  else go(window_store_kernel<T, false>);
+  if (vec && p.T <= 148) go(window_store_kernel<T, true, 1024>, 1024);      // one row per SM at most
+  else if (vec) go(window_store_kernel<T, true, 256>, 256);
+  else go(window_store_kernel<T, false, 256>, 256);
 }
 void launch_window_store(const WindowStore& p, bool f32, cudaStream_t s) {
   if (p.T == 0) return;

@@ -43,6 +43,8 @@ class WindowedAttention(nn.Module):
         self.q_norm = fp32_vector(heads * dim)
         self.k_norm = fp32_vector(kv_heads * dim)
         self.sink = fp32_vector(heads)
+        freq = ops.hybrid.rope_turns(rope_base, rope_dims)
+        self.register_buffer("freq", freq.to(self.sink.device), persistent=False)
         self.vectors = {"q.norm": "q_norm", "k.norm": "k_norm", "sink": "sink"}       # checkpoint name -> parameter
 
     def bind(self, offset: Dict[str, int]) -> None:
@@ -53,5 +55,5 @@ class WindowedAttention(nn.Module):
         return LayerCache(PassCache(), kv=(self.kv_heads, padded_dim(self.dim)))
 
     def forward(self, positions: torch.Tensor, p, cache: PassCache, out: torch.Tensor) -> None:
-        ops.hybrid.windowed_attention(p, self.dims, self.q_norm, self.k_norm, self.sink, self.eps, cache.k_rows,
+        ops.hybrid.windowed_attention(p, self.dims, self.freq, self.q_norm, self.k_norm, self.sink, self.eps, cache.k_rows,
                                       cache.v_rows, positions, get_context(), out)

@@ -6,6 +6,7 @@ in 32-bit); the residual stream, the recurrent states and the small per-head vec
 """
 from __future__ import annotations
 
+import math
 from dataclasses import dataclass
 from typing import Optional
 
@@ -269,11 +270,18 @@ def experts(h, route, weights, w_gate_up, w_down, ff: int, spec: GluSpec):
 ATTN_IMPL = 0           # tests: 1 the general kernel also where a tensor-core form exists
 
 
-def windowed_attention(p, d: WindowDims, q_norm, k_norm, sink, eps: float, k_rows, v_rows, positions, ctx, out):
-    """Norm over the whole projection, rotation, cache store, attention with a sink and output gate, to `out`."""
+def rope_turns(base: float, dims: int):
+    """Rotation frequencies in turns per position, float64."""
+    i = torch.arange(dims // 2, dtype=torch.float64)
+    return float(base) ** (-2 * i / max(1, dims)) / (2 * math.pi)
+
+
+def windowed_attention(p, d: WindowDims, freq, q_norm, k_norm, sink, eps: float, k_rows, v_rows, positions, ctx, out):
+    """Norm over the whole projection, rotation (`freq`: rope_turns), cache store, attention with a sink and output gate, to
+    `out`."""
     if out.is_cuda:
         _n(2)
-        ext().windowed_attention(p, [d.heads, d.kv_heads, d.dim, d.rot_dims, d.window, d.q, d.k, d.g], d.scale, d.base,
+        ext().windowed_attention(p, [d.heads, d.kv_heads, d.dim, d.rot_dims, d.window, d.q, d.k, d.g], d.scale, freq,
                                  q_norm, k_norm, sink, float(eps), k_rows, v_rows, positions, ctx.slot_mapping,
                                  ctx.block_tables, ctx.context_lens, ctx.cu_seqlens_q, ctx.row_seq, ctx.row_ctx,
                                  int(ctx.max_seqlen_q), int(ctx.max_seqlen_k), out, ATTN_IMPL)
