@@ -121,8 +121,9 @@ prefill_attn_tc2_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
     tma_prefetch_desc(&tm_v);
   }
   // V rows past the visible keys are never loaded; 0 * (uninitialised bits) must not produce NaN
-  for (int i = threadIdx.x; i < 2 * P2_TILE_BYTES / 16; i += P2_THREADS)
-    reinterpret_cast<uint4*>(s_v)[i] = make_uint4(0, 0, 0, 0);
+  if (kv_end % P2_BN != 0)
+    for (int i = threadIdx.x; i < 2 * P2_TILE_BYTES / 16; i += P2_THREADS)
+      reinterpret_cast<uint4*>(s_v)[i] = make_uint4(0, 0, 0, 0);
   fence_proxy_async();
   if (warp == 1) {
     tmem_alloc(tmem_slot, 512);
@@ -340,7 +341,14 @@ prefill_attn_tc2_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
 #pragma unroll 1
       for (int c = 0; c < D / 32; ++c) {
         uint32_t r[32];
+        uint4 gates[4];                                      // requested before the wait for the accumulator
         tmem_ld_32x32(to + uint32_t(c * 32), r);
+        if (gate != nullptr && qrow < q_len && (dim & 7) == 0) {
+#pragma unroll
+          for (int q = 0; q < 4; ++q)
+            if (c * 32 + q * 8 < dim) gates[q] = *reinterpret_cast<const uint4*>(gate + c * 32 + q * 8);
+        }
+        __syncwarp();
         tmem_ld_wait();
         if (qrow < q_len && (dim & 7) == 0) {
 #pragma unroll
@@ -351,7 +359,7 @@ prefill_attn_tc2_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
 #pragma unroll
             for (int e = 0; e < 8; ++e) v[e] = __uint_as_float(r[q * 8 + e]) * inv;
             if (gate != nullptr) {
-              const uint4 gu = *reinterpret_cast<const uint4*>(gate + col);
+              const uint4 gu = gates[q];
               const uint32_t gw[4] = {gu.x, gu.y, gu.z, gu.w};
 #pragma unroll
               for (int e = 0; e < 4; ++e) {

@@ -17,7 +17,7 @@ using bf16 = __nv_bfloat16;
 template <typename T, bool VEC, int WS_THREADS>
 __global__ void __launch_bounds__(WS_THREADS)
 window_store_kernel(const WindowStore p) {
-  __shared__ float red[WS_THREADS / 32];
+  __shared__ float2 red[WS_THREADS / 32];
   extern __shared__ __align__(16) float sm[];
   const int nq = p.H * p.D, nk = p.G * p.D, half = p.rot_dims / 2;
   float *s_q = sm, *s_k = sm + nq;
@@ -29,9 +29,9 @@ window_store_kernel(const WindowStore p) {
   T* out = reinterpret_cast<T*>(p.out);
   if (tid < p.pad_out) out[t * p.ld_out + nq + tid] = Elem<T>::put(0.f);
   const double pos = double(p.positions[t]);
-  for (int i = tid; i < half; i += WS_THREADS) turn_angle(pos, p.freq[i], cs[i].x, cs[i].y);
   float sq = 0.f, sk = 0.f;
   if (VEC) {
+#pragma unroll 4
     for (int i = tid * 4; i < nq; i += WS_THREADS * 4) {
       const float4 v = proj_at4<T>(p.proj, t, p.off_q + i);
       *reinterpret_cast<float4*>(s_q + i) = v;
@@ -60,8 +60,18 @@ window_store_kernel(const WindowStore p) {
       sk += v * v;
     }
   }
-  const float iq = rsqrtf(cta_sum<WS_THREADS>(sq, red) / float(nq) + p.eps);
-  const float ik = rsqrtf(cta_sum<WS_THREADS>(sk, red) / float(nk) + p.eps);
+  for (int i = tid; i < half; i += WS_THREADS) turn_angle(pos, p.freq[i], cs[i].x, cs[i].y);
+  sq = warp_sum(sq);
+  sk = warp_sum(sk);
+  if ((tid & 31) == 0) red[tid >> 5] = make_float2(sq, sk);
+  __syncthreads();
+  sq = sk = 0.f;
+#pragma unroll
+  for (int i = 0; i < WS_THREADS / 32; ++i) {
+    sq += red[i].x;
+    sk += red[i].y;
+  }
+  const float iq = rsqrtf(sq / float(nq) + p.eps), ik = rsqrtf(sk / float(nk) + p.eps);
   // column c of a head whose first element is x[0] and norm weight w[0]
   auto turned = [&](const float* x, const float* w, int c, float inv) {
     const float v = x[c] * inv * w[c];
