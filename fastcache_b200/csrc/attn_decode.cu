@@ -18,7 +18,7 @@
 // byte), so the legacy tensor path is enough to keep the memory system busy; the
 // tcgen05 path is used where the work is compute-bound.
 //
-// Options for other designs (AttnOptions): a sliding window (tiles before it are not read), a sink per head (one more
+// Options for other designs (AttnOptions): a sliding window or chunks (tiles before them are not read), a soft cap, a sink per head (one more
 // term of the denominator, added where the splits end up), heads narrower than the rows of the pool, and a gate that
 // multiplies the output.
 #include <cuda_bf16.h>
@@ -29,6 +29,7 @@
 #include <stdexcept>
 #include <string>
 
+#include "attn_options.cuh"
 #include "gemm.h"
 #include "kernels.h"
 #include "launch.h"
@@ -135,7 +136,8 @@ decode_attn_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_consta
   const int g = lane >> 2, t = lane & 3;
 
   const int ctx = context_lens[b];
-  const int first = opt.window > 0 ? max(0, ctx - opt.window) : 0;      // first visible row
+  const int first = attn_first(opt, max(ctx - 1, 0));                   // first visible row
+  const ScoreScale sscale = score_scale(opt, scale_log2);
   const int tile_first = first / DEC_TILE, tile_end = (ctx + DEC_TILE - 1) / DEC_TILE;
   const int tiles_per = (tile_end - tile_first + splits - 1) / splits;
   const int tile0 = tile_first + split * tiles_per;
@@ -244,8 +246,8 @@ decode_attn_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_consta
           sc[n][e] = -INFINITY;
           sc[n][2 + e] = -INFINITY;
         } else {
-          sc[n][e] *= scale_log2;
-          sc[n][2 + e] *= scale_log2;
+          sc[n][e] = scaled_score(sscale, sc[n][e]);
+          sc[n][2 + e] = scaled_score(sscale, sc[n][2 + e]);
         }
         mx0 = fmaxf(mx0, sc[n][e]);
         mx1 = fmaxf(mx1, sc[n][2 + e]);

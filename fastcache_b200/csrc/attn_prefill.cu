@@ -16,6 +16,7 @@
 #include <stdexcept>
 #include <string>
 
+#include "attn_options.cuh"
 #include "kernels.h"
 #include "mma.cuh"
 #include "ptx.cuh"
@@ -54,7 +55,7 @@ prefill_attn_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_cache
   const int g = lane >> 2, t = lane & 3;
 
   const int kv_end = min(kv_len, offset + q0 + PF_BM);      // keys visible to this q tile
-  const int tile0 = opt.window > 0 ? max(0, offset + q0 - opt.window + 1) / PF_BN : 0;      // tiles before the window
+  const int tile0 = attn_first(opt, offset + q0) / PF_BN;   // no row sees a tile before it
   const int n_tiles = (kv_end + PF_BN - 1) / PF_BN - tile0;
 
   // ---- Q tile -> smem
@@ -100,6 +101,9 @@ prefill_attn_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_cache
   uint32_t qa[D / 16][4];
   const int qrow0 = offset + q0 + warp * 16 + g;             // kv position of this thread's first row
   const int qrow1 = qrow0 + 8;
+  const int first0 = attn_first(opt, qrow0), first1 = attn_first(opt, qrow1);
+  const int first_last = attn_first(opt, offset + q0 + warp * 16 + 15);    // of the warp's last row
+  const ScoreScale sscale = score_scale(opt, scale_log2);
 
   for (int it = 0; it < n_tiles; ++it) {
     if (it + 1 < n_tiles) load_tile(it + 1, (it + 1) & 1);
@@ -136,19 +140,18 @@ prefill_attn_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_cache
     }
     // ---- scale, causal mask (only tiles that touch the diagonal or the end), row max
     const int col0 = (tile0 + it) * PF_BN;
-    const int win = opt.window > 0 ? opt.window : 0x40000000;           // visible: row - col < win
     const bool need_mask = (col0 + PF_BN - 1 > offset + q0 + warp * 16) || (col0 + PF_BN > kv_end) ||
-                           (offset + q0 + warp * 16 + 15 - col0 >= win);
+                           first_last > col0;
     float mx0 = -INFINITY, mx1 = -INFINITY;
 #pragma unroll
     for (int n = 0; n < PF_BN / 8; ++n) {
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
         const int col = col0 + n * 8 + 2 * t + e;
-        float a = sc[n][e] * scale_log2, b = sc[n][2 + e] * scale_log2;
+        float a = scaled_score(sscale, sc[n][e]), b = scaled_score(sscale, sc[n][2 + e]);
         if (need_mask) {
-          if (col > qrow0 || col >= kv_end || qrow0 - col >= win) a = -INFINITY;
-          if (col > qrow1 || col >= kv_end || qrow1 - col >= win) b = -INFINITY;
+          if (col > qrow0 || col >= kv_end || col < first0) a = -INFINITY;
+          if (col > qrow1 || col >= kv_end || col < first1) b = -INFINITY;
         }
         sc[n][e] = a;
         sc[n][2 + e] = b;

@@ -15,8 +15,8 @@
 //                back as P.  O is rescaled only when a row maximum grows by more than 2^8 over the
 //                reference (all lanes of the warp then rescale their O row in tensor memory), so
 //                most tiles never touch O; the reference maximum cancels in O / l at the end.
-// Options (AttnOptions): a sliding window (key tiles before the first query's window are skipped), a sink per head, heads
-// narrower than the pool's rows, an output gate.
+// Options (AttnOptions): a sliding window or chunks (key tiles that a query tile does not see are skipped), a soft cap of the
+// scores, a sink per head, heads narrower than the pool's rows, an output gate.
 #include <cuda.h>
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
@@ -25,6 +25,7 @@
 #include <stdexcept>
 #include <string>
 
+#include "attn_options.cuh"
 #include "gemm.h"
 #include "kernels.h"
 #include "ptx.cuh"
@@ -94,11 +95,11 @@ prefill_attn_tc2_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
   // keys visible to each query tile, in tiles of 128
   const int kv_end_a = min(kv_len, offset + q0 + P2_BM);
   const int kv_end_b = act_b ? min(kv_len, offset + q0 + 2 * P2_BM) : 0;
-  const int win = p.opt.window > 0 ? p.opt.window : 0x40000000;       // visible: row - key < win
-  const int tile0 = max(0, offset + q0 - win + 1) / P2_BN;            // tiles before it are out of every row's window
+  const int tile0 = attn_first(p.opt, offset + q0) / P2_BN;           // no row sees a tile before it
   const int n_a = (kv_end_a + P2_BN - 1) / P2_BN - tile0;
   const int n_b = act_b ? (kv_end_b + P2_BN - 1) / P2_BN - tile0 : 0;
-  const int f_b = max(0, offset + q0 + P2_BM - win + 1) / P2_BN - tile0;   // first tile of B's window (0 or 1; A's is 0)
+  // first tile that B sees (A's is 0); never past the one after A's last, so that every tile has a reader
+  const int f_b = attn_first(p.opt, offset + q0 + P2_BM) / P2_BN - tile0;
   const int n_tiles = max(n_a, n_b);
   const int kv_end = max(kv_end_a, kv_end_b);
   const int* bt = p.block_tables + (long long)seq * p.max_blocks;
@@ -259,6 +260,9 @@ prefill_attn_tc2_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
     const uint32_t to = tmem_base + lane_addr + 256u + uint32_t(x * 128);    // O_x
     const int qrow = q0 + x * P2_BM + row;                   // row among the sequence's new tokens
     const int qpos = offset + qrow;                          // last key position this row may see
+    const int first = attn_first(p.opt, qpos), first_last = attn_first(p.opt, offset + q0 + x * P2_BM + P2_BM - 1);
+    const ScoreScale sscale = score_scale(p.opt, p.scale_log2);
+    const float scale_log2 = sscale.cap ? 1.f : p.scale_log2;            // capped scores are in log2 units already
     float m_ref = -INFINITY, l = 0.f;                        // -inf: no visible key yet
     bool ok = true;
     for (int j = f_x; j < n_x && ok; ++j) {
@@ -273,9 +277,21 @@ prefill_attn_tc2_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
       tmem_ld_wait();
       const int col0 = (tile0 + j) * P2_BN;
       const bool need_mask = (col0 + P2_BN - 1 > offset + q0 + x * P2_BM) || (col0 + P2_BN > kv_end_x) ||
-                             (offset + q0 + x * P2_BM + P2_BM - 1 - col0 >= win);
+                             first_last > col0;
+      if (sscale.cap) {
+        float top = 0.f;
+#pragma unroll
+        for (int t = 0; t < 128; ++t) top = fmaxf(top, fabsf(__uint_as_float(s[t])));
+        if (__any_sync(__activemask(), top * sscale.in > TANH_POLY_MAX)) {
+#pragma unroll
+          for (int t = 0; t < 128; ++t) s[t] = __float_as_uint(sscale.out * tanh_exp(__uint_as_float(s[t]) * sscale.in));
+        } else {
+#pragma unroll
+          for (int t = 0; t < 128; ++t) s[t] = __float_as_uint(sscale.out * tanh_poly(__uint_as_float(s[t]) * sscale.in));
+        }
+      }
       if (need_mask) {
-        const int hi = min(qpos, kv_end_x - 1) - col0, lo = qpos - win + 1 - col0;     // visible columns of the tile
+        const int hi = min(qpos, kv_end_x - 1) - col0, lo = first - col0;     // visible columns of the tile
 #pragma unroll
         for (int t = 0; t < 128; ++t)
           if (t > hi || t < lo) s[t] = 0xff800000u;                                     // -inf
@@ -283,7 +299,7 @@ prefill_attn_tc2_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
       float mx = -INFINITY;
 #pragma unroll
       for (int t = 0; t < 128; ++t) mx = fmaxf(mx, __uint_as_float(s[t]));
-      mx *= p.scale_log2;
+      mx *= scale_log2;
       if (j == f_x) {
         m_ref = mx;
       } else if (__any_sync(__activemask(), mx > m_ref + P2_RESCALE_THRESHOLD)) {
@@ -314,8 +330,8 @@ prefill_attn_tc2_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
 #pragma unroll
       for (int t = 0; t < 64; ++t) {
         float e0, e1;
-        const float a0 = fmaf(__uint_as_float(s[2 * t]), p.scale_log2, -base);
-        const float a1 = fmaf(__uint_as_float(s[2 * t + 1]), p.scale_log2, -base);
+        const float a0 = fmaf(__uint_as_float(s[2 * t]), scale_log2, -base);
+        const float a1 = fmaf(__uint_as_float(s[2 * t + 1]), scale_log2, -base);
         asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e0) : "f"(a0));
         asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e1) : "f"(a1));
         rs += e0 + e1;

@@ -1,5 +1,5 @@
 // Launchers of the hybrid-model kernels: norms on an fp32 residual stream and gated activations (resid.cu), recurrent
-// layers (recurrence.cu, recurrence_chunk.cu), latent attention (latent.cu, latent_decode.cu, latent_prefill.cu),
+// layers (recurrence.cu, recurrence_chunk.cu, lru.cu), residual streams (streams.cu), latent attention (latent.cu, latent_decode.cu, latent_prefill.cu),
 // windowed attention (window_attn.cu, with the attn_*.cu kernels), experts (moe.cu, moe_gemm.cu) and the CUDA-core GEMM of
 // 32-bit runs (linear_simt.cu).
 //
@@ -40,6 +40,7 @@ struct SimtLinear {
   long long gx = 0, gw = 0, gy = 0;           // offsets between groups
   ProjSrc gate;                               // p == part == nullptr: no gate
   int gate_off = 0;
+  bool y_f32 = false;                         // y holds fp32 whatever the element type
   const int* group_rows = nullptr;            // [groups + 1]: group g has the rows [g, g + 1) of x and y (gx, gy unused)
   int y_pad = 0;                              // columns [groups * N, y_pad) of y are zeroed (groups stored side by side)
 };
@@ -85,6 +86,30 @@ struct GluMul {
 void launch_glu_mul(const GluMul& p, bool f32, cudaStream_t s);
 void launch_gelu_mul(const ProjSrc& gu, const void* bias, void* out, int T, int up_off, int width, int width_p,
                      bool f32, cudaStream_t s);
+
+// ---- streams.cu: S residual streams x [T, S, W]
+constexpr int STREAM_MAX = 16, STREAM_MAX_WIDTH = 8192;
+// x_t <- sum_s mix[s, t] x_s + out[t] (y + sum_j mix_j experts[row_of_j]);  h = layer norm of sum_t in[t] x_t
+struct StreamMix {
+  int T = 0, S = 0, W = 0, Wp = 0;
+  bool has_y = false;
+  ProjSrc y;
+  float* x = nullptr;
+  const float* connection = nullptr; // this sublayer's [in (S) | out (S) | mix (S * S, from * S + to)]
+  const float* next = nullptr;       // the next one's; nullptr: plain sum, the streams are not written
+  const float *w = nullptr, *b = nullptr;     // the layer norm's
+  void* h = nullptr;                 // [T, ld_h], columns [W, Wp) are zeroed
+  long long ld_h = 0;
+  float eps = 0.f;
+  ProjSrc experts;                   // as in AddNorm
+  const int* row_of = nullptr;
+  const float* mix = nullptr;
+  int top = 0;
+};
+void launch_stream_mix(const StreamMix& p, bool f32, cudaStream_t s);
+// table [vocab, Wp]; connection, y and experts unused
+void launch_embed_streams(const StreamMix& p, const void* ids, const void* table, long long vocab, bool f32, uint32_t* status,
+                          cudaStream_t s);
 
 // ---- recurrence.cu
 struct StepParams {
@@ -158,6 +183,39 @@ void launch_gla_chunk(const StepParams& p, int max_len, cudaStream_t s);
 void launch_delta_chunk(const StepParams& p, int max_len, cudaStream_t s);
 void launch_memory_chunk(const StepParams& p, int max_len, cudaStream_t s);
 
+// ---- lru.cu: real-gated linear recurrent unit, state [slots, C]
+struct LruParams {
+  int T = 0, C = 0, blocks = 1, taps = 1;
+  RunBatch runs;
+  const int* row_seq = nullptr;      // request of every row (nullptr: row b belongs to request b)
+  ProjSrc x, y;                      // branches; y: `gelu` tells whether the activation is still to be applied
+  int off_x = 0, off_y = 0;
+  bool gelu = true;
+  const void *bias_x = nullptr, *bias_y = nullptr;   // [C]; y's is added where gelu is
+  const float *conv_w = nullptr, *conv_b = nullptr;  // [C, taps], [C]
+  float* conv_state = nullptr;       // [slots, taps - 1, C]: the last inputs
+  const void* gate_w = nullptr;      // [2, blocks, n, n]
+  const float* gate_b = nullptr;     // [2, C]
+  const float* lam = nullptr;        // [C]
+  float sharpness = 8.f;
+  float* state = nullptr;
+  void* u = nullptr;                 // [T, C] convolution output
+  const float* z = nullptr;          // general form: gate logits without bias [T, 2, C]
+  void* out = nullptr;
+  long long ld_out = 0;
+  int pad_out = 0;                   // columns after C that are zeroed
+  float* agg = nullptr;              // scratch of the scan in segments [B, segments, 2, C]
+  int max_len = 1;
+  uint32_t* status = nullptr;
+};
+// u; runs of one row (runs.cu == nullptr) also advance conv_state, longer ones leave it to the scan
+void launch_lru_conv(const LruParams& p, bool f32, cudaStream_t s);
+void launch_lru_scan(const LruParams& p, bool f32, cudaStream_t s);        // general: gates from z
+bool lru_tc_supported(const LruParams& p);                                 // bf16 forms that make the gates' products
+void launch_lru_step(const LruParams& p, cudaStream_t s);                  // runs of one row
+int lru_segments(const LruParams& p, int num_sms);
+void launch_lru_scan_tc(const LruParams& p, int segments, cudaStream_t s); // runs of any length
+
 // ---- latent.cu
 struct LatentStore {
   int T = 0, H = 0, D = 0, R = 0, rank = 0, rot_dims = 0, V = 0;
@@ -228,11 +286,14 @@ struct LatentPrefill {
 bool latent_prefill_supported(const LatentPrefill& p);
 void launch_latent_prefill(const LatentPrefill& p, cudaStream_t s);
 
-// ---- window_attn.cu: what surrounds attention over per-head K/V rows whose values are the raw keys
+// ---- window_attn.cu: what surrounds attention over per-head K/V rows
 struct WindowStore {
-  int T = 0, H = 0, G = 0, D = 0, pitch = 0, rot_dims = 0;     // pitch: row width of q and of the pools (>= D, zero-padded)
-  ProjSrc proj;
-  int off_q = 0, off_k = 0, off_g = 0;
+  int T = 0, H = 0, G = 0, D = 0, V = 0, pitch = 0, rot_dims = 0;   // pitch: row width of q and of the pools (>= D and V,
+  ProjSrc proj;                                                     // zero-padded)
+  int off_q = 0, off_k = 0, off_v = -1, off_g = 0;             // off_v < 0: the values are the raw keys (V == D)
+  const void* bias = nullptr;                                  // of the packed projection, by column (nullptr: none)
+  bool half = false;                                           // entry i turns with i + rot_dims / 2 (else 2i with 2i + 1)
+  float rot_size = 1.f;                                        // factor of cos and sin
   const float *q_norm = nullptr, *k_norm = nullptr;            // over the whole projections
   float eps = 0.f;
   const double* freq = nullptr;                                // [rot_dims / 2] turns per position
@@ -242,20 +303,21 @@ struct WindowStore {
   int block_size = 0;
   long long num_rows = 0;                                      // blocks * block
   void* q = nullptr;                                           // [T, H, pitch]
-  void* gate = nullptr;                                        // [T, H * D] copy of the gate projection (nullptr: not wanted)
-  void* out = nullptr;                                         // attention output: columns [H * D, + pad_out) are zeroed
+  void* gate = nullptr;                                        // [T, H * V] copy of the gate projection (nullptr: not wanted)
+  void* out = nullptr;                                         // attention output: columns [H * V, + pad_out) are zeroed
   long long ld_out = 0;
   int pad_out = 0;
   uint32_t* status = nullptr;
 };
 void launch_window_store(const WindowStore& p, bool f32, cudaStream_t s);
 struct WindowAttn {                  // the general form: any head size, bf16 or fp32
-  int T = 0, H = 0, G = 0, D = 0, pitch = 0, window = 0, block_size = 0, max_blocks = 0, num_blocks = 0;
+  int T = 0, H = 0, G = 0, D = 0, V = 0, pitch = 0, window = 0, chunk = 0, block_size = 0, max_blocks = 0, num_blocks = 0;
+  float softcap = 0.f;               // window, chunk, softcap: as in AttnOptions
   const void *q = nullptr, *k_rows = nullptr, *v_rows = nullptr;
   const int *block_tables = nullptr, *row_seq = nullptr, *row_ctx = nullptr;      // as in LatentAttn
-  const float* sink = nullptr;
+  const float* sink = nullptr;       // nullptr: none
   ProjSrc gate;
-  int off_g = 0;
+  int off_g = -1;                    // < 0: no gate
   void* out = nullptr;
   long long ld_out = 0;
   float scale = 1.f;
@@ -282,6 +344,22 @@ struct RouteTable {
   uint32_t* status = nullptr;
 };
 void launch_route_table(const RouteTable& p, cudaStream_t s);
+// choice by score: see route_by_score in ops/hybrid.py
+struct RouteScore {
+  ProjSrc logits;                    // fp32 [T, E], first column 0
+  const float* correction = nullptr; // [E]
+  const int* ctx = nullptr;          // as in RouteTable
+  int T = 0, top = 0, E = 0, groups = 1, keep = 1;
+  float* mix = nullptr;              // [T, top] weights
+  int* row_of = nullptr;
+  int* plan = nullptr;
+  int* ids = nullptr;                // scratch [T, top]
+  int* counts = nullptr;             // scratch [route_score_blocks(T), E]
+  int token_at = 0;                  // (set by the launcher)
+};
+constexpr int ROUTE_ROWS = 64;       // tokens per CTA of the large form
+inline int route_score_blocks(int T) { return (T + ROUTE_ROWS - 1) / ROUTE_ROWS; }
+void launch_route_score(const RouteScore& p, cudaStream_t s);
 // decode-size expert products (moe_gemm.cu): partial [splits, pairs, N] of x [pairs, K] and w [E, N, K]; an expert has at
 // most max_rows <= 256 rows
 int moe_skinny_splits(int max_rows, int pairs, int E, int N, int K);

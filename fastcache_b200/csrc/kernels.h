@@ -29,6 +29,8 @@ void launch_sample(const void* logits, const void* temps, void* out, int B, int 
 // Options of the paged attention kernels; the defaults are plain causal attention.
 struct AttnOptions {
   int window = 0;                  // positions a query sees, itself included (0: all up to itself)
+  int chunk = 0;                   // a query sees no key before the last multiple of it (0: no chunks)
+  float softcap = 0.f;             // c > 0: scores become c tanh(score / c)
   const float* sink = nullptr;     // [Hq] fp32: exp(sink) joins the denominator, without key or value
   int dim = 0;                     // columns of a head that are written (0: all); the pool's rows may be wider
   const void* gate = nullptr;      // bf16 [rows, ld_gate]: the output is multiplied by sigmoid(gate)

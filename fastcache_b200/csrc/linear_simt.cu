@@ -62,7 +62,8 @@ linear_simt_kernel(const SimtLinear a) {
       float v = acc[i][j];
       if (bias != nullptr) v += Elem<T>::get(bias[n]);
       if (gated) v *= sigmoid_t<T>(proj_at<T>(a.gate, m, a.gate_off + g * a.N + n));
-      y[(long long)m * a.ldy + n] = Elem<T>::put(v);
+      if (a.y_f32) reinterpret_cast<float*>(a.y)[g * a.gy + (long long)m * a.ldy + n] = v;
+      else y[(long long)m * a.ldy + n] = Elem<T>::put(v);
     }
     if (g == 0 && blockIdx.x == 0)
       for (int c = a.groups * a.N + (threadIdx.x & 15); c < a.y_pad; c += 16)

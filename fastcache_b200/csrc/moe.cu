@@ -1,5 +1,5 @@
-// Tokens by expert: the plan of a step's routing (which sorted row belongs to which token and expert, which 128-row tile to
-// which expert) and the gather of the tokens into that order.
+// Tokens by expert: the choice of a token's experts (by a table, by scores), the plan of a step's routing (which sorted row
+// belongs to which token and expert, which 128-row tile to which expert) and the gather of the tokens into that order.
 #include <stdexcept>
 #include <string>
 
@@ -70,6 +70,236 @@ void launch_route_table(const RouteTable& a, cudaStream_t s) {
   launch_pdl(PDL_PARTIALS, route_table_kernel, dim3(1), dim3(RT_THREADS), 0, s, p);
   const cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess) throw std::runtime_error(std::string("routing: ") + cudaGetErrorString(e));
+}
+
+// ---- choice by score
+// One warp per token.  s_choice [E]: choice scores, -inf outside the best groups; `put(j, expert, score)` receives the j-th
+// chosen expert on every lane.  Ties go to the lower index.
+struct Best {
+  float v;
+  int i;
+};
+__device__ __forceinline__ Best warp_best(Best b) {
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) {
+    const float v = __shfl_xor_sync(0xffffffffu, b.v, o);
+    const int i = __shfl_xor_sync(0xffffffffu, b.i, o);
+    if (v > b.v || (v == b.v && i < b.i)) b = {v, i};
+  }
+  return b;
+}
+template <typename Put>
+__device__ __forceinline__ void choose_experts(const RouteScore& p, long long t, float* s_choice, float* s_group, Put put) {
+  const int lane = threadIdx.x & 31, size = p.E / p.groups;
+  for (int e = lane; e < p.E; e += 32) s_choice[e] = sigmoid_f(proj_at<float>(p.logits, t, e)) + p.correction[e];
+  __syncwarp();
+  if (p.keep < p.groups) {
+    for (int g = lane; g < p.groups; g += 32) {
+      float a = -INFINITY, b = -INFINITY;                    // the two largest
+      for (int e = g * size; e < (g + 1) * size; ++e) {
+        const float v = s_choice[e];
+        b = fmaxf(b, fminf(a, v));
+        a = fmaxf(a, v);
+      }
+      s_group[g] = size > 1 ? a + b : a;
+    }
+    __syncwarp();
+    // a group takes part if fewer than `keep` groups stand before it
+    for (int g = lane; g < p.groups; g += 32) {
+      const float v = s_group[g];
+      int before = 0;
+      for (int o = 0; o < p.groups; ++o) before += s_group[o] > v || (s_group[o] == v && o < g) ? 1 : 0;
+      if (before >= p.keep)
+        for (int e = g * size; e < (g + 1) * size; ++e) s_choice[e] = -INFINITY;
+    }
+    __syncwarp();
+  }
+  for (int j = 0; j < p.top; ++j) {
+    Best b{-INFINITY, p.E};
+    for (int e = lane; e < p.E; e += 32)
+      if (s_choice[e] > b.v) b = {s_choice[e], e};
+    b = warp_best(b);
+    const int e = min(b.i, p.E - 1);                         // scores that are not numbers choose the last expert
+    put(j, e, b.v - p.correction[e]);
+    __syncwarp();
+    if (lane == 0) s_choice[e] = -INFINITY;
+    __syncwarp();
+  }
+}
+// choice and weights of token t: ids and mix (lane j holds the j-th, `top` <= 32 at a time)
+__device__ __forceinline__ void choose_and_weigh(const RouteScore& p, long long t, float* s_choice, float* s_group, int* ids) {
+  const int lane = threadIdx.x & 31;
+  if (p.ctx != nullptr && p.ctx[t] <= 0) {                   // a padding row has no experts
+    for (int j = lane; j < p.top; j += 32) ids[j] = -1;
+    return;
+  }
+  float total = 0.f;
+  float* mix = p.mix + t * p.top;
+  choose_experts(p, t, s_choice, s_group, [&](int j, int e, float) {
+    const float s = sigmoid_f(proj_at<float>(p.logits, t, e));       // without the rounding of adding the correction
+    total += s;
+    if (lane == 0) {
+      ids[j] = e;
+      mix[j] = s;
+    }
+  });
+  __syncwarp();
+  const float inv = 1.f / (total + 1e-20f);
+  for (int j = lane; j < p.top; j += 32) mix[j] *= inv;
+}
+
+// sums of s_v [n] up to and including each entry, in place, by all threads
+template <int THREADS>
+__device__ __forceinline__ void cta_scan(int* s_v, int n) {
+  for (int o = 1; o < n; o <<= 1) {
+    int add[MOE_MAX_EXPERTS / THREADS];
+#pragma unroll
+    for (int k = 0; k < MOE_MAX_EXPERTS / THREADS; ++k) {
+      const int i = threadIdx.x + k * THREADS;
+      add[k] = i < n && i >= o ? s_v[i - o] : 0;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < MOE_MAX_EXPERTS / THREADS; ++k) {
+      const int i = threadIdx.x + k * THREADS;
+      if (i < n) s_v[i] += add[k];
+    }
+    __syncthreads();
+  }
+}
+// plan's first rows, tile count and tiles from the experts' counts; s_end, s_tile: scratch [E] (s_end: end of each expert's rows)
+template <int THREADS>
+__device__ __forceinline__ void write_plan(const RouteScore& p, const int* s_count, int* s_end, int* s_tile, bool write) {
+  for (int e = threadIdx.x; e < p.E; e += THREADS) {
+    s_end[e] = s_count[e];
+    s_tile[e] = (s_count[e] + MOE_TILE - 1) / MOE_TILE;
+  }
+  __syncthreads();
+  cta_scan<THREADS>(s_end, p.E);
+  cta_scan<THREADS>(s_tile, p.E);
+  if (!write) return;
+  int* tile = p.plan + p.E + 2;
+  for (int e = threadIdx.x; e < p.E; e += THREADS) {
+    const int n = s_count[e], at = s_end[e] - n, tiles = (n + MOE_TILE - 1) / MOE_TILE, first = s_tile[e] - tiles;
+    p.plan[e] = at;
+    for (int k = 0; k < tiles; ++k) {
+      tile[2 * (first + k)] = e;
+      tile[2 * (first + k) + 1] = at + k * MOE_TILE;
+    }
+    if (e == p.E - 1) {
+      p.plan[p.E] = s_end[e];
+      p.plan[p.E + 1] = s_tile[e];
+    }
+  }
+}
+
+// Few tokens: one CTA chooses, counts and places.
+__global__ void __launch_bounds__(RT_THREADS)
+route_score_small_kernel(const RouteScore p) {
+  extern __shared__ float s_scores[];                        // [warps][E + groups]
+  __shared__ int s_count[MOE_MAX_EXPERTS], s_end[MOE_MAX_EXPERTS], s_tile[MOE_MAX_EXPERTS];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int warp = threadIdx.x >> 5, tid = threadIdx.x;
+  float* s_choice = s_scores + warp * (p.E + p.groups);
+  for (int e = tid; e < p.E; e += RT_THREADS) s_count[e] = 0;
+  for (int t = warp; t < p.T; t += RT_THREADS / 32) choose_and_weigh(p, t, s_choice, s_choice + p.E, p.ids + t * p.top);
+  __syncthreads();                                           // also makes ids visible in the CTA
+  for (int i = tid; i < p.T * p.top; i += RT_THREADS)
+    if (p.ids[i] >= 0) atomicAdd(&s_count[p.ids[i]], 1);
+  __syncthreads();
+  write_plan<RT_THREADS>(p, s_count, s_end, s_tile, true);
+  __syncthreads();
+  for (int e = tid; e < p.E; e += RT_THREADS) s_end[e] -= s_count[e];       // next free row
+  __syncthreads();
+  int* token = p.plan + p.token_at;
+  for (int i = tid; i < p.T * p.top; i += RT_THREADS) {
+    const int e = p.ids[i];
+    int r = -1;
+    if (e >= 0) {
+      r = atomicAdd(&s_end[e], 1);
+      token[r] = i / p.top;
+    }
+    p.row_of[i] = r;
+  }
+}
+
+// Many tokens: every CTA chooses for ROUTE_ROWS tokens and leaves its counts; then every CTA places its own.
+constexpr int RS_ROUTE_THREADS = 256;
+__global__ void __launch_bounds__(RS_ROUTE_THREADS)
+route_choose_kernel(const RouteScore p) {
+  extern __shared__ float s_scores[];
+  __shared__ int s_count[MOE_MAX_EXPERTS];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int warp = threadIdx.x >> 5, tid = threadIdx.x, t0 = blockIdx.x * ROUTE_ROWS, t1 = min(p.T, t0 + ROUTE_ROWS);
+  float* s_choice = s_scores + warp * (p.E + p.groups);
+  for (int e = tid; e < p.E; e += RS_ROUTE_THREADS) s_count[e] = 0;
+  for (int t = t0 + warp; t < t1; t += RS_ROUTE_THREADS / 32)
+    choose_and_weigh(p, t, s_choice, s_choice + p.E, p.ids + (long long)t * p.top);
+  __syncthreads();
+  for (int i = t0 * p.top + tid; i < t1 * p.top; i += RS_ROUTE_THREADS)
+    if (p.ids[i] >= 0) atomicAdd(&s_count[p.ids[i]], 1);
+  __syncthreads();
+  for (int e = tid; e < p.E; e += RS_ROUTE_THREADS) p.counts[(long long)blockIdx.x * p.E + e] = s_count[e];
+}
+__global__ void __launch_bounds__(RS_ROUTE_THREADS)
+route_place_kernel(const RouteScore p, int blocks) {
+  __shared__ int s_count[MOE_MAX_EXPERTS], s_before[MOE_MAX_EXPERTS], s_end[MOE_MAX_EXPERTS], s_tile[MOE_MAX_EXPERTS];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int tid = threadIdx.x, t0 = blockIdx.x * ROUTE_ROWS, t1 = min(p.T, t0 + ROUTE_ROWS);
+  for (int e = tid; e < p.E; e += RS_ROUTE_THREADS) s_count[e] = s_before[e] = 0;
+  __syncthreads();
+  // columns of the count table, shared between threads where there are fewer experts than threads
+  const int cols = min(p.E, RS_ROUTE_THREADS), per = RS_ROUTE_THREADS / cols, part = tid / cols;
+  if (part < per)
+    for (int e = tid % cols; e < p.E; e += cols) {
+      int all = 0, before = 0;
+#pragma unroll 4
+      for (int b = part; b < blocks; b += per) {
+        const int n = __ldcg(p.counts + (long long)b * p.E + e);
+        all += n;
+        if (b < int(blockIdx.x)) before += n;
+      }
+      atomicAdd(&s_count[e], all);
+      atomicAdd(&s_before[e], before);
+    }
+  __syncthreads();
+  write_plan<RS_ROUTE_THREADS>(p, s_count, s_end, s_tile, blockIdx.x == 0);
+  __syncthreads();
+  for (int e = tid; e < p.E; e += RS_ROUTE_THREADS) s_end[e] += s_before[e] - s_count[e];
+  __syncthreads();
+  int* token = p.plan + p.token_at;
+  for (int i = t0 * p.top + tid; i < t1 * p.top; i += RS_ROUTE_THREADS) {
+    const int e = __ldcg(p.ids + i), r = e >= 0 ? atomicAdd(&s_end[e], 1) : -1;
+    if (e >= 0) token[r] = i / p.top;
+    p.row_of[i] = r;
+  }
+}
+void launch_route_score(const RouteScore& a, cudaStream_t s) {
+  if (a.T == 0) return;
+  RouteScore p = a;
+  p.token_at = moe_token_offset(p.T * p.top, p.E);
+  if (p.E > MOE_MAX_EXPERTS) throw std::runtime_error("experts are limited to 1024");
+  auto smem = [&](auto kern, int warps) {
+    const int bytes = warps * (p.E + p.groups) * 4;
+    if (bytes > 200 * 1024) throw std::runtime_error("routing: too many experts and groups");
+    if (bytes > 32 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes);
+    return size_t(bytes);
+  };
+  const bool small = p.T <= 256 && p.E + p.groups <= 1024;
+  if (small) {
+    const size_t n = smem(route_score_small_kernel, RT_THREADS / 32);
+    launch_pdl(PDL_PARTIALS, route_score_small_kernel, dim3(1), dim3(RT_THREADS), n, s, p);
+  } else {
+    const int blocks = route_score_blocks(p.T);
+    const size_t n = smem(route_choose_kernel, RS_ROUTE_THREADS / 32);
+    launch_pdl(PDL_PARTIALS, route_choose_kernel, dim3(blocks), dim3(RS_ROUTE_THREADS), n, s, p);
+    launch_pdl(PDL_PARTIALS, route_place_kernel, dim3(blocks), dim3(RS_ROUTE_THREADS), 0, s, p, blocks);
+  }
+  const cudaError_t e = cudaGetLastError();
+  if (e != cudaSuccess) throw std::runtime_error(std::string("routing by score: ") + cudaGetErrorString(e));
 }
 
 // 16-byte pieces, one row per CTA

@@ -1,7 +1,6 @@
 // Python bindings of the kernels of pre-normed layers whose sublayers run in parallel: packed projections that stay
 // partial sums for their readers, windowed attention, matrix memory, gated activations, experts, add + norm.
 #include <ATen/cuda/CUDAContext.h>
-#include <c10/cuda/CUDAGuard.h>
 #include <torch/extension.h>
 
 #include <algorithm>
@@ -9,113 +8,10 @@
 #include <tuple>
 #include <vector>
 
-#include "hybrid_bind.h"
 #include "kernels.h"
+#include "projection.h"
 
 namespace {
-
-constexpr int SMALL_ROWS = 256;         // decode-size products: fp32 partial sums for the readers
-
-// Output of a packed projection on the device.  `src` is what most readers take, `wide` a form with fp32 values (columns
-// counted from wide0).  Partial sums live in the stream's scratch until the next product.
-struct Projection {
-  fc::ProjSrc src, wide;
-  int wide0 = 0;
-  int64_t rows = 0, cols = 0;
-  bool f32 = false;
-  Tensor hold, hold_wide;
-};
-
-void check_rows(const Tensor& t, const char* name) {
-  check_elem(t, name);
-  TORCH_CHECK(t.dim() == 2 && t.stride(1) == 1 && t.stride(0) % 8 == 0 && (reinterpret_cast<uintptr_t>(t.data_ptr()) & 15) == 0,
-              name, " must be a row-major matrix with rows of whole 16-byte pieces");
-}
-void check_product(const Tensor& x, const Tensor& w) {
-  check_rows(x, "x");
-  check_rows(w, "weight");
-  TORCH_CHECK(x.scalar_type() == w.scalar_type() && x.size(1) == w.size(1) && w.size(1) % 8 == 0 && w.size(0) % 8 == 0 &&
-                  w.stride(0) == w.size(1), "projection operands must be padded to multiples of 8");
-}
-void simt(const Tensor& x, const Tensor& w, void* y, int N, long long ldy) {
-  fc::SimtLinear a;
-  a.x = x.data_ptr();
-  a.w = w.data_ptr();
-  a.y = y;
-  a.M = int(x.size(0));
-  a.N = N;
-  a.K = int(x.size(1));
-  a.ldx = x.stride(0);
-  a.ldw = w.size(1);
-  a.ldy = ldy;
-  fc::launch_linear_simt(a, true, stream_now());
-}
-// fp32 partial sums of a decode-size product in the stream's scratch; with `finish` also `hold`
-fc::ProjSrc partial_product(const Tensor& x, const Tensor& w, int N, bool finish, Tensor& hold) {
-  const auto& ws = ws_of(x);
-  const int M = int(x.size(0)), K = int(x.size(1));
-  if (finish) hold = torch::empty({M, N}, x.options());
-  const int splits = fc::gemm_skinny_bf16(x.data_ptr(), w.data_ptr(), finish ? hold.data_ptr() : nullptr, nullptr, M, N, K,
-                                          x.stride(0), K, N, 0, gemm_workspace(ws), fc::stream_sm_limit(stream_now()), 0,
-                                          finish, stream_now(), nullptr, fc::SK_PARTIAL);
-  fc::ProjSrc s;
-  s.part = ws.gemm_scratch;
-  s.splits = splits;
-  s.part_stride = (long long)M * N;
-  s.part_ld = N;
-  return s;
-}
-bool partial_fits(int64_t M, int64_t N) { return M <= SMALL_ROWS && size_t(M) * size_t(N) <= fc::gemm_scratch_bytes() / 4; }
-
-// rows [0, N) of w.  `finish`: readers of `src` need a finished matrix.
-Projection project(const Tensor& x, const Tensor& w, int64_t N, int64_t wide0, int64_t wide_n, bool finish) {
-  check_product(x, w);
-  TORCH_CHECK(N > 0 && N <= w.size(0) && N % 8 == 0 && wide0 >= 0 && wide0 + wide_n <= N, "bad projection columns");
-  c10::cuda::CUDAGuard guard(x.device());
-  Projection r;
-  const int M = int(x.size(0)), K = int(x.size(1));
-  r.rows = M;
-  r.cols = N;
-  r.f32 = is_f32(x);
-  if (!r.f32 && M > 0 && partial_fits(M, N)) {
-    const fc::ProjSrc part = partial_product(x, w, int(N), finish, r.hold);
-    r.src = r.wide = part;
-    if (finish) {
-      r.src = fc::ProjSrc();
-      r.src.p = r.hold.data_ptr();
-      r.src.ld = N;
-    }
-    return r;
-  }
-  r.hold = torch::empty({M, N}, x.options());
-  r.src.p = r.hold.data_ptr();
-  r.src.ld = N;
-  if (M == 0) return r;
-  if (r.f32) {
-    simt(x, w, r.hold.data_ptr(), int(N), N);
-    r.wide = r.src;
-    return r;
-  }
-  const auto& ws = ws_of(x);
-  if (wide_n > 0) {
-    r.hold_wide = torch::empty({M, wide_n}, x.options().dtype(torch::kFloat32));
-    r.wide.p = r.hold_wide.data_ptr();
-    r.wide.ld = wide_n;
-    r.wide0 = int(wide0);
-    fc::gemm_bf16_wide(x.data_ptr(), w.data_ptr(), r.hold.data_ptr(), M, int(N), K, x.stride(0), K, N, int(wide0), int(wide_n),
-                       r.hold_wide.data_ptr<float>(), gemm_workspace(ws), fc::stream_sm_limit(stream_now()), stream_now());
-  } else {
-    fc::gemm_bf16(x.data_ptr(), w.data_ptr(), r.hold.data_ptr(), nullptr, M, int(N), K, x.stride(0), K, N, 0,
-                  gemm_workspace(ws), fc::stream_sm_limit(stream_now()), stream_now());
-  }
-  return r;
-}
-
-void check_out(const Tensor& out, int64_t rows, int64_t width, bool f32) {
-  check_rows(out, "out");
-  TORCH_CHECK(is_f32(out) == f32 && out.size(0) == rows && out.size(1) == pad8(int(width)), "output rows of ", pad8(int(width)),
-              " columns expected");
-}
 
 void glu(const Projection& p, int64_t gate, int64_t up, int64_t width, int64_t kind, double limit, Tensor out) {
   check_out(out, p.rows, width, p.f32);
@@ -338,28 +234,33 @@ Projection experts(const Tensor& h, const Tensor& plan, int64_t top, const Tenso
 }
 
 // ------------------------------------------------------------------ windowed attention
-// d: heads, key heads, head size, rotated dimensions, window, first columns of q, k, gate.  impl: 0 choose, 1 general
-void windowed_attention(const Projection& pr, const std::vector<int64_t>& d, double scale, const Tensor& freq, const Tensor& q_norm,
-                        const Tensor& k_norm, const Tensor& sink, double eps, Tensor k_rows, Tensor v_rows,
-                        const Tensor& positions, const Tensor& slots, const Tensor& block_tables, const Tensor& ctx,
-                        const OptTensor& cu_q, const OptTensor& row_seq, const OptTensor& row_ctx, int64_t max_q,
-                        int64_t max_ctx, Tensor out, int64_t impl) {
-  TORCH_CHECK(d.size() == 8, "windowed attention: eight sizes and offsets");
-  const int H = int(d[0]), G = int(d[1]), D = int(d[2]), rot = int(d[3]), window = int(d[4]);
+// d: heads, key heads, head size, value size, rotated dimensions, window, chunk, first columns of q, k, v (-1: the values are
+// the raw keys) and gate (-1: none), whether halves turn together.  impl: 0 choose, 1 general
+void windowed_attention(const Projection& pr, const std::vector<int64_t>& d, double scale, double softcap, double rot_size,
+                        const Tensor& freq, const OptTensor& bias, const Tensor& q_norm, const Tensor& k_norm, const OptTensor& sink,
+                        double eps, Tensor k_rows, Tensor v_rows, const Tensor& positions, const Tensor& slots,
+                        const Tensor& block_tables, const Tensor& ctx, const OptTensor& cu_q, const OptTensor& row_seq,
+                        const OptTensor& row_ctx, int64_t max_q, int64_t max_ctx, Tensor out, int64_t impl) {
+  TORCH_CHECK(d.size() == 12, "windowed attention: twelve sizes and offsets");
+  const int H = int(d[0]), G = int(d[1]), D = int(d[2]), V = int(d[3]), rot = int(d[4]), window = int(d[5]), chunk = int(d[6]);
+  const int off_q = int(d[7]), off_k = int(d[8]), off_v = int(d[9]), off_g = int(d[10]);
   const int T = int(pr.rows), B = int(ctx.numel());
-  const bool f32 = pr.f32;
+  const bool f32 = pr.f32, gated = off_g >= 0;
   TORCH_CHECK(H > 0 && G > 0 && H % G == 0 && rot % 2 == 0 && rot <= D, "bad head counts or rotated dimensions");
-  TORCH_CHECK(d[5] + H * D <= pr.cols && d[6] + G * D <= pr.cols && d[7] + H * D <= pr.cols, "bad projection columns");
-  check_out(out, T, int64_t(H) * D, f32);
+  TORCH_CHECK(window >= 0 && chunk >= 0 && (off_v >= 0 || V == D), "bad window, chunk or value size");
+  TORCH_CHECK(off_q + H * D <= pr.cols && off_k + G * D <= pr.cols && off_v + G * V <= pr.cols && off_g + H * V <= pr.cols,
+              "bad projection columns");
+  check_out(out, T, int64_t(H) * V, f32);
   for (const Tensor& t : {k_rows, v_rows}) {
     check_elem(t, "cache rows");
-    TORCH_CHECK(is_f32(t) == f32 && t.is_contiguous() && t.dim() == 4 && t.size(1) == G && t.size(3) >= D && t.size(3) % 8 == 0,
-                "cache rows must be [blocks, key heads, block, padded head size]");
+    TORCH_CHECK(is_f32(t) == f32 && t.is_contiguous() && t.dim() == 4 && t.size(1) == G && t.size(3) >= std::max(D, V) &&
+                    t.size(3) % 8 == 0, "cache rows must be [blocks, key heads, block, padded head size]");
   }
   TORCH_CHECK(k_rows.sizes() == v_rows.sizes(), "keys and values need pages of one shape");
   check_f32(q_norm, "query norm", (int64_t)H * D);
   check_f32(k_norm, "key norm", (int64_t)G * D);
-  check_f32(sink, "sink", H);
+  if (sink.has_value()) check_f32(*sink, "sink", H);
+  check_bias(bias, pr.cols, f32);
   TORCH_CHECK(freq.is_cuda() && freq.scalar_type() == torch::kFloat64 && freq.is_contiguous() && freq.numel() == rot / 2,
               "freq must be float64 [rotated dimensions / 2]");
   check_i32(slots, "slot map", T);
@@ -378,12 +279,17 @@ void windowed_attention(const Projection& pr, const std::vector<int64_t>& d, dou
   st.H = H;
   st.G = G;
   st.D = D;
+  st.V = V;
   st.pitch = pitch;
   st.rot_dims = rot;
   st.proj = pr.src;
-  st.off_q = int(d[5]);
-  st.off_k = int(d[6]);
-  st.off_g = int(d[7]);
+  st.off_q = off_q;
+  st.off_k = off_k;
+  st.off_v = off_v;
+  st.off_g = std::max(off_g, 0);
+  if (bias.has_value()) st.bias = bias->data_ptr();
+  st.half = d[11] != 0;
+  st.rot_size = float(rot_size);
   st.q_norm = q_norm.data_ptr<float>();
   st.k_norm = k_norm.data_ptr<float>();
   st.eps = float(eps);
@@ -397,12 +303,12 @@ void windowed_attention(const Projection& pr, const std::vector<int64_t>& d, dou
   st.q = q.data_ptr();
   st.out = out.data_ptr();
   st.ld_out = out.stride(0);
-  st.pad_out = int(out.size(1)) - H * D;
+  st.pad_out = int(out.size(1)) - H * V;
   st.status = ws.status;
   const bool prefill = cu_q.has_value() && cu_q->defined();
   const bool tc = !f32 && impl != 1 && (pitch == 64 || pitch == 128) && bs % 8 == 0 && (prefill || H / G <= 16);
-  if (tc && pr.src.part != nullptr) {
-    gate = torch::empty({T, H * D}, out.options());
+  if (tc && gated && (pr.src.part != nullptr || bias.has_value())) {
+    gate = torch::empty({T, H * V}, out.options());
     st.gate = gate.data_ptr();
   }
   fc::launch_window_store(st, f32, stream_now());
@@ -420,8 +326,11 @@ void windowed_attention(const Projection& pr, const std::vector<int64_t>& d, dou
     a.H = H;
     a.G = G;
     a.D = D;
+    a.V = V;
     a.pitch = pitch;
     a.window = window;
+    a.chunk = chunk;
+    a.softcap = float(softcap);
     a.block_size = bs;
     a.max_blocks = max_blocks;
     a.num_blocks = blocks;
@@ -431,9 +340,10 @@ void windowed_attention(const Projection& pr, const std::vector<int64_t>& d, dou
     a.block_tables = block_tables.data_ptr<int>();
     a.row_seq = prefill ? row_seq->data_ptr<int>() : nullptr;
     a.row_ctx = prefill ? row_ctx->data_ptr<int>() : ctx.data_ptr<int>();
-    a.sink = sink.data_ptr<float>();
+    if (sink.has_value()) a.sink = sink->data_ptr<float>();
+    TORCH_CHECK(!gated || !bias.has_value(), "the general form takes no gate with a bias");
     a.gate = pr.src;
-    a.off_g = st.off_g;
+    a.off_g = off_g;
     a.out = out.data_ptr();
     a.ld_out = out.stride(0);
     a.scale = float(scale);
@@ -443,12 +353,14 @@ void windowed_attention(const Projection& pr, const std::vector<int64_t>& d, dou
   }
   fc::AttnOptions opt;
   opt.window = window;
-  opt.sink = sink.data_ptr<float>();
-  opt.dim = D;
+  opt.chunk = chunk;
+  opt.softcap = float(softcap);
+  if (sink.has_value()) opt.sink = sink->data_ptr<float>();
+  opt.dim = V;
   if (gate.defined()) {
     opt.gate = gate.data_ptr();
-    opt.ld_gate = (long long)H * D;
-  } else {
+    opt.ld_gate = (long long)H * V;
+  } else if (gated) {
     opt.gate = reinterpret_cast<const char*>(pr.src.p) + (long long)st.off_g * 2;
     opt.ld_gate = pr.src.ld;
   }
@@ -456,6 +368,7 @@ void windowed_attention(const Projection& pr, const std::vector<int64_t>& d, dou
   if (!prefill) {
     if (max_ctx <= 0) max_ctx = (int64_t)max_blocks * bs;
     if (window > 0) max_ctx = std::min<int64_t>(max_ctx, window + 64);
+    if (chunk > 0) max_ctx = std::min<int64_t>(max_ctx, chunk + 64);
     int splits = fc::decode_attn_pick_splits(T, G, int(max_ctx), fc::gemm_num_sms());
     while (splits > 1 && ((long long)T * H * splits * pitch > fc::ATTN_WS_FLOATS || (long long)T * H * splits > fc::ATTN_LSE_FLOATS)) --splits;
     fc::launch_decode_attention(q.data_ptr(), k_rows.data_ptr(), v_rows.data_ptr(), block_tables.data_ptr<int>(),
@@ -568,6 +481,8 @@ Projection as_projection(const Tensor& t, int64_t wide0, const OptTensor& wide) 
 
 }  // namespace
 
+void register_streams(pybind11::module_& m);
+
 void register_prenorm(pybind11::module_& m) {
   py::class_<Projection>(m, "Projection", "output of a packed projection, for the ops that read it")
       .def_readonly("rows", &Projection::rows)
@@ -582,4 +497,5 @@ void register_prenorm(pybind11::module_& m) {
   m.def("experts", &experts);
   m.def("windowed_attention", &windowed_attention);
   m.def("matrix_memory", &matrix_memory);
+  register_streams(m);
 }

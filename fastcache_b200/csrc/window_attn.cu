@@ -1,10 +1,11 @@
-// Attention over per-head K/V rows whose values are the raw keys: norm over the whole query and key projections,
-// interleaved rotation, cache store, and the general form of windowed attention with a sink and an output gate (any head
-// size, bf16 or fp32; the tensor-core forms are attn_prefill*.cu and attn_decode.cu with AttnOptions).
+// Attention over per-head K/V rows: bias, norm over the whole query and key projections, rotation, cache store (the values
+// may be the raw keys), and the general form of attention with window, chunks, soft cap, sink and output gate (any head size,
+// bf16 or fp32; the tensor-core forms are attn_prefill*.cu and attn_decode.cu with AttnOptions).
 #include <algorithm>
 #include <stdexcept>
 #include <string>
 
+#include "attn_options.cuh"
 #include "hybrid.cuh"
 #include "launch.h"
 
@@ -13,13 +14,14 @@ namespace fc {
 using bf16 = __nv_bfloat16;
 
 // One CTA per token.  The projections are staged in shared memory as fp32 while their squares are summed; VEC: four
-// columns at a time (head size, pitch and offsets multiples of 4).
+// columns at a time (head sizes, half of the rotated dimensions where halves turn, pitch and offsets multiples of 4).
 template <typename T, bool VEC, int WS_THREADS>
 __global__ void __launch_bounds__(WS_THREADS)
 window_store_kernel(const WindowStore p) {
   __shared__ float2 red[WS_THREADS / 32];
   extern __shared__ __align__(16) float sm[];
   const int nq = p.H * p.D, nk = p.G * p.D, half = p.rot_dims / 2;
+  const T* bias = reinterpret_cast<const T*>(p.bias);
   float *s_q = sm, *s_k = sm + nq;
   float2* cs = reinterpret_cast<float2*>(sm + ((nq + nk + 3) / 4) * 4);      // (cos, sin) of every pair
   pdl_launch_dependents();
@@ -27,40 +29,61 @@ window_store_kernel(const WindowStore p) {
   const long long t = blockIdx.x;
   const int tid = threadIdx.x;
   T* out = reinterpret_cast<T*>(p.out);
-  if (tid < p.pad_out) out[t * p.ld_out + nq + tid] = Elem<T>::put(0.f);
+  if (tid < p.pad_out) out[t * p.ld_out + p.H * p.V + tid] = Elem<T>::put(0.f);
   const double pos = double(p.positions[t]);
   float sq = 0.f, sk = 0.f;
+  // columns of the projection with their bias
+  auto col1 = [&](int c) {
+    const float v = proj_at<T>(p.proj, t, c);
+    return bias != nullptr ? v + Elem<T>::get(bias[c]) : v;
+  };
+  auto col4 = [&](int c) {
+    float4 v = proj_at4<T>(p.proj, t, c);
+    if (bias != nullptr) {
+      v.x += Elem<T>::get(bias[c]);
+      v.y += Elem<T>::get(bias[c + 1]);
+      v.z += Elem<T>::get(bias[c + 2]);
+      v.w += Elem<T>::get(bias[c + 3]);
+    }
+    return v;
+  };
+  const int ng = p.H * p.V;
   if (VEC) {
 #pragma unroll 4
     for (int i = tid * 4; i < nq; i += WS_THREADS * 4) {
-      const float4 v = proj_at4<T>(p.proj, t, p.off_q + i);
+      const float4 v = col4(p.off_q + i);
       *reinterpret_cast<float4*>(s_q + i) = v;
       sq += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
     }
     for (int i = tid * 4; i < nk; i += WS_THREADS * 4) {
-      const float4 v = proj_at4<T>(p.proj, t, p.off_k + i);
+      const float4 v = col4(p.off_k + i);
       *reinterpret_cast<float4*>(s_k + i) = v;
       sk += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
     }
     if (p.gate != nullptr)
-      for (int i = tid * 4; i < nq; i += WS_THREADS * 4) {
-        const float4 v = proj_at4<T>(p.proj, t, p.off_g + i);
-        store4(reinterpret_cast<T*>(p.gate) + t * nq + i, v.x, v.y, v.z, v.w);
+      for (int i = tid * 4; i < ng; i += WS_THREADS * 4) {
+        const float4 v = col4(p.off_g + i);
+        store4(reinterpret_cast<T*>(p.gate) + t * ng + i, v.x, v.y, v.z, v.w);
       }
   } else {
     for (int i = tid; i < nq; i += WS_THREADS) {
-      const float v = proj_at<T>(p.proj, t, p.off_q + i);
+      const float v = col1(p.off_q + i);
       s_q[i] = v;
       sq += v * v;
-      if (p.gate != nullptr) reinterpret_cast<T*>(p.gate)[t * nq + i] = Elem<T>::put(proj_at<T>(p.proj, t, p.off_g + i));
     }
+    if (p.gate != nullptr)
+      for (int i = tid; i < ng; i += WS_THREADS) reinterpret_cast<T*>(p.gate)[t * ng + i] = Elem<T>::put(col1(p.off_g + i));
     for (int i = tid; i < nk; i += WS_THREADS) {
-      const float v = proj_at<T>(p.proj, t, p.off_k + i);
+      const float v = col1(p.off_k + i);
       s_k[i] = v;
       sk += v * v;
     }
   }
-  for (int i = tid; i < half; i += WS_THREADS) turn_angle(pos, p.freq[i], cs[i].x, cs[i].y);
+  for (int i = tid; i < half; i += WS_THREADS) {
+    float c, s;
+    turn_angle(pos, p.freq[i], c, s);
+    cs[i] = make_float2(c * p.rot_size, s * p.rot_size);
+  }
   sq = warp_sum(sq);
   sk = warp_sum(sk);
   if ((tid & 31) == 0) red[tid >> 5] = make_float2(sq, sk);
@@ -76,13 +99,33 @@ window_store_kernel(const WindowStore p) {
   auto turned = [&](const float* x, const float* w, int c, float inv) {
     const float v = x[c] * inv * w[c];
     if (c >= p.rot_dims) return v;
+    if (p.half) {
+      const bool lo = c < half;
+      const int d = lo ? c + half : c - half;
+      const float2 a = cs[lo ? c : d];
+      const float o = x[d] * inv * w[d];
+      return lo ? v * a.x - o * a.y : v * a.x + o * a.y;
+    }
     const float2 a = cs[c >> 1];
     const float o = x[c ^ 1] * inv * w[c ^ 1];
     return (c & 1) ? v * a.x + o * a.y : v * a.x - o * a.y;
   };
-  auto four = [&](const float* x, const float* w, int c, float inv) {
+  auto normed = [&](const float* x, const float* w, int c, float inv) {
     const float4 v = *reinterpret_cast<const float4*>(x + c), g = *reinterpret_cast<const float4*>(w + c);
-    float4 y = make_float4(v.x * inv * g.x, v.y * inv * g.y, v.z * inv * g.z, v.w * inv * g.w);
+    return make_float4(v.x * inv * g.x, v.y * inv * g.y, v.z * inv * g.z, v.w * inv * g.w);
+  };
+  auto four = [&](const float* x, const float* w, int c, float inv) {
+    float4 y = normed(x, w, c, inv);
+    if (p.half) {
+      if (c >= p.rot_dims) return y;
+      const bool lo = c < half;
+      const int d = lo ? c + half : c - half;
+      const float4 o = normed(x, w, d, inv);
+      const float2* a = cs + (lo ? c : d);
+      const float f = lo ? -1.f : 1.f;
+      return make_float4(y.x * a[0].x + f * o.x * a[0].y, y.y * a[1].x + f * o.y * a[1].y, y.z * a[2].x + f * o.z * a[2].y,
+                         y.w * a[3].x + f * o.w * a[3].y);
+    }
     if (c < p.rot_dims) {
       const float2 a = cs[c >> 1];
       y = make_float4(y.x * a.x - y.y * a.y, y.y * a.x + y.x * a.y, y.z, y.w);
@@ -119,11 +162,12 @@ window_store_kernel(const WindowStore p) {
     if (VEC) {
       const float4 y = c < p.D ? four(x, p.k_norm + g * p.D, c, ik) : make_float4(0.f, 0.f, 0.f, 0.f);
       store4(k, y.x, y.y, y.z, y.w);
-      const float4 r = c < p.D ? *reinterpret_cast<const float4*>(x + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+      float4 r = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (c < p.V) r = p.off_v < 0 ? *reinterpret_cast<const float4*>(x + c) : col4(p.off_v + g * p.V + c);
       store4(v, r.x, r.y, r.z, r.w);
     } else {
       *k = Elem<T>::put(c < p.D ? turned(x, p.k_norm + g * p.D, c, ik) : 0.f);
-      *v = Elem<T>::put(c < p.D ? x[c] : 0.f);
+      *v = Elem<T>::put(c >= p.V ? 0.f : p.off_v < 0 ? x[c] : col1(p.off_v + g * p.V + c));
     }
   }
 }
@@ -143,7 +187,10 @@ window_attn_kernel(const WindowAttn p) {
   __syncwarp();
   const int b = p.row_seq != nullptr ? p.row_seq[t] : int(t), ctx = p.row_ctx[t], g = h / (p.H / p.G);
   const int* bt = p.block_tables + (long long)b * p.max_blocks;
-  const int first = p.window > 0 ? max(0, ctx - p.window) : 0;
+  AttnOptions seen;
+  seen.window = p.window;
+  seen.chunk = p.chunk;
+  const int first = attn_first(seen, max(ctx - 1, 0));
   const T *kr = reinterpret_cast<const T*>(p.k_rows), *vr = reinterpret_cast<const T*>(p.v_rows);
   float acc[NACC];
 #pragma unroll
@@ -162,6 +209,7 @@ window_attn_kernel(const WindowAttn p) {
         s = 0.f;
         for (int c = 0; c < p.D; ++c) s = fmaf(s_q[c], Elem<T>::get(kr[row + c]), s);
         s *= p.scale;
+        if (p.softcap > 0.f) s = p.softcap * tanhf(s / p.softcap);
       }
     }
     __syncwarp();
@@ -178,16 +226,18 @@ window_attn_kernel(const WindowAttn p) {
       if (pr < 0) continue;
 #pragma unroll
       for (int i = 0; i < NACC; ++i)
-        if (lane + i * 32 < p.D) acc[i] = fmaf(pe, Elem<T>::get(vr[pr + lane + i * 32]), acc[i]);
+        if (lane + i * 32 < p.V) acc[i] = fmaf(pe, Elem<T>::get(vr[pr + lane + i * 32]), acc[i]);
     }
   }
   if (p.sink != nullptr && m != -INFINITY) l += expf(p.sink[h] - m);
   const float inv = l > 0.f ? 1.f / l : 0.f;
-  T* out = reinterpret_cast<T*>(p.out) + t * p.ld_out + h * p.D;
+  T* out = reinterpret_cast<T*>(p.out) + t * p.ld_out + h * p.V;
 #pragma unroll
   for (int i = 0; i < NACC; ++i) {
     const int c = lane + i * 32;
-    if (c < p.D) out[c] = Elem<T>::put(acc[i] * inv * sigmoid_t<T>(proj_at<T>(p.gate, t, p.off_g + h * p.D + c)));
+    if (c >= p.V) continue;
+    const float gate = p.off_g >= 0 ? sigmoid_t<T>(proj_at<T>(p.gate, t, p.off_g + h * p.V + c)) : 1.f;
+    out[c] = Elem<T>::put(acc[i] * inv * gate);
   }
 }
 
@@ -202,7 +252,8 @@ static void window_store_t(const WindowStore& p, cudaStream_t s) {
   const int n = (p.H + p.G) * p.D;
   const size_t smem = size_t((n + 3) / 4 * 4 + p.rot_dims) * 4;
   if (smem > 200 * 1024) throw std::runtime_error("windowed attention: query and key projections are limited to 50000 columns");
-  const bool vec = p.D % 4 == 0 && p.pitch % 4 == 0 && p.off_q % 4 == 0 && p.off_k % 4 == 0 && p.off_g % 4 == 0;
+  const bool vec = p.D % 4 == 0 && p.V % 4 == 0 && p.pitch % 4 == 0 && p.off_q % 4 == 0 && p.off_k % 4 == 0 && p.off_g % 4 == 0 &&
+                   (p.off_v < 0 || p.off_v % 4 == 0) && (!p.half || p.rot_dims % 8 == 0);
   auto go = [&](auto kern, int threads) {
     if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem));
     launch_pdl(PDL_ROPE, kern, dim3(p.T), dim3(threads), smem, s, p);
@@ -220,15 +271,15 @@ void launch_window_store(const WindowStore& p, bool f32, cudaStream_t s) {
 
 void launch_window_attn(const WindowAttn& p, bool f32, cudaStream_t s) {
   if (p.T == 0) return;
-  if (p.D > 512) throw std::runtime_error("windowed attention: heads are limited to 512 columns");
+  if (p.D > 512 || p.V > 512) throw std::runtime_error("windowed attention: heads are limited to 512 columns");
   const dim3 grid(p.T, (p.H + WA_WARPS - 1) / WA_WARPS);
   const size_t smem = size_t(WA_WARPS) * p.D * 4;
   auto go = [&](auto kern) { kern<<<grid, WA_WARPS * 32, smem, s>>>(p); };
   if (f32) {
-    if (p.D <= 128) go(window_attn_kernel<float, 4>);
+    if (p.V <= 128) go(window_attn_kernel<float, 4>);
     else go(window_attn_kernel<float, 16>);
   } else {
-    if (p.D <= 128) go(window_attn_kernel<bf16, 4>);
+    if (p.V <= 128) go(window_attn_kernel<bf16, 4>);
     else go(window_attn_kernel<bf16, 16>);
   }
   check_launch("windowed attention");

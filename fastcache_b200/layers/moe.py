@@ -1,4 +1,4 @@
-"""Mixture of experts: gated feed-forward experts and a router that reads a table of the token ids."""
+"""Mixture of experts: gated feed-forward experts, a router that reads a table of the token ids and one that scores them."""
 from __future__ import annotations
 
 import torch
@@ -7,7 +7,7 @@ from torch import nn
 from .. import ops
 from ..ops.hybrid import GluSpec
 from ..utils.context import get_context
-from .linear import pad8
+from .linear import PackedLinear, pad8
 
 
 class TableRouter(nn.Module):
@@ -32,6 +32,23 @@ class TableRouter(nn.Module):
     def forward(self, input_ids: torch.Tensor):
         """The step's routing; depends on the ids alone, so passes that run a layer again share it."""
         return ops.hybrid.route_by_table(input_ids, self.table, self.experts, get_context())
+
+
+class ScoreRouter(nn.Module):
+    """Experts by sigmoid scores of a linear map.  A correction per expert takes part in the choice but not in the weights;
+    experts stand in equal groups of neighbours, of which the best `keep` (by their two largest choice scores) take part."""
+
+    def __init__(self, width: int, experts: int, top: int, groups: int = 1, keep: int = 1):
+        super().__init__()
+        if experts % groups or not 0 < keep <= groups or not 0 < top <= keep * (experts // groups):
+            raise ValueError(f"{top} experts per token from {keep} of {groups} groups of {experts} experts")
+        self.experts, self.top, self.groups, self.keep = experts, top, groups, keep
+        self.proj = PackedLinear(width, {"router": experts})
+        self.correction = nn.Parameter(torch.zeros(experts, dtype=torch.float32), requires_grad=False)
+
+    def forward(self, h: torch.Tensor):
+        """(the step's routing, weights)"""
+        return ops.hybrid.route_by_score(h, self.proj.weight, self.correction, self.top, self.groups, self.keep, get_context())
 
 
 class Experts(nn.Module):

@@ -1,4 +1,5 @@
-"""Recurrent mixers with a fixed-size state per request: gated linear attention, the gated delta rule, matrix memory.
+"""Recurrent mixers with a fixed-size state per request: gated linear attention, the gated delta rule, matrix memory,
+real-gated linear recurrent units.
 
 They read the state that earlier steps left in the request's slot (`state`, and `conv_state` for the short
 convolutions), advance it by the rows of the batch and leave it there; prefill portions of any length and decode
@@ -13,7 +14,7 @@ from torch import nn
 
 from .. import ops
 from ..engine.layer_cache import LayerCache, PassCache
-from ..ops.hybrid import DeltaDims, GlaDims, MatrixMemoryDims
+from ..ops.hybrid import DeltaDims, GlaDims, LruDims, MatrixMemoryDims
 from ..utils.context import get_context
 from .linear import PackedLinear
 
@@ -120,3 +121,47 @@ class MatrixMemory(nn.Module):
 
     def forward(self, positions: torch.Tensor, p, cache: PassCache, out: torch.Tensor) -> None:
         ops.hybrid.matrix_memory(p, self.dims, self.i_bias, self.f_bias, self.norm, self.eps, cache, get_context(), out)
+
+
+class RealGatedLRU(nn.Module):
+    """Recurrent block of Griffin (De et al., "Griffin: Mixing Gated Linear Recurrences with Local Attention for Efficient
+    Language Models"): one number of state per channel that fades by a gated factor a and takes sqrt(1 - a^2) of the gated
+    input.  The input passes a short causal convolution, its gates are block-diagonal matrices of it; a second branch
+    (gelu) multiplies the output.  Works between projections that its owner holds."""
+
+    def __init__(self, channels: int, blocks: int, taps: int, sharpness: float = 8.0):
+        super().__init__()
+        if channels % blocks:
+            raise ValueError(f"{channels} channels cannot be cut into {blocks} equal parts")
+        n = channels // blocks
+        self.channels, self.blocks, self.taps, self.sharpness, self.bias = channels, blocks, taps, float(sharpness), True
+        self.sizes: Dict[str, int] = {"y": channels, "x": channels}
+        self.out_width = channels
+        self.conv = fp32_vector(channels, taps)
+        self.conv_bias = fp32_vector(channels)
+        self.gates = nn.Parameter(torch.zeros(2, blocks, n, n), requires_grad=False)      # of the decay, of the input
+        self.gates.weight_loader = self._load_gate
+        self.gate_bias = fp32_vector(2, channels)
+        self.gate_bias.weight_loader = self._load_gate
+        self.lam = fp32_vector(channels)
+        self.lam.data.copy_(torch.linspace(-7.0, -2.0, channels))
+        self.vectors = {"conv": "conv", "conv.b": "conv_bias", "lam": "lam"}
+
+    GATES = {"ra": 0, "ri": 1}
+
+    def _load_gate(self, param: nn.Parameter, loaded: torch.Tensor, shard_id=None) -> None:
+        n = self.channels // self.blocks
+        if loaded.shape != ((self.blocks, n, n) if param is self.gates else (self.blocks, n)):
+            raise ValueError(f"shape mismatch: {tuple(loaded.shape)} for gates of {self.blocks} blocks of {n}")
+        param.data[self.GATES[shard_id]].copy_(loaded.reshape(param.data.shape[1:]))
+
+    def bind(self, offset: Dict[str, int]) -> None:
+        self.dims = LruDims(self.channels, self.blocks, offset["y"], offset["x"], self.sharpness)
+
+    def cache(self) -> LayerCache:
+        return LayerCache(PassCache(), state={"state": (self.channels,), "conv_state": (self.taps - 1, self.channels)})
+
+    def forward(self, positions: torch.Tensor, h: torch.Tensor, proj: PackedLinear, cache: PassCache) -> torch.Tensor:
+        """`proj`: the packed projection (y, x) of h."""
+        return ops.hybrid.real_gated_lru(h, proj.weight, proj.bias, self.dims, self.conv, self.conv_bias, self.gates,
+                                         self.gate_bias, self.lam, cache, get_context())

@@ -24,6 +24,8 @@ def detect_model_type(hf_config: Any) -> str:
         return "bagedra"
     if "lekilix" in mt or "lekilix" in joined:
         return "lekilix"
+    if "duperax" in mt or "duperax" in joined:
+        return "duperax"
     if "llama" in mt or "llama" in joined or "mistral" in mt:
         return "llama"
     raise ValueError(f"unsupported model type {mt!r} / architectures {archs}")
@@ -64,9 +66,14 @@ def _lekilix(cfg):
     return LekilixForCausalLM(cfg)
 
 
+def _duperax(cfg):
+    from .duperax import DuperaxForCausalLM
+    return DuperaxForCausalLM(cfg)
+
+
 MODEL_REGISTRY: Dict[str, Callable] = {
     "llama": _llama, "qwen3": _qwen3, "qwen2": _qwen2, "llava": _llava, "minicpm": _minicpm,
-    "bagedra": _bagedra, "lekilix": _lekilix,
+    "bagedra": _bagedra, "lekilix": _lekilix, "duperax": _duperax,
 }
 
 

@@ -71,18 +71,47 @@ class LatentDims:
 
 @dataclass(frozen=True)
 class WindowDims:
-    """Windowed attention over keys that are also the values; first columns of the packed projections.  `window`: the
-    positions a query sees, itself included (0: all up to itself)."""
+    """Attention over per-head rows: sizes, first columns of the packed projections, and what a query sees.
+
+    `v` None: the values are the raw keys; `g` None: no output gate.  `half`: entry i of a head turns with entry
+    i + rot_dims / 2 (else entries 2i and 2i + 1 turn together), cos and sin are multiplied by `rot_size`.  `window`: the
+    positions a query sees, itself included; `chunk`: it sees no key before the last multiple of it; 0: all up to itself.
+    `softcap` c > 0: scores become c tanh(score / c)."""
     heads: int
     kv_heads: int
     dim: int
     rot_dims: int
-    base: float
     scale: float
     window: int
     q: int
     k: int
-    g: int
+    g: Optional[int] = None
+    v: Optional[int] = None
+    vdim: int = 0
+    chunk: int = 0
+    softcap: float = 0.0
+    half: bool = False
+    rot_size: float = 1.0
+
+    @property
+    def value_dim(self) -> int:
+        return self.vdim or self.dim
+
+    def sizes(self) -> list:
+        """The integers as the extension takes them (-1: no such projection)."""
+        return [self.heads, self.kv_heads, self.dim, self.value_dim, self.rot_dims, self.window, self.chunk, self.q, self.k,
+                -1 if self.v is None else self.v, -1 if self.g is None else self.g, int(self.half)]
+
+
+@dataclass(frozen=True)
+class LruDims:
+    """Real-gated linear recurrent unit: channels, equal parts that the gate matrices work on, first columns of the packed
+    projections; the logarithm of the decay is -sharpness * r * softplus(lam)."""
+    channels: int
+    blocks: int
+    y: int
+    x: int
+    sharpness: float = 8.0
 
 
 @dataclass(frozen=True)
@@ -247,6 +276,31 @@ def linear_glu(h, weight, up: int, width: int, spec: GluSpec, out):
         glu(ref_linear(h, weight), 0, up, width, spec, out)
 
 
+# ------------------------------------------------------------------ several residual streams
+def embed_streams(ids, weight, width: int, streams: int, nxt, eps: float):
+    """(fp32 streams [T, streams, width], all the row of the table; the next sublayer's input).  `nxt` = (connection, norm
+    weight, norm bias), see `linear_mix_norm`."""
+    if weight.is_cuda:
+        _n()
+        return ext().embed_streams(ids, weight, int(width), int(streams), *nxt, float(eps))
+    return ref.embed_streams(ids, weight, width, streams, nxt, eps)
+
+
+def linear_mix_norm(a, weight, x, connection, nxt, eps: float, dtype, experts=None):
+    """The streams after a sublayer that returned y = a @ weight.T (a None: none) + the mixed outputs of `experts`, in fp32
+    and in place: x_t <- sum_s mix[s, t] x_s + out[t] y; returns what the next sublayer reads, the layer norm of
+    sum_s in[s] x_s, in `dtype` (the model's).
+
+    `connection` = [in | out | mix] of this sublayer.  `nxt` = (connection, norm weight, norm bias) of the next one; its
+    connection None: the plain sum, after which the streams are not needed (nor written) any more."""
+    if x.is_cuda:
+        _n(2)
+        y, row_of, mix = experts or (None, None, None)
+        return ext().linear_mix_norm(a, weight, x, connection, *nxt, float(eps), y, row_of, mix)
+    y = ref_linear(a, weight) if a is not None else None
+    return ref.mix_norm(y, x, connection, nxt, eps, dtype, experts)
+
+
 # ------------------------------------------------------------------ experts
 def route_by_table(ids, table, experts: int, ctx):
     """Which rows every expert gets when a token's id names its experts (table [vocab, top], int32).  CPU: [T, top]."""
@@ -254,6 +308,17 @@ def route_by_table(ids, table, experts: int, ctx):
         _n()
         return ext().route_by_table(ids, table, int(experts), None if ctx.is_prefill else ctx.context_lens)
     return table[ids].long()
+
+
+def route_by_score(h, weight, correction, top: int, groups: int, keep: int, ctx):
+    """Which rows every expert gets, and the weights [T, top], from scores sigmoid(h @ weight.T): see
+    `reference_hybrid.route_by_score`.  CPU: ([T, top], weights)."""
+    if h.is_cuda:
+        _n(3)
+        row_of, plan, mix = ext().route_by_score(h, weight, correction, int(top), int(groups), int(keep),
+                                                 None if ctx.is_prefill else ctx.context_lens)
+        return (row_of, plan), mix
+    return ref.route_by_score(ref_linear(h, weight), correction, top, groups, keep)
 
 
 def experts(h, route, weights, w_gate_up, w_down, ff: int, spec: GluSpec):
@@ -270,23 +335,53 @@ def experts(h, route, weights, w_gate_up, w_down, ff: int, spec: GluSpec):
 ATTN_IMPL = 0           # tests: 1 the general kernel also where a tensor-core form exists
 
 
-def rope_turns(base: float, dims: int):
-    """Rotation frequencies in turns per position, float64."""
+def rope_turns(base: float, dims: int, scaling: Optional[dict] = None):
+    """Rotation frequencies in turns per position, float64.  `scaling` (factor, original, fast, slow): YaRN; pairs that turn
+    less than `slow` times over the `original` positions are slowed down by `factor`, those that turn more than `fast` times
+    stay, with a ramp between."""
     i = torch.arange(dims // 2, dtype=torch.float64)
-    return float(base) ** (-2 * i / max(1, dims)) / (2 * math.pi)
+    f = float(base) ** (-2 * i / max(1, dims)) / (2 * math.pi)
+    if scaling:
+        def pair(turns):
+            return dims * math.log(scaling["original"] / (2 * math.pi * turns)) / (2 * math.log(base))
+        lo, hi = max(math.floor(pair(scaling["fast"])), 0), min(math.ceil(pair(scaling["slow"])), dims - 1)
+        ramp = ((i - lo) / max(hi - lo, 0.001)).clamp(0, 1)
+        f = f / scaling["factor"] * ramp + f * (1 - ramp)
+    return f
 
 
-def windowed_attention(p, d: WindowDims, freq, q_norm, k_norm, sink, eps: float, k_rows, v_rows, positions, ctx, out):
-    """Norm over the whole projection, rotation (`freq`: rope_turns), cache store, attention with a sink and output gate, to
-    `out`."""
+def rope_size(scaling: Optional[dict]) -> float:
+    """Factor of cos and sin that goes with `scaling`."""
+    return 0.1 * math.log(scaling["factor"]) + 1.0 if scaling else 1.0
+
+
+def windowed_attention(p, d: WindowDims, freq, q_norm, k_norm, sink, eps: float, k_rows, v_rows, positions, ctx, out,
+                       bias=None):
+    """Bias, norm over the whole projection, rotation (`freq`: rope_turns), cache store, attention (with a sink, an output
+    gate) to `out`.  `bias`: of the packed projection, by column."""
     if out.is_cuda:
         _n(2)
-        ext().windowed_attention(p, [d.heads, d.kv_heads, d.dim, d.rot_dims, d.window, d.q, d.k, d.g], d.scale, freq,
-                                 q_norm, k_norm, sink, float(eps), k_rows, v_rows, positions, ctx.slot_mapping,
-                                 ctx.block_tables, ctx.context_lens, ctx.cu_seqlens_q, ctx.row_seq, ctx.row_ctx,
-                                 int(ctx.max_seqlen_q), int(ctx.max_seqlen_k), out, ATTN_IMPL)
+        ext().windowed_attention(p, d.sizes(), d.scale, d.softcap, d.rot_size, freq, bias, q_norm, k_norm, sink, float(eps),
+                                 k_rows, v_rows, positions, ctx.slot_mapping, ctx.block_tables, ctx.context_lens,
+                                 ctx.cu_seqlens_q, ctx.row_seq, ctx.row_ctx, int(ctx.max_seqlen_q), int(ctx.max_seqlen_k),
+                                 out, ATTN_IMPL)
     else:
-        ref.windowed_attention(p, d, q_norm, k_norm, sink, eps, k_rows, v_rows, positions, ctx, out)
+        ref.windowed_attention(p, d, freq, q_norm, k_norm, sink, eps, k_rows, v_rows, positions, ctx, out, bias)
+
+
+# ------------------------------------------------------------------ real-gated linear recurrent unit
+LRU_IMPL = 0            # tests: 1 the general kernels also where a tensor-core form exists
+
+
+def real_gated_lru(h, weight, bias, d: LruDims, conv_w, conv_b, gate_w, gate_b, lam, cache, ctx):
+    """Projections, convolution, gates and recurrence of a batch of runs up to the output projection.  gate_w [2, blocks, n, n]
+    and gate_b [2, channels]: the gate of the decay, then the gate of the input."""
+    if h.is_cuda:
+        _n(4)
+        return ext().real_gated_lru(h, weight, bias, [d.channels, d.blocks, d.y, d.x], d.sharpness, conv_w, conv_b, gate_w,
+                                    gate_b, lam, cache.conv_state, cache.state, *_run_args(ctx), ctx.row_seq, LRU_IMPL)
+    return ref.real_gated_lru(ref_linear(h, weight, bias), d, conv_w, conv_b, gate_w, gate_b, lam, cache.conv_state,
+                              cache.state, ctx)
 
 
 # ------------------------------------------------------------------ matrix memory

@@ -1,5 +1,6 @@
 """Plain PyTorch statements of the ops of hybrid models: norms on a 32-bit residual, short convolution, gated linear
-attention, gated delta rule, matrix memory, paged latent attention, windowed attention with a sink, experts.
+attention, gated delta rule, matrix memory, real-gated recurrence, paged latent attention, windowed and chunked attention,
+experts, several residual streams.
 
 Like `reference.py`: the execution path on CPU tensors.  A batch is a concatenation of runs of rows, one run per
 request, with the request's state slot and the position of its first row; a run that starts at position 0 starts
@@ -7,6 +8,7 @@ from a zero state.
 """
 from __future__ import annotations
 
+import math
 from typing import List, Optional, Tuple
 
 import torch
@@ -56,13 +58,17 @@ def gelu_tanh_and_mul(gu, up_off: int, width: int):
 # ------------------------------------------------------------------ recurrent layers
 def short_conv(p, conv_w, conv_state, ctx):
     """silu(depthwise causal convolution) of the first C columns of p, per run; updates the kept inputs."""
+    return F.silu(causal_conv(p[:, :conv_w.shape[0]].float(), conv_w, conv_state, ctx))
+
+
+def causal_conv(x, conv_w, conv_state, ctx):
+    """Depthwise causal convolution of x [T, C] fp32, per run; updates the kept inputs."""
     C, taps = conv_w.shape
-    x = p[:, :C].float()
     out = torch.zeros_like(x)
     for _, lo, hi, start, slot in runs(ctx):
         past = x.new_zeros(taps - 1, C) if start == 0 else conv_state[slot]
         seq = torch.cat([past, x[lo:hi]])
-        out[lo:hi] = F.silu(sum(seq[j:j + hi - lo] * conv_w[:, j] for j in range(taps)))
+        out[lo:hi] = sum(seq[j:j + hi - lo] * conv_w[:, j] for j in range(taps))
         if taps > 1:
             conv_state[slot] = seq[hi - lo:]
     return out
@@ -112,6 +118,27 @@ def delta_rule(p, d, conv_w, a_log, dt_bias, norm_w, eps: float, conv_state, sta
             o[t] = torch.einsum("hdv,hd->hv", S, q[t])
         state[slot] = S
     return gated_head_norm(o, p[:, d.g:d.g + H * V], norm_w, eps, p.dtype)
+
+
+def real_gated_lru(p, d, conv_w, conv_b, gate_w, gate_b, lam, conv_state, state, ctx):
+    """d: `ops.hybrid.LruDims`; p packed projections with their biases.  S <- a S + sqrt(1 - a^2) i u per channel with
+    log a = -sharpness r softplus(lam); u = convolution of the x branch, r and i its block-diagonal gates; the y branch
+    multiplies the output."""
+    C, n = d.channels, d.channels // d.blocks
+    u = (causal_conv(p[:, d.x:d.x + C].float(), conv_w, conv_state, ctx) + conv_b).to(p.dtype).float()
+    z = torch.einsum("tbk,gbnk->gtbn", u.view(-1, d.blocks, n), gate_w.float()).reshape(2, -1, C)
+    r, i = torch.sigmoid(z + gate_b[:, None])
+    log_a = -d.sharpness * r * F.softplus(lam)
+    a, write = torch.exp(log_a), torch.sqrt(-torch.expm1(2 * log_a)) * i * u
+    o = torch.zeros_like(u)
+    for _, lo, hi, start, slot in runs(ctx):
+        S = state.new_zeros(C) if start == 0 else state[slot].clone()
+        for t in range(lo, hi):
+            S = a[t] * S + write[t]
+            o[t] = S
+        state[slot] = S
+    y = o * F.gelu(p[:, d.y:d.y + C].float(), approximate="tanh")
+    return _pad_to(y.to(p.dtype), -(-C // 8) * 8)
 
 
 # ------------------------------------------------------------------ latent attention
@@ -169,6 +196,29 @@ def add_norm(y, x, add: bool, norm_w, eps: float, experts=None):
     return _pad_to(n.to(y.dtype), y.shape[1])
 
 
+def embed_streams(ids, weight, width: int, streams: int, nxt, eps: float):
+    x = F.embedding(ids, weight)[:, None, :width].float().repeat(1, streams, 1)
+    return x, _streams_in(x, nxt, eps, weight.shape[1], weight.dtype)
+
+
+def _streams_in(x, nxt, eps: float, width: int, dtype):
+    c, w, b = nxt
+    u = x.sum(1) if c is None else torch.einsum("s,tsw->tw", c[: x.shape[1]], x)
+    u = u - u.mean(-1, keepdim=True)
+    return _pad_to((_rms(u, eps) * w + b).to(dtype), width)
+
+
+def mix_norm(y, x, connection, nxt, eps: float, dtype, experts=None):
+    """x [T, S, W] after a sublayer (in place) and the next one's input; connection [in (S) | out (S) | mix (S * S, from * S +
+    to)]."""
+    S, W = x.shape[1:]
+    width = (y if y is not None else experts).shape[1]
+    total = sum(t[:, :W].float() for t in (y, experts) if t is not None)
+    out, mix = connection[S:2 * S], connection[2 * S:].view(S, S)
+    x.copy_(torch.einsum("st,nsw->ntw", mix, x) + out[:, None] * total[:, None])
+    return _streams_in(x, nxt, eps, width, dtype)
+
+
 def glu(gate, up, act: str, limit: float):
     """act(gate) * up ("silu"), or the clamped form ("clamped"): g * sigmoid(1.702 g) * (u + 1) with g = min(gate, limit)
     and u = up clamped to +-limit."""
@@ -177,6 +227,20 @@ def glu(gate, up, act: str, limit: float):
         return (F.silu(g) * u).to(gate.dtype)
     g, u = g.clamp(max=limit), u.clamp(-limit, limit)
     return (g * torch.sigmoid(1.702 * g) * (u + 1)).to(gate.dtype)
+
+
+def route_by_score(z, correction, top: int, groups: int, keep: int):
+    """Chosen experts [T, top] and their weights: of the `keep` groups (equal, of neighbours) whose two largest choice scores
+    sigmoid(z) + correction have the largest sums, the `top` experts with the largest choice scores; weights are the
+    scores without correction over their sum."""
+    T, E = z.shape[0], correction.numel()
+    s = torch.sigmoid(z[:, :E].float())
+    choice = (s + correction).view(T, groups, -1)
+    best = choice.topk(min(2, choice.shape[2]), -1).values.sum(-1).topk(keep, -1).indices
+    out = torch.ones(T, groups, dtype=torch.bool).scatter(1, best, False)
+    ids = choice.masked_fill(out[..., None], float("-inf")).view(T, E).topk(top, -1).indices
+    w = s.gather(1, ids)
+    return ids, w / (w.sum(-1, keepdim=True) + 1e-20)
 
 
 def experts(h, ids, weights, w_gate_up, w_down, ff: int, act: str, limit: float):
@@ -191,40 +255,57 @@ def experts(h, ids, weights, w_gate_up, w_down, ff: int, act: str, limit: float)
     return out
 
 
-def rope_pairs(x, positions, base: float, dims: int):
-    """Interleaved rotation: columns 2i and 2i + 1 below `dims` of x [T, H, D] turn by position * base^(-2i / dims)."""
-    i = torch.arange(dims // 2, dtype=torch.float64, device=x.device)
-    a = positions.double()[:, None, None] * base ** (-2 * i / dims)
-    c, s = a.cos().float(), a.sin().float()
-    u, v = x[..., 0:dims:2].float(), x[..., 1:dims:2].float()
+def rope_rows(x, positions, turns, dims: int, half: bool, size: float):
+    """Rotation of the first `dims` columns of x [T, H, D] by position * turns: columns 2i and 2i + 1 together, or (half) i
+    and i + dims / 2; cos and sin times `size`."""
+    a = 2 * math.pi * positions.double()[:, None, None] * turns
+    c, s = (size * a.cos()).float(), (size * a.sin()).float()
+    x = x.float()
+    if half:
+        return torch.cat([_rotate(x[..., :dims], c, s), x[..., dims:]], -1)
+    u, v = x[..., 0:dims:2], x[..., 1:dims:2]
     turned = torch.stack([u * c - v * s, v * c + u * s], -1).flatten(-2)
-    return torch.cat([turned, x[..., dims:].float()], -1)
+    return torch.cat([turned, x[..., dims:]], -1)
 
 
-def windowed_attention(p, d, q_norm, k_norm, sink, eps: float, k_rows, v_rows, positions, ctx, out):
-    """Stores the batch's keys and values (the raw keys) in the pages and writes attention times sigmoid(gate) to `out`.
-    d: `ops.hybrid.WindowDims`; a query at position i sees the last d.window positions up to i (0: all)."""
-    T, H, G, D = p.shape[0], d.heads, d.kv_heads, d.dim
+def windowed_attention(p, d, turns, q_norm, k_norm, sink, eps: float, k_rows, v_rows, positions, ctx, out, bias=None):
+    """Stores the batch's keys and values in the pages and writes attention (times sigmoid(gate)) to `out`.
+    d: `ops.hybrid.WindowDims`."""
+    T, H, G, D, V = p.shape[0], d.heads, d.kv_heads, d.dim, d.value_dim
+    if bias is not None:
+        p = p + bias
     q, k = p[:, d.q:d.q + H * D].float(), p[:, d.k:d.k + G * D]
-    q = rope_pairs((_rms(q, eps) * q_norm).view(T, H, D), positions, d.base, d.rot_dims).to(p.dtype)
-    kn = rope_pairs((_rms(k.float(), eps) * k_norm).view(T, G, D), positions, d.base, d.rot_dims)
+    v = k if d.v is None else p[:, d.v:d.v + G * V]
+    rope = positions, turns, d.rot_dims, d.half, d.rot_size
+    q = rope_rows((_rms(q, eps) * q_norm).view(T, H, D), *rope).to(p.dtype)
+    kn = rope_rows((_rms(k.float(), eps) * k_norm).view(T, G, D), *rope)
     ok = ctx.slot_mapping >= 0
     slots = ctx.slot_mapping[ok].long()
     bs = k_rows.shape[2]
     k_rows[slots // bs, :, slots % bs, :D] = kn[ok].to(k_rows.dtype)
-    v_rows[slots // bs, :, slots % bs, :D] = k.reshape(T, G, D)[ok].to(v_rows.dtype)
-    o = torch.zeros(T, H, D)
+    v_rows[slots // bs, :, slots % bs, :V] = v.reshape(T, G, V)[ok].to(v_rows.dtype)
+    o = torch.zeros(T, H, V)
     for i, lo, hi, start, _ in runs(ctx):
         n = start + hi - lo
         blocks = ctx.block_tables[i][: -(-n // bs)].long()
-        ks, vs = (r[blocks][..., :D].transpose(1, 2).reshape(-1, G, D)[:n].float().repeat_interleave(H // G, 1)
-                  for r in (k_rows, v_rows))
+        ks, vs = (r[blocks][..., :w].transpose(1, 2).reshape(-1, G, w)[:n].float().repeat_interleave(H // G, 1)
+                  for r, w in ((k_rows, D), (v_rows, V)))
         s = torch.einsum("ihd,jhd->hij", q[lo:hi].float(), ks) * d.scale
-        back = torch.arange(start, n)[:, None] - torch.arange(n)[None, :]
-        hidden = back < 0 if d.window <= 0 else (back < 0) | (back >= d.window)
-        s = torch.cat([s.masked_fill(hidden, float("-inf")), sink[:, None, None].expand(-1, hi - lo, 1)], -1)
-        o[lo:hi] = torch.einsum("hij,jhd->ihd", torch.softmax(s, -1)[..., :-1], vs)
-    y = o.reshape(T, H * D) * torch.sigmoid(p[:, d.g:d.g + H * D].float())
+        if d.softcap:
+            s = d.softcap * torch.tanh(s / d.softcap)
+        at, key = torch.arange(start, n)[:, None], torch.arange(n)[None, :]
+        hidden = key > at
+        if d.window > 0:
+            hidden |= at - key >= d.window
+        if d.chunk > 0:
+            hidden |= key < at // d.chunk * d.chunk
+        s = s.masked_fill(hidden, float("-inf"))
+        if sink is not None:
+            s = torch.cat([s, sink[:, None, None].expand(-1, hi - lo, 1)], -1)
+        o[lo:hi] = torch.einsum("hij,jhd->ihd", torch.softmax(s, -1)[..., :n], vs)
+    y = o.reshape(T, H * V)
+    if d.g is not None:
+        y = y * torch.sigmoid(p[:, d.g:d.g + H * V].float())
     out.copy_(_pad_to(y.to(p.dtype), out.shape[1]))
 
 
