@@ -28,6 +28,8 @@ class TokenReplay:
         sch, runner = self.llm.scheduler, self.llm.model_runner
         pieces = []
         for e in entries:
+            if any(not 0 <= w < len(e["tokens"]) for w in e.get("want", ())):
+                raise ValueError(f"request {e['id']!r}: a wanted place is not among its {len(e['tokens'])} tokens")
             seq = self.live.get(e["id"])
             if seq is None:
                 seq = self.live[e["id"]] = Sequence(e["tokens"])

@@ -41,9 +41,10 @@ def config(layers, width=72, vocab=110, eps=1e-5, streams=3, logit_scale=1.5, lo
     return cfg
 
 
-def weights(cfg, seed=0):
+def weights(cfg, seed=0, decisive=False):
     """Random tensors by checkpoint name (values exact in bf16).  Attention is peaked, decays range from forgetting to keeping,
-    the feed-forward reaches its clamps, choice scores are of either sign, streams mix without growing."""
+    the feed-forward reaches its clamps, choice scores are of either sign, streams mix without growing.  `decisive`: the
+    corrections alone choose the experts, so that no 16-bit run decides a close call differently (the weights still vary)."""
     g = torch.Generator().manual_seed(seed)
     W, V, S = cfg["width"], cfg["vocab"], cfg["streams"]
     out = {}
@@ -99,6 +100,8 @@ def weights(cfg, seed=0):
                 put(f"{p}e{e}.{n}", *shape)
         put(p + "router", E, W, scale=2 * W ** -0.5)
         put(p + "correction", E, scale=0.3, mean=-0.5)
+        if decisive:
+            out[p + "correction"] = 1.5 * torch.randperm(E, generator=g).float().mul(1.25).sub(E)
     norm("final.norm")
     put("head", V, W)
     return out
