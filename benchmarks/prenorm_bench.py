@@ -100,7 +100,7 @@ def kernel_table():
             add("routing by table", case, lambda: hybrid.route_by_table(ids, table, EXPERTS, ctx), t * (8 + TOP * 12))
     del gu, down, wg, wd
     # ---- windowed attention (norms, rotation, store, attention, gate)
-    cols = [H, G, D, 64, WINDOW, 0, H * D, (H + G) * D]
+    cols = hybrid.WindowDims(H, G, D, 64, D ** -0.5, WINDOW, 0, H * D, (H + G) * D).sizes()
     freq = hybrid.rope_turns(1e4, 64).cuda()
     qn, kn, sink = torch.ones(H * D, device=dev), torch.ones(G * D, device=dev), torch.zeros(H, device=dev)
     cos_sin = torch.ones(16384, D, device=dev, dtype=torch.float32)
@@ -137,7 +137,7 @@ def kernel_table():
         out = torch.empty(t, H * D, device=dev, dtype=bf)
         ctx = (pos + 1).int()
         add(f"norms + store + windowed {kind} attention", case,
-            lambda: e.windowed_attention(pr, cols, D ** -0.5, freq, qn, kn, sink, 1e-6, kc, vc, pos, slots, bt, lens, cu,
+            lambda: e.windowed_attention(pr, cols, D ** -0.5, 0.0, 1.0, freq, None, qn, kn, sink, 1e-6, kc, vc, pos, slots, bt, lens, cu,
                                          seq if prefill else None, ctx if prefill else None, n if prefill else 0, 0, out, 0),
             io + t * H * D * 2 + b * min(n, WINDOW) * kv, seen * H * 4 * D, like=f"rope + store + {kind} attention (dense)")
         del kc, vc, qkv

@@ -101,7 +101,7 @@ def weights(cfg, seed=0, decisive=False):
         put(p + "router", E, W, scale=2 * W ** -0.5)
         put(p + "correction", E, scale=0.3, mean=-0.5)
         if decisive:
-            out[p + "correction"] = 1.5 * torch.randperm(E, generator=g).float().mul(1.25).sub(E)
+            out[p + "correction"] = -2.5 * 2.0 ** torch.randperm(E, generator=g).float()      # sums of two differ as well
     norm("final.norm")
     put("head", V, W)
     return out

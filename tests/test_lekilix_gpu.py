@@ -175,7 +175,7 @@ def _rnd(*shape, scale=1.0, dtype=torch.bfloat16, seed=0):
 def test_windowed_attention_op(H, G, D, page, window):
     """Prefill of several requests (whole, continued, short) and decoding with context splits, peaked scores, strong sinks."""
     from fastcache_b200.layers.windowed_attention import padded_dim
-    from fastcache_b200.ops.hybrid import rope_turns
+    from fastcache_b200.ops.hybrid import WindowDims, rope_turns
     from fastcache_b200.ops.loader import ext
     rot, eps, base, scale = D // 2, 1e-5, 1e4, D ** -0.5
     ctx = [700, 64, 130, 1, 1290]
@@ -187,7 +187,7 @@ def test_windowed_attention_op(H, G, D, page, window):
     q_norm, k_norm = _rnd(H * D, dtype=torch.float32, seed=7).abs() + 1.5, _rnd(G * D, dtype=torch.float32, seed=8).abs() + 0.5
     sink = _rnd(H, scale=3.0, dtype=torch.float32, seed=9)
     freq = rope_turns(base, rot).cuda()
-    cols = [H, G, D, rot, window, 0, H * D, (H + G) * D]
+    cols = WindowDims(H, G, D, rot, scale, window, 0, H * D, (H + G) * D).sizes()
     for prefill in (True, False):
         pools = [torch.full((5 * pages, G, page, P), 50.0, device="cuda", dtype=torch.bfloat16) for _ in range(2)]
 
@@ -199,7 +199,7 @@ def test_windowed_attention_op(H, G, D, page, window):
             out = torch.full((rows.shape[0], -(-H * D // 8) * 8), 7.0, device="cuda", dtype=torch.bfloat16)
             end = torch.tensor([s + n for s, n in zip(start, lens)], dtype=torch.int32, device="cuda")
             cu = torch.tensor([0] + lens, dtype=torch.int32).cumsum(0).int().cuda() if is_prefill else None
-            ext().windowed_attention(ext().as_projection(rows), cols, scale, freq, q_norm, k_norm, sink, eps, *pools, pos, slots,
+            ext().windowed_attention(ext().as_projection(rows), cols, scale, 0.0, 1.0, freq, None, q_norm, k_norm, sink, eps, *pools, pos, slots,
                                      bt.cuda(), end, cu, seq.int().cuda() if is_prefill else None,
                                      (pos + 1).int() if is_prefill else None, max(lens), 0, out, 0)
             return out
