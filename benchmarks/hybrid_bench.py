@@ -255,6 +255,9 @@ def run(steps=5, small=False, kernels=True, model="bagedra"):
     if model == "lekilix":
         from benchmarks import prenorm_bench
         make, table = prenorm_bench.model_config, prenorm_bench.kernel_table
+    elif model == "duperax":
+        from benchmarks import streams_bench
+        make, table = streams_bench.model_config, streams_bench.kernel_table
     sizes = {"2k": SIZES["2k"]} if small else SIZES
     out = {"layers": LAYERS, "sizes": {}}
     for name, size in sizes.items():

@@ -133,17 +133,20 @@ std::tuple<Tensor, Tensor, Tensor> route_by_score(const Tensor& h, const Tensor&
 }
 
 // ------------------------------------------------------------------ real-gated linear recurrent unit
-// d: channels, blocks, first columns of the y and x branches.  impl: 0 choose, 1 general
+// d: channels, blocks, first columns of the y and x branches.  impl: 0 choose, 1 general.  An empty weight: h holds the finished
+// branches (kernel benchmarks; for the form of prefill batches with y's activation applied)
 Tensor real_gated_lru(const Tensor& h, const Tensor& weight, const OptTensor& bias, const std::vector<int64_t>& d, double sharpness,
                       const Tensor& conv_w, const Tensor& conv_b, const Tensor& gate_w, const Tensor& gate_b, const Tensor& lam,
                       Tensor conv_state, Tensor state, const OptTensor& cu, const Tensor& ctx, const Tensor& slots, int64_t max_len,
                       const OptTensor& row_seq, int64_t impl) {
   TORCH_CHECK(d.size() == 4, "recurrent unit: four sizes and offsets");
-  check_product(h, weight);
-  const int64_t T = h.size(0), C = d[0], blocks = d[1], S = state.size(0);
+  const bool finished = weight.numel() == 0;
+  if (finished) check_rows(h, "branches");
+  else check_product(h, weight);
+  const int64_t T = h.size(0), C = d[0], blocks = d[1], S = state.size(0), cols = finished ? h.size(1) : weight.size(0);
   const bool f32 = is_f32(h), prefill = cu.has_value() && cu->defined();
   TORCH_CHECK(C > 0 && blocks > 0 && C % blocks == 0, "channels must split into equal blocks");
-  TORCH_CHECK(d[2] >= 0 && d[3] >= 0 && d[2] % 8 == 0 && d[3] % 8 == 0 && d[2] + C <= weight.size(0) && d[3] + C <= weight.size(0),
+  TORCH_CHECK(d[2] >= 0 && d[3] >= 0 && d[2] % 8 == 0 && d[3] % 8 == 0 && d[2] + C <= cols && d[3] + C <= cols,
               "bad projection columns");
   TORCH_CHECK(conv_w.dim() == 2, "the convolution must be [channels, taps]");
   const int64_t taps = conv_w.size(1), n = C / blocks;
@@ -156,7 +159,7 @@ Tensor real_gated_lru(const Tensor& h, const Tensor& weight, const OptTensor& bi
   check_f32(conv_state, "convolution state", S * (taps - 1) * C);
   check_elem(gate_w, "gates");
   TORCH_CHECK(is_f32(gate_w) == f32 && gate_w.is_contiguous() && gate_w.numel() == 2 * C * n, "gates must be [2, blocks, n, n]");
-  check_bias(bias, weight.size(0), f32);
+  check_bias(bias, cols, f32);
   c10::cuda::CUDAGuard guard(h.device());
   Tensor out = torch::empty({T, pad8(int(C))}, h.options()), u = torch::empty({T, C}, h.options());
   fc::LruParams p;
@@ -192,7 +195,14 @@ Tensor real_gated_lru(const Tensor& h, const Tensor& weight, const OptTensor& bi
   const bool tc = !f32 && impl != 1 && fc::lru_tc_supported(p);
   Projection xy;
   Tensor x, y;
-  if (tc && prefill) {
+  if (finished) {
+    p.x.p = p.y.p = h.data_ptr();
+    p.x.ld = p.y.ld = h.stride(0);
+    p.off_y = int(d[2]);
+    p.off_x = int(d[3]);
+    p.gelu = !(tc && prefill);
+    p.bias_y = bias_at(d[2]);
+  } else if (tc && prefill) {
     // the branches as two finished products, bias and gelu in the epilogue of one
     const auto gw = gemm_workspace(ws_of(h));
     const int sms = fc::stream_sm_limit(stream_now()), K = int(h.size(1));
