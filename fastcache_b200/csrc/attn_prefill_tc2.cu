@@ -262,7 +262,7 @@ prefill_attn_tc2_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
     const int qpos = offset + qrow;                          // last key position this row may see
     const int first = attn_first(p.opt, qpos), first_last = attn_first(p.opt, offset + q0 + x * P2_BM + P2_BM - 1);
     const ScoreScale sscale = score_scale(p.opt, p.scale_log2);
-    const float scale_log2 = sscale.cap ? 1.f : p.scale_log2;            // capped scores are in log2 units already
+    const float scale_log2 = sscale.cap ? sscale.out : p.scale_log2;     // capped: of tanh(score / cap)
     float m_ref = -INFINITY, l = 0.f;                        // -inf: no visible key yet
     bool ok = true;
     for (int j = f_x; j < n_x && ok; ++j) {
@@ -282,12 +282,14 @@ prefill_attn_tc2_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
         float top = 0.f;
 #pragma unroll
         for (int t = 0; t < 128; ++t) top = fmaxf(top, fabsf(__uint_as_float(s[t])));
-        if (__any_sync(__activemask(), top * sscale.in > TANH_POLY_MAX)) {
-#pragma unroll
-          for (int t = 0; t < 128; ++t) s[t] = __float_as_uint(sscale.out * tanh_exp(__uint_as_float(s[t]) * sscale.in));
+        top *= sscale.in;
+        if (!__any_sync(__activemask(), top > TANH_SMALL)) {
+          tanh_poly<3>(s, sscale.in);
+        } else if (!__any_sync(__activemask(), top > TANH_MID)) {
+          tanh_poly<5>(s, sscale.in);
         } else {
 #pragma unroll
-          for (int t = 0; t < 128; ++t) s[t] = __float_as_uint(sscale.out * tanh_poly(__uint_as_float(s[t]) * sscale.in));
+          for (int t = 0; t < 128; ++t) s[t] = __float_as_uint(tanh_exp(__uint_as_float(s[t]) * sscale.in));
         }
       }
       if (need_mask) {

@@ -699,12 +699,20 @@ static GemmParams prefill_params(void* c, int M, int N, int K, long long ldc, co
 void gemm_bf16_wide(const void* x, const void* w, void* c, int M, int N, int K, long long ldx, long long ldw, long long ldc,
                     int wide0, int wide_n, float* wide, const GemmWorkspace& ws, int sm_limit, cudaStream_t stream) {
   if (M <= 0 || N <= 0 || K <= 0) return;
-  constexpr int BN = 256;
   const int sms = sm_limit > 0 ? sm_limit : gemm_num_sms();
   GemmParams p = prefill_params(c, M, N, K, ldc, ws);
   p.wide = wide;
   p.wide0 = wide0;
   p.wide_n = wide_n;
+  if (N <= 128) {
+    constexpr int BN = 128;
+    p.num_n = 1;
+    p.total_work = p.num_m;
+    launch_one<BN, 6, false, GLU_NONE, GF_WIDE>(make_tmap_bf16_2d(x, M, K, ldx, BM, BK), make_tmap_bf16_2d(w, N, K, ldw, BN, BK), p,
+                                                std::min(p.total_work, sms), stream);
+    return;
+  }
+  constexpr int BN = 256;
   p.num_n = (N + BN - 1) / BN;
   p.total_work = p.num_m * p.num_n;
   launch_one<BN, 4, false, GLU_NONE, GF_WIDE>(make_tmap_bf16_2d(x, M, K, ldx, BM, BK), make_tmap_bf16_2d(w, N, K, ldw, BN, BK),

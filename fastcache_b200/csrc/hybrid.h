@@ -346,7 +346,10 @@ struct RouteTable {
 void launch_route_table(const RouteTable& p, cudaStream_t s);
 // choice by score: see route_by_score in ops/hybrid.py
 struct RouteScore {
-  ProjSrc logits;                    // fp32 [T, E], first column 0
+  ProjSrc logits;                    // fp32 [T, E], first column 0; or `h` and the router's weights (up to ROUTE_SMALL tokens)
+  const void *h = nullptr, *w = nullptr;      // [T, ld_h], [E, K]; K a multiple of 8
+  long long ld_h = 0;
+  int K = 0;
   const float* correction = nullptr; // [E]
   const int* ctx = nullptr;          // as in RouteTable
   int T = 0, top = 0, E = 0, groups = 1, keep = 1;
@@ -357,9 +360,9 @@ struct RouteScore {
   int* counts = nullptr;             // scratch [route_score_blocks(T), E]
   int token_at = 0;                  // (set by the launcher)
 };
-constexpr int ROUTE_ROWS = 64;       // tokens per CTA of the large form
+constexpr int ROUTE_ROWS = 64, ROUTE_SMALL = 256;    // tokens per CTA of the large form, most tokens of the small one
 inline int route_score_blocks(int T) { return (T + ROUTE_ROWS - 1) / ROUTE_ROWS; }
-void launch_route_score(const RouteScore& p, cudaStream_t s);
+void launch_route_score(const RouteScore& p, bool f32, cudaStream_t s);
 // decode-size expert products (moe_gemm.cu): partial [splits, pairs, N] of x [pairs, K] and w [E, N, K]; an expert has at
 // most max_rows <= 256 rows
 int moe_skinny_splits(int max_rows, int pairs, int E, int N, int K);

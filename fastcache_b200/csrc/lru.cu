@@ -11,6 +11,7 @@
 #include <algorithm>
 #include <stdexcept>
 #include <string>
+#include <type_traits>
 
 #include "gemm.h"
 #include "hybrid.cuh"
@@ -79,18 +80,29 @@ __device__ __forceinline__ void advance_conv_state(const LruParams& p, const Run
 }
 
 // ================================================================= convolution
-// VEC: a thread owns four channels (C, offsets and pitches multiples of 4) of LC_ROWS rows and slides the window of up to
-// four taps in registers
-constexpr int LC_ROWS = 16;
+// A thread owns four channels (C, offsets and pitches multiples of 4) of some rows and slides the window of up to four taps in
+// registers.  Rows are requested LC_BATCH at a time, one batch ahead.
+constexpr int LC_ROWS = 32, LC_BATCH = 8;
+// four elements of a finished projection as they are
 template <typename T>
-__device__ __forceinline__ void branch_x4(const LruParams& p, long long row, int c, const float (&bias)[4], float (&x)[4]) {
-  const float4 v = proj_at4<T>(p.x, row, p.off_x + c);
-  x[0] = v.x + bias[0];
-  x[1] = v.y + bias[1];
-  x[2] = v.z + bias[2];
-  x[3] = v.w + bias[3];
-}
-template <typename T>
+struct Raw4;
+template <>
+struct Raw4<float> {
+  float4 v;
+  __device__ __forceinline__ void load(const float* p) { v = __ldcg(reinterpret_cast<const float4*>(p)); }
+  __device__ __forceinline__ float4 get() const { return v; }
+};
+template <>
+struct Raw4<bf16> {
+  uint2 v;
+  __device__ __forceinline__ void load(const bf16* p) { v = __ldcg(reinterpret_cast<const uint2*>(p)); }
+  __device__ __forceinline__ float4 get() const {
+    return make_float4(__uint_as_float(v.x << 16), __uint_as_float(v.x & 0xffff0000u), __uint_as_float(v.y << 16),
+                       __uint_as_float(v.y & 0xffff0000u));
+  }
+};
+// PART: the projection is still partial sums
+template <typename T, int BATCH, bool PART>
 __global__ void __launch_bounds__(256)
 lru_conv4_kernel(const LruParams p, int rows) {
   const int c = (blockIdx.x * 256 + threadIdx.x) * 4, t0 = blockIdx.y * rows, t1 = min(p.T, t0 + rows);
@@ -107,54 +119,104 @@ lru_conv4_kernel(const LruParams p, int rows) {
   pdl_wait();
   if (!on) return;
   float x1[4] = {}, x2[4] = {}, x3[4] = {};                  // inputs one, two and three rows back
-  int b = -1;
   Run run{};
-  const bool advance = p.runs.cu == nullptr;
+  int run_end = 0;                                           // row after the current run
   auto back = [&](int t, int j, float (&x)[4]) {             // input j rows before row t of the current run
     x[0] = x[1] = x[2] = x[3] = 0.f;
     const int i = t - run.lo - j;
     if (j >= p.taps || run.slot < 0) return;
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
     if (i >= 0) {
-      branch_x4<T>(p, t - j, c, bias, x);
+      v = proj_at4<T>(p.x, t - j, p.off_x + c);
+      v = make_float4(v.x + bias[0], v.y + bias[1], v.z + bias[2], v.w + bias[3]);
     } else if (run.start + i >= 0) {
-      const float4 s = __ldcg(reinterpret_cast<const float4*>(p.conv_state + ((long long)run.slot * (p.taps - 1) + p.taps - 1 + i) * p.C + c));
-      x[0] = s.x;
-      x[1] = s.y;
-      x[2] = s.z;
-      x[3] = s.w;
+      v = __ldcg(reinterpret_cast<const float4*>(p.conv_state + ((long long)run.slot * (p.taps - 1) + p.taps - 1 + i) * p.C + c));
+    }
+    x[0] = v.x;
+    x[1] = v.y;
+    x[2] = v.z;
+    x[3] = v.w;
+  };
+  Raw4<typename std::conditional<PART, float, T>::type> nxt[BATCH], cur[BATCH];
+  auto request = [&](int t) {
+#pragma unroll
+    for (int i = 0; i < BATCH; ++i) {
+      const long long row = min(t + i, t1 - 1);
+      if constexpr (PART) nxt[i].v = proj_at4<T>(p.x, row, p.off_x + c);
+      else nxt[i].load(reinterpret_cast<const T*>(p.x.p) + row * p.x.ld + p.off_x + c);
     }
   };
-  float nxt[4];
-  branch_x4<T>(p, t0, c, bias, nxt);
-#pragma unroll 2
-  for (int t = t0; t < t1; ++t) {
-    const int bt = p.row_seq != nullptr ? p.row_seq[t] : t;
-    if (bt != b) {
-      b = bt;
-      run = get_run(p.runs, b);
-      back(t, 1, x1);
-      back(t, 2, x2);
-      back(t, 3, x3);
-    }
-    float x0[4], y[4];
+  request(t0);
+  for (int tb = t0; tb < t1; tb += BATCH) {
 #pragma unroll
-    for (int i = 0; i < 4; ++i) x0[i] = nxt[i];
-    if (t + 1 < t1) branch_x4<T>(p, t + 1, c, bias, nxt);
+    for (int i = 0; i < BATCH; ++i) cur[i] = nxt[i];
+    if (tb + BATCH < t1) request(tb + BATCH);
 #pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      y[i] = cb[i] + fmaf(x3[i], w[3][i], fmaf(x2[i], w[2][i], fmaf(x1[i], w[1][i], x0[i] * w[0][i])));
-      x3[i] = x2[i];
-      x2[i] = x1[i];
-      x1[i] = x0[i];
-    }
-    store4(reinterpret_cast<T*>(p.u) + (long long)t * p.C + c, y[0], y[1], y[2], y[3]);
-    if (advance && run.slot >= 0) {                          // a run of one row: this thread read what it now replaces
-      float* s = p.conv_state + (long long)run.slot * (p.taps - 1) * p.C + c;
-      if (p.taps > 1) *reinterpret_cast<float4*>(s + (long long)(p.taps - 2) * p.C) = make_float4(x1[0], x1[1], x1[2], x1[3]);
-      if (p.taps > 2) *reinterpret_cast<float4*>(s + (long long)(p.taps - 3) * p.C) = make_float4(x2[0], x2[1], x2[2], x2[3]);
-      if (p.taps > 3) *reinterpret_cast<float4*>(s + (long long)(p.taps - 4) * p.C) = make_float4(x3[0], x3[1], x3[2], x3[3]);
+    for (int k = 0; k < BATCH; ++k) {
+      const int t = tb + k;
+      if (t >= t1) break;
+      if (t >= run_end) {
+        run = get_run(p.runs, p.row_seq != nullptr ? p.row_seq[t] : t);
+        run_end = run.lo + run.len;
+        back(t, 1, x1);
+        back(t, 2, x2);
+        back(t, 3, x3);
+      }
+      const float4 raw = cur[k].get();
+      const float x0[4] = {raw.x + bias[0], raw.y + bias[1], raw.z + bias[2], raw.w + bias[3]};
+      float y[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        y[i] = cb[i] + fmaf(x3[i], w[3][i], fmaf(x2[i], w[2][i], fmaf(x1[i], w[1][i], x0[i] * w[0][i])));
+        x3[i] = x2[i];
+        x2[i] = x1[i];
+        x1[i] = x0[i];
+      }
+      store4(reinterpret_cast<T*>(p.u) + (long long)t * p.C + c, y[0], y[1], y[2], y[3]);
     }
   }
+}
+// the same for runs of one row: every load that does not depend on another is requested at once
+template <typename T>
+__global__ void __launch_bounds__(256)
+lru_conv4_step_kernel(const LruParams p) {
+  const int c = (blockIdx.x * 256 + threadIdx.x) * 4, t = blockIdx.y, back = p.taps - 1;
+  const bool on = c < p.C;
+  float w[4][4], bias[4], cb[4];                             // w[tap: 0 = current row][channel]
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+#pragma unroll
+    for (int j = 0; j < 4; ++j) w[j][i] = on && j < p.taps ? p.conv_w[(long long)(c + i) * p.taps + p.taps - 1 - j] : 0.f;
+    bias[i] = on && p.bias_x != nullptr ? Elem<T>::get(reinterpret_cast<const T*>(p.bias_x)[c + i]) : 0.f;
+    cb[i] = on ? p.conv_b[c + i] : 0.f;
+  }
+  pdl_launch_dependents();
+  pdl_wait();
+  if (!on) return;
+  const Run run = get_run(p.runs, t);
+  float* s = p.conv_state + (long long)max(run.slot, 0) * back * p.C + c;
+  float4 old[3];                                             // old[j]: input j + 1 rows back
+#pragma unroll
+  for (int j = 0; j < 3; ++j) {
+    old[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (j < back) old[j] = __ldcg(reinterpret_cast<const float4*>(s + (long long)(back - 1 - j) * p.C));
+  }
+  const float4 raw = proj_at4<T>(p.x, t, p.off_x + c);
+  const float4 x = make_float4(raw.x + bias[0], raw.y + bias[1], raw.z + bias[2], raw.w + bias[3]);
+  float4 y = make_float4(fmaf(x.x, w[0][0], cb[0]), fmaf(x.y, w[0][1], cb[1]), fmaf(x.z, w[0][2], cb[2]), fmaf(x.w, w[0][3], cb[3]));
+#pragma unroll
+  for (int j = 0; j < 3; ++j) {
+    if (run.slot < 0 || run.start <= j) old[j] = make_float4(0.f, 0.f, 0.f, 0.f);       // before the start
+    y.x = fmaf(old[j].x, w[j + 1][0], y.x);
+    y.y = fmaf(old[j].y, w[j + 1][1], y.y);
+    y.z = fmaf(old[j].z, w[j + 1][2], y.z);
+    y.w = fmaf(old[j].w, w[j + 1][3], y.w);
+  }
+  store4(reinterpret_cast<T*>(p.u) + (long long)t * p.C + c, y.x, y.y, y.z, y.w);
+  if (run.slot < 0) return;
+#pragma unroll
+  for (int j = 0; j < 3; ++j)
+    if (j < back) *reinterpret_cast<float4*>(s + (long long)(back - 1 - j) * p.C) = j == 0 ? x : old[j - 1];
 }
 // any size: one thread per (row, channel)
 template <typename T>
@@ -210,14 +272,15 @@ lru_scan_kernel(const LruParams p) {
 }
 
 // ================================================================= step: runs of one row, bf16
-// Grid (16 channels, 16 requests); the four warps share the sum over a block's inputs.  The weights do not depend on the
-// kernel before and are requested ahead of the wait for it.
+// Grid (16 channels, 8 NT requests); the four warps share the sum over a block's inputs.  The weights do not depend on the
+// kernel before and are requested ahead of the wait for it; what the recurrence reads is requested before the products.
 constexpr int LS_KSTEPS = 4;             // 16-wide steps per warp: blocks of up to 256 channels
+template <int NT>
 __global__ void __launch_bounds__(128)
 lru_step_kernel(const LruParams p) {
-  __shared__ float s_acc[4][2][16][17];                      // [warp][gate][request][channel]
+  __shared__ float s_acc[4][2][NT * 8][17];                  // [warp][gate][request][channel]
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
-  const int c0 = blockIdx.x * 16, r0 = blockIdx.y * 16, n = p.C / p.blocks, blk = c0 / n, steps = n / 16;
+  const int c0 = blockIdx.x * 16, r0 = blockIdx.y * NT * 8, n = p.C / p.blocks, blk = c0 / n, steps = n / 16;
   uint32_t wa[2][LS_KSTEPS][4];
 #pragma unroll
   for (int m = 0; m < 2; ++m) {
@@ -241,54 +304,78 @@ lru_step_kernel(const LruParams p) {
   pdl_launch_dependents();
   pdl_wait();
   const bf16* u = reinterpret_cast<const bf16*>(p.u);
-  float acc[2][2][4];                                        // [gate][8 requests]
+  // this thread's requests r0 + threadIdx.x / 16 + 8 i; rows past the batch repeat its last one, so that no load is conditional
+  int slot[NT], row_i[NT];
+  float S[NT], y[NT];
+  unsigned short u16[NT];
+  bool first[NT];
+#pragma unroll
+  for (int i = 0; i < NT; ++i) {
+    row_i[i] = min(r0 + (threadIdx.x >> 4) + i * 8, p.T - 1);
+    const Run run = get_run(p.runs, row_i[i]);
+    slot[i] = run.slot;
+    first[i] = run.start <= 0;
+    u16[i] = __ldcg(reinterpret_cast<const unsigned short*>(u) + (long long)row_i[i] * p.C + c);
+    y[i] = p.bias_y != nullptr ? __bfloat162float(reinterpret_cast<const bf16*>(p.bias_y)[c]) : 0.f;
+  }
+#pragma unroll
+  for (int i = 0; i < NT; ++i) S[i] = __ldcg(p.state + (long long)max(slot[i], 0) * p.C + c);
+  if (p.y.part != nullptr) {
+#pragma unroll 4
+    for (int k = 0; k < p.y.splits; ++k)
+#pragma unroll
+      for (int i = 0; i < NT; ++i) y[i] += __ldcg(p.y.part + k * p.y.part_stride + row_i[i] * p.y.part_ld + p.off_y + c);
+  } else {
+#pragma unroll
+    for (int i = 0; i < NT; ++i)
+      y[i] += __uint_as_float(uint32_t(__ldcg(reinterpret_cast<const unsigned short*>(p.y.p) + row_i[i] * p.y.ld + p.off_y + c)) << 16);
+  }
+  float acc[2][NT][4];                                       // [gate][8 requests]
 #pragma unroll
   for (int m = 0; m < 2; ++m)
 #pragma unroll
-    for (int x = 0; x < 2; ++x) acc[m][x][0] = acc[m][x][1] = acc[m][x][2] = acc[m][x][3] = 0.f;
+    for (int x = 0; x < NT; ++x) acc[m][x][0] = acc[m][x][1] = acc[m][x][2] = acc[m][x][3] = 0.f;
 #pragma unroll
   for (int i = 0; i < LS_KSTEPS; ++i) {
     const int ks = warp + i * 4;
     if (ks >= steps) break;
+    uint32_t b0[NT], b1[NT];
 #pragma unroll
-    for (int x = 0; x < 2; ++x) {
-      const int row = r0 + x * 8 + g;
-      uint32_t b0 = 0u, b1 = 0u;
-      if (row < p.T) {
-        const uint32_t* q = reinterpret_cast<const uint32_t*>(u + (long long)row * p.C + blk * n + ks * 16 + 2 * t);
-        b0 = __ldcg(q);
-        b1 = __ldcg(q + 4);
-      }
-      mma_bf16(acc[0][x], wa[0][i], b0, b1);
-      mma_bf16(acc[1][x], wa[1][i], b0, b1);
+    for (int x = 0; x < NT; ++x) {
+      const uint32_t* q = reinterpret_cast<const uint32_t*>(u + (long long)min(r0 + x * 8 + g, p.T - 1) * p.C + blk * n + ks * 16 + 2 * t);
+      b0[x] = __ldcg(q);
+      b1[x] = __ldcg(q + 4);
+    }
+#pragma unroll
+    for (int x = 0; x < NT; ++x) {
+      mma_bf16(acc[0][x], wa[0][i], b0[x], b1[x]);
+      mma_bf16(acc[1][x], wa[1][i], b0[x], b1[x]);
     }
   }
 #pragma unroll
   for (int m = 0; m < 2; ++m)
 #pragma unroll
-    for (int x = 0; x < 2; ++x)
+    for (int x = 0; x < NT; ++x)
 #pragma unroll
       for (int e = 0; e < 4; ++e) s_acc[warp][m][x * 8 + 2 * t + (e & 1)][g + (e >> 1) * 8] = acc[m][x][e];
   __syncthreads();
   bf16* out = reinterpret_cast<bf16*>(p.out);
-  for (int r = threadIdx.x >> 4; r < 16; r += 8) {
-    const int row = r0 + r;
-    if (row >= p.T) break;
-    const Run run = get_run(p.runs, row);
-    if (blockIdx.x == 0 && ch < p.pad_out) out[row * p.ld_out + p.C + ch] = __float2bfloat16(0.f);
-    float zr = br, zi = bi;
 #pragma unroll
-    for (int w = 0; w < 4; ++w) {
-      zr += s_acc[w][0][r][ch];
-      zi += s_acc[w][1][r][ch];
+  for (int i = 0; i < NT; ++i) {
+    const int r = (threadIdx.x >> 4) + i * 8, row = r0 + r;
+    if (row >= p.T) break;
+    if (blockIdx.x == 0 && ch < p.pad_out) out[row * p.ld_out + p.C + ch] = __float2bfloat16(0.f);
+    float zr = br, zi = bi, a, w;
+#pragma unroll
+    for (int v = 0; v < 4; ++v) {
+      zr += s_acc[v][0][r][ch];
+      zi += s_acc[v][1][r][ch];
     }
-    float a, w;
     lru_gates(zr, zi, k, a, w);
-    float S = run.slot >= 0 && run.start > 0 ? __ldcg(p.state + (long long)run.slot * p.C + c) : 0.f;
-    const unsigned short ub = __ldcg(reinterpret_cast<const unsigned short*>(u) + (long long)row * p.C + c);
-    S = fmaf(a, S, w * __bfloat162float(__ushort_as_bfloat16(ub)));
-    if (run.slot >= 0) p.state[(long long)run.slot * p.C + c] = S;
-    out[row * p.ld_out + c] = __float2bfloat16(S * branch_y<bf16>(p, row, c));
+    if (slot[i] < 0 || first[i]) S[i] = 0.f;
+    S[i] = fmaf(a, S[i], w * __uint_as_float(uint32_t(u16[i]) << 16));
+    if (slot[i] >= 0) p.state[(long long)slot[i] * p.C + c] = S[i];
+    out[row * p.ld_out + c] = __float2bfloat16(S[i] * gelu_tanh_t<bf16>(y[i]));
   }
 }
 
@@ -404,7 +491,7 @@ lru_scan_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_consta
     const int c = blk * q.n + (on ? cb + ch : 0);            // lanes past the block repeat its first channel, unwritten
     const uint32_t lane_addr = tmem_base + (uint32_t(group * 32) << 16);
     const float k = lru_rate(p, c), br = p.gate_b[c], bi = p.gate_b[p.C + c];
-    const bf16* yp = reinterpret_cast<const bf16*>(p.y.p) + p.off_y + c;
+    const unsigned short* yp = reinterpret_cast<const unsigned short*>(p.y.p) + p.off_y + c;
     bf16* op = reinterpret_cast<bf16*>(p.out) + c;
     // place of the channel in a u tile: sub-tile, 16-byte chunk (swizzled by the row) and byte inside it
     const int cu = cb + ch < q.subs * 64 ? cb + ch : 0;
@@ -421,15 +508,11 @@ lru_scan_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_consta
     bool ok = true;
     for (int j = 0; j < n_tiles && ok; ++j) {
       const int st = j & 1, t0 = seg0 + j * LT_TOK + half * 32, live = min(32, max(0, seg1 - t0));
-      uint32_t y2[16];                                       // the other branch, requested early, two tokens to a register
+      // the other branch, requested early and used last; rows past the run repeat its last one, so that no load is conditional
+      unsigned short y16[32];
       if (!AGG) {
 #pragma unroll
-        for (int t = 0; t < 32; t += 2) {
-          uint32_t lo = 0u, hi = 0u;
-          if (t < live) lo = *reinterpret_cast<const unsigned short*>(yp + (run.lo + t0 + t) * p.y.ld);
-          if (t + 1 < live) hi = *reinterpret_cast<const unsigned short*>(yp + (run.lo + t0 + t + 1) * p.y.ld);
-          y2[t >> 1] = lo | (hi << 16);
-        }
+        for (int t = 0; t < 32; ++t) y16[t] = __ldcg(yp + (run.lo + min(t0 + t, seg1 - 1)) * p.y.ld);
       }
       // warp-uniform, so that a wait that ran out ends the loop for the whole warp
       ok = __all_sync(0xffffffffu, !*s_abort && mbar_wait(&acc_full[st], uint32_t((j >> 1) & 1), p.status, ST_TIMEOUT_ACC_FULL));
@@ -479,12 +562,9 @@ lru_scan_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_consta
       }
       if (!AGG) {
 #pragma unroll
-        for (int t = 0; t < 32; ++t) {
-          if (t < live && on) {
-            const float y = __uint_as_float((t & 1) ? (y2[t >> 1] & 0xffff0000u) : (y2[t >> 1] << 16));
-            op[(run.lo + t0 + t) * p.ld_out] = __float2bfloat16(__uint_as_float(b[t]) * y);
-          }
-        }
+        for (int t = 0; t < 32; ++t)
+          if (t < live && on)
+            op[(run.lo + t0 + t) * p.ld_out] = __float2bfloat16(__uint_as_float(b[t]) * __uint_as_float(uint32_t(y16[t]) << 16));
         if (blockIdx.x == 0 && ch < p.pad_out)
           for (int t = 0; t < live; ++t) reinterpret_cast<bf16*>(p.out)[(run.lo + t0 + t) * p.ld_out + p.C + ch] = __float2bfloat16(0.f);
       }
@@ -519,8 +599,15 @@ template <typename T>
 static void lru_conv_t(const LruParams& p, cudaStream_t s) {
   const bool vec = p.C % 4 == 0 && p.off_x % 4 == 0 && p.taps <= 4 && (p.x.part != nullptr ? p.x.part_ld % 4 == 0 : p.x.ld % 4 == 0);
   if (vec) {
-    const int rows = p.runs.cu == nullptr ? 1 : LC_ROWS;
-    launch_pdl(PDL_PARTIALS, lru_conv4_kernel<T>, dim3((p.C + 1023) / 1024, (p.T + rows - 1) / rows), dim3(256), 0, s, p, rows);
+    if (p.runs.cu == nullptr) {
+      launch_pdl(PDL_PARTIALS, lru_conv4_step_kernel<T>, dim3((p.C + 1023) / 1024, p.T), dim3(256), 0, s, p);
+      return;
+    }
+    const int rows = p.T >= 2048 ? LC_ROWS : LC_BATCH;
+    const dim3 grid((p.C + 1023) / 1024, (p.T + rows - 1) / rows);
+    auto go = [&](auto kern) { launch_pdl(PDL_PARTIALS, kern, grid, dim3(256), 0, s, p, rows); };
+    if (p.x.part != nullptr) go(lru_conv4_kernel<T, LC_BATCH, true>);
+    else go(lru_conv4_kernel<T, LC_BATCH, false>);
   } else {
     launch_pdl(PDL_PARTIALS, lru_conv_kernel<T>, dim3(p.T, (p.C + 255) / 256), dim3(256), 0, s, p);
   }
@@ -547,7 +634,10 @@ bool lru_tc_supported(const LruParams& p) {
 
 void launch_lru_step(const LruParams& p, cudaStream_t s) {
   if (p.T == 0) return;
-  launch_pdl(PDL_PARTIALS, lru_step_kernel, dim3(p.C / 16, (p.T + 15) / 16), dim3(128), 0, s, p);
+  auto go = [&](auto kern, int nt) { launch_pdl(PDL_PARTIALS, kern, dim3(p.C / 16, (p.T + nt * 8 - 1) / (nt * 8)), dim3(128), 0, s, p); };
+  if (p.T <= 8) go(lru_step_kernel<1>, 1);
+  else if (p.T <= 16) go(lru_step_kernel<2>, 2);
+  else go(lru_step_kernel<4>, 4);
   check_launch("step of the recurrent unit");
 }
 

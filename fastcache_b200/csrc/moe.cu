@@ -193,56 +193,93 @@ __device__ __forceinline__ void write_plan(const RouteScore& p, const int* s_cou
   }
 }
 
-// Few tokens: one CTA chooses, counts and places.
+// Few tokens, scores from h and the router's weights: one CTA per token makes the products (a warp per expert) and chooses.
+constexpr int RF_THREADS = 512;
+template <typename T>
+__global__ void __launch_bounds__(RF_THREADS)
+route_token_kernel(const RouteScore p) {
+  extern __shared__ float s_row[];                           // [K] h, [E] logits, [E + groups]
+  float *s_z = s_row + p.K, *s_choice = s_z + p.E;
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  ProjSrc h;
+  h.p = p.h;
+  h.ld = p.ld_h;
+  for (int c = threadIdx.x * 8; c < p.K; c += RF_THREADS * 8) {
+    float v[8];
+    proj_at8<T>(h, t, c, v);
+    store8(s_row + c, v);
+  }
+  __syncthreads();
+  ProjSrc w;
+  w.p = p.w;
+  w.ld = p.K;
+  for (int e = warp; e < p.E; e += RF_THREADS / 32) {
+    float z = 0.f;
+#pragma unroll 8
+    for (int c = lane * 8; c < p.K; c += 256) {
+      float a[8];
+      proj_at8<T>(w, e, c, a);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) z = fmaf(a[i], s_row[c + i], z);
+    }
+    z = warp_sum(z);
+    if (lane == 0) s_z[e] = z;
+  }
+  __syncthreads();
+  if (warp != 0) return;
+  RouteScore q = p;                                          // this token's logits
+  q.logits = ProjSrc();
+  q.logits.p = s_z;
+  choose_and_weigh(q, t, s_choice, s_choice + p.E, p.ids + (long long)t * p.top);
+}
+// The same from finished logits, `rows` tokens per CTA; with p.counts how often every expert was chosen by the CTA's tokens.
 __global__ void __launch_bounds__(RT_THREADS)
-route_score_small_kernel(const RouteScore p) {
+route_choose_kernel(const RouteScore p, int rows) {
   extern __shared__ float s_scores[];                        // [warps][E + groups]
+  __shared__ int s_count[MOE_MAX_EXPERTS];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int warp = threadIdx.x >> 5, tid = threadIdx.x, t0 = blockIdx.x * rows, t1 = min(p.T, t0 + rows);
+  float* s_choice = s_scores + warp * (p.E + p.groups);
+  for (int e = tid; e < p.E; e += blockDim.x) s_count[e] = 0;
+  for (int t = t0 + warp; t < t1; t += blockDim.x / 32)
+    choose_and_weigh(p, t, s_choice, s_choice + p.E, p.ids + (long long)t * p.top);
+  if (p.counts == nullptr) return;
+  __syncthreads();                                           // also makes ids visible in the CTA
+  for (int i = t0 * p.top + tid; i < t1 * p.top; i += blockDim.x)
+    if (p.ids[i] >= 0) atomicAdd(&s_count[p.ids[i]], 1);
+  __syncthreads();
+  for (int e = tid; e < p.E; e += blockDim.x) p.counts[(long long)blockIdx.x * p.E + e] = s_count[e];
+}
+// Few tokens: one CTA counts and places.
+__global__ void __launch_bounds__(RT_THREADS)
+route_place_small_kernel(const RouteScore p) {
   __shared__ int s_count[MOE_MAX_EXPERTS], s_end[MOE_MAX_EXPERTS], s_tile[MOE_MAX_EXPERTS];
   pdl_launch_dependents();
   pdl_wait();
-  const int warp = threadIdx.x >> 5, tid = threadIdx.x;
-  float* s_choice = s_scores + warp * (p.E + p.groups);
+  const int tid = threadIdx.x, pairs = p.T * p.top;
   for (int e = tid; e < p.E; e += RT_THREADS) s_count[e] = 0;
-  for (int t = warp; t < p.T; t += RT_THREADS / 32) choose_and_weigh(p, t, s_choice, s_choice + p.E, p.ids + t * p.top);
-  __syncthreads();                                           // also makes ids visible in the CTA
-  for (int i = tid; i < p.T * p.top; i += RT_THREADS)
-    if (p.ids[i] >= 0) atomicAdd(&s_count[p.ids[i]], 1);
+  __syncthreads();
+  for (int i = tid; i < pairs; i += RT_THREADS) {
+    const int e = __ldcg(p.ids + i);
+    if (e >= 0) atomicAdd(&s_count[e], 1);
+  }
   __syncthreads();
   write_plan<RT_THREADS>(p, s_count, s_end, s_tile, true);
   __syncthreads();
   for (int e = tid; e < p.E; e += RT_THREADS) s_end[e] -= s_count[e];       // next free row
   __syncthreads();
   int* token = p.plan + p.token_at;
-  for (int i = tid; i < p.T * p.top; i += RT_THREADS) {
-    const int e = p.ids[i];
-    int r = -1;
-    if (e >= 0) {
-      r = atomicAdd(&s_end[e], 1);
-      token[r] = i / p.top;
-    }
+  for (int i = tid; i < pairs; i += RT_THREADS) {
+    const int e = __ldcg(p.ids + i), r = e >= 0 ? atomicAdd(&s_end[e], 1) : -1;
+    if (e >= 0) token[r] = i / p.top;
     p.row_of[i] = r;
   }
 }
-
-// Many tokens: every CTA chooses for ROUTE_ROWS tokens and leaves its counts; then every CTA places its own.
+// Many tokens: every CTA places its ROUTE_ROWS tokens behind those of the CTAs before it.
 constexpr int RS_ROUTE_THREADS = 256;
-__global__ void __launch_bounds__(RS_ROUTE_THREADS)
-route_choose_kernel(const RouteScore p) {
-  extern __shared__ float s_scores[];
-  __shared__ int s_count[MOE_MAX_EXPERTS];
-  pdl_launch_dependents();
-  pdl_wait();
-  const int warp = threadIdx.x >> 5, tid = threadIdx.x, t0 = blockIdx.x * ROUTE_ROWS, t1 = min(p.T, t0 + ROUTE_ROWS);
-  float* s_choice = s_scores + warp * (p.E + p.groups);
-  for (int e = tid; e < p.E; e += RS_ROUTE_THREADS) s_count[e] = 0;
-  for (int t = t0 + warp; t < t1; t += RS_ROUTE_THREADS / 32)
-    choose_and_weigh(p, t, s_choice, s_choice + p.E, p.ids + (long long)t * p.top);
-  __syncthreads();
-  for (int i = t0 * p.top + tid; i < t1 * p.top; i += RS_ROUTE_THREADS)
-    if (p.ids[i] >= 0) atomicAdd(&s_count[p.ids[i]], 1);
-  __syncthreads();
-  for (int e = tid; e < p.E; e += RS_ROUTE_THREADS) p.counts[(long long)blockIdx.x * p.E + e] = s_count[e];
-}
 __global__ void __launch_bounds__(RS_ROUTE_THREADS)
 route_place_kernel(const RouteScore p, int blocks) {
   __shared__ int s_count[MOE_MAX_EXPERTS], s_before[MOE_MAX_EXPERTS], s_end[MOE_MAX_EXPERTS], s_tile[MOE_MAX_EXPERTS];
@@ -277,25 +314,32 @@ route_place_kernel(const RouteScore p, int blocks) {
     p.row_of[i] = r;
   }
 }
-void launch_route_score(const RouteScore& a, cudaStream_t s) {
+void launch_route_score(const RouteScore& a, bool f32, cudaStream_t s) {
   if (a.T == 0) return;
   RouteScore p = a;
   p.token_at = moe_token_offset(p.T * p.top, p.E);
   if (p.E > MOE_MAX_EXPERTS) throw std::runtime_error("experts are limited to 1024");
-  auto smem = [&](auto kern, int warps) {
-    const int bytes = warps * (p.E + p.groups) * 4;
+  auto smem = [&](auto kern, int floats) {
+    const size_t bytes = size_t(floats) * 4;
     if (bytes > 200 * 1024) throw std::runtime_error("routing: too many experts and groups");
-    if (bytes > 32 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes);
-    return size_t(bytes);
+    if (bytes > 32 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, int(bytes));
+    return bytes;
   };
-  const bool small = p.T <= 256 && p.E + p.groups <= 1024;
-  if (small) {
-    const size_t n = smem(route_score_small_kernel, RT_THREADS / 32);
-    launch_pdl(PDL_PARTIALS, route_score_small_kernel, dim3(1), dim3(RT_THREADS), n, s, p);
+  const int each = p.E + p.groups;
+  if (p.h != nullptr) {
+    const int floats = p.K + p.E + each;
+    auto go = [&](auto kern) { launch_pdl(PDL_PARTIALS, kern, dim3(p.T), dim3(RF_THREADS), smem(kern, floats), s, p); };
+    if (f32) go(route_token_kernel<float>);
+    else go(route_token_kernel<__nv_bfloat16>);
+  }
+  if (p.T <= ROUTE_SMALL) {
+    p.counts = nullptr;
+    if (p.h == nullptr)
+      launch_pdl(PDL_PARTIALS, route_choose_kernel, dim3((p.T + 7) / 8), dim3(256), smem(route_choose_kernel, 8 * each), s, p, 8);
+    launch_pdl(PDL_PARTIALS, route_place_small_kernel, dim3(1), dim3(RT_THREADS), 0, s, p);
   } else {
-    const int blocks = route_score_blocks(p.T);
-    const size_t n = smem(route_choose_kernel, RS_ROUTE_THREADS / 32);
-    launch_pdl(PDL_PARTIALS, route_choose_kernel, dim3(blocks), dim3(RS_ROUTE_THREADS), n, s, p);
+    const int blocks = route_score_blocks(p.T), warps = each <= 1024 ? RT_THREADS / 32 : 8;
+    launch_pdl(PDL_PARTIALS, route_choose_kernel, dim3(blocks), dim3(warps * 32), smem(route_choose_kernel, warps * each), s, p, ROUTE_ROWS);
     launch_pdl(PDL_PARTIALS, route_place_kernel, dim3(blocks), dim3(RS_ROUTE_THREADS), 0, s, p, blocks);
   }
   const cudaError_t e = cudaGetLastError();

@@ -114,9 +114,18 @@ std::tuple<Tensor, Tensor, Tensor> route_by_score(const Tensor& h, const Tensor&
     check_i32(*ctx, "context lengths", T);
     r.ctx = ctx->data_ptr<int>();
   }
-  const Projection z = project(h, weight, weight.size(0), 0, weight.size(0), false);
-  TORCH_CHECK(z.cols >= E, "the router needs a row per expert");
-  r.logits = z.wide;
+  check_product(h, weight);
+  TORCH_CHECK(weight.size(0) >= E, "the router needs a row per expert");
+  Projection z;
+  if (T <= fc::ROUTE_SMALL && (int64_t)T * E <= 4096) {     // the weights are read once per token
+    r.h = h.data_ptr();
+    r.ld_h = h.stride(0);
+    r.w = weight.data_ptr();
+    r.K = int(h.size(1));
+  } else {
+    z = project(h, weight, weight.size(0), 0, weight.size(0), false);
+    r.logits = z.wide;
+  }
   r.correction = correction.data_ptr<float>();
   r.T = T;
   r.top = int(top);
@@ -128,7 +137,7 @@ std::tuple<Tensor, Tensor, Tensor> route_by_score(const Tensor& h, const Tensor&
   r.plan = plan.data_ptr<int>();
   r.ids = ids.data_ptr<int>();
   r.counts = counts.data_ptr<int>();
-  fc::launch_route_score(r, stream_now());
+  fc::launch_route_score(r, is_f32(h), stream_now());
   return {row_of, plan, mix};
 }
 

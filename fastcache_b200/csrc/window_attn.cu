@@ -172,6 +172,175 @@ window_store_kernel(const WindowStore p) {
   }
 }
 
+// Many rows of heads that fill the pages' rows (bf16, finished projections).  A thread owns 16-byte pieces of the query and one
+// of the key or the value of several tokens: the next token is requested ahead, the last threads make its angles meanwhile, and
+// halves that turn together are exchanged within the warp.
+constexpr int WR_MAX_HALF = 128;
+__device__ __forceinline__ void unpack8(const uint4& u, float (&v)[8]) {
+  const uint32_t w[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    v[2 * i] = __uint_as_float(w[i] << 16);
+    v[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u);
+  }
+}
+__device__ __forceinline__ void add_bias8(float (&v)[8], const uint4& b) {
+  float f[8];
+  unpack8(b, f);
+#pragma unroll
+  for (int e = 0; e < 8; ++e) v[e] += f[e];
+}
+template <int THREADS, int NQ>
+__global__ void __launch_bounds__(THREADS, NQ == 1 ? 1024 / THREADS : 1)
+window_store_rows_kernel(const WindowStore p, int tokens) {
+  __shared__ float2 red[2][THREADS / 32];
+  __shared__ __align__(16) float2 cs[2][WR_MAX_HALF];
+  const int tid = threadIdx.x, nq = p.H * p.D, nk = p.G * p.D, half = p.rot_dims / 2;
+  const bool is_k = tid < nk / 8, is_v = !is_k && tid < nk / 4;
+  const int at8 = (is_k ? tid : tid - nk / 8) * 8;           // first element of the key or value piece in its row
+  const bf16 *src = reinterpret_cast<const bf16*>(p.proj.p), *bias = reinterpret_cast<const bf16*>(p.bias);
+  const int kv_col = (is_k || p.off_v < 0 ? p.off_k : p.off_v) + at8;
+  const uint4 zero = make_uint4(0, 0, 0, 0);
+  auto piece = [&](const bf16* row, int col) { return __ldcg(reinterpret_cast<const uint4*>(row + col)); };
+  uint4 bq[NQ], bkv = zero;
+#pragma unroll
+  for (int j = 0; j < NQ; ++j) {
+    const int i = (tid + j * THREADS) * 8;
+    bq[j] = bias != nullptr && i < nq ? *reinterpret_cast<const uint4*>(bias + p.off_q + i) : zero;
+  }
+  if ((is_k || is_v) && bias != nullptr) bkv = *reinterpret_cast<const uint4*>(bias + kv_col);
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t0 = blockIdx.x * tokens, t1 = min(p.T, t0 + tokens);
+  if (t0 >= t1) return;
+  uint4 q4[NQ], kv4 = zero;
+#pragma unroll
+  for (int j = 0; j < NQ; ++j) q4[j] = zero;
+  int slot = 0;
+  auto request = [&](int t) {
+    const bf16* row = src + t * p.proj.ld;
+#pragma unroll
+    for (int j = 0; j < NQ; ++j)
+      if ((tid + j * THREADS) * 8 < nq) q4[j] = piece(row, p.off_q + (tid + j * THREADS) * 8);
+    if (is_k || is_v) kv4 = piece(row, kv_col);
+    slot = p.slots[t];
+  };
+  request(t0);
+  const int turn_i = THREADS - 1 - tid;                      // this thread's angle
+  const double freq = turn_i < half ? p.freq[turn_i] : 0.0;
+  auto angles = [&](int t) {
+    if (turn_i >= half) return;
+    float c, s;
+    turn_angle(double(p.positions[t]), freq, c, s);
+    cs[t & 1][turn_i] = make_float2(c * p.rot_size, s * p.rot_size);
+  };
+  angles(t0);
+  // norm weight and rotation of a piece whose first column of the head is c; every lane of the warp takes part
+  auto finish = [&](float (&y)[8], const float* w, float inv, int c, const float2* a, bool on) {
+    if (on) {
+      const float4 w0 = *reinterpret_cast<const float4*>(w), w1 = *reinterpret_cast<const float4*>(w + 4);
+      const float f[8] = {w0.x, w0.y, w0.z, w0.w, w1.x, w1.y, w1.z, w1.w};
+#pragma unroll
+      for (int e = 0; e < 8; ++e) y[e] *= inv * f[e];
+    }
+    if (half == 0) return;
+    if (p.half) {
+      const bool lo = c < half;
+      const float f = lo ? -1.f : 1.f;
+      const float2* g = a + (c < p.rot_dims ? (lo ? c : c - half) : 0);
+#pragma unroll
+      for (int e = 0; e < 8; e += 2) {
+        const float o0 = __shfl_xor_sync(0xffffffffu, y[e], half >> 3), o1 = __shfl_xor_sync(0xffffffffu, y[e + 1], half >> 3);
+        if (c < p.rot_dims) {
+          const float4 gg = *reinterpret_cast<const float4*>(g + e);
+          y[e] = y[e] * gg.x + f * o0 * gg.y;
+          y[e + 1] = y[e + 1] * gg.z + f * o1 * gg.w;
+        }
+      }
+    } else {
+#pragma unroll
+      for (int e = 0; e < 8; e += 2)
+        if (c + e < p.rot_dims) {
+          const float2 g = a[(c + e) >> 1];
+          const float u = y[e], v = y[e + 1];
+          y[e] = u * g.x - v * g.y;
+          y[e + 1] = v * g.x + u * g.y;
+        }
+    }
+  };
+  for (int t = t0; t < t1; ++t) {
+    const int par = t & 1, at = slot;
+    float x[NQ][8], kv[8], sq = 0.f, sk = 0.f;
+#pragma unroll
+    for (int j = 0; j < NQ; ++j) {                           // pieces past the row are zero
+      unpack8(q4[j], x[j]);
+      add_bias8(x[j], bq[j]);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) sq += x[j][e] * x[j][e];
+    }
+    unpack8(kv4, kv);
+    add_bias8(kv, bkv);
+    if (is_k)
+#pragma unroll
+      for (int e = 0; e < 8; ++e) sk += kv[e] * kv[e];
+    if (t + 1 < t1) request(t + 1);
+    sq = warp_sum(sq);
+    sk = warp_sum(sk);
+    if ((tid & 31) == 0) red[par][tid >> 5] = make_float2(sq, sk);
+    __syncthreads();
+    sq = sk = 0.f;
+#pragma unroll
+    for (int i = 0; i < THREADS / 32; ++i) {
+      sq += red[par][i].x;
+      sk += red[par][i].y;
+    }
+    const float iq = rsqrtf(sq / float(nq) + p.eps), ik = rsqrtf(sk / float(nk) + p.eps);
+    const float2* turns = cs[par];
+    if (t + 1 < t1) angles(t + 1);                           // of the buffer that was read before this token's barrier
+    bf16* q = reinterpret_cast<bf16*>(p.q) + (long long)t * nq;
+#pragma unroll
+    for (int j = 0; j < NQ; ++j) {
+      const int i = (tid + j * THREADS) * 8;
+      finish(x[j], p.q_norm + i, iq, i & (p.D - 1), turns, i < nq);
+      if (i < nq) store8(q + i, x[j]);
+    }
+    if (tid < (nk / 8 + 31) / 32 * 32) {                     // whole warps; the value pieces among them stay as they are
+      float y[8];
+#pragma unroll
+      for (int e = 0; e < 8; ++e) y[e] = kv[e];
+      finish(y, p.k_norm + at8, ik, at8 & (p.D - 1), turns, is_k);
+      if (is_k)
+#pragma unroll
+        for (int e = 0; e < 8; ++e) kv[e] = y[e];
+    }
+    if (at < 0 || !(is_k || is_v)) continue;
+    if (at >= p.num_rows) {
+      if (tid == 0) report(p.status, ST_BAD_INDEX);
+      continue;
+    }
+    const int blk = at / p.block_size, off = at - blk * p.block_size;
+    store8(reinterpret_cast<bf16*>(is_k ? p.k_rows : p.v_rows) +
+               (((long long)blk * p.G + at8 / p.D) * p.block_size + off) * p.D + (at8 & (p.D - 1)), kv);
+  }
+}
+static bool window_store_rows_supported(const WindowStore& p) {
+  const int half = p.rot_dims / 2, shift = half / 8;
+  const bool turn = half == 0 || (p.half ? half % 8 == 0 && shift <= 16 && (shift & (shift - 1)) == 0 && p.D % p.rot_dims == 0
+                                         : half <= WR_MAX_HALF);
+  return p.T >= 256 && p.proj.part == nullptr && p.gate == nullptr && (p.D == 64 || p.D == 128) && p.D == p.V && p.D == p.pitch && turn &&
+         p.H * p.D <= 8192 && 2 * p.G * p.D <= (p.H * p.D <= 2048 ? 2048 : 4096) && p.proj.ld % 8 == 0 && p.off_q % 8 == 0 && p.off_k % 8 == 0 &&
+         (p.off_v < 0 || p.off_v % 8 == 0) && p.pad_out == 0;
+}
+static void launch_window_store_rows(const WindowStore& p, cudaStream_t s) {
+  auto go = [&](auto kern, int threads) {                    // two CTAs of 512 threads, four of 256 per SM
+    const int ctas = 148 * 1024 / threads, tokens = std::max(4, (p.T + ctas - 1) / ctas);
+    launch_pdl(PDL_ROPE, kern, dim3((p.T + tokens - 1) / tokens), dim3(threads), 0, s, p, tokens);
+  };
+  if (p.H * p.D <= 2048) go(window_store_rows_kernel<256, 1>, 256);
+  else if (p.H * p.D <= 4096) go(window_store_rows_kernel<512, 1>, 512);
+  else go(window_store_rows_kernel<512, 2>, 512);
+}
+
 // General form: one warp per (row, head).  A lane scores one of 32 keys, then the lanes share the value columns.
 constexpr int WA_WARPS = 4;
 template <typename T, int NACC>
@@ -265,6 +434,7 @@ static void window_store_t(const WindowStore& p, cudaStream_t s) {
 void launch_window_store(const WindowStore& p, bool f32, cudaStream_t s) {
   if (p.T == 0) return;
   if (f32) window_store_t<float>(p, s);
+  else if (window_store_rows_supported(p)) launch_window_store_rows(p, s);
   else window_store_t<bf16>(p, s);
   check_launch("norm, rotation and store of windowed attention");
 }
