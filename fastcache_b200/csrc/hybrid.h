@@ -1,7 +1,7 @@
-// Launchers of the hybrid-model kernels: norms on an fp32 residual stream and gated activations (resid.cu), recurrent
-// layers (recurrence.cu, recurrence_chunk.cu, lru.cu), residual streams (streams.cu), latent attention (latent.cu, latent_decode.cu, latent_prefill.cu),
-// windowed attention (window_attn.cu, with the attn_*.cu kernels), experts (moe.cu, moe_gemm.cu) and the CUDA-core GEMM of
-// 32-bit runs (linear_simt.cu).
+// Launchers of the hybrid-model kernels: norms on an fp32 residual stream and gated activations (resid.cu), several residual
+// streams (streams.cu), recurrent layers (recurrence.cu, recurrence_chunk.cu, lru.cu), latent attention (latent.cu,
+// latent_decode.cu, latent_prefill.cu), attention over per-head rows (window_attn.cu, with the attn_*.cu kernels), experts
+// (moe.cu, moe_gemm.cu) and the CUDA-core GEMM of 32-bit runs (linear_simt.cu).
 //
 // `f32` selects the element type of activations and weights (fp32 or bf16); everything accumulates in fp32.
 #pragma once

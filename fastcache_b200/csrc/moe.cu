@@ -73,8 +73,8 @@ void launch_route_table(const RouteTable& a, cudaStream_t s) {
 }
 
 // ---- choice by score
-// One warp per token.  s_choice [E]: choice scores, -inf outside the best groups; `put(j, expert, score)` receives the j-th
-// chosen expert on every lane.  Ties go to the lower index.
+// One warp per token.  s_choice [E]: choice scores, -inf outside the best groups; `put(j, expert)` receives the j-th chosen
+// expert on every lane.  Ties go to the lower index.
 struct Best {
   float v;
   int i;
@@ -120,13 +120,13 @@ __device__ __forceinline__ void choose_experts(const RouteScore& p, long long t,
       if (s_choice[e] > b.v) b = {s_choice[e], e};
     b = warp_best(b);
     const int e = min(b.i, p.E - 1);                         // scores that are not numbers choose the last expert
-    put(j, e, b.v - p.correction[e]);
+    put(j, e);
     __syncwarp();
     if (lane == 0) s_choice[e] = -INFINITY;
     __syncwarp();
   }
 }
-// choice and weights of token t: ids and mix (lane j holds the j-th, `top` <= 32 at a time)
+// choice and weights of token t: its rows of ids and mix
 __device__ __forceinline__ void choose_and_weigh(const RouteScore& p, long long t, float* s_choice, float* s_group, int* ids) {
   const int lane = threadIdx.x & 31;
   if (p.ctx != nullptr && p.ctx[t] <= 0) {                   // a padding row has no experts
@@ -135,7 +135,7 @@ __device__ __forceinline__ void choose_and_weigh(const RouteScore& p, long long 
   }
   float total = 0.f;
   float* mix = p.mix + t * p.top;
-  choose_experts(p, t, s_choice, s_group, [&](int j, int e, float) {
+  choose_experts(p, t, s_choice, s_group, [&](int j, int e) {
     const float s = sigmoid_f(proj_at<float>(p.logits, t, e));       // without the rounding of adding the correction
     total += s;
     if (lane == 0) {

@@ -227,12 +227,14 @@ window_store_rows_kernel(const WindowStore p, int tokens) {
   };
   request(t0);
   const int turn_i = THREADS - 1 - tid;                      // this thread's angle
+  // halves that turn together read 16 bytes per pair of angles: the same pair of neighbouring pieces lies side by side
+  const int turn_at = p.half ? (((turn_i & 7) >> 1) * (half >> 3) + (turn_i >> 3)) * 2 + (turn_i & 1) : turn_i;
   const double freq = turn_i < half ? p.freq[turn_i] : 0.0;
   auto angles = [&](int t) {
     if (turn_i >= half) return;
     float c, s;
     turn_angle(double(p.positions[t]), freq, c, s);
-    cs[t & 1][turn_i] = make_float2(c * p.rot_size, s * p.rot_size);
+    cs[t & 1][turn_at] = make_float2(c * p.rot_size, s * p.rot_size);
   };
   angles(t0);
   // norm weight and rotation of a piece whose first column of the head is c; every lane of the warp takes part
@@ -247,12 +249,12 @@ window_store_rows_kernel(const WindowStore p, int tokens) {
     if (p.half) {
       const bool lo = c < half;
       const float f = lo ? -1.f : 1.f;
-      const float2* g = a + (c < p.rot_dims ? (lo ? c : c - half) : 0);
+      const float4* g = reinterpret_cast<const float4*>(a) + ((c < p.rot_dims ? (lo ? c : c - half) : 0) >> 3);
 #pragma unroll
       for (int e = 0; e < 8; e += 2) {
         const float o0 = __shfl_xor_sync(0xffffffffu, y[e], half >> 3), o1 = __shfl_xor_sync(0xffffffffu, y[e + 1], half >> 3);
         if (c < p.rot_dims) {
-          const float4 gg = *reinterpret_cast<const float4*>(g + e);
+          const float4 gg = g[(e >> 1) * (half >> 3)];
           y[e] = y[e] * gg.x + f * o0 * gg.y;
           y[e + 1] = y[e + 1] * gg.z + f * o1 * gg.w;
         }
