@@ -131,6 +131,17 @@ __device__ __forceinline__ float glu_t(float g, float u, float limit) {
   return over_one_plus_exp<T>(g, -1.702f * g) * (u + 1.f);
 }
 
+// xIELU: z > 0: a z^2 + z / 2, else b (e^z - 1 - z) + z / 2.  e^z - 1 - z cancels near 0: its series there
+template <typename T>
+__device__ __forceinline__ float xielu_t(float z, float a, float b) {
+  const float n = fminf(z, 0.f);
+  float e;
+  if constexpr (sizeof(T) == 2) e = __expf(n) - 1.f - n;
+  else e = expm1f(n) - n;
+  if (n > -0.25f) e = n * n * (0.5f + n * (0.16666667f + n * (0.041666667f + n * (0.0083333333f + n * 0.0013888889f))));
+  return (z > 0.f ? a * z * z : b * e) + 0.5f * z;
+}
+
 // cos and sin of `position` times a frequency in turns, reduced in double
 __device__ __forceinline__ void turn_angle(double pos, double freq, float& c, float& s) {
   const double turns = pos * freq;

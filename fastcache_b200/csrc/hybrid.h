@@ -52,8 +52,23 @@ void launch_head_linear_mma(const SimtLinear& a, cudaStream_t s);
 // ---- resid.cu
 void launch_embed_scaled(const void* ids, const void* weight, float* x, void* h, int T, int W, int Wp, long long V,
                          float scale, bool f32, uint32_t* status, cudaStream_t s);
-void launch_post_norm_add(const ProjSrc& y, const void* bias, float* x, const float* w, void* h, int T, int W, int Wp,
-                          float eps, bool f32, cudaStream_t s);
+// x += rms(f * (y + bias) + sum_j mix_j experts[row_of_j]) * w in fp32; h = x in the model's type
+struct PostNormAdd {
+  int T = 0, W = 0, Wp = 0;
+  bool has_y = true;
+  ProjSrc y;
+  const float* y_factor = nullptr;   // f [T]; nullptr: 1
+  const void* bias = nullptr;        // [W]; nullptr: none
+  float* x = nullptr;                // [T, W]
+  const float* w = nullptr;
+  void* h = nullptr;                 // [T, Wp], columns [W, Wp) are zeroed
+  float eps = 0.f;
+  ProjSrc experts;                   // as in AddNorm
+  const int* row_of = nullptr;
+  const float* mix = nullptr;
+  int top = 0;
+};
+void launch_post_norm_add(const PostNormAdd& p, bool f32, cudaStream_t s);
 void launch_rms_norm_wide(const float* x, const float* w, void* h, int T, int W, int Wp, float eps, bool f32,
                           cudaStream_t s);
 // x (+)= y + sum_j mix_j experts[row_of_j] in fp32; h = rms(x) * w, or x itself without w
@@ -84,6 +99,8 @@ struct GluMul {
   long long ld_out = 0;
 };
 void launch_glu_mul(const GluMul& p, bool f32, cudaStream_t s);
+// xIELU of columns [0, width): c = [a, b] on the device, z > 0: a z^2 + z / 2, else b (e^z - 1 - z) + z / 2
+void launch_xielu(const ProjSrc& z, const float* c, void* out, int T, int width, int width_p, bool f32, cudaStream_t s);
 void launch_gelu_mul(const ProjSrc& gu, const void* bias, void* out, int T, int up_off, int width, int width_p,
                      bool f32, cudaStream_t s);
 
@@ -220,10 +237,11 @@ void launch_lru_scan_tc(const LruParams& p, int segments, cudaStream_t s); // ru
 struct LatentStore {
   int T = 0, H = 0, D = 0, R = 0, rank = 0, rot_dims = 0, V = 0;
   ProjSrc proj;
-  int off_q = 0, off_kv = -1, off_g = 0;       // off_kv < 0: the layer reads another layer's rows
+  int off_q = 0, off_kv = -1, off_g = 0;       // off_kv < 0: no cache rows to write
   const float* norm_w = nullptr;
   float eps = 0.f;
   double log2_base = 0.0;            // rotation: position * base^(-2 i / rot_dims)
+  bool half = true;                  // entry i turns with i + rot_dims / 2 (else 2i with 2i + 1)
   const long long* positions = nullptr;
   const int* slots = nullptr;
   void* pool = nullptr;
@@ -232,52 +250,70 @@ struct LatentStore {
   void* q = nullptr;                 // [T, H, D + R], or with `q_abs`: [T, H, D] (unrotated part only)
   void* q_abs = nullptr;             // [T, H, rank + R]: the rotated part goes behind the first `rank` columns
   void* gate = nullptr;              // [T, H * V] copy of the gate projection (nullptr: not wanted)
+  // queries from a latent of their own (launch_latent_inputs)
+  int off_dq = 0, q_rank = 0, ld_cq = 0;
+  const float* q_norm_w = nullptr;
+  void* cq = nullptr;                // [T, ld_cq] normed query latent, zero-padded
+  float* head_gate = nullptr;        // [T, H] sigmoid of the columns off_g + head (nullptr: no such gate)
   uint32_t* status = nullptr;
 };
 void launch_latent_store(const LatentStore& p, bool f32, cudaStream_t s);   // q == nullptr: queries stay in `proj`
+// cq, the cache row and head_gate from the projections (the queries are a product of cq)
+void launch_latent_inputs(const LatentStore& p, bool f32, cudaStream_t s);
 bool latent_rotate_supported(const LatentStore& p);
 
-struct LatentAttn {
-  int T = 0, H = 0, rank = 0, R = 0, row_width = 0, block_size = 0, max_blocks = 0, num_blocks = 0;
-  const void* q_abs = nullptr;       // [T, H, rank + R]
+// Attention over cache rows that all heads share: a query scores against the first K columns of a row; the values of head h
+// are its V columns from v_col + h / (H / v_heads) * V on.  Latent rows: v_col = 0, one value head.
+struct RowAttn {
+  int T = 0, H = 0, K = 0, V = 0, v_col = 0, v_heads = 1;
+  int row_width = 0, block_size = 0, max_blocks = 0, num_blocks = 0;
+  int window = 0;                    // rows a query sees, its own included (0: all up to its own)
+  const void* q = nullptr;           // [T, H, K]
   const void* pool = nullptr;
   const int* block_tables = nullptr;
   const int* row_seq = nullptr;      // request of every row (nullptr: row b belongs to request b)
   const int* row_ctx = nullptr;      // visible rows of every query row
-  void* o_lat = nullptr;             // [T, H, rank]
+  const float* sink = nullptr;       // [H] joins the softmax without a key (nullptr: none)
+  const float* head_gate = nullptr;  // [T, H] factor of the output (nullptr: none)
+  void* out = nullptr;               // [T, ld_out], V columns per head
+  long long ld_out = 0;
   float scale = 1.f;
   uint32_t* status = nullptr;
   // split context (latent_decode.cu)
   int splits = 1;
   float *part_o = nullptr, *part_lse = nullptr;
 };
-void launch_latent_attn_simt(const LatentAttn& p, bool f32, cudaStream_t s);
-bool latent_decode_supported(const LatentAttn& p);
-int latent_decode_splits(const LatentAttn& p, int max_ctx, int num_sms);
-void launch_latent_decode(const LatentAttn& p, cudaStream_t s);
+void launch_row_attn_simt(const RowAttn& p, bool f32, cudaStream_t s);
+bool latent_decode_supported(const RowAttn& p);
+int latent_decode_splits(const RowAttn& p, int max_ctx, int num_sms);
+void launch_latent_decode(const RowAttn& p, cudaStream_t s);
 // the same on tcgen05 (latent_decode_tc.cu); both leave partials for launch_latent_merge when splits > 1
-bool latent_decode_tc_supported(const LatentAttn& p);
-int latent_decode_tc_splits(const LatentAttn& p, int max_ctx, int num_sms);
-void launch_latent_decode_tc(const LatentAttn& p, cudaStream_t s);
-void launch_latent_merge(const LatentAttn& p, cudaStream_t s);
+bool latent_decode_tc_supported(const RowAttn& p);
+int latent_decode_tc_splits(const RowAttn& p, int max_ctx, int num_sms);
+void launch_latent_decode_tc(const RowAttn& p, cudaStream_t s);
+void launch_latent_merge(const RowAttn& p, cudaStream_t s);
 
 void launch_gather_rows(const void* pool, const int* block_tables, const int* ctx, const int* cu_kv, void* out,
                         int B, int max_ctx, int row_width, int block_size, int max_blocks, int num_blocks, bool f32,
                         uint32_t* status, cudaStream_t s);
-// expanded causal attention on tcgen05 (latent_prefill.cu)
+// causal attention of many rows on tcgen05 (latent_prefill.cu): keys = D columns per head and R columns that all heads share
 struct LatentPrefill {
-  int T = 0, B = 0, H = 0, D = 0, R = 0, V = 0, rank = 0, max_q = 0;
+  int T = 0, B = 0, H = 0, D = 0, R = 0, V = 0, v_heads = 0, max_q = 0;   // v_heads: value heads (0: H)
   long long total_kv = 0;
+  int window = 0;                    // as in RowAttn
   const void* q = nullptr;           // [T, ld_q]: D + R columns per head
   long long ld_q = 0;
-  const void* k = nullptr;           // [total_kv, ld_kv]: keys, head by head
-  const void* v = nullptr;           // values, head by head, same pitch
-  long long ld_kv = 0;
-  const void* rot = nullptr;         // rotated key part of the gathered rows
+  const void* k = nullptr;           // [total_kv, ld_k]: keys, head by head (D == 0: none)
+  long long ld_k = 0;
+  const void* v = nullptr;           // [total_kv, ld_v]: values, value head by value head
+  long long ld_v = 0;
+  const void* rot = nullptr;         // [total_kv, ld_rot] the shared columns
   long long ld_rot = 0;
   const int *cu_q = nullptr, *cu_kv = nullptr;
-  const void* gate = nullptr;        // first gate column of the packed projections
+  const float* sink = nullptr;       // as in RowAttn
+  const void* gate = nullptr;        // [T, ld_gate] sigmoid(gate) multiplies the output, column by column (nullptr: none)
   long long ld_gate = 0;
+  const float* head_gate = nullptr;  // as in RowAttn
   void* out = nullptr;
   long long ld_out = 0;
   float scale = 1.f;
@@ -285,6 +321,29 @@ struct LatentPrefill {
 };
 bool latent_prefill_supported(const LatentPrefill& p);
 void launch_latent_prefill(const LatentPrefill& p, cudaStream_t s);
+
+// ---- talking.cu: queries and cache rows of attention whose heads mix their scores before the softmax
+// q [T, H, G * D]: the sum over the heads g of key head u of talk[h, g] * query of g, for every u; a query of this width
+// scores against a whole cache row, keys of all G heads side by side, so that mixed scores are ordinary ones
+struct TalkStore {
+  int T = 0, H = 0, G = 0, D = 0, V = 0, rot_dims = 0;
+  ProjSrc proj;
+  int off_q = 0, off_k = -1, off_v = -1;       // off_k < 0: the layer reads another layer's rows
+  const float* talk = nullptr;       // [H, H]
+  float eps = 0.f;
+  const double* freq = nullptr;      // [rot_dims / 2] turns per position; entry i turns with i + rot_dims / 2
+  const long long* positions = nullptr;
+  const int* slots = nullptr;
+  void* pool = nullptr;              // rows [keys G * D | zeros to v_col | values G * V]
+  int row_width = 0, v_col = 0;
+  long long num_rows = 0;
+  void* q = nullptr;                 // [T, H, G * D]
+  void* out = nullptr;               // attention output: columns [H * V, + pad_out) are zeroed
+  long long ld_out = 0;
+  int pad_out = 0;
+  uint32_t* status = nullptr;
+};
+void launch_talk_store(const TalkStore& p, bool f32, cudaStream_t s);
 
 // ---- window_attn.cu: what surrounds attention over per-head K/V rows
 struct WindowStore {
@@ -344,7 +403,7 @@ struct RouteTable {
   uint32_t* status = nullptr;
 };
 void launch_route_table(const RouteTable& p, cudaStream_t s);
-// choice by score: see route_by_score in ops/hybrid.py
+// choice by score: see route_by_score and route_by_logit in ops/hybrid.py
 struct RouteScore {
   ProjSrc logits;                    // fp32 [T, E], first column 0; or `h` and the router's weights (up to ROUTE_SMALL tokens)
   const void *h = nullptr, *w = nullptr;      // [T, ld_h], [E, K]; K a multiple of 8
@@ -353,6 +412,8 @@ struct RouteScore {
   const float* correction = nullptr; // [E]
   const int* ctx = nullptr;          // as in RouteTable
   int T = 0, top = 0, E = 0, groups = 1, keep = 1;
+  bool softmax = false;              // choice by logit + correction, weights: their softmax over the chosen experts
+  float* extra = nullptr;            // [T] sigmoid of the logit behind the experts' (nullptr: none)
   float* mix = nullptr;              // [T, top] weights
   int* row_of = nullptr;
   int* plan = nullptr;

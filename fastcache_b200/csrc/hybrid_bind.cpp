@@ -8,13 +8,14 @@
 #include <tuple>
 #include <vector>
 
-#include "hybrid_bind.h"
+#include "projection.h"
+#include "row_attention.h"
 
 namespace {
 
 // x @ w.T.  `partial`: decode-size bf16 products may stay split-K partial sums in the stream's scratch, valid until
 // the next product on this stream.  `hold` keeps the finished output alive.  An empty w: x is the projection output.
-fc::ProjSrc project(const Tensor& x, const Tensor& w, const OptTensor& bias, bool partial, Tensor& hold) {
+fc::ProjSrc product(const Tensor& x, const Tensor& w, const OptTensor& bias, bool partial, Tensor& hold) {
   check_elem(x, "x");
   if (w.numel() == 0) {
     TORCH_CHECK(x.dim() == 2 && x.stride(1) == 1 && x.stride(0) % 8 == 0, "bad projection output");
@@ -78,7 +79,7 @@ fc::ProjSrc project(const Tensor& x, const Tensor& w, const OptTensor& bias, boo
 Tensor linear_wide(const Tensor& x, const Tensor& w, const OptTensor& bias) {
   c10::cuda::CUDAGuard guard(x.device());
   Tensor y;
-  project(x, w, bias, false, y);
+  product(x, w, bias, false, y);
   return y;
 }
 
@@ -94,25 +95,61 @@ std::tuple<Tensor, Tensor> embed_scaled(const Tensor& ids, const Tensor& weight,
   return {x, h};
 }
 
-// x += rms(a @ w.T + bias) * norm_w; returns x in the element type of a, padded to the width of w's output
-Tensor linear_post_norm_add(const Tensor& a, const Tensor& w, const OptTensor& bias, Tensor x, const Tensor& norm_w,
-                            double eps) {
+// x += rms(f * (a @ w.T + bias) + mixed expert rows) * norm_w; returns x in the element type of a, padded to the width of w's
+// output
+Tensor linear_post_norm_add(const Tensor& a, const Tensor& w, const OptTensor& bias, Tensor x, const Tensor& norm_w, double eps,
+                            const Projection* experts, const OptTensor& row_of, const OptTensor& mix, const OptTensor& factor) {
   c10::cuda::CUDAGuard guard(a.device());
   const int64_t T = a.size(0), W = x.size(1), Wp = w.numel() ? w.size(0) : a.size(1);
   check_f32(x, "residual", T * W);
   check_f32(norm_w, "norm weight", W);
   TORCH_CHECK(Wp >= W, "projection narrower than the residual");
+  const bool f32 = is_f32(a);
+  fc::PostNormAdd n;
   Tensor hold;
-  const void* bp = nullptr;
   if (bias.has_value() && bias->defined()) {
     TORCH_CHECK(bias->scalar_type() == a.scalar_type() && bias->is_contiguous() && bias->numel() == Wp, "bad bias");
-    bp = bias->data_ptr();
+    n.bias = bias->data_ptr();
   }
-  const fc::ProjSrc src = project(a, w, c10::nullopt, true, hold);
+  n.y = product(a, w, c10::nullopt, true, hold);
+  if (factor.has_value()) {
+    check_f32(*factor, "factor", T);
+    n.y_factor = factor->data_ptr<float>();
+  }
+  if (experts != nullptr) {
+    TORCH_CHECK(row_of.has_value() && row_of->dim() == 2 && row_of->size(0) == T && experts->cols == Wp && experts->f32 == f32,
+                "bad expert outputs");
+    check_i32(*row_of, "row_of", T);
+    n.experts = experts->src;
+    n.row_of = row_of->data_ptr<int>();
+    n.top = int(row_of->size(1));
+    if (mix.has_value()) {
+      check_f32(*mix, "expert weights", row_of->numel());
+      n.mix = mix->data_ptr<float>();
+    }
+  }
   Tensor h = torch::empty({T, Wp}, a.options());
-  fc::launch_post_norm_add(src, bp, x.data_ptr<float>(), norm_w.data_ptr<float>(), h.data_ptr(), int(T), int(W), int(Wp),
-                           float(eps), is_f32(a), stream_now());
+  n.T = int(T);
+  n.W = int(W);
+  n.Wp = int(Wp);
+  n.x = x.data_ptr<float>();
+  n.w = norm_w.data_ptr<float>();
+  n.h = h.data_ptr();
+  n.eps = float(eps);
+  fc::launch_post_norm_add(n, f32, stream_now());
   return h;
+}
+
+// xIELU of h @ w.T; coef: [2] fp32 on the device
+Tensor linear_xielu(const Tensor& h, const Tensor& w, const Tensor& coef, int64_t width) {
+  c10::cuda::CUDAGuard guard(h.device());
+  const int64_t T = h.size(0), wp = pad8(int(width)), N = w.numel() ? w.size(0) : h.size(1);
+  check_f32(coef, "xIELU coefficients", 2);
+  TORCH_CHECK(N == wp, "bad width");
+  Tensor hold, out = torch::empty({T, wp}, h.options());
+  const fc::ProjSrc z = product(h, w, c10::nullopt, true, hold);
+  fc::launch_xielu(z, coef.data_ptr<float>(), out.data_ptr(), int(T), int(width), int(wp), is_f32(h), stream_now());
+  return out;
 }
 
 Tensor rms_norm_wide(const Tensor& x, const Tensor& norm_w, double eps, int64_t Wp, bool f32) {
@@ -152,7 +189,7 @@ Tensor linear_gelu_mul(const Tensor& h, const Tensor& w, const OptTensor& bias, 
                   wp, fc::ACT_GEGLU_TANH, gw, fc::stream_sm_limit(stream_now()), stream_now());
     return out;
   }
-  const fc::ProjSrc src = project(h, w, c10::nullopt, true, hold);
+  const fc::ProjSrc src = product(h, w, c10::nullopt, true, hold);
   fc::launch_gelu_mul(src, bp, out.data_ptr(), int(T), int(up_off), int(width), int(wp), is_f32(h), stream_now());
   return out;
 }
@@ -217,13 +254,13 @@ Tensor gla(const Tensor& h, const Tensor& w, const Tensor& w_a2, const Tensor& z
   const bool chunk = !is_f32(h) && max_len >= CHUNK_MIN_ROWS && fc::chunk_supported(D, V);
   Tensor hold, z, out, o_raw;
   const bool decode = p.runs.cu == nullptr;
-  p.proj = project(h, w, c10::nullopt, decode, hold);
+  p.proj = product(h, w, c10::nullopt, decode, hold);
   if (decode) {
     p.w_a2 = w_a2.data_ptr();
     p.ld_a2 = w_a2.size(1);
     p.rank = rank;
   } else {
-    project(hold.narrow(1, d[8], w_a2.size(1)), w_a2, c10::nullopt, false, z);
+    product(hold.narrow(1, d[8], w_a2.size(1)), w_a2, c10::nullopt, false, z);
     p.z = z.data_ptr();
     p.ld_z = z.size(1);
   }
@@ -265,7 +302,7 @@ Tensor delta_rule(const Tensor& h, const Tensor& w, const Tensor& conv_w, const 
   } else {
     TORCH_CHECK(p.runs.B == T, "one row per request expected");
   }
-  p.proj = project(h, w, c10::nullopt, true, hold);
+  p.proj = product(h, w, c10::nullopt, true, hold);
   q.H = H;
   q.K = K;
   q.D = D;
@@ -300,54 +337,35 @@ Tensor delta_rule(const Tensor& h, const Tensor& w, const Tensor& conv_w, const 
   return out;
 }
 
-// absorbed attention: the tensor-core form where it takes the sizes; `po` / `pl` keep its scratch alive
-void absorbed(fc::LatentAttn& at, bool f32, int64_t impl, int64_t max_ctx, const Tensor& like, Tensor& po, Tensor& pl) {
-  const bool tc = !f32 && impl != 1 && impl != 3 && fc::latent_decode_tc_supported(at);
-  if (!tc && (f32 || impl == 1 || !fc::latent_decode_supported(at))) {
-    fc::launch_latent_attn_simt(at, f32, stream_now());
-    return;
-  }
-  at.splits = tc ? fc::latent_decode_tc_splits(at, int(max_ctx), fc::gemm_num_sms())
-                 : fc::latent_decode_splits(at, int(max_ctx), fc::gemm_num_sms());
-  if (at.splits > 1) {
-    const auto opt = like.options().dtype(torch::kFloat32);
-    po = torch::empty({(int64_t)at.T * at.H * at.splits * at.rank}, opt);
-    pl = torch::empty({(int64_t)at.T * at.H * at.splits}, opt);
-    at.part_o = po.data_ptr<float>();
-    at.part_lse = pl.data_ptr<float>();
-  }
-  if (tc) fc::launch_latent_decode_tc(at, stream_now());
-  else fc::launch_latent_decode(at, stream_now());
-  if (at.splits > 1) fc::launch_latent_merge(at, stream_now());
-}
-
 // Projection, cache store and attention of a latent-attention layer (up to the output projection).
-// d: heads, dim, rot, vdim, rank, rot_dims, offsets of q, kv (-1: none), g.  impl: 0 choose, 1 the forms without tensor
-// cores, 2 absorbed also in prefill, 3 the same
-// on mma.sync
+// d: heads, dim, rot, vdim, rank, rot_dims, offsets of q, kv (-1: none), g (-1: none), then the latent of the queries (its
+// offset, its size; 0: none, q is a projection), window (0: none), whether halves turn together, whether the gate has one
+// column per head.  With a latent, `q_norm` and `w_uq` make the queries from it (q's offset is unused).  impl: 0 choose, 1 the
+// forms without tensor cores, 2 absorbed also in prefill, 3 the same on mma.sync.  cu_kv, max_kv, total_kv: the rows that
+// prefill gathers (the last ones of every request, as many as the window needs)
 Tensor latent_attention(const Tensor& h, const Tensor& w, const std::vector<int64_t>& d, double scale, double base,
                         const OptTensor& kv_norm, double eps, const Tensor& w_kv, int64_t off_uv, const Tensor& w_ukt,
                         const Tensor& w_uv, Tensor pool, const Tensor& positions, const OptTensor& slots,
                         const Tensor& block_tables, const Tensor& ctx, const OptTensor& cu_q, const OptTensor& cu_kv,
-                        const OptTensor& row_seq, const OptTensor& row_ctx, int64_t max_q, int64_t max_ctx,
-                        int64_t total_kv, int64_t impl) {
-  TORCH_CHECK(d.size() == 9, "latent attention: nine sizes and offsets");
+                        const OptTensor& row_seq, const OptTensor& row_ctx, int64_t max_q, int64_t max_ctx, int64_t max_kv,
+                        int64_t total_kv, const OptTensor& q_norm, const OptTensor& w_uq, const OptTensor& sink, int64_t impl) {
+  TORCH_CHECK(d.size() == 14, "latent attention: fourteen sizes and offsets");
   const int H = int(d[0]), D = int(d[1]), R = int(d[2]), V = int(d[3]), rank = int(d[4]), rot_dims = int(d[5]);
+  const int off_g = int(d[8]), q_rank = int(d[10]), window = int(d[11]);
+  const bool by_latent = q_rank > 0, head_gate = off_g >= 0 && d[13] != 0;
   c10::cuda::CUDAGuard guard(h.device());
   const int T = int(h.size(0)), B = int(ctx.numel());
   const bool f32 = is_f32(h);
-  check_elem(pool, "cache rows");
-  TORCH_CHECK(pool.scalar_type() == h.scalar_type() && pool.is_contiguous() && pool.dim() == 3 &&
-                  pool.size(2) >= rank + R && pool.size(2) % 8 == 0, "cache rows must be [blocks, block, row width]");
-  TORCH_CHECK(positions.is_cuda() && positions.scalar_type() == torch::kInt64 && positions.is_contiguous() &&
-                  positions.numel() == T, "positions must be int64 [T]");
+  check_pool(pool, rank + R, f32);
+  check_positions(positions, T);
   check_i32(ctx, "context lengths", B);
-  TORCH_CHECK(block_tables.is_cuda() && block_tables.scalar_type() == torch::kInt32 && block_tables.dim() == 2 &&
-                  block_tables.is_contiguous() && block_tables.size(0) >= B, "block_tables must be int32 [B, blocks]");
+  check_block_tables(block_tables, B);
   TORCH_CHECK(w_ukt.is_contiguous() && w_ukt.numel() == (int64_t)H * rank * D && w_uv.is_contiguous() &&
                   w_uv.numel() == (int64_t)H * V * rank && w_ukt.scalar_type() == h.scalar_type() &&
                   w_uv.scalar_type() == h.scalar_type(), "bad expansion weights");
   TORCH_CHECK(rot_dims % 2 == 0 && rot_dims <= R, "rotated dimensions must be even and inside the rotated part");
+  TORCH_CHECK(window >= 0, "bad window");
+  if (sink.has_value()) check_f32(*sink, "sink", H);
   const auto& ws = ws_of(h);
   fc::LatentStore st;
   st.T = T;
@@ -357,9 +375,10 @@ Tensor latent_attention(const Tensor& h, const Tensor& w, const std::vector<int6
   st.V = V;
   st.rank = rank;
   st.rot_dims = rot_dims;
+  st.half = d[12] != 0;
   st.off_q = int(d[6]);
   st.off_kv = int(d[7]);
-  st.off_g = int(d[8]);
+  st.off_g = std::max(off_g, 0);
   st.eps = float(eps);
   st.log2_base = std::log2(base);
   st.positions = reinterpret_cast<const long long*>(positions.data_ptr<int64_t>());
@@ -374,11 +393,33 @@ Tensor latent_attention(const Tensor& h, const Tensor& w, const std::vector<int6
     st.norm_w = kv_norm->data_ptr<float>();
     st.slots = slots->data_ptr<int>();
   }
+  TORCH_CHECK(off_g < 0 || head_gate == by_latent, "a gate per head goes with queries from a latent, a gate per column without");
   const bool prefill = cu_q.has_value() && cu_q->defined();
   Tensor out = torch::empty({T, pad8(H * V)}, h.options());
   if (T == 0) return out;
-  Tensor hold;
-  st.proj = project(h, w, c10::nullopt, true, hold);
+  Tensor hold, cq, hold_q, gates;
+  st.proj = product(h, w, c10::nullopt, true, hold);
+  if (by_latent) {
+    TORCH_CHECK(q_norm.has_value() && w_uq.has_value() && w_uq->dim() == 2 && w_uq->size(1) == pad8(q_rank) &&
+                    w_uq->size(0) >= H * (D + R), "queries from a latent need its norm and their projection");
+    check_f32(*q_norm, "query latent norm", q_rank);
+    cq = torch::empty({T, pad8(q_rank)}, h.options());
+    st.off_dq = int(d[9]);
+    st.q_rank = q_rank;
+    st.ld_cq = pad8(q_rank);
+    st.q_norm_w = q_norm->data_ptr<float>();
+    st.cq = cq.data_ptr();
+    if (head_gate) {
+      gates = torch::empty({T, H}, h.options().dtype(torch::kFloat32));
+      st.head_gate = gates.data_ptr<float>();
+    }
+    fc::launch_latent_inputs(st, f32, stream_now());
+    st.proj = product(cq, *w_uq, c10::nullopt, true, hold_q);
+    st.off_q = 0;
+    st.off_kv = -1;                                         // the cache row is written
+  }
+  const bool column_gate = off_g >= 0 && !head_gate;
+  const float* sinks = sink.has_value() ? sink->data_ptr<float>() : nullptr;
 
   if (prefill && !f32 && impl == 0) {
     // expanded form: the cache rows of every request become per-head keys and values
@@ -389,12 +430,11 @@ Tensor latent_attention(const Tensor& h, const Tensor& w, const std::vector<int6
     a.D = D;
     a.R = R;
     a.V = V;
-    a.rank = rank;
     a.max_q = int(max_q);
     a.total_kv = total_kv;
-    if (fc::latent_prefill_supported(a)) {
+    if (rank % 8 == 0 && D > 0 && R <= 64 && fc::latent_prefill_supported(a)) {
       check_i32(*cu_q, "cu_q", B + 1);
-      check_i32(*cu_kv, "cu_kv", B + 1);
+      TORCH_CHECK(cu_kv.has_value(), "prefill needs the rows to gather");
       Tensor q, gate;
       const bool partial = st.proj.splits > 1;
       if (fc::latent_rotate_supported(st)) {
@@ -406,28 +446,29 @@ Tensor latent_attention(const Tensor& h, const Tensor& w, const std::vector<int6
         a.q = st.q;
         a.ld_q = (long long)H * (D + R);
       }
-      if (partial) {
+      if (partial && column_gate) {
         gate = torch::empty({T, H * V}, h.options());
         st.gate = gate.data_ptr();
       }
       fc::launch_latent_store(st, false, stream_now());
-      Tensor rows = torch::empty({total_kv, pool.size(2)}, h.options());
-      fc::launch_gather_rows(pool.data_ptr(), block_tables.data_ptr<int>(), ctx.data_ptr<int>(), cu_kv->data_ptr<int>(),
-                             rows.data_ptr(), B, int(max_ctx), int(pool.size(2)), int(pool.size(1)),
-                             int(block_tables.size(1)), int(pool.size(0)), false, ws.status, stream_now());
+      Tensor rows = gather_rows(pool, block_tables, ctx, *cu_kv, max_kv, total_kv);
       Tensor kv;
-      project(rows.narrow(1, 0, w_kv.size(1)), w_kv, c10::nullopt, false, kv);
+      product(rows.narrow(1, 0, w_kv.size(1)), w_kv, c10::nullopt, false, kv);
       a.k = kv.data_ptr();
       a.v = reinterpret_cast<const char*>(kv.data_ptr()) + off_uv * 2;
-      a.ld_kv = kv.size(1);
+      a.ld_k = a.ld_v = kv.size(1);
       a.rot = reinterpret_cast<const char*>(rows.data_ptr()) + rank * 2;
       a.ld_rot = rows.size(1);
       a.cu_q = cu_q->data_ptr<int>();
       a.cu_kv = cu_kv->data_ptr<int>();
-      if (partial) {
+      a.window = window;
+      a.sink = sinks;
+      if (head_gate) {
+        a.head_gate = gates.data_ptr<float>();
+      } else if (column_gate && partial) {
         a.gate = gate.data_ptr();
         a.ld_gate = H * V;
-      } else {
+      } else if (column_gate) {
         a.gate = reinterpret_cast<const char*>(st.proj.p) + (long long)st.off_g * 2;
         a.ld_gate = st.proj.ld;
       }
@@ -444,7 +485,7 @@ Tensor latent_attention(const Tensor& h, const Tensor& w, const std::vector<int6
   Tensor gate, o_lat = torch::empty({T, H, rank}, h.options());
   st.q = qn.data_ptr();
   st.q_abs = q_abs.data_ptr();
-  if (st.proj.splits > 1) {
+  if (st.proj.splits > 1 && column_gate) {
     gate = torch::empty({T, H * V}, h.options());
     st.gate = gate.data_ptr();
   }
@@ -468,33 +509,20 @@ Tensor latent_attention(const Tensor& h, const Tensor& w, const std::vector<int6
     else fc::launch_linear_simt(l, f32, stream_now());
   };
   head_linear(a);
-  fc::LatentAttn at;
+  fc::RowAttn at;
   at.T = T;
   at.H = H;
-  at.rank = rank;
-  at.R = R;
-  at.row_width = int(pool.size(2));
-  at.block_size = int(pool.size(1));
-  at.max_blocks = int(block_tables.size(1));
-  at.num_blocks = int(pool.size(0));
-  at.q_abs = q_abs.data_ptr();
-  at.pool = pool.data_ptr();
-  at.block_tables = block_tables.data_ptr<int>();
-  if (prefill) {
-    TORCH_CHECK(row_seq.has_value() && row_ctx.has_value(), "prefill rows need their request and visible rows");
-    check_i32(*row_seq, "row_seq", T);
-    check_i32(*row_ctx, "row_ctx", T);
-    at.row_seq = row_seq->data_ptr<int>();
-    at.row_ctx = row_ctx->data_ptr<int>();
-  } else {
-    TORCH_CHECK(B >= T, "one row per request expected");
-    at.row_ctx = ctx.data_ptr<int>();
-  }
-  at.o_lat = o_lat.data_ptr();
+  at.K = rank + R;
+  at.V = rank;
+  at.window = window;
+  at.q = q_abs.data_ptr();
+  set_pages(at, pool, block_tables, ctx, prefill, row_seq, row_ctx);
+  at.sink = sinks;
+  if (head_gate) at.head_gate = gates.data_ptr<float>();
+  at.out = o_lat.data_ptr();
+  at.ld_out = (long long)H * rank;
   at.scale = float(scale);
-  at.status = ws.status;
-  Tensor po, pl;
-  absorbed(at, f32, impl, max_ctx > 0 ? max_ctx : block_tables.size(1) * pool.size(1), o_lat, po, pl);
+  attend_rows(at, f32, impl, max_ctx, o_lat);
   a = fc::SimtLinear();
   a.x = o_lat.data_ptr();
   a.w = w_uv.data_ptr();
@@ -512,7 +540,7 @@ Tensor latent_attention(const Tensor& h, const Tensor& w, const std::vector<int6
   if (st.gate != nullptr) {
     a.gate.p = st.gate;
     a.gate.ld = H * V;
-  } else {
+  } else if (column_gate) {
     a.gate = st.proj;
     a.gate_off = st.off_g;
   }
@@ -521,47 +549,54 @@ Tensor latent_attention(const Tensor& h, const Tensor& w, const std::vector<int6
   return out;
 }
 
-// Absorbed attention alone: q_abs [T, H, rank + R] over the paged rows, one request per row -> [T, H, rank]
-Tensor latent_decode_rows(const Tensor& q_abs, const Tensor& pool, const Tensor& block_tables, const Tensor& ctx,
-                          int64_t rank, double scale, int64_t impl) {
-  check_elem(q_abs, "q");
-  check_elem(pool, "cache rows");
-  TORCH_CHECK(q_abs.dim() == 3 && q_abs.is_contiguous() && pool.dim() == 3 && pool.is_contiguous() &&
-                  pool.scalar_type() == q_abs.scalar_type() && pool.size(2) >= q_abs.size(2), "bad operands");
-  c10::cuda::CUDAGuard guard(q_abs.device());
-  const int64_t T = q_abs.size(0), H = q_abs.size(1);
+// Attention over shared rows alone: q [T, H, K] over the paged rows, one request per row -> [T, H * V]; the values of head h are
+// columns v_col + h / (H / v_heads) * V ... of a row
+Tensor latent_decode_rows(const Tensor& q, const Tensor& pool, const Tensor& block_tables, const Tensor& ctx, int64_t V, double scale,
+                          int64_t impl, int64_t v_col, int64_t v_heads, int64_t window, const OptTensor& sink,
+                          const OptTensor& head_gate) {
+  check_elem(q, "q");
+  TORCH_CHECK(q.dim() == 3 && q.is_contiguous() && v_heads > 0 && q.size(1) % v_heads == 0, "bad operands");
+  c10::cuda::CUDAGuard guard(q.device());
+  const int64_t T = q.size(0), H = q.size(1);
+  check_pool(pool, int(std::max(q.size(2), v_col + V * v_heads)), is_f32(q));
   check_i32(ctx, "context lengths", T);
-  check_i32(block_tables, "block tables", T);
-  TORCH_CHECK(block_tables.dim() == 2 && block_tables.size(0) >= T, "bad block tables");
-  Tensor o = torch::empty({T, H, rank}, q_abs.options()), po, pl;
-  fc::LatentAttn at;
+  check_block_tables(block_tables, int(T));
+  Tensor o = torch::empty({T, H, V}, q.options());
+  fc::RowAttn at;
   at.T = int(T);
   at.H = int(H);
-  at.rank = int(rank);
-  at.R = int(q_abs.size(2) - rank);
-  at.row_width = int(pool.size(2));
-  at.block_size = int(pool.size(1));
-  at.max_blocks = int(block_tables.size(1));
-  at.num_blocks = int(pool.size(0));
-  at.q_abs = q_abs.data_ptr();
-  at.pool = pool.data_ptr();
-  at.block_tables = block_tables.data_ptr<int>();
-  at.row_ctx = ctx.data_ptr<int>();
-  at.o_lat = o.data_ptr();
+  at.K = int(q.size(2));
+  at.V = int(V);
+  at.v_col = int(v_col);
+  at.v_heads = int(v_heads);
+  at.window = int(window);
+  at.q = q.data_ptr();
+  set_pages(at, pool, block_tables, ctx, false, c10::nullopt, c10::nullopt);
+  if (sink.has_value()) {
+    check_f32(*sink, "sink", H);
+    at.sink = sink->data_ptr<float>();
+  }
+  if (head_gate.has_value()) {
+    check_f32(*head_gate, "head gate", T * H);
+    at.head_gate = head_gate->data_ptr<float>();
+  }
+  at.out = o.data_ptr();
+  at.ld_out = H * V;
   at.scale = float(scale);
-  at.status = ws_of(pool).status;
-  absorbed(at, is_f32(q_abs), impl, block_tables.size(1) * pool.size(1), o, po, pl);
+  attend_rows(at, is_f32(q), impl, 0, o);
   return o;
 }
 
-// Expanded attention alone: q [T, H, D + R], kv [rows, H * D | H * V], rot [rows, R], gate [T, H * V] -> [T, H * V]
-Tensor latent_prefill_rows(const Tensor& q, const Tensor& kv, const Tensor& rot, const Tensor& gate, const Tensor& cu_q,
-                           const Tensor& cu_kv, int64_t D, int64_t V, double scale, int64_t max_q) {
+// Prefill attention alone: q [T, H, D + R], kv [rows, H * D | v_heads * V], rot [rows, R], gate [T, H * V] -> [T, H * V]
+Tensor latent_prefill_rows(const Tensor& q, const Tensor& kv, const Tensor& rot, const OptTensor& gate, const Tensor& cu_q,
+                           const Tensor& cu_kv, int64_t D, int64_t V, double scale, int64_t max_q, int64_t v_heads, int64_t window,
+                           const OptTensor& sink) {
   const int64_t T = q.size(0), H = q.size(1), R = rot.size(1), B = cu_q.numel() - 1;
-  TORCH_CHECK(q.is_contiguous() && kv.is_contiguous() && gate.is_contiguous() && rot.stride(1) == 1 && q.size(2) == D + R &&
-                  kv.size(1) == H * (D + V) && gate.size(1) == H * V && gate.size(0) == T && rot.size(0) == kv.size(0) &&
+  if (v_heads <= 0) v_heads = H;
+  TORCH_CHECK(q.is_contiguous() && kv.stride(1) == 1 && rot.stride(1) == 1 && q.size(2) == D + R &&
+                  kv.size(1) == H * D + v_heads * V && rot.size(0) == kv.size(0) &&
                   q.scalar_type() == torch::kBFloat16 && kv.scalar_type() == torch::kBFloat16 && q.is_cuda() &&
-                  rot.scalar_type() == torch::kBFloat16 && gate.scalar_type() == torch::kBFloat16, "bad operands");
+                  rot.scalar_type() == torch::kBFloat16, "bad operands");
   check_i32(cu_q, "cu_q", B + 1);
   check_i32(cu_kv, "cu_kv", B + 1);
   c10::cuda::CUDAGuard guard(q.device());
@@ -573,21 +608,29 @@ Tensor latent_prefill_rows(const Tensor& q, const Tensor& kv, const Tensor& rot,
   a.D = int(D);
   a.R = int(R);
   a.V = int(V);
-  a.rank = 8;
+  a.v_heads = int(v_heads);
   a.max_q = int(max_q);
   a.total_kv = kv.size(0);
+  a.window = int(window);
   TORCH_CHECK(fc::latent_prefill_supported(a), "sizes without a tensor-core form");
   a.q = q.data_ptr();
   a.ld_q = H * (D + R);
   a.k = kv.data_ptr();
   a.v = reinterpret_cast<const char*>(kv.data_ptr()) + H * D * 2;
-  a.ld_kv = kv.size(1);
+  a.ld_k = a.ld_v = kv.stride(0);
   a.rot = rot.data_ptr();
   a.ld_rot = rot.stride(0);
   a.cu_q = cu_q.data_ptr<int>();
   a.cu_kv = cu_kv.data_ptr<int>();
-  a.gate = gate.data_ptr();
-  a.ld_gate = H * V;
+  if (gate.has_value()) {
+    TORCH_CHECK(gate->is_contiguous() && gate->size(0) == T && gate->size(1) == H * V && gate->scalar_type() == torch::kBFloat16, "bad gate");
+    a.gate = gate->data_ptr();
+    a.ld_gate = H * V;
+  }
+  if (sink.has_value()) {
+    check_f32(*sink, "sink", H);
+    a.sink = sink->data_ptr<float>();
+  }
   a.out = out.data_ptr();
   a.ld_out = H * V;
   a.scale = float(scale);
@@ -602,13 +645,19 @@ void register_hybrid(pybind11::module_& m) {
   m.def("linear_wide", &linear_wide, "x @ w.T (+ bias), bf16 on tcgen05 or true fp32 on the CUDA cores", py::arg("x"),
         py::arg("w"), py::arg("bias") = py::none());
   m.def("embed_scaled", &embed_scaled);
-  m.def("linear_post_norm_add", &linear_post_norm_add);
+  m.def("linear_post_norm_add", &linear_post_norm_add, py::arg("a"), py::arg("w"), py::arg("bias"), py::arg("x"), py::arg("norm_w"),
+        py::arg("eps"), py::arg("experts") = nullptr, py::arg("row_of") = py::none(), py::arg("mix") = py::none(),
+        py::arg("factor") = py::none());
+  m.def("linear_xielu", &linear_xielu);
   m.def("rms_norm_wide", &rms_norm_wide);
   m.def("linear_gelu_mul", &linear_gelu_mul);
   m.def("gla", &gla);
   m.def("delta_rule", &delta_rule);
   m.def("latent_attention", &latent_attention);
   m.def("latent_decode_rows", &latent_decode_rows, py::arg("q"), py::arg("pool"), py::arg("block_tables"), py::arg("ctx"),
-        py::arg("rank"), py::arg("scale"), py::arg("impl") = 0);      // 0 choose, 1 CUDA cores, 3 mma.sync
-  m.def("latent_prefill_rows", &latent_prefill_rows);
+        py::arg("V"), py::arg("scale"), py::arg("impl") = 0, py::arg("v_col") = 0, py::arg("v_heads") = 1, py::arg("window") = 0,
+        py::arg("sink") = py::none(), py::arg("head_gate") = py::none());      // impl: 0 choose, 1 CUDA cores, 3 mma.sync
+  m.def("latent_prefill_rows", &latent_prefill_rows, py::arg("q"), py::arg("kv"), py::arg("rot"), py::arg("gate"), py::arg("cu_q"),
+        py::arg("cu_kv"), py::arg("D"), py::arg("V"), py::arg("scale"), py::arg("max_q"), py::arg("v_heads") = 0, py::arg("window") = 0,
+        py::arg("sink") = py::none());
 }

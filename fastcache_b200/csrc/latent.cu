@@ -1,6 +1,6 @@
-// Latent attention around the cache: norm of the latent, rotation of the shared key part and of the queries, store of
+// Latent attention around the cache: norms of the latents, rotation of the shared key part and of the queries, store of
 // the cache rows, gather of a request's rows for the expanded form, and the general (any size, fp32 or bf16) form of
-// absorbed attention over the paged rows.
+// attention over paged rows that all heads share.
 #include <algorithm>
 #include <stdexcept>
 #include <string>
@@ -12,6 +12,39 @@ namespace fc {
 
 using bf16 = __nv_bfloat16;
 constexpr int LS_THREADS = 256;
+
+// column r of a rotated part whose first column is `col` of the projection; cs: cos | sin, rot_dims / 2 each
+template <typename T>
+__device__ __forceinline__ float turned_at(const LatentStore& p, long long t, int col, int r, const float* cs) {
+  const float v = proj_at<T>(p.proj, t, col + r);
+  if (r >= p.rot_dims) return v;
+  const int half = p.rot_dims / 2;
+  const bool first = p.half ? r < half : (r & 1) == 0;
+  const int i = p.half ? (first ? r : r - half) : r >> 1, step = p.half ? half : 1;
+  const float o = proj_at<T>(p.proj, t, col + r + (first ? step : -step));
+  return first ? v * cs[i] - o * cs[half + i] : v * cs[i] + o * cs[half + i];
+}
+// cache row of token t: normed latent | rotated shared key part; by the whole CTA
+template <typename T, int THREADS>
+__device__ __forceinline__ void store_latent_row(const LatentStore& p, long long t, const float* cs, float* red) {
+  const int slot = p.slots[t];
+  if (slot < 0) return;
+  if (slot >= p.num_rows) {
+    if (threadIdx.x == 0) report(p.status, ST_BAD_INDEX);
+    return;
+  }
+  T* row = reinterpret_cast<T*>(p.pool) + (long long)slot * p.row_width;
+  float ss = 0.f;
+  for (int c = threadIdx.x; c < p.rank; c += THREADS) {
+    const float v = proj_at<T>(p.proj, t, p.off_kv + c);
+    ss += v * v;
+  }
+  const float inv = rsqrtf(cta_sum<THREADS>(ss, red) / float(p.rank) + p.eps);
+  for (int c = threadIdx.x; c < p.rank; c += THREADS)
+    row[c] = Elem<T>::put(proj_at<T>(p.proj, t, p.off_kv + c) * inv * p.norm_w[c]);
+  for (int r = threadIdx.x; r < p.R; r += THREADS)
+    row[p.rank + r] = Elem<T>::put(turned_at<T>(p, t, p.off_kv + p.rank, r, cs));
+}
 
 template <typename T>
 __global__ void __launch_bounds__(LS_THREADS)
@@ -33,14 +66,8 @@ latent_store_kernel(const LatentStore p) {
   const int qw = q_abs != nullptr ? p.D : Q;
   for (int idx = part * LS_THREADS + threadIdx.x; idx < p.H * Q; idx += parts * LS_THREADS) {
     const int h = idx / Q, c = idx - h * Q;
-    float v = proj_at<T>(p.proj, t, p.off_q + idx);
     const int r = c - p.D;
-    if (r >= 0 && r < p.rot_dims) {
-      const bool first = r < half;
-      const int i = first ? r : r - half;
-      const float o = proj_at<T>(p.proj, t, p.off_q + idx + (first ? half : -half));
-      v = first ? v * cs[i] - o * cs[half + i] : v * cs[i] + o * cs[half + i];
-    }
+    const float v = r < 0 ? proj_at<T>(p.proj, t, p.off_q + idx) : turned_at<T>(p, t, p.off_q + idx - r, r, cs);
     if (r < 0 || q_abs == nullptr) q[(t * p.H + h) * qw + c] = Elem<T>::put(v);
     else q_abs[(t * p.H + h) * (p.rank + p.R) + p.rank + r] = Elem<T>::put(v);
   }
@@ -50,33 +77,33 @@ latent_store_kernel(const LatentStore p) {
       gate[t * p.H * p.V + c] = Elem<T>::put(proj_at<T>(p.proj, t, p.off_g + c));
   }
   if (p.off_kv < 0 || part != 0) return;
-  // cache row: normed latent | rotated shared key part
-  const int slot = p.slots[t];
-  if (slot < 0) return;
-  if (slot >= p.num_rows) {
-    if (threadIdx.x == 0) report(p.status, ST_BAD_INDEX);
-    return;
-  }
-  T* row = reinterpret_cast<T*>(p.pool) + (long long)slot * p.row_width;
+  store_latent_row<T, LS_THREADS>(p, t, cs, red);
+}
+
+// Normed query latent, cache row and head gates of a token (the queries are made from the query latent afterwards)
+template <typename T>
+__global__ void __launch_bounds__(LS_THREADS)
+latent_inputs_kernel(const LatentStore p) {
+  __shared__ float red[LS_THREADS / 32];
+  extern __shared__ float cs[];
+  const int half = p.rot_dims / 2;
+  pdl_launch_dependents();
+  pdl_wait();
+  const long long t = blockIdx.x;
+  const double pos = double(p.positions[t]);
+  for (int i = threadIdx.x; i < half; i += LS_THREADS) rope_angle(pos, p.log2_base, i, p.rot_dims, cs[i], cs[half + i]);
   float ss = 0.f;
-  for (int c = threadIdx.x; c < p.rank; c += LS_THREADS) {
-    const float v = proj_at<T>(p.proj, t, p.off_kv + c);
+  for (int c = threadIdx.x; c < p.q_rank; c += LS_THREADS) {
+    const float v = proj_at<T>(p.proj, t, p.off_dq + c);
     ss += v * v;
   }
-  const float inv = rsqrtf(cta_sum<LS_THREADS>(ss, red) / float(p.rank) + p.eps);
-  for (int c = threadIdx.x; c < p.rank; c += LS_THREADS)
-    row[c] = Elem<T>::put(proj_at<T>(p.proj, t, p.off_kv + c) * inv * p.norm_w[c]);
-  for (int r = threadIdx.x; r < p.R; r += LS_THREADS) {
-    const int col = p.off_kv + p.rank + r;
-    float v = proj_at<T>(p.proj, t, col);
-    if (r < p.rot_dims) {
-      const bool first = r < half;
-      const int i = first ? r : r - half;
-      const float o = proj_at<T>(p.proj, t, col + (first ? half : -half));
-      v = first ? v * cs[i] - o * cs[half + i] : v * cs[i] + o * cs[half + i];
-    }
-    row[p.rank + r] = Elem<T>::put(v);
-  }
+  const float inv = rsqrtf(cta_sum<LS_THREADS>(ss, red) / float(p.q_rank) + p.eps);      // also makes cs visible
+  T* cq = reinterpret_cast<T*>(p.cq) + t * p.ld_cq;
+  for (int c = threadIdx.x; c < p.ld_cq; c += LS_THREADS)
+    cq[c] = Elem<T>::put(c < p.q_rank ? proj_at<T>(p.proj, t, p.off_dq + c) * inv * p.q_norm_w[c] : 0.f);
+  if (p.head_gate != nullptr)
+    for (int h = threadIdx.x; h < p.H; h += LS_THREADS) p.head_gate[t * p.H + h] = sigmoid_f(proj_at<T>(p.proj, t, p.off_g + h));
+  if (p.off_kv >= 0) store_latent_row<T, LS_THREADS>(p, t, cs, red);
 }
 
 // The same for many rows of a finished projection whose queries are then read where they are: the rotated parts are
@@ -87,7 +114,7 @@ template <typename T>
 __global__ void __launch_bounds__(LR_WARPS * 32)
 latent_rotate_kernel(const LatentStore p) {
   extern __shared__ float cs[];
-  const int half = p.rot_dims / 2, quads = half / 4;
+  const int half = p.rot_dims / 2, quads = half / 4;        // quads of pairs
   pdl_launch_dependents();
   pdl_wait();
   const long long t = blockIdx.x;
@@ -99,6 +126,15 @@ latent_rotate_kernel(const LatentStore p) {
   auto rotate = [&](const T* su, T* du, int i0) {            // quads at columns i0 and half + i0 of a rotated part
     ProjSrc s;
     s.p = su;
+    if (!p.half) {                                           // columns 2 i0 .. 2 i0 + 7
+#pragma unroll
+      for (int e = 0; e < 4; e += 2) {
+        const float4 a = proj_at4<T>(s, 0, 2 * (i0 + e));
+        const float2 c = *reinterpret_cast<const float2*>(cs + i0 + e), d = *reinterpret_cast<const float2*>(cs + half + i0 + e);
+        store4(du + 2 * (i0 + e), a.x * c.x - a.y * d.x, a.y * c.x + a.x * d.x, a.z * c.y - a.w * d.y, a.w * c.y + a.z * d.y);
+      }
+      return;
+    }
     const float4 u = proj_at4<T>(s, 0, i0), v = proj_at4<T>(s, 0, half + i0);
     const float4 c = *reinterpret_cast<const float4*>(cs + i0), d = *reinterpret_cast<const float4*>(cs + half + i0);
     store4(du + i0, u.x * c.x - v.x * d.x, u.y * c.y - v.y * d.y, u.z * c.z - v.z * d.z, u.w * c.w - v.w * d.w);
@@ -135,6 +171,15 @@ bool latent_rotate_supported(const LatentStore& p) {
   return p.proj.splits <= 1 && p.rot_dims == p.R && p.R % 8 == 0 && p.D % 4 == 0 && p.rank % 4 == 0;
 }
 
+void launch_latent_inputs(const LatentStore& p, bool f32, cudaStream_t s) {
+  if (p.T == 0) return;
+  const size_t smem = size_t(std::max(2, p.rot_dims)) * 4;
+  if (f32) launch_pdl(PDL_ROPE, latent_inputs_kernel<float>, dim3(p.T), dim3(LS_THREADS), smem, s, p);
+  else launch_pdl(PDL_ROPE, latent_inputs_kernel<bf16>, dim3(p.T), dim3(LS_THREADS), smem, s, p);
+  const cudaError_t e = cudaGetLastError();
+  if (e != cudaSuccess) throw std::runtime_error(std::string("latent inputs: ") + cudaGetErrorString(e));
+}
+
 void launch_latent_store(const LatentStore& p, bool f32, cudaStream_t s) {
   if (p.T == 0) return;
   if (p.q == nullptr) {                                      // in place
@@ -157,25 +202,25 @@ void launch_latent_store(const LatentStore& p, bool f32, cudaStream_t s) {
 }
 
 // ------------------------------------------------------------------ gather
-// rows [0, ctx[b]) of every request, one after another (cu_kv), 16 bytes per thread
+// the last cu_kv[b + 1] - cu_kv[b] of the ctx[b] rows of every request, one after another, 16 bytes per thread
 template <int BYTES>
 __global__ void __launch_bounds__(256)
 gather_rows_kernel(const uint8_t* __restrict__ pool, const int* __restrict__ block_tables, const int* __restrict__ ctx,
                    const int* __restrict__ cu_kv, uint8_t* __restrict__ out, int chunks, int block_size,
                    int max_blocks, int num_blocks, uint32_t* status) {
   const int b = blockIdx.y;
-  const int n = min(min(ctx[b], cu_kv[b + 1] - cu_kv[b]), max_blocks * block_size);
+  const int len = min(ctx[b], max_blocks * block_size), n = min(len, cu_kv[b + 1] - cu_kv[b]);
   const int per = 256 / chunks > 0 ? 256 / chunks : 1;
   const int row0 = blockIdx.x * per;
   for (int i = threadIdx.x; i < per * chunks; i += 256) {
     const int row = row0 + i / chunks, c = i % chunks;
     if (row >= n) return;
-    const int blk = block_tables[(long long)b * max_blocks + row / block_size];
+    const int at = len - n + row, blk = block_tables[(long long)b * max_blocks + at / block_size];
     if (blk < 0 || blk >= num_blocks) {
       report(status, ST_BAD_INDEX);
       continue;
     }
-    const long long src = (long long)blk * block_size + row % block_size;
+    const long long src = (long long)blk * block_size + at % block_size;
     reinterpret_cast<uint4*>(out)[((long long)cu_kv[b] + row) * chunks + c] =
         reinterpret_cast<const uint4*>(pool)[src * chunks + c];
   }
@@ -193,31 +238,31 @@ void launch_gather_rows(const void* pool, const int* block_tables, const int* ct
   if (e != cudaSuccess) throw std::runtime_error(std::string("gather rows: ") + cudaGetErrorString(e));
 }
 
-// ------------------------------------------------------------------ absorbed attention, general form
+// ------------------------------------------------------------------ attention over shared rows, general form
 constexpr int LA_THREADS = 128;
 constexpr int LA_TILE = 64;
-constexpr int LA_COLS = 8;           // latent columns per thread: rank <= 1024
+constexpr int LA_COLS = 8;           // value columns per thread: up to 1024 per head
 
 template <typename T>
 __global__ void __launch_bounds__(LA_THREADS)
-latent_attn_simt_kernel(const LatentAttn p) {
-  extern __shared__ float sq[];                    // rank + R query values
+row_attn_simt_kernel(const RowAttn p) {
+  extern __shared__ float sq[];                    // K query values
   __shared__ float ss[LA_TILE];
   __shared__ const T* srow[LA_TILE];
   const int t = blockIdx.x, h = blockIdx.y;
-  const int w = p.rank + p.R;
   const int ctx = min(p.row_ctx[t], p.max_blocks * p.block_size);
   const int b = p.row_seq != nullptr ? p.row_seq[t] : t;
-  const T* q = reinterpret_cast<const T*>(p.q_abs) + ((long long)t * p.H + h) * w;
+  const int first = p.window > 0 ? max(0, ctx - p.window) : 0, vc = p.v_col + h / (p.H / p.v_heads) * p.V;
+  const T* q = reinterpret_cast<const T*>(p.q) + ((long long)t * p.H + h) * p.K;
   const T* pool = reinterpret_cast<const T*>(p.pool);
   const int* bt = p.block_tables + (long long)b * p.max_blocks;
-  for (int c = threadIdx.x; c < w; c += LA_THREADS) sq[c] = ctx > 0 ? Elem<T>::get(q[c]) * p.scale : 0.f;
+  for (int c = threadIdx.x; c < p.K; c += LA_THREADS) sq[c] = ctx > 0 ? Elem<T>::get(q[c]) * p.scale : 0.f;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   float acc[LA_COLS];
 #pragma unroll
   for (int i = 0; i < LA_COLS; ++i) acc[i] = 0.f;
   float m = -INFINITY, l = 0.f;
-  for (int k0 = 0; k0 < ctx; k0 += LA_TILE) {
+  for (int k0 = first; k0 < ctx; k0 += LA_TILE) {
     const int n = min(LA_TILE, ctx - k0);
     __syncthreads();
     if (threadIdx.x < n) {
@@ -232,7 +277,7 @@ latent_attn_simt_kernel(const LatentAttn p) {
     __syncthreads();
     for (int j = warp; j < n; j += LA_THREADS / 32) {
       float d = 0.f;
-      for (int c = lane; c < w; c += 32) d = fmaf(sq[c], Elem<T>::get(srow[j][c]), d);
+      for (int c = lane; c < p.K; c += 32) d = fmaf(sq[c], Elem<T>::get(srow[j][c]), d);
       d = warp_sum(d);
       if (lane == 0) ss[j] = d;
     }
@@ -250,28 +295,37 @@ latent_attn_simt_kernel(const LatentAttn p) {
 #pragma unroll
       for (int i = 0; i < LA_COLS; ++i) {
         const int c = threadIdx.x + i * LA_THREADS;
-        if (c < p.rank) acc[i] = fmaf(e, Elem<T>::get(srow[j][c]), acc[i]);
+        if (c < p.V) acc[i] = fmaf(e, Elem<T>::get(srow[j][vc + c]), acc[i]);
       }
     }
   }
-  const float inv = l > 0.f ? 1.f / l : 0.f;
-  T* o = reinterpret_cast<T*>(p.o_lat) + ((long long)t * p.H + h) * p.rank;
+  if (p.sink != nullptr && ctx > 0) l += expf(p.sink[h] - m);
+  float inv = l > 0.f ? 1.f / l : 0.f;
+  if (p.head_gate != nullptr) inv *= p.head_gate[(long long)t * p.H + h];
+  T* o = reinterpret_cast<T*>(p.out) + t * p.ld_out + h * p.V;
 #pragma unroll
   for (int i = 0; i < LA_COLS; ++i) {
     const int c = threadIdx.x + i * LA_THREADS;
-    if (c < p.rank) o[c] = Elem<T>::put(acc[i] * inv);
+    if (c < p.V) o[c] = Elem<T>::put(acc[i] * inv);
   }
 }
 
-void launch_latent_attn_simt(const LatentAttn& p, bool f32, cudaStream_t s) {
+void launch_row_attn_simt(const RowAttn& p, bool f32, cudaStream_t s) {
   if (p.T == 0) return;
-  if (p.rank > LA_THREADS * LA_COLS) throw std::runtime_error("latent attention: kv_rank is limited to 1024");
+  if (p.V > LA_THREADS * LA_COLS) throw std::runtime_error("attention over shared rows: values are limited to 1024 columns (kv_rank)");
   const dim3 grid(p.T, p.H);
-  const size_t smem = size_t(p.rank + p.R) * 4;
-  if (f32) latent_attn_simt_kernel<float><<<grid, LA_THREADS, smem, s>>>(p);
-  else latent_attn_simt_kernel<bf16><<<grid, LA_THREADS, smem, s>>>(p);
+  const size_t smem = size_t(p.K) * 4;
+  auto go = [&](auto kern) {
+    if (smem > 40 * 1024) {
+      if (smem > 200 * 1024) throw std::runtime_error("attention over shared rows: scores are limited to 50000 columns");
+      cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem));
+    }
+    kern<<<grid, LA_THREADS, smem, s>>>(p);
+  };
+  if (f32) go(row_attn_simt_kernel<float>);
+  else go(row_attn_simt_kernel<bf16>);
   const cudaError_t e = cudaGetLastError();
-  if (e != cudaSuccess) throw std::runtime_error(std::string("latent attention: ") + cudaGetErrorString(e));
+  if (e != cudaSuccess) throw std::runtime_error(std::string("attention over shared rows: ") + cudaGetErrorString(e));
 }
 
 }  // namespace fc

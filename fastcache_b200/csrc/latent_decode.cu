@@ -1,6 +1,7 @@
 // Absorbed latent attention of decode-size batches (bf16): every query row attends to the cache rows of its request as
 // they are, key = [latent | rotated part], value = latent, shared by all heads.
 //
+// Rows before the window are skipped tile by tile and masked; the sink and the head gates join at the end.
 // Grid (query row, group of 16 * MT heads, split of the context).  One tile of 32 cache rows in shared memory is both the
 // keys and the values of all heads of the CTA, so a row is read once.  Two groups of eight warps take alternate tiles, each
 // with its own two-stage TMA ring (128-byte swizzle, boxes that never straddle a page), running maximum and accumulators:
@@ -38,7 +39,7 @@ __device__ __forceinline__ uint32_t ld_swz(int rows, int row, int chunk) {
 
 template <int MT, int NPW>
 __global__ void __launch_bounds__(LD_THREADS, 1)
-latent_decode_kernel(const __grid_constant__ CUtensorMap tm, const LatentAttn p, int box_rows, int nc, float scale_log2) {
+latent_decode_kernel(const __grid_constant__ CUtensorMap tm, const RowAttn p, int box_rows, int nc, float scale_log2) {
   constexpr int HR = MT * 16;                     // head rows of this CTA
   constexpr int TPR = LD_GT / HR;                 // softmax threads per head row
   constexpr int KPT = LD_TILE / TPR;              // keys per softmax thread
@@ -69,19 +70,20 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm, const LatentAttn p,
   asm volatile("fence.proxy.async.global;" ::: "memory");          // rows were written with ordinary stores
   const int ctx = min(p.row_ctx[t], p.max_blocks * p.block_size);
   const int b = p.row_seq != nullptr ? p.row_seq[t] : t;
-  const int tiles = (ctx + LD_TILE - 1) / LD_TILE;
-  const int per = (tiles + p.splits - 1) / p.splits;
-  const int tile0 = split * per, n_tiles = max(0, min(tiles, tile0 + per) - tile0);
+  const int first = p.window > 0 ? max(0, ctx - p.window) : 0;     // first visible row
+  const int tiles = (ctx + LD_TILE - 1) / LD_TILE, start = first / LD_TILE;
+  const int per = (tiles - start + p.splits - 1) / p.splits;
+  const int tile0 = start + split * per, n_tiles = max(0, min(tiles, tile0 + per) - tile0);
   const int n_mine = (n_tiles - grp + LD_GROUPS - 1) / LD_GROUPS;  // tiles grp, grp + 2, ...
   const int* bt = p.block_tables + (long long)b * p.max_blocks;
-  const int w = p.rank + p.R;
+  const int w = p.K;
 
   // Q, zero-padded to whole sub-tiles and head rows
   for (int i = tid; i < HR * nc * 8; i += LD_THREADS) {
     const int r = i / (nc * 8), ch = i - r * (nc * 8);
     uint4 v = make_uint4(0, 0, 0, 0);
     if (h0 + r < p.H && ch * 8 < w)
-      v = __ldcg(reinterpret_cast<const uint4*>(reinterpret_cast<const bf16*>(p.q_abs) +
+      v = __ldcg(reinterpret_cast<const uint4*>(reinterpret_cast<const bf16*>(p.q) +
                                                 ((long long)t * p.H + h0 + r) * w + ch * 8));
     *reinterpret_cast<uint4*>(s_q + ld_swz(HR, r, ch)) = v;
   }
@@ -161,7 +163,8 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm, const LatentAttn p,
     group_sync();
     // ---- softmax of one head row by TPR threads
     {
-      const int valid = ctx - (tile0 + grp + it * LD_GROUPS) * LD_TILE;      // keys of this tile that exist
+      const int row0 = (tile0 + grp + it * LD_GROUPS) * LD_TILE;
+      const int valid = ctx - row0, hidden = first - row0;         // keys of this tile that exist; that lie before the window
       float v[KPT];
       float mx = -INFINITY;
 #pragma unroll
@@ -169,12 +172,12 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm, const LatentAttn p,
         float s = 0.f;
 #pragma unroll
         for (int x = 0; x < LD_PARTS; ++x) s += s_s[(x * HR + srow) * SLD + sk0 + i];
-        v[i] = sk0 + i < valid ? s * scale_log2 : -INFINITY;
+        v[i] = sk0 + i < valid && sk0 + i >= hidden ? s * scale_log2 : -INFINITY;
         mx = fmaxf(mx, v[i]);
       }
 #pragma unroll
       for (int x = 1; x < TPR; x <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, x));
-      const float mn = fmaxf(m_run, mx);                           // a tile has at least one key
+      const float mn = fmaxf(m_run, mx);                           // a tile has at least one visible key
       const float cor = exp2f(m_run - mn);
       m_run = mn;
       float rs = 0.f;
@@ -214,7 +217,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm, const LatentAttn p,
 #pragma unroll
       for (int n = 0; n < NPW; ++n) {
         const int cg = warp + n * LD_WARPS;                        // 16-column group of the latent
-        if (cg * 16 >= p.rank) continue;
+        if (cg * 16 >= p.V) continue;
         uint32_t b0, b1, b2, b3;
         ldsm_x4_t(kv + ld_swz(LD_TILE, ks * 16 + (mat & 1) * 8 + (lane & 7), cg * 2 + (mat >> 1)), b0, b1, b2, b3);
 #pragma unroll
@@ -250,11 +253,15 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm, const LatentAttn p,
   if (gt % TPR == 0) {
     const float m1 = s_m[srow], mm = fmaxf(m_run, m1);
     const float w0 = m_run == -INFINITY ? 0.f : exp2f(m_run - mm), w1 = m1 == -INFINITY ? 0.f : exp2f(m1 - mm);
-    const float l = l_run * w0 + s_m[HR + srow] * w1, inv = l > 0.f ? 1.f / l : 0.f;
+    float l = l_run * w0 + s_m[HR + srow] * w1;
+    const int head = h0 + srow;
+    if (p.splits > 1 && head < p.H)
+      p.part_lse[((long long)t * p.H + head) * p.splits + split] = l > 0.f ? mm + log2f(l) : -INFINITY;
+    if (p.splits == 1 && p.sink != nullptr && head < p.H && l > 0.f) l += exp2f(p.sink[head] * 1.4426950408889634f - mm);
+    float inv = l > 0.f ? 1.f / l : 0.f;
+    if (p.splits == 1 && p.head_gate != nullptr && head < p.H) inv *= p.head_gate[(long long)t * p.H + head];
     s_w[srow] = w0 * inv;
     s_w[HR + srow] = w1 * inv;
-    if (p.splits > 1 && h0 + srow < p.H)
-      p.part_lse[((long long)t * p.H + h0 + srow) * p.splits + split] = l > 0.f ? mm + log2f(l) : -INFINITY;
   }
   group_sync();
 #pragma unroll
@@ -268,51 +275,54 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm, const LatentAttn p,
 #pragma unroll
       for (int n = 0; n < NPW; ++n) {
         const int cg = warp + n * LD_WARPS;
-        if (cg * 16 >= p.rank) continue;
+        if (cg * 16 >= p.V) continue;
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
           const int col = cg * 16 + e * 8 + q4 * 2, i0 = (m * NPW + n) * 8 + e * 4 + half * 2;
           const float a = o[m][n][e][half * 2] * w0 + s_o[i0 * LD_GT + gt] * w1;
           const float c = o[m][n][e][half * 2 + 1] * w0 + s_o[(i0 + 1) * LD_GT + gt] * w1;
           if (p.splits == 1)
-            *reinterpret_cast<uint32_t*>(reinterpret_cast<bf16*>(p.o_lat) + row * p.rank + col) = pack_bf16(a, c);
+            *reinterpret_cast<uint32_t*>(reinterpret_cast<bf16*>(p.out) + t * p.ld_out + (h0 + r) * p.V + col) = pack_bf16(a, c);
           else
-            *reinterpret_cast<float2*>(p.part_o + (row * p.splits + split) * p.rank + col) = make_float2(a, c);
+            *reinterpret_cast<float2*>(p.part_o + (row * p.splits + split) * p.V + col) = make_float2(a, c);
         }
       }
     }
 }
-// o_lat[row] = sum_s 2^(lse_s - max) part_o[row, s] / sum_s 2^(lse_s - max); one CTA per (row, head), 4 columns a thread
+// out[row] = sum_s 2^(lse_s - max) part_o[row, s] / (sum_s 2^(lse_s - max) + sink); one CTA per (row, head), 4 columns a thread
 __global__ void __launch_bounds__(128)
-latent_merge_kernel(const LatentAttn p) {
+latent_merge_kernel(const RowAttn p) {
   __shared__ float s_w[LD_MAX_SPLITS];
   pdl_launch_dependents();
   pdl_wait();
-  const long long row = blockIdx.x;
+  const long long row = blockIdx.x, t = row / p.H;
+  const int h = int(row - t * p.H);
   if (threadIdx.x < 32) {
     const int lane = threadIdx.x;
     const float l = lane < p.splits ? __ldcg(p.part_lse + row * p.splits + lane) : -INFINITY;
     const float mx = warp_max(l);
     const float wgt = l == -INFINITY ? 0.f : exp2f(l - mx);
-    const float den = warp_sum(wgt);
-    s_w[lane] = den > 0.f ? wgt / den : 0.f;
+    float den = warp_sum(wgt);
+    if (p.sink != nullptr && den > 0.f) den += exp2f(p.sink[h] * 1.4426950408889634f - mx);
+    const float f = p.head_gate != nullptr ? p.head_gate[row] : 1.f;
+    s_w[lane] = den > 0.f ? wgt / den * f : 0.f;
   }
   __syncthreads();
-  for (int c = threadIdx.x * 4; c < p.rank; c += 512) {
+  for (int c = threadIdx.x * 4; c < p.V; c += 512) {
     float a[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll 8
     for (int s = 0; s < p.splits; ++s) {
       const float f = s_w[s];
-      const float4 v = __ldcg(reinterpret_cast<const float4*>(p.part_o + (row * p.splits + s) * p.rank + c));
+      const float4 v = __ldcg(reinterpret_cast<const float4*>(p.part_o + (row * p.splits + s) * p.V + c));
       a[0] = fmaf(f, v.x, a[0]);
       a[1] = fmaf(f, v.y, a[1]);
       a[2] = fmaf(f, v.z, a[2]);
       a[3] = fmaf(f, v.w, a[3]);
     }
-    store4(reinterpret_cast<bf16*>(p.o_lat) + row * p.rank + c, a[0], a[1], a[2], a[3]);
+    store4(reinterpret_cast<bf16*>(p.out) + t * p.ld_out + h * p.V + c, a[0], a[1], a[2], a[3]);
   }
 }
-void launch_latent_merge(const LatentAttn& p, cudaStream_t s) {
+void launch_latent_merge(const RowAttn& p, cudaStream_t s) {
   launch_pdl(PDL_DECODE_MERGE, latent_merge_kernel, dim3(unsigned((long long)p.T * p.H)), dim3(128), 0, s, p);
   const cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess) throw std::runtime_error(std::string("latent merge: ") + cudaGetErrorString(e));
@@ -323,24 +333,24 @@ static int ld_box_rows(int block_size) {
   while (box > block_size || block_size % box != 0) box >>= 1;
   return box;
 }
-static int ld_nc(const LatentAttn& p) { return (p.row_width + 63) / 64; }
+static int ld_nc(const RowAttn& p) { return (p.row_width + 63) / 64; }
 static int ld_smem(int mt, int nc) {
   const int hr = mt * 16;
   return LD_GROUPS * LD_STAGES * nc * LD_SUB + nc * hr * 128 + LD_GROUPS * hr * 128 +
          LD_GROUPS * LD_PARTS * hr * (LD_TILE + 4) * 4 + (2 + LD_GROUPS) * hr * 4 + LD_GROUPS * LD_STAGES * 8 + 1024;
 }
-static int ld_mt(const LatentAttn& p) {
+static int ld_mt(const RowAttn& p) {
   int mt = p.H > 32 ? 4 : p.H > 16 ? 2 : 1;
-  while (mt > 1 && (ld_smem(mt, ld_nc(p)) > 227 * 1024 || (mt == 4 && p.rank > 256))) mt >>= 1;
+  while (mt > 1 && (ld_smem(mt, ld_nc(p)) > 227 * 1024 || (mt == 4 && p.V > 256))) mt >>= 1;
   return mt;
 }
 
-bool latent_decode_supported(const LatentAttn& p) {
-  return p.rank % 16 == 0 && p.rank <= 512 && (p.rank + p.R) % 8 == 0 && ld_box_rows(p.block_size) >= 8 &&
+bool latent_decode_supported(const RowAttn& p) {
+  return p.v_col == 0 && p.v_heads == 1 && p.V % 16 == 0 && p.V <= 512 && p.K % 8 == 0 && p.ld_out % 4 == 0 && ld_box_rows(p.block_size) >= 8 &&
          ld_smem(ld_mt(p), ld_nc(p)) <= 227 * 1024;
 }
 
-int latent_decode_splits(const LatentAttn& p, int max_ctx, int num_sms) {
+int latent_decode_splits(const RowAttn& p, int max_ctx, int num_sms) {
   const int hr = ld_mt(p) * 16;
   const int ctas = p.T * ((p.H + hr - 1) / hr);
   const int by_len = std::max(1, max_ctx / (4 * LD_TILE));      // two tiles per group at least
@@ -349,7 +359,7 @@ int latent_decode_splits(const LatentAttn& p, int max_ctx, int num_sms) {
   return s;
 }
 
-void launch_latent_decode(const LatentAttn& p, cudaStream_t s) {
+void launch_latent_decode(const RowAttn& p, cudaStream_t s) {
   if (p.T == 0) return;
   const int box = ld_box_rows(p.block_size), nc = ld_nc(p), mt = ld_mt(p), smem = ld_smem(mt, nc);
   const CUtensorMap tm = make_tmap_bf16_2d(p.pool, (uint64_t)p.num_blocks * p.block_size, p.row_width, p.row_width, box, 64);
@@ -362,8 +372,8 @@ void launch_latent_decode(const LatentAttn& p, cudaStream_t s) {
   };
   auto pick = [&](auto m) {
     constexpr int MT = decltype(m)::value;
-    if (p.rank <= 128) go(latent_decode_kernel<MT, 1>);
-    else if (p.rank <= 256) go(latent_decode_kernel<MT, 2>);
+    if (p.V <= 128) go(latent_decode_kernel<MT, 1>);
+    else if (p.V <= 256) go(latent_decode_kernel<MT, 2>);
     else if constexpr (MT < 4) go(latent_decode_kernel<MT, 4>);    // ld_mt keeps the accumulators in registers
   };
   if (mt == 1) pick(std::integral_constant<int, 1>{});

@@ -1,17 +1,21 @@
-// Absorbed latent attention of decode-size batches on tcgen05 (the general tensor-core form is in latent_decode.cu).
+// Attention of decode-size batches over cache rows that all heads share, on tcgen05 (the general tensor-core form is in
+// latent_decode.cu): latent rows, whose first columns are the values too, or rows with the keys of several key heads side by
+// side and the values behind them.
 //
 // Grid (query row, group of 32 heads, split of the context).  A CTA walks its rows of the cache in tiles of 64.  The wide
 // operand of both products is the cache, not the few heads:
-//     S^T [64 rows x 32 heads]    = rows (latent | rotated part) * Q^T        A: row tile, K-major; B: Q, K-major
-//     O^T [128 latents x 32 heads] += rows^T * P^T, one block per 128 latents  A: the same tile, MN-major; B: P, K-major
+//     S^T [64 rows x 32 heads]    = rows (key columns) * Q^T                   A: row tile, K-major; B: Q, K-major
+//     O^T [128 columns x 32 heads] += rows^T * P^T, one block per 128 value columns  A: MN-major; B: P, K-major
 // (S^T is issued with 128 rows; the upper 64 read the shared memory behind the tile and their lanes are ignored.)  Shared
-// memory holds a tile as pairs of 64-column sub-tiles (128 latents each) in a ring of ten pairs, and the columns behind
-// them in a ring of two sub-tiles; a pair is refilled as soon as its block of O^T is done.
+// memory holds a tile as pairs of 64-column sub-tiles in a ring, and the columns behind latent pairs in a ring of two
+// sub-tiles.  Latent pairs serve both products and are refilled as soon as their block of O^T is done; other rows have pairs
+// of keys, then pairs of values.  Where value heads differ, every head takes its own columns of O^T at the end.
 //   warp 0     TMA, boxes that never straddle a page
-//   warp 1     tcgen05.mma issuer; the scores of the next tile go first, so that they overlap the softmax of this one
-//   warps 2-5  one cache row per thread: P = 2^(s - ref) for all heads against a reference per head (the first row's
-//              score; should a score outgrow it by 2^64, all accumulators move to the new maximum), P to shared memory
-//              as bf16, sums per thread; at the end one latent per thread
+//   warp 1     tcgen05.mma issuer; the scores of the next tile go first, so that they overlap the softmax of this one (where
+//              the ring holds the values of one tile and the keys of the next)
+//   warps 2-5  one cache row per thread: P = 2^(s - ref) for all heads against a reference per head (the score of the first
+//              visible row; should a score outgrow it by 2^64, all accumulators move to the new maximum), P to shared memory
+//              as bf16, sums per thread; at the end one value column per thread
 #include <algorithm>
 #include <stdexcept>
 #include <string>
@@ -23,12 +27,20 @@
 namespace fc {
 
 using bf16 = __nv_bfloat16;
-constexpr int LT_ROWS = 64, LT_HEADS = 32, LT_PAIRS = 10, LT_THREADS = 192;
+constexpr int LT_ROWS = 64, LT_HEADS = 32, LT_MAX_RING = 12, LT_THREADS = 192;
 constexpr int LT_SUB = LT_ROWS * 128;             // bytes of a [64 rows x 64 columns] sub-tile
 constexpr int LT_QSUB = LT_HEADS * 128;           // of a [32 heads x 64 columns] sub-tile
-constexpr int LT_TMEM = 256;                      // S^T of even / odd tiles [0, 32) [32, 64), O^T blocks [64 + 32 b, ...)
+// tensor memory: S^T of even / odd tiles [0, 32) [32, 64), O^T blocks [64 + 32 b, ...)
 constexpr float LT_RANGE = 64.f;                  // log2 units above the reference that P may reach
-constexpr int LT_MAX_SUBS = 9;
+constexpr int LT_MAX_BLOCKS = 14;
+constexpr float LT_LOG2E = 1.4426950408889634f;
+
+// A tile in the ring: `pairs` slots of 128 columns, of which the first `keys` enter the scores and the last `values` make the
+// blocks of O^T; `extra`: 64 more key columns; `shared`: keys and values are the same pairs
+struct LtTile {
+  int pairs, keys, values, extra, ring, ahead, tmem;
+  bool shared;
+};
 
 __device__ __forceinline__ uint64_t lt_sdesc(uint32_t addr, uint32_t lbo_bytes, uint32_t sbo_bytes) {
   uint64_t d = 0;
@@ -74,18 +86,19 @@ __device__ __forceinline__ void lt_load(void* dst, const CUtensorMap* m, uint64_
 }
 
 __global__ void __launch_bounds__(LT_THREADS, 1)
-latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm, const LatentAttn p, int box_rows, int pairs, int extra,
+latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm, const RowAttn p, const LtTile w, int box_rows,
                         float scale_log2) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
-  uint8_t* s_kv = smem;                                            // [LT_PAIRS] pairs of sub-tiles
-  uint8_t* s_x = s_kv + LT_PAIRS * 2 * LT_SUB;                     // the columns behind the pairs
-  uint8_t* s_q = s_x + 2 * LT_SUB;                                 // [LT_MAX_SUBS] sub-tiles
-  uint8_t* s_p = s_q + LT_MAX_SUBS * LT_QSUB;
+  const int subs = w.keys * 2 + w.extra;                           // sub-tiles of Q
+  uint8_t* s_kv = smem;                                            // [ring] pairs of sub-tiles
+  uint8_t* s_x = s_kv + w.ring * 2 * LT_SUB;                       // the columns behind the pairs
+  uint8_t* s_q = s_x + (w.extra ? 2 * LT_SUB : 0);                 // [subs] sub-tiles
+  uint8_t* s_p = s_q + subs * LT_QSUB;
   float* s_ref = reinterpret_cast<float*>(s_p + 2 * LT_QSUB);      // (P of even / odd tiles)  [32] reference
   float* s_red = s_ref + LT_HEADS;                                 // [4][32]
   uint64_t* bars = reinterpret_cast<uint64_t*>(s_red + 4 * LT_HEADS);
-  uint64_t *full = bars, *empty = bars + LT_PAIRS, *x_full = bars + 2 * LT_PAIRS, *x_empty = x_full + 2;
+  uint64_t *full = bars, *empty = bars + LT_MAX_RING, *x_full = bars + 2 * LT_MAX_RING, *x_empty = x_full + 2;
   uint64_t *s_full = x_full + 4, *p_ready = x_full + 6, *o_done = x_full + 7;      // o_done: O^T complete up to a tile
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(x_full + 8);
   volatile int* s_abort = reinterpret_cast<volatile int*>(tmem_slot + 1);
@@ -95,7 +108,7 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm, const LatentAttn
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   pdl_launch_dependents();
   if (tid == 0) {
-    for (int i = 0; i < LT_PAIRS; ++i) {
+    for (int i = 0; i < w.ring; ++i) {
       mbar_init(&full[i], 1);
       mbar_init(&empty[i], 1);
     }
@@ -111,27 +124,27 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm, const LatentAttn
     tma_prefetch_desc(&tm);
   }
   if (warp == 1) {
-    tmem_alloc(tmem_slot, LT_TMEM);
+    tmem_alloc(tmem_slot, uint32_t(w.tmem));
     tmem_relinquish();
   }
   pdl_wait();
   asm volatile("fence.proxy.async.global;" ::: "memory");          // rows were written with ordinary stores
   const int ctx = min(p.row_ctx[t], p.max_blocks * p.block_size);
   const int b = p.row_seq != nullptr ? p.row_seq[t] : t;
-  const int tiles = (ctx + LT_ROWS - 1) / LT_ROWS;
-  const int per = (tiles + p.splits - 1) / p.splits;
-  const int tile0 = split * per, n_tiles = max(0, min(tiles, tile0 + per) - tile0);
+  const int first = p.window > 0 ? max(0, ctx - p.window) : 0;     // first visible row
+  const int tiles = (ctx + LT_ROWS - 1) / LT_ROWS, start = first / LT_ROWS;
+  const int per = (tiles - start + p.splits - 1) / p.splits;
+  const int tile0 = start + split * per, n_tiles = max(0, min(tiles, tile0 + per) - tile0);
   const int* bt = p.block_tables + (long long)b * p.max_blocks;
-  const int w = p.rank + p.R, subs = pairs * 2 + extra;
 
   {                                                                // Q, zero-padded to whole sub-tiles and head rows
-    const uint4* q = reinterpret_cast<const uint4*>(reinterpret_cast<const bf16*>(p.q_abs) + ((long long)t * p.H + h0) * w);
+    const uint4* q = reinterpret_cast<const uint4*>(reinterpret_cast<const bf16*>(p.q) + ((long long)t * p.H + h0) * p.K);
     uint4 v[6];
     for (int ch = lane; ch < subs * 8; ch += 32) {
 #pragma unroll
       for (int i = 0; i < 6; ++i) {
         const int r = warp + i * (LT_THREADS / 32);
-        v[i] = r < LT_HEADS && h0 + r < p.H && ch * 8 < w ? __ldcg(q + (long long)r * (w / 8) + ch) : make_uint4(0, 0, 0, 0);
+        v[i] = r < LT_HEADS && h0 + r < p.H && ch * 8 < p.K ? __ldcg(q + (long long)r * (p.K / 8) + ch) : make_uint4(0, 0, 0, 0);
       }
 #pragma unroll
       for (int i = 0; i < 6; ++i) {
@@ -141,8 +154,8 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm, const LatentAttn
       }
     }
   }
-  if (n_tiles <= LT_PAIRS)                                         // boxes past the context are never loaded: keep it finite
-    for (int i = tid; i < (LT_PAIRS * 2 + 2) * LT_SUB / 16; i += LT_THREADS)
+  if (n_tiles <= LT_MAX_RING)                                      // boxes past the context are never loaded: keep it finite
+    for (int i = tid; i < (w.ring * 2 + (w.extra ? 2 : 0)) * LT_SUB / 16; i += LT_THREADS)
       reinterpret_cast<uint4*>(s_kv)[i] = make_uint4(0, 0, 0, 0);
   fence_proxy_async();
   tc_fence_before();
@@ -189,21 +202,22 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm, const LatentAttn
           for (int pc = 0; pc < pieces; ++pc)
             lt_load(dst + pc * box_rows * 128, &tm, bar, col, reinterpret_cast<volatile int*>(s_at)[pc], el);
         };
-        for (int i = 0; i < pairs; ++i) {
+        for (int i = 0; i < w.pairs; ++i) {
+          const int col = w.shared || i < w.keys ? i * 128 : p.v_col + (i - w.keys) * 128;
           if (!__all_sync(0xffffffffu, mbar_wait(&empty[slot], phase, p.status, ST_TIMEOUT_EMPTY))) {
             if (lane == 0) *s_abort = 1;
             ok = false;
             break;
           }
           lt_expect(&full[slot], 2 * bytes, el);
-          load(s_kv + slot * 2 * LT_SUB, &full[slot], i * 128);
-          load(s_kv + slot * 2 * LT_SUB + LT_SUB, &full[slot], i * 128 + 64);
-          if (++slot == LT_PAIRS) {
+          load(s_kv + slot * 2 * LT_SUB, &full[slot], col);
+          load(s_kv + slot * 2 * LT_SUB + LT_SUB, &full[slot], col + 64);
+          if (++slot == w.ring) {
             slot = 0;
             phase ^= 1;
           }
         }
-        if (extra && ok) {
+        if (w.extra && ok) {
           const int x = j & 1;
           if (!__all_sync(0xffffffffu, mbar_wait(&x_empty[x], (uint32_t(j >> 1) & 1u) ^ 1u, p.status, ST_TIMEOUT_EMPTY))) {
             if (lane == 0) *s_abort = 1;
@@ -211,7 +225,7 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm, const LatentAttn
             break;
           }
           lt_expect(&x_full[x], bytes, el);
-          load(s_x + x * LT_SUB, &x_full[x], pairs * 128);
+          load(s_x + x * LT_SUB, &x_full[x], w.keys * 128);
         }
       }
     }
@@ -221,12 +235,20 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm, const LatentAttn
     {
       constexpr uint32_t idesc_s = make_idesc_bf16(128, LT_HEADS, false, false);
       constexpr uint32_t idesc_o = make_idesc_bf16(128, LT_HEADS, true, false);      // A (rows^T) is MN-major
-      const int ksteps = (p.row_width + 15) / 16;
+      const int ksteps = (p.K + 15) / 16;
       auto wait = [](uint64_t* bar, uint32_t parity, uint32_t* status, uint32_t code) {
         return __all_sync(0xffffffffu, mbar_wait(bar, parity, status, code)) != 0;
       };
-      int slot = 0, sl = 0;                                        // next pair of O^T and of S^T
-      uint32_t ph = 0;
+      int slot = 0, sl = 0;                                        // next pair of O^T and of S^T, their phases
+      uint32_t pho = 0, ph = 0;
+      auto skip = [&](int& at, uint32_t& phase, int n) {
+        at += n;
+        while (at >= w.ring) {
+          at -= w.ring;
+          phase ^= 1;
+        }
+      };
+      skip(slot, pho, w.pairs - w.values);
       // descriptors by addition on their address field (16-byte units)
       const uint64_t d_rows = lt_sdesc(smem_u32(s_kv), 16, 1024), d_x = lt_sdesc(smem_u32(s_x), 16, 1024);
       const uint64_t d_cols = lt_sdesc(smem_u32(s_kv), LT_SUB, 1024);
@@ -241,42 +263,49 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm, const LatentAttn
       };
       auto issue_s = [&](int j) {
         const int x = j & 1;
-        for (int i = 0; i < pairs; ++i) {
+        for (int i = 0; i < w.keys; ++i) {
           if (!wait(&full[sl], ph, p.status, ST_TIMEOUT_FULL)) return false;
           tc_fence_after();
           const uint64_t da = d_rows + uint64_t(sl * (2 * LT_SUB >> 4));
           scores(tmem + LT_HEADS * uint32_t(x), da, i * 2);
           scores(tmem + LT_HEADS * uint32_t(x), da + uint64_t(LT_SUB >> 4), i * 2 + 1);
-          if (++sl == LT_PAIRS) {
-            sl = 0;
-            ph ^= 1;
-          }
+          if (!w.shared) lt_commit(&empty[sl], el);
+          skip(sl, ph, 1);
         }
-        if (extra) {
+        skip(sl, ph, w.pairs - w.keys);
+        if (w.extra) {
           if (!wait(&x_full[x], uint32_t(j >> 1) & 1u, p.status, ST_TIMEOUT_FULL)) return false;
           tc_fence_after();
-          scores(tmem + LT_HEADS * uint32_t(x), d_x + uint64_t(x * (LT_SUB >> 4)), pairs * 2);
+          scores(tmem + LT_HEADS * uint32_t(x), d_x + uint64_t(x * (LT_SUB >> 4)), w.keys * 2);
         }
         lt_commit(&s_full[x], el);
-        if (extra) lt_commit(&x_empty[x], el);
+        if (w.extra) lt_commit(&x_empty[x], el);
         return true;
       };
       bool ok = n_tiles == 0 || issue_s(0);
       for (int j = 0; j < n_tiles && ok; ++j) {
-        if (j + 1 < n_tiles) ok = issue_s(j + 1);
+        if (w.ahead && j + 1 < n_tiles) ok = issue_s(j + 1);
         ok = ok && wait(p_ready, uint32_t(j) & 1u, p.status, ST_TIMEOUT_FULL);
         if (!ok) break;
         tc_fence_after();
-        for (int i = 0; i < pairs; ++i) {
+        for (int i = 0; i < w.values && ok; ++i) {
+          if (!w.shared) {
+            ok = wait(&full[slot], pho, p.status, ST_TIMEOUT_FULL);
+            if (!ok) break;
+            tc_fence_after();
+          }
           const uint64_t dv = d_cols + uint64_t(slot * (2 * LT_SUB >> 4)), dp = d_p + uint64_t((j & 1) * (LT_QSUB >> 4));
           const uint32_t tm_o = tmem + LT_HEADS * uint32_t(2 + i);
 #pragma unroll
           for (int kk = 0; kk < LT_ROWS / 16; ++kk)
             lt_mma(tm_o, dv + uint64_t(kk * 128), dp + uint64_t(kk * 2), idesc_o, (j > 0 || kk > 0) ? 1u : 0u, el);
           lt_commit(&empty[slot], el);
-          if (++slot == LT_PAIRS) slot = 0;
+          skip(slot, pho, 1);
         }
+        skip(slot, pho, w.pairs - w.values);
+        if (!ok) break;
         lt_commit(o_done, el);
+        if (!w.ahead && j + 1 < n_tiles) ok = issue_s(j + 1);
       }
       if (!ok && lane == 0) *s_abort = 1;
     }
@@ -311,9 +340,10 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm, const LatentAttn
       uint32_t s[LT_HEADS];
       tmem_ld_32x32(tmem + lanes + LT_HEADS * uint32_t(j & 1), s);
       tmem_ld_wait();
-      const bool valid = mine && (tile0 + j) * LT_ROWS + row < ctx;
+      const int at = (tile0 + j) * LT_ROWS + row;
+      const bool valid = mine && at < ctx && at >= first;
       if (j == 0) {
-        if (row == 0)
+        if (row == max(0, first - tile0 * LT_ROWS))
 #pragma unroll
           for (int h = 0; h < LT_HEADS; ++h) s_ref[h] = __uint_as_float(s[h]) * scale_log2;
         sync_or(false);
@@ -350,7 +380,7 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm, const LatentAttn
         if (j > 0 && ok) ok = mbar_wait(o_done, uint32_t(j - 1) & 1u, p.status, ST_TIMEOUT_ACC_FULL);
         tc_fence_after();
         if (j > 0)
-          for (int i = 0; i < pairs; ++i) {
+          for (int i = 0; i < w.values; ++i) {
             uint32_t r[32];
             tmem_ld_32x32(tmem + lanes + LT_HEADS * uint32_t(2 + i), r);
             tmem_ld_wait();
@@ -376,13 +406,13 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm, const LatentAttn
           *reinterpret_cast<bf16*>(prow + (j & 1) * LT_QSUB + h * 128 + ((chunk ^ (h & 7)) << 4)) = __float2bfloat16(e);
         }
       }
+      // the last two phases of o_done one by one, a parity cannot tell a phase from the one two before it: the scores of the
+      // last tile only say that the third-last product is done, and the last one cannot be before this arrival
+      if (j == n_tiles - 1 && j > 0 && ok) ok = mbar_wait(o_done, uint32_t(j - 1) & 1u, p.status, ST_TIMEOUT_ACC_FULL);
       fence_proxy_async();
       tc_fence_before();
       mbar_arrive(p_ready);
     }
-    // the last two phases one by one: the scores of the last tile only say that the third-last product is done, and a
-    // parity cannot tell a phase from the one two before it
-    if (ok && n_tiles > 1) ok = mbar_wait(o_done, uint32_t(n_tiles - 2) & 1u, p.status, ST_TIMEOUT_ACC_FULL);
     if (ok && n_tiles > 0) ok = mbar_wait(o_done, uint32_t(n_tiles - 1) & 1u, p.status, ST_TIMEOUT_ACC_FULL);
     if (!ok) *s_abort = 1;
     tc_fence_after();
@@ -404,11 +434,21 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm, const LatentAttn
     if (et < LT_HEADS) {
       const float x = s_red[et] + s_red[LT_HEADS + et] + s_red[2 * LT_HEADS + et] + s_red[3 * LT_HEADS + et];
       const bool has = good && x > 0.f;
-      if (p.splits > 1 && h0 + et < p.H)
-        p.part_lse[((long long)t * p.H + h0 + et) * p.splits + split] = has ? s_ref[et] + log2f(x) : -INFINITY;
-      s_red[et] = has ? 1.f / x : 0.f;
+      const int head = h0 + et;
+      if (p.splits > 1 && head < p.H)
+        p.part_lse[((long long)t * p.H + head) * p.splits + split] = has ? s_ref[et] + log2f(x) : -INFINITY;
+      float f = 0.f;
+      if (has) {
+        f = 1.f / x;
+        if (p.splits == 1 && head < p.H) {
+          if (p.sink != nullptr) f = 1.f / (x + exp2f(p.sink[head] * LT_LOG2E - s_ref[et]));
+          if (p.head_gate != nullptr) f *= p.head_gate[(long long)t * p.H + head];
+        }
+      }
+      s_red[et] = f;
     }
-    for (int i = 0; i < pairs; ++i) {
+    const int heads_per = p.H / p.v_heads;
+    for (int i = 0; i < w.values; ++i) {
       sync_or(false);                                              // s_red is there, the block before is written
       if (good) {
         uint32_t r[32];
@@ -418,17 +458,20 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm, const LatentAttn
         for (int h = 0; h < LT_HEADS; ++h) s_o[h * 132 + row] = __uint_as_float(r[h]);
       }
       sync_or(false);
-      const int c = i * 128 + (et & 31) * 4;                       // a warp writes 128 latents of a head
-      if (c < p.rank)
+      const int c = i * 128 + (et & 31) * 4;                       // a warp writes 128 columns of a head
+      const int vh = c / p.V;                                      // the value head they belong to (V is a multiple of 4)
+      if (vh < p.v_heads)
         for (int h = et >> 5; h < LT_HEADS && h0 + h < p.H; h += 4) {
+          if ((h0 + h) / heads_per != vh) continue;
           const float inv = s_red[h];
           float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
           if (inv != 0.f) x = *reinterpret_cast<const float4*>(s_o + h * 132 + (et & 31) * 4);
           const long long at = (long long)t * p.H + h0 + h;
+          const int cv = c - vh * p.V;
           if (p.splits == 1)
-            store4(reinterpret_cast<bf16*>(p.o_lat) + at * p.rank + c, x.x * inv, x.y * inv, x.z * inv, x.w * inv);
+            store4(reinterpret_cast<bf16*>(p.out) + t * p.ld_out + (h0 + h) * p.V + cv, x.x * inv, x.y * inv, x.z * inv, x.w * inv);
           else
-            store4(p.part_o + (at * p.splits + split) * p.rank + c, x.x * inv, x.y * inv, x.z * inv, x.w * inv);
+            store4(p.part_o + (at * p.splits + split) * p.V + cv, x.x * inv, x.y * inv, x.z * inv, x.w * inv);
         }
     }
   }
@@ -436,7 +479,7 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm, const LatentAttn
   __syncthreads();
   if (warp == 1) {
     tc_fence_after();
-    tmem_dealloc(tmem, LT_TMEM);
+    tmem_dealloc(tmem, uint32_t(w.tmem));
   }
 }
 
@@ -446,30 +489,55 @@ static int lt_box_rows(int block_size) {
   return box;
 }
 
-bool latent_decode_tc_supported(const LatentAttn& p) {
-  const int pairs = (p.rank + 127) / 128;
-  return p.rank % 8 == 0 && (p.rank + p.R) % 8 == 0 && pairs <= 4 && p.row_width - pairs * 128 <= 64 &&
-         lt_box_rows(p.block_size) >= 8;
+static int lt_smem(const LtTile& w) {
+  return w.ring * 2 * LT_SUB + (w.extra ? 2 * LT_SUB : 0) + (w.keys * 2 + w.extra + 2) * LT_QSUB + 5 * LT_HEADS * 4 +
+         (2 * LT_MAX_RING + 8) * 8 + 16 + LT_ROWS / 2 + 1024;
+}
+// how a tile lies in the ring; ring 0: these sizes do not fit
+static LtTile lt_tile(const RowAttn& p) {
+  LtTile w{};
+  const int vw = p.v_heads * p.V;
+  w.shared = p.v_col == 0;
+  w.values = (vw + 127) / 128;
+  if (w.shared) {
+    w.pairs = w.keys = w.values;
+    w.extra = p.K > w.keys * 128 ? 1 : 0;
+    if (p.K - w.keys * 128 > 64 || vw > p.K) return w;
+  } else {
+    w.keys = (p.K + 127) / 128;
+    w.pairs = w.keys + w.values;
+  }
+  if (w.values > LT_MAX_BLOCKS) return w;
+  w.tmem = w.values <= 6 ? 256 : 512;
+  w.ring = w.shared ? 10 : LT_MAX_RING;
+  while (w.ring > 0 && lt_smem(w) > 227 * 1024) --w.ring;
+  if (w.ring < 4 || (w.shared && w.ring < 2 * w.pairs)) w.ring = 0;
+  w.ahead = w.shared || w.keys + w.values <= w.ring ? 1 : 0;
+  return w;
 }
 
-int latent_decode_tc_splits(const LatentAttn& p, int max_ctx, int num_sms) {
+bool latent_decode_tc_supported(const RowAttn& p) {
+  return p.V % 8 == 0 && p.K % 8 == 0 && p.v_col % 8 == 0 && p.row_width % 8 == 0 && p.ld_out % 4 == 0 && p.H % p.v_heads == 0 &&
+         lt_box_rows(p.block_size) >= 8 && lt_tile(p).ring > 0;
+}
+
+int latent_decode_tc_splits(const RowAttn& p, int max_ctx, int num_sms) {
   const int ctas = p.T * ((p.H + LT_HEADS - 1) / LT_HEADS);
   if (ctas * 3 > num_sms * 2) return 1;                            // nearly a full wave already
   return std::max(1, std::min({num_sms / std::max(1, ctas), max_ctx / (2 * LT_ROWS), 32}));
 }
 
-void launch_latent_decode_tc(const LatentAttn& p, cudaStream_t s) {
+void launch_latent_decode_tc(const RowAttn& p, cudaStream_t s) {
   if (p.T == 0) return;
-  const int box = lt_box_rows(p.block_size), pairs = (p.rank + 127) / 128, extra = p.row_width > pairs * 128 ? 1 : 0;
+  const LtTile w = lt_tile(p);
+  const int box = lt_box_rows(p.block_size), smem = lt_smem(w);
+  if (w.ring == 0) throw std::runtime_error("attention over shared rows (tcgen05): unsupported sizes");
   const CUtensorMap tm = make_tmap_bf16_2d(p.pool, (uint64_t)p.num_blocks * p.block_size, p.row_width, p.row_width, box, 64);
-  constexpr int smem = (LT_PAIRS * 2 + 2) * LT_SUB + (LT_MAX_SUBS + 2) * LT_QSUB + 5 * LT_HEADS * 4 +
-                       (2 * LT_PAIRS + 8) * 8 + 16 + LT_ROWS / 2 + 1024;
-  static_assert(smem <= 227 * 1024, "shared memory of a CTA");
   cudaFuncSetAttribute(latent_decode_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
   launch_pdl(PDL_DECODE_ATTN, latent_decode_tc_kernel, dim3(p.T, (p.H + LT_HEADS - 1) / LT_HEADS, p.splits),
-             dim3(LT_THREADS), smem, s, tm, p, box, pairs, extra, p.scale * 1.4426950408889634f);
+             dim3(LT_THREADS), smem, s, tm, p, w, box, p.scale * LT_LOG2E);
   const cudaError_t e = cudaGetLastError();
-  if (e != cudaSuccess) throw std::runtime_error(std::string("latent decode (tcgen05): ") + cudaGetErrorString(e));
+  if (e != cudaSuccess) throw std::runtime_error(std::string("attention over shared rows (tcgen05): ") + cudaGetErrorString(e));
 }
 
 }  // namespace fc

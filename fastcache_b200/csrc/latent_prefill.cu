@@ -1,17 +1,21 @@
-// Causal prefill attention of latent layers on tcgen05: per-head keys and values expanded from the cache rows of each
-// request (contiguous, see launch_gather_rows), key = [dim unrotated | rot shared by all heads], value of another size.
+// Causal prefill attention on tcgen05 over the gathered cache rows of each request (contiguous, see launch_gather_rows): keys
+// of D columns per head and R columns that all heads share, values of another size.  Latent attention: D and values expanded
+// from the rows, R the rotated part.  Heads that mix their scores: D = 0, R the keys of all key heads side by side, values of
+// a group of heads.  Options: sliding window (key tiles before a query tile's window are neither loaded nor multiplied), sink.
 //
 // One CTA owns 128 query rows of one head and walks the visible keys in tiles of 128.  Even and odd key tiles have
 // separate score and output accumulators in tensor memory and separate softmax warps, so that one parity's matrices
 // run while the other's softmax does; the two partial results are merged at the end:
 //     S_0 [0,128)  S_1 [128,256)  O_0 [256,384)  O_1 [384,512)
-//   warp 0       TMA: the Q tile once, then K (unrotated sub-tiles + rotated sub-tile) and V tiles; stage = parity.
-//                Three-dimensional boxes (column, head, row) zero-fill the columns past a head's width
+//   warp 0       TMA: the Q tile once, K in sub-tiles of 64 columns through a ring, V tiles.  Queries of more than eight
+//                sub-tiles do not stay: every slot of the ring takes a sub-tile of K and of Q.  Three-dimensional boxes
+//                (column, head, row) zero-fill the columns past a head's width
 //   warp 1       tcgen05.mma issuer: S_x = Q K(j)^T, then O_x += P_x V(j) with P_x in tensor memory over S_x
 //   warps 2-5    softmax of even tiles, warps 6-9 of odd tiles: one query row per thread, reference maximum as in
 //                attn_prefill_tc2.cu (O is rescaled only when a row outgrows its reference by 2^8)
-// The epilogue multiplies with sigmoid(gate) and writes bf16.
+// The epilogue multiplies with the output gate, if there is one, and writes bf16.
 #include <cuda.h>
+#include <algorithm>
 #include <stdexcept>
 #include <string>
 
@@ -24,6 +28,9 @@ using bf16 = __nv_bfloat16;
 constexpr int LP_BM = 128, LP_BN = 128, LP_THREADS = 320;
 constexpr int LP_SUB = 128 * 128;                 // bytes of a [128 rows x 64 columns] sub-tile
 constexpr float LP_RESCALE = 8.f;                 // log2 units
+constexpr int LP_SLOTS = 14;                      // sub-tiles of shared memory: Q, K ring, V
+constexpr int LP_RING = 8;                        // most slots of the K ring
+constexpr float LP_LOG2E = 1.4426950408889634f;
 
 __device__ __forceinline__ uint64_t lp_sdesc(uint32_t addr, uint32_t lbo_bytes, uint32_t sbo_bytes) {
   uint64_t d = 0;
@@ -41,30 +48,34 @@ struct LpMaps {
 struct LpParams {
   const int *cu_q, *cu_kv;
   const bf16* gate;
+  const float *head_gate, *sink;
   bf16* out;
   long long ld_gate, ld_out;
-  int D, R, V;
+  int D, R, V, heads_per_value, window;
+  int nd, nr;                                     // sub-tiles of the keys' own and shared columns
+  int ring, v_stages;
   float scale_log2;
   uint32_t* status;
 };
 
-// ND / NV: 64-column sub-tiles of the unrotated key part and of the values
-template <int ND, int NV>
+// NV: 64-column sub-tiles of the values; STREAM_Q: Q comes with K through the ring
+template <int NV, bool STREAM_Q>
 __global__ void __launch_bounds__(LP_THREADS, 1)
 latent_prefill_kernel(const __grid_constant__ LpMaps tm, const LpParams p) {
-  constexpr int NQ = ND + 1;                       // sub-tiles of a Q or K tile: unrotated, then rotated
-  constexpr int K_BYTES = NQ * LP_SUB, V_BYTES = NV * LP_SUB;
+  constexpr int SLOT = STREAM_Q ? 2 * LP_SUB : LP_SUB;   // K sub-tile, then Q's
+  constexpr int V_BYTES = NV * LP_SUB;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
-  uint8_t* s_q = smem;
-  uint8_t* s_k = s_q + K_BYTES;                    // 2 stages
-  uint8_t* s_v = s_k + 2 * K_BYTES;                // 2 stages
-  uint64_t* bars = reinterpret_cast<uint64_t*>(s_v + 2 * V_BYTES);
-  uint64_t *q_full = bars, *k_full = bars + 1, *k_empty = bars + 3, *v_full = bars + 5, *v_empty = bars + 7;
-  uint64_t *s_full = bars + 9, *p_ready = bars + 11, *o_done = bars + 13;
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 15);
+  const int nq = p.nd + p.nr;                      // sub-tiles of a Q or K tile
+  uint8_t* s_k = smem;                             // ring
+  uint8_t* s_v = s_k + p.ring * SLOT;              // v_stages
+  uint8_t* s_q = s_v + p.v_stages * V_BYTES;
+  uint64_t* bars = reinterpret_cast<uint64_t*>(smem + LP_SLOTS * LP_SUB);
+  uint64_t *q_full = bars, *k_full = bars + 1, *k_empty = k_full + LP_RING, *v_full = k_empty + LP_RING, *v_empty = v_full + 2;
+  uint64_t *s_full = v_empty + 2, *p_ready = s_full + 2, *o_done = p_ready + 2;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(o_done + 2);
   volatile int* s_abort = reinterpret_cast<volatile int*>(tmem_slot + 1);
-  float* s_ml = reinterpret_cast<float*>(bars + 16);   // [2][128] reference maximum and sum of the odd tiles
+  float* s_ml = reinterpret_cast<float*>(o_done + 3);   // [2][128] reference maximum and sum of the odd tiles
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int seq = blockIdx.z, h = blockIdx.y;
@@ -74,13 +85,17 @@ latent_prefill_kernel(const __grid_constant__ LpMaps tm, const LpParams p) {
   const int kv_begin = p.cu_kv[seq], kv_len = p.cu_kv[seq + 1] - kv_begin;
   const int offset = kv_len - q_len;
   const int kv_end = min(kv_len, offset + q0 + LP_BM);
-  const int n_tiles = (kv_end + LP_BN - 1) / LP_BN;
+  const int first_key = p.window > 0 ? max(0, offset + q0 - p.window + 1) : 0;      // of the tile's first row
+  const int tile0 = first_key / LP_BN;
+  const int n_tiles = (kv_end + LP_BN - 1) / LP_BN - tile0;
 
   if (threadIdx.x == 0) {
     mbar_init(q_full, 1);
-    for (int s = 0; s < 2; ++s) {
+    for (int s = 0; s < p.ring; ++s) {
       mbar_init(&k_full[s], 1);
       mbar_init(&k_empty[s], 1);
+    }
+    for (int s = 0; s < 2; ++s) {
       mbar_init(&v_full[s], 1);
       mbar_init(&v_empty[s], 1);
       mbar_init(&s_full[s], 1);
@@ -102,74 +117,86 @@ latent_prefill_kernel(const __grid_constant__ LpMaps tm, const LpParams p) {
   if (warp == 0) {
     // ------------------------------------------------------------------ TMA loader
     if (lane == 0) {
-      mbar_expect_tx(q_full, K_BYTES);
-#pragma unroll
-      for (int s = 0; s < ND; ++s) tma_load_3d(s_q + s * LP_SUB, &tm.qn, q_full, s * 64, h, q_begin + q0);
-      tma_load_3d(s_q + ND * LP_SUB, &tm.qr, q_full, 0, h, q_begin + q0);
-      for (int j = 0; j < n_tiles && !*s_abort; ++j) {
-        const int st = j & 1;
-        const uint32_t ph = ((j >> 1) & 1) ^ 1;
-        const int row = kv_begin + j * LP_BN;
-        if (!mbar_wait(&k_empty[st], ph, p.status, ST_TIMEOUT_EMPTY)) {
-          *s_abort = 1;
-          break;
+      auto load_q = [&](uint8_t* dst, uint64_t* bar, int i) {
+        if (i < p.nd) tma_load_3d(dst, &tm.qn, bar, i * 64, h, q_begin + q0);
+        else tma_load_3d(dst, &tm.qr, bar, (i - p.nd) * 64, h, q_begin + q0);
+      };
+      if (!STREAM_Q) {
+        mbar_expect_tx(q_full, uint32_t(nq) * LP_SUB);
+        for (int i = 0; i < nq; ++i) load_q(s_q + i * LP_SUB, q_full, i);
+      }
+      int slot = 0;
+      uint32_t phase = 1;
+      bool ok = true;
+      for (int j = 0; j < n_tiles && ok && !*s_abort; ++j) {
+        const int row = kv_begin + (tile0 + j) * LP_BN;
+        for (int i = 0; i < nq; ++i) {
+          ok = mbar_wait(&k_empty[slot], phase, p.status, ST_TIMEOUT_EMPTY);
+          if (!ok) break;
+          uint8_t* dk = s_k + slot * SLOT;
+          mbar_expect_tx(&k_full[slot], SLOT);
+          if (i < p.nd) tma_load_3d(dk, &tm.kn, &k_full[slot], i * 64, h, row);
+          else tma_load_2d(dk, &tm.kr, &k_full[slot], (i - p.nd) * 64, row);
+          if (STREAM_Q) load_q(dk + LP_SUB, &k_full[slot], i);
+          if (++slot == p.ring) {
+            slot = 0;
+            phase ^= 1;
+          }
         }
-        mbar_expect_tx(&k_full[st], K_BYTES);
-        uint8_t* dk = s_k + st * K_BYTES;
-#pragma unroll
-        for (int s = 0; s < ND; ++s) tma_load_3d(dk + s * LP_SUB, &tm.kn, &k_full[st], s * 64, h, row);
-        tma_load_2d(dk + ND * LP_SUB, &tm.kr, &k_full[st], 0, row);
-        if (!mbar_wait(&v_empty[st], ph, p.status, ST_TIMEOUT_EMPTY)) {
-          *s_abort = 1;
-          break;
-        }
+        if (!ok) break;
+        const int st = p.v_stages == 2 ? j & 1 : 0;
+        const uint32_t use = uint32_t(p.v_stages == 2 ? j >> 1 : j) & 1u;
+        ok = mbar_wait(&v_empty[st], use ^ 1u, p.status, ST_TIMEOUT_EMPTY);
+        if (!ok) break;
         mbar_expect_tx(&v_full[st], V_BYTES);
 #pragma unroll
-        for (int s = 0; s < NV; ++s) tma_load_3d(s_v + st * V_BYTES + s * LP_SUB, &tm.v, &v_full[st], s * 64, h, row);
+        for (int s = 0; s < NV; ++s) tma_load_3d(s_v + st * V_BYTES + s * LP_SUB, &tm.v, &v_full[st], s * 64, h / p.heads_per_value, row);
       }
+      if (!ok) *s_abort = 1;
     }
   } else if (warp == 1) {
     // ------------------------------------------------------------------ MMA issuer
     if (lane == 0) {
       constexpr uint32_t idesc_s = make_idesc_bf16(128, 128, false, false);
       constexpr uint32_t idesc_o = make_idesc_bf16(128, NV * 64, false, true);     // B (= V) is MN-major
-      const int steps_d = (p.D + 15) / 16, steps_r = (p.R + 15) / 16;
+      int slot = 0;
+      uint32_t phase = 0;
       auto issue_s = [&](int j) {
         const int x = j & 1;
-        if (!mbar_wait(&k_full[x], uint32_t(j >> 1) & 1u, p.status, ST_TIMEOUT_FULL)) return false;
-        tc_fence_after();
-        const uint32_t qa = smem_u32(s_q), ka = smem_u32(s_k + x * K_BYTES);
-        for (int kk = 0; kk < steps_d; ++kk) {
-          const uint32_t off = uint32_t(kk >> 2) * LP_SUB + uint32_t(kk & 3) * 32;
-          tc_mma_f16(tmem_base + uint32_t(x * 128), lp_sdesc(qa + off, 16, 1024), lp_sdesc(ka + off, 16, 1024), idesc_s,
-                     kk > 0 ? 1u : 0u);
-        }
-        for (int kk = 0; kk < steps_r; ++kk) {
-          const uint32_t off = uint32_t(ND) * LP_SUB + uint32_t(kk) * 32;
-          tc_mma_f16(tmem_base + uint32_t(x * 128), lp_sdesc(qa + off, 16, 1024), lp_sdesc(ka + off, 16, 1024), idesc_s,
-                     1u);
+        for (int i = 0; i < nq; ++i) {
+          if (!mbar_wait(&k_full[slot], phase, p.status, ST_TIMEOUT_FULL)) return false;
+          tc_fence_after();
+          const uint32_t ka = smem_u32(s_k + slot * SLOT), qa = STREAM_Q ? ka + LP_SUB : smem_u32(s_q + i * LP_SUB);
+          const int left = i < p.nd ? p.D - i * 64 : p.R - (i - p.nd) * 64, steps = min(4, (left + 15) / 16);
+          for (int kk = 0; kk < steps; ++kk)
+            tc_mma_f16(tmem_base + uint32_t(x * 128), lp_sdesc(qa + uint32_t(kk) * 32, 16, 1024),
+                       lp_sdesc(ka + uint32_t(kk) * 32, 16, 1024), idesc_s, (i > 0 || kk > 0) ? 1u : 0u);
+          tc_commit(&k_empty[slot]);
+          if (++slot == p.ring) {
+            slot = 0;
+            phase ^= 1;
+          }
         }
         tc_commit(&s_full[x]);
-        tc_commit(&k_empty[x]);
         return true;
       };
-      bool ok = mbar_wait(q_full, 0, p.status, ST_TIMEOUT_FULL);
+      bool ok = STREAM_Q || mbar_wait(q_full, 0, p.status, ST_TIMEOUT_FULL);
       if (ok) ok = issue_s(0);
       if (ok && n_tiles > 1) ok = issue_s(1);
       for (int j = 0; j < n_tiles && ok; ++j) {
         const int x = j & 1;
-        const uint32_t use = uint32_t(j >> 1) & 1u;
-        ok = mbar_wait(&p_ready[x], use, p.status, ST_TIMEOUT_FULL) &&
-             mbar_wait(&v_full[x], use, p.status, ST_TIMEOUT_FULL);
+        const int st = p.v_stages == 2 ? x : 0;
+        ok = mbar_wait(&p_ready[x], uint32_t(j >> 1) & 1u, p.status, ST_TIMEOUT_FULL) &&
+             mbar_wait(&v_full[st], uint32_t(p.v_stages == 2 ? j >> 1 : j) & 1u, p.status, ST_TIMEOUT_FULL);
         if (!ok) break;
         tc_fence_after();
-        const uint32_t va = smem_u32(s_v + x * V_BYTES);
+        const uint32_t va = smem_u32(s_v + st * V_BYTES);
 #pragma unroll
         for (int kk = 0; kk < 8; ++kk)
           tc_mma_f16_ts(tmem_base + 256u + uint32_t(x * 128), tmem_base + uint32_t(x * 128) + uint32_t(kk * 8),
                         lp_sdesc(va + uint32_t(kk) * 2048, LP_SUB, 1024), idesc_o, (j > 1 || kk > 0) ? 1u : 0u);
         tc_commit(&o_done[x]);
-        tc_commit(&v_empty[x]);
+        tc_commit(&v_empty[st]);
         if (j + 2 < n_tiles) ok = issue_s(j + 2);
       }
       if (!ok) *s_abort = 1;
@@ -198,13 +225,19 @@ latent_prefill_kernel(const __grid_constant__ LpMaps tm, const LpParams p) {
 #pragma unroll
       for (int c = 0; c < 4; ++c) tmem_ld_32x32(ts + uint32_t(c * 32), *reinterpret_cast<uint32_t(*)[32]>(&s[c * 32]));
       tmem_ld_wait();
-      const int col0 = j * LP_BN;
+      const int col0 = (tile0 + j) * LP_BN;
       if ((col0 + LP_BN - 1 > offset + q0) || (col0 + LP_BN > kv_end)) {
 #pragma unroll
         for (int t = 0; t < 128; ++t) {
           const int col = col0 + t;
           if (col > qpos || col >= kv_end) s[t] = 0xff800000u;          // -inf
         }
+      }
+      if (p.window > 0 && col0 <= offset + q0 + LP_BM - 1 - p.window) {  // the last row's window starts behind col0
+        const int hidden = qpos - p.window - col0;
+#pragma unroll
+        for (int t = 0; t < 128; ++t)
+          if (t <= hidden) s[t] = 0xff800000u;
       }
       float mx = -INFINITY;
 #pragma unroll
@@ -259,7 +292,7 @@ latent_prefill_kernel(const __grid_constant__ LpMaps tm, const LpParams p) {
     tc_fence_after();
     // every matrix of both parities is done after this barrier: the K stages are free for the odd tiles' result
     asm volatile("bar.sync 1, 256;" ::: "memory");
-    float* s_o = reinterpret_cast<float*>(s_k);                  // [NV * 64 columns][128 rows]
+    float* s_o = reinterpret_cast<float*>(s_k);                  // [NV * 64 columns][128 rows]: two slots per 64 columns
     const bool two = n_tiles > 1 && !*s_abort;
     if (x == 1) {
       if (two) {
@@ -278,18 +311,21 @@ latent_prefill_kernel(const __grid_constant__ LpMaps tm, const LpParams p) {
     } else {
       asm volatile("bar.sync 1, 256;" ::: "memory");
       if (ok) {
-        float w0 = 1.f, w1 = 0.f;
+        float w0 = 1.f, w1 = 0.f, mm = m_ref;                    // a row sees itself: one of the maxima is finite
         if (two) {
-          const float m1 = s_ml[row], mm = fmaxf(m_ref, m1);
-          w0 = exp2f(m_ref - mm);                                // key 0 is visible to every row: m_ref is finite
+          const float m1 = s_ml[row];
+          mm = fmaxf(m_ref, m1);
+          w0 = m_ref == -INFINITY ? 0.f : exp2f(m_ref - mm);
           w1 = m1 == -INFINITY ? 0.f : exp2f(m1 - mm);
           l = l * w0 + s_ml[128 + row] * w1;
         }
-        const float inv = l > 0.f ? 1.f / l : 0.f;
+        if (p.sink != nullptr && l > 0.f) l += exp2f(p.sink[h] * LP_LOG2E - mm);
+        float inv = l > 0.f ? 1.f / l : 0.f;
+        if (p.head_gate != nullptr && qrow < q_len) inv *= p.head_gate[(long long)(q_begin + qrow) * gridDim.y + h];
         w0 *= inv;
         w1 *= inv;
         bf16* dst = p.out + (long long)(q_begin + qrow) * p.ld_out + h * p.V;
-        const bf16* gate = p.gate + (long long)(q_begin + qrow) * p.ld_gate + h * p.V;
+        const bf16* gate = p.gate != nullptr ? p.gate + (long long)(q_begin + qrow) * p.ld_gate + h * p.V : nullptr;
 #pragma unroll 1
         for (int c = 0; c < NV * 2; ++c) {
           uint32_t r[32];
@@ -299,7 +335,7 @@ latent_prefill_kernel(const __grid_constant__ LpMaps tm, const LpParams p) {
           for (int q = 0; q < 4; ++q) {
             const int col = c * 32 + q * 8;
             if (qrow >= q_len || col >= p.V) continue;           // V is a multiple of 8
-            const uint4 gu = *reinterpret_cast<const uint4*>(gate + col);
+            const uint4 gu = gate != nullptr ? *reinterpret_cast<const uint4*>(gate + col) : make_uint4(0, 0, 0, 0);
             const uint32_t gw[4] = {gu.x, gu.y, gu.z, gu.w};
             uint32_t ow[4];
 #pragma unroll
@@ -309,8 +345,12 @@ latent_prefill_kernel(const __grid_constant__ LpMaps tm, const LpParams p) {
                 a = fmaf(s_o[(col + 2 * e) * 128 + row], w1, a);
                 b = fmaf(s_o[(col + 2 * e + 1) * 128 + row], w1, b);
               }
-              const float2 g = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&gw[e]));
-              ow[e] = pack_bf16(a * sigmoid_t<bf16>(g.x), b * sigmoid_t<bf16>(g.y));
+              if (gate != nullptr) {
+                const float2 g = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&gw[e]));
+                a *= sigmoid_t<bf16>(g.x);
+                b *= sigmoid_t<bf16>(g.y);
+              }
+              ow[e] = pack_bf16(a, b);
             }
             *reinterpret_cast<uint4*>(dst + col) = make_uint4(ow[0], ow[1], ow[2], ow[3]);
           }
@@ -327,14 +367,16 @@ latent_prefill_kernel(const __grid_constant__ LpMaps tm, const LpParams p) {
 }
 
 bool latent_prefill_supported(const LatentPrefill& p) {
-  return p.D % 8 == 0 && p.D <= 128 && p.R % 8 == 0 && p.R <= 64 && p.V % 8 == 0 && p.V <= 128 && p.rank % 8 == 0 &&
-         p.D > 0 && p.R > 0 && p.V > 0;
+  return p.D % 8 == 0 && p.D <= 128 && p.R % 8 == 0 && p.V % 8 == 0 && p.V <= 128 && p.R > 0 && p.V > 0 && p.D >= 0 &&
+         (p.v_heads == 0 || p.H % p.v_heads == 0);
 }
 
-template <int ND, int NV>
+template <int NV, bool STREAM_Q>
 static void launch_lp(const LpMaps& tm, const LpParams& q, const LatentPrefill& p, cudaStream_t s) {
-  constexpr int smem = 3 * (ND + 1) * LP_SUB + 2 * NV * LP_SUB + 128 + 1024 + 1024;
-  auto kern = latent_prefill_kernel<ND, NV>;
+  // barriers and maxima behind the sub-tiles, then the slack of the alignment
+  constexpr int smem = LP_SLOTS * LP_SUB + (2 * LP_RING + 14) * 8 + 1024 + 1024;
+  static_assert(smem <= 227 * 1024, "shared memory of a CTA");
+  auto kern = latent_prefill_kernel<NV, STREAM_Q>;
   cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
   kern<<<dim3((p.max_q + LP_BM - 1) / LP_BM, p.H, p.B), LP_THREADS, smem, s>>>(tm, q);
 }
@@ -343,30 +385,41 @@ void launch_latent_prefill(const LatentPrefill& p, cudaStream_t s) {
   if (p.T == 0 || p.B == 0 || p.max_q == 0) return;
   LpMaps tm;
   const uint64_t Q = uint64_t(p.D + p.R);
+  const int vh = p.v_heads > 0 ? p.v_heads : p.H;
   const bf16* q = reinterpret_cast<const bf16*>(p.q);
-  tm.qn = make_tmap_bf16_3d(q, p.D, p.H, p.T, Q, p.ld_q, 64, 1, LP_BM);
   tm.qr = make_tmap_bf16_3d(q + p.D, p.R, p.H, p.T, Q, p.ld_q, 64, 1, LP_BM);
-  tm.kn = make_tmap_bf16_3d(p.k, p.D, p.H, p.total_kv, p.D, p.ld_kv, 64, 1, LP_BN);
-  tm.v = make_tmap_bf16_3d(p.v, p.V, p.H, p.total_kv, p.V, p.ld_kv, 64, 1, LP_BN);
   tm.kr = make_tmap_bf16_2d(p.rot, p.total_kv, p.R, p.ld_rot, LP_BN, 64);
+  tm.qn = p.D > 0 ? make_tmap_bf16_3d(q, p.D, p.H, p.T, Q, p.ld_q, 64, 1, LP_BM) : tm.qr;
+  tm.kn = p.D > 0 ? make_tmap_bf16_3d(p.k, p.D, p.H, p.total_kv, p.D, p.ld_k, 64, 1, LP_BN) : tm.kr;
+  tm.v = make_tmap_bf16_3d(p.v, p.V, vh, p.total_kv, p.V, p.ld_v, 64, 1, LP_BN);
   LpParams a;
   a.cu_q = p.cu_q;
   a.cu_kv = p.cu_kv;
   a.gate = reinterpret_cast<const bf16*>(p.gate);
+  a.head_gate = p.head_gate;
+  a.sink = p.sink;
   a.out = reinterpret_cast<bf16*>(p.out);
   a.ld_gate = p.ld_gate;
   a.ld_out = p.ld_out;
   a.D = p.D;
   a.R = p.R;
   a.V = p.V;
-  a.scale_log2 = p.scale * 1.4426950408889634f;
+  a.heads_per_value = p.H / vh;
+  a.window = p.window;
+  a.scale_log2 = p.scale * LP_LOG2E;
   a.status = p.status;
-  if (p.D <= 64 && p.V <= 64) launch_lp<1, 1>(tm, a, p, s);
-  else if (p.D <= 64) launch_lp<1, 2>(tm, a, p, s);
-  else if (p.V <= 64) launch_lp<2, 1>(tm, a, p, s);
-  else launch_lp<2, 2>(tm, a, p, s);
+  a.nd = (p.D + 63) / 64;
+  a.nr = (p.R + 63) / 64;
+  const int nv = p.V <= 64 ? 1 : 2, nq = a.nd + a.nr;
+  const bool stream = nq > 8;
+  // at least four slots for K; two stages of V where they leave that much
+  const int left = LP_SLOTS - (stream ? 0 : nq);
+  a.v_stages = left - 2 * nv >= (stream ? 8 : 4) ? 2 : 1;
+  a.ring = std::min(LP_RING, (left - a.v_stages * nv) / (stream ? 2 : 1));
+  if (nv == 1) stream ? launch_lp<1, true>(tm, a, p, s) : launch_lp<1, false>(tm, a, p, s);
+  else stream ? launch_lp<2, true>(tm, a, p, s) : launch_lp<2, false>(tm, a, p, s);
   const cudaError_t e = cudaGetLastError();
-  if (e != cudaSuccess) throw std::runtime_error(std::string("latent prefill: ") + cudaGetErrorString(e));
+  if (e != cudaSuccess) throw std::runtime_error(std::string("prefill over gathered rows: ") + cudaGetErrorString(e));
 }
 
 }  // namespace fc

@@ -91,7 +91,10 @@ __device__ __forceinline__ Best warp_best(Best b) {
 template <typename Put>
 __device__ __forceinline__ void choose_experts(const RouteScore& p, long long t, float* s_choice, float* s_group, Put put) {
   const int lane = threadIdx.x & 31, size = p.E / p.groups;
-  for (int e = lane; e < p.E; e += 32) s_choice[e] = sigmoid_f(proj_at<float>(p.logits, t, e)) + p.correction[e];
+  for (int e = lane; e < p.E; e += 32) {
+    const float z = proj_at<float>(p.logits, t, e);
+    s_choice[e] = (p.softmax ? z : sigmoid_f(z)) + p.correction[e];
+  }
   __syncwarp();
   if (p.keep < p.groups) {
     for (int g = lane; g < p.groups; g += 32) {
@@ -131,12 +134,17 @@ __device__ __forceinline__ void choose_and_weigh(const RouteScore& p, long long 
   const int lane = threadIdx.x & 31;
   if (p.ctx != nullptr && p.ctx[t] <= 0) {                   // a padding row has no experts
     for (int j = lane; j < p.top; j += 32) ids[j] = -1;
+    if (p.extra != nullptr && lane == 0) p.extra[t] = 0.f;
     return;
   }
-  float total = 0.f;
+  if (p.extra != nullptr && lane == 0) p.extra[t] = sigmoid_f(proj_at<float>(p.logits, t, p.E));
+  float total = 0.f, first = 0.f;
   float* mix = p.mix + t * p.top;
   choose_experts(p, t, s_choice, s_group, [&](int j, int e) {
-    const float s = sigmoid_f(proj_at<float>(p.logits, t, e));       // without the rounding of adding the correction
+    const float z = proj_at<float>(p.logits, t, e);
+    if (p.softmax && j == 0) first = z + p.correction[e];            // the largest
+    // sigmoid: without the rounding of adding the correction
+    const float s = p.softmax ? expf(z + p.correction[e] - first) : sigmoid_f(z);
     total += s;
     if (lane == 0) {
       ids[j] = e;
@@ -144,7 +152,7 @@ __device__ __forceinline__ void choose_and_weigh(const RouteScore& p, long long 
     }
   });
   __syncwarp();
-  const float inv = 1.f / (total + 1e-20f);
+  const float inv = 1.f / (p.softmax ? total : total + 1e-20f);
   for (int j = lane; j < p.top; j += 32) mix[j] *= inv;
 }
 
@@ -198,8 +206,9 @@ constexpr int RF_THREADS = 512;
 template <typename T>
 __global__ void __launch_bounds__(RF_THREADS)
 route_token_kernel(const RouteScore p) {
-  extern __shared__ float s_row[];                           // [K] h, [E] logits, [E + groups]
-  float *s_z = s_row + p.K, *s_choice = s_z + p.E;
+  extern __shared__ float s_row[];                           // [K] h, [n] logits, [E + groups]
+  const int n = p.E + (p.extra != nullptr ? 1 : 0);
+  float *s_z = s_row + p.K, *s_choice = s_z + n;
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -215,7 +224,7 @@ route_token_kernel(const RouteScore p) {
   ProjSrc w;
   w.p = p.w;
   w.ld = p.K;
-  for (int e = warp; e < p.E; e += RF_THREADS / 32) {
+  for (int e = warp; e < n; e += RF_THREADS / 32) {
     float z = 0.f;
 #pragma unroll 8
     for (int c = lane * 8; c < p.K; c += 256) {
@@ -231,7 +240,7 @@ route_token_kernel(const RouteScore p) {
   if (warp != 0) return;
   RouteScore q = p;                                          // this token's logits
   q.logits = ProjSrc();
-  q.logits.p = s_z;
+  q.logits.p = s_z;                                          // pitch 0
   choose_and_weigh(q, t, s_choice, s_choice + p.E, p.ids + (long long)t * p.top);
 }
 // The same from finished logits, `rows` tokens per CTA; with p.counts how often every expert was chosen by the CTA's tokens.
@@ -327,7 +336,7 @@ void launch_route_score(const RouteScore& a, bool f32, cudaStream_t s) {
   };
   const int each = p.E + p.groups;
   if (p.h != nullptr) {
-    const int floats = p.K + p.E + each;
+    const int floats = p.K + p.E + 1 + each;
     auto go = [&](auto kern) { launch_pdl(PDL_PARTIALS, kern, dim3(p.T), dim3(RF_THREADS), smem(kern, floats), s, p); };
     if (f32) go(route_token_kernel<float>);
     else go(route_token_kernel<__nv_bfloat16>);

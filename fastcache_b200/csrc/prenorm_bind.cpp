@@ -482,6 +482,7 @@ Projection as_projection(const Tensor& t, int64_t wide0, const OptTensor& wide) 
 }  // namespace
 
 void register_streams(pybind11::module_& m);
+void register_talking(pybind11::module_& m);
 
 void register_prenorm(pybind11::module_& m) {
   py::class_<Projection>(m, "Projection", "output of a packed projection, for the ops that read it")
@@ -498,4 +499,5 @@ void register_prenorm(pybind11::module_& m) {
   m.def("windowed_attention", &windowed_attention);
   m.def("matrix_memory", &matrix_memory);
   register_streams(m);
+  register_talking(m);
 }

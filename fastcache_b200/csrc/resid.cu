@@ -33,59 +33,93 @@ embed_scaled_kernel(const long long* __restrict__ ids, const T* __restrict__ wei
   }
 }
 
-// x += rms(y + bias) * w;  h = x in the model's type, zero-padded from W to Wp columns
-template <typename T, bool VEC>
+// x += rms(f (y + bias) + mixed expert rows) * w;  h = x in the model's type, zero-padded from W to Wp columns.  NC: 4-column
+// chunks per thread
+template <typename T, bool VEC, int NC>
 __global__ void __launch_bounds__(RS_THREADS)
-post_norm_add_kernel(const ProjSrc y, const T* __restrict__ bias, float* __restrict__ x, const float* __restrict__ w,
-                     T* __restrict__ h, int W, int Wp, float eps) {
+post_norm_add_kernel(const PostNormAdd p) {
   __shared__ float red[RS_THREADS / 32];
   pdl_launch_dependents();
   pdl_wait();
   const long long row = blockIdx.x;
-  float v[RS_CHUNKS][4];
-  float ss = 0.f;
+  const int W = p.W;
+  const T* bias = reinterpret_cast<const T*>(p.bias);
+  auto col_of = [&](int c) { return (int(threadIdx.x) + c * RS_THREADS) * 4; };
+  float v[NC][4];
 #pragma unroll
-  for (int c = 0; c < RS_CHUNKS; ++c) {
-    const int col = (threadIdx.x + c * RS_THREADS) * 4;
-    if (col >= W) continue;
-    const float4 a = proj_at4<T>(y, row, col);           // the pad columns of a projection exist and are zero
+  for (int c = 0; c < NC; ++c) {
+    const int col = col_of(c);
+    v[c][0] = v[c][1] = v[c][2] = v[c][3] = 0.f;
+    if (col >= W || !p.has_y) continue;
+    const float4 a = proj_at4<T>(p.y, row, col);         // the pad columns of a projection exist and are zero
     v[c][0] = a.x;
     v[c][1] = a.y;
     v[c][2] = a.z;
     v[c][3] = a.w;
+    if (bias != nullptr)
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+        if (VEC || col + i < W) v[c][i] += Elem<T>::get(bias[col + i]);
+  }
+  if (p.y_factor != nullptr) {
+    const float f = p.y_factor[row];
+#pragma unroll
+    for (int c = 0; c < NC; ++c)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) v[c][i] *= f;
+  }
+  for (int j = 0; j < p.top; ++j) {
+    const int r = p.row_of[row * p.top + j];
+    if (r < 0) continue;
+    const float f = p.mix != nullptr ? p.mix[row * p.top + j] : 1.f / float(p.top);
+    float4 e[NC];
+#pragma unroll
+    for (int c = 0; c < NC; ++c)
+      if (col_of(c) < W) e[c] = proj_at4<T>(p.experts, r, col_of(c));
+#pragma unroll
+    for (int c = 0; c < NC; ++c)
+      if (col_of(c) < W) {
+        v[c][0] = fmaf(e[c].x, f, v[c][0]);
+        v[c][1] = fmaf(e[c].y, f, v[c][1]);
+        v[c][2] = fmaf(e[c].z, f, v[c][2]);
+        v[c][3] = fmaf(e[c].w, f, v[c][3]);
+      }
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int c = 0; c < NC; ++c)
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
-      if (bias != nullptr) v[c][i] += Elem<T>::get(bias[col + i]);
-      if (!VEC && col + i >= W) v[c][i] = 0.f;
+      if (!VEC && col_of(c) + i >= W) v[c][i] = 0.f;
       ss += v[c][i] * v[c][i];
     }
-  }
-  const float inv = rsqrtf(cta_sum<RS_THREADS>(ss, red) / float(W) + eps);
+  const float inv = rsqrtf(cta_sum<RS_THREADS>(ss, red) / float(W) + p.eps);
+  float* x = p.x + row * W;
+  T* h = reinterpret_cast<T*>(p.h) + row * p.Wp;
 #pragma unroll
-  for (int c = 0; c < RS_CHUNKS; ++c) {
-    const int col = (threadIdx.x + c * RS_THREADS) * 4;
+  for (int c = 0; c < NC; ++c) {
+    const int col = col_of(c);
     if (col >= W) continue;
-    float* xr = x + row * W + col;
     if (VEC) {
-      float4 xv = *reinterpret_cast<const float4*>(xr);
-      const float4 wv = *reinterpret_cast<const float4*>(w + col);
+      float4 xv = *reinterpret_cast<const float4*>(x + col);
+      const float4 wv = *reinterpret_cast<const float4*>(p.w + col);
       xv.x += v[c][0] * inv * wv.x;
       xv.y += v[c][1] * inv * wv.y;
       xv.z += v[c][2] * inv * wv.z;
       xv.w += v[c][3] * inv * wv.w;
-      *reinterpret_cast<float4*>(xr) = xv;
-      store4(h + row * Wp + col, xv.x, xv.y, xv.z, xv.w);
+      *reinterpret_cast<float4*>(x + col) = xv;
+      store4(h + col, xv.x, xv.y, xv.z, xv.w);
     } else {
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
         if (col + i >= W) break;
-        const float n = xr[i] + v[c][i] * inv * w[col + i];
-        xr[i] = n;
-        h[row * Wp + col + i] = Elem<T>::put(n);
+        const float n = x[col + i] + v[c][i] * inv * p.w[col + i];
+        x[col + i] = n;
+        h[col + i] = Elem<T>::put(n);
       }
     }
   }
-  for (int c = W + threadIdx.x; c < Wp; c += RS_THREADS) h[row * Wp + c] = Elem<T>::put(0.f);
+  for (int c = W + threadIdx.x; c < p.Wp; c += RS_THREADS) h[c] = Elem<T>::put(0.f);
 }
 
 // x (+)= y + mixed expert rows;  h = rms(x) * w (or x) in the model's type, zero-padded from W to Wp columns.  NC: 4-column
@@ -195,6 +229,25 @@ glu_mul_kernel(const GluMul a) {
   }
 }
 
+// the same grid; one input
+template <typename T>
+__global__ void __launch_bounds__(RS_THREADS)
+xielu_kernel(const ProjSrc z, const float* __restrict__ coef, T* __restrict__ out, int rows, int width, int width_p) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int col = (blockIdx.x * RS_THREADS + threadIdx.x) * 8;
+  if (col >= width_p) return;
+  const float a = coef[0], b = coef[1];
+#pragma unroll 2
+  for (int row = blockIdx.y; row < rows; row += gridDim.y) {
+    float v[8];
+    proj_at8<T>(z, row, col, v);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) v[j] = col + j < width ? xielu_t<T>(v[j], a, b) : 0.f;
+    store8(out + (long long)row * width_p + col, v);
+  }
+}
+
 template <typename T>
 __global__ void __launch_bounds__(RS_THREADS)
 rms_norm_wide_kernel(const float* __restrict__ x, const float* __restrict__ w, T* __restrict__ h, int W, int Wp,
@@ -259,22 +312,23 @@ void launch_embed_scaled(const void* ids, const void* weight, float* x, void* h,
   check_launch("embedding");
 }
 
-template <typename T>
-static void post_norm_t(const ProjSrc& y, const void* bias, float* x, const float* w, void* h, int T_, int W, int Wp,
-                        float eps, cudaStream_t s) {
-  if (W % 4 == 0)
-    launch_pdl(PDL_NORM, post_norm_add_kernel<T, true>, dim3(T_), dim3(RS_THREADS), 0, s, y, (const T*)bias, x, w,
-               (T*)h, W, Wp, eps);
-  else
-    launch_pdl(PDL_NORM, post_norm_add_kernel<T, false>, dim3(T_), dim3(RS_THREADS), 0, s, y, (const T*)bias, x, w,
-               (T*)h, W, Wp, eps);
-}
-void launch_post_norm_add(const ProjSrc& y, const void* bias, float* x, const float* w, void* h, int T, int W, int Wp,
-                          float eps, bool f32, cudaStream_t s) {
-  if (T == 0) return;
-  if (W > RS_THREADS * RS_CHUNKS * 4) throw std::runtime_error("norm rows are limited to 8192 columns");
-  if (f32) post_norm_t<float>(y, bias, x, w, h, T, W, Wp, eps, s);
-  else post_norm_t<bf16>(y, bias, x, w, h, T, W, Wp, eps, s);
+void launch_post_norm_add(const PostNormAdd& p, bool f32, cudaStream_t s) {
+  if (p.T == 0) return;
+  if (p.W > RS_THREADS * RS_CHUNKS * 4) throw std::runtime_error("norm rows are limited to 8192 columns");
+  auto go = [&](auto kern) { launch_pdl(PDL_NORM, kern, dim3(p.T), dim3(RS_THREADS), 0, s, p); };
+  const int chunks = (p.W + RS_THREADS * 4 - 1) / (RS_THREADS * 4);
+  if (p.W % 4 != 0) {
+    if (f32) go(post_norm_add_kernel<float, false, RS_CHUNKS>);
+    else go(post_norm_add_kernel<bf16, false, RS_CHUNKS>);
+  } else if (f32) {
+    go(post_norm_add_kernel<float, true, RS_CHUNKS>);
+  } else if (chunks <= 2) {
+    go(post_norm_add_kernel<bf16, true, 2>);
+  } else if (chunks <= 4) {
+    go(post_norm_add_kernel<bf16, true, 4>);
+  } else {
+    go(post_norm_add_kernel<bf16, true, RS_CHUNKS>);
+  }
   check_launch("norm + add");
 }
 
@@ -323,6 +377,15 @@ void launch_glu_mul(const GluMul& p, bool f32, cudaStream_t s) {
     else go(glu_mul_kernel<bf16, GLU_ACT_CLAMPED>);
   }
   check_launch("gated activation");
+}
+
+void launch_xielu(const ProjSrc& z, const float* c, void* out, int T, int width, int width_p, bool f32, cudaStream_t s) {
+  if (T == 0) return;
+  const int cols = (width_p / 8 + RS_THREADS - 1) / RS_THREADS;
+  const dim3 grid(cols, std::min(T, std::max(1, 148 * 8 / cols)));
+  if (f32) launch_pdl(PDL_PARTIALS, xielu_kernel<float>, grid, dim3(RS_THREADS), 0, s, z, c, (float*)out, T, width, width_p);
+  else launch_pdl(PDL_PARTIALS, xielu_kernel<bf16>, grid, dim3(RS_THREADS), 0, s, z, c, (bf16*)out, T, width, width_p);
+  check_launch("xIELU");
 }
 
 void launch_gelu_mul(const ProjSrc& gu, const void* bias, void* out, int T, int up_off, int width, int width_p,

@@ -98,9 +98,8 @@ Tensor mix_norm(const Projection& y, Tensor x, const Tensor& connection, const O
   return h;
 }
 
-// (row_of, plan, weights)
-std::tuple<Tensor, Tensor, Tensor> route_by_score(const Tensor& h, const Tensor& weight, const Tensor& correction, int64_t top,
-                                                  int64_t groups, int64_t keep, const OptTensor& ctx) {
+std::tuple<Tensor, Tensor, Tensor> route(const Tensor& h, const Tensor& weight, const Tensor& correction, int64_t top, int64_t groups,
+                                         int64_t keep, const OptTensor& ctx, bool softmax, float* extra) {
   const int T = int(h.size(0)), E = int(correction.numel());
   check_f32(correction, "correction", E);
   TORCH_CHECK(groups > 0 && E % groups == 0 && keep > 0 && keep <= groups && top > 0 && top <= keep * (E / groups), "bad routing sizes");
@@ -115,7 +114,7 @@ std::tuple<Tensor, Tensor, Tensor> route_by_score(const Tensor& h, const Tensor&
     r.ctx = ctx->data_ptr<int>();
   }
   check_product(h, weight);
-  TORCH_CHECK(weight.size(0) >= E, "the router needs a row per expert");
+  TORCH_CHECK(weight.size(0) >= E + (extra != nullptr ? 1 : 0), "the router needs a row per expert");
   Projection z;
   if (T <= fc::ROUTE_SMALL && (int64_t)T * E <= 4096) {     // the weights are read once per token
     r.h = h.data_ptr();
@@ -132,6 +131,8 @@ std::tuple<Tensor, Tensor, Tensor> route_by_score(const Tensor& h, const Tensor&
   r.E = E;
   r.groups = int(groups);
   r.keep = int(keep);
+  r.softmax = softmax;
+  r.extra = extra;
   r.mix = mix.data_ptr<float>();
   r.row_of = row_of.data_ptr<int>();
   r.plan = plan.data_ptr<int>();
@@ -139,6 +140,20 @@ std::tuple<Tensor, Tensor, Tensor> route_by_score(const Tensor& h, const Tensor&
   r.counts = counts.data_ptr<int>();
   fc::launch_route_score(r, is_f32(h), stream_now());
   return {row_of, plan, mix};
+}
+
+// (row_of, plan, weights)
+std::tuple<Tensor, Tensor, Tensor> route_by_score(const Tensor& h, const Tensor& weight, const Tensor& correction, int64_t top,
+                                                  int64_t groups, int64_t keep, const OptTensor& ctx) {
+  return route(h, weight, correction, top, groups, keep, ctx, false, nullptr);
+}
+// (row_of, plan, weights, factor of the shared expert: the sigmoid of the row behind the experts')
+std::tuple<Tensor, Tensor, Tensor, OptTensor> route_by_logit(const Tensor& h, const Tensor& weight, const Tensor& bias, int64_t top,
+                                                             bool shared, const OptTensor& ctx) {
+  OptTensor extra;
+  if (shared) extra = torch::empty({h.size(0)}, h.options().dtype(torch::kFloat32));
+  auto [row_of, plan, mix] = route(h, weight, bias, top, 1, 1, ctx, true, shared ? extra->data_ptr<float>() : nullptr);
+  return {row_of, plan, mix, extra};
 }
 
 // ------------------------------------------------------------------ real-gated linear recurrent unit
@@ -274,5 +289,6 @@ void register_streams(pybind11::module_& m) {
   m.def("linear_mix_norm", &linear_mix_norm);
   m.def("mix_norm", &mix_norm);
   m.def("route_by_score", &route_by_score);
+  m.def("route_by_logit", &route_by_logit);
   m.def("real_gated_lru", &real_gated_lru);
 }

@@ -376,7 +376,8 @@ class ModelRunner:
         return {"state_slots": self._to_dev(self._state_slots(seqs), torch.int32),
                 "row_seq": self._to_dev(np.repeat(np.arange(len(seqs), dtype=np.int32), lens), torch.int32),
                 "row_ctx": self._to_dev(ctx, torch.int32),
-                "cu_seqlens_kv": self._to_dev(cu_kv.astype(np.int32), torch.int32), "total_kv": int(cu_kv[-1])}
+                "cu_seqlens_kv": self._to_dev(cu_kv.astype(np.int32), torch.int32), "total_kv": int(cu_kv[-1]),
+                "q_lens": lens, "kv_lens": kv_lens}
 
     def prepare_decode(self, seqs: Seq[Sequence]):
         bs = self.block_size

@@ -1,4 +1,5 @@
-"""Mixture of experts: gated feed-forward experts, a router that reads a table of the token ids and one that scores them."""
+"""Mixture of experts: gated feed-forward experts, one that every token uses, and routers: by a table of the token ids, by
+sigmoid scores within groups, by logits."""
 from __future__ import annotations
 
 import torch
@@ -8,6 +9,7 @@ from .. import ops
 from ..ops.hybrid import GluSpec
 from ..utils.context import get_context
 from .linear import PackedLinear, pad8
+from .recurrent import fp32_vector
 
 
 class TableRouter(nn.Module):
@@ -49,6 +51,38 @@ class ScoreRouter(nn.Module):
     def forward(self, h: torch.Tensor):
         """(the step's routing, weights)"""
         return ops.hybrid.route_by_score(h, self.proj.weight, self.correction, self.top, self.groups, self.keep, get_context())
+
+
+class LogitRouter(nn.Module):
+    """The `top` experts with the largest logits of a linear map with bias; their weights are the softmax of these logits.
+    `shared`: one more row of the map gives a shared expert's factor, through a sigmoid."""
+
+    def __init__(self, width: int, experts: int, top: int, shared: bool = False):
+        super().__init__()
+        if not 0 < top <= experts:
+            raise ValueError(f"{top} experts per token of {experts}")
+        self.experts, self.top, self.shared = experts, top, shared
+        self.proj = PackedLinear(width, dict({"router": experts}, **({"sg": 1} if shared else {})), tight=("sg",))
+        self.bias = fp32_vector(experts)
+
+    def forward(self, h: torch.Tensor):
+        """(the step's routing, weights, factor of the shared expert or None)"""
+        return ops.hybrid.route_by_logit(h, self.proj.weight, self.bias, self.top, self.shared, get_context())
+
+
+class GatedFeedForward(nn.Module):
+    """Gated feed-forward up to its down projection, without biases (a shared expert)."""
+
+    def __init__(self, width: int, ff: int, spec: GluSpec):
+        super().__init__()
+        self.ff, self.spec = int(ff), spec
+        self.gate_up = PackedLinear(width, {"gate": self.ff, "up": self.ff})
+        self.down = PackedLinear(self.ff, {"down": width})
+
+    def forward(self, h: torch.Tensor) -> torch.Tensor:
+        a = h.new_empty(h.shape[0], pad8(self.ff))
+        ops.hybrid.linear_glu(h, self.gate_up.weight, self.gate_up.offset["up"], self.ff, self.spec, a)
+        return a
 
 
 class Experts(nn.Module):

@@ -26,6 +26,8 @@ def detect_model_type(hf_config: Any) -> str:
         return "lekilix"
     if "duperax" in mt or "duperax" in joined:
         return "duperax"
+    if "darusun" in mt or "darusun" in joined:
+        return "darusun"
     if "llama" in mt or "llama" in joined or "mistral" in mt:
         return "llama"
     raise ValueError(f"unsupported model type {mt!r} / architectures {archs}")
@@ -71,9 +73,15 @@ def _duperax(cfg):
     return DuperaxForCausalLM(cfg)
 
 
+def _darusun(cfg):
+    from .darusun import DarusunForCausalLM
+    return DarusunForCausalLM(cfg)
+
+
 MODEL_REGISTRY: Dict[str, Callable] = {
     "llama": _llama, "qwen3": _qwen3, "qwen2": _qwen2, "llava": _llava, "minicpm": _minicpm,
     "bagedra": _bagedra, "lekilix": _lekilix, "duperax": _duperax,
+    "darusun": _darusun,
 }
 
 

@@ -55,7 +55,11 @@ class DeltaDims:
 
 @dataclass(frozen=True)
 class LatentDims:
-    """Latent attention; `kv` is None for a layer that reads another layer's cache rows."""
+    """Latent attention; `kv` is None for a layer that reads another layer's cache rows.
+
+    `g` None: no output gate; `head_gate`: one column per head.  `dq`: first column of the latent (of `q_rank`) that the
+    queries are made from; None: they are the columns from `q` on.  `half`: entry i of a rotated part turns with entry
+    i + rot_dims / 2 (else entries 2i and 2i + 1).  `window`: the positions a query sees, itself included (0: all up to itself)."""
     heads: int
     dim: int
     rot: int
@@ -65,8 +69,38 @@ class LatentDims:
     base: float
     rot_dims: int
     q: int
-    g: int
+    g: Optional[int]
     kv: Optional[int]
+    dq: Optional[int] = None
+    q_rank: int = 0
+    window: int = 0
+    half: bool = True
+    head_gate: bool = False
+
+    def sizes(self) -> list:
+        """The integers as the extension takes them (-1: no such projection)."""
+        return [self.heads, self.dim, self.rot, self.vdim, self.rank, self.rot_dims, self.q, -1 if self.kv is None else self.kv,
+                -1 if self.g is None else self.g, self.dq or 0, self.q_rank, self.window, int(self.half), int(self.head_gate)]
+
+
+@dataclass(frozen=True)
+class TalkDims:
+    """Attention whose heads mix their scores: sizes, first columns of the packed projections (`k` and `v` None: another
+    layer's cache rows), first value column of a cache row."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    rot_dims: int
+    scale: float
+    q: int
+    k: Optional[int]
+    v: Optional[int]
+    v_col: int
+
+    def sizes(self) -> list:
+        return [self.heads, self.kv_heads, self.dim, self.vdim, self.rot_dims, self.q, -1 if self.k is None else self.k,
+                -1 if self.v is None else self.v, self.v_col]
 
 
 @dataclass(frozen=True)
@@ -151,12 +185,23 @@ def embed_scaled(ids, weight, width: int, scale: float):
     return ref.embed_scaled(ids, weight, width, scale)
 
 
-def linear_post_norm_add(a, weight, bias, x, norm_w, eps: float):
-    """x += RMSNorm(a @ weight.T + bias) * norm_w in fp32, in place; returns x in the model's dtype (padded width)."""
+def linear_post_norm_add(a, weight, bias, x, norm_w, eps: float, experts=None, factor=None):
+    """x += RMSNorm(factor * (a @ weight.T + bias) + the mixed outputs of `experts`) * norm_w in fp32, in place; returns x in
+    the model's dtype (padded width).  `factor` [T] fp32, or None: 1."""
     if a.is_cuda:
         _n(2)
-        return ext().linear_post_norm_add(a, weight, bias, x, norm_w, float(eps))
-    return ref.post_norm_add(ref_linear(a, weight, bias), x, norm_w, eps)
+        y, row_of, mix = experts if experts is not None else (None, None, None)
+        return ext().linear_post_norm_add(a, weight, bias, x, norm_w, float(eps), y, row_of, mix, factor)
+    return ref.post_norm_add(ref_linear(a, weight, bias), x, norm_w, eps, experts, factor)
+
+
+def linear_xielu(h, weight, coef, width: int):
+    """xIELU of h @ weight.T (see `reference_hybrid.xielu`; coef [2] fp32), padded to 8 columns."""
+    if h.is_cuda:
+        _n(2)
+        return ext().linear_xielu(h, weight, coef, int(width))
+    z = ref_linear(h, weight)
+    return ref._pad_to(ref.xielu(z[:, :width].float(), coef).to(h.dtype), z.shape[1])
 
 
 def rms_norm_wide(x, norm_w, eps: float, width: int, dtype):
@@ -209,23 +254,43 @@ def _run_args(ctx):
 
 
 # ------------------------------------------------------------------ latent attention
-def latent_attention(h, weight, d: LatentDims, kv_norm_w, eps: float, kv_proj, w_ukt, w_uv, pool, positions, ctx):
+def latent_attention(h, weight, d: LatentDims, kv_norm_w, eps: float, kv_proj, w_ukt, w_uv, pool, positions, ctx, q_norm_w=None,
+                     q_weight=None, sink=None):
     """Projections, cache store, attention and output gate of a latent-attention layer up to the output projection.
+    `q_norm_w`, `q_weight`: norm and projection of the queries' latent; `sink` [H] joins the softmax without a key.
 
     `kv_proj` (packed uk | uv) expands cache rows to keys and values (prefill); `w_ukt` [H, rank, dim] and `w_uv`
     [H, vdim, rank] are the same weights for the absorbed form (decode), which never expands a row."""
     if h.is_cuda:
         _n(6)
+        cu_kv, max_kv, total_kv = ctx.kv_span(d.window)
         return ext().latent_attention(
-            h, weight, [d.heads, d.dim, d.rot, d.vdim, d.rank, d.rot_dims, d.q, -1 if d.kv is None else d.kv, d.g],
-            d.scale, d.base, kv_norm_w, float(eps), kv_proj.weight, kv_proj.offset["uv"], w_ukt, w_uv, pool, positions,
-            ctx.slot_mapping, ctx.block_tables, ctx.context_lens, ctx.cu_seqlens_q, ctx.cu_seqlens_kv, ctx.row_seq,
-            ctx.row_ctx, int(ctx.max_seqlen_q), int(ctx.max_seqlen_k), int(ctx.total_kv), LATENT_IMPL)
+            h, weight, d.sizes(), d.scale, d.base, kv_norm_w, float(eps), kv_proj.weight, kv_proj.offset["uv"], w_ukt, w_uv, pool,
+            positions, ctx.slot_mapping, ctx.block_tables, ctx.context_lens, ctx.cu_seqlens_q, cu_kv, ctx.row_seq, ctx.row_ctx,
+            int(ctx.max_seqlen_q), int(ctx.max_seqlen_k), max_kv, total_kv, q_norm_w, q_weight, sink, LATENT_IMPL)
     p = ref_linear(h, weight)
-    q = ref.latent_project(p, d, kv_norm_w, eps, positions, pool, ctx.slot_mapping)
+    q_in = p[:, d.q:] if d.dq is None else ref_linear(ref.latent_of_queries(p, d, q_norm_w, eps, q_weight.shape[1]), q_weight)
+    q = ref.latent_project(p, q_in, d, kv_norm_w, eps, positions, pool, ctx.slot_mapping)
     w, off = kv_proj.weight, kv_proj.offset
-    return ref.latent_attention(q, p[:, d.g:d.g + d.heads * d.vdim], d, w[off["uk"]:off["uk"] + d.heads * d.dim],
-                                w[off["uv"]:off["uv"] + d.heads * d.vdim], pool, ctx)
+    gate = None if d.g is None else p[:, d.g:d.g + d.heads * (1 if d.head_gate else d.vdim)]
+    return ref.latent_attention(q, gate, d, w[off["uk"]:off["uk"] + d.heads * d.dim],
+                                w[off["uv"]:off["uv"] + d.heads * d.vdim], pool, ctx, sink)
+
+
+# ------------------------------------------------------------------ attention whose heads mix their scores
+TALK_IMPL = 0           # tests: 1 the general kernels also where a tensor-core form exists, 2 the decode form also in prefill
+
+
+def talking_attention(p, d: TalkDims, freq, talk, eps: float, pool, positions, ctx, out):
+    """Rotation (`freq`: rope_turns), norm per head, cache store, attention with scores talk @ scores to `out`.  talk [H, H]
+    fp32, to and from; cache rows [keys | values] of all key heads."""
+    if out.is_cuda:
+        _n(3)
+        ext().talking_attention(p, d.sizes(), d.scale, freq, talk, float(eps), pool, positions, ctx.slot_mapping, ctx.block_tables,
+                                ctx.context_lens, ctx.cu_seqlens_q, ctx.cu_seqlens_kv, ctx.row_seq, ctx.row_ctx,
+                                int(ctx.max_seqlen_q), int(ctx.max_seqlen_k), int(ctx.total_kv), out, TALK_IMPL)
+    else:
+        ref.talking_attention(p, d, freq, talk, eps, pool, positions, ctx, out)
 
 
 # ------------------------------------------------------------------ pre-normed layers with parallel sublayers
@@ -319,6 +384,17 @@ def route_by_score(h, weight, correction, top: int, groups: int, keep: int, ctx)
                                                  None if ctx.is_prefill else ctx.context_lens)
         return (row_of, plan), mix
     return ref.route_by_score(ref_linear(h, weight), correction, top, groups, keep)
+
+
+def route_by_logit(h, weight, bias, top: int, shared: bool, ctx):
+    """Which rows every expert gets, their weights [T, top], the softmax of the chosen logits h @ weight.T + bias, and (shared)
+    the factor of a shared expert, the sigmoid of the row of `weight` behind the experts'.  CPU: ([T, top], weights, factor)."""
+    if h.is_cuda:
+        _n(3)
+        row_of, plan, mix, factor = ext().route_by_logit(h, weight, bias, int(top), bool(shared),
+                                                         None if ctx.is_prefill else ctx.context_lens)
+        return (row_of, plan), mix, factor
+    return ref.route_by_logit(ref_linear(h, weight), bias, top, shared)
 
 
 def experts(h, route, weights, w_gate_up, w_down, ff: int, spec: GluSpec):

@@ -1,6 +1,6 @@
 """Plain PyTorch statements of the ops of hybrid models: norms on a 32-bit residual, short convolution, gated linear
-attention, gated delta rule, matrix memory, real-gated recurrence, paged latent attention, windowed and chunked attention,
-experts, several residual streams.
+attention, gated delta rule, matrix memory, real-gated recurrence, paged latent attention, attention with mixed heads, windowed
+and chunked attention, experts, several residual streams.
 
 Like `reference.py`: the execution path on CPU tensors.  A batch is a concatenation of runs of rows, one run per
 request, with the request's state slot and the position of its first row; a run that starts at position 0 starts
@@ -41,9 +41,20 @@ def embed_scaled(ids, weight, width: int, scale: float):
     return x, _pad_to(x.to(weight.dtype), weight.shape[1])
 
 
-def post_norm_add(y, x, weight, eps: float):
-    x += _rms(y[:, : x.shape[1]].float(), eps) * weight
+def post_norm_add(y, x, weight, eps: float, experts=None, factor=None):
+    s = y[:, : x.shape[1]].float()
+    if factor is not None:
+        s = s * factor[:, None]
+    if experts is not None:
+        s = s + experts[:, : x.shape[1]].float()
+    x += _rms(s, eps) * weight
     return _pad_to(x.to(y.dtype), y.shape[1])
+
+
+def xielu(z, coef):
+    """coef[0] z^2 + z / 2 above 0, coef[1] (exp(z) - 1 - z) + z / 2 below."""
+    n = z.clamp(max=0)
+    return torch.where(z > 0, coef[0] * z * z, coef[1] * (torch.expm1(n) - n)) + z / 2
 
 
 def rms_norm_wide(x, weight, eps: float, width: int, dtype):
@@ -142,31 +153,35 @@ def real_gated_lru(p, d, conv_w, conv_b, gate_w, gate_b, lam, conv_state, state,
 
 
 # ------------------------------------------------------------------ latent attention
-def _rope(x, positions, base: float, dims: int):
-    i = torch.arange(dims // 2, dtype=torch.float64, device=x.device)
-    a = positions.double()[:, None, None] * base ** (-2 * i / dims)
-    cos, sin = a.cos().float(), a.sin().float()
-    return torch.cat([_rotate(x[..., :dims].float(), cos, sin), x[..., dims:].float()], -1).to(x.dtype)
+def latent_of_queries(p, d, norm_w, eps: float, width: int):
+    c = _rms(p[:, d.dq:d.dq + d.q_rank].float(), eps) * norm_w
+    return _pad_to(c.to(p.dtype), width)
 
 
-def latent_project(p, d, norm_w, eps: float, positions, pool, slots):
+def latent_project(p, q_in, d, norm_w, eps: float, positions, pool, slots):
     """Writes the cache rows (normed latent | rotated shared key part) of a layer that owns a cache and returns the
-    queries with their rotated part rotated, [T, H, dim + rot]."""
+    queries (first columns of `q_in`) with their rotated part rotated, [T, H, dim + rot]."""
     T = p.shape[0]
-    q = p[:, d.q:d.q + d.heads * (d.dim + d.rot)].reshape(T, d.heads, d.dim + d.rot).clone()
-    q[..., d.dim:] = _rope(q[..., d.dim:], positions, d.base, d.rot_dims)
+    i = torch.arange(d.rot_dims // 2, dtype=torch.float64, device=p.device)
+    turns = d.base ** (-2 * i / max(1, d.rot_dims)) / (2 * math.pi)
+
+    def turned(x):
+        return rope_rows(x, positions, turns, d.rot_dims, d.half, 1.0).to(x.dtype)
+
+    q = q_in[:, :d.heads * (d.dim + d.rot)].reshape(T, d.heads, d.dim + d.rot).clone()
+    q[..., d.dim:] = turned(q[..., d.dim:])
     if d.kv is not None:
         kv = p[:, d.kv:d.kv + d.rank + d.rot]
         c = (_rms(kv[:, : d.rank].float(), eps) * norm_w).to(p.dtype)
-        r = _rope(kv[:, None, d.rank:], positions, d.base, d.rot_dims)[:, 0]
+        r = turned(kv[:, None, d.rank:])[:, 0]
         ok = slots >= 0
         flat = pool.view(-1, pool.shape[-1])
         flat[slots[ok].long(), : d.rank + d.rot] = torch.cat([c, r], -1)[ok].to(pool.dtype)
     return q
 
 
-def latent_attention(q, gate, d, w_uk, w_uv, pool, ctx):
-    """Causal attention of the rows of `q` over the cache rows of their requests, times sigmoid(gate)."""
+def latent_attention(q, gate, d, w_uk, w_uv, pool, ctx, sink=None):
+    """Causal attention of the rows of `q` over the cache rows of their requests (inside the window), times sigmoid(gate)."""
     T, H = q.shape[0], d.heads
     out = torch.zeros(T, H, d.vdim, dtype=torch.float32)
     for i, lo, hi, start, _ in runs(ctx):
@@ -178,10 +193,55 @@ def latent_attention(q, gate, d, w_uk, w_uv, pool, ctx):
         v = (c @ w_uv[:, : d.rank].float().T).view(n, H, d.vdim)
         s = torch.einsum("ihd,jhd->hij", q[lo:hi, :, : d.dim].float(), kn)
         s = (s + torch.einsum("ihd,jd->hij", q[lo:hi, :, d.dim:].float(), r)) * d.scale
-        hidden = torch.arange(n)[None, :] > torch.arange(start, n)[:, None]
-        out[lo:hi] = torch.einsum("hij,jhv->ihv", torch.softmax(s.masked_fill(hidden, float("-inf")), -1), v)
-    y = out.reshape(T, H * d.vdim) * torch.sigmoid(gate.float())
+        at, key = torch.arange(start, n)[:, None], torch.arange(n)[None, :]
+        hidden = key > at
+        if d.window > 0:
+            hidden |= at - key >= d.window
+        out[lo:hi] = torch.einsum("hij,jhv->ihv", softmax_with_sink(s.masked_fill(hidden, float("-inf")), sink), v)
+    if gate is not None:
+        g = torch.sigmoid(gate.float())
+        out = out * (g[:, :, None] if d.head_gate else g.view(T, H, d.vdim))
+    y = out.reshape(T, H * d.vdim)
     return _pad_to(y.to(q.dtype), -(-H * d.vdim // 8) * 8)
+
+
+def softmax_with_sink(s, sink):
+    """Softmax of s [H, i, j] over j whose denominator also holds exp(sink [H]) (None: not)."""
+    if sink is None:
+        return torch.softmax(s, -1)
+    n = s.shape[-1]
+    return torch.softmax(torch.cat([s, sink[:, None, None].expand(-1, s.shape[1], 1)], -1), -1)[..., :n]
+
+
+# ------------------------------------------------------------------ attention whose heads mix their scores
+def talking_attention(p, d, turns, talk, eps: float, pool, positions, ctx, out):
+    """Stores the batch's keys and values in the pages (layers that own them) and writes attention to `out`.  d:
+    `ops.hybrid.TalkDims`."""
+    T, H, G, D, V = p.shape[0], d.heads, d.kv_heads, d.dim, d.vdim
+
+    def turned(off, heads):
+        x = p[:, off:off + heads * D].reshape(T, heads, D)
+        return _rms(rope_rows(x, positions, turns, d.rot_dims, True, 1.0), eps)
+
+    q = turned(d.q, H)
+    if d.k is not None:
+        ok = ctx.slot_mapping >= 0
+        rows = torch.zeros(T, pool.shape[-1])
+        rows[:, :G * D] = turned(d.k, G).reshape(T, G * D)
+        rows[:, d.v_col:d.v_col + G * V] = p[:, d.v:d.v + G * V].float()
+        pool.view(-1, pool.shape[-1])[ctx.slot_mapping[ok].long()] = rows[ok].to(pool.dtype)
+    o = torch.zeros(T, H, V)
+    for i, lo, hi, start, _ in runs(ctx):
+        n = start + hi - lo
+        blocks = ctx.block_tables[i][: -(-n // pool.shape[1])].long()
+        rows = pool[blocks].reshape(-1, pool.shape[-1])[:n].float()
+        k, v = rows[:, :G * D].reshape(n, G, D), rows[:, d.v_col:d.v_col + G * V].reshape(n, G, V)
+        s = torch.einsum("ihd,jhd->hij", q[lo:hi], k.repeat_interleave(H // G, 1)) * d.scale
+        s = torch.einsum("hg,gij->hij", talk, s)
+        hidden = torch.arange(n)[None, :] > torch.arange(start, n)[:, None]
+        o[lo:hi] = torch.einsum("hij,jhv->ihv", torch.softmax(s.masked_fill(hidden, float("-inf")), -1),
+                                v.repeat_interleave(H // G, 1))
+    out.copy_(_pad_to(o.reshape(T, H * V).to(p.dtype), out.shape[1]))
 
 
 # ------------------------------------------------------------------ pre-normed layers
@@ -243,6 +303,14 @@ def route_by_score(z, correction, top: int, groups: int, keep: int):
     return ids, w / (w.sum(-1, keepdim=True) + 1e-20)
 
 
+def route_by_logit(z, bias, top: int, shared: bool):
+    """Chosen experts [T, top] (largest logits z + bias), the softmax of their logits, and the sigmoid of the column of z behind
+    the experts' (or None)."""
+    E = bias.numel()
+    best = (z[:, :E].float() + bias).topk(top, -1)
+    return best.indices, torch.softmax(best.values, -1), torch.sigmoid(z[:, E].float()) if shared else None
+
+
 def experts(h, ids, weights, w_gate_up, w_down, ff: int, act: str, limit: float):
     """Sum over a token's experts `ids` [T, top] of weight * down(glu(gate, up)); weights None: equal ones."""
     out = torch.zeros(h.shape[0], w_down.shape[1], dtype=torch.float32, device=h.device)
@@ -299,10 +367,7 @@ def windowed_attention(p, d, turns, q_norm, k_norm, sink, eps: float, k_rows, v_
             hidden |= at - key >= d.window
         if d.chunk > 0:
             hidden |= key < at // d.chunk * d.chunk
-        s = s.masked_fill(hidden, float("-inf"))
-        if sink is not None:
-            s = torch.cat([s, sink[:, None, None].expand(-1, hi - lo, 1)], -1)
-        o[lo:hi] = torch.einsum("hij,jhd->ihd", torch.softmax(s, -1)[..., :n], vs)
+        o[lo:hi] = torch.einsum("hij,jhd->ihd", softmax_with_sink(s.masked_fill(hidden, float("-inf")), sink), vs)
     y = o.reshape(T, H * V)
     if d.g is not None:
         y = y * torch.sigmoid(p[:, d.g:d.g + H * V].float())

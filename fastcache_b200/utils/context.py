@@ -7,9 +7,10 @@ store, for prefill and decode alike.
 """
 from __future__ import annotations
 
-from dataclasses import dataclass
-from typing import Any, Optional
+from dataclasses import dataclass, field
+from typing import Any, Dict, Optional, Sequence, Tuple
 
+import numpy as np
 import torch
 
 
@@ -39,6 +40,23 @@ class Context:
     # latent attention in prefill: first row of every request in the batch's gathered cache rows, their total
     cu_seqlens_kv: Optional[torch.Tensor] = None
     total_kv: int = 0
+    # the same on the host: rows of every request in this step and after it
+    q_lens: Optional[Sequence[int]] = None
+    kv_lens: Optional[Sequence[int]] = None
+    _spans: Dict[int, Tuple[Any, int, int]] = field(default_factory=dict)
+
+    def kv_span(self, window: int) -> Tuple[Optional[torch.Tensor], int, int]:
+        """The last cache rows of every request that its rows of this step see through a window (0: all): (boundaries, most
+        rows of a request, total)."""
+        if window <= 0 or self.kv_lens is None:
+            return self.cu_seqlens_kv, int(self.max_seqlen_k), int(self.total_kv)
+        if window not in self._spans:
+            n = np.minimum(np.asarray(self.kv_lens), np.asarray(self.q_lens) + window - 1)
+            cu = torch.from_numpy(np.concatenate([[0], np.cumsum(n)]).astype(np.int32))
+            if self.cu_seqlens_kv.is_cuda:
+                cu = cu.pin_memory().to(self.cu_seqlens_kv.device, non_blocking=True)
+            self._spans[window] = cu, int(n.max()), int(n.sum())
+        return self._spans[window]
 
 
 _CONTEXT = Context()

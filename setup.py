@@ -15,7 +15,7 @@ SRC = os.path.join("fastcache_b200", "csrc")
 CORE = os.environ.get("FC_EXT") == "core"
 CORE_SOURCES = ("attn_decode.cu", "attn_prefill.cu", "attn_prefill_tc2.cu", "bindings.cpp", "elementwise.cu", "gemm.cu", "gemm_2cta.cu", "gemm_skinny.cu", "gemm_streamk.cu",
                 "hybrid_bind.cpp", "latent.cu", "latent_decode.cu", "latent_decode_tc.cu", "latent_prefill.cu", "linear_simt.cu", "lru.cu", "moe.cu", "moe_gemm.cu", "partials.cu", "prenorm_bind.cpp",
-                "recurrence.cu", "recurrence_chunk.cu", "resid.cu", "streams.cu", "streams_bind.cpp", "window_attn.cu")
+                "recurrence.cu", "recurrence_chunk.cu", "resid.cu", "streams.cu", "streams_bind.cpp", "talking.cu", "talking_bind.cpp", "window_attn.cu")
 sources = [os.path.join(SRC, f) for f in CORE_SOURCES] if CORE else sorted(glob.glob(os.path.join(SRC, "*.cu")) + glob.glob(os.path.join(SRC, "*.cpp")))
 
 nvcc_flags = ["-O3", "-std=c++17", "-lineinfo", "-gencode", "arch=compute_100a,code=sm_100a",
