@@ -678,7 +678,7 @@ def main():
     ap.add_argument("--check", action="store_true",
                     help="instead of timing: first tokens under --gpus N against the same prompts on one GPU "
                          "(shrunken config, greedy)")
-    ap.add_argument("--layers", nargs="?", const="bagedra", default="", choices=["bagedra", "lekilix", "duperax"],
+    ap.add_argument("--layers", nargs="?", const="bagedra", default="", choices=["bagedra", "lekilix", "duperax", "darusun"],
                     help="instead of the job: prefill and decode throughput of a hybrid model's layers beside the dense "
                          "decoder at a few equal sizes, and the roofline of their kernels (1 GPU)")
     ap.add_argument("--small", action="store_true", help="--layers: the smallest size only")

@@ -258,6 +258,9 @@ def run(steps=5, small=False, kernels=True, model="bagedra"):
     elif model == "duperax":
         from benchmarks import streams_bench
         make, table = streams_bench.model_config, streams_bench.kernel_table
+    elif model == "darusun":
+        from benchmarks import talking_bench
+        make, table = talking_bench.model_config, talking_bench.kernel_table
     sizes = {"2k": SIZES["2k"]} if small else SIZES
     out = {"layers": LAYERS, "sizes": {}}
     for name, size in sizes.items():

@@ -36,6 +36,7 @@
 #include <unordered_map>
 
 #include "gemm.h"
+#include "hybrid.cuh"
 #include "ptx.cuh"
 
 namespace fc {
@@ -67,6 +68,7 @@ struct GemmParams {
   const int* plan;        // GF_GROUPED: rows sorted by group, see gemm_bf16_grouped
   int groups, group_rows; // groups, rows of W per group
   float limit;            // GLU_CLAMPED
+  const float* coef;      // GF_XIELU: its two factors
 };
 
 __device__ __forceinline__ float apply_act(float v, int act) {
@@ -123,7 +125,7 @@ struct SmemLayout {
 
 // GLU: gated epilogue, out = act(gate) * up of w = [gate; up]
 enum Glu : int { GLU_NONE = 0, GLU_SILU = 1, GLU_GELU_TANH = 2, GLU_CLAMPED = 3 };   // GLU_GELU_TANH takes a bias [gate | up]
-enum GemmForm : int { GF_PLAIN = 0, GF_WIDE = 1, GF_ACC = 2, GF_GROUPED = 3 };
+enum GemmForm : int { GF_PLAIN = 0, GF_WIDE = 1, GF_ACC = 2, GF_GROUPED = 3, GF_XIELU = 4 };
 
 template <int BN, int STAGES, bool TRANS_OUT, int GLU = GLU_NONE, int FORM = GF_PLAIN>
 __global__ void __launch_bounds__(GEMM_THREADS, 1)
@@ -371,7 +373,13 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_constan
                 for (int t = 0; t < 32; ++t) v[t] += __bfloat162float(p.bias[jb + t]);
               }
             }
-            apply_act_chunk(v, p.act);
+            if constexpr (FORM == GF_XIELU) {
+              const float a = __ldg(p.coef), b = __ldg(p.coef + 1);
+#pragma unroll
+              for (int t = 0; t < 32; ++t) v[t] = xielu_t<__nv_bfloat16>(v[t], a, b);
+            } else {
+              apply_act_chunk(v, p.act);
+            }
 #pragma unroll
             for (int q = 0; q < 4; ++q) {
               uint32_t u[4];
@@ -385,7 +393,9 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_constan
               if (jb + t < p.N) {
                 float a = v[t] + bi;
                 if (p.bias != nullptr && !p.bias_on_i) a += __bfloat162float(p.bias[jb + t]);
-                dst[t] = __float2bfloat16(apply_act(a, p.act));
+                if constexpr (FORM == GF_XIELU) a = xielu_t<__nv_bfloat16>(a, __ldg(p.coef), __ldg(p.coef + 1));
+                else a = apply_act(a, p.act);
+                dst[t] = __float2bfloat16(a);
               }
             }
           }
@@ -747,6 +757,18 @@ void gemm_bf16_clamped_glu(const void* x, const void* w, void* c, int M, int wid
   launch_one<BN, 4, false, GLU_CLAMPED>(make_tmap_bf16_2d(x, M, K, ldx, BM, BK),
                                         make_tmap_bf16_2d(w, 2 * width, K, ldw, BN / 2, BK), p,
                                         std::min(p.total_work, sm_limit > 0 ? sm_limit : gemm_num_sms()), stream);
+}
+
+void gemm_bf16_xielu(const void* x, const void* w, void* c, const float* coef, int M, int N, int K, long long ldx, long long ldw,
+                     long long ldc, const GemmWorkspace& ws, int sm_limit, cudaStream_t stream) {
+  if (M <= 0 || N <= 0 || K <= 0) return;
+  constexpr int BN = 256;
+  GemmParams p = prefill_params(c, M, N, K, ldc, ws);
+  p.coef = coef;
+  p.num_n = (N + BN - 1) / BN;
+  p.total_work = p.num_m * p.num_n;
+  launch_one<BN, 4, false, GLU_NONE, GF_XIELU>(make_tmap_bf16_2d(x, M, K, ldx, BM, BK), make_tmap_bf16_2d(w, N, K, ldw, BN, BK), p,
+                                               std::min(p.total_work, sm_limit > 0 ? sm_limit : gemm_num_sms()), stream);
 }
 
 void gemm_bf16_grouped(const void* x, const void* w, void* c, const int* plan, int rows, int groups, int max_tiles, int N,

@@ -66,6 +66,9 @@ void gemm_bf16_acc(const void* x, const void* w, float* y, int M, int N, int K, 
 // clamped_glu: w = [gate; up], c [M, width] = g sigmoid(1.702 g) (u + 1), g = min(gate, limit), u = up clamped to +-limit.
 void gemm_bf16_clamped_glu(const void* x, const void* w, void* c, int M, int width, int K, long long ldx, long long ldw,
                            long long ldc, float limit, const GemmWorkspace& ws, int sm_limit, cudaStream_t stream);
+// xielu: c [M, N] = xIELU of the product (see launch_xielu in hybrid.h).
+void gemm_bf16_xielu(const void* x, const void* w, void* c, const float* coef, int M, int N, int K, long long ldx, long long ldw,
+                     long long ldc, const GemmWorkspace& ws, int sm_limit, cudaStream_t stream);
 // grouped: rows of x sorted by group, w [groups, N, K]; `plan` (device): [groups + 1] first row of every group, [1] number
 // of 128-row tiles, then (group, first row) of every tile (at most max_tiles).  glu_kind -1: c [rows, N]; 0 silu, 1 clamped:
 // w[g] = [gate; up], c [rows, N / 2].

@@ -136,20 +136,19 @@ template <typename T>
 __device__ __forceinline__ float xielu_t(float z, float a, float b) {
   const float n = fminf(z, 0.f);
   float e;
-  if constexpr (sizeof(T) == 2) e = __expf(n) - 1.f - n;
-  else e = expm1f(n) - n;
-  if (n > -0.25f) e = n * n * (0.5f + n * (0.16666667f + n * (0.041666667f + n * (0.0083333333f + n * 0.0013888889f))));
+  if constexpr (sizeof(T) == 2) {
+    e = __expf(n) - 1.f - n;
+    if (n > -0.0625f) e = n * n * (0.5f + n * (0.16666667f + n * 0.041666667f));
+  } else {
+    e = expm1f(n) - n;
+    if (n > -0.25f) e = n * n * (0.5f + n * (0.16666667f + n * (0.041666667f + n * (0.0083333333f + n * 0.0013888889f))));
+  }
   return (z > 0.f ? a * z * z : b * e) + 0.5f * z;
 }
 
-// cos and sin of `position` times a frequency in turns, reduced in double
+// cos and sin of `position` times a frequency in turns: reduced in double, so that far positions lose nothing
 __device__ __forceinline__ void turn_angle(double pos, double freq, float& c, float& s) {
   const double turns = pos * freq;
-  sincospif(float(2.0 * (turns - rint(turns))), &s, &c);
-}
-// cos and sin of position * base^(-2 i / dims): the angle is reduced in double, so that far positions lose nothing
-__device__ __forceinline__ void rope_angle(double pos, double log2_base, int i, int dims, float& c, float& s) {
-  const double turns = pos * exp2(-log2_base * (2.0 * i / dims)) * 0.15915494309189535;   // 1 / (2 pi)
   sincospif(float(2.0 * (turns - rint(turns))), &s, &c);
 }
 

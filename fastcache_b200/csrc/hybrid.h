@@ -240,7 +240,7 @@ struct LatentStore {
   int off_q = 0, off_kv = -1, off_g = 0;       // off_kv < 0: no cache rows to write
   const float* norm_w = nullptr;
   float eps = 0.f;
-  double log2_base = 0.0;            // rotation: position * base^(-2 i / rot_dims)
+  const double* freq = nullptr;      // [rot_dims / 2] turns per position
   bool half = true;                  // entry i turns with i + rot_dims / 2 (else 2i with 2i + 1)
   const long long* positions = nullptr;
   const int* slots = nullptr;

@@ -147,6 +147,12 @@ Tensor linear_xielu(const Tensor& h, const Tensor& w, const Tensor& coef, int64_
   check_f32(coef, "xIELU coefficients", 2);
   TORCH_CHECK(N == wp, "bad width");
   Tensor hold, out = torch::empty({T, wp}, h.options());
+  if (w.numel() && !is_f32(h) && T > SMALL_ROWS) {           // prefill sizes: in the GEMM's epilogue (pad columns are zero anyway)
+    check_product(h, w);
+    fc::gemm_bf16_xielu(h.data_ptr(), w.data_ptr(), out.data_ptr(), coef.data_ptr<float>(), int(T), int(N), int(h.size(1)), h.stride(0),
+                        w.size(1), wp, gemm_workspace(ws_of(h)), fc::stream_sm_limit(stream_now()), stream_now());
+    return out;
+  }
   const fc::ProjSrc z = product(h, w, c10::nullopt, true, hold);
   fc::launch_xielu(z, coef.data_ptr<float>(), out.data_ptr(), int(T), int(width), int(wp), is_f32(h), stream_now());
   return out;
@@ -343,7 +349,7 @@ Tensor delta_rule(const Tensor& h, const Tensor& w, const Tensor& conv_w, const 
 // column per head.  With a latent, `q_norm` and `w_uq` make the queries from it (q's offset is unused).  impl: 0 choose, 1 the
 // forms without tensor cores, 2 absorbed also in prefill, 3 the same on mma.sync.  cu_kv, max_kv, total_kv: the rows that
 // prefill gathers (the last ones of every request, as many as the window needs)
-Tensor latent_attention(const Tensor& h, const Tensor& w, const std::vector<int64_t>& d, double scale, double base,
+Tensor latent_attention(const Tensor& h, const Tensor& w, const std::vector<int64_t>& d, double scale, const Tensor& freq,
                         const OptTensor& kv_norm, double eps, const Tensor& w_kv, int64_t off_uv, const Tensor& w_ukt,
                         const Tensor& w_uv, Tensor pool, const Tensor& positions, const OptTensor& slots,
                         const Tensor& block_tables, const Tensor& ctx, const OptTensor& cu_q, const OptTensor& cu_kv,
@@ -380,7 +386,9 @@ Tensor latent_attention(const Tensor& h, const Tensor& w, const std::vector<int6
   st.off_kv = int(d[7]);
   st.off_g = std::max(off_g, 0);
   st.eps = float(eps);
-  st.log2_base = std::log2(base);
+  TORCH_CHECK(freq.is_cuda() && freq.scalar_type() == torch::kFloat64 && freq.is_contiguous() && freq.numel() == rot_dims / 2,
+              "freq must be float64 [rotated dimensions / 2]");
+  st.freq = freq.data_ptr<double>();
   st.positions = reinterpret_cast<const long long*>(positions.data_ptr<int64_t>());
   st.pool = pool.data_ptr();
   st.row_width = int(pool.size(2));

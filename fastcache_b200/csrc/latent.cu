@@ -56,7 +56,7 @@ latent_store_kernel(const LatentStore p) {
   pdl_wait();
   const long long t = blockIdx.x;
   const double pos = double(p.positions[t]);
-  for (int i = threadIdx.x; i < half; i += LS_THREADS) rope_angle(pos, p.log2_base, i, p.rot_dims, cs[i], cs[half + i]);
+  for (int i = threadIdx.x; i < half; i += LS_THREADS) turn_angle(pos, p.freq[i], cs[i], cs[half + i]);
   __syncthreads();
   const int part = blockIdx.y, parts = gridDim.y;
   // queries: every (head, column) of this part
@@ -80,30 +80,143 @@ latent_store_kernel(const LatentStore p) {
   store_latent_row<T, LS_THREADS>(p, t, cs, red);
 }
 
-// Normed query latent, cache row and head gates of a token (the queries are made from the query latent afterwards)
+// The queries alone, four columns per access (sizes and offsets multiples of 4; where halves turn, half a rotated part as well)
 template <typename T>
 __global__ void __launch_bounds__(LS_THREADS)
-latent_inputs_kernel(const LatentStore p) {
-  __shared__ float red[LS_THREADS / 32];
+latent_queries_kernel(const LatentStore p) {
   extern __shared__ float cs[];
-  const int half = p.rot_dims / 2;
+  const int half = p.rot_dims / 2, Q = p.D + p.R, n = p.H * Q;
   pdl_launch_dependents();
   pdl_wait();
   const long long t = blockIdx.x;
+  const int idx = (blockIdx.y * LS_THREADS + threadIdx.x) * 4, h = idx / Q, c = idx - h * Q, r = c - p.D;
+  float4 v, o;
+  const bool on = idx < n, turn = on && r >= 0 && r < p.rot_dims;
+  if (on) v = proj_at4<T>(p.proj, t, p.off_q + idx);
+  if (turn && p.half) o = proj_at4<T>(p.proj, t, p.off_q + idx + (r < half ? half : -half));
   const double pos = double(p.positions[t]);
-  for (int i = threadIdx.x; i < half; i += LS_THREADS) rope_angle(pos, p.log2_base, i, p.rot_dims, cs[i], cs[half + i]);
-  float ss = 0.f;
-  for (int c = threadIdx.x; c < p.q_rank; c += LS_THREADS) {
-    const float v = proj_at<T>(p.proj, t, p.off_dq + c);
-    ss += v * v;
+  for (int i = threadIdx.x; i < half; i += LS_THREADS) turn_angle(pos, p.freq[i], cs[i], cs[half + i]);
+  __syncthreads();
+  if (!on) return;
+  if (turn && p.half) {
+    const int i = r < half ? r : r - half;
+    const float f = r < half ? -1.f : 1.f;
+    const float4 a = *reinterpret_cast<const float4*>(cs + i), b = *reinterpret_cast<const float4*>(cs + half + i);
+    v = make_float4(v.x * a.x + f * o.x * b.x, v.y * a.y + f * o.y * b.y, v.z * a.z + f * o.z * b.z, v.w * a.w + f * o.w * b.w);
+  } else if (turn) {
+    const float2 a = *reinterpret_cast<const float2*>(cs + r / 2), b = *reinterpret_cast<const float2*>(cs + half + r / 2);
+    v = make_float4(v.x * a.x - v.y * b.x, v.y * a.x + v.x * b.x, v.z * a.y - v.w * b.y, v.w * a.y + v.z * b.y);
   }
-  const float inv = rsqrtf(cta_sum<LS_THREADS>(ss, red) / float(p.q_rank) + p.eps);      // also makes cs visible
+  T* q = reinterpret_cast<T*>(p.q);
+  if (p.q_abs == nullptr) store4(q + t * n + idx, v.x, v.y, v.z, v.w);
+  else if (r < 0) store4(q + (t * p.H + h) * p.D + c, v.x, v.y, v.z, v.w);
+  else store4(reinterpret_cast<T*>(p.q_abs) + (t * p.H + h) * (p.rank + p.R) + p.rank + r, v.x, v.y, v.z, v.w);
+}
+static bool latent_queries_supported(const LatentStore& p) {
+  return p.off_kv < 0 && p.gate == nullptr && p.D % 4 == 0 && p.R % 4 == 0 && p.rank % 4 == 0 && p.off_q % 4 == 0 && p.rot_dims % 4 == 0 &&
+         (!p.half || p.rot_dims % 8 == 0);
+}
+
+// Normed query latent, cache row and head gates of a token (the queries are made from the query latent afterwards).  VEC: four
+// columns per access, everything read ahead of one barrier
+constexpr int LI_Q = 4, LI_KV = 1;                       // four-column pieces per thread: q_rank up to 4096, rank up to 1024
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(LS_THREADS)
+latent_inputs_kernel(const LatentStore p) {
+  __shared__ float2 red2[LS_THREADS / 32];
+  __shared__ float red[LS_THREADS / 32];
+  extern __shared__ float cs[];
+  const int half = p.rot_dims / 2, tid = threadIdx.x;
+  pdl_launch_dependents();
+  pdl_wait();
+  const long long t = blockIdx.x;
   T* cq = reinterpret_cast<T*>(p.cq) + t * p.ld_cq;
-  for (int c = threadIdx.x; c < p.ld_cq; c += LS_THREADS)
-    cq[c] = Elem<T>::put(c < p.q_rank ? proj_at<T>(p.proj, t, p.off_dq + c) * inv * p.q_norm_w[c] : 0.f);
-  if (p.head_gate != nullptr)
-    for (int h = threadIdx.x; h < p.H; h += LS_THREADS) p.head_gate[t * p.H + h] = sigmoid_f(proj_at<T>(p.proj, t, p.off_g + h));
-  if (p.off_kv >= 0) store_latent_row<T, LS_THREADS>(p, t, cs, red);
+  if constexpr (!VEC) {
+    const double pos = double(p.positions[t]);
+    for (int i = tid; i < half; i += LS_THREADS) turn_angle(pos, p.freq[i], cs[i], cs[half + i]);
+    float ss = 0.f;
+    for (int c = tid; c < p.q_rank; c += LS_THREADS) {
+      const float v = proj_at<T>(p.proj, t, p.off_dq + c);
+      ss += v * v;
+    }
+    const float inv = rsqrtf(cta_sum<LS_THREADS>(ss, red) / float(p.q_rank) + p.eps);      // also makes cs visible
+    for (int c = tid; c < p.ld_cq; c += LS_THREADS)
+      cq[c] = Elem<T>::put(c < p.q_rank ? proj_at<T>(p.proj, t, p.off_dq + c) * inv * p.q_norm_w[c] : 0.f);
+    if (p.head_gate != nullptr)
+      for (int h = tid; h < p.H; h += LS_THREADS) p.head_gate[t * p.H + h] = sigmoid_f(proj_at<T>(p.proj, t, p.off_g + h));
+    if (p.off_kv >= 0) store_latent_row<T, LS_THREADS>(p, t, cs, red);
+  } else {
+    float4 q[LI_Q], kv[LI_KV];
+    float sq = 0.f, sk = 0.f;
+#pragma unroll
+    for (int i = 0; i < LI_Q; ++i) {
+      const int c = (tid + i * LS_THREADS) * 4;
+      if (c < p.q_rank) q[i] = proj_at4<T>(p.proj, t, p.off_dq + c);
+    }
+#pragma unroll
+    for (int i = 0; i < LI_KV; ++i) {
+      const int c = (tid + i * LS_THREADS) * 4;
+      if (c < p.rank) kv[i] = proj_at4<T>(p.proj, t, p.off_kv + c);
+    }
+    // rotated part and gates by the last threads
+    const int lt = LS_THREADS - 1 - tid, slot = p.slots[t];
+    const bool turn = lt < half;
+    float u = 0.f, v = 0.f, c = 1.f, s = 0.f;
+    const int cu = p.half ? lt : 2 * lt, cv = p.half ? half + lt : 2 * lt + 1, rot = p.off_kv + p.rank;
+    if (turn) {
+      u = proj_at<T>(p.proj, t, rot + cu);
+      v = proj_at<T>(p.proj, t, rot + cv);
+      turn_angle(double(p.positions[t]), p.freq[lt], c, s);
+    }
+    if (p.head_gate != nullptr)
+      for (int h = tid; h < p.H; h += LS_THREADS) p.head_gate[t * p.H + h] = sigmoid_f(proj_at<T>(p.proj, t, p.off_g + h));
+#pragma unroll
+    for (int i = 0; i < LI_Q; ++i)
+      if ((tid + i * LS_THREADS) * 4 < p.q_rank) sq += q[i].x * q[i].x + q[i].y * q[i].y + q[i].z * q[i].z + q[i].w * q[i].w;
+#pragma unroll
+    for (int i = 0; i < LI_KV; ++i)
+      if ((tid + i * LS_THREADS) * 4 < p.rank) sk += kv[i].x * kv[i].x + kv[i].y * kv[i].y + kv[i].z * kv[i].z + kv[i].w * kv[i].w;
+    sq = warp_sum(sq);
+    sk = warp_sum(sk);
+    if ((tid & 31) == 0) red2[tid >> 5] = make_float2(sq, sk);
+    __syncthreads();
+    sq = sk = 0.f;
+#pragma unroll
+    for (int i = 0; i < LS_THREADS / 32; ++i) {
+      sq += red2[i].x;
+      sk += red2[i].y;
+    }
+    const float iq = rsqrtf(sq / float(p.q_rank) + p.eps), ik = rsqrtf(sk / float(p.rank) + p.eps);
+    auto put = [&](T* dst, const float4& x, const float* w, float inv) {
+      const float4 g = *reinterpret_cast<const float4*>(w);
+      store4(dst, x.x * inv * g.x, x.y * inv * g.y, x.z * inv * g.z, x.w * inv * g.w);
+    };
+#pragma unroll
+    for (int i = 0; i < LI_Q; ++i) {
+      const int at = (tid + i * LS_THREADS) * 4;
+      if (at < p.q_rank) put(cq + at, q[i], p.q_norm_w + at, iq);
+    }
+    for (int at = p.q_rank + tid; at < p.ld_cq; at += LS_THREADS) cq[at] = Elem<T>::put(0.f);
+    if (slot < 0) return;
+    if (slot >= p.num_rows) {
+      if (tid == 0) report(p.status, ST_BAD_INDEX);
+      return;
+    }
+    T* row = reinterpret_cast<T*>(p.pool) + (long long)slot * p.row_width;
+#pragma unroll
+    for (int i = 0; i < LI_KV; ++i) {
+      const int at = (tid + i * LS_THREADS) * 4;
+      if (at < p.rank) put(row + at, kv[i], p.norm_w + at, ik);
+    }
+    if (turn) {
+      row[p.rank + cu] = Elem<T>::put(u * c - v * s);
+      row[p.rank + cv] = Elem<T>::put(v * c + u * s);
+    }
+  }
+}
+static bool latent_inputs_vec(const LatentStore& p) {
+  return p.off_kv >= 0 && p.q_rank % 4 == 0 && p.q_rank <= LS_THREADS * 4 * LI_Q && p.rank % 4 == 0 && p.rank <= LS_THREADS * 4 * LI_KV &&
+         p.off_dq % 4 == 0 && p.off_kv % 4 == 0 && p.rot_dims == p.R && p.R <= 2 * LS_THREADS;
 }
 
 // The same for many rows of a finished projection whose queries are then read where they are: the rotated parts are
@@ -120,7 +233,7 @@ latent_rotate_kernel(const LatentStore p) {
   const long long t = blockIdx.x;
   const int tid = threadIdx.x, lane = tid & 31;
   const double pos = double(p.positions[t]);
-  for (int i = tid; i < half; i += LR_WARPS * 32) rope_angle(pos, p.log2_base, i, p.rot_dims, cs[i], cs[half + i]);
+  for (int i = tid; i < half; i += LR_WARPS * 32) turn_angle(pos, p.freq[i], cs[i], cs[half + i]);
   __syncthreads();
   T* row = const_cast<T*>(reinterpret_cast<const T*>(p.proj.p)) + t * p.proj.ld;
   auto rotate = [&](const T* su, T* du, int i0) {            // quads at columns i0 and half + i0 of a rotated part
@@ -174,8 +287,10 @@ bool latent_rotate_supported(const LatentStore& p) {
 void launch_latent_inputs(const LatentStore& p, bool f32, cudaStream_t s) {
   if (p.T == 0) return;
   const size_t smem = size_t(std::max(2, p.rot_dims)) * 4;
-  if (f32) launch_pdl(PDL_ROPE, latent_inputs_kernel<float>, dim3(p.T), dim3(LS_THREADS), smem, s, p);
-  else launch_pdl(PDL_ROPE, latent_inputs_kernel<bf16>, dim3(p.T), dim3(LS_THREADS), smem, s, p);
+  auto go = [&](auto kern) { launch_pdl(PDL_ROPE, kern, dim3(p.T), dim3(LS_THREADS), smem, s, p); };
+  const bool vec = latent_inputs_vec(p);
+  if (f32) vec ? go(latent_inputs_kernel<float, true>) : go(latent_inputs_kernel<float, false>);
+  else vec ? go(latent_inputs_kernel<bf16, true>) : go(latent_inputs_kernel<bf16, false>);
   const cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess) throw std::runtime_error(std::string("latent inputs: ") + cudaGetErrorString(e));
 }
@@ -192,6 +307,15 @@ void launch_latent_store(const LatentStore& p, bool f32, cudaStream_t s) {
     return;
   }
   const int work = p.H * (p.D + p.R);
+  if (latent_queries_supported(p)) {
+    const dim3 grid(p.T, (work + LS_THREADS * 4 - 1) / (LS_THREADS * 4));
+    const size_t smem = size_t(std::max(2, p.rot_dims)) * 4;
+    if (f32) launch_pdl(PDL_ROPE, latent_queries_kernel<float>, grid, dim3(LS_THREADS), smem, s, p);
+    else launch_pdl(PDL_ROPE, latent_queries_kernel<bf16>, grid, dim3(LS_THREADS), smem, s, p);
+    const cudaError_t e = cudaGetLastError();
+    if (e != cudaSuccess) throw std::runtime_error(std::string("latent store: ") + cudaGetErrorString(e));
+    return;
+  }
   const int parts = p.T >= 592 ? 1 : std::max(1, std::min(16, (work + LS_THREADS * 4 - 1) / (LS_THREADS * 4)));
   const dim3 grid(p.T, parts);
   const size_t smem = size_t(std::max(2, p.rot_dims)) * 4;

@@ -23,6 +23,7 @@
 #include "gemm.h"
 #include "hybrid.cuh"
 #include "launch.h"
+#include "one_lane.cuh"
 
 namespace fc {
 
@@ -50,39 +51,6 @@ __device__ __forceinline__ uint64_t lt_sdesc(uint32_t addr, uint32_t lbo_bytes, 
   d |= uint64_t(1) << 46;
   d |= uint64_t(2) << 61;
   return d;
-}
-
-// issue by one lane of a warp that is converged otherwise: loops and descriptors stay warp-uniform
-__device__ __forceinline__ void lt_mma(uint32_t tmem_d, uint64_t a, uint64_t b, uint32_t idesc, uint32_t accumulate,
-                                       uint32_t issue) {
-  asm volatile(
-      "{\n\t.reg .pred p, q;\n\t"
-      "setp.ne.b32 p, %4, 0;\n\tsetp.ne.b32 q, %5, 0;\n\t"
-      "@q tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t}"
-      ::"r"(tmem_d), "l"(a), "l"(b), "r"(idesc), "r"(accumulate), "r"(issue)
-      : "memory");
-}
-__device__ __forceinline__ void lt_commit(uint64_t* bar, uint32_t issue) {
-  asm volatile(
-      "{\n\t.reg .pred q;\n\tsetp.ne.b32 q, %1, 0;\n\t"
-      "@q tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];\n\t}"
-      ::"r"(smem_u32(bar)), "r"(issue)
-      : "memory");
-}
-
-__device__ __forceinline__ void lt_expect(uint64_t* bar, uint32_t bytes, uint32_t issue) {
-  asm volatile(
-      "{\n\t.reg .pred q;\n\tsetp.ne.b32 q, %2, 0;\n\t"
-      "@q mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;\n\t}"
-      ::"r"(smem_u32(bar)), "r"(bytes), "r"(issue)
-      : "memory");
-}
-__device__ __forceinline__ void lt_load(void* dst, const CUtensorMap* m, uint64_t* bar, int x, int y, uint32_t issue) {
-  asm volatile(
-      "{\n\t.reg .pred q;\n\tsetp.ne.b32 q, %5, 0;\n\t"
-      "@q cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4}], [%2];\n\t}"
-      ::"r"(smem_u32(dst)), "l"(reinterpret_cast<uint64_t>(m)), "r"(smem_u32(bar)), "r"(x), "r"(y), "r"(issue)
-      : "memory");
 }
 
 __global__ void __launch_bounds__(LT_THREADS, 1)
@@ -200,7 +168,7 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm, const RowAttn p,
         auto load = [&](uint8_t* dst, uint64_t* bar, int col) {
 #pragma unroll 1
           for (int pc = 0; pc < pieces; ++pc)
-            lt_load(dst + pc * box_rows * 128, &tm, bar, col, reinterpret_cast<volatile int*>(s_at)[pc], el);
+            one_load_2d(dst + pc * box_rows * 128, &tm, bar, col, reinterpret_cast<volatile int*>(s_at)[pc], el);
         };
         for (int i = 0; i < w.pairs; ++i) {
           const int col = w.shared || i < w.keys ? i * 128 : p.v_col + (i - w.keys) * 128;
@@ -209,7 +177,7 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm, const RowAttn p,
             ok = false;
             break;
           }
-          lt_expect(&full[slot], 2 * bytes, el);
+          one_expect(&full[slot], 2 * bytes, el);
           load(s_kv + slot * 2 * LT_SUB, &full[slot], col);
           load(s_kv + slot * 2 * LT_SUB + LT_SUB, &full[slot], col + 64);
           if (++slot == w.ring) {
@@ -224,7 +192,7 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm, const RowAttn p,
             ok = false;
             break;
           }
-          lt_expect(&x_full[x], bytes, el);
+          one_expect(&x_full[x], bytes, el);
           load(s_x + x * LT_SUB, &x_full[x], w.keys * 128);
         }
       }
@@ -259,7 +227,7 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm, const RowAttn p,
 #pragma unroll
         for (int kk = 0; kk < 4; ++kk)
           if (kk < left)
-            lt_mma(tm_s, da + uint64_t(kk * 2), dq + uint64_t(kk * 2), idesc_s, (sub > 0 || kk > 0) ? 1u : 0u, el);
+            one_mma(tm_s, da + uint64_t(kk * 2), dq + uint64_t(kk * 2), idesc_s, (sub > 0 || kk > 0) ? 1u : 0u, el);
       };
       auto issue_s = [&](int j) {
         const int x = j & 1;
@@ -269,7 +237,7 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm, const RowAttn p,
           const uint64_t da = d_rows + uint64_t(sl * (2 * LT_SUB >> 4));
           scores(tmem + LT_HEADS * uint32_t(x), da, i * 2);
           scores(tmem + LT_HEADS * uint32_t(x), da + uint64_t(LT_SUB >> 4), i * 2 + 1);
-          if (!w.shared) lt_commit(&empty[sl], el);
+          if (!w.shared) one_commit(&empty[sl], el);
           skip(sl, ph, 1);
         }
         skip(sl, ph, w.pairs - w.keys);
@@ -278,8 +246,8 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm, const RowAttn p,
           tc_fence_after();
           scores(tmem + LT_HEADS * uint32_t(x), d_x + uint64_t(x * (LT_SUB >> 4)), w.keys * 2);
         }
-        lt_commit(&s_full[x], el);
-        if (w.extra) lt_commit(&x_empty[x], el);
+        one_commit(&s_full[x], el);
+        if (w.extra) one_commit(&x_empty[x], el);
         return true;
       };
       bool ok = n_tiles == 0 || issue_s(0);
@@ -298,13 +266,13 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm, const RowAttn p,
           const uint32_t tm_o = tmem + LT_HEADS * uint32_t(2 + i);
 #pragma unroll
           for (int kk = 0; kk < LT_ROWS / 16; ++kk)
-            lt_mma(tm_o, dv + uint64_t(kk * 128), dp + uint64_t(kk * 2), idesc_o, (j > 0 || kk > 0) ? 1u : 0u, el);
-          lt_commit(&empty[slot], el);
+            one_mma(tm_o, dv + uint64_t(kk * 128), dp + uint64_t(kk * 2), idesc_o, (j > 0 || kk > 0) ? 1u : 0u, el);
+          one_commit(&empty[slot], el);
           skip(slot, pho, 1);
         }
         skip(slot, pho, w.pairs - w.values);
         if (!ok) break;
-        lt_commit(o_done, el);
+        one_commit(o_done, el);
         if (!w.ahead && j + 1 < n_tiles) ok = issue_s(j + 1);
       }
       if (!ok && lane == 0) *s_abort = 1;

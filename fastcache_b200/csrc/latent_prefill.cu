@@ -21,6 +21,7 @@
 
 #include "gemm.h"
 #include "hybrid.cuh"
+#include "one_lane.cuh"
 
 namespace fc {
 
@@ -116,91 +117,94 @@ latent_prefill_kernel(const __grid_constant__ LpMaps tm, const LpParams p) {
 
   if (warp == 0) {
     // ------------------------------------------------------------------ TMA loader
-    if (lane == 0) {
-      auto load_q = [&](uint8_t* dst, uint64_t* bar, int i) {
-        if (i < p.nd) tma_load_3d(dst, &tm.qn, bar, i * 64, h, q_begin + q0);
-        else tma_load_3d(dst, &tm.qr, bar, (i - p.nd) * 64, h, q_begin + q0);
-      };
-      if (!STREAM_Q) {
-        mbar_expect_tx(q_full, uint32_t(nq) * LP_SUB);
-        for (int i = 0; i < nq; ++i) load_q(s_q + i * LP_SUB, q_full, i);
-      }
-      int slot = 0;
-      uint32_t phase = 1;
-      bool ok = true;
-      for (int j = 0; j < n_tiles && ok && !*s_abort; ++j) {
-        const int row = kv_begin + (tile0 + j) * LP_BN;
-        for (int i = 0; i < nq; ++i) {
-          ok = mbar_wait(&k_empty[slot], phase, p.status, ST_TIMEOUT_EMPTY);
-          if (!ok) break;
-          uint8_t* dk = s_k + slot * SLOT;
-          mbar_expect_tx(&k_full[slot], SLOT);
-          if (i < p.nd) tma_load_3d(dk, &tm.kn, &k_full[slot], i * 64, h, row);
-          else tma_load_2d(dk, &tm.kr, &k_full[slot], (i - p.nd) * 64, row);
-          if (STREAM_Q) load_q(dk + LP_SUB, &k_full[slot], i);
-          if (++slot == p.ring) {
-            slot = 0;
-            phase ^= 1;
-          }
-        }
-        if (!ok) break;
-        const int st = p.v_stages == 2 ? j & 1 : 0;
-        const uint32_t use = uint32_t(p.v_stages == 2 ? j >> 1 : j) & 1u;
-        ok = mbar_wait(&v_empty[st], use ^ 1u, p.status, ST_TIMEOUT_EMPTY);
-        if (!ok) break;
-        mbar_expect_tx(&v_full[st], V_BYTES);
-#pragma unroll
-        for (int s = 0; s < NV; ++s) tma_load_3d(s_v + st * V_BYTES + s * LP_SUB, &tm.v, &v_full[st], s * 64, h / p.heads_per_value, row);
-      }
-      if (!ok) *s_abort = 1;
+    const uint32_t el = elect_one() ? 1u : 0u;
+    auto load_q = [&](uint8_t* dst, uint64_t* bar, int i) {
+      if (i < p.nd) one_load_3d(dst, &tm.qn, bar, i * 64, h, q_begin + q0, el);
+      else one_load_3d(dst, &tm.qr, bar, (i - p.nd) * 64, h, q_begin + q0, el);
+    };
+    if (!STREAM_Q) {
+      one_expect(q_full, uint32_t(nq) * LP_SUB, el);
+      for (int i = 0; i < nq; ++i) load_q(s_q + i * LP_SUB, q_full, i);
     }
+    const int hv = h / p.heads_per_value;
+    int slot = 0;
+    uint32_t phase = 1;
+    bool ok = true;
+    for (int j = 0; j < n_tiles && ok; ++j) {
+      const int row = kv_begin + (tile0 + j) * LP_BN;
+      ok = !__any_sync(0xffffffffu, *s_abort != 0);
+      for (int i = 0; i < nq && ok; ++i) {
+        ok = warp_wait(&k_empty[slot], phase, p.status, ST_TIMEOUT_EMPTY);
+        if (!ok) break;
+        uint8_t* dk = s_k + slot * SLOT;
+        one_expect(&k_full[slot], SLOT, el);
+        if (i < p.nd) one_load_3d(dk, &tm.kn, &k_full[slot], i * 64, h, row, el);
+        else one_load_2d(dk, &tm.kr, &k_full[slot], (i - p.nd) * 64, row, el);
+        if (STREAM_Q) load_q(dk + LP_SUB, &k_full[slot], i);
+        if (++slot == p.ring) {
+          slot = 0;
+          phase ^= 1;
+        }
+      }
+      if (!ok) break;
+      const int st = p.v_stages == 2 ? j & 1 : 0;
+      const uint32_t use = uint32_t(p.v_stages == 2 ? j >> 1 : j) & 1u;
+      ok = warp_wait(&v_empty[st], use ^ 1u, p.status, ST_TIMEOUT_EMPTY);
+      if (!ok) break;
+      one_expect(&v_full[st], V_BYTES, el);
+#pragma unroll
+      for (int s = 0; s < NV; ++s) one_load_3d(s_v + st * V_BYTES + s * LP_SUB, &tm.v, &v_full[st], s * 64, hv, row, el);
+    }
+    if (!ok && lane == 0) *s_abort = 1;
   } else if (warp == 1) {
     // ------------------------------------------------------------------ MMA issuer
-    if (lane == 0) {
-      constexpr uint32_t idesc_s = make_idesc_bf16(128, 128, false, false);
-      constexpr uint32_t idesc_o = make_idesc_bf16(128, NV * 64, false, true);     // B (= V) is MN-major
-      int slot = 0;
-      uint32_t phase = 0;
-      auto issue_s = [&](int j) {
-        const int x = j & 1;
-        for (int i = 0; i < nq; ++i) {
-          if (!mbar_wait(&k_full[slot], phase, p.status, ST_TIMEOUT_FULL)) return false;
-          tc_fence_after();
-          const uint32_t ka = smem_u32(s_k + slot * SLOT), qa = STREAM_Q ? ka + LP_SUB : smem_u32(s_q + i * LP_SUB);
-          const int left = i < p.nd ? p.D - i * 64 : p.R - (i - p.nd) * 64, steps = min(4, (left + 15) / 16);
-          for (int kk = 0; kk < steps; ++kk)
-            tc_mma_f16(tmem_base + uint32_t(x * 128), lp_sdesc(qa + uint32_t(kk) * 32, 16, 1024),
-                       lp_sdesc(ka + uint32_t(kk) * 32, 16, 1024), idesc_s, (i > 0 || kk > 0) ? 1u : 0u);
-          tc_commit(&k_empty[slot]);
-          if (++slot == p.ring) {
-            slot = 0;
-            phase ^= 1;
-          }
-        }
-        tc_commit(&s_full[x]);
-        return true;
-      };
-      bool ok = STREAM_Q || mbar_wait(q_full, 0, p.status, ST_TIMEOUT_FULL);
-      if (ok) ok = issue_s(0);
-      if (ok && n_tiles > 1) ok = issue_s(1);
-      for (int j = 0; j < n_tiles && ok; ++j) {
-        const int x = j & 1;
-        const int st = p.v_stages == 2 ? x : 0;
-        ok = mbar_wait(&p_ready[x], uint32_t(j >> 1) & 1u, p.status, ST_TIMEOUT_FULL) &&
-             mbar_wait(&v_full[st], uint32_t(p.v_stages == 2 ? j >> 1 : j) & 1u, p.status, ST_TIMEOUT_FULL);
-        if (!ok) break;
+    const uint32_t el = elect_one() ? 1u : 0u;
+    constexpr uint32_t idesc_s = make_idesc_bf16(128, 128, false, false);
+    constexpr uint32_t idesc_o = make_idesc_bf16(128, NV * 64, false, true);     // B (= V) is MN-major
+    // descriptors by addition on their address field (16-byte units)
+    const uint64_t d_k = lp_sdesc(smem_u32(s_k), 16, 1024), d_q = lp_sdesc(smem_u32(s_q), 16, 1024);
+    const uint64_t d_v = lp_sdesc(smem_u32(s_v), LP_SUB, 1024);
+    int slot = 0;
+    uint32_t phase = 0;
+    auto issue_s = [&](int j) {
+      const uint32_t ts = tmem_base + uint32_t(j & 1) * 128u;
+      for (int i = 0; i < nq; ++i) {
+        if (!warp_wait(&k_full[slot], phase, p.status, ST_TIMEOUT_FULL)) return false;
         tc_fence_after();
-        const uint32_t va = smem_u32(s_v + st * V_BYTES);
+        const uint64_t dk = d_k + uint64_t(slot * (SLOT >> 4)), dq = STREAM_Q ? dk + uint64_t(LP_SUB >> 4) : d_q + uint64_t(i * (LP_SUB >> 4));
+        const int left = i < p.nd ? p.D - i * 64 : p.R - (i - p.nd) * 64;
 #pragma unroll
-        for (int kk = 0; kk < 8; ++kk)
-          tc_mma_f16_ts(tmem_base + 256u + uint32_t(x * 128), tmem_base + uint32_t(x * 128) + uint32_t(kk * 8),
-                        lp_sdesc(va + uint32_t(kk) * 2048, LP_SUB, 1024), idesc_o, (j > 1 || kk > 0) ? 1u : 0u);
-        tc_commit(&o_done[x]);
-        tc_commit(&v_empty[st]);
-        if (j + 2 < n_tiles) ok = issue_s(j + 2);
+        for (int kk = 0; kk < 4; ++kk)
+          if (kk * 16 < left)
+            one_mma(ts, dq + uint64_t(kk * 2), dk + uint64_t(kk * 2), idesc_s, (i > 0 || kk > 0) ? 1u : 0u, el);
+        one_commit(&k_empty[slot], el);
+        if (++slot == p.ring) {
+          slot = 0;
+          phase ^= 1;
+        }
       }
-      if (!ok) *s_abort = 1;
+      one_commit(&s_full[j & 1], el);
+      return true;
+    };
+    bool ok = STREAM_Q || warp_wait(q_full, 0, p.status, ST_TIMEOUT_FULL);
+    if (ok) ok = issue_s(0);
+    if (ok && n_tiles > 1) ok = issue_s(1);
+    for (int j = 0; j < n_tiles && ok; ++j) {
+      const int x = j & 1, st = p.v_stages == 2 ? x : 0;
+      ok = warp_wait(&p_ready[x], uint32_t(j >> 1) & 1u, p.status, ST_TIMEOUT_FULL) &&
+           warp_wait(&v_full[st], uint32_t(p.v_stages == 2 ? j >> 1 : j) & 1u, p.status, ST_TIMEOUT_FULL);
+      if (!ok) break;
+      tc_fence_after();
+      const uint64_t dv = d_v + uint64_t(st * (V_BYTES >> 4));
+#pragma unroll
+      for (int kk = 0; kk < 8; ++kk)
+        one_mma_ts(tmem_base + 256u + uint32_t(x * 128), tmem_base + uint32_t(x * 128) + uint32_t(kk * 8), dv + uint64_t(kk * 128), idesc_o,
+                   (j > 1 || kk > 0) ? 1u : 0u, el);
+      one_commit(&o_done[x], el);
+      one_commit(&v_empty[st], el);
+      if (j + 2 < n_tiles) ok = issue_s(j + 2);
     }
+    if (!ok && lane == 0) *s_abort = 1;
   } else {
     // ------------------------------------------------ softmax of the even (x = 0) or odd (x = 1) key tiles
     const int x = (warp - 2) >> 2;

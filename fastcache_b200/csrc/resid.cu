@@ -34,92 +34,103 @@ embed_scaled_kernel(const long long* __restrict__ ids, const T* __restrict__ wei
 }
 
 // x += rms(f (y + bias) + mixed expert rows) * w;  h = x in the model's type, zero-padded from W to Wp columns.  NC: 4-column
-// chunks per thread
+// chunks per thread.  What does not depend on the norm is requested first
+constexpr int PN_THREADS = 512, PN_TOP = 4;
 template <typename T, bool VEC, int NC>
-__global__ void __launch_bounds__(RS_THREADS)
+__global__ void __launch_bounds__(PN_THREADS)
 post_norm_add_kernel(const PostNormAdd p) {
-  __shared__ float red[RS_THREADS / 32];
+  __shared__ float red[PN_THREADS / 32];
   pdl_launch_dependents();
   pdl_wait();
   const long long row = blockIdx.x;
   const int W = p.W;
   const T* bias = reinterpret_cast<const T*>(p.bias);
-  auto col_of = [&](int c) { return (int(threadIdx.x) + c * RS_THREADS) * 4; };
-  float v[NC][4];
+  float* x = p.x + row * W;
+  T* h = reinterpret_cast<T*>(p.h) + row * p.Wp;
+  auto col_of = [&](int c) { return (int(threadIdx.x) + c * PN_THREADS) * 4; };
+  int r[PN_TOP];
+  float f[PN_TOP];
+#pragma unroll
+  for (int j = 0; j < PN_TOP; ++j) {
+    r[j] = j < p.top ? p.row_of[row * p.top + j] : -1;
+    f[j] = j >= p.top ? 0.f : p.mix != nullptr ? p.mix[row * p.top + j] : 1.f / float(p.top);
+  }
+  const float fy = p.y_factor != nullptr ? p.y_factor[row] : 1.f;
+  float4 xv[NC], v[NC];
 #pragma unroll
   for (int c = 0; c < NC; ++c) {
     const int col = col_of(c);
-    v[c][0] = v[c][1] = v[c][2] = v[c][3] = 0.f;
-    if (col >= W || !p.has_y) continue;
-    const float4 a = proj_at4<T>(p.y, row, col);         // the pad columns of a projection exist and are zero
-    v[c][0] = a.x;
-    v[c][1] = a.y;
-    v[c][2] = a.z;
-    v[c][3] = a.w;
-    if (bias != nullptr)
-#pragma unroll
-      for (int i = 0; i < 4; ++i)
-        if (VEC || col + i < W) v[c][i] += Elem<T>::get(bias[col + i]);
+    v[c] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (col >= W) continue;
+    if (VEC) xv[c] = __ldcg(reinterpret_cast<const float4*>(x + col));
+    if (p.has_y) v[c] = proj_at4<T>(p.y, row, col);      // the pad columns of a projection exist and are zero
   }
-  if (p.y_factor != nullptr) {
-    const float f = p.y_factor[row];
-#pragma unroll
-    for (int c = 0; c < NC; ++c)
-#pragma unroll
-      for (int i = 0; i < 4; ++i) v[c][i] *= f;
-  }
-  for (int j = 0; j < p.top; ++j) {
-    const int r = p.row_of[row * p.top + j];
-    if (r < 0) continue;
-    const float f = p.mix != nullptr ? p.mix[row * p.top + j] : 1.f / float(p.top);
+  auto add = [&](int rj, float fj) {
+    if (rj < 0) return;
     float4 e[NC];
 #pragma unroll
     for (int c = 0; c < NC; ++c)
-      if (col_of(c) < W) e[c] = proj_at4<T>(p.experts, r, col_of(c));
+      if (col_of(c) < W) e[c] = proj_at4<T>(p.experts, rj, col_of(c));
 #pragma unroll
     for (int c = 0; c < NC; ++c)
       if (col_of(c) < W) {
-        v[c][0] = fmaf(e[c].x, f, v[c][0]);
-        v[c][1] = fmaf(e[c].y, f, v[c][1]);
-        v[c][2] = fmaf(e[c].z, f, v[c][2]);
-        v[c][3] = fmaf(e[c].w, f, v[c][3]);
+        v[c].x = fmaf(e[c].x, fj, v[c].x);
+        v[c].y = fmaf(e[c].y, fj, v[c].y);
+        v[c].z = fmaf(e[c].z, fj, v[c].z);
+        v[c].w = fmaf(e[c].w, fj, v[c].w);
       }
+  };
+#pragma unroll
+  for (int c = 0; c < NC; ++c) {
+    const int col = col_of(c);
+    if (bias != nullptr && col < W) {
+      v[c].x += Elem<T>::get(bias[col]);
+      if (VEC || col + 1 < W) v[c].y += Elem<T>::get(bias[col + 1]);
+      if (VEC || col + 2 < W) v[c].z += Elem<T>::get(bias[col + 2]);
+      if (VEC || col + 3 < W) v[c].w += Elem<T>::get(bias[col + 3]);
+    }
+    v[c].x *= fy;
+    v[c].y *= fy;
+    v[c].z *= fy;
+    v[c].w *= fy;
   }
+#pragma unroll
+  for (int j = 0; j < PN_TOP; ++j) add(r[j], f[j]);
+  for (int j = PN_TOP; j < p.top; ++j) add(p.row_of[row * p.top + j], p.mix != nullptr ? p.mix[row * p.top + j] : 1.f / float(p.top));
   float ss = 0.f;
 #pragma unroll
-  for (int c = 0; c < NC; ++c)
-#pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      if (!VEC && col_of(c) + i >= W) v[c][i] = 0.f;
-      ss += v[c][i] * v[c][i];
+  for (int c = 0; c < NC; ++c) {
+    if (!VEC) {
+      const int col = col_of(c);
+      if (col + 1 >= W) v[c].y = 0.f;
+      if (col + 2 >= W) v[c].z = 0.f;
+      if (col + 3 >= W) v[c].w = 0.f;
     }
-  const float inv = rsqrtf(cta_sum<RS_THREADS>(ss, red) / float(W) + p.eps);
-  float* x = p.x + row * W;
-  T* h = reinterpret_cast<T*>(p.h) + row * p.Wp;
+    ss += v[c].x * v[c].x + v[c].y * v[c].y + v[c].z * v[c].z + v[c].w * v[c].w;
+  }
+  const float inv = rsqrtf(cta_sum<PN_THREADS>(ss, red) / float(W) + p.eps);
 #pragma unroll
   for (int c = 0; c < NC; ++c) {
     const int col = col_of(c);
     if (col >= W) continue;
     if (VEC) {
-      float4 xv = *reinterpret_cast<const float4*>(x + col);
-      const float4 wv = *reinterpret_cast<const float4*>(p.w + col);
-      xv.x += v[c][0] * inv * wv.x;
-      xv.y += v[c][1] * inv * wv.y;
-      xv.z += v[c][2] * inv * wv.z;
-      xv.w += v[c][3] * inv * wv.w;
-      *reinterpret_cast<float4*>(x + col) = xv;
-      store4(h + col, xv.x, xv.y, xv.z, xv.w);
+      const float4 w = *reinterpret_cast<const float4*>(p.w + col);
+      const float4 n = make_float4(xv[c].x + v[c].x * inv * w.x, xv[c].y + v[c].y * inv * w.y, xv[c].z + v[c].z * inv * w.z,
+                                   xv[c].w + v[c].w * inv * w.w);
+      *reinterpret_cast<float4*>(x + col) = n;
+      store4(h + col, n.x, n.y, n.z, n.w);
     } else {
+      const float a[4] = {v[c].x, v[c].y, v[c].z, v[c].w};
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
         if (col + i >= W) break;
-        const float n = x[col + i] + v[c][i] * inv * p.w[col + i];
+        const float n = x[col + i] + a[i] * inv * p.w[col + i];
         x[col + i] = n;
         h[col + i] = Elem<T>::put(n);
       }
     }
   }
-  for (int c = W + threadIdx.x; c < p.Wp; c += RS_THREADS) h[c] = Elem<T>::put(0.f);
+  for (int c = W + threadIdx.x; c < p.Wp; c += PN_THREADS) h[c] = Elem<T>::put(0.f);
 }
 
 // x (+)= y + mixed expert rows;  h = rms(x) * w (or x) in the model's type, zero-padded from W to Wp columns.  NC: 4-column
@@ -314,20 +325,19 @@ void launch_embed_scaled(const void* ids, const void* weight, float* x, void* h,
 
 void launch_post_norm_add(const PostNormAdd& p, bool f32, cudaStream_t s) {
   if (p.T == 0) return;
-  if (p.W > RS_THREADS * RS_CHUNKS * 4) throw std::runtime_error("norm rows are limited to 8192 columns");
-  auto go = [&](auto kern) { launch_pdl(PDL_NORM, kern, dim3(p.T), dim3(RS_THREADS), 0, s, p); };
-  const int chunks = (p.W + RS_THREADS * 4 - 1) / (RS_THREADS * 4);
+  if (p.W > PN_THREADS * 16) throw std::runtime_error("norm rows are limited to 8192 columns");
+  auto go = [&](auto kern) { launch_pdl(PDL_NORM, kern, dim3(p.T), dim3(PN_THREADS), 0, s, p); };
   if (p.W % 4 != 0) {
-    if (f32) go(post_norm_add_kernel<float, false, RS_CHUNKS>);
-    else go(post_norm_add_kernel<bf16, false, RS_CHUNKS>);
+    if (f32) go(post_norm_add_kernel<float, false, 4>);
+    else go(post_norm_add_kernel<bf16, false, 4>);
   } else if (f32) {
-    go(post_norm_add_kernel<float, true, RS_CHUNKS>);
-  } else if (chunks <= 2) {
+    go(post_norm_add_kernel<float, true, 4>);
+  } else if (p.W <= PN_THREADS * 4) {
+    go(post_norm_add_kernel<bf16, true, 1>);
+  } else if (p.W <= PN_THREADS * 8) {
     go(post_norm_add_kernel<bf16, true, 2>);
-  } else if (chunks <= 4) {
-    go(post_norm_add_kernel<bf16, true, 4>);
   } else {
-    go(post_norm_add_kernel<bf16, true, RS_CHUNKS>);
+    go(post_norm_add_kernel<bf16, true, 4>);
   }
   check_launch("norm + add");
 }

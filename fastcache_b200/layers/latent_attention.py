@@ -51,8 +51,10 @@ class LatentAttention(nn.Module):
         self.kv_proj = PackedLinear(kv_rank, {"uk": heads * dim, "uv": heads * vdim})
         self.o_proj = PackedLinear(heads * vdim, {"o": width})
         o = self.in_proj.offset
-        self.dims = LatentDims(heads, dim, rot_dim, vdim, kv_rank, float(scale), float(rope_base), rope_dims,
+        self.dims = LatentDims(heads, dim, rot_dim, vdim, kv_rank, float(scale), rope_dims,
                                o.get("q", 0), o["g"], o.get("dkv"), o.get("dq"), q_rank, int(window), half, head_gate)
+        freq = ops.hybrid.rope_turns(rope_base, rope_dims)
+        self.register_buffer("freq", freq.to(self.o_proj.weight.device), persistent=False)
         self.row_width = pad8(kv_rank + rot_dim) if owner is None else 0
         self.rows: Optional[torch.Tensor] = None            # [blocks, block, row_width], bound by the runner
         self.w_ukt: Optional[torch.Tensor] = None
@@ -74,6 +76,6 @@ class LatentAttention(nn.Module):
         rows = self.rows if owner is None else owner.rows
         if rows is None:
             raise RuntimeError("latent attention used before its cache rows were bound")
-        return ops.hybrid.latent_attention(h, self.in_proj.weight, self.dims, self.kv_norm, self.eps,
+        return ops.hybrid.latent_attention(h, self.in_proj.weight, self.dims, self.freq, self.kv_norm, self.eps,
                                            self.kv_proj, self.w_ukt, self.w_uv, rows, positions, get_context(), self.q_norm,
                                            None if self.q_proj is None else self.q_proj.weight, self.sink)

@@ -66,7 +66,6 @@ class LatentDims:
     vdim: int
     rank: int
     scale: float
-    base: float
     rot_dims: int
     q: int
     g: Optional[int]
@@ -254,10 +253,10 @@ def _run_args(ctx):
 
 
 # ------------------------------------------------------------------ latent attention
-def latent_attention(h, weight, d: LatentDims, kv_norm_w, eps: float, kv_proj, w_ukt, w_uv, pool, positions, ctx, q_norm_w=None,
+def latent_attention(h, weight, d: LatentDims, freq, kv_norm_w, eps: float, kv_proj, w_ukt, w_uv, pool, positions, ctx, q_norm_w=None,
                      q_weight=None, sink=None):
     """Projections, cache store, attention and output gate of a latent-attention layer up to the output projection.
-    `q_norm_w`, `q_weight`: norm and projection of the queries' latent; `sink` [H] joins the softmax without a key.
+    `freq`: rope_turns; `q_norm_w`, `q_weight`: norm and projection of the queries' latent; `sink` [H] joins the softmax without a key.
 
     `kv_proj` (packed uk | uv) expands cache rows to keys and values (prefill); `w_ukt` [H, rank, dim] and `w_uv`
     [H, vdim, rank] are the same weights for the absorbed form (decode), which never expands a row."""
@@ -265,12 +264,12 @@ def latent_attention(h, weight, d: LatentDims, kv_norm_w, eps: float, kv_proj, w
         _n(6)
         cu_kv, max_kv, total_kv = ctx.kv_span(d.window)
         return ext().latent_attention(
-            h, weight, d.sizes(), d.scale, d.base, kv_norm_w, float(eps), kv_proj.weight, kv_proj.offset["uv"], w_ukt, w_uv, pool,
+            h, weight, d.sizes(), d.scale, freq, kv_norm_w, float(eps), kv_proj.weight, kv_proj.offset["uv"], w_ukt, w_uv, pool,
             positions, ctx.slot_mapping, ctx.block_tables, ctx.context_lens, ctx.cu_seqlens_q, cu_kv, ctx.row_seq, ctx.row_ctx,
             int(ctx.max_seqlen_q), int(ctx.max_seqlen_k), max_kv, total_kv, q_norm_w, q_weight, sink, LATENT_IMPL)
     p = ref_linear(h, weight)
     q_in = p[:, d.q:] if d.dq is None else ref_linear(ref.latent_of_queries(p, d, q_norm_w, eps, q_weight.shape[1]), q_weight)
-    q = ref.latent_project(p, q_in, d, kv_norm_w, eps, positions, pool, ctx.slot_mapping)
+    q = ref.latent_project(p, q_in, d, freq, kv_norm_w, eps, positions, pool, ctx.slot_mapping)
     w, off = kv_proj.weight, kv_proj.offset
     gate = None if d.g is None else p[:, d.g:d.g + d.heads * (1 if d.head_gate else d.vdim)]
     return ref.latent_attention(q, gate, d, w[off["uk"]:off["uk"] + d.heads * d.dim],

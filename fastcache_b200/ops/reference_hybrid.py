@@ -158,12 +158,10 @@ def latent_of_queries(p, d, norm_w, eps: float, width: int):
     return _pad_to(c.to(p.dtype), width)
 
 
-def latent_project(p, q_in, d, norm_w, eps: float, positions, pool, slots):
+def latent_project(p, q_in, d, turns, norm_w, eps: float, positions, pool, slots):
     """Writes the cache rows (normed latent | rotated shared key part) of a layer that owns a cache and returns the
     queries (first columns of `q_in`) with their rotated part rotated, [T, H, dim + rot]."""
     T = p.shape[0]
-    i = torch.arange(d.rot_dims // 2, dtype=torch.float64, device=p.device)
-    turns = d.base ** (-2 * i / max(1, d.rot_dims)) / (2 * math.pi)
 
     def turned(x):
         return rope_rows(x, positions, turns, d.rot_dims, d.half, 1.0).to(x.dtype)
