@@ -387,6 +387,7 @@ static void launch_lp(const LpMaps& tm, const LpParams& q, const LatentPrefill& 
 
 void launch_latent_prefill(const LatentPrefill& p, cudaStream_t s) {
   if (p.T == 0 || p.B == 0 || p.max_q == 0) return;
+  if (paired_prefill_supported(p)) return launch_paired_prefill(p, s);
   LpMaps tm;
   const uint64_t Q = uint64_t(p.D + p.R);
   const int vh = p.v_heads > 0 ? p.v_heads : p.H;

@@ -133,6 +133,115 @@ post_norm_add_kernel(const PostNormAdd p) {
   for (int c = W + threadIdx.x; c < p.Wp; c += PN_THREADS) h[c] = Elem<T>::put(0.f);
 }
 
+// The same for many rows of finished projections (bf16, W a multiple of 4, at most TOP expert rows per token): a CTA walks rows
+// and has the next one's loads in flight while it norms and writes this one
+template <int NC, int TOP>
+__global__ void __launch_bounds__(PN_THREADS, NC <= 2 ? 2 : 1)
+post_norm_rows_kernel(const PostNormAdd p) {
+  constexpr int E = TOP > 0 ? TOP : 1;
+  __shared__ float red[2][PN_THREADS / 32];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int W = p.W, tid = threadIdx.x, step = gridDim.x;
+  auto col_of = [&](int c) { return (tid + c * PN_THREADS) * 4; };
+  const bf16 *y = reinterpret_cast<const bf16*>(p.y.p), *ey = reinterpret_cast<const bf16*>(p.experts.p);
+  uint2 y4[NC], e4[E][NC];
+  float4 x4[NC];
+  int r[E];
+  float f[E], fn[E], fy = 1.f;                               // factors of this row; of the next one
+  auto index = [&](int row) {
+#pragma unroll
+    for (int j = 0; j < TOP; ++j) {
+      const bool on = row < p.T && j < p.top;
+      r[j] = on ? p.row_of[row * p.top + j] : -1;
+      fn[j] = !on ? 0.f : p.mix != nullptr ? p.mix[row * p.top + j] : 1.f / float(p.top);
+    }
+  };
+  auto request = [&](int row) {                              // index(row) is there
+#pragma unroll
+    for (int c = 0; c < NC; ++c) {
+      const int col = col_of(c);
+      if (col >= W) continue;
+      y4[c] = __ldcg(reinterpret_cast<const uint2*>(y + row * p.y.ld + col));
+      x4[c] = __ldcg(reinterpret_cast<const float4*>(p.x + (long long)row * W + col));
+#pragma unroll
+      for (int j = 0; j < TOP; ++j)
+        e4[j][c] = r[j] >= 0 ? __ldcg(reinterpret_cast<const uint2*>(ey + r[j] * p.experts.ld + col)) : make_uint2(0, 0);
+    }
+    if (p.y_factor != nullptr) fy = p.y_factor[row];
+#pragma unroll
+    for (int j = 0; j < TOP; ++j) f[j] = fn[j];
+  };
+  auto wide = [](const uint2& u) {
+    return make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xffff0000u), __uint_as_float(u.y << 16),
+                       __uint_as_float(u.y & 0xffff0000u));
+  };
+  int row = blockIdx.x;
+  index(row);
+  if (row < p.T) request(row);
+  index(row + step);
+  for (int par = 0; row < p.T; row += step, par ^= 1) {
+    float4 v[NC], x[NC];
+    float ss = 0.f;
+#pragma unroll
+    for (int c = 0; c < NC; ++c) {
+      v[c] = x[c] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (col_of(c) >= W) continue;
+      const float4 a = wide(y4[c]);
+      v[c] = make_float4(a.x * fy, a.y * fy, a.z * fy, a.w * fy);
+#pragma unroll
+      for (int j = 0; j < TOP; ++j) {
+        const float4 e = wide(e4[j][c]);
+        v[c].x = fmaf(e.x, f[j], v[c].x);
+        v[c].y = fmaf(e.y, f[j], v[c].y);
+        v[c].z = fmaf(e.z, f[j], v[c].z);
+        v[c].w = fmaf(e.w, f[j], v[c].w);
+      }
+      x[c] = x4[c];
+      ss += v[c].x * v[c].x + v[c].y * v[c].y + v[c].z * v[c].z + v[c].w * v[c].w;
+    }
+    if (row + step < p.T) {
+      request(row + step);
+      index(row + 2 * step);
+    }
+    ss = warp_sum(ss);
+    if ((tid & 31) == 0) red[par][tid >> 5] = ss;
+    __syncthreads();
+    ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < PN_THREADS / 32; ++i) ss += red[par][i];
+    const float inv = rsqrtf(ss / float(W) + p.eps);
+#pragma unroll
+    for (int c = 0; c < NC; ++c) {
+      const int col = col_of(c);
+      if (col >= W) continue;
+      const float4 w = *reinterpret_cast<const float4*>(p.w + col);
+      const float4 n = make_float4(x[c].x + v[c].x * inv * w.x, x[c].y + v[c].y * inv * w.y, x[c].z + v[c].z * inv * w.z,
+                                   x[c].w + v[c].w * inv * w.w);
+      *reinterpret_cast<float4*>(p.x + (long long)row * W + col) = n;
+      store4(reinterpret_cast<bf16*>(p.h) + (long long)row * p.Wp + col, n.x, n.y, n.z, n.w);
+    }
+    if (tid < p.Wp - W) reinterpret_cast<bf16*>(p.h)[(long long)row * p.Wp + W + tid] = __float2bfloat16(0.f);
+  }
+}
+static bool post_norm_rows(const PostNormAdd& p, cudaStream_t s) {
+  if (p.T < 1024 || p.W % 4 != 0 || !p.has_y || p.y.part != nullptr || p.bias != nullptr || p.top > 4 ||
+      (p.top > 0 && p.experts.part != nullptr))
+    return false;
+  auto go = [&](auto kern, int ctas) { launch_pdl(PDL_NORM, kern, dim3(148 * ctas), dim3(PN_THREADS), 0, s, p); };
+  auto pick = [&](auto nc) {
+    constexpr int NC = decltype(nc)::value;
+    constexpr int ctas = NC <= 2 ? 2 : 1;
+    if (p.top == 0) go(post_norm_rows_kernel<NC, 0>, ctas);
+    else if (p.top <= 2) go(post_norm_rows_kernel<NC, 2>, ctas);
+    else go(post_norm_rows_kernel<NC, 4>, ctas);
+  };
+  if (p.W <= PN_THREADS * 4) pick(std::integral_constant<int, 1>{});
+  else if (p.W <= PN_THREADS * 8) pick(std::integral_constant<int, 2>{});
+  else pick(std::integral_constant<int, 4>{});
+  return true;
+}
+
 // x (+)= y + mixed expert rows;  h = rms(x) * w (or x) in the model's type, zero-padded from W to Wp columns.  NC: 4-column
 // chunks per thread
 template <typename T, bool VEC, int NC>
@@ -327,7 +436,8 @@ void launch_post_norm_add(const PostNormAdd& p, bool f32, cudaStream_t s) {
   if (p.T == 0) return;
   if (p.W > PN_THREADS * 16) throw std::runtime_error("norm rows are limited to 8192 columns");
   auto go = [&](auto kern) { launch_pdl(PDL_NORM, kern, dim3(p.T), dim3(PN_THREADS), 0, s, p); };
-  if (p.W % 4 != 0) {
+  if (!f32 && post_norm_rows(p, s)) {
+  } else if (p.W % 4 != 0) {
     if (f32) go(post_norm_add_kernel<float, false, 4>);
     else go(post_norm_add_kernel<bf16, false, 4>);
   } else if (f32) {

@@ -231,7 +231,8 @@ def test_absorbed_attention_with_window_sink_and_gate(H, rank, R, page, window, 
     assert ext().read_status(0) == 0
 
 
-@pytest.mark.parametrize("H,G,D,R,V,window,sink", [(4, 2, 0, 64, 64, 0, False), (8, 2, 0, 256, 128, 0, False), (6, 3, 0, 336, 80, 0, False),
+@pytest.mark.parametrize("H,G,D,R,V,window,sink", [(4, 2, 0, 64, 64, 0, False), (3, 1, 0, 256, 128, 0, False), (6, 1, 0, 40, 24, 0, False),
+                                                   (4, 1, 0, 136, 72, 0, False), (16, 2, 0, 192, 128, 0, False), (8, 2, 0, 256, 128, 0, False), (6, 3, 0, 336, 80, 0, False),
                                                    (4, 4, 0, 512, 128, 0, True), (4, 1, 0, 384, 56, 50, False), (10, 5, 0, 640, 128, 0, False),
                                                    (8, 8, 0, 1024, 64, 129, True), (3, 3, 128, 64, 128, 100, True), (2, 2, 40, 24, 16, 1, True),
                                                    (2, 2, 128, 64, 128, 128, False)])
