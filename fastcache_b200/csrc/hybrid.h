@@ -321,9 +321,6 @@ struct LatentPrefill {
 };
 bool latent_prefill_supported(const LatentPrefill& p);
 void launch_latent_prefill(const LatentPrefill& p, cudaStream_t s);
-// the same for shared keys alone, two heads of one value head at a time (paired_prefill.cu); launch_latent_prefill takes it where it can
-bool paired_prefill_supported(const LatentPrefill& p);
-void launch_paired_prefill(const LatentPrefill& p, cudaStream_t s);
 
 // ---- talking.cu: queries and cache rows of attention whose heads mix their scores before the softmax
 // q [T, H, G * D]: the sum over the heads g of key head u of talk[h, g] * query of g, for every u; a query of this width

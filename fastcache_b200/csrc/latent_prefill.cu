@@ -7,9 +7,9 @@
 // separate score and output accumulators in tensor memory and separate softmax warps, so that one parity's matrices
 // run while the other's softmax does; the two partial results are merged at the end:
 //     S_0 [0,128)  S_1 [128,256)  O_0 [256,384)  O_1 [384,512)
-//   warp 0       TMA: the Q tile once, K in sub-tiles of 64 columns through a ring, V tiles.  Queries of more than eight
-//                sub-tiles do not stay: every slot of the ring takes a sub-tile of K and of Q.  Three-dimensional boxes
-//                (column, head, row) zero-fill the columns past a head's width
+//   warp 0       TMA: the Q tile once, K through a ring whose slots take one or more sub-tiles of 64 columns (a whole tile
+//                where two fit), V tiles.  Queries of more than eight sub-tiles do not stay: every slot then takes a sub-tile
+//                of K and of Q.  Three-dimensional boxes (column, head, row) zero-fill the columns past a head's width
 //   warp 1       tcgen05.mma issuer: S_x = Q K(j)^T, then O_x += P_x V(j) with P_x in tensor memory over S_x
 //   warps 2-5    softmax of even tiles, warps 6-9 of odd tiles: one query row per thread, reference maximum as in
 //                attn_prefill_tc2.cu (O is rescaled only when a row outgrows its reference by 2^8)
@@ -54,7 +54,7 @@ struct LpParams {
   long long ld_gate, ld_out;
   int D, R, V, heads_per_value, window;
   int nd, nr;                                     // sub-tiles of the keys' own and shared columns
-  int ring, v_stages;
+  int ring, per_slot, v_stages;                   // slots of the K ring, sub-tiles of K in a slot
   float scale_log2;
   uint32_t* status;
 };
@@ -63,13 +63,13 @@ struct LpParams {
 template <int NV, bool STREAM_Q>
 __global__ void __launch_bounds__(LP_THREADS, 1)
 latent_prefill_kernel(const __grid_constant__ LpMaps tm, const LpParams p) {
-  constexpr int SLOT = STREAM_Q ? 2 * LP_SUB : LP_SUB;   // K sub-tile, then Q's
+  const int slot_bytes = STREAM_Q ? 2 * LP_SUB : p.per_slot * LP_SUB;    // STREAM_Q: K sub-tile, then Q's
   constexpr int V_BYTES = NV * LP_SUB;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   const int nq = p.nd + p.nr;                      // sub-tiles of a Q or K tile
   uint8_t* s_k = smem;                             // ring
-  uint8_t* s_v = s_k + p.ring * SLOT;              // v_stages
+  uint8_t* s_v = s_k + p.ring * slot_bytes;              // v_stages
   uint8_t* s_q = s_v + p.v_stages * V_BYTES;
   uint64_t* bars = reinterpret_cast<uint64_t*>(smem + LP_SLOTS * LP_SUB);
   uint64_t *q_full = bars, *k_full = bars + 1, *k_empty = k_full + LP_RING, *v_full = k_empty + LP_RING, *v_empty = v_full + 2;
@@ -79,9 +79,9 @@ latent_prefill_kernel(const __grid_constant__ LpMaps tm, const LpParams p) {
   float* s_ml = reinterpret_cast<float*>(o_done + 3);   // [2][128] reference maximum and sum of the odd tiles
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int seq = blockIdx.z, h = blockIdx.y;
+  const int seq = blockIdx.z, h = blockIdx.x;
   const int q_begin = p.cu_q[seq], q_len = p.cu_q[seq + 1] - q_begin;
-  const int q0 = (gridDim.x - 1 - blockIdx.x) * LP_BM;            // late (long) tiles first
+  const int q0 = (gridDim.y - 1 - blockIdx.y) * LP_BM;            // late (long) tiles first
   if (q0 >= q_len) return;
   const int kv_begin = p.cu_kv[seq], kv_len = p.cu_kv[seq + 1] - kv_begin;
   const int offset = kv_len - q_len;
@@ -133,14 +133,15 @@ latent_prefill_kernel(const __grid_constant__ LpMaps tm, const LpParams p) {
     for (int j = 0; j < n_tiles && ok; ++j) {
       const int row = kv_begin + (tile0 + j) * LP_BN;
       ok = !__any_sync(0xffffffffu, *s_abort != 0);
-      for (int i = 0; i < nq && ok; ++i) {
+      for (int i0 = 0; i0 < nq && ok; i0 += p.per_slot) {
         ok = warp_wait(&k_empty[slot], phase, p.status, ST_TIMEOUT_EMPTY);
         if (!ok) break;
-        uint8_t* dk = s_k + slot * SLOT;
-        one_expect(&k_full[slot], SLOT, el);
-        if (i < p.nd) one_load_3d(dk, &tm.kn, &k_full[slot], i * 64, h, row, el);
-        else one_load_2d(dk, &tm.kr, &k_full[slot], (i - p.nd) * 64, row, el);
-        if (STREAM_Q) load_q(dk + LP_SUB, &k_full[slot], i);
+        uint8_t* dk = s_k + slot * slot_bytes;
+        one_expect(&k_full[slot], slot_bytes, el);
+        for (int i = i0; i < i0 + p.per_slot; ++i, dk += LP_SUB)
+          if (i < p.nd) one_load_3d(dk, &tm.kn, &k_full[slot], i * 64, h, row, el);
+          else one_load_2d(dk, &tm.kr, &k_full[slot], (i - p.nd) * 64, row, el);
+        if (STREAM_Q) load_q(dk, &k_full[slot], i0);
         if (++slot == p.ring) {
           slot = 0;
           phase ^= 1;
@@ -168,15 +169,19 @@ latent_prefill_kernel(const __grid_constant__ LpMaps tm, const LpParams p) {
     uint32_t phase = 0;
     auto issue_s = [&](int j) {
       const uint32_t ts = tmem_base + uint32_t(j & 1) * 128u;
-      for (int i = 0; i < nq; ++i) {
+      for (int i0 = 0; i0 < nq; i0 += p.per_slot) {
         if (!warp_wait(&k_full[slot], phase, p.status, ST_TIMEOUT_FULL)) return false;
         tc_fence_after();
-        const uint64_t dk = d_k + uint64_t(slot * (SLOT >> 4)), dq = STREAM_Q ? dk + uint64_t(LP_SUB >> 4) : d_q + uint64_t(i * (LP_SUB >> 4));
-        const int left = i < p.nd ? p.D - i * 64 : p.R - (i - p.nd) * 64;
+        uint64_t dk = d_k + uint64_t(slot * (slot_bytes >> 4)), dq = STREAM_Q ? dk + uint64_t(LP_SUB >> 4) : d_q + uint64_t(i0 * (LP_SUB >> 4));
+        for (int i = i0; i < i0 + p.per_slot; ++i, dk += uint64_t(LP_SUB >> 4), dq += uint64_t(LP_SUB >> 4)) {
+          const int left = i < p.nd ? p.D - i * 64 : p.R - (i - p.nd) * 64;
+          if (elect_one())
 #pragma unroll
-        for (int kk = 0; kk < 4; ++kk)
-          if (kk * 16 < left)
-            one_mma(ts, dq + uint64_t(kk * 2), dk + uint64_t(kk * 2), idesc_s, (i > 0 || kk > 0) ? 1u : 0u, el);
+            for (int kk = 0; kk < 4; ++kk)
+              if (kk * 16 < left)
+                tc_mma_f16(ts, dq + uint64_t(kk * 2), dk + uint64_t(kk * 2), idesc_s, (i > 0 || kk > 0) ? 1u : 0u);
+          __syncwarp();
+        }
         one_commit(&k_empty[slot], el);
         if (++slot == p.ring) {
           slot = 0;
@@ -196,10 +201,12 @@ latent_prefill_kernel(const __grid_constant__ LpMaps tm, const LpParams p) {
       if (!ok) break;
       tc_fence_after();
       const uint64_t dv = d_v + uint64_t(st * (V_BYTES >> 4));
+      if (elect_one())
 #pragma unroll
-      for (int kk = 0; kk < 8; ++kk)
-        one_mma_ts(tmem_base + 256u + uint32_t(x * 128), tmem_base + uint32_t(x * 128) + uint32_t(kk * 8), dv + uint64_t(kk * 128), idesc_o,
-                   (j > 1 || kk > 0) ? 1u : 0u, el);
+        for (int kk = 0; kk < 8; ++kk)
+          tc_mma_f16_ts(tmem_base + 256u + uint32_t(x * 128), tmem_base + uint32_t(x * 128) + uint32_t(kk * 8), dv + uint64_t(kk * 128),
+                        idesc_o, (j > 1 || kk > 0) ? 1u : 0u);
+      __syncwarp();
       one_commit(&o_done[x], el);
       one_commit(&v_empty[st], el);
       if (j + 2 < n_tiles) ok = issue_s(j + 2);
@@ -243,10 +250,10 @@ latent_prefill_kernel(const __grid_constant__ LpMaps tm, const LpParams p) {
         for (int t = 0; t < 128; ++t)
           if (t <= hidden) s[t] = 0xff800000u;
       }
-      float mx = -INFINITY;
+      float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};        // four chains
 #pragma unroll
-      for (int t = 0; t < 128; ++t) mx = fmaxf(mx, __uint_as_float(s[t]));
-      mx *= p.scale_log2;
+      for (int t = 0; t < 128; ++t) mx4[t & 3] = fmaxf(mx4[t & 3], __uint_as_float(s[t]));
+      const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * p.scale_log2;
       if (i == 0) {
         m_ref = mx;
       } else if (__any_sync(__activemask(), mx > m_ref + LP_RESCALE)) {
@@ -272,7 +279,7 @@ latent_prefill_kernel(const __grid_constant__ LpMaps tm, const LpParams p) {
         tmem_st_wait();
       }
       const float base = m_ref == -INFINITY ? 0.f : m_ref;
-      float rs = 0.f;
+      float rs[4] = {0.f, 0.f, 0.f, 0.f};
       uint32_t u[64];
 #pragma unroll
       for (int t = 0; t < 64; ++t) {
@@ -281,7 +288,7 @@ latent_prefill_kernel(const __grid_constant__ LpMaps tm, const LpParams p) {
         const float a1 = fmaf(__uint_as_float(s[2 * t + 1]), p.scale_log2, -base);
         asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e0) : "f"(a0));
         asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e1) : "f"(a1));
-        rs += e0 + e1;
+        rs[t & 3] += e0 + e1;
         u[t] = pack_bf16(e0, e1);
       }
       tmem_st_32x32(ts, *reinterpret_cast<uint32_t(*)[32]>(&u[0]));
@@ -289,7 +296,7 @@ latent_prefill_kernel(const __grid_constant__ LpMaps tm, const LpParams p) {
       tmem_st_wait();
       tc_fence_before();
       mbar_arrive(&p_ready[x]);
-      l += rs;
+      l += (rs[0] + rs[1]) + (rs[2] + rs[3]);
     }
     if (ok && n_x > 0) ok = mbar_wait(&o_done[x], uint32_t(n_x - 1) & 1u, p.status, ST_TIMEOUT_ACC_FULL);
     if (!ok) *s_abort = 1;
@@ -325,7 +332,7 @@ latent_prefill_kernel(const __grid_constant__ LpMaps tm, const LpParams p) {
         }
         if (p.sink != nullptr && l > 0.f) l += exp2f(p.sink[h] * LP_LOG2E - mm);
         float inv = l > 0.f ? 1.f / l : 0.f;
-        if (p.head_gate != nullptr && qrow < q_len) inv *= p.head_gate[(long long)(q_begin + qrow) * gridDim.y + h];
+        if (p.head_gate != nullptr && qrow < q_len) inv *= p.head_gate[(long long)(q_begin + qrow) * gridDim.x + h];
         w0 *= inv;
         w1 *= inv;
         bf16* dst = p.out + (long long)(q_begin + qrow) * p.ld_out + h * p.V;
@@ -382,12 +389,11 @@ static void launch_lp(const LpMaps& tm, const LpParams& q, const LatentPrefill& 
   static_assert(smem <= 227 * 1024, "shared memory of a CTA");
   auto kern = latent_prefill_kernel<NV, STREAM_Q>;
   cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
-  kern<<<dim3((p.max_q + LP_BM - 1) / LP_BM, p.H, p.B), LP_THREADS, smem, s>>>(tm, q);
+  kern<<<dim3(p.H, (p.max_q + LP_BM - 1) / LP_BM, p.B), LP_THREADS, smem, s>>>(tm, q);
 }
 
 void launch_latent_prefill(const LatentPrefill& p, cudaStream_t s) {
   if (p.T == 0 || p.B == 0 || p.max_q == 0) return;
-  if (paired_prefill_supported(p)) return launch_paired_prefill(p, s);
   LpMaps tm;
   const uint64_t Q = uint64_t(p.D + p.R);
   const int vh = p.v_heads > 0 ? p.v_heads : p.H;
@@ -420,7 +426,9 @@ void launch_latent_prefill(const LatentPrefill& p, cudaStream_t s) {
   // at least four slots for K; two stages of V where they leave that much
   const int left = LP_SLOTS - (stream ? 0 : nq);
   a.v_stages = left - 2 * nv >= (stream ? 8 : 4) ? 2 : 1;
-  a.ring = std::min(LP_RING, (left - a.v_stages * nv) / (stream ? 2 : 1));
+  const int subs = left - a.v_stages * nv;                 // of the ring
+  a.per_slot = stream ? 1 : 2 * nq <= subs ? nq : nq % 2 == 0 ? 2 : 1;
+  a.ring = std::min(LP_RING, subs / (stream ? 2 : a.per_slot));
   if (nv == 1) stream ? launch_lp<1, true>(tm, a, p, s) : launch_lp<1, false>(tm, a, p, s);
   else stream ? launch_lp<2, true>(tm, a, p, s) : launch_lp<2, false>(tm, a, p, s);
   const cudaError_t e = cudaGetLastError();

@@ -44,16 +44,6 @@ __device__ __forceinline__ void one_load_3d(void* dst, const CUtensorMap* m, uin
       ::"r"(smem_u32(dst)), "l"(reinterpret_cast<uint64_t>(m)), "r"(smem_u32(bar)), "r"(x), "r"(y), "r"(z), "r"(issue)
       : "memory");
 }
-// D[tmem] (+)= A[tmem] * B[smem desc], see tc_mma_f16_ts
-__device__ __forceinline__ void one_mma_ts(uint32_t tmem_d, uint32_t tmem_a, uint64_t b, uint32_t idesc, uint32_t accumulate,
-                                           uint32_t issue) {
-  asm volatile(
-      "{\n\t.reg .pred p, q;\n\t"
-      "setp.ne.b32 p, %4, 0;\n\tsetp.ne.b32 q, %5, 0;\n\t"
-      "@q tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, p;\n\t}"
-      ::"r"(tmem_d), "r"(tmem_a), "l"(b), "r"(idesc), "r"(accumulate), "r"(issue)
-      : "memory");
-}
 // a wait by every lane, with one answer
 __device__ __forceinline__ bool warp_wait(uint64_t* bar, uint32_t parity, uint32_t* status, uint32_t code) {
   return __all_sync(0xffffffffu, mbar_wait(bar, parity, status, code)) != 0;

@@ -14,7 +14,7 @@ SRC = os.path.join("fastcache_b200", "csrc")
 # parallelism need (ops/loader.py takes it where the whole extension is not built)
 CORE = os.environ.get("FC_EXT") == "core"
 CORE_SOURCES = ("attn_decode.cu", "attn_prefill.cu", "attn_prefill_tc2.cu", "bindings.cpp", "elementwise.cu", "gemm.cu", "gemm_2cta.cu", "gemm_skinny.cu", "gemm_streamk.cu",
-                "hybrid_bind.cpp", "latent.cu", "latent_decode.cu", "latent_decode_tc.cu", "latent_prefill.cu", "linear_simt.cu", "lru.cu", "moe.cu", "moe_gemm.cu", "paired_prefill.cu", "partials.cu", "prenorm_bind.cpp",
+                "hybrid_bind.cpp", "latent.cu", "latent_decode.cu", "latent_decode_tc.cu", "latent_prefill.cu", "linear_simt.cu", "lru.cu", "moe.cu", "moe_gemm.cu", "partials.cu", "prenorm_bind.cpp",
                 "recurrence.cu", "recurrence_chunk.cu", "resid.cu", "streams.cu", "streams_bind.cpp", "talking.cu", "talking_bind.cpp", "window_attn.cu")
 sources = [os.path.join(SRC, f) for f in CORE_SOURCES] if CORE else sorted(glob.glob(os.path.join(SRC, "*.cu")) + glob.glob(os.path.join(SRC, "*.cpp")))
 
