@@ -68,7 +68,8 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm, const RowAttn p,
   uint64_t* bars = reinterpret_cast<uint64_t*>(s_red + 4 * LT_HEADS);
   uint64_t *full = bars, *empty = bars + LT_MAX_RING, *x_full = bars + 2 * LT_MAX_RING, *x_empty = x_full + 2;
   uint64_t *s_full = x_full + 4, *p_ready = x_full + 6, *o_done = x_full + 7;      // o_done: O^T complete up to a tile
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(x_full + 8);
+  uint64_t* q_ready = x_full + 8;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(x_full + 9);
   volatile int* s_abort = reinterpret_cast<volatile int*>(tmem_slot + 1);
   int* s_at = reinterpret_cast<int*>(tmem_slot + 2);               // [LT_ROWS / 8]
 
@@ -86,6 +87,7 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm, const RowAttn p,
       mbar_init(&s_full[i], 1);
     }
     mbar_init(p_ready, 128);
+    mbar_init(q_ready, 128);
     mbar_init(o_done, 1);
     *s_abort = 0;
     fence_barrier_init();
@@ -105,27 +107,6 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm, const RowAttn p,
   const int tile0 = start + split * per, n_tiles = max(0, min(tiles, tile0 + per) - tile0);
   const int* bt = p.block_tables + (long long)b * p.max_blocks;
 
-  {                                                                // Q, zero-padded to whole sub-tiles and head rows
-    const uint4* q = reinterpret_cast<const uint4*>(reinterpret_cast<const bf16*>(p.q) + ((long long)t * p.H + h0) * p.K);
-    uint4 v[6];
-    for (int ch = lane; ch < subs * 8; ch += 32) {
-#pragma unroll
-      for (int i = 0; i < 6; ++i) {
-        const int r = warp + i * (LT_THREADS / 32);
-        v[i] = r < LT_HEADS && h0 + r < p.H && ch * 8 < p.K ? __ldcg(q + (long long)r * (p.K / 8) + ch) : make_uint4(0, 0, 0, 0);
-      }
-#pragma unroll
-      for (int i = 0; i < 6; ++i) {
-        const int r = warp + i * (LT_THREADS / 32);
-        if (r < LT_HEADS)
-          *reinterpret_cast<uint4*>(s_q + (ch >> 3) * LT_QSUB + r * 128 + (((ch & 7) ^ (r & 7)) << 4)) = v[i];
-      }
-    }
-  }
-  if (n_tiles <= LT_MAX_RING)                                      // boxes past the context are never loaded: keep it finite
-    for (int i = tid; i < (w.ring * 2 + (w.extra ? 2 : 0)) * LT_SUB / 16; i += LT_THREADS)
-      reinterpret_cast<uint4*>(s_kv)[i] = make_uint4(0, 0, 0, 0);
-  fence_proxy_async();
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
@@ -139,13 +120,15 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm, const RowAttn p,
       bool ok = true;
       uint32_t phase = 1;
       constexpr int MAX_PIECES = LT_ROWS / 8;
+      const int pieces = LT_ROWS / box_rows;
       int next[MAX_PIECES];                                        // pool row of every piece of a tile, one tile ahead
       auto find = [&](int j) {
         const int row0 = (tile0 + j) * LT_ROWS;
 #pragma unroll
         for (int pc = 0; pc < MAX_PIECES; ++pc) {
-          const int tok = row0 + pc * box_rows;
-          if (j >= n_tiles || pc * box_rows >= LT_ROWS || tok >= ctx) continue;
+          if (j >= n_tiles || pc * box_rows >= LT_ROWS) continue;
+          // a box past the context is loaded from the last one inside: what its rows hold must only be finite
+          const int tok = min(row0 + pc * box_rows, (ctx - 1) / box_rows * box_rows);
           int blk = bt[tok / p.block_size];
           if (blk < 0 || blk >= p.num_blocks) {
             if (lane == 0) report(p.status, ST_BAD_INDEX);
@@ -156,8 +139,6 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm, const RowAttn p,
       };
       find(0);
       for (int j = 0; j < n_tiles && ok; ++j) {
-        const int pieces = min(LT_ROWS / box_rows, (ctx - (tile0 + j) * LT_ROWS + box_rows - 1) / box_rows);
-        const uint32_t bytes = uint32_t(pieces) * box_rows * 128;
         // through shared memory: the issue loop stays one instruction sequence for any number of pieces
         ok = !__any_sync(0xffffffffu, *s_abort != 0);                // also: every lane is done with the tile before
 #pragma unroll
@@ -177,7 +158,7 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm, const RowAttn p,
             ok = false;
             break;
           }
-          one_expect(&full[slot], 2 * bytes, el);
+          one_expect(&full[slot], 2 * LT_SUB, el);
           load(s_kv + slot * 2 * LT_SUB, &full[slot], col);
           load(s_kv + slot * 2 * LT_SUB + LT_SUB, &full[slot], col + 64);
           if (++slot == w.ring) {
@@ -192,7 +173,7 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm, const RowAttn p,
             ok = false;
             break;
           }
-          one_expect(&x_full[x], bytes, el);
+          one_expect(&x_full[x], LT_SUB, el);
           load(s_x + x * LT_SUB, &x_full[x], w.keys * 128);
         }
       }
@@ -224,10 +205,11 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm, const RowAttn p,
       auto scores = [&](uint32_t tm_s, uint64_t da, int sub) {
         const uint64_t dq = d_q + uint64_t(sub * (LT_QSUB >> 4));
         const int left = ksteps - sub * 4;
+        if (elect_one())
 #pragma unroll
-        for (int kk = 0; kk < 4; ++kk)
-          if (kk < left)
-            one_mma(tm_s, da + uint64_t(kk * 2), dq + uint64_t(kk * 2), idesc_s, (sub > 0 || kk > 0) ? 1u : 0u, el);
+          for (int kk = 0; kk < 4; ++kk)
+            if (kk < left) tc_mma_f16(tm_s, da + uint64_t(kk * 2), dq + uint64_t(kk * 2), idesc_s, (sub > 0 || kk > 0) ? 1u : 0u);
+        __syncwarp();
       };
       auto issue_s = [&](int j) {
         const int x = j & 1;
@@ -250,7 +232,7 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm, const RowAttn p,
         if (w.extra) one_commit(&x_empty[x], el);
         return true;
       };
-      bool ok = n_tiles == 0 || issue_s(0);
+      bool ok = n_tiles == 0 || (wait(q_ready, 0, p.status, ST_TIMEOUT_FULL) && issue_s(0));
       for (int j = 0; j < n_tiles && ok; ++j) {
         if (w.ahead && j + 1 < n_tiles) ok = issue_s(j + 1);
         ok = ok && wait(p_ready, uint32_t(j) & 1u, p.status, ST_TIMEOUT_FULL);
@@ -264,9 +246,11 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm, const RowAttn p,
           }
           const uint64_t dv = d_cols + uint64_t(slot * (2 * LT_SUB >> 4)), dp = d_p + uint64_t((j & 1) * (LT_QSUB >> 4));
           const uint32_t tm_o = tmem + LT_HEADS * uint32_t(2 + i);
+          if (elect_one())
 #pragma unroll
-          for (int kk = 0; kk < LT_ROWS / 16; ++kk)
-            one_mma(tm_o, dv + uint64_t(kk * 128), dp + uint64_t(kk * 2), idesc_o, (j > 0 || kk > 0) ? 1u : 0u, el);
+            for (int kk = 0; kk < LT_ROWS / 16; ++kk)
+              tc_mma_f16(tm_o, dv + uint64_t(kk * 128), dp + uint64_t(kk * 2), idesc_o, (j > 0 || kk > 0) ? 1u : 0u);
+          __syncwarp();
           one_commit(&empty[slot], el);
           skip(slot, pho, 1);
         }
@@ -278,7 +262,26 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm, const RowAttn p,
       if (!ok && lane == 0) *s_abort = 1;
     }
   } else {
-    // ------------------------------------------------------------------ softmax, then epilogue
+    // ------------------------------------------------------------------ Q; softmax; epilogue
+    if (n_tiles > 0) {                                             // zero-padded to whole sub-tiles and head rows
+      const uint4* q = reinterpret_cast<const uint4*>(reinterpret_cast<const bf16*>(p.q) + ((long long)t * p.H + h0) * p.K);
+      constexpr int N = LT_HEADS / 4;
+      for (int ch = lane; ch < subs * 8; ch += 32) {
+        uint4 v[N];
+#pragma unroll
+        for (int i = 0; i < N; ++i) {
+          const int r = warp - 2 + i * 4;
+          v[i] = h0 + r < p.H && ch * 8 < p.K ? __ldcg(q + (long long)r * (p.K / 8) + ch) : make_uint4(0, 0, 0, 0);
+        }
+#pragma unroll
+        for (int i = 0; i < N; ++i) {
+          const int r = warp - 2 + i * 4;
+          *reinterpret_cast<uint4*>(s_q + (ch >> 3) * LT_QSUB + r * 128 + (((ch & 7) ^ (r & 7)) << 4)) = v[i];
+        }
+      }
+      fence_proxy_async();
+      mbar_arrive(q_ready);
+    }
     const int group = warp & 3;                                    // TMEM lanes this warp may touch
     const int row = group * 32 + lane;
     const uint32_t lanes = uint32_t(group * 32) << 16;
@@ -384,10 +387,9 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm, const RowAttn p,
     if (ok && n_tiles > 0) ok = mbar_wait(o_done, uint32_t(n_tiles - 1) & 1u, p.status, ST_TIMEOUT_ACC_FULL);
     if (!ok) *s_abort = 1;
     tc_fence_after();
-    // every product is done: the ring is free.  Sums over the rows, then O^T block by block through shared memory
+    // every product is done: the ring is free.  Sums over the rows, then O^T block by block, a lane per value column
     const bool good = !sync_or(!ok) && n_tiles > 0;
     float* s_l = reinterpret_cast<float*>(s_kv);                   // [LT_ROWS][33]
-    float* s_o = s_l + LT_ROWS * 33;                               // [32 heads][128 latents + 4]
     const int et = tid - 64;                                       // 0..127
     if (mine)
 #pragma unroll
@@ -415,32 +417,31 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm, const RowAttn p,
       }
       s_red[et] = f;
     }
-    const int heads_per = p.H / p.v_heads;
+    sync_or(false);
+    const int heads_per = p.H / p.v_heads, here = min(LT_HEADS, p.H - h0);
+    const long long head0 = (long long)t * p.H + h0;
+    // short loops: this code runs once per CTA, and fetching it is what it waits for
+#pragma unroll 1
     for (int i = 0; i < w.values; ++i) {
-      sync_or(false);                                              // s_red is there, the block before is written
-      if (good) {
-        uint32_t r[32];
-        tmem_ld_32x32(tmem + lanes + LT_HEADS * uint32_t(2 + i), r);
+      const int c = i * 128 + row, vh = c / p.V, cv = c - vh * p.V;    // the value head of this column takes it
+      const int lo = vh * heads_per - h0, hi = vh < p.v_heads ? min(here, lo + heads_per) : 0;
+      bf16* out = reinterpret_cast<bf16*>(p.out) + t * p.ld_out + (long long)h0 * p.V + cv;
+      float* part = p.part_o + (head0 * p.splits + split) * p.V + cv;
+      const int step = p.splits == 1 ? p.V : p.splits * p.V;
+#pragma unroll 1
+      for (int h8 = 0; h8 < here; h8 += 8) {
+        uint32_t r[8];
+        tmem_ld_32x8(tmem + lanes + LT_HEADS * uint32_t(2 + i) + uint32_t(h8), r);
         tmem_ld_wait();
 #pragma unroll
-        for (int h = 0; h < LT_HEADS; ++h) s_o[h * 132 + row] = __uint_as_float(r[h]);
-      }
-      sync_or(false);
-      const int c = i * 128 + (et & 31) * 4;                       // a warp writes 128 columns of a head
-      const int vh = c / p.V;                                      // the value head they belong to (V is a multiple of 4)
-      if (vh < p.v_heads)
-        for (int h = et >> 5; h < LT_HEADS && h0 + h < p.H; h += 4) {
-          if ((h0 + h) / heads_per != vh) continue;
-          const float inv = s_red[h];
-          float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
-          if (inv != 0.f) x = *reinterpret_cast<const float4*>(s_o + h * 132 + (et & 31) * 4);
-          const long long at = (long long)t * p.H + h0 + h;
-          const int cv = c - vh * p.V;
-          if (p.splits == 1)
-            store4(reinterpret_cast<bf16*>(p.out) + t * p.ld_out + (h0 + h) * p.V + cv, x.x * inv, x.y * inv, x.z * inv, x.w * inv);
-          else
-            store4(p.part_o + (at * p.splits + split) * p.V + cv, x.x * inv, x.y * inv, x.z * inv, x.w * inv);
+        for (int e = 0; e < 8; ++e) {
+          const int h = h8 + e;
+          if (h < lo || h >= hi) continue;
+          const float f = s_red[h], x = f != 0.f ? __uint_as_float(r[e]) * f : 0.f;      // 0: no row was seen
+          if (p.splits == 1) out[(long long)h * step] = __float2bfloat16(x);
+          else part[(long long)h * step] = x;
         }
+      }
     }
   }
   tc_fence_before();
@@ -459,7 +460,7 @@ static int lt_box_rows(int block_size) {
 
 static int lt_smem(const LtTile& w) {
   return w.ring * 2 * LT_SUB + (w.extra ? 2 * LT_SUB : 0) + (w.keys * 2 + w.extra + 2) * LT_QSUB + 5 * LT_HEADS * 4 +
-         (2 * LT_MAX_RING + 8) * 8 + 16 + LT_ROWS / 2 + 1024;
+         (2 * LT_MAX_RING + 9) * 8 + 16 + LT_ROWS / 2 + 1024;
 }
 // how a tile lies in the ring; ring 0: these sizes do not fit
 static LtTile lt_tile(const RowAttn& p) {
@@ -502,8 +503,8 @@ void launch_latent_decode_tc(const RowAttn& p, cudaStream_t s) {
   if (w.ring == 0) throw std::runtime_error("attention over shared rows (tcgen05): unsupported sizes");
   const CUtensorMap tm = make_tmap_bf16_2d(p.pool, (uint64_t)p.num_blocks * p.block_size, p.row_width, p.row_width, box, 64);
   cudaFuncSetAttribute(latent_decode_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
-  launch_pdl(PDL_DECODE_ATTN, latent_decode_tc_kernel, dim3(p.T, (p.H + LT_HEADS - 1) / LT_HEADS, p.splits),
-             dim3(LT_THREADS), smem, s, tm, p, w, box, p.scale * LT_LOG2E);
+  launch_pdl(PDL_DECODE_ATTN, latent_decode_tc_kernel, dim3(p.T, (p.H + LT_HEADS - 1) / LT_HEADS, p.splits), dim3(LT_THREADS), smem, s,
+             tm, p, w, box, p.scale * LT_LOG2E);
   const cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess) throw std::runtime_error(std::string("attention over shared rows (tcgen05): ") + cudaGetErrorString(e));
 }

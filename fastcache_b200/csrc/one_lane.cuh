@@ -1,21 +1,12 @@
 // Instructions issued by one lane of a warp that is converged otherwise: only the instruction is predicated, loops, addresses and
-// descriptors stay warp-uniform.  (Inside a divergent single-lane branch every TMA load and MMA costs hundreds of cycles of issue.)
+// descriptors stay warp-uniform.  (Inside a long divergent single-lane branch every TMA load and MMA
+// costs hundreds of cycles of issue; a few MMAs in a row stand best in an `if (elect_one())` of their own.)
 // `issue`: 1 on the issuing lane, 0 on the others.
 #pragma once
 #include "ptx.cuh"
 
 namespace fc {
 
-// D[tmem] (+)= A[smem desc] * B[smem desc]
-__device__ __forceinline__ void one_mma(uint32_t tmem_d, uint64_t a, uint64_t b, uint32_t idesc, uint32_t accumulate,
-                                       uint32_t issue) {
-  asm volatile(
-      "{\n\t.reg .pred p, q;\n\t"
-      "setp.ne.b32 p, %4, 0;\n\tsetp.ne.b32 q, %5, 0;\n\t"
-      "@q tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t}"
-      ::"r"(tmem_d), "l"(a), "l"(b), "r"(idesc), "r"(accumulate), "r"(issue)
-      : "memory");
-}
 __device__ __forceinline__ void one_commit(uint64_t* bar, uint32_t issue) {
   asm volatile(
       "{\n\t.reg .pred q;\n\tsetp.ne.b32 q, %1, 0;\n\t"
