@@ -67,9 +67,10 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm, const RowAttn p,
   float* s_red = s_ref + LT_HEADS;                                 // [4][32]
   uint64_t* bars = reinterpret_cast<uint64_t*>(s_red + 4 * LT_HEADS);
   uint64_t *full = bars, *empty = bars + LT_MAX_RING, *x_full = bars + 2 * LT_MAX_RING, *x_empty = x_full + 2;
-  uint64_t *s_full = x_full + 4, *p_ready = x_full + 6, *o_done = x_full + 7;      // o_done: O^T complete up to a tile
-  uint64_t* q_ready = x_full + 8;
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(x_full + 9);
+  // o_done: O^T complete up to a tile.  p_ready of even / odd tiles apart: the scores of the next tile are issued before the issuer
+  // waits for this one's P, so one barrier could be two phases ahead of its wait
+  uint64_t *s_full = x_full + 4, *p_ready = x_full + 6, *o_done = x_full + 8, *q_ready = x_full + 9;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(x_full + 10);
   volatile int* s_abort = reinterpret_cast<volatile int*>(tmem_slot + 1);
   int* s_at = reinterpret_cast<int*>(tmem_slot + 2);               // [LT_ROWS / 8]
 
@@ -85,8 +86,8 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm, const RowAttn p,
       mbar_init(&x_full[i], 1);
       mbar_init(&x_empty[i], 1);
       mbar_init(&s_full[i], 1);
+      mbar_init(&p_ready[i], 128);
     }
-    mbar_init(p_ready, 128);
     mbar_init(q_ready, 128);
     mbar_init(o_done, 1);
     *s_abort = 0;
@@ -235,7 +236,7 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm, const RowAttn p,
       bool ok = n_tiles == 0 || (wait(q_ready, 0, p.status, ST_TIMEOUT_FULL) && issue_s(0));
       for (int j = 0; j < n_tiles && ok; ++j) {
         if (w.ahead && j + 1 < n_tiles) ok = issue_s(j + 1);
-        ok = ok && wait(p_ready, uint32_t(j) & 1u, p.status, ST_TIMEOUT_FULL);
+        ok = ok && wait(&p_ready[j & 1], uint32_t(j >> 1) & 1u, p.status, ST_TIMEOUT_FULL);
         if (!ok) break;
         tc_fence_after();
         for (int i = 0; i < w.values && ok; ++i) {
@@ -382,7 +383,7 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm, const RowAttn p,
       if (j == n_tiles - 1 && j > 0 && ok) ok = mbar_wait(o_done, uint32_t(j - 1) & 1u, p.status, ST_TIMEOUT_ACC_FULL);
       fence_proxy_async();
       tc_fence_before();
-      mbar_arrive(p_ready);
+      mbar_arrive(&p_ready[j & 1]);
     }
     if (ok && n_tiles > 0) ok = mbar_wait(o_done, uint32_t(n_tiles - 1) & 1u, p.status, ST_TIMEOUT_ACC_FULL);
     if (!ok) *s_abort = 1;
@@ -431,6 +432,7 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm, const RowAttn p,
 #pragma unroll 1
       for (int h8 = 0; h8 < here; h8 += 8) {
         uint32_t r[8];
+        __syncwarp();
         tmem_ld_32x8(tmem + lanes + LT_HEADS * uint32_t(2 + i) + uint32_t(h8), r);
         tmem_ld_wait();
 #pragma unroll
@@ -460,7 +462,7 @@ static int lt_box_rows(int block_size) {
 
 static int lt_smem(const LtTile& w) {
   return w.ring * 2 * LT_SUB + (w.extra ? 2 * LT_SUB : 0) + (w.keys * 2 + w.extra + 2) * LT_QSUB + 5 * LT_HEADS * 4 +
-         (2 * LT_MAX_RING + 9) * 8 + 16 + LT_ROWS / 2 + 1024;
+         (2 * LT_MAX_RING + 10) * 8 + 16 + LT_ROWS / 2 + 1024;
 }
 // how a tile lies in the ring; ring 0: these sizes do not fit
 static LtTile lt_tile(const RowAttn& p) {
