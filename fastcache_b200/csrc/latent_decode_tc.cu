@@ -2,11 +2,12 @@
 // latent_decode.cu): latent rows, whose first columns are the values too, or rows with the keys of several key heads side by
 // side and the values behind them.
 //
-// Grid (query row, group of 32 heads, split of the context).  A CTA walks its rows of the cache in tiles of 64.  The wide
-// operand of both products is the cache, not the few heads:
-//     S^T [64 rows x 32 heads]    = rows (key columns) * Q^T                   A: row tile, K-major; B: Q, K-major
+// Grid (query row, group of 32 heads, split of the context).  A CTA walks its rows of the cache in tiles of 128 rows, or of 64
+// where wider tiles would leave no room for the next one's keys.  The wide operand of both products is the cache, not the few
+// heads:
+//     S^T [rows x 32 heads]        = rows (key columns) * Q^T                  A: row tile, K-major; B: Q, K-major
 //     O^T [128 columns x 32 heads] += rows^T * P^T, one block per 128 value columns  A: MN-major; B: P, K-major
-// (S^T is issued with 128 rows; the upper 64 read the shared memory behind the tile and their lanes are ignored.)  Shared
+// (S^T is issued with 128 rows; of a tile of 64 the upper ones read the shared memory behind it, their lanes are ignored.)  Shared
 // memory holds a tile as pairs of 64-column sub-tiles in a ring, and the columns behind latent pairs in a ring of two
 // sub-tiles.  Latent pairs serve both products and are refilled as soon as their block of O^T is done; other rows have pairs
 // of keys, then pairs of values.  Where value heads differ, every head takes its own columns of O^T at the end.
@@ -28,8 +29,7 @@
 namespace fc {
 
 using bf16 = __nv_bfloat16;
-constexpr int LT_ROWS = 64, LT_HEADS = 32, LT_MAX_RING = 12, LT_THREADS = 192;
-constexpr int LT_SUB = LT_ROWS * 128;             // bytes of a [64 rows x 64 columns] sub-tile
+constexpr int LT_HEADS = 32, LT_MAX_RING = 12, LT_THREADS = 192;
 constexpr int LT_QSUB = LT_HEADS * 128;           // of a [32 heads x 64 columns] sub-tile
 // tensor memory: S^T of even / odd tiles [0, 32) [32, 64), O^T blocks [64 + 32 b, ...)
 constexpr float LT_RANGE = 64.f;                  // log2 units above the reference that P may reach
@@ -39,7 +39,7 @@ constexpr float LT_LOG2E = 1.4426950408889634f;
 // A tile in the ring: `pairs` slots of 128 columns, of which the first `keys` enter the scores and the last `values` make the
 // blocks of O^T; `extra`: 64 more key columns; `shared`: keys and values are the same pairs
 struct LtTile {
-  int pairs, keys, values, extra, ring, ahead, tmem;
+  int rows, pairs, keys, values, extra, ring, ahead, tmem;
   bool shared;
 };
 
@@ -53,9 +53,12 @@ __device__ __forceinline__ uint64_t lt_sdesc(uint32_t addr, uint32_t lbo_bytes, 
   return d;
 }
 
+template <int LT_ROWS>
 __global__ void __launch_bounds__(LT_THREADS, 1)
 latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm, const RowAttn p, const LtTile w, int box_rows,
                         float scale_log2) {
+  constexpr int LT_SUB = LT_ROWS * 128;                            // bytes of a [rows x 64 columns] sub-tile
+  constexpr int PSUBS = LT_ROWS / 64;                              // sub-tiles of P
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   const int subs = w.keys * 2 + w.extra;                           // sub-tiles of Q
@@ -63,7 +66,7 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm, const RowAttn p,
   uint8_t* s_x = s_kv + w.ring * 2 * LT_SUB;                       // the columns behind the pairs
   uint8_t* s_q = s_x + (w.extra ? 2 * LT_SUB : 0);                 // [subs] sub-tiles
   uint8_t* s_p = s_q + subs * LT_QSUB;
-  float* s_ref = reinterpret_cast<float*>(s_p + 2 * LT_QSUB);      // (P of even / odd tiles)  [32] reference
+  float* s_ref = reinterpret_cast<float*>(s_p + 2 * PSUBS * LT_QSUB);      // (P of even / odd tiles)  [32] reference
   float* s_red = s_ref + LT_HEADS;                                 // [4][32]
   uint64_t* bars = reinterpret_cast<uint64_t*>(s_red + 4 * LT_HEADS);
   uint64_t *full = bars, *empty = bars + LT_MAX_RING, *x_full = bars + 2 * LT_MAX_RING, *x_empty = x_full + 2;
@@ -245,12 +248,12 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm, const RowAttn p,
             if (!ok) break;
             tc_fence_after();
           }
-          const uint64_t dv = d_cols + uint64_t(slot * (2 * LT_SUB >> 4)), dp = d_p + uint64_t((j & 1) * (LT_QSUB >> 4));
+          const uint64_t dv = d_cols + uint64_t(slot * (2 * LT_SUB >> 4)), dp = d_p + uint64_t((j & 1) * (PSUBS * LT_QSUB >> 4));
           const uint32_t tm_o = tmem + LT_HEADS * uint32_t(2 + i);
           if (elect_one())
 #pragma unroll
             for (int kk = 0; kk < LT_ROWS / 16; ++kk)
-              tc_mma_f16(tm_o, dv + uint64_t(kk * 128), dp + uint64_t(kk * 2), idesc_o, (j > 0 || kk > 0) ? 1u : 0u);
+              tc_mma_f16(tm_o, dv + uint64_t(kk * 128), dp + uint64_t((kk >> 2) * (LT_QSUB >> 4) + (kk & 3) * 2), idesc_o, (j > 0 || kk > 0) ? 1u : 0u);
           __syncwarp();
           one_commit(&empty[slot], el);
           skip(slot, pho, 1);
@@ -298,9 +301,9 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm, const RowAttn p,
     float l[LT_HEADS];
 #pragma unroll
     for (int h = 0; h < LT_HEADS; ++h) l[h] = 0.f;
-    uint8_t* prow = s_p + (row & 7) * 2;
+    uint8_t* prow = s_p + (PSUBS > 1 ? (row >> 6) * LT_QSUB : 0) + (row & 7) * 2;
     const int chunk = (row & 63) >> 3;
-    const bool mine = row < LT_ROWS;                               // warp-uniform: the upper lanes hold no cache row
+    const bool mine = row < LT_ROWS;                               // warp-uniform: of 64 rows the upper lanes hold none
     bool ok = true;
     for (int j = 0; j < n_tiles; ++j) {
       if (ok) ok = !*s_abort && mbar_wait(&s_full[j & 1], uint32_t(j >> 1) & 1u, p.status, ST_TIMEOUT_ACC_FULL);
@@ -375,7 +378,7 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm, const RowAttn p,
           float e;
           asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(valid ? v[h] : -INFINITY));
           l[h] += e;
-          *reinterpret_cast<bf16*>(prow + (j & 1) * LT_QSUB + h * 128 + ((chunk ^ (h & 7)) << 4)) = __float2bfloat16(e);
+          *reinterpret_cast<bf16*>(prow + (j & 1) * PSUBS * LT_QSUB + h * 128 + ((chunk ^ (h & 7)) << 4)) = __float2bfloat16(e);
         }
       }
       // the last two phases of o_done one by one, a parity cannot tell a phase from the one two before it: the scores of the
@@ -454,20 +457,22 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm, const RowAttn p,
   }
 }
 
-static int lt_box_rows(int block_size) {
-  int box = LT_ROWS;
+static int lt_box_rows(int block_size, int rows) {
+  int box = rows;
   while (box > block_size || block_size % box != 0) box >>= 1;
   return box;
 }
 
 static int lt_smem(const LtTile& w) {
-  return w.ring * 2 * LT_SUB + (w.extra ? 2 * LT_SUB : 0) + (w.keys * 2 + w.extra + 2) * LT_QSUB + 5 * LT_HEADS * 4 +
-         (2 * LT_MAX_RING + 10) * 8 + 16 + LT_ROWS / 2 + 1024;
+  const int sub = w.rows * 128;
+  return w.ring * 2 * sub + (w.extra ? 2 * sub : 0) + (w.keys * 2 + w.extra + 2 * (w.rows / 64)) * LT_QSUB + 5 * LT_HEADS * 4 +
+         (2 * LT_MAX_RING + 10) * 8 + 16 + w.rows / 2 + 1024;
 }
 // how a tile lies in the ring; ring 0: these sizes do not fit
 static LtTile lt_tile(const RowAttn& p) {
   LtTile w{};
   const int vw = p.v_heads * p.V;
+  w.rows = 64;
   w.shared = p.v_col == 0;
   w.values = (vw + 127) / 128;
   if (w.shared) {
@@ -480,8 +485,18 @@ static LtTile lt_tile(const RowAttn& p) {
   }
   if (w.values > LT_MAX_BLOCKS) return w;
   w.tmem = w.values <= 6 ? 256 : 512;
-  w.ring = w.shared ? 10 : LT_MAX_RING;
-  while (w.ring > 0 && lt_smem(w) > 227 * 1024) --w.ring;
+  auto fit = [](LtTile& x, int most) {
+    x.ring = most;
+    while (x.ring > 0 && lt_smem(x) > 227 * 1024) --x.ring;
+  };
+  if (!w.shared) {
+    LtTile wide = w;
+    wide.rows = 128;
+    wide.ahead = 1;
+    fit(wide, LT_MAX_RING / 2);
+    if (wide.ring >= w.keys + w.values) return wide;
+  }
+  fit(w, w.shared ? 10 : LT_MAX_RING);
   if (w.ring < 4 || (w.shared && w.ring < 2 * w.pairs)) w.ring = 0;
   w.ahead = w.shared || w.keys + w.values <= w.ring ? 1 : 0;
   return w;
@@ -489,24 +504,28 @@ static LtTile lt_tile(const RowAttn& p) {
 
 bool latent_decode_tc_supported(const RowAttn& p) {
   return p.V % 8 == 0 && p.K % 8 == 0 && p.v_col % 8 == 0 && p.row_width % 8 == 0 && p.ld_out % 4 == 0 && p.H % p.v_heads == 0 &&
-         lt_box_rows(p.block_size) >= 8 && lt_tile(p).ring > 0;
+         lt_box_rows(p.block_size, 64) >= 8 && lt_tile(p).ring > 0;
 }
 
 int latent_decode_tc_splits(const RowAttn& p, int max_ctx, int num_sms) {
   const int ctas = p.T * ((p.H + LT_HEADS - 1) / LT_HEADS);
   if (ctas * 3 > num_sms * 2) return 1;                            // nearly a full wave already
-  return std::max(1, std::min({num_sms / std::max(1, ctas), max_ctx / (2 * LT_ROWS), 32}));
+  return std::max(1, std::min({num_sms / std::max(1, ctas), max_ctx / 128, 32}));
 }
 
 void launch_latent_decode_tc(const RowAttn& p, cudaStream_t s) {
   if (p.T == 0) return;
   const LtTile w = lt_tile(p);
-  const int box = lt_box_rows(p.block_size), smem = lt_smem(w);
+  const int box = lt_box_rows(p.block_size, w.rows), smem = lt_smem(w);
   if (w.ring == 0) throw std::runtime_error("attention over shared rows (tcgen05): unsupported sizes");
   const CUtensorMap tm = make_tmap_bf16_2d(p.pool, (uint64_t)p.num_blocks * p.block_size, p.row_width, p.row_width, box, 64);
-  cudaFuncSetAttribute(latent_decode_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
-  launch_pdl(PDL_DECODE_ATTN, latent_decode_tc_kernel, dim3(p.T, (p.H + LT_HEADS - 1) / LT_HEADS, p.splits), dim3(LT_THREADS), smem, s,
-             tm, p, w, box, p.scale * LT_LOG2E);
+  auto go = [&](auto kern) {
+    cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    launch_pdl(PDL_DECODE_ATTN, kern, dim3(p.T, (p.H + LT_HEADS - 1) / LT_HEADS, p.splits), dim3(LT_THREADS), smem, s, tm, p, w, box,
+               p.scale * LT_LOG2E);
+  };
+  if (w.rows == 128) go(latent_decode_tc_kernel<128>);
+  else go(latent_decode_tc_kernel<64>);
   const cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess) throw std::runtime_error(std::string("attention over shared rows (tcgen05): ") + cudaGetErrorString(e));
 }
