@@ -214,6 +214,89 @@ latent_inputs_kernel(const LatentStore p) {
     }
   }
 }
+// The same for many rows of a finished projection (bf16): one warp per token, everything in flight at once.  NQ: 16-byte pieces of
+// the query latent per lane
+constexpr int LW_WARPS = 8, LW_KV = 4;
+template <int NQ>
+__global__ void __launch_bounds__(LW_WARPS * 32)
+latent_inputs_rows_kernel(const LatentStore p) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int lane = threadIdx.x & 31;
+  const long long t = (long long)blockIdx.x * LW_WARPS + (threadIdx.x >> 5);
+  if (t >= p.T) return;
+  const bf16* row = reinterpret_cast<const bf16*>(p.proj.p) + t * p.proj.ld;
+  uint4 q[NQ], kv[LW_KV];
+#pragma unroll
+  for (int i = 0; i < NQ; ++i) {
+    const int c = (lane + i * 32) * 8;
+    q[i] = c < p.q_rank ? __ldcg(reinterpret_cast<const uint4*>(row + p.off_dq + c)) : make_uint4(0, 0, 0, 0);
+  }
+#pragma unroll
+  for (int i = 0; i < LW_KV; ++i) {
+    const int c = (lane + i * 32) * 8;
+    kv[i] = c < p.rank ? __ldcg(reinterpret_cast<const uint4*>(row + p.off_kv + c)) : make_uint4(0, 0, 0, 0);
+  }
+  const int slot = p.slots[t], half = p.rot_dims / 2, rot = p.off_kv + p.rank;
+  const double pos = double(p.positions[t]);
+  if (p.head_gate != nullptr)
+    for (int h = lane; h < p.H; h += 32) p.head_gate[t * p.H + h] = sigmoid_f(Elem<bf16>::get(row[p.off_g + h]));
+  auto squares = [](const uint4& u) {
+    const uint32_t w[4] = {u.x, u.y, u.z, u.w};
+    float s = 0.f;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const float a = __uint_as_float(w[e] << 16), b = __uint_as_float(w[e] & 0xffff0000u);
+      s += a * a + b * b;
+    }
+    return s;
+  };
+  auto put = [](bf16* dst, const uint4& u, const float* g, float inv) {
+    const float4 a = *reinterpret_cast<const float4*>(g), b = *reinterpret_cast<const float4*>(g + 4);
+    const uint32_t w[4] = {u.x, u.y, u.z, u.w};
+    const float f[8] = {a.x, a.y, a.z, a.w, b.x, b.y, b.z, b.w};
+    uint32_t o[4];
+#pragma unroll
+    for (int e = 0; e < 4; ++e)
+      o[e] = pack_bf16(__uint_as_float(w[e] << 16) * inv * f[2 * e], __uint_as_float(w[e] & 0xffff0000u) * inv * f[2 * e + 1]);
+    *reinterpret_cast<uint4*>(dst) = make_uint4(o[0], o[1], o[2], o[3]);
+  };
+  float sq = 0.f, sk = 0.f;
+#pragma unroll
+  for (int i = 0; i < NQ; ++i) sq += squares(q[i]);
+#pragma unroll
+  for (int i = 0; i < LW_KV; ++i) sk += squares(kv[i]);
+  const float iq = rsqrtf(warp_sum(sq) / float(p.q_rank) + p.eps), ik = rsqrtf(warp_sum(sk) / float(p.rank) + p.eps);
+  bf16* cq = reinterpret_cast<bf16*>(p.cq) + t * p.ld_cq;    // ld_cq == q_rank: a multiple of 8
+#pragma unroll
+  for (int i = 0; i < NQ; ++i) {
+    const int c = (lane + i * 32) * 8;
+    if (c < p.q_rank) put(cq + c, q[i], p.q_norm_w + c, iq);
+  }
+  if (slot < 0) return;
+  if (slot >= p.num_rows) {
+    if (lane == 0) report(p.status, ST_BAD_INDEX);
+    return;
+  }
+  bf16* dst = reinterpret_cast<bf16*>(p.pool) + (long long)slot * p.row_width;
+#pragma unroll
+  for (int i = 0; i < LW_KV; ++i) {
+    const int c = (lane + i * 32) * 8;
+    if (c < p.rank) put(dst + c, kv[i], p.norm_w + c, ik);
+  }
+  for (int i = lane; i < half; i += 32) {
+    const int cu = p.half ? i : 2 * i, cv = p.half ? half + i : 2 * i + 1;
+    const float u = Elem<bf16>::get(row[rot + cu]), v = Elem<bf16>::get(row[rot + cv]);
+    float c, s;
+    turn_angle(pos, p.freq[i], c, s);
+    dst[p.rank + cu] = Elem<bf16>::put(u * c - v * s);
+    dst[p.rank + cv] = Elem<bf16>::put(v * c + u * s);
+  }
+}
+static bool latent_inputs_rows(const LatentStore& p) {
+  return p.T >= 256 && p.proj.part == nullptr && p.off_kv >= 0 && p.q_rank % 8 == 0 && p.q_rank <= 12 * 256 && p.rank % 8 == 0 &&
+         p.rank <= LW_KV * 256 && p.off_dq % 8 == 0 && p.off_kv % 8 == 0 && p.proj.ld % 8 == 0 && p.row_width % 8 == 0 && p.rot_dims == p.R;
+}
 static bool latent_inputs_vec(const LatentStore& p) {
   return p.off_kv >= 0 && p.q_rank % 4 == 0 && p.q_rank <= LS_THREADS * 4 * LI_Q && p.rank % 4 == 0 && p.rank <= LS_THREADS * 4 * LI_KV &&
          p.off_dq % 4 == 0 && p.off_kv % 4 == 0 && p.rot_dims == p.R && p.R <= 2 * LS_THREADS;
@@ -287,6 +370,15 @@ bool latent_rotate_supported(const LatentStore& p) {
 void launch_latent_inputs(const LatentStore& p, bool f32, cudaStream_t s) {
   if (p.T == 0) return;
   const size_t smem = size_t(std::max(2, p.rot_dims)) * 4;
+  if (!f32 && latent_inputs_rows(p)) {
+    auto go = [&](auto kern) { launch_pdl(PDL_ROPE, kern, dim3((p.T + LW_WARPS - 1) / LW_WARPS), dim3(LW_WARPS * 32), 0, s, p); };
+    if (p.q_rank <= 4 * 256) go(latent_inputs_rows_kernel<4>);
+    else if (p.q_rank <= 8 * 256) go(latent_inputs_rows_kernel<8>);
+    else go(latent_inputs_rows_kernel<12>);
+    const cudaError_t e = cudaGetLastError();
+    if (e != cudaSuccess) throw std::runtime_error(std::string("latent inputs: ") + cudaGetErrorString(e));
+    return;
+  }
   auto go = [&](auto kern) { launch_pdl(PDL_ROPE, kern, dim3(p.T), dim3(LS_THREADS), smem, s, p); };
   const bool vec = latent_inputs_vec(p);
   if (f32) vec ? go(latent_inputs_kernel<float, true>) : go(latent_inputs_kernel<float, false>);

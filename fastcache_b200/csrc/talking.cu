@@ -137,10 +137,11 @@ talk_store_kernel(const TalkStore p, int tokens) {
 // Many rows of a finished projection (bf16), heads of 32, 64 or 128 columns.  D / 4 lanes hold a head, rotate and norm it in
 // registers and leave it in shared memory as the sum of two bf16 terms.  The mix runs on mma.sync with talk as the 16-row operand,
 // also as two terms: hi hi + hi lo + lo hi.  Inside a block of 32 columns, column 8 q + 2 j + e lies at 8 j + 2 q + e, so that a
-// lane's four pairs of accumulators are eight neighbouring columns.
+// lane's four pairs of accumulators are eight neighbouring columns.  The next token's heads are requested before this one's mix.
+// NR: query heads per D / 4 lanes, at most
 constexpr int TR_THREADS = 256, TR_WARPS = TR_THREADS / 32;
-template <int D>
-__global__ void __launch_bounds__(TR_THREADS, 3)
+template <int D, int NR>
+__global__ void __launch_bounds__(TR_THREADS, NR <= 4 ? 3 : 2)
 talk_store_rows_kernel(const TalkStore p, int tokens) {
   constexpr int L = D / 4, PER_WARP = 32 / L, PITCH = D + 8;  // lanes per head; pitch: rows 16 bytes apart modulo 128
   extern __shared__ __align__(16) uint8_t raw[];
@@ -179,23 +180,42 @@ talk_store_rows_kernel(const TalkStore p, int tokens) {
   const int mat = lane >> 3;
   const uint32_t talk_u = smem_u32(s_talk), q_u = smem_u32(s_q);
   const uint32_t talk_lo = uint32_t(G * hp * tp) * 2, q_lo = uint32_t((H + 16) * PITCH) * 2;
+  // one head per round: query heads, then (round NR) key heads
+  auto head_of = [&](int r) {
+    const int i = (r < NR ? r * TR_WARPS + warp : warp) * PER_WARP + sub;
+    return r < NR ? (i < H ? i : -1) : keys && i < G ? H + i : -1;
+  };
+  uint2 in[NR + 1];
+  uint4 val = make_uint4(0, 0, 0, 0);
+  int next_slot = -1;
+  auto request = [&](int t) {
+    const bf16* row = src + (long long)t * p.proj.ld;
+#pragma unroll
+    for (int r = 0; r <= NR; ++r) {
+      const int h = head_of(r);
+      in[r] = h < 0 ? make_uint2(0, 0)
+                    : __ldcg(reinterpret_cast<const uint2*>(row + (h < H ? p.off_q + h * D : p.off_k + (h - H) * D) + c0));
+    }
+    if (keys) {
+      if (tid * 8 < G * V) val = __ldcg(reinterpret_cast<const uint4*>(row + p.off_v + tid * 8));
+      next_slot = p.slots[t];
+    }
+  };
+  if (t0 < t1) request(t0);
   for (int t = t0; t < t1; ++t) {
     __syncthreads();                                         // angles are there, the mix of the token before is done
-    const bf16* row = src + (long long)t * p.proj.ld;
     const float2* cs = s_cs + (t & 1) * half;
-    int slot = keys ? p.slots[t] : -1;
+    int slot = next_slot;
     if (slot >= p.num_rows) {
       if (tid == 0) report(p.status, ST_BAD_INDEX);
       slot = -1;
     }
     bf16* dst = reinterpret_cast<bf16*>(p.pool) + (slot >= 0 ? (long long)slot * p.row_width : 0);
-    const int heads = H + (slot >= 0 ? G : 0);
-#pragma unroll 2
-    for (int h0 = warp * PER_WARP; h0 < heads; h0 += TR_WARPS * PER_WARP) {
-      const int h = h0 + sub;
-      const bool on = h < heads;
-      uint2 raw2 = make_uint2(0, 0);
-      if (on) raw2 = __ldcg(reinterpret_cast<const uint2*>(row + (h < H ? p.off_q + h * D : p.off_k + (h - H) * D) + c0));
+#pragma unroll
+    for (int r = 0; r <= NR; ++r) {
+      const int h = head_of(r);
+      const bool on = h >= 0 && (h < H || slot >= 0);
+      const uint2 raw2 = in[r];
       float x[4] = {__uint_as_float(raw2.x << 16), __uint_as_float(raw2.x & 0xffff0000u), __uint_as_float(raw2.y << 16),
                     __uint_as_float(raw2.y & 0xffff0000u)};
       if (half > 0) {
@@ -232,9 +252,8 @@ talk_store_rows_kernel(const TalkStore p, int tokens) {
         *reinterpret_cast<uint2*>(dst + (h - H) * D + c0) = make_uint2(a, b);
       }
     }
-    if (slot >= 0)
-      for (int i = tid * 8; i < G * V; i += TR_THREADS * 8)
-        *reinterpret_cast<uint4*>(dst + p.v_col + i) = __ldcg(reinterpret_cast<const uint4*>(row + p.off_v + i));
+    if (slot >= 0 && tid * 8 < G * V) *reinterpret_cast<uint4*>(dst + p.v_col + tid * 8) = val;
+    if (t + 1 < t1) request(t + 1);
     __syncthreads();
     angles(t + 1);
     bf16* q = reinterpret_cast<bf16*>(p.q) + (long long)t * H * nk;
@@ -282,7 +301,8 @@ static bool talk_rows_supported(const TalkStore& p) {
   const int half = p.rot_dims / 2;
   return p.T > 296 && p.proj.part == nullptr && (p.D == 32 || p.D == 64 || p.D == 128) && half % 4 == 0 && half <= TR_THREADS &&
          (p.G * p.V) % 8 == 0 && p.proj.ld % 8 == 0 && p.off_q % 8 == 0 && (p.off_k < 0 || (p.off_k % 8 == 0 && p.off_v % 8 == 0)) &&
-         p.v_col % 8 == 0 && p.row_width % 8 == 0 && p.pad_out == 0 && talk_rows_smem(p) <= 100 * 1024;
+         p.v_col % 8 == 0 && p.row_width % 8 == 0 && p.pad_out == 0 && talk_rows_smem(p) <= 100 * 1024 &&
+         p.H <= 8 * TR_WARPS * (128 / p.D) && p.G <= TR_WARPS * (128 / p.D) && p.G * p.V <= TR_THREADS * 8;
 }
 static void launch_talk_rows(const TalkStore& p, cudaStream_t s) {
   const size_t smem = talk_rows_smem(p);
@@ -291,9 +311,10 @@ static void launch_talk_rows(const TalkStore& p, cudaStream_t s) {
     if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem));
     launch_pdl(PDL_ROPE, kern, dim3((p.T + tokens - 1) / tokens), dim3(TR_THREADS), smem, s, p, tokens);
   };
-  if (p.D == 32) go(talk_store_rows_kernel<32>);
-  else if (p.D == 64) go(talk_store_rows_kernel<64>);
-  else go(talk_store_rows_kernel<128>);
+  const bool few = p.H <= 4 * TR_WARPS * (128 / p.D);
+  if (p.D == 32) few ? go(talk_store_rows_kernel<32, 4>) : go(talk_store_rows_kernel<32, 8>);
+  else if (p.D == 64) few ? go(talk_store_rows_kernel<64, 4>) : go(talk_store_rows_kernel<64, 8>);
+  else few ? go(talk_store_rows_kernel<128, 4>) : go(talk_store_rows_kernel<128, 8>);
 }
 
 template <typename T>
