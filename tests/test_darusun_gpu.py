@@ -189,7 +189,7 @@ def _softmax(s, sink):
 
 
 @pytest.mark.parametrize("impl", [0, 1])
-@pytest.mark.parametrize("H,G,D,V,page,window,sink", [(32, 2, 128, 128, 64, 0, False), (8, 2, 64, 32, 16, 0, False), (33, 3, 40, 24, 8, 100, True),
+@pytest.mark.parametrize("H,G,D,V,page,window,sink", [(32, 2, 128, 128, 64, 0, False), (8, 2, 64, 40, 16, 0, False), (33, 3, 40, 24, 8, 100, True),
                                                       (32, 8, 128, 128, 64, 0, True), (6, 6, 64, 72, 32, 65, False), (16, 4, 128, 128, 64, 700, False),
                                                       (12, 1, 128, 96, 256, 1, True), (48, 4, 96, 128, 64, 64, True)])
 def test_attention_over_rows_with_several_value_heads(H, G, D, V, page, window, sink, impl):
