@@ -110,7 +110,7 @@ def _mixer(kind: str, m: dict, width: int, eps: float, mixers: List[nn.Module]) 
                                 m["rot"]["dims"], eps, owner)
     if kind == "latent_attention":
         return LatentAttention(width, m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"], m["scale"], m["rot"]["base"],
-                               m["rot"]["dims"], eps, q_rank=m["q_rank"], window=int(m["mask"]["size"]), half=False,
+                               m["rot"]["dims"], eps, q_rank=m["q_rank"], window=int((m.get("mask") or {}).get("size") or 0), half=False,
                                head_gate=True, sink=True)
     raise ValueError(f"unknown mixer type {kind!r}")
 
